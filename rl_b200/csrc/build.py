@@ -30,6 +30,8 @@ NVCC_FLAGS = [
     "-Xcompiler", "-fPIC,-fvisibility=hidden",
     "--use_fast_math",
 ]
+# sources whose tanh / sine / cosine / exponential / division must be the accurate ones
+PRECISE = {"mixers.cu", "retention.cu"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread"]
 
 
@@ -57,7 +59,7 @@ def _compile_one(src: Path, verbose: bool, ptxas_v: bool) -> tuple[Path, str]:
     obj = BUILD / (src.name + ".o")
     stamp = BUILD / (src.name + ".sha")
     if src.suffix == ".cu":
-        flags = list(NVCC_FLAGS) + (["-Xptxas", "-v"] if ptxas_v else [])
+        flags = [f for f in NVCC_FLAGS if src.name not in PRECISE or f != "--use_fast_math"] + (["-Xptxas", "-v"] if ptxas_v else [])
         cmd = [_nvcc(), *flags, "-I", str(CSRC), "-c", str(src), "-o", str(obj)]
     else:
         flags = list(CXX_FLAGS)

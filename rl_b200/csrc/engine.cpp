@@ -20,7 +20,7 @@
 
 namespace {
 
-enum SeqState : int { WAITING = 0, RUNNING = 1, FINISHED = 2 };
+enum SeqState : int { WAITING = 0, RUNNING = 1, FINISHED = 2, STEPPED = 3 };
 
 struct Seq {
   long long id = 0;
@@ -423,6 +423,39 @@ RLB_API int rlb_engine_commit_first(void* h, const long long* ids, int n, int* f
     }
   }
   return retired;
+}
+
+// Stepped sequences: the caller (GenerationEngine.step) decides which tokens run when; this class only keeps their pages. They never
+// wait, decode or get preempted through schedule(), and share the block pool with the scheduled ones.
+RLB_API int rlb_engine_open(void* h, long long id) {
+  Engine* e = static_cast<Engine*>(h);
+  if (e->seqs.count(id)) return -1;
+  Seq s;
+  s.id = id;
+  s.state = STEPPED;
+  s.arrival = e->clock++;
+  e->seqs.emplace(id, std::move(s));
+  return 0;
+}
+// Makes room for `count` more tokens. Returns the position of the first of them, -1 for an unknown id, -2 when blocks run out (then
+// nothing changes).
+RLB_API int rlb_engine_extend(void* h, long long id, int count) {
+  Engine* e = static_cast<Engine*>(h);
+  auto it = e->seqs.find(id);
+  if (it == e->seqs.end() || it->second.state != STEPPED || count < 0) return -1;
+  Seq& s = it->second;
+  if (!e->ensure_capacity(s, s.num_tokens + count)) return -2;
+  const int first = s.num_tokens;
+  s.num_tokens += count;
+  return first;
+}
+RLB_API int rlb_engine_close(void* h, long long id) {
+  Engine* e = static_cast<Engine*>(h);
+  auto it = e->seqs.find(id);
+  if (it == e->seqs.end() || it->second.state != STEPPED) return -1;
+  e->release_seq(it->second);
+  e->seqs.erase(it);
+  return 0;
 }
 
 RLB_API int rlb_engine_seq_info(void* h, long long id, int* num_tokens, int* num_generated, int* state) {

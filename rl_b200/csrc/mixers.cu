@@ -1,0 +1,460 @@
+// Kernels of parallel mixer layers (models/mixers.py) that run for every size and for bf16 and fp32 models alike: the residual
+// stream's start, a plain product with the layer epilogues, the latent-attention and retention mixers one row at a time.
+//
+// The batch of an engine step mixes single decoded tokens and portions of prompts; every row knows its position, its cache slot and
+// its sequence's pages or state row, so nothing here depends on how a prompt was cut or on what else is in the batch. The mixers
+// read their projections from the rows of the fused input product and write their gated output over the gate columns of the same
+// rows, which the output product then reads in place.
+//
+// This file is compiled without fast math: tanh, sine, cosine, exponentials, square roots and divisions are the accurate ones.
+// The tensor-core forms for bf16 are in latent_attention.cu, latent_decode.cu and retention.cu.
+#include "common.cuh"
+
+#include <math.h>
+
+namespace {
+using namespace rlb;
+
+template <typename T>
+__device__ __forceinline__ float ld(const T* p) {
+  return static_cast<float>(*p);
+}
+template <>
+__device__ __forceinline__ float ld<__nv_bfloat16>(const __nv_bfloat16* p) {
+  return __bfloat162float(*p);
+}
+template <typename T>
+__device__ __forceinline__ void st(T* p, float v) {
+  *p = static_cast<T>(v);
+}
+template <>
+__device__ __forceinline__ void st<__nv_bfloat16>(__nv_bfloat16* p, float v) {
+  *p = __float2bfloat16(v);
+}
+
+// ---------------------------------------------------------------- start of the residual stream
+// x = table[id] * scale (kept in e), + step; h = w * tanh(alpha x) + b
+template <typename T>
+__global__ void embed_rows_kernel(const void* ids, int ids64, const T* __restrict__ table, float* __restrict__ x, float* __restrict__ e,
+                                  T* __restrict__ h, const T* __restrict__ step, const T* __restrict__ alpha, const T* __restrict__ nw,
+                                  const T* __restrict__ nb, int d, int vocab, float scale, int* status) {
+  const long long row = blockIdx.x;
+  long long id = ids64 ? static_cast<const long long*>(ids)[row] : static_cast<const int*>(ids)[row];
+  if (id < 0 || id >= vocab) {
+    if (threadIdx.x == 0 && status) atomicCAS(status, 0, RLB_ERR_BOUNDS);
+    id = 0;
+  }
+  const float a = ld(alpha);
+  for (int c = threadIdx.x; c < d; c += blockDim.x) {
+    float v = ld(table + id * d + c) * scale;
+    if (e) e[row * d + c] = v;
+    if (step) v += ld(step + c);
+    x[row * d + c] = v;
+    st(h + row * d + c, tanhf(a * v) * ld(nw + c) + ld(nb + c));
+  }
+}
+
+// ---------------------------------------------------------------- product with the layer epilogues
+struct RowsGemm {
+  const void* a;
+  const void* w;
+  void* out;
+  int M, N, K;
+  long long lda, ldw, ldo;
+  int act_from;        // squared ReLU on columns >= act_from
+  float* x;            // residual stream (null: plain store): x += acc (+ e) (+ step), out = dynamic tanh of x
+  long long ldx;
+  const float* e;
+  const void* step;
+  const void* alpha;
+  const void* nw;
+  const void* nb;
+};
+
+constexpr int RG_T = 64, RG_K = 16;
+
+template <typename TI, typename TO>
+__global__ void __launch_bounds__(256) gemm_rows_kernel(RowsGemm g) {
+  __shared__ float as[RG_K][RG_T + 4], ws[RG_K][RG_T + 4];
+  const TI* A = static_cast<const TI*>(g.a);
+  const TI* W = static_cast<const TI*>(g.w);
+  const int m0 = blockIdx.y * RG_T, n0 = blockIdx.x * RG_T;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < g.K; k0 += RG_K) {
+    for (int i = threadIdx.x; i < RG_T * RG_K; i += 256) {
+      const int r = i / RG_K, k = i % RG_K;
+      as[k][r] = (m0 + r < g.M && k0 + k < g.K) ? ld(A + static_cast<long long>(m0 + r) * g.lda + k0 + k) : 0.f;
+      ws[k][r] = (n0 + r < g.N && k0 + k < g.K) ? ld(W + static_cast<long long>(n0 + r) * g.ldw + k0 + k) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < RG_K; ++k) {
+      float av[4], wv[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        av[i] = as[k][ty * 4 + i];
+        wv[i] = ws[k][tx * 4 + i];
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], wv[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+  const float alpha = g.x ? ld(static_cast<const TI*>(g.alpha)) : 0.f;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int m = m0 + ty * 4 + i;
+    if (m >= g.M) continue;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + tx * 4 + j;
+      if (n >= g.N) continue;
+      float v = acc[i][j];
+      TO* o = static_cast<TO*>(g.out) + static_cast<long long>(m) * g.ldo + n;
+      if (g.x) {
+        float* xp = g.x + static_cast<long long>(m) * g.ldx + n;
+        v += *xp;
+        if (g.e) v += g.e[static_cast<long long>(m) * g.ldx + n];
+        if (g.step) v += ld(static_cast<const TI*>(g.step) + n);
+        *xp = v;
+        v = tanhf(alpha * v) * ld(static_cast<const TI*>(g.nw) + n) + ld(static_cast<const TI*>(g.nb) + n);
+      } else if (n >= g.act_from) {
+        v = fmaxf(v, 0.f);
+        v *= v;
+      }
+      st(o, v);
+    }
+  }
+}
+
+// ---------------------------------------------------------------- latent attention
+struct LatentShape {
+  long long ldp;                       // row stride of the projected rows
+  int q_off, lat_off, mix_off;         // columns of queries, latent and gate
+  int heads, dim, rot_dim, vdim, rank; // per head: dim unrotated + rot_dim rotated query / key dimensions
+  int width;                           // row width of the latent cache
+  int block_size, num_blocks;
+};
+
+// Per row: latent / rms * w and rotated shared key into the cache row of the token; rotated query parts in place.
+template <typename T>
+__global__ void latent_prep_kernel(T* __restrict__ p, LatentShape s, const int* __restrict__ positions, const long long* __restrict__ slots,
+                                   const T* __restrict__ norm_w, const float* __restrict__ freq, int half, float gain, float eps,
+                                   T* __restrict__ cache, int* status) {
+  extern __shared__ float sm[];
+  __shared__ float red[32];
+  float* cs = sm;              // [half] cosine, then [half] sine
+  const long long row = blockIdx.x;
+  T* pr = p + row * s.ldp;
+  const float pos = static_cast<float>(positions[row]);
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float sn, c;
+    sincosf(pos * freq[i], &sn, &c);
+    cs[i] = c * gain;
+    cs[half + i] = sn * gain;
+  }
+  float ss = 0.f;
+  for (int r = threadIdx.x; r < s.rank; r += blockDim.x) {
+    const float v = ld(pr + s.lat_off + r);
+    ss += v * v;
+  }
+  ss = block_sum(ss, red);
+  const float rstd = 1.f / sqrtf(ss / static_cast<float>(s.rank) + eps);
+  __syncthreads();
+  const long long slot = slots[row];
+  if (slot >= static_cast<long long>(s.num_blocks) * s.block_size) {
+    if (threadIdx.x == 0 && status) atomicCAS(status, 0, RLB_ERR_BOUNDS);
+  } else if (slot >= 0) {
+    T* cr = cache + slot * s.width;
+    for (int r = threadIdx.x; r < s.width; r += blockDim.x) {
+      float v = 0.f;
+      if (r < s.rank) {
+        v = ld(pr + s.lat_off + r) * rstd * ld(norm_w + r);
+      } else if (r < s.rank + s.rot_dim) {
+        const int j = r - s.rank;
+        v = ld(pr + s.lat_off + r);
+        if (j < 2 * half) {
+          const float o = ld(pr + s.lat_off + s.rank + (j ^ 1));
+          v = (j & 1) ? v * cs[j >> 1] + o * cs[half + (j >> 1)] : v * cs[j >> 1] - o * cs[half + (j >> 1)];
+        }
+      }
+      st(cr + r, v);
+    }
+  }
+  const int qd = s.dim + s.rot_dim;
+  for (int i = threadIdx.x; i < s.heads * half; i += blockDim.x) {
+    T* q = pr + s.q_off + (i / half) * qd + s.dim + 2 * (i % half);
+    const float c = cs[i % half], sn = cs[half + i % half], u = ld(q), v = ld(q + 1);
+    st(q, u * c - v * sn);
+    st(q + 1, v * c + u * sn);
+  }
+}
+
+// One CTA per (row, head): the query is carried into the latent space (q^T W_uk), the keys are the cached rows, the weighted
+// latent is carried to the values (W_uv) and gated. Everything in fp32.
+constexpr int LR_TILE = 128;
+template <typename T>
+__global__ void __launch_bounds__(128)
+latent_rows_kernel(T* __restrict__ p, LatentShape s, const T* __restrict__ cache, const int* __restrict__ block_table, int bt_stride,
+                   const int* __restrict__ seq_lens, const T* __restrict__ kv_up, float scale, int* status) {
+  extern __shared__ float sm[];
+  __shared__ float red[32];
+  float* qa = sm;                       // [width]
+  float* o = qa + s.width;              // [rank]
+  float* sc = o + s.rank;               // [LR_TILE]
+  long long* rows = reinterpret_cast<long long*>(sm + ((s.width + s.rank + LR_TILE + 1) & ~1));   // [LR_TILE]
+  const int row = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  T* pr = p + row * s.ldp;
+  const T* q = pr + s.q_off + h * (s.dim + s.rot_dim);
+  for (int r = tid; r < s.width; r += 128) {
+    float v = 0.f;
+    if (r < s.rank) {
+      for (int d = 0; d < s.dim; ++d) v = fmaf(ld(q + d), ld(kv_up + static_cast<long long>(h * s.dim + d) * s.rank + r), v);
+    } else if (r < s.rank + s.rot_dim) {
+      v = ld(q + s.dim + r - s.rank);
+    }
+    qa[r] = v * scale;
+  }
+  for (int r = tid; r < s.rank; r += 128) o[r] = 0.f;
+  const int len = min(seq_lens[row], bt_stride * s.block_size);
+  float m = -INFINITY, l = 0.f;
+  for (int t0 = 0; t0 < len; t0 += LR_TILE) {
+    const int n = min(LR_TILE, len - t0);
+    __syncthreads();
+    if (tid < n) {
+      const int t = t0 + tid;
+      int blk = block_table[static_cast<long long>(row) * bt_stride + t / s.block_size];
+      if (blk < 0 || blk >= s.num_blocks) {
+        if (status) atomicCAS(status, 0, RLB_ERR_BOUNDS);
+        blk = 0;
+      }
+      rows[tid] = (static_cast<long long>(blk) * s.block_size + t % s.block_size) * s.width;
+    }
+    __syncthreads();
+    for (int j = warp; j < n; j += 4) {
+      const T* cr = cache + rows[j];
+      float v = 0.f;
+      for (int r = lane; r < s.width; r += 32) v = fmaf(qa[r], ld(cr + r), v);
+      v = warp_sum(v);
+      if (lane == 0) sc[j] = v;
+    }
+    __syncthreads();
+    const float mine = tid < n ? sc[tid] : -INFINITY;
+    const float mn = fmaxf(m, block_max(mine, red));
+    const float pj = tid < n ? expf(mine - mn) : 0.f;
+    const float c = m == -INFINITY ? 0.f : expf(m - mn);
+    l = l * c + block_sum(pj, red);
+    m = mn;
+    if (tid < n) sc[tid] = pj;
+    __syncthreads();
+    for (int r = tid; r < s.rank; r += 128) {
+      float v = o[r] * c;
+      for (int j = 0; j < n; ++j) v = fmaf(sc[j], ld(cache + rows[j] + r), v);
+      o[r] = v;
+    }
+  }
+  __syncthreads();
+  const float inv = l > 0.f ? 1.f / l : 0.f;
+  for (int v = warp; v < s.vdim; v += 4) {
+    const T* w = kv_up + static_cast<long long>(s.heads * s.dim + h * s.vdim + v) * s.rank;
+    float y = 0.f;
+    for (int r = lane; r < s.rank; r += 32) y = fmaf(o[r], ld(w + r), y);
+    y = warp_sum(y) * inv;
+    if (lane == 0) {
+      T* g = pr + s.mix_off + h * s.vdim + v;
+      st(g, y / (1.f + expf(-ld(g))));
+    }
+  }
+}
+
+// ---------------------------------------------------------------- retention
+struct RetentionShape {
+  long long ldp;
+  int q_off, k_off, v_off, mix_off;
+  int heads, dim, vdim;
+};
+
+// One CTA per (sequence piece, head), token after token: S = decay S + k v^T, o = S^T q, unit RMS over the head, SiLU gate. A piece
+// whose first token stands at position 0 starts from a zero state, whatever its state row held before.
+template <typename T>
+__global__ void __launch_bounds__(256)
+retention_rows_kernel(T* __restrict__ p, RetentionShape s, int row0, const int* __restrict__ cu, const int* __restrict__ positions,
+                      const long long* __restrict__ state_rows, float* __restrict__ state, long long num_states,
+                      const float* __restrict__ decay, const float* __restrict__ freq, int half, float gain, float kscale, float eps, int* status) {
+  extern __shared__ float sm[];
+  __shared__ float red[32];
+  float* q = sm;                 // [dim]
+  float* k = q + s.dim;          // [dim]
+  float* o = k + s.dim;          // [vdim]
+  float* part = o + s.vdim;      // [256] partial sums over slices of dim (vdim < 256)
+  const int seq = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+  const int begin = cu ? cu[seq] : seq, end = cu ? cu[seq + 1] : seq + 1;
+  const long long sr = state_rows[seq];
+  if (sr < 0 || sr >= num_states) {
+    if (tid == 0 && status) atomicCAS(status, 0, RLB_ERR_BOUNDS);
+    return;
+  }
+  float* S = state + (sr * s.heads + h) * static_cast<long long>(s.dim) * s.vdim;
+  const float dec = decay[h];
+  const int slices = s.vdim >= 256 ? 1 : 256 / s.vdim;
+  const int slice = s.vdim >= 256 ? 0 : tid / s.vdim;
+  for (int t = begin; t < end; ++t) {
+    T* pr = p + (row0 + t) * s.ldp;
+    const float pos = static_cast<float>(positions[row0 + t]);
+    const bool fresh = positions[row0 + t] == 0;
+    for (int i = tid; i < s.dim; i += 256) {
+      float qv = ld(pr + s.q_off + h * s.dim + i), kv = ld(pr + s.k_off + h * s.dim + i);
+      if (i < 2 * half) {
+        const int f = i < half ? i : i - half, oi = i < half ? i + half : i - half;
+        float sn, c;
+        sincosf(pos * freq[f], &sn, &c);
+        c *= gain;
+        sn *= i < half ? -gain : gain;
+        qv = qv * c + ld(pr + s.q_off + h * s.dim + oi) * sn;
+        kv = kv * c + ld(pr + s.k_off + h * s.dim + oi) * sn;
+      }
+      q[i] = qv;
+      k[i] = kv * kscale;
+    }
+    __syncthreads();
+    if (slice < slices) {
+      for (int v = s.vdim >= 256 ? tid : tid % s.vdim; v < s.vdim; v += 256) {
+        const float vv = ld(pr + s.v_off + h * s.vdim + v);
+        float acc = 0.f;
+        for (int i = slice; i < s.dim; i += slices) {
+          float* sp = S + static_cast<long long>(i) * s.vdim + v;
+          const float nv = fresh ? k[i] * vv : fmaf(dec, *sp, k[i] * vv);
+          *sp = nv;
+          acc = fmaf(nv, q[i], acc);
+        }
+        if (slices > 1) {
+          part[tid] = acc;
+          break;
+        }
+        o[v] = acc;
+      }
+    }
+    __syncthreads();
+    if (slices > 1 && tid < s.vdim) {
+      float acc = 0.f;
+      for (int j = 0; j < slices; ++j) acc += part[j * s.vdim + tid];
+      o[tid] = acc;
+    }
+    float ss = 0.f;
+    for (int v = tid; v < s.vdim; v += 256) ss += o[v] * o[v];   // each thread reads what it wrote
+    ss = block_sum(ss, red);
+    const float rstd = 1.f / sqrtf(ss / static_cast<float>(s.vdim) + eps);
+    for (int v = tid; v < s.vdim; v += 256) {
+      T* g = pr + s.mix_off + h * s.vdim + v;
+      const float gv = ld(g);
+      st(g, o[v] * rstd * (gv / (1.f + expf(-gv))));
+    }
+    __syncthreads();
+  }
+}
+
+int smem_attr(const void* kernel, size_t bytes) {
+  if (bytes <= 48 * 1024) return 0;
+  if (bytes > 220 * 1024) return -2;
+  return static_cast<int>(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes)));
+}
+}  // namespace
+
+RLB_API int rlb_embed_rows(const void* ids, int ids64, const void* table, int f32, float* x, float* e, void* h, const void* step,
+                           const void* alpha, const void* nw, const void* nb, long long rows, int d, int vocab, float scale, int* status,
+                           void* stream) {
+  if (rows <= 0) return 0;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (f32)
+    embed_rows_kernel<float><<<static_cast<unsigned>(rows), 256, 0, s>>>(ids, ids64, static_cast<const float*>(table), x, e, static_cast<float*>(h),
+        static_cast<const float*>(step), static_cast<const float*>(alpha), static_cast<const float*>(nw), static_cast<const float*>(nb), d, vocab, scale, status);
+  else
+    embed_rows_kernel<__nv_bfloat16><<<static_cast<unsigned>(rows), 256, 0, s>>>(ids, ids64, static_cast<const __nv_bfloat16*>(table), x, e,
+        static_cast<__nv_bfloat16*>(h), static_cast<const __nv_bfloat16*>(step), static_cast<const __nv_bfloat16*>(alpha),
+        static_cast<const __nv_bfloat16*>(nw), static_cast<const __nv_bfloat16*>(nb), d, vocab, scale, status);
+  return static_cast<int>(cudaGetLastError());
+}
+
+// out = A W^T for any sizes (A, W both bf16 or both fp32; out bf16 or fp32), squared ReLU on columns >= act_from. With `x`:
+// x += A W^T (+ e) (+ step) in place (fp32, row stride ldx, as is e) and out = nw * tanh(alpha x) + nb.
+RLB_API int rlb_gemm_rows(const void* a, const void* w, void* out, int M, int N, int K, long long lda, long long ldw, long long ldo, int in_f32,
+                          int out_f32, int act_from, float* x, long long ldx, const float* e, const void* step, const void* alpha,
+                          const void* nw, const void* nb, void* stream) {
+  if (M <= 0 || N <= 0 || K <= 0) return 0;
+  if (x && (!alpha || !nw || !nb)) return -2;
+  RowsGemm g{a, w, out, M, N, K, lda, ldw, ldo, act_from, x, ldx, e, step, alpha, nw, nb};
+  const dim3 grid((N + RG_T - 1) / RG_T, (M + RG_T - 1) / RG_T);
+  if (grid.y > 65535) return -2;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (in_f32 && out_f32) gemm_rows_kernel<float, float><<<grid, 256, 0, s>>>(g);
+  else if (in_f32) gemm_rows_kernel<float, __nv_bfloat16><<<grid, 256, 0, s>>>(g);
+  else if (out_f32) gemm_rows_kernel<__nv_bfloat16, float><<<grid, 256, 0, s>>>(g);
+  else gemm_rows_kernel<__nv_bfloat16, __nv_bfloat16><<<grid, 256, 0, s>>>(g);
+  return static_cast<int>(cudaGetLastError());
+}
+
+RLB_API int rlb_latent_prep(void* p, int f32, long long rows, long long ldp, int q_off, int lat_off, int heads, int dim, int rot_dim, int rank,
+                            int width, int block_size, int num_blocks, const int* positions, const long long* slots, const void* norm_w,
+                            const float* freq, int half, float gain, float eps, void* cache, int* status, void* stream) {
+  if (rows <= 0) return 0;
+  if (2 * half > rot_dim || rank + rot_dim > width) return -2;
+  LatentShape s{ldp, q_off, lat_off, 0, heads, dim, rot_dim, 0, rank, width, block_size, num_blocks};
+  const size_t sm = sizeof(float) * 2 * (half + 1);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (f32)
+    latent_prep_kernel<float><<<static_cast<unsigned>(rows), 256, sm, st>>>(static_cast<float*>(p), s, positions, slots, static_cast<const float*>(norm_w),
+                                                                            freq, half, gain, eps, static_cast<float*>(cache), status);
+  else
+    latent_prep_kernel<__nv_bfloat16><<<static_cast<unsigned>(rows), 256, sm, st>>>(static_cast<__nv_bfloat16*>(p), s, positions, slots,
+        static_cast<const __nv_bfloat16*>(norm_w), freq, half, gain, eps, static_cast<__nv_bfloat16*>(cache), status);
+  return static_cast<int>(cudaGetLastError());
+}
+
+RLB_API int rlb_latent_rows(void* p, int f32, int rows, long long ldp, int q_off, int mix_off, int heads, int dim, int rot_dim, int vdim, int rank,
+                            int width, int block_size, int num_blocks, const void* cache, const int* block_table, int bt_stride,
+                            const int* seq_lens, const void* kv_up, float scale, int* status, void* stream) {
+  if (rows <= 0) return 0;
+  if (rank + rot_dim > width || heads > 65535) return -2;
+  LatentShape s{ldp, q_off, 0, mix_off, heads, dim, rot_dim, vdim, rank, width, block_size, num_blocks};
+  const size_t sm = sizeof(float) * ((width + rank + LR_TILE + 1) & ~1) + sizeof(long long) * LR_TILE;
+  const dim3 grid(rows, heads);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  int rc;
+  if (f32) {
+    if ((rc = smem_attr(reinterpret_cast<const void*>(latent_rows_kernel<float>), sm))) return rc;
+    latent_rows_kernel<float><<<grid, 128, sm, st>>>(static_cast<float*>(p), s, static_cast<const float*>(cache), block_table, bt_stride, seq_lens,
+                                                     static_cast<const float*>(kv_up), scale, status);
+  } else {
+    if ((rc = smem_attr(reinterpret_cast<const void*>(latent_rows_kernel<__nv_bfloat16>), sm))) return rc;
+    latent_rows_kernel<__nv_bfloat16><<<grid, 128, sm, st>>>(static_cast<__nv_bfloat16*>(p), s, static_cast<const __nv_bfloat16*>(cache), block_table,
+                                                             bt_stride, seq_lens, static_cast<const __nv_bfloat16*>(kv_up), scale, status);
+  }
+  return static_cast<int>(cudaGetLastError());
+}
+
+// `cu` (offsets of the pieces, counted from row0) null: piece i is the single row row0 + i.
+RLB_API int rlb_retention_rows(void* p, int f32, int row0, int pieces, long long ldp, int q_off, int k_off, int v_off, int mix_off, int heads,
+                               int dim, int vdim, const int* cu, const int* positions, const long long* state_rows, float* state,
+                               long long num_states, const float* decay, const float* freq, int half, float gain, float kscale, float eps,
+                               int* status, void* stream) {
+  if (pieces <= 0) return 0;
+  if (2 * half > dim || heads > 65535) return -2;
+  RetentionShape s{ldp, q_off, k_off, v_off, mix_off, heads, dim, vdim};
+  const size_t sm = sizeof(float) * (2 * dim + vdim + 256);
+  const dim3 grid(pieces, heads);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  int rc;
+  if (f32) {
+    if ((rc = smem_attr(reinterpret_cast<const void*>(retention_rows_kernel<float>), sm))) return rc;
+    retention_rows_kernel<float><<<grid, 256, sm, st>>>(static_cast<float*>(p), s, row0, cu, positions, state_rows, state, num_states, decay, freq, half,
+                                                        gain, kscale, eps, status);
+  } else {
+    if ((rc = smem_attr(reinterpret_cast<const void*>(retention_rows_kernel<__nv_bfloat16>), sm))) return rc;
+    retention_rows_kernel<__nv_bfloat16><<<grid, 256, sm, st>>>(static_cast<__nv_bfloat16*>(p), s, row0, cu, positions, state_rows, state, num_states,
+                                                                decay, freq, half, gain, kscale, eps, status);
+  }
+  return static_cast<int>(cudaGetLastError());
+}

@@ -25,6 +25,7 @@ from rl_b200.models.transformer import CausalLM, PackedBatch
 from rl_b200.ops import engine_ops as E
 from rl_b200.ops import functional as F
 from rl_b200.ops import lib as _L
+from rl_b200.ops import mixer_ops as X
 from rl_b200.parallel.tensor import gather_cols, row_linear
 
 _P, _I, _LL = C.c_void_p, C.c_int, C.c_longlong
@@ -50,6 +51,9 @@ _ENGINE_SIGS = {
     "rlb_engine_cached_prefix": ([_P, _LL], _I),
     "rlb_engine_register_prefix": ([_P, _LL], _I),
     "rlb_engine_cache_stats": ([_P, _P, _P, _P, _P], None),
+    "rlb_engine_open": ([_P, _LL], _I),
+    "rlb_engine_extend": ([_P, _LL, _I], _I),
+    "rlb_engine_close": ([_P, _LL], _I),
 }
 _bound = False
 
@@ -208,6 +212,32 @@ class _PyScheduler:
                 del self.seqs[sid]
         return out
 
+    # stepped sequences: the caller decides which tokens run when, the scheduler only keeps their pages
+    def open(self, sid):
+        if sid in self.seqs:
+            return -1
+        self.seqs[sid] = dict(id=sid, prompt_len=0, max_new=0, num_tokens=0, num_generated=0, running=False, share_with=-1,
+                              prefilled=False, arrival=self.clock, blocks=[], stepped=True)
+        self.clock += 1
+        return 0
+
+    def extend(self, sid, count):
+        s = self.seqs.get(sid)
+        if s is None or not s.get("stepped") or count < 0:
+            return -1
+        if not self._ensure(s, s["num_tokens"] + count):
+            return -2
+        s["num_tokens"] += count
+        return s["num_tokens"] - count
+
+    def close(self, sid):
+        s = self.seqs.get(sid)
+        if s is None or not s.get("stepped"):
+            return -1
+        self._release(s)
+        del self.seqs[sid]
+        return 0
+
     @property
     def num_free_blocks(self):
         return len(self.free)
@@ -302,6 +332,15 @@ class _NativeScheduler:
         self.lib.rlb_engine_cache_stats(self.h, *[C.byref(x) for x in v])
         return dict(zip(("hits", "queries", "evictions", "cached_blocks"), (x.value for x in v)))
 
+    def open(self, sid):
+        return self.lib.rlb_engine_open(self.h, sid)
+
+    def extend(self, sid, count):
+        return self.lib.rlb_engine_extend(self.h, sid, count)
+
+    def close(self, sid):
+        return self.lib.rlb_engine_close(self.h, sid)
+
     @property
     def window(self) -> int:
         return self.lib.rlb_engine_window(self.h)
@@ -392,6 +431,10 @@ class GenerationEngine:
         # ``_hybrid_block``. Prefixes are not shared between sequences (pages carry no state) and decode runs eagerly.
         self.hybrid = bool(self.cfg.is_hybrid)
         self._attn_layers = [i for i, l in enumerate(model.layers) if l.self_attn is not None]
+        # layer-list models (Gadarax): one cache or state pool per layer RUN (a looped layer has one per pass), see ``_mixer_forward``
+        self.mixer = bool(self.cfg.is_mixer)
+        self.runs = self.cfg.layer_runs if self.mixer else []
+        self.stateful = bool(self.cfg.is_recurrent)   # sequences own a row of the state pools: prefixes are not shared by pages
         if self.hybrid:
             ep_h = getattr(model, "ep", None)
             if self.tpw > 1 or (ep_h is not None and ep_h.world > 1):
@@ -405,6 +448,10 @@ class GenerationEngine:
         self._r3_buf: list = []
         self.mamba_conv: Optional[list] = None
         self.mamba_ssm: Optional[list] = None
+        self.latent_cache: Optional[list] = None      # per run: [pages, page size, latent width] (latent attention)
+        self.ret_state: Optional[list] = None         # per run: [state rows, heads, dim, vdim] fp32 (retention)
+        self._step_ids: dict = {}                     # requests driven through ``step``: caller's id -> sequence id
+        self._step_next = 0
         self._state_row: dict[int, int] = {}
         self._free_rows: list[int] = []
         self._decode_rows: Optional[torch.Tensor] = None
@@ -427,6 +474,8 @@ class GenerationEngine:
             elif self.device.type == "cuda":
                 free, _ = torch.cuda.mem_get_info(self.device)
                 per_block = 2 * max(1, len(self._attn_layers)) * self.hkv * block_size * c.head_dim * 2
+                if self.mixer:
+                    per_block = max(1, sum(self._latent_width(i) for i, _ in self.runs)) * block_size * model.embed_tokens.element_size()
                 num_blocks = max(16, int(free * gpu_memory_utilization) // per_block)
             else:
                 num_blocks = 256
@@ -444,7 +493,7 @@ class GenerationEngine:
         # Prefix cache: full prompt blocks stay addressable by the hash of the token prefix they end, across requests and
         # generate calls (until the weights change: ``sleep`` resets it). A later prompt with the same prefix, e.g. the next
         # turn of a multi-turn rollout, prefills only its new tokens.
-        self.prefix_caching = bool(enable_prefix_caching) and isinstance(self.sched, _NativeScheduler) and not self.hybrid
+        self.prefix_caching = bool(enable_prefix_caching) and isinstance(self.sched, _NativeScheduler) and not self.stateful
         self._graphs: dict[int, tuple] = {}
         self._agreed_bucket = 0
         self._static: Optional[dict] = None
@@ -487,6 +536,11 @@ class GenerationEngine:
         if self.k_cache is not None:
             return
         c = self.cfg
+        if self.stateful:
+            self._state_row, self._free_rows = {}, list(range(self.max_running, 0, -1))
+        if self.mixer:
+            self._wake_mixer()
+            return
         shape = (self.num_blocks, self.hkv, self.block_size, c.head_dim)
         dt = self.model.dtype
         attn = set(self._attn_layers)
@@ -498,24 +552,42 @@ class GenerationEngine:
                                for l in self.model.layers]
             self.mamba_ssm = [torch.zeros((R, c.mamba_num_heads, c.mamba_head_dim, c.ssm_state_size), dtype=torch.float32, device=self.device)
                               if l.kind == "mamba" else None for l in self.model.layers]
-            self._state_row, self._free_rows = {}, list(range(R - 1, 0, -1))
+
+    def _latent_width(self, layer: int) -> int:
+        m = self.model.layers[layer].mixer
+        return m.latent_width if m.kind == "latent_attention" else 0
+
+    def _wake_mixer(self) -> None:
+        """Pools of a layer-list model, one per layer run: latent pages for latent attention, fp32 state rows (row 0 is scratch for the
+        padding rows of a decode batch) for retention."""
+        dt, dev = self.model.dtype, self.device
+        mx = [self.model.layers[i].mixer for i, _ in self.runs]
+        self.k_cache = self.v_cache = []     # (no key / value pages)
+        self.latent_cache = [torch.zeros((self.num_blocks, self.block_size, m.latent_width), dtype=dt, device=dev)
+                             if m.kind == "latent_attention" else None for m in mx]
+        self.ret_state = [torch.zeros((self.max_running + 1, m.heads, m.dim, m.vdim), dtype=torch.float32, device=dev)
+                          if m.kind == "retention" else None for m in mx]
 
     def sleep(self, free_kv_cache: bool = True) -> None:
         """Ends a generation phase: drops all requests; optionally returns the KV cache memory (captured graphs are
         tied to the cache addresses and are dropped with it)."""
         self.sched.reset()
-        if self.hybrid:
+        self._step_ids = {}
+        if self.stateful:
             self._state_row, self._free_rows = {}, list(range(self.max_running, 0, -1))
         if free_kv_cache:
             self._graphs.clear()
             self._static = None
             self.k_cache = self.v_cache = None
             self.mamba_conv = self.mamba_ssm = None
+            self.latent_cache = self.ret_state = None
             if self.device.type == "cuda":
                 torch.cuda.empty_cache()
 
     def kv_cache_bytes(self) -> int:
         c = self.cfg
+        if self.mixer:
+            return sum(self._latent_width(i) for i, _ in self.runs) * self.num_blocks * self.block_size * self.model.embed_tokens.element_size()
         return 2 * len(self._attn_layers) * self.num_blocks * self.hkv * self.block_size * c.head_dim * self.model.dtype.itemsize if hasattr(self.model.dtype, "itemsize") else 0
 
     # ------------------------------------------------------------------ routed-expert recording (rollout routing replay)
@@ -780,8 +852,123 @@ class GenerationEngine:
             h, x = comm.allreduce_rows(part, h, next_w, eps)
         return self._output_logits(x, logits_out)
 
+    # ------------------------------------------------------------------ layer-list models
+    @torch.no_grad()
+    def _mixer_forward(self, b: "X.TokenBatch", rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """One pass over the rows of ``b`` (single decoded tokens and portions of prompts alike); logits of ``rows`` (None: all).
+        Per layer run: fused input product, mixer, fused output product; the last one's epilogue also updates the fp32 residual
+        stream, makes the loop's additions and applies the next layer's norm."""
+        m, c, runs = self.model, self.cfg, self.runs
+        norms = [m.layers[i].norm for i, _ in runs] + [m.norm]
+
+        def begins(r):    # (embeddings are added again, step vector) when run r is the first of a pass of the loop
+            i, t = runs[r] if r < len(runs) else (None, None)
+            return (t > 0, m.loop_step[t]) if t is not None and i == c.layer_loop["start"] else (False, None)
+
+        x, e, h = X.embed_rows(b.ids, m.embed_tokens, c.embed_scale, begins(0)[1], norms[0],
+                               keep=c.layer_loop is not None and c.layer_loop["times"] > 1)
+        for r, (i, _) in enumerate(runs):
+            layer = m.layers[i]
+            mx = layer.mixer
+            p = X.in_proj(h, layer.in_proj, layer.up_off)
+            if mx.kind == "latent_attention":
+                X.latent_attention_(p, mx, b, self.latent_cache[r])
+            else:
+                X.retention_(p, mx, b, self.ret_state[r])
+            again, step = begins(r + 1)
+            h = X.out_proj_(x, p[:, mx.mix_off : mx.mix_off + layer.out_width], layer.out_proj, e if again else None, step, norms[r + 1])
+        if rows is not None:
+            h = h.index_select(0, rows)
+        return X.logits(h, m.output_weight, self.logits_dtype)
+
+    def _token_batch(self, items) -> tuple:
+        """Rows of one step from ``items`` = [(sequence id, tokens, first position)]. Single tokens come first, then portions in order of
+        length; returns (batch, first row of every item in the order of ``items``)."""
+        dev = self.device
+        order = sorted(range(len(items)), key=lambda j: len(items[j][1]))
+        first, toks, pos, slots, lens = [0] * len(items), [], [], [], []
+        for j in order:
+            sid, seq, p = items[j]
+            first[j] = len(toks)
+            toks.extend(seq)
+            lens.append(len(seq))
+            pos.append(torch.arange(p, p + len(seq), dtype=torch.int32))
+            slots.append(self.sched.slots(sid, p, len(seq)))
+        n_single = sum(1 for n in lens if n == 1)
+        pos = torch.cat(pos)
+        ids = _L.to_device(torch.tensor(toks, dtype=torch.int32 if self.native else torch.int64), dev)
+        sids = [items[j][0] for j in order]
+        bt, _, _ = self.sched.tables(sids, self.max_blocks_per_seq)
+        of_row = torch.repeat_interleave(torch.arange(len(lens)), torch.tensor(lens))
+        b = X.TokenBatch(ids=ids, positions=pos.to(dev), slots=torch.cat(slots).to(dev), n_single=n_single, n_paged=len(toks),
+                         block_table=bt[of_row].to(dev), seq_lens=(pos + 1).to(dev), max_ctx=int(pos.max()) + 1)
+        if self.stateful:
+            b.state_rows = torch.tensor([self._state_row[s] for s in sids], dtype=torch.int64, device=dev)
+        if n_single < len(lens):
+            cu = torch.zeros(len(lens) - n_single + 1, dtype=torch.int32)
+            cu[1:] = torch.tensor(lens[n_single:], dtype=torch.int64).cumsum(0)
+            b.cu, b.max_portion = cu.to(dev), lens[-1]
+        return b, first
+
+    @torch.no_grad()
+    def step(self, entries, end=()) -> list:
+        """Runs exactly the given tokens as one batch, from the cache and state that earlier calls left, and returns the wanted logits.
+        ``entries`` = [(request, tokens, places wanted among them)], ``end`` = requests whose pages and state are given back
+        afterwards. A request is admitted by its first entry; nothing is sampled. Returns one [wanted, vocab] tensor per entry.
+
+        The forward pass is the one :meth:`generate` uses: single tokens run as decode rows, longer entries as prompt portions
+        that continue after the cached tokens."""
+        self.wake()
+        self.model.eval()
+        names = [r for r, _, _ in entries]
+        if len(set(names)) != len(names):
+            raise ValueError("a request has two entries in one step")
+        items = []
+        for name, toks, _ in entries:
+            if not toks:
+                raise ValueError(f"request {name!r}: an entry without tokens")
+            if name not in self._step_ids:
+                sid = (1 << 40) + self._step_next
+                self._step_next += 1
+                if len(self._step_ids) >= self.max_running or self.sched.open(sid):
+                    raise RuntimeError(f"request {name!r}: more than {self.max_running} live requests")
+                if self.stateful:
+                    self._state_row[sid] = self._free_rows.pop()
+                self._step_ids[name] = sid
+            sid = self._step_ids[name]
+            p = self.sched.extend(sid, len(toks))
+            if p < 0:
+                raise RuntimeError(f"request {name!r}: the cache has no room for {len(toks)} more tokens")
+            if p + len(toks) > self.max_model_len:
+                raise ValueError(f"request {name!r} grows beyond {self.max_model_len} tokens")
+            items.append((sid, [int(t) for t in toks], p))
+        out = []
+        if self.mixer and items:
+            b, first = self._token_batch(items)
+            rows = [first[j] + w for j, (_, _, want) in enumerate(entries) for w in want]
+            z = self._mixer_forward(b, torch.tensor(rows, dtype=torch.int64, device=self.device))
+        elif items:
+            z = self._prefill_round([(sid, [0] * p + toks, p, len(toks)) for sid, toks, p in items], self.device,
+                                    wants=[want for _, _, want in entries])
+        at = 0
+        for _, _, want in entries:
+            out.append(z[at : at + len(want)])
+            at += len(want)
+        for name in end:
+            sid = self._step_ids.pop(name)
+            self.sched.close(sid)
+            if self.stateful:
+                self._free_rows.append(self._state_row.pop(sid))
+        if self.native:
+            _L.raise_on_status("GenerationEngine.step", self.device)
+        return out
+
     @torch.no_grad()
     def _decode_forward(self, ids, positions, slots, block_table, seq_lens, num_splits, scratch, logits_out=None):
+        if self.mixer:
+            n = ids.shape[0]
+            return self._mixer_forward(X.TokenBatch(ids=ids, positions=positions, slots=slots, n_single=n, n_paged=n, block_table=block_table,
+                                                    seq_lens=seq_lens, state_rows=self._decode_rows, max_ctx=self.max_model_len))
         if self._can_fuse_decode(ids.shape[0]):
             return self._decode_forward_fused(ids, positions, slots, block_table, seq_lens, num_splits, scratch, logits_out)
         if self._can_fuse_decode_tp(ids.shape[0]):
@@ -944,6 +1131,10 @@ class GenerationEngine:
 
     def _prefill_plain(self, items, reqs, dev) -> dict:
         """Whole prompts in one packed batch (nothing cached, nothing longer than the prefill budget)."""
+        if self.mixer:
+            z = self._prefill_round([(sid, seq, 0, len(seq)) for sid, seq, _ in items], dev)
+            self.stats["prefill_tokens"] += sum(len(seq) for _, seq, _ in items)
+            return {sid: z[j] for j, (sid, _, _) in enumerate(items)}
         toks, lens, slots = [], [], []
         for sid, seq, _ in items:
             toks.extend(seq)
@@ -994,9 +1185,16 @@ class GenerationEngine:
         return out
 
     @torch.no_grad()
-    def _prefill_round(self, round_items, dev) -> torch.Tensor:
+    def _prefill_round(self, round_items, dev, wants=None) -> torch.Tensor:
         """One packed forward over the NEW tokens of several sequences: sequence i contributes tokens [p_i, p_i + n_i) and
-        attends to its p_i cached tokens. Returns the logits of every sequence's last new token."""
+        attends to its p_i cached tokens. Returns the logits of every sequence's last new token, or of the places ``wants[i]``
+        among its new tokens."""
+        if wants is None:
+            wants = [[n - 1] for _, _, _, n in round_items]
+        if self.mixer:
+            b, first = self._token_batch([(sid, seq[p : p + n], p) for sid, seq, p, n in round_items])
+            rows = [first[j] + w for j, want in enumerate(wants) for w in want]
+            return self._mixer_forward(b, torch.tensor(rows, dtype=torch.int64, device=dev))
         m, c = self.model, self.cfg
         hq, hkv, D = self.hq, self.hkv, c.head_dim
         idt = torch.int32 if self.native else torch.int64
@@ -1012,7 +1210,7 @@ class GenerationEngine:
             new_idx.append(torch.arange(row + p, row + p + n))
             row += p + n
             full_lens.append(p + n)
-            last.append(len(toks) - 1)
+            last.extend(len(toks) - n + w for w in wants[len(full_lens) - 1])
         ids = _L.to_device(torch.tensor(toks, dtype=idt), dev)
         self._r3_rows([sid for sid, _, _, n in round_items for _ in range(n)], torch.cat(pos))
         positions = torch.cat(pos).to(dev)
@@ -1086,7 +1284,7 @@ class GenerationEngine:
             ids_np[j] = r.out_tokens[-1]
             keys_np[j] = self._row_key(r, sp)
             rem_np[j] = r.max_new - len(r.out_tokens)
-        if self.hybrid:
+        if self.stateful:
             hb["state_rows"].zero_()    # padding rows use the scratch row
             for j, sid in enumerate(decode):
                 hb["state_rows"][j] = self._state_row[sid]
@@ -1182,7 +1380,7 @@ class GenerationEngine:
             mm = mm_inputs[i] if mm_inputs is not None else None
             if mm is not None and mm[0] is None:
                 mm = None
-            if share_prefixes and not self.hybrid and not self.record_routing:   # (shared pages carry no state / no routing record)
+            if share_prefixes and not self.stateful and not self.record_routing:   # (shared pages carry no state / no routing record)
                 key = tuple(p)
                 if mm is not None:   # equal prompts share their prefix only if they show the same images
                     from rl_b200.data.multimodal_utils import content_key
@@ -1241,7 +1439,7 @@ class GenerationEngine:
                                       sum(1 for r in reqs.values() if not r.finished)))
             if not idle and not prefill and not shared and not decode:
                 raise RuntimeError("scheduler made no progress (KV cache too small for a single request)")
-            if self.hybrid:
+            if self.stateful:
                 self._claim_state_rows(set(prefill) | set(decode))
             agreed_steps = None
             if lock:
@@ -1283,7 +1481,7 @@ class GenerationEngine:
                     r = reqs[sid]
                     ids_np[j] = r.out_tokens[-1]
                     keys_np[j] = self._row_key(r, sp)
-                    if self.hybrid:
+                    if self.stateful:
                         hb["state_rows"][j] = self._state_row[sid]
                 st["blob"].copy_(st["host_blob"], non_blocking=True)
                 self._step_counter += 1
@@ -1327,6 +1525,10 @@ class GenerationEngine:
                 if copies:
                     src = torch.tensor([a for a, _ in copies], dtype=torch.int32, device=dev)
                     dst = torch.tensor([b for _, b in copies], dtype=torch.int32, device=dev)
+                    for cache in (self.latent_cache or []):
+                        if cache is not None:
+                            raw = cache.view(torch.bfloat16)
+                            E.block_copy(raw, raw, src, dst)
                     for li in self._attn_layers:
                         E.block_copy(self.k_cache[li], self.v_cache[li], src, dst)
                 new = list(prefill) + list(shared)

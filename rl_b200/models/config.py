@@ -4,6 +4,9 @@ One dataclass covers Llama (2/3/3.1/3.2), Mistral, Qwen2/2.5, Qwen3, Qwen3-MoE a
 (QKV bias, per-head q/k RMSNorm, tied embeddings, RoPE scaling, mixture-of-experts FFN; for Gemma 3: tanh-GELU gate, norms
 before and after each block, scaled embeddings, sliding-window layers with their own RoPE base, a fixed attention scale). ``from_hf_dict`` reads a
 HuggingFace ``config.json`` dictionary; ``PRESETS`` names the architectures used by the benchmark configs.
+
+Models described layer by layer (Gadarax) keep their layer list in ``mixers``: each entry names the sequence mixer, its sizes and its
+MLP; ``layer_loop`` runs a range of layers several times with the same weights.
 """
 
 from __future__ import annotations
@@ -90,9 +93,32 @@ class ModelConfig:
     moe_latent_size: Optional[int] = None      # routed experts work in a narrower space between two shared projections
     moe_shared_expert_intermediate_size: int = 0
 
+    # Gadarax: every layer is one norm whose output feeds a sequence mixer and an MLP side by side; the layers differ
+    mixers: Optional[list] = None      # per layer: {"type": "latent_attention" | "retention", "mixer": {sizes}, "mlp": {"kind", "ff"} or None}
+    layer_loop: Optional[dict] = None  # {"start", "stop", "times"}: layers start .. stop - 1 run `times` times in a row with the same weights
+    norm_kind: str = "rms"             # "rms" | "dyt" (dynamic tanh: w * tanh(alpha x) + b, no statistics)
+
     @property
     def is_hybrid(self) -> bool:
         return self.layers_block_type is not None
+
+    @property
+    def is_mixer(self) -> bool:
+        return self.mixers is not None
+
+    @property
+    def is_recurrent(self) -> bool:
+        """Some layer carries a per-sequence state beside (or instead of) cache pages: prefixes cannot be shared by pages."""
+        return self.is_hybrid or (self.mixers is not None and any(m["type"] == "retention" for m in self.mixers))
+
+    @property
+    def layer_runs(self) -> list:
+        """[(layer, pass)] in execution order; pass counts from 0 inside the loop and is None outside it."""
+        lp, n = self.layer_loop, self.num_hidden_layers
+        if not lp:
+            return [(i, None) for i in range(n)]
+        body = [(i, t) for t in range(lp["times"]) for i in range(lp["start"], lp["stop"])]
+        return [(i, None) for i in range(lp["start"])] + body + [(i, None) for i in range(lp["stop"], n)]
 
     def block_type(self, i: int) -> str:
         """"mamba" | "attention" | "mlp" | "moe" for hybrid models, "decoder" (attention + MLP in one layer) otherwise."""
@@ -136,6 +162,18 @@ class ModelConfig:
 
     def num_parameters(self) -> int:
         d, L = self.hidden_size, self.num_hidden_layers
+        if self.mixers is not None:
+            n = self.vocab_size * d + 2 * d + 1 + (self.layer_loop["times"] * d if self.layer_loop else 0)
+            for e in self.mixers:
+                m = e["mixer"]
+                H, kd, vd = m["heads"], m["dim"], m["vdim"]
+                if e["type"] == "latent_attention":
+                    R, rd = m["kv_rank"], m["rot_dim"]
+                    n += d * (H * (kd + rd) + R + rd + 2 * H * vd) + R + H * (kd + vd) * R
+                else:
+                    n += d * (2 * H * kd + 3 * H * vd)
+                n += 2 * d * (e["mlp"]["ff"] if e.get("mlp") else 0) + 2 * d + 1
+            return n
         if self.layers_block_type is not None:
             I, C, H = self.mamba_inner, self.mamba_conv_dim, self.mamba_num_heads
             din = self.moe_latent_size or d
@@ -155,11 +193,17 @@ class ModelConfig:
         return L * (attn + ffn + norms) + emb + d
 
     def to_hf_dict(self) -> dict:
+        if self.is_mixer:
+            out = {"architecture": "Gadarax", "vocab": self.vocab_size, "width": self.hidden_size, "embedding": {"scale": self.embed_scale},
+                   "norm": {"eps": self.rms_norm_eps}, "layers": self.mixers, "torch_dtype": self.torch_dtype}
+            return dict(out, loop=self.layer_loop) if self.layer_loop else out
         arch = {"llama": "LlamaForCausalLM", "mistral": "MistralForCausalLM", "qwen2": "Qwen2ForCausalLM",
                 "qwen3": "Qwen3ForCausalLM", "qwen3_moe": "Qwen3MoeForCausalLM",
                 "gemma3_text": "Gemma3ForCausalLM", "deepseek_v3": "DeepseekV3ForCausalLM",
                 "nemotron_h": "NemotronHForCausalLM"}.get(self.model_type, "LlamaForCausalLM")
         d = asdict(self)
+        for k in ("mixers", "layer_loop", "norm_kind"):
+            d.pop(k)
         nh = {k: d.pop(k) for k in ("layers_block_type", "use_rope", "mlp_gated", "mlp_bias", "mamba_num_heads", "mamba_head_dim", "ssm_state_size",
                                     "mamba_n_groups", "mamba_d_conv", "mamba_chunk_size", "mamba_conv_bias", "mamba_proj_bias", "mamba_dt_limit",
                                     "moe_latent_size", "moe_shared_expert_intermediate_size")}
@@ -200,6 +244,8 @@ class ModelConfig:
 
     @classmethod
     def from_hf_dict(cls, hf: dict, **overrides) -> "ModelConfig":
+        if hf.get("architecture") == "Gadarax":
+            return cls._from_layer_list(hf, **overrides)
         mt = hf.get("model_type", "llama")
         if mt == "gemma3" and "text_config" in hf:      # the multimodal wrapper: the language model's settings are nested
             hf = dict(hf["text_config"], model_type="gemma3_text")
@@ -306,6 +352,39 @@ class ModelConfig:
         return cfg
 
     @classmethod
+    def _from_layer_list(cls, hf: dict, **overrides) -> "ModelConfig":
+        """Configurations that describe the model layer by layer (Gadarax)."""
+        layers = hf["layers"]
+        for i, e in enumerate(layers):
+            need = {"latent_attention": ("heads", "dim", "rot_dim", "vdim", "kv_rank", "scale", "rot"),
+                    "retention": ("heads", "dim", "vdim", "decay", "rot")}.get(e["type"])
+            if need is None:
+                raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
+            missing = [k for k in need if k not in e["mixer"]]
+            if missing:
+                raise ValueError(f"layer {i}: the {e['type']} mixer lacks {missing}")
+            if e.get("mlp") and e["mlp"].get("kind", "dense") != "dense":
+                raise ValueError(f"layer {i}: unknown MLP kind {e['mlp']['kind']!r}")
+            m = e["mixer"]
+            if e["type"] == "retention" and len(m["decay"]) != m["heads"]:
+                raise ValueError(f"layer {i}: {len(m['decay'])} decays for {m['heads']} heads")
+            limit = m["rot_dim"] if e["type"] == "latent_attention" else m["dim"]
+            if m["rot"]["dims"] > limit or m["rot"]["dims"] % 2:
+                raise ValueError(f"layer {i}: {m['rot']['dims']} rotated dimensions in a part of {limit}")
+        lp = hf.get("loop")
+        if lp and not (0 <= lp["start"] < lp["stop"] <= len(layers) and lp["times"] >= 1):
+            raise ValueError(f"layer loop {lp} does not fit {len(layers)} layers")
+        m0 = layers[0]["mixer"]
+        cfg = cls(model_type="gadarax", vocab_size=hf["vocab"], hidden_size=hf["width"], num_hidden_layers=len(layers),
+                  intermediate_size=max([e["mlp"]["ff"] for e in layers if e.get("mlp")] or [0]), num_attention_heads=m0["heads"],
+                  num_key_value_heads=m0["heads"], head_dim=m0["dim"], rms_norm_eps=float(hf["norm"]["eps"]), tie_word_embeddings=True,
+                  mlp_gated=False, hidden_act="relu2", embed_scale=float(hf["embedding"]["scale"]), norm_kind="dyt", mixers=layers,
+                  layer_loop=dict(lp) if lp else None, torch_dtype=str(hf.get("torch_dtype", "bfloat16")).replace("torch.", ""))
+        for k, v in overrides.items():
+            setattr(cfg, k, v)
+        return cfg
+
+    @classmethod
     def from_pretrained(cls, path: str, **overrides) -> "ModelConfig":
         with open(os.path.join(path, "config.json")) as f:
             return cls.from_hf_dict(json.load(f), **overrides)
@@ -349,6 +428,26 @@ def rope_inv_freq(cfg: ModelConfig, device=None) -> torch.Tensor:
         ramp = ((torch.arange(D // 2, dtype=torch.float32) - lo) / max(hi - lo, 1e-3)).clamp(0, 1)
         inv = inv / factor * ramp + inv * (1 - ramp)
     return inv.to(device) if device is not None else inv
+
+
+def rotary_table(rot: dict) -> tuple[torch.Tensor, float]:
+    """Angle per position of each rotated pair [dims / 2] (fp32) and the factor on cosine and sine, for a rotation described by
+    ``{"dims", "base"}`` and optionally ``"scaling"`` = YaRN's ``{"factor", "original", "fast", "slow"}``: pairs that turn more than
+    ``fast`` times within the original context keep their frequency, pairs that turn less than ``slow`` times are slowed down by
+    ``factor``, with a linear ramp between the two (upper end clamped at the last dimension)."""
+    n, base = int(rot["dims"]), float(rot["base"])
+    f = base ** (-2.0 * torch.arange(n // 2, dtype=torch.float64) / n) if n else torch.zeros(0, dtype=torch.float64)
+    s = rot.get("scaling")
+    if not s:
+        return f.float(), 1.0
+    factor = float(s["factor"])
+
+    def dim_of(turns):
+        return n * math.log(float(s["original"]) / (2 * math.pi * float(turns))) / (2 * math.log(base))
+
+    lo, hi = max(math.floor(dim_of(s["fast"])), 0), min(math.ceil(dim_of(s["slow"])), n - 1)
+    ramp = ((torch.arange(n // 2, dtype=torch.float64) - lo) / max(hi - lo, 1e-3)).clamp(0, 1)
+    return (f / factor * ramp + f * (1 - ramp)).float(), 0.1 * math.log(factor) + 1.0
 
 
 PRESETS: dict[str, dict] = {

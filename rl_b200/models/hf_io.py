@@ -173,6 +173,17 @@ def _model_map(model: CausalLM):
 def iter_hf_shards(model: CausalLM) -> Iterator[tuple[str, torch.Tensor, Optional[tuple[int, int, int]]]]:
     """Yields (hf_name, local tensor view, hf_slice) for every logical HF tensor (or shard of one) this rank holds."""
     cfg = model.cfg
+    if cfg.is_mixer:    # layer-list models (Gadarax) keep their checkpoint's own tensor names
+        yield "embed", model.embed_tokens, None
+        if model.loop_step is not None:
+            yield "loop.step", model.loop_step, None
+        for i, layer in enumerate(model.layers):
+            for name, view in layer.tensor_views(f"l{i}."):
+                yield name, view, None
+        yield "final.norm", model.norm.weight, None
+        yield "final.norm.b", model.norm.bias, None
+        yield "final.norm.alpha", model.norm.alpha, None
+        return
     params = _local(model)
     ep_rank, ep_size = (model.ep.rank, model.ep.world) if model.ep is not None else (0, 1)
     per = cfg.num_experts // ep_size if cfg.is_moe else 0

@@ -1,0 +1,242 @@
+"""Sequence mixers that sit beside an MLP in one parallel layer, and that layer.
+
+A parallel layer computes ``h = norm(x)`` once and adds ``mixer(h) + mlp(h)`` to the residual stream, so all its input projections
+read the same rows and both its output projections write the same rows. The layer therefore holds two fused weights:
+
+    in_proj  [mixer projections | gate | MLP up, d]     one product of ``h``; squared ReLU rides on the ``up`` columns
+    out_proj [d, mixed | MLP ff]                        one product whose left operand is the [gate | up] range of the first
+                                                        product's rows: the mixer writes its gated output over the gate columns
+
+Segments start at multiples of 8 columns (16-byte rows for TMA); padding rows and columns hold zeros. The residual stream is fp32.
+
+Mixers:
+  * ``LatentAttentionMixer``: causal attention whose keys and values are decompressed from one normalised latent per token; only
+    the latent and a rotated key part shared by the heads are cached. Own softmax scale, output gate, interleaved rotation.
+  * ``RetentionMixer``: linear attention with one fixed decay per head, a unit-RMS norm per head and a SiLU gate. The state
+    [heads, dim, vdim] is fp32.
+
+The modules' ``sequence`` methods are the differentiable PyTorch statement over packed sequences (training, CPU); the generation
+engine runs the same weights through ``rl_b200/ops/mixer_ops.py``.
+"""
+
+from __future__ import annotations
+
+import torch
+import torch.nn as nn
+import torch.nn.functional as TF
+
+from rl_b200.ops import functional as F
+
+from .config import ModelConfig, rotary_table
+
+
+def pad8(n: int) -> int:
+    return -(-n // 8) * 8
+
+
+class DynamicTanh(nn.Module):
+    """y = w * tanh(alpha x) + b: a norm without statistics. Evaluated in fp32, returned in ``out_dtype``."""
+
+    def __init__(self, d: int, dtype, device):
+        super().__init__()
+        self.weight = nn.Parameter(torch.ones(d, dtype=dtype, device=device))
+        self.bias = nn.Parameter(torch.zeros(d, dtype=dtype, device=device))
+        self.alpha = nn.Parameter(torch.full((), 0.5, dtype=dtype, device=device))
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        y = torch.tanh(self.alpha.float() * x.float()) * self.weight.float() + self.bias.float()
+        return y.to(self.weight.dtype)
+
+
+def rotate_pairs(x: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor, gain: float, interleaved: bool) -> torch.Tensor:
+    """fp32 rotation of the leading ``2 * len(freq)`` dimensions of ``x`` [T, H, n]; pairs are (2i, 2i + 1) when ``interleaved``,
+    else (i, i + len(freq)). Cosine and sine are multiplied by ``gain``."""
+    x = x.float()
+    half = freq.numel()
+    if half == 0:
+        return x
+    ang = positions.float()[:, None] * freq[None, :]
+    c, s = (ang.cos() * gain)[:, None, :], (ang.sin() * gain)[:, None, :]
+    head, rest = x[..., : 2 * half], x[..., 2 * half :]
+    u, v = (head[..., 0::2], head[..., 1::2]) if interleaved else (head[..., :half], head[..., half:])
+    a, b = u * c - v * s, v * c + u * s
+    rot = torch.stack([a, b], dim=-1).flatten(-2) if interleaved else torch.cat([a, b], dim=-1)
+    return torch.cat([rot, rest], dim=-1)
+
+
+class LatentAttentionMixer(nn.Module):
+    kind = "latent_attention"
+
+    def __init__(self, spec: dict, cfg: ModelConfig, dtype, device):
+        super().__init__()
+        self.heads, self.dim, self.rot_dim, self.vdim = spec["heads"], spec["dim"], spec["rot_dim"], spec["vdim"]
+        self.rank, self.scale, self.eps = spec["kv_rank"], float(spec["scale"]), cfg.rms_norm_eps
+        self.qdim = self.dim + self.rot_dim
+        self.latent_width = pad8(self.rank + self.rot_dim)       # row width of the cache: [latent | rotated key | padding]
+        H = self.heads
+        self.q_off, self.lat_off = 0, pad8(H * self.qdim)
+        self.mix_off = self.lat_off + pad8(self.rank + self.rot_dim)
+        self.mix_width = pad8(H * self.vdim)
+        self.in_width = self.mix_off + self.mix_width
+        self.kv_norm = nn.Parameter(torch.ones(self.rank, dtype=dtype, device=device))
+        self.kv_up = nn.Parameter(torch.empty(H * (self.dim + self.vdim), self.rank, dtype=dtype, device=device))   # [keys | values]
+        freq, self.gain = rotary_table(spec["rot"])
+        self.register_buffer("freq", freq.to(device), persistent=False)
+
+    def in_rows(self) -> list:
+        """(checkpoint leaf, first row, rows) of this mixer's slices of ``in_proj``."""
+        H = self.heads
+        return [("q", self.q_off, H * self.qdim), ("dkv", self.lat_off, self.rank + self.rot_dim), ("g", self.mix_off, H * self.vdim)]
+
+    def own_tensors(self) -> list:
+        """(checkpoint leaf, parameter name, first row, rows or None)."""
+        H = self.heads
+        return [("dkv.norm", "kv_norm", 0, None), ("uk", "kv_up", 0, H * self.dim), ("uv", "kv_up", H * self.dim, H * self.vdim)]
+
+    def key_parts(self, p: torch.Tensor, positions: torch.Tensor):
+        """From the projected rows: normalised latent [T, rank] and rotated shared key [T, rot_dim], both fp32."""
+        lat = p[:, self.lat_off : self.lat_off + self.rank].float()
+        lat = lat * torch.rsqrt(lat.pow(2).mean(-1, keepdim=True) + self.eps) * self.kv_norm.float()
+        kr = p[:, self.lat_off + self.rank : self.lat_off + self.rank + self.rot_dim]
+        return lat, rotate_pairs(kr[:, None], positions, self.freq, self.gain, True)[:, 0]
+
+    def queries(self, p: torch.Tensor, positions: torch.Tensor):
+        q = p[:, self.q_off : self.q_off + self.heads * self.qdim].reshape(-1, self.heads, self.qdim)
+        return torch.cat([q[..., : self.dim].float(), rotate_pairs(q[..., self.dim :], positions, self.freq, self.gain, True)], dim=-1)
+
+    def sequence(self, p: torch.Tensor, positions: torch.Tensor, cu_seqlens: torch.Tensor) -> torch.Tensor:
+        """Gated head outputs [T, heads * vdim] of packed whole sequences."""
+        T, H = p.shape[0], self.heads
+        lat, kr = self.key_parts(p, positions)
+        lat = lat.to(p.dtype)
+        k = TF.linear(lat, self.kv_up[: H * self.dim]).reshape(T, H, self.dim)
+        v = TF.linear(lat, self.kv_up[H * self.dim :]).reshape(T, H, self.vdim).float()
+        k = torch.cat([k.float(), kr[:, None].expand(T, H, self.rot_dim)], dim=-1)
+        q = self.queries(p, positions)
+        out = []
+        cu = cu_seqlens.tolist()
+        for s, e in zip(cu[:-1], cu[1:]):
+            z = torch.einsum("ihd,jhd->hij", q[s:e], k[s:e]) * self.scale
+            z = z.masked_fill(torch.ones(e - s, e - s, dtype=torch.bool, device=z.device).triu(1), float("-inf"))
+            out.append(torch.einsum("hij,jhd->ihd", torch.softmax(z, -1), v[s:e]))
+        y = torch.cat(out).reshape(T, H * self.vdim)
+        return (y * torch.sigmoid(p[:, self.mix_off : self.mix_off + H * self.vdim].float())).to(p.dtype)
+
+
+class RetentionMixer(nn.Module):
+    kind = "retention"
+
+    def __init__(self, spec: dict, cfg: ModelConfig, dtype, device):
+        super().__init__()
+        self.heads, self.dim, self.vdim, self.eps = spec["heads"], spec["dim"], spec["vdim"], cfg.rms_norm_eps
+        H = self.heads
+        self.q_off = 0
+        self.k_off = pad8(H * self.dim)
+        self.v_off = self.k_off + pad8(H * self.dim)
+        self.mix_off = self.v_off + pad8(H * self.vdim)
+        self.mix_width = pad8(H * self.vdim)
+        self.in_width = self.mix_off + self.mix_width
+        freq, self.gain = rotary_table(spec["rot"])
+        self.register_buffer("freq", freq.to(device), persistent=False)
+        self.register_buffer("decay", torch.tensor(spec["decay"], dtype=torch.float32, device=device), persistent=False)
+        # log2 of the decays from the configuration's own precision: powers of a decay are taken as exp2(n * log2 decay)
+        self.register_buffer("log2_decay", torch.tensor(spec["decay"], dtype=torch.float64).log2().clamp(min=-1e4).float().to(device), persistent=False)
+
+    def in_rows(self) -> list:
+        H = self.heads
+        return [("q", self.q_off, H * self.dim), ("k", self.k_off, H * self.dim), ("v", self.v_off, H * self.vdim), ("g", self.mix_off, H * self.vdim)]
+
+    def own_tensors(self) -> list:
+        return []
+
+    def qkv(self, p: torch.Tensor, positions: torch.Tensor):
+        """fp32 rotated queries, rotated and scaled keys [T, H, dim], values [T, H, vdim]."""
+        H = self.heads
+        q = rotate_pairs(p[:, self.q_off : self.q_off + H * self.dim].reshape(-1, H, self.dim), positions, self.freq, self.gain, False)
+        k = rotate_pairs(p[:, self.k_off : self.k_off + H * self.dim].reshape(-1, H, self.dim), positions, self.freq, self.gain, False)
+        v = p[:, self.v_off : self.v_off + H * self.vdim].reshape(-1, H, self.vdim).float()
+        return q, k * self.dim ** -0.5, v
+
+    def finish(self, o: torch.Tensor, p: torch.Tensor) -> torch.Tensor:
+        """Unit-RMS norm per head and SiLU gate of the head outputs ``o`` [T, H, vdim] (fp32)."""
+        H = self.heads
+        o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + self.eps)
+        g = p[:, self.mix_off : self.mix_off + H * self.vdim].float()
+        return (o.reshape(-1, H * self.vdim) * TF.silu(g)).to(p.dtype)
+
+    def scan(self, q, k, v, S, chunk: int = 64):
+        """Outputs [L, H, vdim] of one sequence (piece) starting from state ``S`` [H, dim, vdim], and the state it leaves. Chunk by
+        chunk: the products inside a chunk are one masked score matrix, only chunk borders are visited one after the other."""
+        outs = []
+        ld = self.log2_decay.to(q.dtype)
+        for s in range(0, q.shape[0], chunk):
+            qc, kc, vc = q[s : s + chunk], k[s : s + chunk], v[s : s + chunk]
+            n = qc.shape[0]
+            i = torch.arange(n, device=q.device)
+            gap = (i[:, None] - i[None, :]).to(q.dtype)
+            w = torch.where(gap >= 0, torch.exp2(gap.clamp(min=0) * ld[:, None, None]), torch.zeros((), device=q.device, dtype=q.dtype))
+            o = torch.einsum("hij,jhv->ihv", torch.einsum("ihd,jhd->hij", qc, kc) * w, vc)
+            o = o + torch.einsum("ihd,hdv->ihv", qc, S) * torch.exp2((i + 1)[:, None].to(q.dtype) * ld)[..., None]
+            tail = torch.exp2((n - 1 - i)[:, None].to(q.dtype) * ld)
+            S = S * torch.exp2(n * ld)[:, None, None] + torch.einsum("jhd,jhv->hdv", kc * tail[..., None], vc)
+            outs.append(o)
+        return torch.cat(outs), S
+
+    def sequence(self, p: torch.Tensor, positions: torch.Tensor, cu_seqlens: torch.Tensor) -> torch.Tensor:
+        q, k, v = self.qkv(p, positions)
+        cu = cu_seqlens.tolist()
+        zero = torch.zeros(self.heads, self.dim, self.vdim, dtype=torch.float32, device=p.device)
+        return self.finish(torch.cat([self.scan(q[s:e], k[s:e], v[s:e], zero)[0] for s, e in zip(cu[:-1], cu[1:])]), p)
+
+
+MIXERS = {m.kind: m for m in (LatentAttentionMixer, RetentionMixer)}
+
+
+class ParallelBlock(nn.Module):
+    """x <- x + mixer(norm(x)) + mlp(norm(x)); the MLP may be absent."""
+
+    def __init__(self, cfg: ModelConfig, dtype, device, tp=None, ep=None, cp=None, lora=None, layer_idx: int = 0):
+        super().__init__()
+        assert (tp is None or tp.world == 1) and (cp is None or cp.world == 1) and not lora, \
+            "parallel mixer layers: no tensor / context parallelism, no LoRA"
+        self.cfg, self.layer_idx, self.window = cfg, layer_idx, 0
+        entry = cfg.mixers[layer_idx]
+        d = cfg.hidden_size
+        self.norm = DynamicTanh(d, dtype, device)
+        self.mixer = MIXERS[entry["type"]](entry["mixer"], cfg, dtype, device)
+        self.ff = entry["mlp"]["ff"] if entry.get("mlp") else 0
+        self.up_off = self.mixer.in_width                  # first MLP column of the projected rows; squared ReLU from here on
+        self.in_width = self.up_off + pad8(self.ff)
+        self.out_width = self.mixer.mix_width + pad8(self.ff)
+        self.in_proj = nn.Parameter(torch.zeros(self.in_width, d, dtype=dtype, device=device))
+        self.out_proj = nn.Parameter(torch.zeros(d, self.out_width, dtype=dtype, device=device))
+        self.self_attn = self.mlp = None                   # (the names other families' walkers look for)
+
+    def tensor_views(self, prefix: str) -> list:
+        """(checkpoint name, view of a parameter) of every tensor of this layer."""
+        m = self.mixer
+        out = [(f"{prefix}norm1", self.norm.weight), (f"{prefix}norm1.b", self.norm.bias), (f"{prefix}norm1.alpha", self.norm.alpha)]
+        out += [(f"{prefix}mix.{leaf}", self.in_proj[r : r + n]) for leaf, r, n in m.in_rows()]
+        for leaf, pname, r, n in m.own_tensors():
+            p = getattr(m, pname)
+            out.append((f"{prefix}mix.{leaf}", p if n is None else p[r : r + n]))
+        out.append((f"{prefix}mix.o", self.out_proj[:, : m.heads * m.vdim]))
+        if self.ff:
+            out += [(f"{prefix}mlp.up", self.in_proj[self.up_off : self.up_off + self.ff]),
+                    (f"{prefix}mlp.down", self.out_proj[:, m.mix_width : m.mix_width + self.ff])]
+        return out
+
+    def forward(self, x, positions, inv_freq, cu_seqlens, max_seqlen):
+        h = self.norm(x)
+        p = _linear(h, self.in_proj)
+        parts = [TF.pad(self.mixer.sequence(p, positions, cu_seqlens), (0, self.mixer.mix_width - self.mixer.heads * self.mixer.vdim))]
+        if self.ff:
+            parts.append(F.plain_act(p[:, self.up_off :].float(), "relu2").to(p.dtype))
+        return x + _linear(torch.cat(parts, dim=1), self.out_proj).float()
+
+
+def _linear(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """The framework's GEMM where its kernels take the shape and type; otherwise the library's."""
+    if x.dtype == torch.bfloat16 and w.shape[0] % 8 == 0 and w.shape[1] % 8 == 0:
+        return F.linear(x, w)
+    return TF.linear(x, w)

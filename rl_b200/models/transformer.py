@@ -520,20 +520,27 @@ class CausalLM(nn.Module):
         else:
             self.embed_tokens = None
         block = HybridBlock if cfg.is_hybrid else DecoderLayer
+        if cfg.is_mixer:
+            from .mixers import DynamicTanh, ParallelBlock as block
+
+            if tpw > 1 or pp_size > 1 or self.cp is not None or (ep is not None and ep.world > 1) or self.lora_cfg or cfg.value_head:
+                raise NotImplementedError("layer-list models run data parallel only, without LoRA or value heads")
         if cfg.is_hybrid and self.tp.sequence_parallel:
             raise NotImplementedError("sequence parallelism is not available for hybrid state-space models")
         self.layers = nn.ModuleList([block(cfg, dtype, device, self.tp, ep, self.cp, self.lora_cfg, layer_idx=self.layer_ids[i])
                                      for i in range(n_local)])
         self.lm_head = None
         if self.last_stage:
-            self.norm = nn.Parameter(torch.ones(d, dtype=dtype, device=device))
+            self.norm = DynamicTanh(d, dtype, device) if cfg.norm_kind == "dyt" else nn.Parameter(torch.ones(d, dtype=dtype, device=device))
             if cfg.value_head:
                 self.score = nn.Parameter(torch.empty(8, d, dtype=dtype, device=device))  # row 0 is the head; 8 rows keep TMA alignment
             elif not tied:
                 self.lm_head = nn.Parameter(torch.empty(self.vocab_local, d, dtype=dtype, device=device))
         else:
             self.norm = None
-        self.register_buffer("inv_freq", rope_inv_freq(cfg, device), persistent=False)
+        # looped layers: one learned vector per pass joins the residual stream when the pass begins
+        self.loop_step = nn.Parameter(torch.zeros(cfg.layer_loop["times"], d, dtype=dtype, device=device)) if cfg.layer_loop else None
+        self.register_buffer("inv_freq", rope_inv_freq(cfg, device) if not cfg.is_mixer else torch.zeros(0, device=device), persistent=False)
         if cfg.rope_local_theta:   # sliding-window layers rotate with their own base and no long-context scaling
             from dataclasses import replace
 
@@ -583,7 +590,7 @@ class CausalLM(nn.Module):
         from .hf_io import iter_hf_shards, hf_full_shape
 
         for name, p in self.named_parameters():
-            if name.endswith("norm") or name.endswith("layernorm"):
+            if name.endswith("norm") or name.endswith("layernorm") or name.endswith("norm.weight"):
                 p.fill_(1.0)
             elif name.endswith("bias"):
                 p.zero_()
@@ -601,6 +608,8 @@ class CausalLM(nn.Module):
             if hf.endswith("norm.weight") or hf.endswith("layernorm.weight") or hf.endswith("norm_f.weight") or hf.endswith(".bias"):
                 continue
             if hf.endswith(".A_log") or hf.endswith(".D") or hf.endswith(".dt_bias"):
+                continue
+            if self.cfg.is_mixer and dst.dim() < 2:   # norms of layer-list models
                 continue
             if hf.endswith("e_score_correction_bias"):
                 dst.zero_()
@@ -695,6 +704,8 @@ class CausalLM(nn.Module):
     def embed(self, batch: PackedBatch) -> torch.Tensor:
         h = self._embed(batch)
         s = self.cfg.embed_scale
+        if self.cfg.is_mixer:      # fp32 residual stream
+            return h.float() * s
         return h if s == 1.0 else h * torch.tensor(s, dtype=h.dtype, device=h.device)   # the scale is rounded to the model dtype first
 
     def _embed(self, batch: PackedBatch) -> torch.Tensor:
@@ -710,7 +721,25 @@ class CausalLM(nn.Module):
             return F.embedding(batch.input_ids[self.cp.local_index(batch.input_ids.numel(), batch.input_ids.device)], self.embed_tokens)
         return F.embedding(batch.input_ids, self.embed_tokens)
 
+    def _run_layer_runs(self, h: torch.Tensor, batch: PackedBatch) -> torch.Tensor:
+        """Layers in the order of ``cfg.layer_runs``. A pass of the loop begins with the embeddings added again (not in the first)
+        and with its step vector added."""
+        e, loop = h, self.cfg.layer_loop
+        for i, t in self.cfg.layer_runs:
+            if t is not None and i == loop["start"]:
+                h = (h + e if t else h) + self.loop_step[t].float()
+            args = (h, batch.positions, None, batch.cu_seqlens, batch.max_seqlen)
+            h = ckpt.checkpoint(self.layers[i], *args, use_reentrant=False) if (self.activation_checkpointing and torch.is_grad_enabled()) else self.layers[i](*args)
+        return h
+
+    def final_norm(self, h: torch.Tensor) -> torch.Tensor:
+        return self.norm(h) if self.cfg.norm_kind == "dyt" else F.rmsnorm(h, self.norm, self.cfg.rms_norm_eps)
+
     def run_layers(self, h: torch.Tensor, batch: PackedBatch) -> torch.Tensor:
+        if self.cfg.is_mixer:
+            if self.sharder is not None or self.capture_layers is not None:
+                raise NotImplementedError("fully sharded parameters and draft heads are not available for layer-list models")
+            return self._run_layer_runs(h, batch)
         inv_freq = self.rope_freqs()
         if self.sharder is not None:
             for i, layer in enumerate(self.layers):
@@ -737,7 +766,7 @@ class CausalLM(nn.Module):
         h = self.run_layers(h, batch)
         if self.sharder is not None:
             return self.sharder.run("head", lambda x: F.rmsnorm(x, self.norm, self.cfg.rms_norm_eps), h)
-        out = F.rmsnorm(h, self.norm, self.cfg.rms_norm_eps) if self.at_output else h
+        out = self.final_norm(h) if self.at_output else h
         if self.capture_layers is not None and self.at_output:
             self.captured["final"] = out
         return out

@@ -73,6 +73,16 @@ def available() -> bool:
     return _LIB_PATH.exists()
 
 
+def stale() -> bool:
+    """True when the library is missing or was built from other sources than those in the tree."""
+    stamp = _LIB_PATH.with_name(_LIB_PATH.name + ".sources")
+    if not _LIB_PATH.exists() or not stamp.exists():
+        return True
+    from rl_b200.tools.fingerprint import source_hash
+
+    return stamp.read_text().strip() != source_hash()
+
+
 def _warn_if_stale() -> None:
     """The build records a hash of the native sources beside the library; when the sources have changed since, say so once
     (``RLB_STRICT_NATIVE=1``: refuse to run). The analogue of the reference's container fingerprint check at import
