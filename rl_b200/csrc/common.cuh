@@ -332,6 +332,59 @@ __device__ __forceinline__ float warp_max(float v) {
   for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
   return v;
 }
+// tanh that keeps its relative accuracy near zero whatever math mode the file is compiled with: the odd Taylor series below 1/4
+// (remainder under 1e-8 relative), 1 - 2 / (1 + exp(2|x|)) above.
+__device__ __forceinline__ float tanh_acc(float x) {
+  const float a = fabsf(x);
+  if (a < 0.25f) {
+    const float q = x * x;
+    return x * (1.f + q * (-1.f / 3.f + q * (2.f / 15.f + q * (-17.f / 315.f + q * (62.f / 2835.f)))));
+  }
+  return copysignf(1.f - 2.f / (1.f + expf(2.f * a)), x);
+}
+
+// Epilogue of the two products of a parallel mixer layer. With `x`: the fp32 residual stream x[row, col] += acc (+ e) (+ step) is
+// updated in place and the output is the dynamic-tanh norm w * tanh(alpha x) + b of the new value. Without: the output is acc,
+// squared ReLU on columns >= act_from.
+struct LayerEpilogue {
+  float* x;
+  long long ldx;             // row stride of x and e
+  const float* e;
+  const __nv_bfloat16* step;
+  const __nv_bfloat16* alpha;
+  const __nv_bfloat16* nw;
+  const __nv_bfloat16* nb;
+  int act_from;
+};
+// Four consecutive columns of one row (col a multiple of 4).
+__device__ __forceinline__ float4 layer_epilogue4(const LayerEpilogue& le, float4 v, long long row, int col, float alpha) {
+  if (le.x) {
+    float4* xp = reinterpret_cast<float4*>(le.x + row * le.ldx + col);
+    const float4 old = *xp;
+    v.x += old.x; v.y += old.y; v.z += old.z; v.w += old.w;
+    if (le.e) {
+      const float4 ev = *reinterpret_cast<const float4*>(le.e + row * le.ldx + col);
+      v.x += ev.x; v.y += ev.y; v.z += ev.z; v.w += ev.w;
+    }
+    if (le.step) {
+      const uint2 sv = *reinterpret_cast<const uint2*>(le.step + col);
+      const float2 s0 = unpack_bf16x2(sv.x), s1 = unpack_bf16x2(sv.y);
+      v.x += s0.x; v.y += s0.y; v.z += s1.x; v.w += s1.y;
+    }
+    *xp = v;
+    const uint2 wv = *reinterpret_cast<const uint2*>(le.nw + col), bv = *reinterpret_cast<const uint2*>(le.nb + col);
+    const float2 w0 = unpack_bf16x2(wv.x), w1 = unpack_bf16x2(wv.y), b0 = unpack_bf16x2(bv.x), b1 = unpack_bf16x2(bv.y);
+    v.x = tanh_acc(alpha * v.x) * w0.x + b0.x;
+    v.y = tanh_acc(alpha * v.y) * w0.y + b0.y;
+    v.z = tanh_acc(alpha * v.z) * w1.x + b1.x;
+    v.w = tanh_acc(alpha * v.w) * w1.y + b1.y;
+  } else if (col >= le.act_from) {   // act_from is a multiple of 8
+    v.x = fmaxf(v.x, 0.f); v.y = fmaxf(v.y, 0.f); v.z = fmaxf(v.z, 0.f); v.w = fmaxf(v.w, 0.f);
+    v.x *= v.x; v.y *= v.y; v.z *= v.z; v.w *= v.w;
+  }
+  return v;
+}
+
 // Block-wide sum; `red` is shared scratch of >= 32 floats. All threads get the result.
 __device__ __forceinline__ float block_sum(float v, float* red) {
   const int lane = threadIdx.x & 31, w = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;

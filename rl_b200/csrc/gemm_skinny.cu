@@ -12,7 +12,7 @@
 //     on HBM for the projections of one layer (N = 4096 would otherwise occupy 16 of the 148 SMs).
 // The epilogue adds an optional bias and residual (the transformer's skip connection) and can emit fp32 (logits).
 //
-// Three optional epilogue fusions remove the small kernels that would otherwise sit between the projections of a decoder
+// Optional epilogue fusions remove the small kernels that would otherwise sit between the projections of a decoder
 // layer (each costs more in launch and dependency latency than in work at 64 tokens):
 //   * RMSNorm on the INPUT, split in two. The kernel that produces the residual stream h (o_proj / down_proj with the
 //     residual add) also writes hw = h * w_norm (the per-channel weight of the NEXT norm) and, per 128-column tile, the
@@ -20,6 +20,8 @@
 //     rstd = rsqrt(sum of the partials / d + eps) in its epilogue: the row scale commutes with the product.
 //   * SwiGLU: for the [gate | up] weight, a tile is 64 gate rows stacked on the 64 matching up rows (two TMA boxes into
 //     one 128-row operand, no re-layout of the weight), and the epilogue writes silu(gate) * up.
+//   * The products of parallel mixer layers (LayerEpilogue in common.cuh): squared ReLU on a column range, or the fp32
+//     residual update followed by the next layer's dynamic-tanh norm.
 //
 // Counterpart in the reference: the cuBLAS / vLLM GEMMs behind every decode-step nn.Linear
 // (nemo_rl/models/generation/vllm/vllm_worker.py:570-597).
@@ -71,6 +73,8 @@ struct SkinnyParams {
   __nv_bfloat16* Y2;
   long long ldy2;
   int swiglu;  // W is [2F, K] = [gate | up]; the output is silu(gate) * up of width F = N
+  int use_layer;
+  LayerEpilogue layer;
 };
 
 __device__ __forceinline__ uint32_t cluster_ctarank() {
@@ -252,6 +256,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
     const int out_cols = p.swiglu ? 64 : SK_BM;      // output columns of this tile
     const int groups = out_cols / 4;                 // work item: (token m, 4 consecutive output columns)
     const int n0 = n_blk * out_cols;
+    const float layer_alpha = p.use_layer && p.layer.x ? __bfloat162float(*p.layer.alpha) : 0.f;
     // a warp always works on one token (groups is 16 or 32, the stride a multiple of 32), so the per-token sum of
     // squares for the next norm is one warp reduction
     const int items = max(m_end - m_begin, 0) * groups;
@@ -292,6 +297,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
           const float2 r0 = unpack_bf16x2(rv.x), r1 = unpack_bf16x2(rv.y);
           acc.x += r0.x; acc.y += r0.y; acc.z += r1.x; acc.w += r1.y;
         }
+        if (p.use_layer) acc = layer_epilogue4(p.layer, acc, m, n, layer_alpha);
         if (p.out_fp32) {
           *reinterpret_cast<float4*>(reinterpret_cast<float*>(p.Y) + static_cast<long long>(m) * p.ldy + n) = acc;
         } else {
@@ -352,6 +358,15 @@ int launch_skinny(const CUtensorMap& tw, const CUtensorMap& tx, const SkinnyPara
   cfg.numAttrs = rlb_pdl_enabled() ? 2 : 1;
   cudaError_t e = cudaLaunchKernelEx(&cfg, kern, tw, tx, p);
   return static_cast<int>(e);
+}
+
+int launch_skinny_nt(int NT, const CUtensorMap& tw, const CUtensorMap& tx, const SkinnyParams& p, int split, cudaStream_t s) {
+  switch (NT) {
+    case 32: return launch_skinny<32>(tw, tx, p, split, s);
+    case 64: return launch_skinny<64>(tw, tx, p, split, s);
+    case 128: return launch_skinny<128>(tw, tx, p, split, s);
+    default: return launch_skinny<256>(tw, tx, p, split, s);
+  }
 }
 
 }  // namespace
@@ -438,15 +453,41 @@ RLB_API int rlb_gemm_skinny_fused(const void* X, const void* W, void* Y, int M, 
   p.Y2 = reinterpret_cast<__nv_bfloat16*>(Y2);
   p.ldy2 = ldy2;
   p.swiglu = swiglu ? 1 : 0;
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
-  switch (NT) {
-    case 32: return launch_skinny<32>(tw, tx, p, split, s);
-    case 64: return launch_skinny<64>(tw, tx, p, split, s);
-    case 128: return launch_skinny<128>(tw, tx, p, split, s);
-    default: return launch_skinny<256>(tw, tx, p, split, s);
-  }
+  p.use_layer = 0;
+  p.layer = LayerEpilogue{};
+  return launch_skinny_nt(NT, tw, tx, p, split, static_cast<cudaStream_t>(stream));
 }
 
+// rlb_gemm_layer for M <= 256 rows on the weight-streaming kernel.
+RLB_API int rlb_gemm_skinny_layer(const void* X, const void* W, void* out, int M, int N, int K, long long ldx_in, long long ldw, long long ldo,
+                                  int act_from, float* x, long long ldx, const float* e, const void* step, const void* alpha,
+                                  const void* nw, const void* nb, int* status, void* stream) {
+  if (M <= 0 || N <= 0 || K <= 0) return 0;
+  if (M > 256) return -7;
+  if ((ldx_in % 8) || (ldw % 8) || (ldo % 8) || (N % 8) || (K % 8) || (act_from % 8) || (ldx % 4)) return -2;
+  if (x && (!alpha || !nw || !nb)) return -2;
+  if ((reinterpret_cast<uintptr_t>(X) | reinterpret_cast<uintptr_t>(W) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(x) |
+       reinterpret_cast<uintptr_t>(e) | reinterpret_cast<uintptr_t>(step) | reinterpret_cast<uintptr_t>(nw) | reinterpret_cast<uintptr_t>(nb)) & 15)
+    return -3;
+  const int NT = M <= 32 ? 32 : (M <= 64 ? 64 : (M <= 128 ? 128 : 256));
+  CUtensorMap tw, tx;
+  int rc = rlb_make_tmap_2d(&tw, W, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, K, N, ldw * 2, SK_BK, SK_BM, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (rc) return -100 - rc;
+  rc = rlb_make_tmap_2d(&tx, X, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, K, M, ldx_in * 2, SK_BK, NT, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (rc) return -100 - rc;
+  SkinnyParams p{};
+  p.Y = out;
+  p.ldy = ldo;
+  p.M = M;
+  p.N = N;
+  p.K = K;
+  p.w_static = g_sk_static_w;
+  p.status = status;
+  p.use_layer = 1;
+  p.layer = LayerEpilogue{x, ldx, e, static_cast<const __nv_bfloat16*>(step), static_cast<const __nv_bfloat16*>(alpha),
+                          static_cast<const __nv_bfloat16*>(nw), static_cast<const __nv_bfloat16*>(nb), act_from};
+  return launch_skinny_nt(NT, tw, tx, p, rlb_gemm_skinny_split(N, K), static_cast<cudaStream_t>(stream));
+}
 RLB_API int rlb_gemm_skinny(const void* X, const void* W, void* Y, int M, int N, int K, long long ldx, long long ldw,
                             long long ldy, int out_fp32, const float* bias, const void* residual, long long ldr,
                             int split, int* status, void* stream) {

@@ -19,6 +19,8 @@
 //   EPI_LOGPROB  for a vocab projection: per (row, n-tile) online-softmax partials (max, sum-exp,
 //                sum of z*exp) and the target logit; logits are never written. A small second
 //                kernel folds the partials into logprob / entropy / logsumexp per row.
+//   EPI_LAYER    products of a parallel mixer layer (LayerEpilogue in common.cuh): squared ReLU on a column range, or
+//                residual update + dynamic-tanh norm
 //   EPI_DLOGITS  recomputes the logits tile and writes coef[row]*(onehot - softmax)*inv_temp in
 //                bf16, the gradient that the dH / dW GEMMs consume.
 // Replaces the cuBLAS calls behind nn.Linear and the chunked hidden->logprob path of the reference
@@ -48,7 +50,7 @@ constexpr int NUM_THREADS = 192;
 constexpr int TMEM_COLS = 512;
 constexpr int GROUP_M = 16;  // rasterisation: 16 m-tiles share each sweep over n
 
-enum { EPI_STORE = 0, EPI_LOGPROB = 1, EPI_DLOGITS = 2 };
+enum { EPI_STORE = 0, EPI_LOGPROB = 1, EPI_DLOGITS = 2, EPI_LAYER = 3 };
 
 struct EpiParams {
   void* C;              // output (EPI_STORE, EPI_DLOGITS)
@@ -69,6 +71,7 @@ struct EpiParams {
   const float* coef;    // [M] upstream gradient of the log-probability (EPI_DLOGITS)
   const float* ent_coef;  // [M] upstream gradient of the entropy, or null (EPI_DLOGITS)
   const float* entropy;   // [M] entropy per row, needed with ent_coef
+  LayerEpilogue layer;    // EPI_LAYER
 };
 
 __device__ __forceinline__ void tile_coords(int tile, int num_m, int num_n, int& m_blk, int& n_blk) {
@@ -295,6 +298,26 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
                 o.w = pack_bf16x2(v[q * 8 + 6], v[q * 8 + 7]);
                 *reinterpret_cast<uint4*>(dst + q * 8) = o;
               }
+            }
+          }
+        }
+      } else if (EPI == EPI_LAYER) {
+        const float alpha = ep.layer.x ? __bfloat162float(*ep.layer.alpha) : 0.f;
+        for (int c = 0; c < BN / 32; ++c) {
+          uint32_t r[32];
+          tmem_ld_32x32b_x32(taddr + c * 32, r);
+          tmem_ld_wait();
+          const int col = col0 + c * 32;
+          if (!row_ok || col >= N) continue;
+          __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(ep.C) + static_cast<long long>(row) * ep.ldc + col;
+#pragma unroll
+          for (int q = 0; q < 4; ++q) {
+            if (col + q * 8 < N) {
+              const float4 a = layer_epilogue4(ep.layer, make_float4(__uint_as_float(r[q * 8]), __uint_as_float(r[q * 8 + 1]),
+                                                                     __uint_as_float(r[q * 8 + 2]), __uint_as_float(r[q * 8 + 3])), row, col + q * 8, alpha);
+              const float4 b = layer_epilogue4(ep.layer, make_float4(__uint_as_float(r[q * 8 + 4]), __uint_as_float(r[q * 8 + 5]),
+                                                                     __uint_as_float(r[q * 8 + 6]), __uint_as_float(r[q * 8 + 7])), row, col + q * 8 + 4, alpha);
+              *reinterpret_cast<uint4*>(dst + q * 8) = make_uint4(pack_bf16x2(a.x, a.y), pack_bf16x2(a.z, a.w), pack_bf16x2(b.x, b.y), pack_bf16x2(b.z, b.w));
             }
           }
         }
@@ -536,6 +559,27 @@ RLB_API int rlb_gemm_bf16(const void* A, const void* B, void* C, int M, int N, i
   ep.accumulate = accumulate;
   return dispatch_layout<EPI_STORE>(a_mn_major != 0, b_mn_major != 0, ta, tb, M, N, K, ep, status, max_ctas,
                                     static_cast<cudaStream_t>(stream));
+}
+
+// out[M, N] (bf16) = epilogue(A W^T) with LayerEpilogue's fields; N, K and all row strides multiples of 8, ldx of 4.
+RLB_API int rlb_gemm_layer(const void* A, const void* W, void* out, int M, int N, int K, long long lda, long long ldw, long long ldo,
+                           int act_from, float* x, long long ldx, const float* e, const void* step, const void* alpha, const void* nw,
+                           const void* nb, int* status, void* stream) {
+  if (M <= 0 || N <= 0 || K <= 0) return 0;
+  if ((lda % 8) || (ldw % 8) || (ldo % 8) || (N % 8) || (K % 8) || (act_from % 8) || (ldx % 4)) return -2;
+  if (x && (!alpha || !nw || !nb)) return -2;
+  if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(x) |
+       reinterpret_cast<uintptr_t>(e) | reinterpret_cast<uintptr_t>(step) | reinterpret_cast<uintptr_t>(nw) | reinterpret_cast<uintptr_t>(nb)) & 15)
+    return -3;
+  CUtensorMap ta, tb;
+  int rc = make_operand_maps(A, W, M, N, K, lda, ldw, false, false, &ta, &tb);
+  if (rc) return -100 - rc;
+  EpiParams ep{};
+  ep.C = out;
+  ep.ldc = ldo;
+  ep.layer = LayerEpilogue{x, ldx, e, static_cast<const __nv_bfloat16*>(step), static_cast<const __nv_bfloat16*>(alpha),
+                           static_cast<const __nv_bfloat16*>(nw), static_cast<const __nv_bfloat16*>(nb), act_from};
+  return launch_gemm<false, false, EPI_LAYER>(ta, tb, M, N, K, ep, status, 0, static_cast<cudaStream_t>(stream));
 }
 
 // Number of n-tiles the vocab-projection epilogues split N into (size of the partial buffers).

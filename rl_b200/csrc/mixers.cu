@@ -139,11 +139,12 @@ struct LatentShape {
   int block_size, num_blocks;
 };
 
-// Per row: latent / rms * w and rotated shared key into the cache row of the token; rotated query parts in place.
+// Per row: latent / rms * w and rotated shared key into the cache row of the token; rotated query parts in place, and for the first
+// `q_rows` rows also behind the latent columns of q_lat [rows, heads, width] (the decode kernels' queries).
 template <typename T>
 __global__ void latent_prep_kernel(T* __restrict__ p, LatentShape s, const int* __restrict__ positions, const long long* __restrict__ slots,
                                    const T* __restrict__ norm_w, const float* __restrict__ freq, int half, float gain, float eps,
-                                   T* __restrict__ cache, int* status) {
+                                   T* __restrict__ cache, T* __restrict__ q_lat, int q_rows, int* status) {
   extern __shared__ float sm[];
   __shared__ float red[32];
   float* cs = sm;              // [half] cosine, then [half] sine
@@ -190,6 +191,14 @@ __global__ void latent_prep_kernel(T* __restrict__ p, LatentShape s, const int* 
     const float c = cs[i % half], sn = cs[half + i % half], u = ld(q), v = ld(q + 1);
     st(q, u * c - v * sn);
     st(q + 1, v * c + u * sn);
+  }
+  if (q_lat && row < q_rows) {
+    __syncthreads();
+    const int tail = s.width - s.rank;
+    for (int i = threadIdx.x; i < s.heads * tail; i += blockDim.x) {
+      const int h = i / tail, j = i % tail;
+      st(q_lat + (row * s.heads + h) * s.width + s.rank + j, j < s.rot_dim ? ld(pr + s.q_off + h * qd + s.dim + j) : 0.f);
+    }
   }
 }
 
@@ -398,7 +407,7 @@ RLB_API int rlb_gemm_rows(const void* a, const void* w, void* out, int M, int N,
 
 RLB_API int rlb_latent_prep(void* p, int f32, long long rows, long long ldp, int q_off, int lat_off, int heads, int dim, int rot_dim, int rank,
                             int width, int block_size, int num_blocks, const int* positions, const long long* slots, const void* norm_w,
-                            const float* freq, int half, float gain, float eps, void* cache, int* status, void* stream) {
+                            const float* freq, int half, float gain, float eps, void* cache, void* q_lat, int q_rows, int* status, void* stream) {
   if (rows <= 0) return 0;
   if (2 * half > rot_dim || rank + rot_dim > width) return -2;
   LatentShape s{ldp, q_off, lat_off, 0, heads, dim, rot_dim, 0, rank, width, block_size, num_blocks};
@@ -406,10 +415,11 @@ RLB_API int rlb_latent_prep(void* p, int f32, long long rows, long long ldp, int
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (f32)
     latent_prep_kernel<float><<<static_cast<unsigned>(rows), 256, sm, st>>>(static_cast<float*>(p), s, positions, slots, static_cast<const float*>(norm_w),
-                                                                            freq, half, gain, eps, static_cast<float*>(cache), status);
+                                                                            freq, half, gain, eps, static_cast<float*>(cache), static_cast<float*>(q_lat), q_rows, status);
   else
     latent_prep_kernel<__nv_bfloat16><<<static_cast<unsigned>(rows), 256, sm, st>>>(static_cast<__nv_bfloat16*>(p), s, positions, slots,
-        static_cast<const __nv_bfloat16*>(norm_w), freq, half, gain, eps, static_cast<__nv_bfloat16*>(cache), status);
+        static_cast<const __nv_bfloat16*>(norm_w), freq, half, gain, eps, static_cast<__nv_bfloat16*>(cache),
+        static_cast<__nv_bfloat16*>(q_lat), q_rows, status);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -567,6 +567,8 @@ class GenerationEngine:
                              if m.kind == "latent_attention" else None for m in mx]
         self.ret_state = [torch.zeros((self.max_running + 1, m.heads, m.dim, m.vdim), dtype=torch.float32, device=dev)
                           if m.kind == "retention" else None for m in mx]
+        # portions of prompts attend tile-wise when every latent-attention layer has a shape the tensor-core kernel takes
+        self._portion_tiles = self.native and all(X.portion_tiles(m, dt) for m in mx if m.kind == "latent_attention")
 
     def sleep(self, free_kv_cache: bool = True) -> None:
         """Ends a generation phase: drops all requests; optionally returns the KV cache memory (captured graphs are
@@ -900,8 +902,19 @@ class GenerationEngine:
         sids = [items[j][0] for j in order]
         bt, _, _ = self.sched.tables(sids, self.max_blocks_per_seq)
         of_row = torch.repeat_interleave(torch.arange(len(lens)), torch.tensor(lens))
-        b = X.TokenBatch(ids=ids, positions=pos.to(dev), slots=torch.cat(slots).to(dev), n_single=n_single, n_paged=len(toks),
-                         block_table=bt[of_row].to(dev), seq_lens=(pos + 1).to(dev), max_ctx=int(pos.max()) + 1)
+        tiled = [j for j, n in enumerate(lens) if n > X.PAGED_PORTION] if self._portion_tiles else []
+        n_paged = sum(lens[: tiled[0]]) if tiled else len(toks)
+        b = X.TokenBatch(ids=ids, positions=pos.to(dev), slots=torch.cat(slots).to(dev), n_single=n_single, n_paged=n_paged,
+                         block_table=bt[of_row[:n_paged]].to(dev), seq_lens=(pos[:n_paged] + 1).to(dev),
+                         max_ctx=int(pos[:n_paged].max()) + 1 if n_paged else 0)
+        if tiled:
+            ctx = [items[order[j]][2] + lens[j] for j in tiled]
+            cu = torch.zeros((2, len(tiled) + 1), dtype=torch.int32)
+            cu[0, 1:] = torch.tensor([lens[j] for j in tiled], dtype=torch.int64).cumsum(0)
+            cu[1, 1:] = torch.tensor(ctx, dtype=torch.int64).cumsum(0)
+            cu = cu.to(dev)
+            b.cu_q, b.cu_ctx, b.q_tiles = cu[0], cu[1], sum(-(-lens[j] // 128) for j in tiled)
+            b.ctx_slots = torch.cat([self.sched.slots(sids[j], 0, n) for j, n in zip(tiled, ctx)]).to(dev)
         if self.stateful:
             b.state_rows = torch.tensor([self._state_row[s] for s in sids], dtype=torch.int64, device=dev)
         if n_single < len(lens):

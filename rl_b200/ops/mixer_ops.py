@@ -17,17 +17,26 @@ from typing import Optional
 
 import torch
 
+from . import functional as F
 from . import lib as _L
 from .lib import F as CF
 from .lib import I, L as LL, P, call, ptr, register, stream_ptr, use_native
 
 register("rlb_embed_rows", [P, I, P, I, P, P, P, P, P, P, P, LL, I, I, CF, P, P])
 register("rlb_gemm_rows", [P, P, P, I, I, I, LL, LL, LL, I, I, I, P, LL, P, P, P, P, P, P])
-register("rlb_latent_prep", [P, I, LL, LL, I, I, I, I, I, I, I, I, I, P, P, P, P, I, CF, CF, P, P, P])
+register("rlb_gemm_layer", [P, P, P, I, I, I, LL, LL, LL, I, P, LL, P, P, P, P, P, P, P])
+register("rlb_gemm_skinny_layer", [P, P, P, I, I, I, LL, LL, LL, I, P, LL, P, P, P, P, P, P, P])
+register("rlb_latent_prep", [P, I, LL, LL, I, I, I, I, I, I, I, I, I, P, P, P, P, I, CF, CF, P, P, I, P, P])
+register("rlb_latent_gather", [P, P, P, LL, I, LL, P, P])
+register("rlb_flash_latent_supported", [I, I, I, I])
+register("rlb_flash_latent", [P, LL, LL, I, I, P, P, LL, I, P, P, I, I, I, I, I, I, I, I, CF, I, P, P])
+register("rlb_latent_decode_supported", [I, I, I, I, I, I])
+register("rlb_latent_decode", [P, I, LL, I, I, I, I, I, I, I, I, I, I, I, P, P, I, P, P, CF, P, P, I, P, P, P, P])
 register("rlb_latent_rows", [P, I, I, LL, I, I, I, I, I, I, I, I, I, I, P, P, I, P, P, CF, P, P])
 register("rlb_retention_rows", [P, I, I, I, LL, I, I, I, I, I, I, I, P, P, P, P, LL, P, P, I, CF, CF, CF, P, P])
 
 NO_ACT = 1 << 30
+PAGED_PORTION = 16   # portions of at most this many tokens attend row by row over the pages (decode kernels)
 
 
 @dataclass
@@ -48,13 +57,12 @@ class TokenBatch:
     seq_lens: torch.Tensor           # int32 [n_paged]
     state_rows: Optional[torch.Tensor] = None   # int64 [sequences]
     cu: Optional[torch.Tensor] = None           # int32
-    max_portion: int = 0
+    max_portion: int = 0             # tokens of the longest portion
     cu_q: Optional[torch.Tensor] = None         # int32
     cu_ctx: Optional[torch.Tensor] = None       # int32
     ctx_slots: Optional[torch.Tensor] = None    # int64
-    max_q: int = 0
+    q_tiles: int = 0                 # 128-row query tiles of those portions
     max_ctx: int = 0                 # upper bound of seq_lens (a host number, fixed while a graph is captured)
-    num_splits: int = 1
 
     @property
     def rows(self) -> int:
@@ -88,10 +96,23 @@ def embed_rows(ids, table, scale: float, step: Optional[torch.Tensor], norm, kee
 
 
 # --------------------------------------------------------------------------------------- products
-def _rows_gemm(a, w, out, act_from=NO_ACT, x=None, e=None, step=None, norm=None):
-    call("rlb_gemm_rows", ptr(a), ptr(w), ptr(out), a.shape[0], w.shape[0], w.shape[1], a.stride(0), w.stride(0), out.stride(0),
-         _f32(a), _f32(out), act_from, ptr(x), x.stride(0) if x is not None else 0, ptr(e), ptr(step),
-         *((ptr(norm.alpha), ptr(norm.weight), ptr(norm.bias)) if norm is not None else (None, None, None)), stream_ptr())
+def _aligned(*ts) -> bool:
+    """bf16 matrices whose rows start on 16-byte boundaries (what TMA can fetch)."""
+    return all(t.dtype == torch.bfloat16 and t.data_ptr() % 16 == 0 and t.stride(0) % 8 == 0 for t in ts)
+
+
+def _product(a, w, out, act_from=NO_ACT, x=None, e=None, step=None, norm=None):
+    """out = epilogue(a w^T): the tensor-core kernels for bf16 shapes that TMA can address, else the plain kernel (any size, fp32)."""
+    M, (N, K) = a.shape[0], w.shape
+    lay = (ptr(x), x.stride(0) if x is not None else 0, ptr(e), ptr(step),
+           *((ptr(norm.alpha), ptr(norm.weight), ptr(norm.bias)) if norm is not None else (None, None, None)))
+    if _aligned(a, w, out) and N % 8 == 0 and K % 8 == 0:
+        name = "rlb_gemm_skinny_layer" if M <= 256 and K >= 256 else "rlb_gemm_layer"
+        call(name, ptr(a), ptr(w), ptr(out), M, N, K, a.stride(0), w.stride(0), out.stride(0), act_from, *lay,
+             ptr(_L.status_word(a.device)), stream_ptr())
+    else:
+        call("rlb_gemm_rows", ptr(a), ptr(w), ptr(out), M, N, K, a.stride(0), w.stride(0), out.stride(0), _f32(a), _f32(out), act_from, *lay,
+             stream_ptr())
     return out
 
 
@@ -102,7 +123,7 @@ def in_proj(h: torch.Tensor, w: torch.Tensor, act_from: int) -> torch.Tensor:
         if act_from < p.shape[1]:
             p[:, act_from:] = torch.relu(p[:, act_from:]).square()
         return p
-    return _rows_gemm(h, w, torch.empty((h.shape[0], w.shape[0]), dtype=h.dtype, device=h.device), act_from)
+    return _product(h, w, torch.empty((h.shape[0], w.shape[0]), dtype=h.dtype, device=h.device), act_from)
 
 
 def out_proj_(x: torch.Tensor, a: torch.Tensor, w: torch.Tensor, e: Optional[torch.Tensor], step: Optional[torch.Tensor], norm) -> torch.Tensor:
@@ -114,13 +135,15 @@ def out_proj_(x: torch.Tensor, a: torch.Tensor, w: torch.Tensor, e: Optional[tor
         if step is not None:
             x += step.float()
         return _dyt_ref(x, norm)
-    return _rows_gemm(a, w, torch.empty((a.shape[0], w.shape[0]), dtype=a.dtype, device=a.device), NO_ACT, x, e, step, norm)
+    return _product(a, w, torch.empty((a.shape[0], w.shape[0]), dtype=a.dtype, device=a.device), NO_ACT, x, e, step, norm)
 
 
 def logits(h: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype = torch.float32) -> torch.Tensor:
     if not use_native(h):
         return (h.float() @ w.float().t()).to(out_dtype)
-    return _rows_gemm(h, w, torch.empty((h.shape[0], w.shape[0]), dtype=out_dtype, device=h.device))
+    if _aligned(h, w) and w.shape[0] % 8 == 0 and w.shape[1] % 8 == 0:
+        return F.gemm(h, w, out_dtype=out_dtype)
+    return _product(h, w, torch.empty((h.shape[0], w.shape[0]), dtype=out_dtype, device=h.device))
 
 
 # --------------------------------------------------------------------------------------- latent attention
@@ -155,12 +178,53 @@ def latent_attention_(p: torch.Tensor, m, b: TokenBatch, cache: torch.Tensor) ->
             y = torch.einsum("hr,hvr->hv", w @ c[:, : m.rank], uv).reshape(-1)
             g.copy_((y * torch.sigmoid(g.float())).to(p.dtype))
         return
-    st = ptr(_L.status_word(p.device))
-    call("rlb_latent_prep", ptr(p), _f32(p), p.shape[0], p.stride(0), m.q_off, m.lat_off, m.heads, m.dim, m.rot_dim, m.rank, m.latent_width, bs,
-         cache.shape[0], ptr(b.positions), ptr(b.slots), ptr(m.kv_norm), ptr(m.freq), m.freq.numel(), float(m.gain), float(m.eps), ptr(cache), st,
-         stream_ptr())
-    call("rlb_latent_rows", ptr(p), _f32(p), b.n_paged, p.stride(0), m.q_off, m.mix_off, m.heads, m.dim, m.rot_dim, m.vdim, m.rank, m.latent_width,
-         bs, cache.shape[0], ptr(cache), ptr(b.block_table), b.block_table.stride(0), ptr(b.seq_lens), ptr(m.kv_up), float(m.scale), st, stream_ptr())
+    dev, T, H, W = p.device, p.shape[0], m.heads, m.latent_width
+    st = ptr(_L.status_word(dev))
+    decode = b.n_paged > 0 and decode_tiles(p, m, bs)
+    q_lat = torch.empty((b.n_paged, H, W), dtype=p.dtype, device=dev) if decode else None
+    call("rlb_latent_prep", ptr(p), _f32(p), T, p.stride(0), m.q_off, m.lat_off, H, m.dim, m.rot_dim, m.rank, W, bs, cache.shape[0], ptr(b.positions),
+         ptr(b.slots), ptr(m.kv_norm), ptr(m.freq), m.freq.numel(), float(m.gain), float(m.eps), ptr(cache), ptr(q_lat),
+         b.n_paged if decode else 0, st, stream_ptr())
+    if decode:
+        splits = split_count(b.n_paged * -(-H // (32 if H > 16 else 16)), b.max_ctx)
+        o_lat = torch.empty((b.n_paged, H * m.rank), dtype=p.dtype, device=dev)
+        po = torch.empty(b.n_paged * H * splits * m.rank, dtype=torch.float32, device=dev) if splits > 1 else None
+        pml = torch.empty(b.n_paged * H * splits * 2, dtype=torch.float32, device=dev) if splits > 1 else None
+        call("rlb_latent_decode", ptr(p), b.n_paged, p.stride(0), p.shape[1], m.q_off, m.mix_off, H, m.dim, m.rot_dim, m.vdim, m.rank, W, bs,
+             cache.shape[0], ptr(cache), ptr(b.block_table), b.block_table.stride(0), ptr(b.seq_lens), ptr(m.kv_up), float(m.scale), ptr(q_lat),
+             ptr(o_lat), splits, ptr(po), ptr(pml), st, stream_ptr())
+    elif b.n_paged:
+        call("rlb_latent_rows", ptr(p), _f32(p), b.n_paged, p.stride(0), m.q_off, m.mix_off, H, m.dim, m.rot_dim, m.vdim, m.rank, W, bs,
+             cache.shape[0], ptr(cache), ptr(b.block_table), b.block_table.stride(0), ptr(b.seq_lens), ptr(m.kv_up), float(m.scale), st, stream_ptr())
+    if b.n_paged < T:
+        n = b.ctx_slots.numel()
+        lat = torch.empty((n, W), dtype=p.dtype, device=dev)
+        call("rlb_latent_gather", ptr(cache), ptr(b.ctx_slots), ptr(lat), n, W, cache.shape[0] * bs, st, stream_ptr())
+        kv = F.gemm(lat[:, : m.rank], m.kv_up)
+        call("rlb_flash_latent", ptr(p), T, p.stride(0), p.shape[1], b.n_paged, ptr(kv), ptr(lat), n, W, ptr(b.cu_q), ptr(b.cu_ctx),
+             b.cu_q.numel() - 1, H, m.dim, m.rot_dim, m.vdim, m.rank, m.q_off, m.mix_off, float(m.scale), b.q_tiles, st, stream_ptr())
+
+
+def decode_tiles(p: torch.Tensor, m, block_size: int) -> bool:
+    """Whether the tensor-core decode kernels take this layer's shape."""
+    return p.dtype == torch.bfloat16 and (m.dim + m.rot_dim) % 8 == 0 and \
+        bool(_L.lib().rlb_latent_decode_supported(m.dim, m.rot_dim, m.vdim, m.rank, m.latent_width, block_size))
+
+
+def portion_tiles(m, dtype: torch.dtype) -> bool:
+    """Whether the tensor-core prefill kernel takes this layer's shape."""
+    return dtype == torch.bfloat16 and (m.dim + m.rot_dim) % 8 == 0 and (m.heads * (m.dim + m.vdim)) % 8 == 0 and \
+        bool(_L.lib().rlb_flash_latent_supported(m.dim, m.rot_dim, m.vdim, m.rank))
+
+
+def split_count(ctas: int, max_ctx: int, sms: int = 148) -> int:
+    """Context splits of the decode attention (one CTA per SM): the count whose waves waste least, at least 256 tokens per split."""
+    best, cost = 1, float("inf")
+    for s in range(1, min(32, max(1, max_ctx // 256)) + 1):
+        c = -(-ctas * s // sms) / s + 0.01 * s
+        if c < cost - 1e-9:
+            best, cost = s, c
+    return best
 
 
 # --------------------------------------------------------------------------------------- retention
