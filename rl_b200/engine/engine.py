@@ -920,7 +920,8 @@ class GenerationEngine:
         if n_single < len(lens):
             cu = torch.zeros(len(lens) - n_single + 1, dtype=torch.int32)
             cu[1:] = torch.tensor(lens[n_single:], dtype=torch.int64).cumsum(0)
-            b.cu, b.max_portion = cu.to(dev), lens[-1]
+            b.cu = cu.to(dev)
+            b.piece_chunk, b.chunk_row, b.chunk_rows = (t.to(dev) for t in X.chunk_lists(lens[n_single:]))
         return b, first
 
     @torch.no_grad()

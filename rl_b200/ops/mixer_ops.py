@@ -34,9 +34,25 @@ register("rlb_latent_decode_supported", [I, I, I, I, I, I])
 register("rlb_latent_decode", [P, I, LL, I, I, I, I, I, I, I, I, I, I, I, P, P, I, P, P, CF, P, P, I, P, P, P, P])
 register("rlb_latent_rows", [P, I, I, LL, I, I, I, I, I, I, I, I, I, I, P, P, I, P, P, CF, P, P])
 register("rlb_retention_rows", [P, I, I, I, LL, I, I, I, I, I, I, I, P, P, P, P, LL, P, P, I, CF, CF, CF, P, P])
+register("rlb_retention_supported", [I, I])
+register("rlb_retention_step", [P, I, LL, I, I, I, I, I, I, I, P, P, P, LL, P, P, I, CF, CF, CF, P, P])
+register("rlb_retention_portions", [P, LL, LL, I, I, I, I, I, I, I, I, I, I, I, P, P, P, P, P, P, LL, P, P, I, CF, CF, CF, P, P, P, P])
 
 NO_ACT = 1 << 30
+CHUNK = 128          # rows per chunk of the chunked recurrences
 PAGED_PORTION = 16   # portions of at most this many tokens attend row by row over the pages (decode kernels)
+
+
+def chunk_lists(lens) -> tuple:
+    """(piece_chunk, chunk_row, chunk_rows) int32 of portions of ``lens`` rows that stand one after another."""
+    first, row, rows, at = [0], [], [], 0
+    for n in lens:
+        for c in range(0, n, CHUNK):
+            row.append(at + c)
+            rows.append(min(CHUNK, n - c))
+        at += n
+        first.append(len(row))
+    return tuple(torch.tensor(x, dtype=torch.int32) for x in (first, row, rows))
 
 
 @dataclass
@@ -57,7 +73,9 @@ class TokenBatch:
     seq_lens: torch.Tensor           # int32 [n_paged]
     state_rows: Optional[torch.Tensor] = None   # int64 [sequences]
     cu: Optional[torch.Tensor] = None           # int32
-    max_portion: int = 0             # tokens of the longest portion
+    piece_chunk: Optional[torch.Tensor] = None  # int32 [n + 1]: chunks (of at most CHUNK rows) of every portion
+    chunk_row: Optional[torch.Tensor] = None    # int32: first row of every chunk, counted from n_single
+    chunk_rows: Optional[torch.Tensor] = None   # int32
     cu_q: Optional[torch.Tensor] = None         # int32
     cu_ctx: Optional[torch.Tensor] = None       # int32
     ctx_slots: Optional[torch.Tensor] = None    # int64
@@ -248,6 +266,20 @@ def retention_(p: torch.Tensor, m, b: TokenBatch, state: torch.Tensor) -> None:
              ptr(b.positions), ptr(rows), ptr(state), state.shape[0], ptr(m.decay), ptr(m.freq), m.freq.numel(), float(m.gain), m.dim ** -0.5,
              float(m.eps), st, stream_ptr())
 
+    if p.dtype == torch.bfloat16 and _L.lib().rlb_retention_supported(m.dim, m.vdim):
+        if b.n_single:
+            call("rlb_retention_step", ptr(p), b.n_single, p.stride(0), m.q_off, m.k_off, m.v_off, m.mix_off, m.heads, m.dim, m.vdim, ptr(b.positions),
+                 ptr(b.state_rows), ptr(state), state.shape[0], ptr(m.decay), ptr(m.freq), m.freq.numel(), float(m.gain), m.dim ** -0.5, float(m.eps),
+                 st, stream_ptr())
+        if b.cu is not None:
+            n = b.chunk_row.numel()
+            cs = torch.empty((p.shape[0] - b.n_single) * 2 * m.freq.numel() + 4, dtype=torch.float32, device=p.device)
+            sums = torch.empty((n, m.heads, m.dim, m.vdim), dtype=torch.float32, device=p.device)
+            call("rlb_retention_portions", ptr(p), p.shape[0], p.stride(0), p.shape[1], b.n_single, m.q_off, m.k_off, m.v_off, m.mix_off, m.heads, m.dim,
+                 m.vdim, b.cu.numel() - 1, n, ptr(b.piece_chunk), ptr(b.chunk_row), ptr(b.chunk_rows), ptr(b.positions),
+                 ptr(b.state_rows[b.n_single :]), ptr(state), state.shape[0], ptr(m.log2_decay), ptr(m.freq), m.freq.numel(), float(m.gain),
+                 m.dim ** -0.5, float(m.eps), ptr(cs), ptr(sums), st, stream_ptr())
+        return
     if b.n_single:
         run(0, b.n_single, None, b.state_rows)
     if b.cu is not None:
