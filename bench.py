@@ -3,6 +3,7 @@
     python bench.py --gpus N --steps K --warmup W            (N > 1: launched once per GPU by torch.distributed.run)
     python bench.py --config qwen3-32b-tp4dp2 --gpus 8 ...   (other model / layout configurations, see CONFIGS)
     python bench.py --config refit-sweep --gpus 8            (weight re-shard times, trainer layout -> serving layouts)
+    python bench.py --config gadarax-serving                 (prefill / decode of a layer-list model beside Llama at equal size)
     python bench.py --impl reference ...                     (the unmodified reference, when it can be installed)
 
 Default (headline) configuration ``llama8b-dp``: one GRPO step (generation + refit + log-probabilities + training) on
@@ -47,6 +48,7 @@ CONFIGS = {
     "qwen3-30b-a3b-ep8": dict(model="qwen3-30b-a3b", tp=1, ep=0, gen_tp=0, prompts_per_gpu=4, generations=8, prompt_len=512, max_new_tokens=2048,
                               train_mb_tokens=8192, logprob_mb_tokens=16384, act_ckpt="on"),
     "refit-sweep": dict(),
+    "gadarax-serving": dict(),
 }
 
 
@@ -168,6 +170,17 @@ def main() -> int:
         from rl_b200.refit.bench_refit import sweep_main
 
         return sweep_main(steps=args.steps, warmup=args.warmup)
+
+    if args.config == "gadarax-serving":
+        from rl_b200.csrc.build import build_all
+        from rl_b200.engine.bench_mixers import main as serving_main
+        from rl_b200.ops import lib as L
+
+        if not L.available():
+            build_all()
+        sampler = ClockSampler(0)
+        sampler.start()
+        return serving_main(steps=args.steps, warmup=args.warmup, clocks=sampler.stop)
 
     import torch
     import torch.distributed as dist

@@ -1,0 +1,308 @@
+"""Serving throughput of layer-list models (Gadarax) beside the Llama architecture at equal size, and the kernels' distance from
+their rooflines beside the like kernels of the Llama path.
+
+    python bench.py --config gadarax-serving [--steps K --warmup W]
+
+Random weights, random prompts. Whole-model figures come from ``GenerationEngine``: prefill of packed prompts (device time of the
+forward pass) and decoding through the captured step (device time of the graph replays). Kernel figures are CUDA-event times of a
+captured graph that runs the operator over buffer sets larger than L2 together.
+"""
+
+from __future__ import annotations
+
+import json
+import math
+import os
+
+import torch
+
+from rl_b200.engine.engine import GenerationEngine, SamplingParams
+from rl_b200.models.config import ModelConfig, preset
+from rl_b200.models.transformer import build_model
+from rl_b200.ops import engine_ops as E
+from rl_b200.ops import functional as F
+from rl_b200.ops import lib as L
+from rl_b200.ops import mixer_ops as X
+
+SIZES = {   # (preset, Llama twin: same width and run count, MHA with 128-wide heads, MLP sized to equal weights per layer run)
+    "gadarax-1b": dict(hidden_size=2048, num_attention_heads=16),
+    "gadarax-4b": dict(hidden_size=4096, num_attention_heads=32),
+}
+PREFILL = ((1, 4096), (8, 1024))      # (prompts, tokens each)
+DECODE = ((16, 4096), (64, 2048))     # (sequences, context)
+
+
+def llama_twin(name: str) -> ModelConfig:
+    """Llama-architecture model of the same width, the same number of layer runs and the same weight bytes streamed per token."""
+    c = preset(name)
+    base = SIZES[name]
+    d, runs = c.hidden_size, c.layer_runs
+    per_run = []
+    for i, _ in runs:
+        m, ff = c.mixers[i]["mixer"], c.mixers[i]["mlp"]["ff"]
+        H, kd, vd = m["heads"], m["dim"], m["vdim"]
+        if c.mixers[i]["type"] == "latent_attention":
+            per_run.append(d * (H * (kd + m["rot_dim"]) + m["kv_rank"] + m["rot_dim"] + 2 * H * vd) + H * (kd + vd) * m["kv_rank"] + 2 * d * ff)
+        else:
+            per_run.append(d * (2 * H * kd + 3 * H * vd) + 2 * d * ff)
+    mean = sum(per_run) / len(per_run)
+    ff = round((mean - 4 * d * d) / (3 * d) / 128) * 128
+    return ModelConfig(model_type="llama", vocab_size=c.vocab_size, intermediate_size=ff, num_hidden_layers=len(runs), head_dim=128,
+                       num_key_value_heads=base["num_attention_heads"], rms_norm_eps=1e-5, rope_theta=500000.0, tie_word_embeddings=True, **base)
+
+
+def timed(fn, steps: int, warmup: int) -> float:
+    """Mean ms per call, CUDA events around ``steps`` calls after ``warmup``."""
+    for _ in range(warmup):
+        fn()
+    torch.cuda.synchronize()
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    a.record()
+    for _ in range(steps):
+        fn()
+    b.record()
+    torch.cuda.synchronize()
+    return a.elapsed_time(b) / steps
+
+
+def timed_graph(fns, steps: int = 5, warmup: int = 3) -> float:
+    """Mean ms per operator call: ``fns`` (the operator over different buffers, together larger than L2) captured one after another."""
+    side = torch.cuda.Stream()
+    side.wait_stream(torch.cuda.current_stream())
+    with torch.cuda.stream(side):
+        for f in fns:
+            f()
+    torch.cuda.current_stream().wait_stream(side)
+    torch.cuda.synchronize()
+    g = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(g):
+        for f in fns:
+            f()
+    return timed(g.replay, steps, warmup) / len(fns)
+
+
+def engine_for(cfg: ModelConfig, tokens: int, seqs: int, max_len: int):
+    model = build_model(cfg, device="cuda", dtype=torch.bfloat16, seed=0)
+    return GenerationEngine(model, block_size=64, num_blocks=tokens // 64 + 2 * seqs + 2, max_running=seqs, max_model_len=max_len, max_prefill_tokens=16384,
+                            enable_prefix_caching=False)
+
+
+def prefill_ms(eng, n: int, length: int, steps: int, warmup: int) -> float:
+    g = torch.Generator().manual_seed(1)
+    eng.wake()
+    items = []
+    for j in range(n):
+        toks = torch.randint(0, eng.cfg.vocab_size, (length,), generator=g).tolist()
+        eng.sched.open(j)
+        eng.sched.extend(j, length)
+        if eng.stateful:
+            eng._state_row[j] = eng._free_rows.pop()
+        items.append((j, toks, 0, length))
+    if eng.mixer:     # the forward pass alone: batch tensors are built once
+        b, _ = eng._token_batch([(sid, t, 0) for sid, t, _, _ in items])
+        rows = torch.arange(1, n + 1, device="cuda") * length - 1
+        ms = timed(lambda: eng._mixer_forward(b, rows), steps, warmup)
+    else:
+        from rl_b200.models.transformer import PackedBatch
+
+        ids = torch.tensor([t for _, ts, _, _ in items for t in ts], dtype=torch.int32, device="cuda")
+        cu = torch.arange(0, n + 1, dtype=torch.int32, device="cuda") * length
+        batch = PackedBatch(ids, torch.arange(length, dtype=torch.int32, device="cuda").repeat(n), cu, length)
+        slots = torch.cat([eng.sched.slots(j, 0, length) for j in range(n)]).cuda()
+        ms = timed(lambda: eng._prefill_forward(batch, slots, (cu[1:] - 1).long()), steps, warmup)
+    for j in range(n):
+        eng.sched.close(j)
+        if eng.stateful:
+            eng._free_rows.append(eng._state_row.pop(j))
+    return ms
+
+
+def decode_ms(eng, n: int, ctx: int, steps: int, warmup: int) -> float:
+    """Device time of one captured decode step (forward, sampling, advance) at about ``ctx`` cached tokens per sequence."""
+    eng.wake()
+    st = eng._static_buffers()
+    B = eng._bucket(n)
+    eng._n_stop = 0
+    per = ctx // 64
+    perm = torch.randperm(eng.num_blocks)[: n * per].to(torch.int32)
+    st["block_table"].zero_()
+    st["block_table"][:n, :per] = perm.view(n, per).cuda()
+    st["win_step"].zero_()
+    st["active"].fill_(0)
+    st["state_rows"][:n] = torch.arange(1, n + 1, device="cuda")
+    sp = SamplingParams(greedy=True, max_new_tokens=1)
+
+    def reset():     # the same step every time: the last token of each sequence
+        st["ids"][:n] = 5
+        st["positions"][:n] = ctx - 1
+        st["seq_lens"][:n] = ctx
+        st["slots"][:n] = (st["block_table"][:n, per - 1].long() * 64 + 63)
+
+    prev = E.skinny_static_weights(True)
+    splits = E.choose_splits(B, eng.hkv, max(eng.max_model_len // 2, 1), 64, eng._sm_count)
+    no, nml = E.decode_scratch_sizes(B, eng.hq, splits, eng.cfg.head_dim)
+    scratch = (torch.empty(no, dtype=torch.float32, device="cuda"), torch.empty(nml, dtype=torch.float32, device="cuda")) if splits > 1 else None
+    reset()
+    with torch.no_grad():
+        ms = timed_graph([lambda: eng._decode_body(st, B, sp, splits, scratch)], max(steps, 10), warmup)
+    E.skinny_static_weights(bool(prev))
+    return ms
+
+
+def peaks() -> dict:
+    path = os.path.join(os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__)))), "MEASURED_PEAKS.json")
+    try:
+        p = json.load(open(path))
+        return dict(hbm=p["hbm_gbs"] * 1e9, flops=p["bf16_tflops"] * 1e12, of="measured")
+    except OSError:
+        return dict(hbm=6.65e12, flops=1.59e15, of="fallback")
+
+
+def kernel_table(name: str) -> list:
+    """[(kernel, ms, roofline ms, fraction of roofline)] of the operators at the preset's sizes, each followed by the like kernel of the
+    Llama path (marked 'like:')."""
+    pk = peaks()
+    c = preset(name)
+    model = build_model(c, device="cuda", dtype=torch.bfloat16, seed=0)
+    att = next(l for l in model.layers if l.mixer.kind == "latent_attention")
+    ret = next(l for l in model.layers if l.mixer.kind == "retention")
+    d = c.hidden_size
+    dev, bf = "cuda", torch.bfloat16
+    out = []
+
+    def add(label, ms, flops=0.0, nbytes=0.0):
+        roof = max(flops / pk["flops"], nbytes / pk["hbm"]) * 1e3
+        out.append(dict(kernel=label, ms=round(ms, 4), roofline_ms=round(roof, 4), fraction=round(roof / ms, 3)))
+
+    def copies(make, nbytes):
+        return [make() for _ in range(max(2, min(24, math.ceil(200e6 / max(1, nbytes)))))]
+
+    def rows_batch(n, ctx):
+        pages = ctx // 64
+        bt = torch.arange(n * pages, dtype=torch.int32, device=dev).view(n, pages)
+        pos = torch.full((n,), ctx - 1, dtype=torch.int32, device=dev)
+        return X.TokenBatch(ids=None, positions=pos, slots=bt[:, -1].long() * 64 + 63, n_single=n, n_paged=n, block_table=bt,
+                            seq_lens=pos + 1, state_rows=torch.arange(n, device=dev), max_ctx=ctx)
+
+    def portion_batch(n, length):
+        T, pages = n * length, length // 64
+        cu = torch.arange(n + 1, dtype=torch.int32, device=dev) * length
+        slots = torch.arange(T, device=dev)
+        pos = torch.arange(length, dtype=torch.int32, device=dev).repeat(n)
+        pc, cr, cn = (t.to(dev) for t in X.chunk_lists([length] * n))
+        bt = torch.zeros((0, pages), dtype=torch.int32, device=dev)
+        return X.TokenBatch(ids=None, positions=pos, slots=slots, n_single=0, n_paged=0, block_table=bt, seq_lens=pos[:0],
+                            state_rows=torch.arange(n, device=dev), cu=cu, piece_chunk=pc, chunk_row=cr, chunk_rows=cn, cu_q=cu, cu_ctx=cu,
+                            ctx_slots=slots, q_tiles=n * -(-length // 128))
+
+    with torch.no_grad():
+        # products (decode and prefill rows)
+        for T in (64, 4096):
+            for label, layer in (("in_proj attention layer", att), ("out_proj attention layer", att)):
+                w = layer.in_proj if label.startswith("in") else layer.out_proj
+                N, K = w.shape
+                nb = 2 * (N * K + T * (N + K)) + (8 * T * N if label.startswith("out") else 0)
+                sets = copies(lambda: (torch.randn(T, K, device=dev).to(bf), w.detach().clone(), torch.randn(T, N, device=dev) if label.startswith("out") else None), nb)
+                if label.startswith("in"):
+                    ms = timed_graph([lambda s=s: X.in_proj(s[0], s[1], layer.up_off) for s in sets])
+                else:
+                    ms = timed_graph([lambda s=s: X.out_proj_(s[2], s[0], s[1], None, None, layer.norm) for s in sets])
+                add(f"{label}, {T} rows", ms, 2.0 * T * N * K, nb)
+                plain = timed_graph([lambda s=s: F.gemm(s[0], s[1]) for s in sets])
+                add(f"like: plain GEMM, {T} rows", plain, 2.0 * T * N * K, 2 * (N * K + T * (N + K)))
+                del sets
+        # decode attention
+        m = att.mixer
+        for n, ctx in DECODE:
+            b = rows_batch(n, ctx)
+            nb = n * ctx * m.latent_width * 2 + m.kv_up.numel() * 2
+            sets = copies(lambda: (torch.randn(n, att.in_width, device=dev).to(bf), torch.randn(n * ctx // 64, 64, m.latent_width, device=dev).to(bf)), nb)
+            add(f"latent attention decode (all kernels), {n} x {ctx}", timed_graph([lambda s=s: X.latent_attention_(s[0], m, b, s[1]) for s in sets]),
+                2.0 * n * ctx * m.heads * (2 * m.rank + m.rot_dim), nb)
+            del sets
+            H = m.heads
+            nb = n * ctx * H * 128 * 2 * 2
+            sets = copies(lambda: (torch.randn(n, 3 * H * 128, device=dev).to(bf), torch.randn(n * ctx // 64, H, 64, 128, device=dev).to(bf),
+                                   torch.randn(n * ctx // 64, H, 64, 128, device=dev).to(bf)), nb)
+            sp = E.choose_splits(n, H, ctx // 2, 64)
+            add(f"like: paged decode attention, {n} x {ctx}", timed_graph([lambda s=s: E.paged_decode(s[0], s[1], s[2], b.block_table, b.seq_lens, H, H, 128,
+                                                                                                   num_splits=sp) for s in sets]), 4.0 * n * ctx * H * 128, nb)
+            del sets
+        # prefill attention
+        for n, length in PREFILL:
+            b = portion_batch(n, length)
+            T = n * length
+            pairs = n * length * length / 2
+            cache = torch.zeros((T // 64, 64, m.latent_width), dtype=bf, device=dev)
+            nb = 2 * T * (att.in_width + 2 * m.heads * (m.dim + m.vdim))
+            sets = copies(lambda: torch.randn(T, att.in_width, device=dev).to(bf), nb)
+            fl = 2.0 * pairs * m.heads * (m.dim + m.rot_dim + m.vdim) + 2.0 * T * m.kv_up.numel()
+            add(f"latent attention prefill (all kernels), {n} x {length}", timed_graph([lambda s=s: X.latent_attention_(s, m, b, cache) for s in sets]), fl, nb)
+            H = m.heads
+            sets = copies(lambda: torch.randn(T, 3 * H * 128, device=dev).to(bf), nb)
+            add(f"like: flash attention, {n} x {length}", timed_graph([lambda s=s: F.attention_varlen(s, b.cu_q, length, H, H, 128) for s in sets]),
+                4.0 * pairs * H * 128, 2 * T * 4 * H * 128)
+            del sets
+        # retention
+        r = ret.mixer
+        for n, _ in DECODE:
+            b = rows_batch(n, 64)
+            nb = n * r.heads * r.dim * r.vdim * 8
+            sets = copies(lambda: (torch.randn(n, ret.in_width, device=dev).to(bf), torch.randn(n, r.heads, r.dim, r.vdim, device=dev)), nb)
+            add(f"retention decode, {n} rows", timed_graph([lambda s=s: X.retention_(s[0], r, b, s[1]) for s in sets]), 0.0, nb)
+            del sets
+        for n, length in PREFILL:
+            b = portion_batch(n, length)
+            T, C = n * length, X.CHUNK
+            S = torch.zeros((n, r.heads, r.dim, r.vdim), device=dev)
+            nb = 2 * T * r.heads * (3 * r.dim + 3 * r.vdim) + (T // C) * r.heads * r.dim * r.vdim * 16
+            fl = 2.0 * T * r.heads * (C / 2 * (r.dim + r.vdim) + 2 * r.dim * r.vdim)
+            sets = copies(lambda: torch.randn(T, ret.in_width, device=dev).to(bf), 2 * T * ret.in_width)
+            add(f"retention prefill (all kernels), {n} x {length}", timed_graph([lambda s=s: X.retention_(s, r, b, S) for s in sets]), fl, nb)
+            del sets
+        mc = ModelConfig(model_type="nemotron_h", vocab_size=64, hidden_size=d, intermediate_size=64, num_hidden_layers=1, layers_block_type=["mamba"],
+                         num_attention_heads=1, num_key_value_heads=1, head_dim=64, use_rope=False, mlp_gated=False, mamba_num_heads=r.heads,
+                         mamba_head_dim=r.vdim, ssm_state_size=r.dim, mamba_n_groups=r.heads, mamba_chunk_size=128)
+        from rl_b200.models.mamba import ssd_scan, ssd_step
+
+        A = -torch.rand(r.heads, device=dev)
+        n, length = PREFILL[1]
+        x, dt = torch.randn(n, length, r.heads, r.vdim, device=dev), torch.rand(n, length, r.heads, device=dev) * 0.1
+        Bm, Cm = torch.randn(n, length, r.heads, r.dim, device=dev), torch.randn(n, length, r.heads, r.dim, device=dev)
+        T = n * length
+        add(f"like: Mamba-2 scan, {n} x {length}", timed(lambda: ssd_scan(x, dt, A, Bm, Cm, 128), 3, 2), 2.0 * T * r.heads * (64 * (r.dim + r.vdim) + 2 * r.dim * r.vdim),
+            4 * T * r.heads * (2 * r.dim + 2 * r.vdim) + (T // 128) * r.heads * r.dim * r.vdim * 16)
+        n = DECODE[1][0]
+        S = torch.randn(n, r.heads, r.vdim, r.dim, device=dev)
+        add(f"like: Mamba-2 step, {n} rows", timed(lambda: ssd_step(x[:1, :n].transpose(0, 1)[:, 0], dt[0, :n], A, Bm[0, :n], Cm[0, :n], S), 5, 3), 0.0, S.numel() * 8)
+        del mc
+    return out
+
+
+def main(steps: int = 5, warmup: int = 3, sizes=None, clocks=None) -> int:
+    torch.backends.cuda.matmul.allow_tf32 = False
+    L.lib()
+    res = dict(metric="layer-list model serving (device time)", unit="tokens/s", dtype="bf16", data="synthetic (random weights and tokens)", models={}, kernels={})
+    for name in sizes or SIZES:
+        for kind in ("gadarax", "llama"):
+            cfg = preset(name) if kind == "gadarax" else llama_twin(name)
+            row = dict(weights_gb=round(2e-9 * cfg.num_parameters(), 2), runs=len(cfg.layer_runs))
+            need = max(max(n * c for n, c in DECODE), max(n * c for n, c in PREFILL))
+            eng = engine_for(cfg, need, max(n for n, _ in DECODE), max(c for _, c in DECODE) + 64)
+            for n, length in PREFILL:
+                ms = prefill_ms(eng, n, length, steps, warmup)
+                row[f"prefill {n}x{length}"] = dict(ms=round(ms, 3), tokens_per_s=round(n * length / ms * 1e3))
+            for n, ctx in DECODE:
+                ms = decode_ms(eng, n, ctx, steps, warmup)
+                row[f"decode {n}x{ctx}"] = dict(ms=round(ms, 3), tokens_per_s=round(n / ms * 1e3))
+            res["models"][f"{name}:{kind}"] = row
+            eng.sleep(True)
+            del eng
+            torch.cuda.empty_cache()
+        res["kernels"][name] = kernel_table(name)
+        torch.cuda.empty_cache()
+    res["status"] = L.check_status()
+    if clocks is not None:
+        res["clocks"] = clocks()
+    print(json.dumps(res), flush=True)
+    return 0

@@ -450,7 +450,27 @@ def rotary_table(rot: dict) -> tuple[torch.Tensor, float]:
     return (f / factor * ramp + f * (1 - ramp)).float(), 0.1 * math.log(factor) + 1.0
 
 
+def _layer_list(width: int, ff: int, latent: dict, retention: dict, kinds: str, loop: Optional[dict], vocab: int) -> dict:
+    """Preset of a layer-list model: ``kinds`` has one letter per layer (A latent attention, R retention)."""
+    rot = {"dims": latent["rot_dim"], "base": 500000.0, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}
+    att = dict(latent, scale=(latent["dim"] + latent["rot_dim"]) ** -0.5, rot=rot)
+    ret = dict(retention, rot={"dims": retention["dim"], "base": 10000.0},
+               decay=[1.0 - 2.0 ** -(5 + 7 * i / max(1, retention["heads"] - 1)) for i in range(retention["heads"])])
+    layers = [{"type": "latent_attention" if k == "A" else "retention", "mixer": att if k == "A" else ret, "mlp": {"kind": "dense", "ff": ff}} for k in kinds]
+    return dict(model_type="gadarax", vocab_size=vocab, hidden_size=width, intermediate_size=ff, num_hidden_layers=len(layers),
+                num_attention_heads=latent["heads"], num_key_value_heads=latent["heads"], head_dim=latent["dim"], rms_norm_eps=1e-6,
+                tie_word_embeddings=True, mlp_gated=False, hidden_act="relu2", embed_scale=float(width) ** 0.5, norm_kind="dyt", mixers=layers,
+                layer_loop=loop)
+
+
 PRESETS: dict[str, dict] = {
+    # Gadarax at the size of small production models: latent attention and retention layers, three of them looped twice
+    "gadarax-1b": _layer_list(2048, 8192, dict(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512), dict(heads=16, dim=128, vdim=128),
+                              "AARARARARARA", dict(start=1, stop=4, times=2), 65536),
+    "gadarax-4b": _layer_list(4096, 16384, dict(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512), dict(heads=16, dim=256, vdim=256),
+                              "AARARARARARA", dict(start=1, stop=4, times=2), 65536),
+    "tiny-gadarax": _layer_list(96, 160, dict(heads=3, dim=16, rot_dim=8, vdim=24, kv_rank=40), dict(heads=4, dim=24, vdim=16), "ARAR",
+                                dict(start=1, stop=3, times=2), 264),
     # Llama-3.1-8B: 32 layers, d 4096, GQA 32q/8kv, SwiGLU 14336, vocab 128256, RoPE theta 5e5 (llama3 scaling)
     "llama3.1-8b": dict(model_type="llama", vocab_size=128256, hidden_size=4096, intermediate_size=14336,
                         num_hidden_layers=32, num_attention_heads=32, num_key_value_heads=8, head_dim=128,

@@ -777,6 +777,10 @@ class CausalLM(nn.Module):
             h = self.run_layers(self.embed(batch), batch)
             return self.sharder.run("head", lambda x: F.linear(F.rmsnorm(x, self.norm, self.cfg.rms_norm_eps), self.output_weight).float(), h)
         h = self.hidden_states(batch, h_in)
+        if self.cfg.is_mixer:
+            from .mixers import _linear
+
+            return _linear(h, self.output_weight).float()
         if self.tp.world == 1:
             return F.linear(h, self.output_weight).float()
         from rl_b200.parallel.tensor import gather_cols

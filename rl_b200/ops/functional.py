@@ -505,7 +505,7 @@ class _Embedding(torch.autograd.Function):
 
 
 def embedding(ids: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
-    if not use_native(table):
+    if not use_native(table) or table.dtype != BF16:
         return tF.embedding(ids, table)
     return _Embedding.apply(ids, table)
 
