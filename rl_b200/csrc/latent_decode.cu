@@ -2,14 +2,17 @@
 // with its own page table. Keys and values are never decompressed: all heads of a row read the same cached latent rows.
 //
 //   heads GEMM   q_lat[t, h, :] = q[t, h, :dim] W_uk[h]         the unrotated query carried into the latent space (W_uk read MN-major)
-//   attention    S^T[128 tokens, HN heads] = L Q^T               one CTA per (row, group of HN heads, split of the context); the tile of
+//   attention    S^T[64 tokens, HN heads] = L Q^T                one CTA per (row, group of HN heads, split of the context); the tile of
 //                O^T[128 dims, HN] (x rank / 128) += L^T P        latent rows is both K and V: it is fetched once
 //   combine      joins the splits
 //   heads GEMM   y[t, h, :] = o[t, h, :] W_uv[h]^T * sigmoid(gate), written over the gate columns of the projected rows
 //
-// The attention kernel streams the latent tile as 32 KB slots (two 64-column groups of 128 tokens) through a ring: the QK product
-// consumes slots as they land, the PV product gives them back one by one, so the next tile streams in under the rest of the PV
-// product and the softmax. O stays in TMEM over all tiles; it is rescaled only when a running maximum grew by more than 2^8.
+// The attention kernel streams latent tiles of 64 tokens as 16 KB slots (two 64-column groups) through a ring that holds at least
+// two tiles: the scores of tile i + 1 are computed under the softmax of tile i, and the PV product gives slots back one by one, so
+// the stream from memory never stops. The score product is issued with 128 rows; rows 64.. read the neighbouring slot and their
+// results are ignored (the instruction's cost is hidden under the stream). The narrow MMAs are bound by the issuing thread, so
+// every descriptor is a precomputed base plus a constant. O stays in TMEM over all tiles; it is rescaled only when a running
+// maximum grew by more than 2^8.
 #include "common.cuh"
 
 #include <math.h>
@@ -18,8 +21,13 @@ namespace {
 using namespace rlb;
 
 // ---------------------------------------------------------------------------------------------------- per-head GEMM
-constexpr int HG_T = 128, HG_K = 64, HG_STAGES = 4, HG_STAGE = 2 * HG_T * HG_K * 2;   // 32 KB per stage
-constexpr int HG_SMEM = HG_STAGES * HG_STAGE + 256 + 1024;
+constexpr int HG_T = 128, HG_K = 64;      // rows of A per tile, reduction step
+template <int BN, int STAGES>
+struct HgCfg {
+  static constexpr int STAGE = (HG_T + BN) * HG_K * 2;
+  static constexpr int SMEM = STAGES * STAGE + 256 + 1024;
+  static constexpr int TMEM = BN < 32 ? 32 : BN;
+};
 constexpr int HG_THREADS = 192;
 
 struct HeadsGemm {
@@ -33,9 +41,11 @@ struct HeadsGemm {
   int* status;
 };
 
-template <bool B_MN>
+template <bool B_MN, int BN, int STAGES>
 __global__ void __launch_bounds__(HG_THREADS, 1)
 gemm_heads_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ CUtensorMap tmap_b, HeadsGemm g) {
+  static_assert(!B_MN || BN == 128, "the MN-major operand is fetched as two 64-column boxes");
+  constexpr int HG_STAGES = STAGES, HG_STAGE = HgCfg<BN, STAGES>::STAGE;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint64_t* full = reinterpret_cast<uint64_t*>(smem + HG_STAGES * HG_STAGE);
@@ -57,7 +67,7 @@ gemm_heads_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_const
     prefetch_tmap(&tmap_b);
   }
   if (warp == 1) {
-    tmem_alloc(smem_u32(tmem_slot), 128);
+    tmem_alloc(smem_u32(tmem_slot), HgCfg<BN, STAGES>::TMEM);
     tmem_relinquish();
   }
   tc_fence_before();
@@ -65,7 +75,7 @@ gemm_heads_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_const
   tc_fence_after();
   pdl_sync();
   const uint32_t tmem = *tmem_slot;
-  const int n0 = blockIdx.x * HG_T, m0 = blockIdx.y * HG_T, head = blockIdx.z;
+  const int n0 = blockIdx.x * BN, m0 = blockIdx.y * HG_T, head = blockIdx.z;
   const int num_k = (g.K + HG_K - 1) / HG_K;
 
   if (warp == 0) {
@@ -87,7 +97,7 @@ gemm_heads_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_const
     }
   } else if (warp == 1) {
     if (lane == 0) {
-      constexpr uint32_t idesc = make_idesc_bf16(HG_T, HG_T, false, B_MN);
+      constexpr uint32_t idesc = make_idesc_bf16(HG_T, BN, false, B_MN);
       bool ok = true;
       for (int kb = 0; kb < num_k; ++kb) {
         const int s = kb % HG_STAGES;
@@ -110,7 +120,7 @@ gemm_heads_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_const
     if (mbar_wait(smem_u32(acc_bar), 0, abort_flag, g.status, RLB_ERR_WAIT_TMEM_FULL)) {
       tc_fence_after();
       __nv_bfloat16* o = g.out + static_cast<long long>(row) * g.ldo + g.o_off + static_cast<long long>(head) * g.o_head + n0;
-      for (int c = 0; c < HG_T && n0 + c < g.N; c += 32) {
+      for (int c = 0; c < BN && n0 + c < g.N; c += 32) {
         uint32_t r[32];
         tmem_ld_32x32b_x32(tmem + (static_cast<uint32_t>(quarter * 32) << 16) + c, r);
         tmem_ld_wait();
@@ -141,15 +151,15 @@ gemm_heads_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_const
   __syncthreads();
   if (warp == 1) {
     tc_fence_after();
-    tmem_dealloc(tmem, 128);
+    tmem_dealloc(tmem, HgCfg<BN, STAGES>::TMEM);
   }
 }
 
 // ---------------------------------------------------------------------------------------------------- attention
-constexpr int LD_TOK = 128;
-constexpr int LD_CHUNK = LD_TOK * 128;       // 128 tokens x 64 columns
-constexpr int LD_SLOT = 2 * LD_CHUNK;        // 32 KB
-constexpr int LD_MAX_SLOTS = 6;
+constexpr int LD_TOK = 64;
+constexpr int LD_CHUNK = LD_TOK * 128;       // 64 tokens x 64 columns
+constexpr int LD_SLOT = 2 * LD_CHUNK;        // 16 KB
+constexpr int LD_MAX_SLOTS = 12;
 constexpr int LD_THREADS = 192;
 constexpr float LD_LOG2E = 1.4426950408889634f;
 constexpr float LD_RESCALE = 8.0f;
@@ -173,10 +183,7 @@ struct LdParams {
 };
 
 __device__ __forceinline__ void ld_bar_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
-__device__ __forceinline__ uint32_t ld_sw128(int row, int col, int chunk_bytes) {
-  const int chunk = col >> 6, c = col & 63;
-  return chunk * chunk_bytes + row * 128 + ((((c * 2) >> 4) ^ (row & 7)) << 4) + ((c * 2) & 15);
-}
+__device__ __forceinline__ uint32_t ld_sw128(int row, int c) { return row * 128 + (((c >> 3) ^ (row & 7)) << 4) + ((c * 2) & 15); }
 
 // Butterfly over the warp that reduces N values per lane at once: after log2(N) exchanges each lane holds one value's partial
 // result, the rest of the exchanges complete it. Returns the reduced value `lane / (32 / N)`.
@@ -214,7 +221,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_lat, const __grid_
   uint8_t* ring = smem;
   uint8_t* q_sm = ring + p.slots * LD_SLOT;
   uint8_t* p_sm = q_sm + p.chunks * QP;
-  float* red = reinterpret_cast<float*>(p_sm + 2 * QP);    // [4][HN]
+  float* red = reinterpret_cast<float*>(p_sm + QP);        // [4][HN]
   uint64_t* bars = reinterpret_cast<uint64_t*>(red + 4 * HN);
   uint64_t *full = bars, *empty = bars + LD_MAX_SLOTS, *q_full = bars + 2 * LD_MAX_SLOTS;
   uint64_t *s_full = q_full + 1, *s_empty = q_full + 2, *p_ready = q_full + 3, *o_done = q_full + 4;
@@ -255,18 +262,18 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_lat, const __grid_
       for (int c = 0; c < p.chunks; ++c) tma_load_2d(smem_u32(q_sm + c * QP), &tmap_q, smem_u32(q_full), c * 64, row * p.heads + h0);
       const int* bt = p.block_table + static_cast<long long>(row) * p.bt_stride;
       const int box = bs < LD_TOK ? bs : LD_TOK, nbox = LD_TOK / box;
-      int it = 0;
+      int slot = 0;
+      uint32_t phase = 0;
       bool ok = true;
       for (int i = 0; i < n_tiles && ok; ++i) {
         const int t0 = t_begin + i * LD_TOK;
-        for (int j = 0; j < p.slots_tile; ++j, ++it) {
-          const int s = it % p.slots;
-          if (!mbar_wait(smem_u32(empty + s), ((it / p.slots) & 1) ^ 1, abort_flag, p.status, RLB_ERR_WAIT_EMPTY)) {
+        for (int j = 0; j < p.slots_tile; ++j) {
+          if (!mbar_wait(smem_u32(empty + slot), phase ^ 1, abort_flag, p.status, RLB_ERR_WAIT_EMPTY)) {
             ok = false;
             break;
           }
           const int nch = min(2, p.chunks - 2 * j);
-          const uint32_t bar = smem_u32(full + s), dst = smem_u32(ring + s * LD_SLOT);
+          const uint32_t bar = smem_u32(full + slot), dst = smem_u32(ring + slot * LD_SLOT);
           mbar_arrive_expect_tx(bar, nch * LD_CHUNK);
           for (int b = 0; b < nbox; ++b) {
             // tokens past the end read pages of valid (if unrelated) content; their scores are masked before the softmax
@@ -274,43 +281,59 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_lat, const __grid_
             const int crow = bt[min(t / bs, p.bt_stride - 1)] * bs + t % bs;
             for (int c = 0; c < nch; ++c) tma_load_2d(dst + c * LD_CHUNK + b * box * 128, &tmap_lat, bar, (2 * j + c) * 64, crow);
           }
+          if (++slot == p.slots) {
+            slot = 0;
+            phase ^= 1;
+          }
         }
       }
     }
   } else if (warp == 1) {
     if (lane == 0 && n_tiles > 0) {
-      constexpr uint32_t idesc_qk = make_idesc_bf16(LD_TOK, HN, false, false);
+      constexpr uint32_t idesc_qk = make_idesc_bf16(128, HN, false, false);
       constexpr uint32_t idesc_pv = make_idesc_bf16(128, HN, true, false);
-      bool ok = mbar_wait(smem_u32(q_full), 0, abort_flag, p.status, RLB_ERR_WAIT_FULL);
-      for (int i = 0; i < n_tiles && ok; ++i) {
-        const uint32_t ph = i & 1;
-        if (!mbar_wait(smem_u32(s_empty), ph ^ 1, abort_flag, p.status, RLB_ERR_WAIT_TMEM_EMPTY)) break;
-        for (int j = 0; j < p.slots_tile && ok; ++j) {
-          const int it = i * p.slots_tile + j, s = it % p.slots;
-          if (!mbar_wait(smem_u32(full + s), (it / p.slots) & 1, abort_flag, p.status, RLB_ERR_WAIT_FULL)) {
-            ok = false;
-            break;
-          }
+      const uint64_t k_desc = make_smem_desc_sw128(smem_u32(ring), 16, 1024), v_desc = make_smem_desc_sw128(smem_u32(ring), LD_CHUNK, 1024);
+      const uint64_t q_desc = make_smem_desc_sw128(smem_u32(q_sm), 16, 1024), p_desc = make_smem_desc_sw128(smem_u32(p_sm), 16, 1024);
+      int qk_slot = 0, pv_slot = 0;
+      uint32_t qk_phase = 0;
+      auto issue_qk = [&](int i) -> bool {
+        if (!mbar_wait(smem_u32(s_empty), (i & 1) ^ 1, abort_flag, p.status, RLB_ERR_WAIT_TMEM_EMPTY)) return false;
+        uint64_t qd = q_desc;
+        for (int j = 0; j < p.slots_tile; ++j) {
+          if (!mbar_wait(smem_u32(full + qk_slot), qk_phase, abort_flag, p.status, RLB_ERR_WAIT_FULL)) return false;
           tc_fence_after();
-          const uint32_t base = smem_u32(ring + s * LD_SLOT);
-          const int nch = min(2, p.chunks - 2 * j);
-          for (int kk = 0; kk < nch * 4; ++kk)
-            umma_f16(tmem_s, make_smem_desc_sw128(base + (kk >> 2) * LD_CHUNK + (kk & 3) * 32, 16, 1024),
-                     make_smem_desc_sw128(smem_u32(q_sm) + (2 * j + (kk >> 2)) * QP + (kk & 3) * 32, 16, 1024), idesc_qk, (j | kk) != 0 ? 1u : 0u);
-          if (j >= p.pairs) umma_commit(smem_u32(empty + s));    // holds only the rotated key part
-        }
-        if (!ok) break;
-        umma_commit(smem_u32(s_full));
-        if (!mbar_wait(smem_u32(p_ready), ph, abort_flag, p.status, RLB_ERR_WAIT_FLAG)) break;
-        tc_fence_after();
-        for (int j = 0; j < p.pairs; ++j) {
-          const int s = (i * p.slots_tile + j) % p.slots;
-          const uint32_t base = smem_u32(ring + s * LD_SLOT);
+          const uint64_t kd = k_desc + static_cast<uint32_t>(qk_slot * (LD_SLOT >> 4));
+          const bool two = 2 * j + 1 < p.chunks;
 #pragma unroll
-          for (int kk = 0; kk < LD_TOK / 16; ++kk)
-            umma_f16(tmem_o + j * HN, make_smem_desc_sw128(base + kk * 2048, LD_CHUNK, 1024),
-                     make_smem_desc_sw128(smem_u32(p_sm) + (kk >> 2) * QP + (kk & 3) * 32, 16, 1024), idesc_pv, (i | kk) != 0 ? 1u : 0u);
-          umma_commit(smem_u32(empty + s));
+          for (int kk = 0; kk < 4; ++kk) umma_f16(tmem_s, kd + kk * 2, qd + kk * 2, idesc_qk, (j | kk) != 0 ? 1u : 0u);
+          if (two) {
+#pragma unroll
+            for (int kk = 0; kk < 4; ++kk) umma_f16(tmem_s, kd + (LD_CHUNK >> 4) + kk * 2, qd + (QP >> 4) + kk * 2, idesc_qk, 1u);
+          }
+          qd += 2 * (QP >> 4);
+          if (j >= p.pairs) umma_commit(smem_u32(empty + qk_slot));    // holds only the rotated key part
+          if (++qk_slot == p.slots) {
+            qk_slot = 0;
+            qk_phase ^= 1;
+          }
+        }
+        umma_commit(smem_u32(s_full));
+        return true;
+      };
+      bool ok = mbar_wait(smem_u32(q_full), 0, abort_flag, p.status, RLB_ERR_WAIT_FULL);
+      if (ok) ok = issue_qk(0);
+      for (int i = 0; i < n_tiles && ok; ++i) {
+        if (i + 1 < n_tiles && !issue_qk(i + 1)) break;     // under the softmax of tile i
+        if (!mbar_wait(smem_u32(p_ready), i & 1, abort_flag, p.status, RLB_ERR_WAIT_FLAG)) break;
+        tc_fence_after();
+        for (int j = 0; j < p.slots_tile; ++j) {
+          if (j < p.pairs) {
+            const uint64_t vd = v_desc + static_cast<uint32_t>(pv_slot * (LD_SLOT >> 4));
+#pragma unroll
+            for (int kk = 0; kk < LD_TOK / 16; ++kk) umma_f16(tmem_o + j * HN, vd + kk * 128, p_desc + kk * 2, idesc_pv, (i | kk) != 0 ? 1u : 0u);
+            umma_commit(smem_u32(empty + pv_slot));
+          }
+          if (++pv_slot == p.slots) pv_slot = 0;
         }
         umma_commit(smem_u32(o_done));
       }
@@ -337,7 +360,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_lat, const __grid_
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(s_empty));
-      const bool valid = t_begin + i * LD_TOK + r < t_end;
+      const bool valid = r < LD_TOK && t_begin + i * LD_TOK + r < t_end;
       float s[HN], mx[HN];
 #pragma unroll
       for (int g = 0; g < HN; ++g) mx[g] = s[g] = valid ? __uint_as_float(sr[g]) * p.scale_log2 : -INFINITY;
@@ -376,8 +399,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_lat, const __grid_
           tmem_st_wait();
         }
       }
+      if (r < LD_TOK) {
 #pragma unroll
-      for (int g = 0; g < HN; ++g) *reinterpret_cast<__nv_bfloat16*>(p_sm + ld_sw128(g, r, QP)) = __float2bfloat16(s[g]);
+        for (int g = 0; g < HN; ++g) *reinterpret_cast<__nv_bfloat16*>(p_sm + ld_sw128(g, r)) = __float2bfloat16(s[g]);
+      }
       fence_proxy_async();
       tc_fence_before();
       ld_bar_sync();      // the maxima of this tile have been read by everyone before the next tile overwrites them
@@ -429,34 +454,45 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_lat, const __grid_
   }
 }
 
-__global__ void latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int num_splits, int rank,
-                                      __nv_bfloat16* __restrict__ out) {
+__global__ void __launch_bounds__(128)
+latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int num_splits, int rank, __nv_bfloat16* __restrict__ out) {
+  __shared__ float w[32];
   pdl_sync();
   const long long rh = blockIdx.x;
-  float mm = -INFINITY, ll = 0.f;
-  for (int s = 0; s < num_splits; ++s) mm = fmaxf(mm, part_ml[(rh * num_splits + s) * 2]);
-  for (int s = 0; s < num_splits; ++s) {
-    const float ms = part_ml[(rh * num_splits + s) * 2];
-    if (ms != -INFINITY) ll += part_ml[(rh * num_splits + s) * 2 + 1] * exp2f(ms - mm);
+  if (threadIdx.x < 32) {     // num_splits <= 32: one lane per split
+    const int s = threadIdx.x;
+    const float m = s < num_splits ? part_ml[(rh * num_splits + s) * 2] : -INFINITY;
+    const float l = s < num_splits ? part_ml[(rh * num_splits + s) * 2 + 1] : 0.f;
+    const float mm = warp_max(m);
+    const float f = m == -INFINITY ? 0.f : exp2f(m - mm);
+    const float ll = warp_sum(l * f);
+    w[s] = ll > 0.f ? f / ll : 0.f;
   }
-  const float inv = ll > 0.f ? 1.f / ll : 0.f;
-  for (int d = threadIdx.x; d < rank; d += blockDim.x) {
-    float acc = 0.f;
+  __syncthreads();
+  const float4* src = reinterpret_cast<const float4*>(part_o + rh * num_splits * rank);
+  const int n4 = rank / 4;
+  for (int d = threadIdx.x; d < n4; d += 128) {
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
     for (int s = 0; s < num_splits; ++s) {
-      const float ms = part_ml[(rh * num_splits + s) * 2];
-      if (ms != -INFINITY) acc += part_o[(rh * num_splits + s) * rank + d] * exp2f(ms - mm);
+      const float4 v = src[s * n4 + d];
+      acc.x = fmaf(v.x, w[s], acc.x);
+      acc.y = fmaf(v.y, w[s], acc.y);
+      acc.z = fmaf(v.z, w[s], acc.z);
+      acc.w = fmaf(v.w, w[s], acc.w);
     }
-    out[rh * rank + d] = __float2bfloat16(acc * inv);
+    *reinterpret_cast<uint2*>(out + rh * rank + d * 4) = make_uint2(pack_bf16x2(acc.x, acc.y), pack_bf16x2(acc.z, acc.w));
   }
 }
 
 template <int HN>
 int launch_latent_decode(const CUtensorMap& tl, const CUtensorMap& tq, LdParams p, int rows, cudaStream_t s) {
-  const int fixed = p.chunks * HN * 128 + 2 * HN * 128 + 4 * HN * 4 + (2 * LD_MAX_SLOTS + 6) * 8 + 1024;
+  // behind the ring: queries, weights, reductions, barriers, and at least the 8 KB that the score product may read past the last slot
+  const int fixed = LD_CHUNK + p.chunks * HN * 128 + HN * 128 + 4 * HN * 4 + (2 * LD_MAX_SLOTS + 6) * 8 + 1024;
   int slots = (227 * 1024 - fixed) / LD_SLOT;
   if (slots > LD_MAX_SLOTS) slots = LD_MAX_SLOTS;
-  if (p.slots_tile * 2 < slots) slots = p.slots_tile * 2;      // two whole tiles in flight are enough
-  if (slots < p.slots_tile) return -2;
+  if (p.slots_tile * 4 < slots) slots = p.slots_tile * 4;
+  if (slots < 2 * p.slots_tile) return -2;      // the scores run one tile ahead of the PV product
   p.slots = slots;
   const int cols = (1 + p.pairs) * HN;
   p.tmem_cols = cols <= 32 ? 32 : (cols <= 64 ? 64 : (cols <= 128 ? 128 : (cols <= 256 ? 256 : 512)));
@@ -484,7 +520,7 @@ RLB_API int rlb_latent_decode(void* p, int rows, long long ldp, int in_width, in
                               const int* seq_lens, const void* kv_up, float scale, void* q_lat, void* o_lat, int num_splits, float* part_o,
                               float* part_ml, int* status, void* stream) {
   if (rows <= 0) return 0;
-  if (!rlb_latent_decode_supported(dim, rot_dim, vdim, rank, width, block_size) || heads > 65535 || num_splits < 1) return -2;
+  if (!rlb_latent_decode_supported(dim, rot_dim, vdim, rank, width, block_size) || heads > 65535 || num_splits < 1 || num_splits > 32) return -2;
   if (ldp % 8 || q_off % 8 || mix_off % 8 || (dim + rot_dim) % 8 || (num_splits > 1 && (!part_o || !part_ml))) return -2;
   if ((reinterpret_cast<uintptr_t>(p) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(kv_up) | reinterpret_cast<uintptr_t>(q_lat) |
        reinterpret_cast<uintptr_t>(o_lat)) & 15)
@@ -492,8 +528,8 @@ RLB_API int rlb_latent_decode(void* p, int rows, long long ldp, int in_width, in
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(gemm_heads_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, HG_SMEM);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_heads_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, HG_SMEM);
+    cudaError_t e = cudaFuncSetAttribute(gemm_heads_kernel<true, 128, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, HgCfg<128, 4>::SMEM);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_heads_kernel<false, 32, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, HgCfg<32, 8>::SMEM);
     if (e != cudaSuccess) return static_cast<int>(e);
     configured = true;
   }
@@ -504,7 +540,7 @@ RLB_API int rlb_latent_decode(void* p, int rows, long long ldp, int in_width, in
   if (!rc) rc = rlb_make_tmap_2d(&tb, kv_up, BF, 2, rank, static_cast<uint64_t>(heads) * (dim + vdim), static_cast<uint64_t>(rank) * 2, 64, HG_K, SW);
   if (rc) return -100 - rc;
   HeadsGemm g{rows, rank, dim, q_off, dim + rot_dim, 0, dim, static_cast<__nv_bfloat16*>(q_lat), static_cast<long long>(heads) * width, 0, width, 0, status};
-  cudaError_t e = rlb_launch_pdl(gemm_heads_kernel<true>, dim3((rank + HG_T - 1) / HG_T, (rows + HG_T - 1) / HG_T, heads), dim3(HG_THREADS), HG_SMEM, s, ta, tb, g);
+  cudaError_t e = rlb_launch_pdl(gemm_heads_kernel<true, 128, 4>, dim3((rank + 127) / 128, (rows + HG_T - 1) / HG_T, heads), dim3(HG_THREADS), HgCfg<128, 4>::SMEM, s, ta, tb, g);
   if (e != cudaSuccess) return static_cast<int>(e);
 
   LdParams d{};
@@ -536,9 +572,9 @@ RLB_API int rlb_latent_decode(void* p, int rows, long long ldp, int in_width, in
     if (e != cudaSuccess) return static_cast<int>(e);
   }
   rc = rlb_make_tmap_2d(&ta, o_lat, BF, 2, static_cast<uint64_t>(heads) * rank, rows, static_cast<uint64_t>(heads) * rank * 2, HG_K, HG_T, SW);
-  if (!rc) rc = rlb_make_tmap_2d(&tb, kv_up, BF, 2, rank, static_cast<uint64_t>(heads) * (dim + vdim), static_cast<uint64_t>(rank) * 2, HG_K, HG_T, SW);
+  if (!rc) rc = rlb_make_tmap_2d(&tb, kv_up, BF, 2, rank, static_cast<uint64_t>(heads) * (dim + vdim), static_cast<uint64_t>(rank) * 2, HG_K, 32, SW);
   if (rc) return -100 - rc;
   HeadsGemm u{rows, vdim, rank, 0, rank, heads * dim, vdim, static_cast<__nv_bfloat16*>(p), ldp, mix_off, vdim, 1, status};
-  e = rlb_launch_pdl(gemm_heads_kernel<false>, dim3((vdim + HG_T - 1) / HG_T, (rows + HG_T - 1) / HG_T, heads), dim3(HG_THREADS), HG_SMEM, s, ta, tb, u);
+  e = rlb_launch_pdl(gemm_heads_kernel<false, 32, 8>, dim3((vdim + 31) / 32, (rows + HG_T - 1) / HG_T, heads), dim3(HG_THREADS), HgCfg<32, 8>::SMEM, s, ta, tb, u);
   return static_cast<int>(e);
 }

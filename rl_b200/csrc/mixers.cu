@@ -148,6 +148,7 @@ __global__ void latent_prep_kernel(T* __restrict__ p, LatentShape s, const int* 
   extern __shared__ float sm[];
   __shared__ float red[32];
   float* cs = sm;              // [half] cosine, then [half] sine
+  pdl_sync();
   const long long row = blockIdx.x;
   T* pr = p + row * s.ldp;
   const float pos = static_cast<float>(positions[row]);
@@ -413,11 +414,12 @@ RLB_API int rlb_latent_prep(void* p, int f32, long long rows, long long ldp, int
   LatentShape s{ldp, q_off, lat_off, 0, heads, dim, rot_dim, 0, rank, width, block_size, num_blocks};
   const size_t sm = sizeof(float) * 2 * (half + 1);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const dim3 grid(static_cast<unsigned>(rows)), block(rows > 1024 ? 128 : 256);
   if (f32)
-    latent_prep_kernel<float><<<static_cast<unsigned>(rows), 256, sm, st>>>(static_cast<float*>(p), s, positions, slots, static_cast<const float*>(norm_w),
+    rlb_launch_pdl(latent_prep_kernel<float>, grid, block, sm, st, static_cast<float*>(p), s, positions, slots, static_cast<const float*>(norm_w),
                                                                             freq, half, gain, eps, static_cast<float*>(cache), static_cast<float*>(q_lat), q_rows, status);
   else
-    latent_prep_kernel<__nv_bfloat16><<<static_cast<unsigned>(rows), 256, sm, st>>>(static_cast<__nv_bfloat16*>(p), s, positions, slots,
+    rlb_launch_pdl(latent_prep_kernel<__nv_bfloat16>, grid, block, sm, st, static_cast<__nv_bfloat16*>(p), s, positions, slots,
         static_cast<const __nv_bfloat16*>(norm_w), freq, half, gain, eps, static_cast<__nv_bfloat16*>(cache),
         static_cast<__nv_bfloat16*>(q_lat), q_rows, status);
   return static_cast<int>(cudaGetLastError());

@@ -38,7 +38,7 @@ struct RetShape {
 };
 
 constexpr int RT_C = 128;                 // tokens per chunk
-constexpr int RT_THREADS = 256;
+constexpr int RT_THREADS = 512;
 constexpr int RT_ATOM = RT_C * 128;       // 128 rows x 64 columns of bf16
 constexpr int RT_SATOM = 64 * 128;        // 64 state rows x 64 value columns
 
@@ -69,31 +69,40 @@ __device__ __forceinline__ void store_split(uint8_t* hi, uint8_t* lo, uint32_t o
   *reinterpret_cast<uint4*>(lo + off) = make_uint4(l[0], l[1], l[2], l[3]);
 }
 
-// Eight consecutive dimensions d0.. of one head's row, rotated (halves layout) in fp32. d0 is a multiple of 8 and below dim.
-__device__ __forceinline__ void load_rotated(const __nv_bfloat16* row, int d0, int half, const float* cs, float (&v)[8]) {
-  const uint4 raw = *reinterpret_cast<const uint4*>(row + d0);
-  const uint32_t w[4] = {raw.x, raw.y, raw.z, raw.w};
+// Eight consecutive dimensions d0.. of one head's row: the raw piece and, where the halves layout rotates whole pieces, its partner.
+struct RawPiece {
+  uint4 own, other;
+};
+__device__ __forceinline__ RawPiece load_piece(const __nv_bfloat16* row, int d0, int half) {
+  RawPiece r;
+  r.own = *reinterpret_cast<const uint4*>(row + d0);
+  if (d0 < 2 * half && half % 8 == 0) r.other = *reinterpret_cast<const uint4*>(row + (d0 < half ? d0 + half : d0 - half));
+  else r.other = make_uint4(0, 0, 0, 0);
+  return r;
+}
+__device__ __forceinline__ void unpack8(const uint4& r, float (&v)[8]) {
+  const uint32_t w[4] = {r.x, r.y, r.z, r.w};
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const float2 f = unpack_bf16x2(w[i]);
     v[2 * i] = f.x;
     v[2 * i + 1] = f.y;
   }
+}
+// The rotation of that piece in fp32 (d0 a multiple of 8).
+__device__ __forceinline__ void rotate_piece(const RawPiece& raw, const __nv_bfloat16* row, int d0, int half, const float* cs, float (&v)[8]) {
+  unpack8(raw.own, v);
   if (d0 >= 2 * half) return;
   if (half % 8 == 0) {
     const bool low = d0 < half;
     const int f0 = low ? d0 : d0 - half;
-    const uint4 oraw = *reinterpret_cast<const uint4*>(row + (low ? d0 + half : d0 - half));
-    const uint32_t ow[4] = {oraw.x, oraw.y, oraw.z, oraw.w};
     const float4 c0 = *reinterpret_cast<const float4*>(cs + f0), c1 = *reinterpret_cast<const float4*>(cs + f0 + 4);
     const float4 s0 = *reinterpret_cast<const float4*>(cs + half + f0), s1 = *reinterpret_cast<const float4*>(cs + half + f0 + 4);
     const float c[8] = {c0.x, c0.y, c0.z, c0.w, c1.x, c1.y, c1.z, c1.w}, s[8] = {s0.x, s0.y, s0.z, s0.w, s1.x, s1.y, s1.z, s1.w};
+    float o[8];
+    unpack8(raw.other, o);
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      const float2 of = unpack_bf16x2(ow[i / 2]);
-      const float o = (i & 1) ? of.y : of.x;
-      v[i] = low ? v[i] * c[i] - o * s[i] : v[i] * c[i] + o * s[i];
-    }
+    for (int i = 0; i < 8; ++i) v[i] = low ? v[i] * c[i] - o[i] * s[i] : v[i] * c[i] + o[i] * s[i];
   } else {
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
@@ -108,22 +117,37 @@ __device__ __forceinline__ void load_rotated(const __nv_bfloat16* row, int d0, i
 }
 
 // One 64-dimension atom [128 rows x 64] of rotated, scaled queries or keys, split into hi and lo; rows past the chunk and dimensions past
-// dim are zero. `weight` (null or [128]) multiplies the rows.
-__device__ __forceinline__ void fill_atom(const RetShape& p, uint8_t* hi, uint8_t* lo, int off, int head, int row_first, int rows, int dim0, float scale,
-                                          const float* weight) {
-  for (int i = threadIdx.x; i < RT_C * 8; i += RT_THREADS) {
-    const int r = i >> 3, piece = i & 7, d0 = dim0 + piece * 8;
-    float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-    if (r < rows && d0 < p.dim) {
-      load_rotated(p.p + static_cast<long long>(p.row0 + row_first + r) * p.ldp + off + head * p.dim, d0, p.half,
-                   p.cs + static_cast<long long>(row_first + r) * 2 * p.half, v);
-      const float s = weight ? scale * weight[r] : scale;
-#pragma unroll
-      for (int k = 0; k < 8; ++k) v[k] *= s;
-    }
-    store_split(hi, lo, rt_sw(r, piece), v);
+// dim are zero. `weight` (null or [128]) multiplies the rows. All loads of a thread are issued before the first is used: `fetch` and
+// `store` are separate so that a caller can have several atoms in flight.
+constexpr int RT_FILL = RT_C * 8 / RT_THREADS;
+struct AtomFill {
+  RawPiece raw[RT_FILL];
+  __device__ __forceinline__ const __nv_bfloat16* row(const RetShape& p, int off, int head, int row_first, int r) const {
+    return p.p + static_cast<long long>(p.row0 + row_first + r) * p.ldp + off + head * p.dim;
   }
-}
+  __device__ __forceinline__ void fetch(const RetShape& p, int off, int head, int row_first, int rows, int dim0) {
+#pragma unroll
+    for (int n = 0; n < RT_FILL; ++n) {
+      const int i = threadIdx.x + n * RT_THREADS, r = i >> 3, d0 = dim0 + (i & 7) * 8;
+      if (r < rows && d0 < p.dim) raw[n] = load_piece(row(p, off, head, row_first, r), d0, p.half);
+    }
+  }
+  __device__ __forceinline__ void store(const RetShape& p, uint8_t* hi, uint8_t* lo, int off, int head, int row_first, int rows, int dim0, float scale,
+                                        const float* weight) {
+#pragma unroll
+    for (int n = 0; n < RT_FILL; ++n) {
+      const int i = threadIdx.x + n * RT_THREADS, r = i >> 3, piece = i & 7, d0 = dim0 + piece * 8;
+      float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      if (r < rows && d0 < p.dim) {
+        rotate_piece(raw[n], row(p, off, head, row_first, r), d0, p.half, p.cs + static_cast<long long>(row_first + r) * 2 * p.half, v);
+        const float s = weight ? scale * weight[r] : scale;
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v[k] *= s;
+      }
+      store_split(hi, lo, rt_sw(r, piece), v);
+    }
+  }
+};
 
 // ---------------------------------------------------------------- sums of the chunks
 __global__ void __launch_bounds__(RT_THREADS, 1)
@@ -165,7 +189,12 @@ retention_state_kernel(const __grid_constant__ CUtensorMap tmap_v, RetShape p, i
   float* out = p.sums + (static_cast<long long>(chunk) * p.heads + head) * p.dim * p.vdim;
   bool ok = true;
   for (int d0 = 0, m = 0; d0 < p.dim; d0 += 128, ++m) {
-    for (int a = 0; a < 2; ++a) fill_atom(p, k_hi + a * RT_ATOM, k_lo + a * RT_ATOM, p.k_off, head, row_first, rows, d0 + a * 64, p.kscale, weight);
+    AtomFill f[2];
+#pragma unroll
+    for (int a = 0; a < 2; ++a) f[a].fetch(p, p.k_off, head, row_first, rows, d0 + a * 64);
+#pragma unroll
+    for (int a = 0; a < 2; ++a)
+      f[a].store(p, k_hi + a * RT_ATOM, k_lo + a * RT_ATOM, p.k_off, head, row_first, rows, d0 + a * 64, p.kscale, weight);
     fence_proxy_async();
     tc_fence_before();
     __syncthreads();
@@ -184,7 +213,7 @@ retention_state_kernel(const __grid_constant__ CUtensorMap tmap_v, RetShape p, i
     __syncwarp();
     tc_fence_after();
     const int d = d0 + quarter * 32 + lane;
-    for (int c = side * 32; c < p.vdim; c += 64) {
+    for (int c = side * 32; c < p.vdim; c += RT_THREADS / 4) {
       uint32_t r[32];
       tmem_ld_32x32b_x32(tmem + (static_cast<uint32_t>(quarter * 32) << 16) + c, r);
       tmem_ld_wait();
@@ -224,7 +253,7 @@ retention_scan_kernel(float* __restrict__ sums, const int* __restrict__ piece_ch
   const float ld = log2_decay[head];
   const long long step = static_cast<long long>(heads) * elems;
   float4* q = reinterpret_cast<float4*>(sums + (static_cast<long long>(c0) * heads + head) * elems + e);
-  constexpr int AHEAD = 4;
+  constexpr int AHEAD = 8;
   for (int c = c0; c < c1; c += AHEAD) {
     float4 add[AHEAD];
 #pragma unroll
@@ -255,8 +284,8 @@ retention_out_kernel(const __grid_constant__ CUtensorMap tmap_v, RetShape p, int
   uint8_t* s_lo = s_hi + atoms_v * RT_SATOM;
   uint8_t* v_s = s_lo + atoms_v * RT_SATOM;
   float* pw = reinterpret_cast<float*>(v_s + atoms_v * RT_ATOM);   // [129] powers of the decay
-  float* ssq = pw + 132;                                           // [2][128]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(ssq + 2 * RT_C);
+  float* ssq = pw + 132;                                           // [column groups][128]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(ssq + RT_THREADS);
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 2);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -288,22 +317,35 @@ retention_out_kernel(const __grid_constant__ CUtensorMap tmap_v, RetShape p, int
   bool ok = true;
   int done = 0;      // commits waited for
   for (int d0 = 0; d0 < p.dim; d0 += 64) {
+    // the loads of queries, keys and start state are in flight together
+    AtomFill fq, fk;
+    fq.fetch(p, p.q_off, head, row_first, rows, d0);
+    fk.fetch(p, p.k_off, head, row_first, rows, d0);
+    const int groups = atoms_v * 8;      // 8-column pieces of a state row
+    float4 sx[4], sy[4];
+#pragma unroll
+    for (int n = 0; n < 4; ++n) {        // 64 rows x at most 32 pieces
+      const int i = threadIdx.x + n * RT_THREADS, r = i / groups, v0 = (i % groups) * 8;
+      sx[n] = sy[n] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < 64 * groups && d0 + r < p.dim && v0 < p.vdim) {
+        sx[n] = *reinterpret_cast<const float4*>(S0 + static_cast<long long>(d0 + r) * p.vdim + v0);
+        sy[n] = *reinterpret_cast<const float4*>(S0 + static_cast<long long>(d0 + r) * p.vdim + v0 + 4);
+      }
+    }
     if (d0 > 0) {    // the previous products have read the stage
       ok = mbar_wait(smem_u32(bars + 1), done & 1, abort_flag, p.status, RLB_ERR_WAIT_EMPTY) && ok;
       ++done;
       __syncthreads();
     }
-    fill_atom(p, q_hi, q_lo, p.q_off, head, row_first, rows, d0, 1.f, nullptr);
-    fill_atom(p, k_hi, k_lo, p.k_off, head, row_first, rows, d0, p.kscale, nullptr);
-    for (int i = threadIdx.x; i < 64 * atoms_v * 8; i += RT_THREADS) {
-      const int r = i / (atoms_v * 8), g = i % (atoms_v * 8), v0 = g * 8;
-      float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-      if (d0 + r < p.dim && v0 < p.vdim) {
-        const float4 x = *reinterpret_cast<const float4*>(S0 + static_cast<long long>(d0 + r) * p.vdim + v0);
-        const float4 y = *reinterpret_cast<const float4*>(S0 + static_cast<long long>(d0 + r) * p.vdim + v0 + 4);
-        v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w; v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
+    fq.store(p, q_hi, q_lo, p.q_off, head, row_first, rows, d0, 1.f, nullptr);
+    fk.store(p, k_hi, k_lo, p.k_off, head, row_first, rows, d0, p.kscale, nullptr);
+#pragma unroll
+    for (int n = 0; n < 4; ++n) {
+      const int i = threadIdx.x + n * RT_THREADS, r = i / groups, g = i % groups;
+      if (i < 64 * groups) {
+        const float v[8] = {sx[n].x, sx[n].y, sx[n].z, sx[n].w, sy[n].x, sy[n].y, sy[n].z, sy[n].w};
+        store_split(s_hi, s_lo, (g >> 3) * RT_SATOM + rt_sw(r, g & 7), v);
       }
-      store_split(s_hi, s_lo, (g >> 3) * RT_SATOM + rt_sw(r, g & 7), v);
     }
     fence_proxy_async();
     tc_fence_before();
@@ -326,26 +368,25 @@ retention_out_kernel(const __grid_constant__ CUtensorMap tmap_v, RetShape p, int
   ++done;
   __syncwarp();
   tc_fence_after();
-  // warps 0-3 and 4-7 share the rows and split the columns
+  // groups of four warps share the rows and split the columns
   const int quarter = warp & 3, side = warp >> 2, i = quarter * 32 + lane;
   const uint32_t lane_addr = static_cast<uint32_t>(quarter * 32) << 16;
-#pragma unroll
-  for (int c = 0; c < 64; c += 32) {
+  for (int c = side * 32; c < RT_C; c += RT_THREADS / 4) {
     uint32_t r[32];
-    tmem_ld_32x32b_x32(tmem_s + lane_addr + side * 64 + c, r);
+    tmem_ld_32x32b_x32(tmem_s + lane_addr + c, r);
     tmem_ld_wait();
 #pragma unroll
     for (int q = 0; q < 4; ++q) {
       float v[8];
 #pragma unroll
       for (int k = 0; k < 8; ++k) {
-        const int j = side * 64 + c + q * 8 + k;
+        const int j = c + q * 8 + k;
         v[k] = j <= i ? __uint_as_float(r[q * 8 + k]) * pw[i - j] : 0.f;
       }
-      store_split(w_hi, w_lo, side * RT_ATOM + rt_sw(i, (c >> 3) + q), v);
+      store_split(w_hi, w_lo, (c >> 6) * RT_ATOM + rt_sw(i, ((c & 63) >> 3) + q), v);
     }
   }
-  for (int c = side * 32; c < vcols; c += 64) {     // start-state term: row i is d^(i+1) times what stands in O
+  for (int c = side * 32; c < vcols; c += RT_THREADS / 4) {     // start-state term: row i is d^(i+1) times what stands in O
     uint32_t r[16];
     const float f = pw[i + 1];
 #pragma unroll
@@ -378,7 +419,7 @@ retention_out_kernel(const __grid_constant__ CUtensorMap tmap_v, RetShape p, int
   __syncwarp();
   tc_fence_after();
   float ss = 0.f;
-  for (int c = side * 32; c < p.vdim; c += 64) {
+  for (int c = side * 32; c < p.vdim; c += RT_THREADS / 4) {
     uint32_t r[32];
     tmem_ld_32x32b_x32(tmem_o + lane_addr + c, r);
     tmem_ld_wait();
@@ -388,9 +429,12 @@ retention_out_kernel(const __grid_constant__ CUtensorMap tmap_v, RetShape p, int
   }
   ssq[side * RT_C + i] = ss;
   __syncthreads();
-  const float rstd = 1.f / sqrtf((ssq[i] + ssq[RT_C + i]) / static_cast<float>(p.vdim) + p.eps);
+  ss = 0.f;
+#pragma unroll
+  for (int g = 0; g < RT_THREADS / 128; ++g) ss += ssq[g * RT_C + i];
+  const float rstd = 1.f / sqrtf(ss / static_cast<float>(p.vdim) + p.eps);
   __nv_bfloat16* dst = p.p + static_cast<long long>(p.row0 + row_first + i) * p.ldp + p.mix_off + head * p.vdim;
-  for (int c = side * 32; c < p.vdim; c += 64) {
+  for (int c = side * 32; c < p.vdim; c += RT_THREADS / 4) {
     uint32_t r[32];
     tmem_ld_32x32b_x32(tmem_o + lane_addr + c, r);
     tmem_ld_wait();
@@ -547,7 +591,7 @@ RLB_API int rlb_retention_portions(void* p, long long rows, long long ldp, int i
   if (rc) return -100 - rc;
   const int av = (vdim + 63) / 64;
   const int smem_state = (4 + av) * RT_ATOM + RT_C * 4 + 64 + 1024;
-  const int smem_out = 4 * RT_ATOM + 2 * av * RT_SATOM + av * RT_ATOM + (132 + 2 * RT_C) * 4 + 64 + 1024;
+  const int smem_out = 4 * RT_ATOM + 2 * av * RT_SATOM + av * RT_ATOM + (132 + RT_THREADS) * 4 + 64 + 1024;
   static int conf_state = 0, conf_out = 0;
   if (smem_state > conf_state) {
     cudaError_t e = cudaFuncSetAttribute(retention_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_state);

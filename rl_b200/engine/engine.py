@@ -1107,12 +1107,18 @@ class GenerationEngine:
             if g is None:
                 no, nml = E.decode_scratch_sizes(B, self.hq, num_splits, c.head_dim)
                 scratch = (torch.empty(no, dtype=torch.float32, device=self.device), torch.empty(nml, dtype=torch.float32, device=self.device)) if num_splits > 1 else None
-                # warm-up outside capture (sets kernel attributes, sizes the allocator), then capture
+                # warm-up outside capture (sets kernel attributes, sizes the allocator), then capture. The warm-up must leave no trace:
+                # it writes no cache slot, works on the scratch state row, and the step inputs and outputs are put back
+                saved, saved_out = st["blob"].clone(), st["out_blob"].clone()
+                st["slots"].fill_(-1)
+                st["state_rows"].zero_()
                 side = torch.cuda.Stream(device=self.device)
                 side.wait_stream(torch.cuda.current_stream())
                 with torch.cuda.stream(side):
                     self._decode_body(st, B, sp, num_splits, scratch)
                 torch.cuda.current_stream().wait_stream(side)
+                st["blob"].copy_(saved)
+                st["out_blob"].copy_(saved_out)
                 torch.cuda.synchronize()
                 graph = torch.cuda.CUDAGraph()
                 before = _L.Counters.launches

@@ -246,9 +246,10 @@ def split_count(ctas: int, max_ctx: int, sms: int = 148) -> int:
 
 
 # --------------------------------------------------------------------------------------- retention
-def retention_(p: torch.Tensor, m, b: TokenBatch, state: torch.Tensor) -> None:
+def retention_(p: torch.Tensor, m, b: TokenBatch, state: torch.Tensor, plain: bool = False) -> None:
     """Retention of all rows of ``p``: every sequence's row of ``state`` [rows, heads, dim, vdim] (fp32) is advanced by its tokens. A
-    piece that starts at position 0 starts from zero. ``m``: the layer's ``RetentionMixer``."""
+    piece that starts at position 0 starts from zero. ``m``: the layer's ``RetentionMixer``. ``plain``: the token-by-token kernel for
+    every shape (it serves fp32 models and odd sizes)."""
     if not use_native(p):
         cuts = list(range(b.n_single)) + ([b.n_single + c for c in b.cu.tolist()] if b.cu is not None else [b.n_single])
         q, k, v = m.qkv(p, b.positions)
@@ -266,7 +267,7 @@ def retention_(p: torch.Tensor, m, b: TokenBatch, state: torch.Tensor) -> None:
              ptr(b.positions), ptr(rows), ptr(state), state.shape[0], ptr(m.decay), ptr(m.freq), m.freq.numel(), float(m.gain), m.dim ** -0.5,
              float(m.eps), st, stream_ptr())
 
-    if p.dtype == torch.bfloat16 and _L.lib().rlb_retention_supported(m.dim, m.vdim):
+    if not plain and p.dtype == torch.bfloat16 and _L.lib().rlb_retention_supported(m.dim, m.vdim):
         if b.n_single:
             call("rlb_retention_step", ptr(p), b.n_single, p.stride(0), m.q_off, m.k_off, m.v_off, m.mix_off, m.heads, m.dim, m.vdim, ptr(b.positions),
                  ptr(b.state_rows), ptr(state), state.shape[0], ptr(m.decay), ptr(m.freq), m.freq.numel(), float(m.gain), m.dim ** -0.5, float(m.eps),
