@@ -1,18 +1,16 @@
-// Decode form of latent attention on the tensor cores (tcgen05 + TMEM + TMA), bf16 in / fp32 accumulate. Every row is one query token
-// with its own page table. Keys and values are never decompressed: all heads of a row read the same cached latent rows.
+// Decode form of latent attention, bf16 in / fp32 accumulate. Every row is one query token with its own page table. Keys and values are
+// never decompressed: all heads of a row read the same cached latent rows.
 //
-//   heads GEMM   q_lat[t, h, :] = q[t, h, :dim] W_uk[h]         the unrotated query carried into the latent space (W_uk read MN-major)
-//   attention    S^T[64 tokens, HN heads] = L Q^T                one CTA per (row, group of HN heads, split of the context); the tile of
-//                O^T[128 dims, HN] (x rank / 128) += L^T P        latent rows is both K and V: it is fetched once
+//   heads GEMM   q_lat[t, h, :] = q[t, h, :dim] W_uk[h]         the unrotated query carried into the latent space (tcgen05, W_uk MN-major)
+//   attention    one CTA per (row, group of HN heads, split of the context): a tile of 64 latent rows is both K and V and is fetched once,
+//                by TMA, into a ring of 64-column chunks
 //   combine      joins the splits
-//   heads GEMM   y[t, h, :] = o[t, h, :] W_uv[h]^T * sigmoid(gate), written over the gate columns of the projected rows
+//   heads GEMM   y[t, h, :] = o[t, h, :] W_uv[h]^T * sigmoid(gate) (tcgen05), written over the gate columns of the projected rows
 //
-// The attention kernel streams latent tiles of 64 tokens as 16 KB slots (two 64-column groups) through a ring that holds at least
-// two tiles: the scores of tile i + 1 are computed under the softmax of tile i, and the PV product gives slots back one by one, so
-// the stream from memory never stops. The score product is issued with 128 rows; rows 64.. read the neighbouring slot and their
-// results are ignored (the instruction's cost is hidden under the stream). The narrow MMAs are bound by the issuing thread, so
-// every descriptor is a precomputed base plus a constant. O stays in TMEM over all tiles; it is rescaled only when a running
-// maximum grew by more than 2^8.
+// The attention products have 16 or 32 rows (heads) only. A tcgen05.mma with 128 latent rows on the M side and 16 heads on the N side
+// occupies its pipe for about 120 cycles (measured: the issuing thread is held that long per instruction, although the tensor pipe is
+// active for 32), which makes the 52 instructions of a 64-token tile take twice the time its 72 KB take to arrive. m16n8k16 warp
+// MMAs fit 16 heads exactly, keep the queries and the output in registers, and leave the kernel bound by the stream.
 #include "common.cuh"
 
 #include <math.h>
@@ -156,98 +154,77 @@ gemm_heads_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_const
 }
 
 // ---------------------------------------------------------------------------------------------------- attention
-constexpr int LD_TOK = 64;
-constexpr int LD_CHUNK = LD_TOK * 128;       // 64 tokens x 64 columns
-constexpr int LD_SLOT = 2 * LD_CHUNK;        // 16 KB
-constexpr int LD_MAX_SLOTS = 12;
-constexpr int LD_THREADS = 192;
+constexpr int LD_TOK = 64;                   // tokens per tile
+constexpr int LD_CHUNK = LD_TOK * 128;       // 64 tokens x 64 columns: 8 KB, 128-byte swizzle
+constexpr int LD_MAX_RING = 24;              // chunks in the ring
+constexpr int LD_HALF = 5;                   // 64-column groups of a latent row that one half of the warps multiplies (rows up to 640)
+constexpr int LD_WARPS = 8;
+constexpr int LD_THREADS = 32 * LD_WARPS;
+constexpr int LD_PSTRIDE = LD_TOK + 8;       // weights: 144-byte rows, free of bank conflicts
+constexpr int LD_SSTRIDE = LD_TOK + 4;       // partial scores (fp32)
 constexpr float LD_LOG2E = 1.4426950408889634f;
-constexpr float LD_RESCALE = 8.0f;
 
 struct LdParams {
   const int* block_table;
   int bt_stride;
   const int* seq_lens;
-  int heads, rank, block_size;
+  int heads, rank, width, block_size;
   int chunks;         // 64-column groups of a latent row
-  int pairs;          // 128-dim output tiles
-  int slots_tile;     // ring slots of one tile: ceil(chunks / 2)
-  int slots;          // ring size
-  int tmem_cols;
+  int ring;           // chunk slots
   float scale_log2;
   int num_splits;
+  const __nv_bfloat16* q;   // [rows, heads, width]
   float* part_o;      // [rows, heads, splits, rank]
   float* part_ml;     // [rows, heads, splits, 2]
   __nv_bfloat16* out; // [rows, heads * rank]
   int* status;
 };
 
-__device__ __forceinline__ void ld_bar_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
-__device__ __forceinline__ uint32_t ld_sw128(int row, int c) { return row * 128 + (((c >> 3) ^ (row & 7)) << 4) + ((c * 2) & 15); }
-
-// Butterfly over the warp that reduces N values per lane at once: after log2(N) exchanges each lane holds one value's partial
-// result, the rest of the exchanges complete it. Returns the reduced value `lane / (32 / N)`.
-template <int N, typename Op>
-__device__ __forceinline__ float warp_reduce_many(float (&v)[N], int lane, Op op) {
-  int n = N, off = 16;
-#pragma unroll
-  for (int step = 0; step < 5; ++step, off >>= 1) {
-    if (n > 1) {
-      n >>= 1;
-      const bool up = lane & off;
-#pragma unroll
-      for (int k = 0; k < N / 2; ++k) {
-        if (k < n) {
-          const float keep = up ? v[k + n] : v[k], send = up ? v[k] : v[k + n];
-          v[k] = op(keep, __shfl_xor_sync(0xffffffffu, send, off));
-        }
-      }
-    } else {
-      v[0] = op(v[0], __shfl_xor_sync(0xffffffffu, v[0], off));
-    }
-  }
-  return v[0];
+__device__ __forceinline__ void ld_bar_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
+__device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm_x4_trans(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(addr)
+               : "memory");
+}
+__device__ __forceinline__ void mma_16x8x16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-__device__ __forceinline__ void ld_tmem_ld16(uint32_t addr, uint32_t* r) { tmem_ld_32x32b_x16(addr, *reinterpret_cast<uint32_t(*)[16]>(r)); }
-__device__ __forceinline__ void ld_tmem_st16(uint32_t addr, uint32_t* r) { tmem_st_32x32b_x16(addr, *reinterpret_cast<uint32_t(*)[16]>(r)); }
-
+// HN heads (16 or 32) of one row against one split of its context. Eight warps (a ninth would cost the others a quarter of their
+// registers); one thread of the last one requests the chunks of later tiles by TMA when the barrier after a tile's scores has shown that
+// everybody is done with the tile before it.
+//   scores   warp = (head group of 16, token group, half of the latent row): its queries stay in registers as A fragments, the two
+//            halves' partial scores meet in shared memory
+//   softmax  256 / HN threads per head, running maximum and sum in registers
+//   PV       warp w owns output columns 64 w .. 64 w + 63 of all heads in registers
 template <int HN>
 __global__ void __launch_bounds__(LD_THREADS, 1)
-latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_lat, const __grid_constant__ CUtensorMap tmap_q, LdParams p) {
+latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_lat, LdParams p) {
+  constexpr int HG = HN / 16, TG = 4 / HG, TW = LD_TOK / TG;   // head groups, token groups, tokens per group
+  constexpr int PER = 256 / HN, TPT = LD_TOK / PER;            // softmax threads per head, tokens per thread
   extern __shared__ uint8_t smem_raw[];
-  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  constexpr int QP = HN * 128;     // one 64-column group of Q or of P^T
-  uint8_t* ring = smem;
-  uint8_t* q_sm = ring + p.slots * LD_SLOT;
-  uint8_t* p_sm = q_sm + p.chunks * QP;
-  float* red = reinterpret_cast<float*>(p_sm + QP);        // [4][HN]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(red + 4 * HN);
-  uint64_t *full = bars, *empty = bars + LD_MAX_SLOTS, *q_full = bars + 2 * LD_MAX_SLOTS;
-  uint64_t *s_full = q_full + 1, *s_empty = q_full + 2, *p_ready = q_full + 3, *o_done = q_full + 4;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(q_full + 5);
-  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  uint8_t* ring = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  float* sred = reinterpret_cast<float*>(ring + p.ring * LD_CHUNK);                          // [2][HN][LD_SSTRIDE]
+  __nv_bfloat16* pw = reinterpret_cast<__nv_bfloat16*>(sred + 2 * HN * LD_SSTRIDE);           // [HN][LD_PSTRIDE]
+  float* fac = reinterpret_cast<float*>(pw + HN * LD_PSTRIDE);                                // [HN] rescale factors, at the end 1 / sum
+  uint64_t* full = reinterpret_cast<uint64_t*>(fac + HN);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(full + LD_MAX_RING);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
-    for (int s = 0; s < 2 * LD_MAX_SLOTS + 2; ++s) mbar_init(smem_u32(bars + s), 1);
-    mbar_init(smem_u32(s_empty), 4);
-    mbar_init(smem_u32(p_ready), 128);
-    mbar_init(smem_u32(o_done), 1);
+    for (int s = 0; s < LD_MAX_RING; ++s) mbar_init(smem_u32(full + s), 1);
     *abort_flag = 0;
     mbar_fence_init();
     fence_proxy_async();
     prefetch_tmap(&tmap_lat);
-    prefetch_tmap(&tmap_q);
   }
-  if (warp == 1) {
-    tmem_alloc(smem_u32(tmem_slot), p.tmem_cols);
-    tmem_relinquish();
-  }
-  tc_fence_before();
   __syncthreads();
-  tc_fence_after();
   pdl_sync();
-  const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + HN;
 
   const int row = blockIdx.x, h0 = blockIdx.y * HN, split = blockIdx.z;
   const int bs = p.block_size;
@@ -256,201 +233,210 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_lat, const __grid_
   const int t_begin = split * per_split, t_end = min(len, t_begin + per_split);
   const int n_tiles = t_end > t_begin ? (t_end - t_begin + LD_TOK - 1) / LD_TOK : 0;
 
-  if (warp == 0) {
-    if (lane == 0 && n_tiles > 0) {
-      mbar_arrive_expect_tx(smem_u32(q_full), p.chunks * QP);
-      for (int c = 0; c < p.chunks; ++c) tma_load_2d(smem_u32(q_sm + c * QP), &tmap_q, smem_u32(q_full), c * 64, row * p.heads + h0);
-      const int* bt = p.block_table + static_cast<long long>(row) * p.bt_stride;
-      const int box = bs < LD_TOK ? bs : LD_TOK, nbox = LD_TOK / box;
-      int slot = 0;
-      uint32_t phase = 0;
-      bool ok = true;
-      for (int i = 0; i < n_tiles && ok; ++i) {
-        const int t0 = t_begin + i * LD_TOK;
-        for (int j = 0; j < p.slots_tile; ++j) {
-          if (!mbar_wait(smem_u32(empty + slot), phase ^ 1, abort_flag, p.status, RLB_ERR_WAIT_EMPTY)) {
-            ok = false;
-            break;
-          }
-          const int nch = min(2, p.chunks - 2 * j);
-          const uint32_t bar = smem_u32(full + slot), dst = smem_u32(ring + slot * LD_SLOT);
-          mbar_arrive_expect_tx(bar, nch * LD_CHUNK);
-          for (int b = 0; b < nbox; ++b) {
-            // tokens past the end read pages of valid (if unrelated) content; their scores are masked before the softmax
-            const int t = t0 + b * box;
-            const int crow = bt[min(t / bs, p.bt_stride - 1)] * bs + t % bs;
-            for (int c = 0; c < nch; ++c) tma_load_2d(dst + c * LD_CHUNK + b * box * 128, &tmap_lat, bar, (2 * j + c) * 64, crow);
-          }
-          if (++slot == p.slots) {
-            slot = 0;
-            phase ^= 1;
-          }
+  // TMA requests in order: chunk after chunk, tile after tile
+  int rq_tile = 0, rq_chunk = 0, rq_slot = 0;
+  auto request = [&](int count) {
+    const int* bt = p.block_table + static_cast<long long>(row) * p.bt_stride;
+    const int box = bs < LD_TOK ? bs : LD_TOK, nbox = LD_TOK / box;
+    int crow[4];
+    for (int done = 0; done < count && rq_tile < n_tiles; ++done) {
+      if (done == 0 || rq_chunk == 0) {
+#pragma unroll
+        for (int b = 0; b < 4; ++b) {
+          // tokens past the end read pages of valid (if unrelated) content; their scores are masked before the softmax
+          const int t = t_begin + rq_tile * LD_TOK + b * box;
+          crow[b] = b < nbox ? bt[min(t / bs, p.bt_stride - 1)] * bs + t % bs : 0;
         }
       }
-    }
-  } else if (warp == 1) {
-    if (lane == 0 && n_tiles > 0) {
-      constexpr uint32_t idesc_qk = make_idesc_bf16(128, HN, false, false);
-      constexpr uint32_t idesc_pv = make_idesc_bf16(128, HN, true, false);
-      const uint64_t k_desc = make_smem_desc_sw128(smem_u32(ring), 16, 1024), v_desc = make_smem_desc_sw128(smem_u32(ring), LD_CHUNK, 1024);
-      const uint64_t q_desc = make_smem_desc_sw128(smem_u32(q_sm), 16, 1024), p_desc = make_smem_desc_sw128(smem_u32(p_sm), 16, 1024);
-      int qk_slot = 0, pv_slot = 0;
-      uint32_t qk_phase = 0;
-      auto issue_qk = [&](int i) -> bool {
-        if (!mbar_wait(smem_u32(s_empty), (i & 1) ^ 1, abort_flag, p.status, RLB_ERR_WAIT_TMEM_EMPTY)) return false;
-        uint64_t qd = q_desc;
-        for (int j = 0; j < p.slots_tile; ++j) {
-          if (!mbar_wait(smem_u32(full + qk_slot), qk_phase, abort_flag, p.status, RLB_ERR_WAIT_FULL)) return false;
-          tc_fence_after();
-          const uint64_t kd = k_desc + static_cast<uint32_t>(qk_slot * (LD_SLOT >> 4));
-          const bool two = 2 * j + 1 < p.chunks;
+      const uint32_t bar = smem_u32(full + rq_slot), dst = smem_u32(ring + rq_slot * LD_CHUNK);
+      mbar_arrive_expect_tx(bar, LD_CHUNK);
 #pragma unroll
-          for (int kk = 0; kk < 4; ++kk) umma_f16(tmem_s, kd + kk * 2, qd + kk * 2, idesc_qk, (j | kk) != 0 ? 1u : 0u);
-          if (two) {
-#pragma unroll
-            for (int kk = 0; kk < 4; ++kk) umma_f16(tmem_s, kd + (LD_CHUNK >> 4) + kk * 2, qd + (QP >> 4) + kk * 2, idesc_qk, 1u);
-          }
-          qd += 2 * (QP >> 4);
-          if (j >= p.pairs) umma_commit(smem_u32(empty + qk_slot));    // holds only the rotated key part
-          if (++qk_slot == p.slots) {
-            qk_slot = 0;
-            qk_phase ^= 1;
-          }
-        }
-        umma_commit(smem_u32(s_full));
-        return true;
-      };
-      bool ok = mbar_wait(smem_u32(q_full), 0, abort_flag, p.status, RLB_ERR_WAIT_FULL);
-      if (ok) ok = issue_qk(0);
-      for (int i = 0; i < n_tiles && ok; ++i) {
-        if (i + 1 < n_tiles && !issue_qk(i + 1)) break;     // under the softmax of tile i
-        if (!mbar_wait(smem_u32(p_ready), i & 1, abort_flag, p.status, RLB_ERR_WAIT_FLAG)) break;
-        tc_fence_after();
-        for (int j = 0; j < p.slots_tile; ++j) {
-          if (j < p.pairs) {
-            const uint64_t vd = v_desc + static_cast<uint32_t>(pv_slot * (LD_SLOT >> 4));
-#pragma unroll
-            for (int kk = 0; kk < LD_TOK / 16; ++kk) umma_f16(tmem_o + j * HN, vd + kk * 128, p_desc + kk * 2, idesc_pv, (i | kk) != 0 ? 1u : 0u);
-            umma_commit(smem_u32(empty + pv_slot));
-          }
-          if (++pv_slot == p.slots) pv_slot = 0;
-        }
-        umma_commit(smem_u32(o_done));
+      for (int b = 0; b < 4; ++b)
+        if (b < nbox) tma_load_2d(dst + b * box * 128, &tmap_lat, bar, rq_chunk * 64, crow[b]);
+      if (++rq_chunk == p.chunks) {
+        rq_chunk = 0;
+        ++rq_tile;
       }
+      if (++rq_slot == p.ring) rq_slot = 0;
     }
-  } else {
-    const int quarter = warp & 3, r = quarter * 32 + lane;
-    const uint32_t lane_addr = static_cast<uint32_t>(quarter * 32) << 16;
-    float m_ref[HN], l[HN];
+  };
+  const bool requester = threadIdx.x == LD_THREADS - 32;
+  if (requester) request(p.ring);
+
+  const int kh = warp & 1, tg = (warp >> 1) % TG, hg = (warp >> 1) / TG;
+  const int c_begin = kh ? (p.chunks + 1) / 2 : 0, c_end = kh ? p.chunks : (p.chunks + 1) / 2;
+  // query fragments of this warp's heads and half of the row
+  uint32_t qf[LD_HALF * 4][4];
+  {
+    const int r0 = h0 + hg * 16 + (lane >> 2);
 #pragma unroll
-    for (int g = 0; g < HN; ++g) {
-      m_ref[g] = -INFINITY;
-      l[g] = 0.f;
-    }
-    bool ok = true;
-    for (int i = 0; i < n_tiles; ++i) {
-      const uint32_t ph = i & 1;
-      // a wait that ran out clears `ok` but leaves no loop early: every warp passes the same named barriers
-      ok = ok && mbar_wait(smem_u32(s_full), ph, abort_flag, p.status, RLB_ERR_WAIT_TMEM_FULL);
-      tc_fence_after();
-      uint32_t sr[HN];
+    for (int k = 0; k < LD_HALF * 4; ++k) {
 #pragma unroll
-      for (int c = 0; c < HN; c += 16) ld_tmem_ld16(tmem_s + lane_addr + c, sr + c);
-      tmem_ld_wait();
-      tc_fence_before();
-      __syncwarp();
-      if (lane == 0) mbar_arrive(smem_u32(s_empty));
-      const bool valid = r < LD_TOK && t_begin + i * LD_TOK + r < t_end;
-      float s[HN], mx[HN];
-#pragma unroll
-      for (int g = 0; g < HN; ++g) mx[g] = s[g] = valid ? __uint_as_float(sr[g]) * p.scale_log2 : -INFINITY;
-      const float wm = warp_reduce_many<HN>(mx, lane, [](float a, float b) { return fmaxf(a, b); });
-      if (lane % (32 / HN) == 0) red[quarter * HN + lane / (32 / HN)] = wm;
-      ld_bar_sync();
-      float f[HN];
-      bool need = false;
-#pragma unroll
-      for (int g = 0; g < HN; ++g) {
-        const float mt = fmaxf(fmaxf(red[g], red[HN + g]), fmaxf(red[2 * HN + g], red[3 * HN + g]));
-        f[g] = 1.f;
-        if (mt > m_ref[g] + LD_RESCALE || m_ref[g] == -INFINITY) {
-          f[g] = m_ref[g] == -INFINITY ? 0.f : exp2f(m_ref[g] - mt);
-          need = true;
-          m_ref[g] = mt;
-        }
-        s[g] = s[g] == -INFINITY ? 0.f : exp2f(s[g] - m_ref[g]);
-        l[g] = l[g] * f[g] + s[g];
-      }
-      if (i > 0) {
-        ok = ok && mbar_wait(smem_u32(o_done), (i - 1) & 1, abort_flag, p.status, RLB_ERR_WAIT_TMEM_EMPTY);
-        tc_fence_after();
-        if (need) {     // the same decision in every thread: the maxima are shared
-          for (int j = 0; j < p.pairs; ++j) {
-#pragma unroll
-            for (int c = 0; c < HN; c += 16) {
-              uint32_t o[16];
-              ld_tmem_ld16(tmem_o + lane_addr + j * HN + c, o);
-              tmem_ld_wait();
-#pragma unroll
-              for (int g = 0; g < 16; ++g) o[g] = __float_as_uint(__uint_as_float(o[g]) * f[c + g]);
-              ld_tmem_st16(tmem_o + lane_addr + j * HN + c, o);
-            }
-          }
-          tmem_st_wait();
-        }
-      }
-      if (r < LD_TOK) {
-#pragma unroll
-        for (int g = 0; g < HN; ++g) *reinterpret_cast<__nv_bfloat16*>(p_sm + ld_sw128(g, r)) = __float2bfloat16(s[g]);
-      }
-      fence_proxy_async();
-      tc_fence_before();
-      ld_bar_sync();      // the maxima of this tile have been read by everyone before the next tile overwrites them
-      mbar_arrive(smem_u32(p_ready));
-    }
-    if (ok && n_tiles > 0) ok = mbar_wait(smem_u32(o_done), (n_tiles - 1) & 1, abort_flag, p.status, RLB_ERR_WAIT_TMEM_EMPTY);
-    tc_fence_after();
-    float lw[HN];
-#pragma unroll
-    for (int g = 0; g < HN; ++g) lw[g] = l[g];
-    const float ws = warp_reduce_many<HN>(lw, lane, [](float a, float b) { return a + b; });
-    if (lane % (32 / HN) == 0) red[quarter * HN + lane / (32 / HN)] = ws;
-    ld_bar_sync();
-#pragma unroll
-    for (int g = 0; g < HN; ++g) l[g] = (red[g] + red[HN + g]) + (red[2 * HN + g] + red[3 * HN + g]);
-    for (int j = 0; j < p.pairs; ++j) {
-      uint32_t o[HN];
-#pragma unroll
-      for (int c = 0; c < HN; c += 16) ld_tmem_ld16(tmem_o + lane_addr + j * HN + c, o + c);
-      tmem_ld_wait();
-      const int d = j * 128 + r;
-      if (d >= p.rank) continue;
-#pragma unroll
-      for (int g = 0; g < HN; ++g) {
-        if (h0 + g >= p.heads) continue;
-        const float v = (ok && n_tiles > 0) ? __uint_as_float(o[g]) : 0.f;
-        const long long rh = static_cast<long long>(row) * p.heads + h0 + g;
-        if (p.num_splits == 1)
-          p.out[rh * p.rank + d] = __float2bfloat16(l[g] > 0.f ? v / l[g] : 0.f);
-        else
-          p.part_o[(rh * p.num_splits + split) * p.rank + d] = v;
-      }
-    }
-    if (p.num_splits > 1 && r == 0) {
-#pragma unroll
-      for (int g = 0; g < HN; ++g) {
-        if (h0 + g >= p.heads) continue;
-        const long long i = ((static_cast<long long>(row) * p.heads + h0 + g) * p.num_splits + split) * 2;
-        p.part_ml[i] = m_ref[g];
-        p.part_ml[i + 1] = l[g];
+      for (int e = 0; e < 4; ++e) {
+        const int h = r0 + (e & 1) * 8, col = c_begin * 64 + k * 16 + (lane & 3) * 2 + (e >> 1) * 8;
+        qf[k][e] = (h < p.heads && col < p.width && k < (c_end - c_begin) * 4)
+                       ? *reinterpret_cast<const uint32_t*>(p.q + (static_cast<long long>(row) * p.heads + h) * p.width + col)
+                       : 0u;
       }
     }
   }
-  tc_fence_before();
-  __syncthreads();
-  if (warp == 1) {
-    tc_fence_after();
-    tmem_dealloc(tmem_s, p.tmem_cols);
+  float o[HG][8][4];
+#pragma unroll
+  for (int g = 0; g < HG; ++g)
+#pragma unroll
+    for (int n = 0; n < 8; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[g][n][e] = 0.f;
+  const int sh = threadIdx.x / PER, st0 = (threadIdx.x % PER) * TPT;     // softmax: this thread's head and first token
+  float m_run = -INFINITY, l_run = 0.f;
+  const bool owns = warp * 64 < p.rank;
+  const uint32_t p_addr = smem_u32(pw);
+  int base = 0;             // ring slot of the tile's first chunk
+  uint32_t phase = 0;       // its phase
+  bool ok = true;
+
+  for (int i = 0; i < n_tiles; ++i) {
+    // ---- scores. A wait that ran out clears `ok` but leaves no loop early: every warp passes the same barriers.
+    float s[TW / 8][4];
+#pragma unroll
+    for (int n = 0; n < TW / 8; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[n][e] = 0.f;
+#pragma unroll
+    for (int cc = 0; cc < LD_HALF; ++cc) {
+      if (c_begin + cc < c_end) {
+        int slot = base + c_begin + cc;
+        const bool wrap = slot >= p.ring;
+        if (wrap) slot -= p.ring;
+        ok = ok && mbar_wait(smem_u32(full + slot), phase ^ (wrap ? 1u : 0u), abort_flag, p.status, RLB_ERR_WAIT_FULL);
+        __syncwarp();
+        const uint32_t chunk = smem_u32(ring + slot * LD_CHUNK);
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) {
+#pragma unroll
+          for (int t = 0; t < TW / 16; ++t) {
+            const int tok = tg * TW + t * 16 + (lane & 7) + ((lane >> 4) << 3), piece = 2 * kk + ((lane >> 3) & 1);
+            uint32_t b[4];
+            ldsm_x4(chunk + tok * 128 + ((piece ^ (tok & 7)) << 4), b);
+            mma_16x8x16(s[2 * t], qf[cc * 4 + kk], b[0], b[1]);
+            mma_16x8x16(s[2 * t + 1], qf[cc * 4 + kk], b[2], b[3]);
+          }
+        }
+      }
+    }
+    {
+      float* dst = sred + (kh * HN + hg * 16 + (lane >> 2)) * LD_SSTRIDE + tg * TW + (lane & 3) * 2;
+#pragma unroll
+      for (int n = 0; n < TW / 8; ++n) {
+        *reinterpret_cast<float2*>(dst + n * 8) = make_float2(s[n][0], s[n][1]);
+        *reinterpret_cast<float2*>(dst + 8 * LD_SSTRIDE + n * 8) = make_float2(s[n][2], s[n][3]);
+      }
+    }
+    ld_bar_sync();
+    if (requester && i > 0) request(p.chunks);      // tile i - 1 has been read by everyone
+    // ---- softmax
+    {
+      float v[TPT];
+      float mx = -INFINITY;
+#pragma unroll
+      for (int k = 0; k < TPT; k += 4) {
+        const float4 a = *reinterpret_cast<const float4*>(sred + sh * LD_SSTRIDE + st0 + k), b = *reinterpret_cast<const float4*>(sred + (HN + sh) * LD_SSTRIDE + st0 + k);
+        const float t[4] = {a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          v[k + e] = t_begin + i * LD_TOK + st0 + k + e < t_end ? t[e] * p.scale_log2 : -INFINITY;
+          mx = fmaxf(mx, v[k + e]);
+        }
+      }
+#pragma unroll
+      for (int off = PER / 2; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+      const float mn = fmaxf(m_run, mx);       // finite: every tile holds a valid token
+      const float f = m_run == -INFINITY ? 0.f : exp2f(m_run - mn);
+      m_run = mn;
+      float sum = 0.f;
+#pragma unroll
+      for (int k = 0; k < TPT; k += 2) {
+        const float a = exp2f(v[k] - mn), b = exp2f(v[k + 1] - mn);
+        sum += a + b;
+        *reinterpret_cast<uint32_t*>(pw + sh * LD_PSTRIDE + st0 + k) = pack_bf16x2(a, b);
+      }
+      l_run = l_run * f + sum;                 // this thread's tokens; joined at the end
+      if (threadIdx.x % PER == 0) fac[sh] = f;
+    }
+    ld_bar_sync();
+    // ---- PV
+    if (owns) {
+      int slot = base + warp;
+      if (slot >= p.ring) slot -= p.ring;
+      const uint32_t chunk = smem_u32(ring + slot * LD_CHUNK);     // (its scores have been read, so it is there)
+#pragma unroll
+      for (int g = 0; g < HG; ++g) {
+        const float f0 = fac[g * 16 + (lane >> 2)], f1 = fac[g * 16 + (lane >> 2) + 8];
+#pragma unroll
+        for (int n = 0; n < 8; ++n) {
+          o[g][n][0] *= f0;
+          o[g][n][1] *= f0;
+          o[g][n][2] *= f1;
+          o[g][n][3] *= f1;
+        }
+      }
+#pragma unroll
+      for (int ks = 0; ks < LD_TOK / 16; ++ks) {
+        uint32_t a[HG][4];
+#pragma unroll
+        for (int g = 0; g < HG; ++g)
+          ldsm_x4(p_addr + ((g * 16 + (lane & 15)) * LD_PSTRIDE + ks * 16 + (lane >> 4) * 8) * 2, a[g]);
+        const int tok = ks * 16 + (lane & 15);
+#pragma unroll
+        for (int n2 = 0; n2 < 4; ++n2) {
+          uint32_t b[4];
+          ldsm_x4_trans(chunk + tok * 128 + (((n2 * 2 + (lane >> 4)) ^ (tok & 7)) << 4), b);
+#pragma unroll
+          for (int g = 0; g < HG; ++g) {
+            mma_16x8x16(o[g][2 * n2], a[g], b[0], b[1]);
+            mma_16x8x16(o[g][2 * n2 + 1], a[g], b[2], b[3]);
+          }
+        }
+      }
+    }
+    base += p.chunks;
+    if (base >= p.ring) {
+      base -= p.ring;
+      phase ^= 1;
+    }
+  }
+#pragma unroll
+  for (int off = PER / 2; off > 0; off >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, off);
+  ld_bar_sync();            // the last factors have been read
+  if (threadIdx.x % PER == 0) {
+    fac[sh] = p.num_splits > 1 ? 1.f : ((ok && l_run > 0.f) ? 1.f / l_run : 0.f);
+    if (p.num_splits > 1 && h0 + sh < p.heads) {
+      const long long k = ((static_cast<long long>(row) * p.heads + h0 + sh) * p.num_splits + split) * 2;
+      p.part_ml[k] = m_run;
+      p.part_ml[k + 1] = l_run;
+    }
+  }
+  ld_bar_sync();
+  if (!owns) return;
+#pragma unroll
+  for (int g = 0; g < HG; ++g) {
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int hl = g * 16 + half * 8 + (lane >> 2);
+      if (h0 + hl >= p.heads) continue;
+      const float f = fac[hl];
+      const long long rh = static_cast<long long>(row) * p.heads + h0 + hl;
+#pragma unroll
+      for (int n = 0; n < 8; ++n) {
+        const int d = warp * 64 + n * 8 + (lane & 3) * 2;
+        if (d >= p.rank) continue;
+        const float a = o[g][n][half * 2] * f, b = o[g][n][half * 2 + 1] * f;
+        if (p.num_splits == 1)
+          *reinterpret_cast<uint32_t*>(p.out + rh * p.rank + d) = pack_bf16x2(a, b);
+        else
+          *reinterpret_cast<float2*>(p.part_o + (rh * p.num_splits + split) * p.rank + d) = make_float2(a, b);
+      }
+    }
   }
 }
 
@@ -486,24 +472,20 @@ latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict_
 }
 
 template <int HN>
-int launch_latent_decode(const CUtensorMap& tl, const CUtensorMap& tq, LdParams p, int rows, cudaStream_t s) {
-  // behind the ring: queries, weights, reductions, barriers, and at least the 8 KB that the score product may read past the last slot
-  const int fixed = LD_CHUNK + p.chunks * HN * 128 + HN * 128 + 4 * HN * 4 + (2 * LD_MAX_SLOTS + 6) * 8 + 1024;
-  int slots = (227 * 1024 - fixed) / LD_SLOT;
-  if (slots > LD_MAX_SLOTS) slots = LD_MAX_SLOTS;
-  if (p.slots_tile * 4 < slots) slots = p.slots_tile * 4;
-  if (slots < 2 * p.slots_tile) return -2;      // the scores run one tile ahead of the PV product
-  p.slots = slots;
-  const int cols = (1 + p.pairs) * HN;
-  p.tmem_cols = cols <= 32 ? 32 : (cols <= 64 ? 64 : (cols <= 128 ? 128 : (cols <= 256 ? 256 : 512)));
-  const int smem = slots * LD_SLOT + fixed;
+int launch_latent_decode(const CUtensorMap& tl, LdParams p, int rows, cudaStream_t s) {
+  const int fixed = 2 * HN * LD_SSTRIDE * 4 + HN * LD_PSTRIDE * 2 + HN * 4 + LD_MAX_RING * 8 + 16 + 1024;
+  p.ring = (227 * 1024 - fixed) / LD_CHUNK;
+  if (p.ring > LD_MAX_RING) p.ring = LD_MAX_RING;
+  if (p.ring > 3 * p.chunks) p.ring = 3 * p.chunks;
+  if (p.ring < p.chunks || p.chunks > 2 * LD_HALF) return -2;
+  const int smem = p.ring * LD_CHUNK + fixed;
   static int configured = 0;
   if (smem > configured) {
     cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<HN>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return static_cast<int>(e);
     configured = smem;
   }
-  return static_cast<int>(rlb_launch_pdl(latent_decode_kernel<HN>, dim3(rows, (p.heads + HN - 1) / HN, p.num_splits), dim3(LD_THREADS), smem, s, tl, tq, p));
+  return static_cast<int>(rlb_launch_pdl(latent_decode_kernel<HN>, dim3(rows, (p.heads + HN - 1) / HN, p.num_splits), dim3(LD_THREADS), smem, s, tl, p));
 }
 }  // namespace
 
@@ -535,7 +517,7 @@ RLB_API int rlb_latent_decode(void* p, int rows, long long ldp, int in_width, in
   }
   const auto BF = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   const auto SW = CU_TENSOR_MAP_SWIZZLE_128B;
-  CUtensorMap ta, tb, tl, tq;
+  CUtensorMap ta, tb, tl;
   int rc = rlb_make_tmap_2d(&ta, p, BF, 2, in_width, rows, ldp * 2, HG_K, HG_T, SW);
   if (!rc) rc = rlb_make_tmap_2d(&tb, kv_up, BF, 2, rank, static_cast<uint64_t>(heads) * (dim + vdim), static_cast<uint64_t>(rank) * 2, 64, HG_K, SW);
   if (rc) return -100 - rc;
@@ -550,9 +532,9 @@ RLB_API int rlb_latent_decode(void* p, int rows, long long ldp, int in_width, in
   d.heads = heads;
   d.rank = rank;
   d.block_size = block_size;
+  d.width = width;
   d.chunks = (width + 63) / 64;
-  d.pairs = (rank + 127) / 128;
-  d.slots_tile = (d.chunks + 1) / 2;
+  d.q = static_cast<const __nv_bfloat16*>(q_lat);
   d.scale_log2 = scale * LD_LOG2E;
   d.num_splits = num_splits;
   d.part_o = part_o;
@@ -562,9 +544,8 @@ RLB_API int rlb_latent_decode(void* p, int rows, long long ldp, int in_width, in
   const int hn = heads > 16 ? 32 : 16;
   rc = rlb_make_tmap_2d(&tl, cache, BF, 2, width, static_cast<uint64_t>(num_blocks) * block_size, static_cast<uint64_t>(width) * 2, 64,
                         block_size < LD_TOK ? block_size : LD_TOK, SW);
-  if (!rc) rc = rlb_make_tmap_2d(&tq, q_lat, BF, 2, width, static_cast<uint64_t>(rows) * heads, static_cast<uint64_t>(width) * 2, 64, hn, SW);
   if (rc) return -100 - rc;
-  rc = hn == 32 ? launch_latent_decode<32>(tl, tq, d, rows, s) : launch_latent_decode<16>(tl, tq, d, rows, s);
+  rc = hn == 32 ? launch_latent_decode<32>(tl, d, rows, s) : launch_latent_decode<16>(tl, d, rows, s);
   if (rc) return rc;
   if (num_splits > 1) {
     e = rlb_launch_pdl(latent_combine_kernel, dim3(static_cast<unsigned>(rows) * heads), dim3(128), 0, s, part_o, part_ml, num_splits, rank,
