@@ -159,7 +159,9 @@ constexpr int LD_CHUNK = LD_TOK * 128;       // 64 tokens x 64 columns: 8 KB, 12
 constexpr int LD_MAX_RING = 24;              // chunks in the ring
 constexpr int LD_HALF = 5;                   // 64-column groups of a latent row that one half of the warps multiplies (rows up to 640)
 constexpr int LD_WARPS = 8;
-constexpr int LD_THREADS = 32 * LD_WARPS;
+constexpr int LD_THREADS = 32 * LD_WARPS + 128;
+constexpr int LD_REGS_LOAD = 24, LD_REGS_COMPUTE = 240;   // per thread after the split; 384 threads are launched with 168 each
+static_assert(128 * LD_REGS_LOAD + 256 * LD_REGS_COMPUTE <= LD_THREADS * 168, "the split exceeds what the block was launched with");
 constexpr int LD_PSTRIDE = LD_TOK + 8;       // weights: 144-byte rows, free of bank conflicts
 constexpr int LD_SSTRIDE = LD_TOK + 4;       // partial scores (fp32)
 constexpr float LD_LOG2E = 1.4426950408889634f;
@@ -196,9 +198,9 @@ __device__ __forceinline__ void mma_16x8x16(float (&d)[4], const uint32_t (&a)[4
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-// HN heads (16 or 32) of one row against one split of its context. Eight warps (a ninth would cost the others a quarter of their
-// registers); one thread of the last one requests the chunks of later tiles by TMA when the barrier after a tile's scores has shown that
-// everybody is done with the tile before it.
+// HN heads (16 or 32) of one row against one split of its context. Two warpgroups compute; the third one's first thread requests the
+// chunks by TMA (a request waits for the queue whenever memory is the limit, so it must not stand in a computing warp's way) and gives
+// its registers to the others.
 //   scores   warp = (head group of 16, token group, half of the latent row): its queries stay in registers as A fragments, the two
 //            halves' partial scores meet in shared memory
 //   softmax  256 / HN threads per head, running maximum and sum in registers
@@ -214,10 +216,12 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_lat, LdParams p) {
   __nv_bfloat16* pw = reinterpret_cast<__nv_bfloat16*>(sred + 2 * HN * LD_SSTRIDE);           // [HN][LD_PSTRIDE]
   float* fac = reinterpret_cast<float*>(pw + HN * LD_PSTRIDE);                                // [HN] rescale factors, at the end 1 / sum
   uint64_t* full = reinterpret_cast<uint64_t*>(fac + HN);
-  volatile int* abort_flag = reinterpret_cast<volatile int*>(full + LD_MAX_RING);
+  uint64_t* tile_done = full + LD_MAX_RING;      // [2], tiles alternate
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tile_done + 2);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
     for (int s = 0; s < LD_MAX_RING; ++s) mbar_init(smem_u32(full + s), 1);
+    for (int s = 0; s < 2; ++s) mbar_init(smem_u32(tile_done + s), LD_WARPS);
     *abort_flag = 0;
     mbar_fence_init();
     fence_proxy_async();
@@ -233,35 +237,43 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_lat, LdParams p) {
   const int t_begin = split * per_split, t_end = min(len, t_begin + per_split);
   const int n_tiles = t_end > t_begin ? (t_end - t_begin + LD_TOK - 1) / LD_TOK : 0;
 
-  // TMA requests in order: chunk after chunk, tile after tile
-  int rq_tile = 0, rq_chunk = 0, rq_slot = 0;
-  auto request = [&](int count) {
-    const int* bt = p.block_table + static_cast<long long>(row) * p.bt_stride;
-    const int box = bs < LD_TOK ? bs : LD_TOK, nbox = LD_TOK / box;
-    int crow[4];
-    for (int done = 0; done < count && rq_tile < n_tiles; ++done) {
-      if (done == 0 || rq_chunk == 0) {
+  if (warp >= LD_WARPS) {
+    asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(LD_REGS_LOAD));
+    if (warp == LD_WARPS && lane == 0) {
+      const int* bt = p.block_table + static_cast<long long>(row) * p.bt_stride;
+      const int box = bs < LD_TOK ? bs : LD_TOK, nbox = LD_TOK / box;
+      int slot = 0, free_chunks = p.ring, freed = 0;      // tiles that have been given back
+      bool ok = true;
+      for (int i = 0; i < n_tiles && ok; ++i) {
+        int crow[4];
 #pragma unroll
         for (int b = 0; b < 4; ++b) {
           // tokens past the end read pages of valid (if unrelated) content; their scores are masked before the softmax
-          const int t = t_begin + rq_tile * LD_TOK + b * box;
+          const int t = t_begin + i * LD_TOK + b * box;
           crow[b] = b < nbox ? bt[min(t / bs, p.bt_stride - 1)] * bs + t % bs : 0;
         }
-      }
-      const uint32_t bar = smem_u32(full + rq_slot), dst = smem_u32(ring + rq_slot * LD_CHUNK);
-      mbar_arrive_expect_tx(bar, LD_CHUNK);
+        for (int c = 0; c < p.chunks; ++c) {
+          if (free_chunks == 0) {
+            if (!mbar_wait(smem_u32(tile_done + (freed & 1)), (freed >> 1) & 1, abort_flag, p.status, RLB_ERR_WAIT_EMPTY)) {
+              ok = false;
+              break;
+            }
+            ++freed;
+            free_chunks = p.chunks;
+          }
+          --free_chunks;
+          const uint32_t bar = smem_u32(full + slot), dst = smem_u32(ring + slot * LD_CHUNK);
+          mbar_arrive_expect_tx(bar, LD_CHUNK);
 #pragma unroll
-      for (int b = 0; b < 4; ++b)
-        if (b < nbox) tma_load_2d(dst + b * box * 128, &tmap_lat, bar, rq_chunk * 64, crow[b]);
-      if (++rq_chunk == p.chunks) {
-        rq_chunk = 0;
-        ++rq_tile;
+          for (int b = 0; b < 4; ++b)
+            if (b < nbox) tma_load_2d(dst + b * box * 128, &tmap_lat, bar, c * 64, crow[b]);
+          if (++slot == p.ring) slot = 0;
+        }
       }
-      if (++rq_slot == p.ring) rq_slot = 0;
     }
-  };
-  const bool requester = threadIdx.x == LD_THREADS - 32;
-  if (requester) request(p.ring);
+    return;
+  }
+  asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(LD_REGS_COMPUTE));
 
   const int kh = warp & 1, tg = (warp >> 1) % TG, hg = (warp >> 1) / TG;
   const int c_begin = kh ? (p.chunks + 1) / 2 : 0, c_end = kh ? p.chunks : (p.chunks + 1) / 2;
@@ -333,7 +345,6 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_lat, LdParams p) {
       }
     }
     ld_bar_sync();
-    if (requester && i > 0) request(p.chunks);      // tile i - 1 has been read by everyone
     // ---- softmax
     {
       float v[TPT];
@@ -399,6 +410,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_lat, LdParams p) {
         }
       }
     }
+    __syncwarp();
+    if (lane == 0) mbar_arrive(smem_u32(tile_done + (i & 1)));
     base += p.chunks;
     if (base >= p.ring) {
       base -= p.ring;
@@ -473,7 +486,7 @@ latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict_
 
 template <int HN>
 int launch_latent_decode(const CUtensorMap& tl, LdParams p, int rows, cudaStream_t s) {
-  const int fixed = 2 * HN * LD_SSTRIDE * 4 + HN * LD_PSTRIDE * 2 + HN * 4 + LD_MAX_RING * 8 + 16 + 1024;
+  const int fixed = 2 * HN * LD_SSTRIDE * 4 + HN * LD_PSTRIDE * 2 + HN * 4 + (LD_MAX_RING + 2) * 8 + 16 + 1024;
   p.ring = (227 * 1024 - fixed) / LD_CHUNK;
   if (p.ring > LD_MAX_RING) p.ring = LD_MAX_RING;
   if (p.ring > 3 * p.chunks) p.ring = 3 * p.chunks;
