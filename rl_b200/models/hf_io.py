@@ -28,6 +28,8 @@ def hf_name_map(cfg: ModelConfig, tp_rank: int = 0, tp_size: int = 1, layer_offs
     is rows ``local_rows`` of the local parameter (of global expert ``e`` when the local parameter is expert-stacked).
     Local layer ``j`` is HF layer ``layer_offset + j`` (pipeline stages own contiguous layer ranges), or ``layer_ids[j]`` when
     the stage interleaves several runs of layers."""
+    if cfg.is_mixer:    # their tensors are row AND column ranges of fused weights: iter_hf_shards names them
+        raise NotImplementedError("layer-list models have no row map: sharded parameters, quantisation-aware training and re-sharding refits do not cover them")
     n_layers = cfg.num_hidden_layers - layer_offset if num_local_layers is None else num_local_layers
     ids = list(layer_ids) if layer_ids is not None else [layer_offset + j for j in range(n_layers)]
     n_layers = len(ids)

@@ -229,12 +229,28 @@ def gemma3_flops(hf, seq: int) -> float:
     return total + head_flops(seq, d, _g(hf, "vocab_size"))
 
 
+def gadarax_flops(hf, seq: int) -> float:
+    """Layer-list models: latent attention (plain query projection, output gate) or retention beside a two-matrix MLP; looped layers
+    count once per pass. ``hf`` is the model configuration object."""
+    d, total = _g(hf, "hidden_size"), 0.0
+    for i, _ in _g(hf, "layer_runs"):
+        e = _g(hf, "mixers")[i]
+        m = e["mixer"]
+        H, kd, vd = m["heads"], m["dim"], m["vdim"]
+        if e["type"] == "latent_attention":
+            total += mla_attention_flops(seq, d, H, 0, m["kv_rank"], kd, m["rot_dim"], vd) + 2 * seq * d * H * vd
+        else:      # projections q, k, v, gate, output; state update and readout
+            total += 2 * seq * d * H * (2 * kd + 3 * vd) + 4 * seq * H * kd * vd
+        total += mlp_flops(seq, d, e["mlp"]["ff"], gated=False) if e.get("mlp") else 0.0
+    return total + head_flops(seq, d, _g(hf, "vocab_size"))
+
+
 FAMILY_FLOPS = {
     "llama": llama_flops, "mistral": mistral_flops, "qwen2": qwen2_flops, "qwen3": qwen3_flops, "gemma3": gemma3_flops,
     "gemma3_text": gemma3_flops,
     "gpt2": gpt_flops, "gpt3": gpt_flops, "nemotron": nemotron_flops, "mixtral": mixtral_flops, "qwen3_moe": qwen3_moe_flops,
     "qwen2_moe": moe_decoder_flops, "deepseek_v3": deepseek_v3_flops, "deepseek_v2": deepseek_v3_flops, "nemotron_h": nemotron_h_flops,
-    "bert": bert_flops,
+    "bert": bert_flops, "gadarax": gadarax_flops,
 }
 
 

@@ -157,6 +157,28 @@ def test_random_init_and_presets():
         build_model(preset("tiny-gadarax"), pp_size=2)
 
 
+def test_worker_trains_and_generates():
+    """The policy worker around the model: rollout log-probabilities equal the trainer's, and a few steps lower the loss."""
+    from rl_b200.algorithms.loss.loss_functions import NLLLossFn
+    from rl_b200.distributed.batched_data_dict import BatchedDataDict
+    from rl_b200.policy.worker import PolicyWorker
+    from rl_b200.utils.flops import model_flops
+
+    mc = preset("tiny-gadarax")
+    assert model_flops(mc, 20) > 0
+    p = PolicyWorker(dict(precision="float32", train_global_batch_size=4, train_micro_batch_size=2, max_total_sequence_length=64,
+                          optimizer=dict(name="torch.optim.AdamW", kwargs=dict(lr=1e-3)),
+                          generation=dict(max_new_tokens=8, stop_token_ids=[], kv_cache_tokens=1024, block_size=16, max_running=4)),
+                     model_cfg=mc, device="cpu", init_reference_model=False)
+    recs = p.build_generation().engine.generate([G.tokens({"vocab": 264}, 12, s) for s in range(4)], SamplingParams(max_new_tokens=8, seed=1))
+    ids = torch.tensor([r.prompt + r.out_tokens for r in recs])
+    data = BatchedDataDict(input_ids=ids, input_lengths=torch.full((4,), 20), token_mask=torch.ones(4, 20), sample_mask=torch.ones(4))
+    lp = p.get_logprobs(data)["logprobs"][:, 12:]
+    assert torch.allclose(lp, torch.tensor([r.out_logprobs for r in recs]), atol=1e-5)
+    losses = [float(p.train(data, NLLLossFn(), gbs=4, mbs=2)["loss"]) for _ in range(3)]
+    assert losses[2] < losses[0]
+
+
 # ------------------------------------------------------------------------------------------------ engine
 @pytest.mark.parametrize("cuts", [[1000], [1], [2], [3], [16], [17, 2, 33, 1], [50, 1]])
 def test_portions_equal_the_oracle(case, cuts):
