@@ -139,68 +139,87 @@ struct LatentShape {
   int block_size, num_blocks;
 };
 
-// Per row: latent / rms * w and rotated shared key into the cache row of the token; rotated query parts in place, and for the first
-// `q_rows` rows also behind the latent columns of q_lat [rows, heads, width] (the decode kernels' queries).
+// Two CTAs per row. blockIdx.y 0: latent / rms * w and the rotated shared key into the cache row of the token. blockIdx.y 1: the
+// rotated query parts, in place, and for the first `q_rows` rows also behind the latent columns of q_lat [rows, heads, width]
+// (the decode kernels' queries). Few rows are a matter of latency: every load is issued before the first is used, angles are computed
+// by the thread that needs them.
+constexpr int LP_KEEP = 8;     // latent columns a thread keeps in registers
 template <typename T>
-__global__ void latent_prep_kernel(T* __restrict__ p, LatentShape s, const int* __restrict__ positions, const long long* __restrict__ slots,
-                                   const T* __restrict__ norm_w, const float* __restrict__ freq, int half, float gain, float eps,
-                                   T* __restrict__ cache, T* __restrict__ q_lat, int q_rows, int* status) {
-  extern __shared__ float sm[];
+__global__ void __launch_bounds__(128)
+latent_prep_kernel(T* __restrict__ p, LatentShape s, const int* __restrict__ positions, const long long* __restrict__ slots,
+                   const T* __restrict__ norm_w, const float* __restrict__ freq, int half, float gain, float eps,
+                   T* __restrict__ cache, T* __restrict__ q_lat, int q_rows, int* status) {
   __shared__ float red[32];
-  float* cs = sm;              // [half] cosine, then [half] sine
+  const int tid = threadIdx.x;
   pdl_sync();
   const long long row = blockIdx.x;
   T* pr = p + row * s.ldp;
   const float pos = static_cast<float>(positions[row]);
-  for (int i = threadIdx.x; i < half; i += blockDim.x) {
-    float sn, c;
-    sincosf(pos * freq[i], &sn, &c);
-    cs[i] = c * gain;
-    cs[half + i] = sn * gain;
+  if (blockIdx.y == 1) {
+    const int tail = s.width - s.rank, pairs = (tail + 1) / 2, qd = s.dim + s.rot_dim;
+    const bool decode = q_lat && row < q_rows;
+    for (int i = tid; i < s.heads * pairs; i += 128) {
+      const int h = i / pairs, f = i % pairs, j = 2 * f;
+      T* q = pr + s.q_off + h * qd + s.dim + j;
+      float u = j < s.rot_dim ? ld(q) : 0.f, v = j + 1 < s.rot_dim ? ld(q + 1) : 0.f;
+      if (f < half) {
+        float sn, c;
+        sincosf(pos * freq[f], &sn, &c);
+        c *= gain;
+        sn *= gain;
+        const float a = u * c - v * sn, b = v * c + u * sn;
+        st(q, a);
+        st(q + 1, b);
+        u = a;
+        v = b;
+      }
+      if (decode) {
+        T* o = q_lat + (row * s.heads + h) * s.width + s.rank + j;
+        st(o, u);
+        if (j + 1 < tail) st(o + 1, v);
+      }
+    }
+    return;
   }
+  const long long slot = slots[row];
+  const T* lat = pr + s.lat_off;
+  float keep[LP_KEEP];
   float ss = 0.f;
-  for (int r = threadIdx.x; r < s.rank; r += blockDim.x) {
-    const float v = ld(pr + s.lat_off + r);
+#pragma unroll
+  for (int k = 0; k < LP_KEEP; ++k) {
+    const int r = tid + k * 128;
+    keep[k] = r < s.rank ? ld(lat + r) : 0.f;
+  }
+#pragma unroll
+  for (int k = 0; k < LP_KEEP; ++k) ss += keep[k] * keep[k];
+  for (int r = tid + LP_KEEP * 128; r < s.rank; r += 128) {
+    const float v = ld(lat + r);
     ss += v * v;
   }
-  ss = block_sum(ss, red);
-  const float rstd = 1.f / sqrtf(ss / static_cast<float>(s.rank) + eps);
-  __syncthreads();
-  const long long slot = slots[row];
-  if (slot >= static_cast<long long>(s.num_blocks) * s.block_size) {
-    if (threadIdx.x == 0 && status) atomicCAS(status, 0, RLB_ERR_BOUNDS);
-  } else if (slot >= 0) {
-    T* cr = cache + slot * s.width;
-    for (int r = threadIdx.x; r < s.width; r += blockDim.x) {
-      float v = 0.f;
-      if (r < s.rank) {
-        v = ld(pr + s.lat_off + r) * rstd * ld(norm_w + r);
-      } else if (r < s.rank + s.rot_dim) {
-        const int j = r - s.rank;
-        v = ld(pr + s.lat_off + r);
-        if (j < 2 * half) {
-          const float o = ld(pr + s.lat_off + s.rank + (j ^ 1));
-          v = (j & 1) ? v * cs[j >> 1] + o * cs[half + (j >> 1)] : v * cs[j >> 1] - o * cs[half + (j >> 1)];
-        }
+  const bool bad = slot >= static_cast<long long>(s.num_blocks) * s.block_size;
+  if (bad && tid == 0 && status) atomicCAS(status, 0, RLB_ERR_BOUNDS);
+  T* cr = cache + slot * s.width;
+  if (slot >= 0 && !bad) {
+    for (int j = tid; j < s.width - s.rank; j += 128) {      // rotated key part, then padding
+      float v = j < s.rot_dim ? ld(lat + s.rank + j) : 0.f;
+      if (j < 2 * half) {
+        float sn, c;
+        sincosf(pos * freq[j >> 1], &sn, &c);
+        const float o = ld(lat + s.rank + (j ^ 1));
+        v = ((j & 1) ? v * c + o * sn : v * c - o * sn) * gain;
       }
-      st(cr + r, v);
+      st(cr + s.rank + j, v);
     }
   }
-  const int qd = s.dim + s.rot_dim;
-  for (int i = threadIdx.x; i < s.heads * half; i += blockDim.x) {
-    T* q = pr + s.q_off + (i / half) * qd + s.dim + 2 * (i % half);
-    const float c = cs[i % half], sn = cs[half + i % half], u = ld(q), v = ld(q + 1);
-    st(q, u * c - v * sn);
-    st(q + 1, v * c + u * sn);
+  ss = block_sum(ss, red);
+  if (slot < 0 || bad) return;
+  const float rstd = 1.f / sqrtf(ss / static_cast<float>(s.rank) + eps);
+#pragma unroll
+  for (int k = 0; k < LP_KEEP; ++k) {
+    const int r = tid + k * 128;
+    if (r < s.rank) st(cr + r, keep[k] * rstd * ld(norm_w + r));
   }
-  if (q_lat && row < q_rows) {
-    __syncthreads();
-    const int tail = s.width - s.rank;
-    for (int i = threadIdx.x; i < s.heads * tail; i += blockDim.x) {
-      const int h = i / tail, j = i % tail;
-      st(q_lat + (row * s.heads + h) * s.width + s.rank + j, j < s.rot_dim ? ld(pr + s.q_off + h * qd + s.dim + j) : 0.f);
-    }
-  }
+  for (int r = tid + LP_KEEP * 128; r < s.rank; r += 128) st(cr + r, ld(lat + r) * rstd * ld(norm_w + r));
 }
 
 // One CTA per (row, head): the query is carried into the latent space (q^T W_uk), the keys are the cached rows, the weighted
@@ -412,14 +431,13 @@ RLB_API int rlb_latent_prep(void* p, int f32, long long rows, long long ldp, int
   if (rows <= 0) return 0;
   if (2 * half > rot_dim || rank + rot_dim > width) return -2;
   LatentShape s{ldp, q_off, lat_off, 0, heads, dim, rot_dim, 0, rank, width, block_size, num_blocks};
-  const size_t sm = sizeof(float) * 2 * (half + 1);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const dim3 grid(static_cast<unsigned>(rows)), block(rows > 1024 ? 128 : 256);
+  const dim3 grid(static_cast<unsigned>(rows), 2), block(128);
   if (f32)
-    rlb_launch_pdl(latent_prep_kernel<float>, grid, block, sm, st, static_cast<float*>(p), s, positions, slots, static_cast<const float*>(norm_w),
+    rlb_launch_pdl(latent_prep_kernel<float>, grid, block, 0, st, static_cast<float*>(p), s, positions, slots, static_cast<const float*>(norm_w),
                                                                             freq, half, gain, eps, static_cast<float*>(cache), static_cast<float*>(q_lat), q_rows, status);
   else
-    rlb_launch_pdl(latent_prep_kernel<__nv_bfloat16>, grid, block, sm, st, static_cast<__nv_bfloat16*>(p), s, positions, slots,
+    rlb_launch_pdl(latent_prep_kernel<__nv_bfloat16>, grid, block, 0, st, static_cast<__nv_bfloat16*>(p), s, positions, slots,
         static_cast<const __nv_bfloat16*>(norm_w), freq, half, gain, eps, static_cast<__nv_bfloat16*>(cache),
         static_cast<__nv_bfloat16*>(q_lat), q_rows, status);
   return static_cast<int>(cudaGetLastError());
