@@ -337,15 +337,16 @@ def test_trace_runner(tmp_path, monkeypatch, capsys):
     assert G.gap(read(2), torch.stack([zb[8], za[20]])) < TOL
 
 
-def test_trace_runner_serves_other_families(tmp_path, monkeypatch):
+@pytest.mark.parametrize("family", ["llama", "nemotron_h"])
+def test_step_serves_other_families(family):
     """The same step function drives the other model families (whole prompts, portions and single tokens in one batch)."""
-    mc = ModelConfig(vocab_size=97, hidden_size=32, intermediate_size=64, num_hidden_layers=2, num_attention_heads=4, num_key_value_heads=2,
-                     head_dim=8, torch_dtype="float32")
+    mc = preset("tiny-nemotron-h") if family == "nemotron_h" else ModelConfig(
+        vocab_size=97, hidden_size=32, intermediate_size=64, num_hidden_layers=2, num_attention_heads=4, num_key_value_heads=2, head_dim=8)
     m = build_model(mc, seed=1, dtype=torch.float32)
     eng = G.engine(m, pages=12)
-    seqs = {"a": torch.randint(0, 97, (30,)).tolist(), "b": torch.randint(0, 97, (23,)).tolist()}
+    seqs = {"a": G.tokens({"vocab": mc.vocab_size}, 30, 1), "b": G.tokens({"vocab": mc.vocab_size}, 23, 2)}
     got = G.run_schedule(eng, [{"a": 17}, {"a": 1, "b": 9}, {"b": 1, "a": 2}, {"a": 10, "b": 13}], seqs)
     for r, t in seqs.items():
         n = len(t)
         z = m.logits(PackedBatch(torch.tensor(t), torch.arange(n).int(), torch.tensor([0, n], dtype=torch.int32), n)).detach()
-        assert (got[r] - z).abs().max() < 1e-4
+        assert (got[r] - z).abs().max() < 1e-3 * z.abs().max()

@@ -158,7 +158,7 @@ def latent_outputs(H, dim, rot, vdim, R, lens, news, bs):
     return run(False, True), run(False, False), run(True, False)
 
 
-@pytest.mark.parametrize("shape", [(8, 32, 16, 32, 136, [300, 77, 5, 129, 640], [1, 77, 5, 100, 17], 64),
+@pytest.mark.parametrize("shape", [(9, 32, 24, 40, 136, [300, 77, 5, 129, 640], [1, 77, 5, 100, 17], 64),
                                    (16, 128, 64, 128, 512, [1000, 200, 130, 129, 1], [1, 200, 128, 2, 1], 64),
                                    (4, 48, 8, 40, 72, [300, 77, 70], [1, 77, 33], 64),
                                    (40, 64, 32, 96, 256, [300, 1000, 70], [300, 1, 33], 32),
@@ -173,7 +173,7 @@ def test_latent_kernels(shape):
 
 
 @pytest.mark.parametrize("H,dim,vdim,rd,lens,starts,decay", [
-    (6, 64, 32, 64, [1, 2, 100, 300, 128, 1], [5, 0, 77, 0, 128, 0], None), (4, 128, 128, 128, [1, 129, 1000], [0, 0, 300], None),
+    (5, 64, 48, 64, [1, 2, 100, 300, 128, 1], [5, 0, 77, 0, 128, 0], None), (4, 128, 128, 128, [1, 129, 1000], [0, 0, 300], None),
     (2, 256, 256, 256, [1, 129, 400], [9, 0, 300], None), (3, 40, 24, 12, [1, 17, 140, 3], [9, 0, 300, 4], None),
     (5, 72, 136, 72, [260, 64], [0, 64], [1.0, 0.5, 0.25, 0.999, 0.9]), (2, 8, 8, 0, [5, 1], [3, 0], [0.75, 0.5])])
 def test_retention_kernels(H, dim, vdim, rd, lens, starts, decay):
