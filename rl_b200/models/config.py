@@ -5,8 +5,10 @@ One dataclass covers Llama (2/3/3.1/3.2), Mistral, Qwen2/2.5, Qwen3, Qwen3-MoE a
 before and after each block, scaled embeddings, sliding-window layers with their own RoPE base, a fixed attention scale). ``from_hf_dict`` reads a
 HuggingFace ``config.json`` dictionary; ``PRESETS`` names the architectures used by the benchmark configs.
 
-Models described layer by layer (Gadarax) keep their layer list in ``mixers``: each entry names the sequence mixer, its sizes and its
-MLP; ``layer_loop`` runs a range of layers several times with the same weights.
+Models described layer by layer (Gadarax, Redarax) keep their layer list in ``mixers``: each entry names the sequence mixer, its sizes
+and its MLP. ``LAYER_LISTS`` says which mixers and MLPs each architecture has and how its configuration maps to ``ModelConfig``:
+Gadarax runs mixer and MLP side by side behind one norm (``layer_loop`` repeats a range of layers with the same weights), Redarax runs
+them one after the other and norms what they return (``norm_place`` "post"), with an input per layer and token (``token_side``).
 """
 
 from __future__ import annotations
@@ -59,7 +61,7 @@ class ModelConfig:
     layer_types: Optional[list] = None  # per layer: "full_attention" | "sliding_attention"
     rope_local_theta: float = 0.0      # RoPE base of the sliding-window layers (0: same as rope_theta, scaling included)
     attn_scale: Optional[float] = None  # softmax scale when it is not head_dim ** -0.5 (query_pre_attn_scalar ** -0.5)
-    final_logit_softcap: float = 0.0   # logits <- cap * tanh(logits / cap) (Gemma 2; 0: off)
+    final_logit_softcap: float = 0.0   # logits <- cap * tanh(logits / cap) (Gemma 2, Redarax; 0: off)
 
     # DeepSeek-V3: multi-head latent attention and its mixture of experts
     kv_lora_rank: int = 0              # > 0: attention is MLA (keys / values decompressed from a latent of this width)
@@ -93,10 +95,14 @@ class ModelConfig:
     moe_latent_size: Optional[int] = None      # routed experts work in a narrower space between two shared projections
     moe_shared_expert_intermediate_size: int = 0
 
-    # Gadarax: every layer is one norm whose output feeds a sequence mixer and an MLP side by side; the layers differ
-    mixers: Optional[list] = None      # per layer: {"type": "latent_attention" | "retention", "mixer": {sizes}, "mlp": {"kind", "ff"} or None}
+    # models described layer by layer (Gadarax, Redarax): the layers differ in their mixers, sizes and MLPs
+    mixers: Optional[list] = None      # per layer: {"type": name of the mixer, "mixer": {sizes}, "mlp": {"kind", sizes} or None}
     layer_loop: Optional[dict] = None  # {"start", "stop", "times"}: layers start .. stop - 1 run `times` times in a row with the same weights
     norm_kind: str = "rms"             # "rms" | "dyt" (dynamic tanh: w * tanh(alpha x) + b, no statistics)
+    norm_place: str = "pre"            # "pre": sublayers read norm(x); "post": they read x, and norm(output) joins the residual stream
+    residual_mult: float = 1.0         # what sublayer outputs are multiplied by when they join the residual stream
+    token_side: Optional[dict] = None  # {"dim"}: every layer adds an input looked up by token in a table of its own (gated by the stream)
+    logit_scale: float = 1.0           # logits are multiplied by this (before the soft cap)
 
     @property
     def is_hybrid(self) -> bool:
@@ -109,7 +115,12 @@ class ModelConfig:
     @property
     def is_recurrent(self) -> bool:
         """Some layer carries a per-sequence state beside (or instead of) cache pages: prefixes cannot be shared by pages."""
-        return self.is_hybrid or (self.mixers is not None and any(m["type"] == "retention" for m in self.mixers))
+        return self.is_hybrid or (self.mixers is not None and any(m["type"] in RECURRENT_MIXERS for m in self.mixers))
+
+    @property
+    def caps_logits(self) -> bool:
+        """Logits are more than the product with the output weight (a scale or a soft cap follows)."""
+        return self.logit_scale != 1.0 or bool(self.final_logit_softcap)
 
     @property
     def layer_runs(self) -> list:
@@ -162,6 +173,27 @@ class ModelConfig:
 
     def num_parameters(self) -> int:
         d, L = self.hidden_size, self.num_hidden_layers
+        if self.model_type == "redarax":
+            sd = self.token_side["dim"] if self.token_side else 0
+            n = 2 * self.vocab_size * d + d + self.vocab_size * L * sd
+            for e in self.mixers:
+                m, mlp = e["mixer"], e.get("mlp")
+                H, vd = m["heads"], m["vdim"]
+                if e["type"] == "attention":
+                    G, kd = m["kv_heads"], m["dim"]
+                    n += (d + 1) * (H * kd + G * kd + G * vd) + 2 * kd + (H * vd + 1) * d
+                elif e["type"] == "mamba2":
+                    C = H * vd + 2 * m["groups"] * m["state"]
+                    n += d * (H * vd + C + H) + C * (m["conv"] + 1) + 3 * H + H * vd + H * vd * d
+                else:
+                    C = 2 * m["kv_heads"] * m["dim"] + H * vd
+                    n += d * (C + 2 * H + 2 * H * vd) + C * m["conv"] + 2 * H + vd
+                n += d
+                if mlp:
+                    r = mlp.get("router")
+                    n += d + (r["experts"] * (3 * d * mlp["expert"]["ff"] + d + 1) if r else 3 * d * mlp["ff"])
+                n += 2 * d * sd + (d if sd else 0)
+            return n
         if self.mixers is not None:
             n = self.vocab_size * d + 2 * d + 1 + (self.layer_loop["times"] * d if self.layer_loop else 0)
             for e in self.mixers:
@@ -193,6 +225,12 @@ class ModelConfig:
         return L * (attn + ffn + norms) + emb + d
 
     def to_hf_dict(self) -> dict:
+        if self.model_type == "redarax":
+            out = {"architecture": "Redarax", "vocab": self.vocab_size, "width": self.hidden_size, "norm": {"eps": self.rms_norm_eps},
+                   "residual_mult": self.residual_mult, "logit_scale": self.logit_scale, "layers": self.mixers, "torch_dtype": self.torch_dtype}
+            if self.token_side:
+                out["token_side"] = self.token_side
+            return dict(out, logit_softcap=self.final_logit_softcap) if self.final_logit_softcap else out
         if self.is_mixer:
             out = {"architecture": "Gadarax", "vocab": self.vocab_size, "width": self.hidden_size, "embedding": {"scale": self.embed_scale},
                    "norm": {"eps": self.rms_norm_eps}, "layers": self.mixers, "torch_dtype": self.torch_dtype}
@@ -202,7 +240,7 @@ class ModelConfig:
                 "gemma3_text": "Gemma3ForCausalLM", "deepseek_v3": "DeepseekV3ForCausalLM",
                 "nemotron_h": "NemotronHForCausalLM"}.get(self.model_type, "LlamaForCausalLM")
         d = asdict(self)
-        for k in ("mixers", "layer_loop", "norm_kind"):
+        for k in ("mixers", "layer_loop", "norm_kind", "norm_place", "residual_mult", "token_side", "logit_scale"):
             d.pop(k)
         nh = {k: d.pop(k) for k in ("layers_block_type", "use_rope", "mlp_gated", "mlp_bias", "mamba_num_heads", "mamba_head_dim", "ssm_state_size",
                                     "mamba_n_groups", "mamba_d_conv", "mamba_chunk_size", "mamba_conv_bias", "mamba_proj_bias", "mamba_dt_limit",
@@ -244,7 +282,7 @@ class ModelConfig:
 
     @classmethod
     def from_hf_dict(cls, hf: dict, **overrides) -> "ModelConfig":
-        if hf.get("architecture") == "Gadarax":
+        if hf.get("architecture") in LAYER_LISTS:
             return cls._from_layer_list(hf, **overrides)
         mt = hf.get("model_type", "llama")
         if mt == "gemma3" and "text_config" in hf:      # the multimodal wrapper: the language model's settings are nested
@@ -353,33 +391,31 @@ class ModelConfig:
 
     @classmethod
     def _from_layer_list(cls, hf: dict, **overrides) -> "ModelConfig":
-        """Configurations that describe the model layer by layer (Gadarax)."""
-        layers = hf["layers"]
+        """Configurations that describe the model layer by layer (``LAYER_LISTS``)."""
+        layers, (mixers, mlps, settings) = hf["layers"], LAYER_LISTS[hf["architecture"]]
         for i, e in enumerate(layers):
-            need = {"latent_attention": ("heads", "dim", "rot_dim", "vdim", "kv_rank", "scale", "rot"),
-                    "retention": ("heads", "dim", "vdim", "decay", "rot")}.get(e["type"])
+            need = MIXER_SIZES[e["type"]] if e["type"] in mixers else None
             if need is None:
                 raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
             missing = [k for k in need if k not in e["mixer"]]
             if missing:
                 raise ValueError(f"layer {i}: the {e['type']} mixer lacks {missing}")
-            if e.get("mlp") and e["mlp"].get("kind", "dense") != "dense":
+            if e.get("mlp") and e["mlp"].get("kind", "dense") not in mlps:
                 raise ValueError(f"layer {i}: unknown MLP kind {e['mlp']['kind']!r}")
-            m = e["mixer"]
-            if e["type"] == "retention" and len(m["decay"]) != m["heads"]:
-                raise ValueError(f"layer {i}: {len(m['decay'])} decays for {m['heads']} heads")
-            limit = m["rot_dim"] if e["type"] == "latent_attention" else m["dim"]
-            if m["rot"]["dims"] > limit or m["rot"]["dims"] % 2:
-                raise ValueError(f"layer {i}: {m['rot']['dims']} rotated dimensions in a part of {limit}")
+            _check_mixer(i, e["type"], e["mixer"])
+            if e.get("mlp") and e["mlp"].get("kind") == "moe":
+                r = e["mlp"]["router"]
+                g = r.get("groups") or {"count": 1, "keep": 1}
+                if r["experts"] % g["count"] or not 1 <= g["keep"] <= g["count"] or not 1 <= r["top"] <= g["keep"] * (r["experts"] // g["count"]):
+                    raise ValueError(f"layer {i}: router {r} does not fit its groups")
         lp = hf.get("loop")
         if lp and not (0 <= lp["start"] < lp["stop"] <= len(layers) and lp["times"] >= 1):
             raise ValueError(f"layer loop {lp} does not fit {len(layers)} layers")
         m0 = layers[0]["mixer"]
-        cfg = cls(model_type="gadarax", vocab_size=hf["vocab"], hidden_size=hf["width"], num_hidden_layers=len(layers),
-                  intermediate_size=max([e["mlp"]["ff"] for e in layers if e.get("mlp")] or [0]), num_attention_heads=m0["heads"],
-                  num_key_value_heads=m0["heads"], head_dim=m0["dim"], rms_norm_eps=float(hf["norm"]["eps"]), tie_word_embeddings=True,
-                  mlp_gated=False, hidden_act="relu2", embed_scale=float(hf["embedding"]["scale"]), norm_kind="dyt", mixers=layers,
-                  layer_loop=dict(lp) if lp else None, torch_dtype=str(hf.get("torch_dtype", "bfloat16")).replace("torch.", ""))
+        cfg = cls(vocab_size=hf["vocab"], hidden_size=hf["width"], num_hidden_layers=len(layers),
+                  intermediate_size=max([_ff_width(e["mlp"]) for e in layers if e.get("mlp")] or [0]), num_attention_heads=m0["heads"],
+                  num_key_value_heads=m0["heads"], head_dim=m0.get("dim", m0["vdim"]), rms_norm_eps=float(hf["norm"]["eps"]), mixers=layers,
+                  layer_loop=dict(lp) if lp else None, torch_dtype=str(hf.get("torch_dtype", "bfloat16")).replace("torch.", ""), **settings(hf))
         for k, v in overrides.items():
             setattr(cfg, k, v)
         return cfg
@@ -393,6 +429,51 @@ class ModelConfig:
         os.makedirs(path, exist_ok=True)
         with open(os.path.join(path, "config.json"), "w") as f:
             json.dump(self.to_hf_dict(), f, indent=2)
+
+
+# what a mixer's description must name
+MIXER_SIZES = {
+    "latent_attention": ("heads", "dim", "rot_dim", "vdim", "kv_rank", "scale", "rot"),
+    "retention": ("heads", "dim", "vdim", "decay", "rot"),
+    "attention": ("heads", "kv_heads", "dim", "vdim", "scale", "rot"),
+    "mamba2": ("heads", "vdim", "state", "groups", "norm_groups", "conv"),
+    "delta": ("heads", "kv_heads", "dim", "vdim", "conv"),
+}
+RECURRENT_MIXERS = ("retention", "mamba2", "delta")
+
+
+def _check_mixer(i: int, kind: str, m: dict) -> None:
+    if kind == "retention" and len(m["decay"]) != m["heads"]:
+        raise ValueError(f"layer {i}: {len(m['decay'])} decays for {m['heads']} heads")
+    if "rot" in m:
+        limit = m["rot_dim"] if kind == "latent_attention" else m["dim"]
+        if m["rot"]["dims"] > limit or m["rot"]["dims"] % 2:
+            raise ValueError(f"layer {i}: {m['rot']['dims']} rotated dimensions in a part of {limit}")
+    for part in ("kv_heads", "groups"):
+        if part in m and m["heads"] % m[part]:
+            raise ValueError(f"layer {i}: {m['heads']} heads do not divide into {m[part]} {part}")
+    if "norm_groups" in m and (m["heads"] * m["vdim"]) % m["norm_groups"]:
+        raise ValueError(f"layer {i}: {m['heads'] * m['vdim']} channels do not divide into {m['norm_groups']} norm groups")
+    if m.get("conv", 1) < 1:
+        raise ValueError(f"layer {i}: a convolution needs at least one tap")
+
+
+def _ff_width(mlp: dict) -> int:
+    return mlp["expert"]["ff"] if mlp.get("kind") == "moe" else mlp["ff"]
+
+
+def _gadarax(hf: dict) -> dict:
+    return dict(model_type="gadarax", tie_word_embeddings=True, mlp_gated=False, hidden_act="relu2", embed_scale=float(hf["embedding"]["scale"]), norm_kind="dyt")
+
+
+def _redarax(hf: dict) -> dict:
+    return dict(model_type="redarax", norm_place="post", residual_mult=float(hf["residual_mult"]), logit_scale=float(hf["logit_scale"]),
+                final_logit_softcap=float(hf.get("logit_softcap") or 0.0), token_side=dict(hf["token_side"]) if hf.get("token_side") else None)
+
+
+# architecture -> (its mixers, its kinds of MLP, configuration -> further ModelConfig fields)
+LAYER_LISTS = {"Gadarax": (("latent_attention", "retention"), ("dense",), _gadarax),
+               "Redarax": (("attention", "mamba2", "delta"), ("dense", "moe"), _redarax)}
 
 
 def rope_inv_freq(cfg: ModelConfig, device=None) -> torch.Tensor:
@@ -463,7 +544,29 @@ def _layer_list(width: int, ff: int, latent: dict, retention: dict, kinds: str, 
                 layer_loop=loop)
 
 
+def _redarax_preset(width: int, kinds: str, attention: dict, mamba2: dict, delta: dict, ff: int, moe: dict, side: int, vocab: int) -> dict:
+    """Preset of a post-norm layer-list model: ``kinds`` has two letters per layer, the mixer (A attention, M Mamba-2, D delta rule) and the
+    feed-forward (d dense, e experts, - none)."""
+    mix = {"A": ("attention", dict(attention, scale=attention["dim"] ** -0.5)), "M": ("mamba2", mamba2), "D": ("delta", delta)}
+    mlp = {"d": {"kind": "dense", "ff": ff, "limit": 7.0}, "e": dict(moe, kind="moe"), "-": None}
+    layers = [{"type": mix[k][0], "mixer": mix[k][1], "mlp": mlp[f]} for k, f in zip(kinds[::2], kinds[1::2])]
+    m0 = layers[0]["mixer"]
+    return dict(model_type="redarax", vocab_size=vocab, hidden_size=width, num_hidden_layers=len(layers), intermediate_size=max(ff, moe["expert"]["ff"]),
+                num_attention_heads=m0["heads"], num_key_value_heads=m0["heads"], head_dim=m0.get("dim", m0["vdim"]), rms_norm_eps=1e-6, mixers=layers,
+                norm_place="post", residual_mult=0.5, logit_scale=0.5, final_logit_softcap=30.0, token_side={"dim": side} if side else None)
+
+
 PRESETS: dict[str, dict] = {
+    # Redarax at the size of small production models: delta-rule, Mamba-2 and grouped-query attention layers, dense and expert feed-forwards
+    "redarax-2b": _redarax_preset(2048, "DdDeMeAeDdDeMeAe", dict(heads=16, kv_heads=4, dim=128, vdim=128, rot={"dims": 64, "base": 1e6}),
+                                  dict(heads=32, vdim=128, state=128, groups=4, norm_groups=4, conv=4), dict(heads=16, kv_heads=8, dim=128, vdim=128, conv=4),
+                                  6144, dict(expert={"ff": 768, "limit": 7.0}, router={"experts": 64, "top": 8, "groups": {"count": 8, "keep": 4}}), 256, 65536),
+    "redarax-7b": _redarax_preset(4096, "DdDeMeAeDdDeMeAe", dict(heads=32, kv_heads=8, dim=128, vdim=128, rot={"dims": 64, "base": 1e6}),
+                                  dict(heads=64, vdim=128, state=128, groups=8, norm_groups=8, conv=4), dict(heads=32, kv_heads=16, dim=128, vdim=128, conv=4),
+                                  12288, dict(expert={"ff": 1536, "limit": 7.0}, router={"experts": 64, "top": 8, "groups": {"count": 8, "keep": 4}}), 256, 65536),
+    "tiny-redarax": _redarax_preset(96, "MeDdAeD-", dict(heads=4, kv_heads=2, dim=24, vdim=16, rot={"dims": 16, "base": 1e4}),
+                                    dict(heads=6, vdim=16, state=24, groups=2, norm_groups=3, conv=3), dict(heads=4, kv_heads=2, dim=16, vdim=24, conv=4),
+                                    160, dict(expert={"ff": 48, "limit": 2.0}, router={"experts": 8, "top": 2, "groups": {"count": 4, "keep": 2}}), 8, 264),
     # Gadarax at the size of small production models: latent attention and retention layers, three of them looped twice
     "gadarax-1b": _layer_list(2048, 8192, dict(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512), dict(heads=16, dim=128, vdim=128),
                               "AARARARARARA", dict(start=1, stop=4, times=2), 65536),

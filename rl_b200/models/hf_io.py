@@ -175,13 +175,20 @@ def _model_map(model: CausalLM):
 def iter_hf_shards(model: CausalLM) -> Iterator[tuple[str, torch.Tensor, Optional[tuple[int, int, int]]]]:
     """Yields (hf_name, local tensor view, hf_slice) for every logical HF tensor (or shard of one) this rank holds."""
     cfg = model.cfg
-    if cfg.is_mixer:    # layer-list models (Gadarax) keep their checkpoint's own tensor names
+    if cfg.is_mixer:    # layer-list models (Gadarax, Redarax) keep their checkpoint's own tensor names
         yield "embed", model.embed_tokens, None
+        if model.side_embed is not None:
+            yield "side.embed", model.side_embed, None
         if model.loop_step is not None:
             yield "loop.step", model.loop_step, None
         for i, layer in enumerate(model.layers):
             for name, view in layer.tensor_views(f"l{i}."):
                 yield name, view, None
+        if model.lm_head is not None:
+            yield "head", model.lm_head, None
+        if cfg.norm_kind == "rms":
+            yield "final.norm", model.norm, None
+            return
         yield "final.norm", model.norm.weight, None
         yield "final.norm.b", model.norm.bias, None
         yield "final.norm.alpha", model.norm.alpha, None

@@ -23,6 +23,7 @@ chunked-scan kernel is not written); the reference reaches the same math through
 
 from __future__ import annotations
 
+import math
 from typing import Optional
 
 import torch
@@ -122,6 +123,17 @@ def _proj(x: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor]) -> torch.
     return TF.linear(x, w, b)
 
 
+@torch.no_grad()
+def init_decay(A_log: torch.Tensor, dt_bias: torch.Tensor, gen: torch.Generator, dt_min: float = 1e-3, dt_max: float = 0.1,
+               dt_floor: float = 1e-4) -> None:
+    """Decay rates 1..H and step sizes log-uniform in [dt_min, dt_max], stored through the inverse of softplus."""
+    H = A_log.numel()
+    A_log.copy_(torch.arange(1, H + 1, dtype=torch.float32).log())
+    u = torch.rand(H, generator=gen, device=dt_bias.device, dtype=torch.float32)
+    dt = (u * (math.log(dt_max) - math.log(dt_min)) + math.log(dt_min)).exp().clamp(min=dt_floor)
+    dt_bias.copy_(dt + torch.log(-torch.expm1(-dt)))
+
+
 class Mamba2Mixer(nn.Module):
     """Parameters in the HuggingFace layout: ``in_proj`` rows are [gate | x | B | C | dt]."""
 
@@ -209,14 +221,8 @@ class Mamba2Mixer(nn.Module):
     def reset_special(self, gen: torch.Generator, dt_min: float = 1e-3, dt_max: float = 0.1, dt_floor: float = 1e-4) -> None:
         """The initial values that are not plain normal draws: decay rates 1..H, unit skip, step sizes log-uniform in
         [dt_min, dt_max] (stored through the inverse of softplus)."""
-        H = self.cfg.mamba_num_heads
-        self.A_log.copy_(torch.arange(1, H + 1, dtype=torch.float32).log())
+        init_decay(self.A_log, self.dt_bias, gen, dt_min, dt_max, dt_floor)
         self.D.fill_(1.0)
         self.norm.fill_(1.0)
-        import math
-
-        u = torch.rand(H, generator=gen, device=self.dt_bias.device, dtype=torch.float32)
-        dt = (u * (math.log(dt_max) - math.log(dt_min)) + math.log(dt_min)).exp().clamp(min=dt_floor)
-        self.dt_bias.copy_(dt + torch.log(-torch.expm1(-dt)))
         if self.conv_bias is not None:
             self.conv_bias.zero_()

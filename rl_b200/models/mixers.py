@@ -1,4 +1,5 @@
-"""Sequence mixers that sit beside an MLP in one parallel layer, and that layer.
+"""Sequence mixers of models that are described layer by layer, and the parallel layer (mixer and MLP side by side); the layer whose
+sublayers run one after the other is in ``post_norm.py``.
 
 A parallel layer computes ``h = norm(x)`` once and adds ``mixer(h) + mlp(h)`` to the residual stream, so all its input projections
 read the same rows and both its output projections write the same rows. The layer therefore holds two fused weights:
@@ -14,9 +15,13 @@ Mixers:
     the latent and a rotated key part shared by the heads are cached. Own softmax scale, output gate, interleaved rotation.
   * ``RetentionMixer``: linear attention with one fixed decay per head, a unit-RMS norm per head and a SiLU gate. The state
     [heads, dim, vdim] is fp32.
+  * ``GroupedAttentionMixer``: causal attention with fewer key / value heads than query heads, biases, RMS norms per head on queries and
+    keys, interleaved partial rotation, own scale, keys and values of unequal size.
+  * ``Mamba2LayerMixer``: state-space duality with a short convolution in front and a gated norm in equal parts behind.
+  * ``DeltaMixer``: gated delta rule: a linear-attention state that forgets by a decay per token and corrects what it stores under a key.
 
 The modules' ``sequence`` methods are the differentiable PyTorch statement over packed sequences (training, CPU); the generation
-engine runs the same weights through ``rl_b200/ops/mixer_ops.py``.
+engine runs the same weights through ``rl_b200/ops/mixer_ops.py`` (latent attention, retention) and ``rl_b200/ops/sequence_ops.py``.
 """
 
 from __future__ import annotations
@@ -28,6 +33,7 @@ import torch.nn.functional as TF
 from rl_b200.ops import functional as F
 
 from .config import ModelConfig, rotary_table
+from .mamba import gated_group_norm, init_decay, ssd_scan
 
 
 def pad8(n: int) -> int:
@@ -189,7 +195,205 @@ class RetentionMixer(nn.Module):
         return self.finish(torch.cat([self.scan(q[s:e], k[s:e], v[s:e], zero)[0] for s, e in zip(cu[:-1], cu[1:])]), p)
 
 
-MIXERS = {m.kind: m for m in (LatentAttentionMixer, RetentionMixer)}
+def rms_unit(x: torch.Tensor, eps: float) -> torch.Tensor:
+    return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+
+
+class GroupedAttentionMixer(nn.Module):
+    kind = "attention"
+
+    def __init__(self, spec: dict, cfg: ModelConfig, dtype, device):
+        super().__init__()
+        self.heads, self.kv_heads, self.dim, self.vdim = spec["heads"], spec["kv_heads"], spec["dim"], spec["vdim"]
+        self.scale, self.eps = float(spec["scale"]), cfg.rms_norm_eps
+        self.q_off, self.k_off = 0, pad8(self.heads * self.dim)
+        self.v_off = self.k_off + pad8(self.kv_heads * self.dim)
+        self.in_width = self.v_off + pad8(self.kv_heads * self.vdim)
+        self.mix_width = pad8(self.heads * self.vdim)
+        d = cfg.hidden_size
+        self.in_proj = nn.Parameter(torch.zeros(self.in_width, d, dtype=dtype, device=device))
+        self.in_bias = nn.Parameter(torch.zeros(self.in_width, dtype=dtype, device=device))
+        self.out_proj = nn.Parameter(torch.zeros(d, self.mix_width, dtype=dtype, device=device))
+        self.out_bias = nn.Parameter(torch.zeros(d, dtype=dtype, device=device))
+        self.q_norm = nn.Parameter(torch.ones(self.dim, dtype=dtype, device=device))
+        self.k_norm = nn.Parameter(torch.ones(self.dim, dtype=dtype, device=device))
+        freq, self.gain = rotary_table(spec["rot"])
+        self.register_buffer("freq", freq.to(device), persistent=False)
+
+    def tensors(self) -> list:
+        """(checkpoint leaf, view of a parameter)."""
+        out = []
+        for leaf, r, n in (("q", self.q_off, self.heads * self.dim), ("k", self.k_off, self.kv_heads * self.dim), ("v", self.v_off, self.kv_heads * self.vdim)):
+            out += [(leaf, self.in_proj[r : r + n]), (leaf + ".b", self.in_bias[r : r + n])]
+        return out + [("q.norm", self.q_norm), ("k.norm", self.k_norm), ("o", self.out_proj[:, : self.heads * self.vdim]), ("o.b", self.out_bias)]
+
+    def qkv(self, p: torch.Tensor, positions: torch.Tensor):
+        """fp32 normed and rotated queries [T, heads, dim] and keys [T, kv_heads, dim], values [T, kv_heads, vdim]."""
+        q = p[:, self.q_off : self.q_off + self.heads * self.dim].reshape(-1, self.heads, self.dim).float()
+        k = p[:, self.k_off : self.k_off + self.kv_heads * self.dim].reshape(-1, self.kv_heads, self.dim).float()
+        v = p[:, self.v_off : self.v_off + self.kv_heads * self.vdim].reshape(-1, self.kv_heads, self.vdim).float()
+        q = rotate_pairs(rms_unit(q, self.eps) * self.q_norm.float(), positions, self.freq, self.gain, True)
+        k = rotate_pairs(rms_unit(k, self.eps) * self.k_norm.float(), positions, self.freq, self.gain, True)
+        return q, k, v
+
+    def sequence(self, p: torch.Tensor, positions: torch.Tensor, cu_seqlens: torch.Tensor) -> torch.Tensor:
+        """Head outputs [T, heads * vdim] of packed whole sequences."""
+        q, k, v = self.qkv(p, positions)
+        n = self.heads // self.kv_heads
+        k, v = k.repeat_interleave(n, dim=1), v.repeat_interleave(n, dim=1)
+        out = []
+        cu = cu_seqlens.tolist()
+        for s, e in zip(cu[:-1], cu[1:]):
+            z = torch.einsum("ihd,jhd->hij", q[s:e], k[s:e]) * self.scale
+            z = z.masked_fill(torch.ones(e - s, e - s, dtype=torch.bool, device=z.device).triu(1), float("-inf"))
+            out.append(torch.einsum("hij,jhd->ihd", torch.softmax(z, -1), v[s:e]))
+        return torch.cat(out).reshape(-1, self.heads * self.vdim).to(p.dtype)
+
+
+class RecurrentMixer(nn.Module):
+    """What the mixers with a short convolution and a state per sequence share: the convolved channels are one column range of the
+    projected rows, [conv_off, conv_off + channels), and the state is [heads, dim, vdim] in fp32."""
+
+    in_bias = out_bias = None
+
+    def piece_bounds(self, cu_seqlens: torch.Tensor) -> list:
+        cu = cu_seqlens.tolist()
+        return list(zip(cu[:-1], cu[1:]))
+
+    def convolve(self, x: torch.Tensor, before: torch.Tensor) -> torch.Tensor:
+        """silu of the causal convolution of one sequence piece's rows [L, channels]; ``before`` [taps - 1, channels] stood in front."""
+        L, n = x.shape[0], self.taps
+        xp = torch.cat([before.to(x.dtype), x]).float()
+        y = sum(xp[j : j + L] * self.conv[:, j].float() for j in range(n))
+        if self.conv_bias is not None:
+            y = y + self.conv_bias.float()
+        return TF.silu(y).to(x.dtype)
+
+    def sequence(self, p: torch.Tensor, positions: torch.Tensor, cu_seqlens: torch.Tensor) -> torch.Tensor:
+        """Mixer outputs (before the output product) of packed whole sequences."""
+        out = []
+        for s, e in self.piece_bounds(cu_seqlens):
+            u = self.convolve(p[s:e, self.conv_off : self.conv_off + self.channels], p.new_zeros(self.taps - 1, self.channels))
+            zero = torch.zeros(self.heads, self.dim, self.vdim, dtype=torch.float32, device=p.device)
+            out.append(self.finish(self.scan(u, p[s:e], zero)[0], p[s:e]))
+        return torch.cat(out)
+
+
+class Mamba2LayerMixer(RecurrentMixer):
+    """S <- exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x per head; dt = softplus(projection + dt_bias). Heads in equal runs share a
+    group's B and C. ``dim`` is the state width."""
+
+    kind = "mamba2"
+
+    def __init__(self, spec: dict, cfg: ModelConfig, dtype, device):
+        super().__init__()
+        self.heads, self.vdim, self.dim, self.groups = spec["heads"], spec["vdim"], spec["state"], spec["groups"]
+        self.norm_groups, self.taps, self.eps = spec["norm_groups"], spec["conv"], cfg.rms_norm_eps
+        self.inner = self.heads * self.vdim
+        self.channels = self.inner + 2 * self.groups * self.dim
+        self.z_off, self.conv_off, self.dt_off = 0, self.inner, self.inner + self.channels      # (one checkpoint tensor: no padding between)
+        self.in_width, self.mix_width = pad8(self.dt_off + self.heads), pad8(self.inner)
+        P = lambda *shape: nn.Parameter(torch.zeros(*shape, dtype=dtype, device=device))   # noqa: E731
+        self.in_proj, self.out_proj = P(self.in_width, cfg.hidden_size), P(cfg.hidden_size, self.mix_width)
+        self.conv, self.conv_bias = P(self.channels, self.taps), P(self.channels)
+        self.A_log, self.dt_bias, self.D = P(self.heads), P(self.heads), nn.Parameter(torch.ones(self.heads, dtype=dtype, device=device))
+        self.norm = nn.Parameter(torch.ones(self.inner, dtype=dtype, device=device))
+
+    def tensors(self) -> list:
+        return [("in", self.in_proj[: self.dt_off + self.heads]), ("conv", self.conv),
+                ("conv.b", self.conv_bias), ("dt_bias", self.dt_bias), ("A_log", self.A_log), ("D", self.D), ("norm", self.norm), ("o", self.out_proj[:, : self.inner])]
+
+    def reset_special(self, gen: torch.Generator) -> None:
+        init_decay(self.A_log, self.dt_bias, gen)
+
+    def parts(self, u: torch.Tensor, p: torch.Tensor):
+        """fp32 x [T, heads, vdim], B and C [T, groups, dim], step sizes and log decays [T, heads]."""
+        u, n = u.float(), self.groups * self.dim
+        dt = TF.softplus(p[:, self.dt_off : self.dt_off + self.heads].float() + self.dt_bias.float())
+        return (u[:, : self.inner].reshape(-1, self.heads, self.vdim), u[:, self.inner : self.inner + n].reshape(-1, self.groups, self.dim),
+                u[:, self.inner + n :].reshape(-1, self.groups, self.dim), dt, -self.A_log.float().exp() * dt)
+
+    def scan(self, u: torch.Tensor, p: torch.Tensor, S: torch.Tensor, chunk: int = 64):
+        """(outputs [L, heads, vdim], state left) of one piece that starts from state ``S`` [heads, dim, vdim]."""
+        x, B, C, dt, _ = self.parts(u, p)
+        y, S = ssd_scan(x[None], dt[None], -self.A_log.float().exp(), B[None], C[None], chunk, S.transpose(1, 2)[None])
+        return y[0] + self.D.float()[:, None] * x, S[0].transpose(1, 2)
+
+    def finish(self, y: torch.Tensor, p: torch.Tensor) -> torch.Tensor:
+        return gated_group_norm(y.reshape(-1, self.inner), p[:, self.z_off : self.z_off + self.inner], self.norm, self.norm_groups, self.eps)
+
+
+class DeltaMixer(RecurrentMixer):
+    """S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q per head, with unit keys and queries, beta = sigmoid(W_b h) and
+    g = exp(-exp(A_log) softplus(W_a h + dt_bias)); then an RMS norm per head and a SiLU gate."""
+
+    kind = "delta"
+    conv_bias = None
+    unit_eps = 1e-6        # under the root of the unit norms of queries and keys
+
+    def __init__(self, spec: dict, cfg: ModelConfig, dtype, device):
+        super().__init__()
+        self.heads, self.kv_heads, self.dim, self.vdim = spec["heads"], spec["kv_heads"], spec["dim"], spec["vdim"]
+        self.taps, self.eps = spec["conv"], cfg.rms_norm_eps
+        H, n = self.heads, self.kv_heads * self.dim
+        self.channels, self.conv_off = 2 * n + H * self.vdim, 0
+        self.g_off = pad8(self.channels)
+        self.b_off = self.g_off + pad8(H * self.vdim)
+        self.a_off = self.b_off + pad8(H)
+        self.in_width, self.mix_width = self.a_off + pad8(H), pad8(H * self.vdim)
+        P = lambda *shape: nn.Parameter(torch.zeros(*shape, dtype=dtype, device=device))   # noqa: E731
+        self.in_proj, self.out_proj = P(self.in_width, cfg.hidden_size), P(cfg.hidden_size, self.mix_width)
+        self.conv = P(self.channels, self.taps)
+        self.A_log, self.dt_bias = P(H), P(H)
+        self.norm = nn.Parameter(torch.ones(self.vdim, dtype=dtype, device=device))
+
+    def tensors(self) -> list:
+        H, n, hv = self.heads, self.kv_heads * self.dim, self.heads * self.vdim
+        out = []
+        for leaf, r, k in (("q", 0, n), ("k", n, n), ("v", 2 * n, hv)):
+            out += [(leaf, self.in_proj[r : r + k]), (leaf + ".conv", self.conv[r : r + k])]
+        out += [(leaf, self.in_proj[r : r + k]) for leaf, r, k in (("g", self.g_off, hv), ("b", self.b_off, H), ("a", self.a_off, H))]
+        return out + [("A_log", self.A_log), ("dt_bias", self.dt_bias), ("norm", self.norm), ("o", self.out_proj[:, :hv])]
+
+    def reset_special(self, gen: torch.Generator) -> None:
+        init_decay(self.A_log, self.dt_bias, gen)
+
+    def parts(self, u: torch.Tensor, p: torch.Tensor):
+        """fp32 unit queries (scaled by dim^-1/2) and keys [T, heads, dim], values, step sizes beta and log decays [T, heads]."""
+        u, n, H = u.float(), self.kv_heads * self.dim, self.heads
+        q, k = (t.reshape(-1, self.kv_heads, self.dim) for t in (u[:, :n], u[:, n : 2 * n]))
+        q, k = (t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) + self.unit_eps) for t in (q, k))
+        rep = H // self.kv_heads
+        beta = torch.sigmoid(p[:, self.b_off : self.b_off + H].float())
+        lg = -self.A_log.float().exp() * TF.softplus(p[:, self.a_off : self.a_off + H].float() + self.dt_bias.float())
+        return (q.repeat_interleave(rep, 1) * self.dim ** -0.5, k.repeat_interleave(rep, 1), u[:, 2 * n :].reshape(-1, H, self.vdim), beta, lg)
+
+    def scan(self, u: torch.Tensor, p: torch.Tensor, S: torch.Tensor, chunk: int = 64):
+        """(outputs [L, heads, vdim], state left) of one piece. Inside a chunk with start state S the writes U solve the unit lower
+        triangular system (I + A) U = beta (V - decay K S), A_ij = beta_i decay_i / decay_j k_i . k_j for j < i."""
+        outs = []
+        q, k, v, beta, lg = (t.transpose(0, 1) for t in self.parts(u, p))          # [heads, L, ...]
+        for s in range(0, q.shape[1], chunk):
+            qc, kc, vc, bc = q[:, s : s + chunk], k[:, s : s + chunk], v[:, s : s + chunk], beta[:, s : s + chunk, None]
+            cum = lg[:, s : s + chunk].cumsum(-1)
+            n = qc.shape[1]
+            low = torch.ones(n, n, dtype=torch.bool, device=q.device).tril()
+            ratio = torch.where(low, cum[:, :, None] - cum[:, None, :], torch.full((), float("-inf"), device=q.device)).exp()
+            A = (bc * ratio * (kc @ kc.transpose(1, 2))).tril(-1)
+            eye = torch.eye(n, device=q.device)
+            U = torch.linalg.solve_triangular(eye + A, bc * (vc - cum.exp()[..., None] * (kc @ S)), upper=False, unitriangular=True)
+            outs.append(cum.exp()[..., None] * (qc @ S) + (ratio * (qc @ kc.transpose(1, 2))) @ U)
+            end = cum[:, -1:]
+            S = end.exp()[..., None] * S + (kc * (end - cum).exp()[..., None]).transpose(1, 2) @ U
+        return torch.cat(outs, 1).transpose(0, 1), S
+
+    def finish(self, o: torch.Tensor, p: torch.Tensor) -> torch.Tensor:
+        hv = self.heads * self.vdim
+        y = (rms_unit(o, self.eps) * self.norm.float()).reshape(-1, hv)
+        return (y * TF.silu(p[:, self.g_off : self.g_off + hv].float())).to(p.dtype)
+
+
+MIXERS = {m.kind: m for m in (LatentAttentionMixer, RetentionMixer, GroupedAttentionMixer, Mamba2LayerMixer, DeltaMixer)}
 
 
 class ParallelBlock(nn.Module):

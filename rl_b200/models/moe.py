@@ -19,6 +19,17 @@ from rl_b200.ops import functional as F
 from .config import ModelConfig
 
 
+def limit_groups(choice: torch.Tensor, groups: int, keep: int, masked: float) -> torch.Tensor:
+    """Group-limited selection: of ``groups`` equal runs of neighbouring experts only the ``keep`` whose two best choice scores sum
+    highest stay eligible; the others' choice scores [T, E] become ``masked``."""
+    if groups <= 1:
+        return choice
+    g = choice.view(choice.shape[0], groups, -1)
+    gs = g.topk(min(2, g.shape[-1]), dim=-1)[0].sum(-1)
+    kept = torch.zeros_like(gs).scatter_(1, gs.topk(keep, dim=-1, sorted=False)[1], 1.0).bool()
+    return g.masked_fill(~kept.unsqueeze(-1), masked).reshape(choice.shape)
+
+
 class MoEMLP(nn.Module):
     def __init__(self, cfg: ModelConfig, dtype, device, ep=None):
         super().__init__()
@@ -68,12 +79,7 @@ class MoEMLP(nn.Module):
         if forced is not None and bool((forced >= 0).all()):
             idx = forced
         else:
-            choice = scores + self.e_score_correction_bias
-            if c.n_group > 1:
-                g = choice.view(-1, c.n_group, E // c.n_group)
-                gs = g.topk(2, dim=-1)[0].sum(-1)
-                keep = torch.zeros_like(gs).scatter_(1, gs.topk(c.topk_group, dim=-1, sorted=False)[1], 1.0)
-                choice = choice.masked_fill(~keep.bool().unsqueeze(-1).expand_as(g).reshape(-1, E), 0.0)
+            choice = limit_groups(scores + self.e_score_correction_bias, c.n_group, c.topk_group, 0.0)
             idx = choice.topk(k, dim=-1, sorted=False)[1]
             if forced is not None:
                 idx = torch.where((forced >= 0).all(-1, keepdim=True), forced.clamp(min=0), idx)

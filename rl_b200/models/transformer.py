@@ -521,8 +521,10 @@ class CausalLM(nn.Module):
             self.embed_tokens = None
         block = HybridBlock if cfg.is_hybrid else DecoderLayer
         if cfg.is_mixer:
-            from .mixers import DynamicTanh, ParallelBlock as block
+            from .mixers import DynamicTanh, ParallelBlock
+            from .post_norm import PostNormBlock
 
+            block = PostNormBlock if cfg.norm_place == "post" else ParallelBlock
             if tpw > 1 or pp_size > 1 or self.cp is not None or (ep is not None and ep.world > 1) or self.lora_cfg or cfg.value_head:
                 raise NotImplementedError("layer-list models run data parallel only, without LoRA or value heads")
         if cfg.is_hybrid and self.tp.sequence_parallel:
@@ -538,6 +540,9 @@ class CausalLM(nn.Module):
                 self.lm_head = nn.Parameter(torch.empty(self.vocab_local, d, dtype=dtype, device=device))
         else:
             self.norm = None
+        # token inputs of the layers: one table, the layers' columns side by side
+        side = cfg.token_side["dim"] * L if cfg.token_side else 0
+        self.side_embed = nn.Parameter(torch.empty(cfg.vocab_size, side, dtype=dtype, device=device)) if side else None
         # looped layers: one learned vector per pass joins the residual stream when the pass begins
         self.loop_step = nn.Parameter(torch.zeros(cfg.layer_loop["times"], d, dtype=dtype, device=device)) if cfg.layer_loop else None
         self.register_buffer("inv_freq", rope_inv_freq(cfg, device) if not cfg.is_mixer else torch.zeros(0, device=device), persistent=False)
@@ -548,7 +553,7 @@ class CausalLM(nn.Module):
                                  persistent=False)
         else:
             self.inv_freq_local = None
-        if cfg.final_logit_softcap:
+        if cfg.final_logit_softcap and not cfg.is_mixer:
             raise NotImplementedError("final logit soft-capping (Gemma 2) is not supported by the fused log-probability paths")
         self.activation_checkpointing = activation_checkpointing
         if init:
@@ -590,7 +595,7 @@ class CausalLM(nn.Module):
         from .hf_io import iter_hf_shards, hf_full_shape
 
         for name, p in self.named_parameters():
-            if name.endswith("norm") or name.endswith("layernorm") or name.endswith("norm.weight"):
+            if name.endswith("norm") or name.rsplit(".", 1)[-1] in ("norm1", "norm2") or name.endswith("layernorm") or name.endswith("norm.weight"):
                 p.fill_(1.0)
             elif name.endswith("bias"):
                 p.zero_()
@@ -728,12 +733,30 @@ class CausalLM(nn.Module):
         for i, t in self.cfg.layer_runs:
             if t is not None and i == loop["start"]:
                 h = (h + e if t else h) + self.loop_step[t].float()
-            args = (h, batch.positions, None, batch.cu_seqlens, batch.max_seqlen)
+            args = (h, batch.positions, self.side_rows(batch.input_ids, i), batch.cu_seqlens, batch.max_seqlen)
             h = ckpt.checkpoint(self.layers[i], *args, use_reentrant=False) if (self.activation_checkpointing and torch.is_grad_enabled()) else self.layers[i](*args)
         return h
 
+    def side_rows(self, ids: torch.Tensor, layer: int) -> Optional[torch.Tensor]:
+        """The token input of ``layer`` (None where the model has none)."""
+        if self.side_embed is None:
+            return None
+        n = self.cfg.token_side["dim"]
+        return nn.functional.embedding(ids.long(), self.side_embed)[:, layer * n : (layer + 1) * n]
+
     def final_norm(self, h: torch.Tensor) -> torch.Tensor:
-        return self.norm(h) if self.cfg.norm_kind == "dyt" else F.rmsnorm(h, self.norm, self.cfg.rms_norm_eps)
+        if self.cfg.norm_kind == "dyt":
+            return self.norm(h)
+        if self.cfg.is_mixer:      # the stream is fp32
+            return (h * torch.rsqrt(h.pow(2).mean(-1, keepdim=True) + self.cfg.rms_norm_eps) * self.norm.float()).to(self.norm.dtype)
+        return F.rmsnorm(h, self.norm, self.cfg.rms_norm_eps)
+
+    def cap_logits(self, z: torch.Tensor) -> torch.Tensor:
+        """What follows the output product: scale and soft cap (fp32 logits)."""
+        c = self.cfg
+        if c.logit_scale != 1.0:
+            z = z * c.logit_scale
+        return c.final_logit_softcap * torch.tanh(z / c.final_logit_softcap) if c.final_logit_softcap else z
 
     def run_layers(self, h: torch.Tensor, batch: PackedBatch) -> torch.Tensor:
         if self.cfg.is_mixer:
@@ -780,12 +803,28 @@ class CausalLM(nn.Module):
         if self.cfg.is_mixer:
             from .mixers import _linear
 
-            return _linear(h, self.output_weight).float()
+            return self.cap_logits(_linear(h, self.output_weight).float())
         if self.tp.world == 1:
             return F.linear(h, self.output_weight).float()
         from rl_b200.parallel.tensor import gather_cols
 
         return gather_cols(column_linear(h, self.output_weight, None, self.tp), self.tp).float()
+
+    def _capped_logprobs(self, h, targets, temperature: float, want_entropy: bool, chunk_rows: int = 2048):
+        """Per-row log-probability of ``targets`` (and entropy) where the logits are scaled or soft-capped: they are materialised
+        ``chunk_rows`` rows at a time (and again in the backward pass)."""
+        from .mixers import _linear
+
+        def rows(hr, tg):
+            z = torch.log_softmax(self.cap_logits(_linear(hr, self.output_weight).float()) / (temperature if temperature > 0 else 1.0), dim=-1)
+            return z.gather(-1, tg[:, None])[:, 0], -(z.exp() * z).sum(-1) if want_entropy else z.new_zeros(z.shape[0])
+
+        out = []
+        for r0 in range(0, h.shape[0], chunk_rows):
+            args = (h[r0 : r0 + chunk_rows], targets[r0 : r0 + chunk_rows])
+            out.append(ckpt.checkpoint(rows, *args, use_reentrant=False) if torch.is_grad_enabled() else rows(*args))
+        lp, ent = (torch.cat(t) for t in zip(*out))
+        return lp, ent if want_entropy else None
 
     def logprobs_from_hidden(self, h: torch.Tensor, batch: PackedBatch, temperature: float = 1.0, want_entropy: bool = False):
         """``h``: normed final hidden states (this rank's rows). out[t] = log p(ids[t] | ids[<t]), 0 at sequence starts."""
@@ -796,7 +835,9 @@ class CausalLM(nn.Module):
         is_start[starts[starts < T]] = True
         # hidden state t predicts token t+1: every row is scored against the next token, then shifted by one
         targets = torch.roll(ids, -1)
-        if self.cp is not None:
+        if self.cfg.caps_logits:
+            lp_rows, ent_rows = self._capped_logprobs(h, targets, temperature, want_entropy)
+        elif self.cp is not None:
             # local rows are scored locally; the [T]-sized results are gathered (backward: each rank keeps its rows' share)
             from rl_b200.parallel.context import gather_to_stream
 
@@ -848,7 +889,7 @@ class CausalLM(nn.Module):
         def score_rows(hr, tg, w):   # rows with the whole vocabulary on this rank
             out = []
             for r0 in range(0, hr.shape[0], chunk_rows):
-                z = F.linear(hr[r0 : r0 + chunk_rows], w).float() / inv_t
+                z = self.cap_logits(F.linear(hr[r0 : r0 + chunk_rows], w).float()) / inv_t
                 z, _ = apply_top_k_top_p(z, top_k, top_p)
                 lp = torch.log_softmax(z, dim=-1).gather(-1, tg[r0 : r0 + chunk_rows, None])[:, 0]
                 out.append(torch.where(torch.isfinite(lp), lp, torch.full_like(lp, -1e4)))   # a token outside the kept set

@@ -245,12 +245,35 @@ def gadarax_flops(hf, seq: int) -> float:
     return total + head_flops(seq, d, _g(hf, "vocab_size"))
 
 
+def redarax_flops(hf, seq: int) -> float:
+    """Post-norm layer-list models: attention, Mamba-2 or delta-rule mixers, dense or expert gated units, token inputs."""
+    d, total = _g(hf, "hidden_size"), 0.0
+    side = (_g(hf, "token_side") or {"dim": 0})["dim"]
+    for e in _g(hf, "mixers"):
+        m, mlp = e["mixer"], e.get("mlp")
+        H, vd = m["heads"], m["vdim"]
+        if e["type"] == "attention":
+            total += 2 * seq * d * (H * m["dim"] + m["kv_heads"] * (m["dim"] + vd) + H * vd) + seq * seq * H * (m["dim"] + vd)
+        elif e["type"] == "mamba2":
+            conv = H * vd + 2 * m["groups"] * m["state"]
+            total += 2 * seq * d * (2 * H * vd + conv - H * vd + H + H * vd) + 2 * seq * conv * m["conv"] + 4 * seq * H * m["state"] * vd
+        else:      # the state is read twice and written once per token
+            conv = 2 * m["kv_heads"] * m["dim"] + H * vd
+            total += 2 * seq * d * (conv + 2 * H + 2 * H * vd) + 2 * seq * conv * m["conv"] + 6 * seq * H * m["dim"] * vd
+        if mlp and mlp.get("kind") == "moe":
+            total += 2 * seq * d * mlp["router"]["experts"] + mlp["router"]["top"] * mlp_flops(seq, d, mlp["expert"]["ff"], gated=True)
+        elif mlp:
+            total += mlp_flops(seq, d, mlp["ff"], gated=True)
+        total += 4 * seq * d * side
+    return total + head_flops(seq, d, _g(hf, "vocab_size"))
+
+
 FAMILY_FLOPS = {
     "llama": llama_flops, "mistral": mistral_flops, "qwen2": qwen2_flops, "qwen3": qwen3_flops, "gemma3": gemma3_flops,
     "gemma3_text": gemma3_flops,
     "gpt2": gpt_flops, "gpt3": gpt_flops, "nemotron": nemotron_flops, "mixtral": mixtral_flops, "qwen3_moe": qwen3_moe_flops,
     "qwen2_moe": moe_decoder_flops, "deepseek_v3": deepseek_v3_flops, "deepseek_v2": deepseek_v3_flops, "nemotron_h": nemotron_h_flops,
-    "bert": bert_flops, "gadarax": gadarax_flops,
+    "bert": bert_flops, "gadarax": gadarax_flops, "redarax": redarax_flops,
 }
 
 
