@@ -1,0 +1,234 @@
+// Grouped-query attention of layer-list models (GroupedAttentionMixer): the step between the projection and the attention kernels, the gather
+// of cached keys and values for prompt portions, and attention one row at a time for every size and for bf16 and fp32 models.
+//
+// Keys and values live in pages [page, kv head, token, dim] / [page, kv head, token, vdim]. The tensor-core forms are in
+// latent_attention.cu (portions of prompts) and paged_decode_mma.cu (single rows, head dimension 128).
+//
+// This file is compiled without fast math.
+#include "common.cuh"
+
+#include <math.h>
+
+namespace {
+using namespace rlb;
+
+template <typename T>
+__device__ __forceinline__ float ldf(const T* p) {
+  return static_cast<float>(*p);
+}
+template <>
+__device__ __forceinline__ float ldf<__nv_bfloat16>(const __nv_bfloat16* p) {
+  return __bfloat162float(*p);
+}
+__device__ __forceinline__ void stf(float* p, float v) { *p = v; }
+__device__ __forceinline__ void stf(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+
+struct GqaShape {
+  long long ldp;
+  int q_off, k_off, v_off;
+  int heads, kv_heads, dim, vdim;
+  int block_size, num_blocks;
+};
+
+// One warp per head of a row: RMS norm and rotation of a query or key head in place, keys and values into the cache. A lane keeps pairs
+// (2i, 2i + 1), which is also what the rotation turns.
+constexpr int GP_WARPS = 8, GP_KEEP = 4;      // pairs a lane keeps in registers
+template <typename T>
+__global__ void __launch_bounds__(GP_WARPS * 32)
+gqa_prep_kernel(T* __restrict__ p, GqaShape s, const int* __restrict__ positions, const long long* __restrict__ slots, const T* __restrict__ q_norm,
+                const T* __restrict__ k_norm, const float* __restrict__ freq, int half, float gain, float eps, T* __restrict__ k_cache,
+                T* __restrict__ v_cache, int* status) {
+  pdl_sync();
+  const int lane = threadIdx.x & 31;
+  const long long row = blockIdx.x;
+  const int unit = blockIdx.y * GP_WARPS + (threadIdx.x >> 5);
+  if (unit >= s.heads + 2 * s.kv_heads) return;
+  T* pr = p + row * s.ldp;
+  const bool is_q = unit < s.heads, is_k = !is_q && unit < s.heads + s.kv_heads;
+  const int head = is_q ? unit : (is_k ? unit - s.heads : unit - s.heads - s.kv_heads);
+  const long long slot = slots[row];
+  const bool bad = slot >= static_cast<long long>(s.num_blocks) * s.block_size;
+  if (bad && lane == 0 && status) atomicCAS(status, 0, RLB_ERR_BOUNDS);
+  const bool cached = slot >= 0 && !bad;
+  const long long page = cached ? slot / s.block_size : 0, off = cached ? slot % s.block_size : 0;
+  if (!is_q && !is_k) {
+    if (!cached) return;
+    const T* v = pr + s.v_off + head * s.vdim;
+    T* c = v_cache + ((page * s.kv_heads + head) * s.block_size + off) * s.vdim;
+    for (int i = lane; i < s.vdim; i += 32) c[i] = v[i];
+    return;
+  }
+  T* x = pr + (is_q ? s.q_off : s.k_off) + head * s.dim;
+  const T* w = is_q ? q_norm : k_norm;
+  T* c = is_k && cached ? k_cache + ((page * s.kv_heads + head) * s.block_size + off) * s.dim : nullptr;
+  const int pairs = (s.dim + 1) / 2;
+  float u[GP_KEEP], v[GP_KEEP];
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < GP_KEEP; ++j) {
+    const int i = lane + j * 32;
+    u[j] = 2 * i < s.dim ? ldf(x + 2 * i) : 0.f;
+    v[j] = 2 * i + 1 < s.dim ? ldf(x + 2 * i + 1) : 0.f;
+    ss += u[j] * u[j] + v[j] * v[j];
+  }
+  for (int i = lane + GP_KEEP * 32; i < pairs; i += 32) {
+    const float a = ldf(x + 2 * i), b = 2 * i + 1 < s.dim ? ldf(x + 2 * i + 1) : 0.f;
+    ss += a * a + b * b;
+  }
+  ss = warp_sum(ss);
+  const float rstd = 1.f / sqrtf(ss / static_cast<float>(s.dim) + eps);
+  const float pos = static_cast<float>(positions[row]);
+  auto finish = [&](int i, float a, float b) {
+    if (2 * i >= s.dim) return;
+    const bool two = 2 * i + 1 < s.dim;
+    a *= rstd * ldf(w + 2 * i);
+    if (two) b *= rstd * ldf(w + 2 * i + 1);
+    if (i < half) {
+      float sn, cs;
+      sincosf(pos * freq[i], &sn, &cs);
+      sn *= gain;
+      cs *= gain;
+      const float a0 = a;
+      a = a0 * cs - b * sn;
+      b = b * cs + a0 * sn;
+    }
+    stf(x + 2 * i, a);
+    if (two) stf(x + 2 * i + 1, b);
+    if (c) {
+      stf(c + 2 * i, a);
+      if (two) stf(c + 2 * i + 1, b);
+    }
+  };
+#pragma unroll
+  for (int j = 0; j < GP_KEEP; ++j) finish(lane + j * 32, u[j], v[j]);
+  for (int i = lane + GP_KEEP * 32; i < pairs; i += 32) finish(i, ldf(x + 2 * i), 2 * i + 1 < s.dim ? ldf(x + 2 * i + 1) : 0.f);
+}
+
+// One CTA per (row, query head): tiles of 128 keys, online softmax, everything in fp32.
+constexpr int GR_TILE = 128;
+template <typename T>
+__global__ void __launch_bounds__(128)
+gqa_rows_kernel(const T* __restrict__ p, GqaShape s, const T* __restrict__ k_cache, const T* __restrict__ v_cache, const int* __restrict__ block_table,
+                int bt_stride, const int* __restrict__ seq_lens, float scale, T* __restrict__ y, long long ldy, int* status) {
+  extern __shared__ float sm[];
+  __shared__ float red[32];
+  float* q = sm;                        // [dim]
+  float* o = q + s.dim;                 // [vdim]
+  float* sc = o + s.vdim;               // [GR_TILE]
+  long long* rows = reinterpret_cast<long long*>(sm + ((s.dim + s.vdim + GR_TILE + 1) & ~1));   // [GR_TILE] token row of the head in the cache
+  const int row = blockIdx.x, h = blockIdx.y, g = h / (s.heads / s.kv_heads), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const T* qp = p + row * s.ldp + s.q_off + h * s.dim;
+  for (int i = tid; i < s.dim; i += 128) q[i] = ldf(qp + i) * scale;
+  for (int i = tid; i < s.vdim; i += 128) o[i] = 0.f;
+  const int len = min(seq_lens[row], bt_stride * s.block_size);
+  float m = -INFINITY, l = 0.f;
+  for (int t0 = 0; t0 < len; t0 += GR_TILE) {
+    const int n = min(GR_TILE, len - t0);
+    __syncthreads();
+    if (tid < n) {
+      const int t = t0 + tid;
+      int blk = block_table[static_cast<long long>(row) * bt_stride + t / s.block_size];
+      if (blk < 0 || blk >= s.num_blocks) {
+        if (status) atomicCAS(status, 0, RLB_ERR_BOUNDS);
+        blk = 0;
+      }
+      rows[tid] = (static_cast<long long>(blk) * s.kv_heads + g) * s.block_size + t % s.block_size;
+    }
+    __syncthreads();
+    for (int j = warp; j < n; j += 4) {
+      const T* k = k_cache + rows[j] * s.dim;
+      float v = 0.f;
+      for (int i = lane; i < s.dim; i += 32) v = fmaf(q[i], ldf(k + i), v);
+      v = warp_sum(v);
+      if (lane == 0) sc[j] = v;
+    }
+    __syncthreads();
+    const float mine = tid < n ? sc[tid] : -INFINITY;
+    const float mn = fmaxf(m, block_max(mine, red));
+    const float pj = tid < n ? expf(mine - mn) : 0.f;
+    const float c = m == -INFINITY ? 0.f : expf(m - mn);
+    l = l * c + block_sum(pj, red);
+    m = mn;
+    if (tid < n) sc[tid] = pj;
+    __syncthreads();
+    for (int i = tid; i < s.vdim; i += 128) {
+      float v = o[i] * c;
+      for (int j = 0; j < n; ++j) v = fmaf(sc[j], ldf(v_cache + rows[j] * s.vdim + i), v);
+      o[i] = v;
+    }
+  }
+  const float inv = l > 0.f ? 1.f / l : 0.f;
+  for (int i = tid; i < s.vdim; i += 128) stf(y + row * ldy + h * s.vdim + i, o[i] * inv);     // (each thread reads what it wrote)
+}
+
+// out[i] = [keys of all kv heads | values of all kv heads] of cache slot slots[i]; dim and vdim in 16-byte pieces.
+__global__ void gqa_gather_kernel(const uint4* __restrict__ k_cache, const uint4* __restrict__ v_cache, const long long* __restrict__ slots,
+                                  uint4* __restrict__ out, long long n, int kv_heads, int dv, int vv, int block_size, long long num_slots, int* status) {
+  const int per = kv_heads * (dv + vv);
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < n * per; i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long t = i / per;
+    int c = static_cast<int>(i - t * per);
+    const long long s = slots[t];
+    if (s < 0 || s >= num_slots) {
+      if (status) atomicCAS(status, 0, RLB_ERR_BOUNDS);
+      out[i] = make_uint4(0, 0, 0, 0);
+      continue;
+    }
+    const bool is_k = c < kv_heads * dv;
+    if (!is_k) c -= kv_heads * dv;
+    const int w = is_k ? dv : vv, g = c / w;
+    out[i] = (is_k ? k_cache : v_cache)[((s / block_size * kv_heads + g) * block_size + s % block_size) * w + (c - g * w)];
+  }
+}
+}  // namespace
+
+// In place on the projected rows p: RMS norm (weight [dim]) and rotation of the first 2 * half dimensions (interleaved pairs) of every query
+// and key head; keys and values of rows with a slot go to the cache.
+RLB_API int rlb_gqa_prep(void* p, int f32, long long rows, long long ldp, int q_off, int k_off, int v_off, int heads, int kv_heads, int dim, int vdim,
+                         int block_size, int num_blocks, const int* positions, const long long* slots, const void* q_norm, const void* k_norm,
+                         const float* freq, int half, float gain, float eps, void* k_cache, void* v_cache, int* status, void* stream) {
+  if (rows <= 0) return 0;
+  if (2 * half > dim || kv_heads < 1 || heads % kv_heads) return -2;
+  GqaShape s{ldp, q_off, k_off, v_off, heads, kv_heads, dim, vdim, block_size, num_blocks};
+  const dim3 grid(static_cast<unsigned>(rows), (heads + 2 * kv_heads + GP_WARPS - 1) / GP_WARPS), block(GP_WARPS * 32);
+  if (grid.y > 65535) return -2;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (f32)
+    return static_cast<int>(rlb_launch_pdl(gqa_prep_kernel<float>, grid, block, 0, st, static_cast<float*>(p), s, positions, slots,
+                                           static_cast<const float*>(q_norm), static_cast<const float*>(k_norm), freq, half, gain, eps,
+                                           static_cast<float*>(k_cache), static_cast<float*>(v_cache), status));
+  return static_cast<int>(rlb_launch_pdl(gqa_prep_kernel<__nv_bfloat16>, grid, block, 0, st, static_cast<__nv_bfloat16*>(p), s, positions, slots,
+                                         static_cast<const __nv_bfloat16*>(q_norm), static_cast<const __nv_bfloat16*>(k_norm), freq, half, gain, eps,
+                                         static_cast<__nv_bfloat16*>(k_cache), static_cast<__nv_bfloat16*>(v_cache), status));
+}
+
+RLB_API int rlb_gqa_rows(const void* p, int f32, int rows, long long ldp, int q_off, int heads, int kv_heads, int dim, int vdim, int block_size,
+                         int num_blocks, const void* k_cache, const void* v_cache, const int* block_table, int bt_stride, const int* seq_lens,
+                         float scale, void* y, long long ldy, int* status, void* stream) {
+  if (rows <= 0) return 0;
+  if (kv_heads < 1 || heads % kv_heads || heads > 65535 || dim + vdim > 12000) return -2;
+  GqaShape s{ldp, q_off, 0, 0, heads, kv_heads, dim, vdim, block_size, num_blocks};
+  const size_t sm = sizeof(float) * ((dim + vdim + GR_TILE + 1) & ~1) + sizeof(long long) * GR_TILE;
+  if (sm > 48 * 1024) return -2;
+  const dim3 grid(rows, heads);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (f32)
+    gqa_rows_kernel<float><<<grid, 128, sm, st>>>(static_cast<const float*>(p), s, static_cast<const float*>(k_cache), static_cast<const float*>(v_cache),
+                                                  block_table, bt_stride, seq_lens, scale, static_cast<float*>(y), ldy, status);
+  else
+    gqa_rows_kernel<__nv_bfloat16><<<grid, 128, sm, st>>>(static_cast<const __nv_bfloat16*>(p), s, static_cast<const __nv_bfloat16*>(k_cache),
+                                                          static_cast<const __nv_bfloat16*>(v_cache), block_table, bt_stride, seq_lens, scale,
+                                                          static_cast<__nv_bfloat16*>(y), ldy, status);
+  return static_cast<int>(cudaGetLastError());
+}
+
+RLB_API int rlb_gqa_gather(const void* k_cache, const void* v_cache, const long long* slots, void* out, long long n, int kv_heads, int dim, int vdim,
+                           int block_size, long long num_slots, int* status, void* stream) {
+  if (n <= 0) return 0;
+  if (dim % 8 || vdim % 8) return -2;
+  const long long want = (n * kv_heads * ((dim + vdim) / 8) + 255) / 256;
+  gqa_gather_kernel<<<static_cast<unsigned>(want < 148 * 16 ? want : 148 * 16), 256, 0, static_cast<cudaStream_t>(stream)>>>(
+      static_cast<const uint4*>(k_cache), static_cast<const uint4*>(v_cache), slots, static_cast<uint4*>(out), n, kv_heads, dim / 8, vdim / 8, block_size,
+      num_slots, status);
+  return static_cast<int>(cudaGetLastError());
+}

@@ -343,9 +343,38 @@ __device__ __forceinline__ float tanh_acc(float x) {
   return copysignf(1.f - 2.f / (1.f + expf(2.f * a)), x);
 }
 
-// Epilogue of the two products of a parallel mixer layer. With `x`: the fp32 residual stream x[row, col] += acc (+ e) (+ step) is
-// updated in place and the output is the dynamic-tanh norm w * tanh(alpha x) + b of the new value. Without: the output is acc,
-// squared ReLU on columns >= act_from.
+// What follows a product in a layer-list model. LIN_GLU: columns 2i and 2i + 1 are gate and up of a clamped gated unit, the output has
+// N / 2 columns. LIN_GELU_MUL: gelu_tanh times a table row chosen by the row's token. LIN_CAP: scale, then soft cap (cap > 0).
+enum RlbLinearAct : int { LIN_NONE = 0, LIN_GLU = 1, LIN_GELU_MUL = 2, LIN_CAP = 3 };
+struct LinearEpi {
+  const void* bias;      // [N] in the weights' type, or null: added to the product
+  int act;
+  float limit;           // LIN_GLU
+  float scale, cap;      // LIN_CAP
+  const void* table;     // LIN_GELU_MUL: [vocab, ld_table] in the weights' type, columns [table_off, table_off + table_cols)
+  long long ld_table;
+  int table_off, table_cols, vocab;
+  const void* ids;       // [rows] int32 or int64
+  int ids64;
+};
+__device__ __forceinline__ float clamped_glu(float g, float u, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
+}
+__device__ __forceinline__ float gelu_tanh_acc(float z) { return 0.5f * z * (1.f + tanh_acc(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+__device__ __forceinline__ float soft_cap(float z, float scale, float cap) {
+  z *= scale;
+  return cap > 0.f ? cap * tanh_acc(z / cap) : z;
+}
+__device__ __forceinline__ long long lin_token(const LinearEpi& e, long long row) {
+  const long long id = e.ids64 ? static_cast<const long long*>(e.ids)[row] : static_cast<const int*>(e.ids)[row];
+  return id < 0 || id >= e.vocab ? 0 : id;      // (the embedding reports bad ids)
+}
+
+// Epilogue of the products of layer-list models. With `x`: the fp32 residual stream x[row, col] += acc (+ e) (+ step) is
+// updated in place and the output is the dynamic-tanh norm w * tanh(alpha x) + b of the new value. Without: the output is acc after
+// `lin`, squared ReLU on columns >= act_from.
 struct LayerEpilogue {
   float* x;
   long long ldx;             // row stride of x and e
@@ -355,9 +384,15 @@ struct LayerEpilogue {
   const __nv_bfloat16* nw;
   const __nv_bfloat16* nb;
   int act_from;
+  LinearEpi lin;
 };
-// Four consecutive columns of one row (col a multiple of 4).
+// Four consecutive columns of one row (col a multiple of 4). LIN_GLU: the two outputs are in .x and .y.
 __device__ __forceinline__ float4 layer_epilogue4(const LayerEpilogue& le, float4 v, long long row, int col, float alpha) {
+  if (le.lin.bias) {
+    const uint2 bv = *reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(le.lin.bias) + col);
+    const float2 b0 = unpack_bf16x2(bv.x), b1 = unpack_bf16x2(bv.y);
+    v.x += b0.x; v.y += b0.y; v.z += b1.x; v.w += b1.y;
+  }
   if (le.x) {
     float4* xp = reinterpret_cast<float4*>(le.x + row * le.ldx + col);
     const float4 old = *xp;
@@ -378,6 +413,17 @@ __device__ __forceinline__ float4 layer_epilogue4(const LayerEpilogue& le, float
     v.y = tanh_acc(alpha * v.y) * w0.y + b0.y;
     v.z = tanh_acc(alpha * v.z) * w1.x + b1.x;
     v.w = tanh_acc(alpha * v.w) * w1.y + b1.y;
+  } else if (le.lin.act == LIN_GLU) {
+    v.x = clamped_glu(v.x, v.y, le.lin.limit);
+    v.y = clamped_glu(v.z, v.w, le.lin.limit);
+  } else if (le.lin.act == LIN_GELU_MUL) {
+    const __nv_bfloat16* t = static_cast<const __nv_bfloat16*>(le.lin.table) + lin_token(le.lin, row) * le.lin.ld_table + le.lin.table_off;
+    float* f = reinterpret_cast<float*>(&v);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) f[i] = col + i < le.lin.table_cols ? gelu_tanh_acc(f[i]) * __bfloat162float(t[col + i]) : 0.f;
+  } else if (le.lin.act == LIN_CAP) {
+    v.x = soft_cap(v.x, le.lin.scale, le.lin.cap); v.y = soft_cap(v.y, le.lin.scale, le.lin.cap);
+    v.z = soft_cap(v.z, le.lin.scale, le.lin.cap); v.w = soft_cap(v.w, le.lin.scale, le.lin.cap);
   } else if (col >= le.act_from) {   // act_from is a multiple of 8
     v.x = fmaxf(v.x, 0.f); v.y = fmaxf(v.y, 0.f); v.z = fmaxf(v.z, 0.f); v.w = fmaxf(v.w, 0.f);
     v.x *= v.x; v.y *= v.y; v.z *= v.z; v.w *= v.w;
@@ -408,6 +454,27 @@ __device__ __forceinline__ float block_max(float v, float* red) {
 }
 
 }  // namespace rlb
+
+// A product and what follows it: out = epilogue(a w^T), for rlb_linear_rows (any size, bf16 or fp32), rlb_linear_tiled and
+// rlb_linear_skinny (bf16 shapes that TMA can address) and rlb_linear_grouped. Grouped: 128-row tile t of `a` belongs to expert
+// tile_expert[t] (-1: unused) whose weight is w + expert * N * ldw; rlb_linear_rows may read row r of `a` from a_rows[r] (-1: zeros).
+struct RlbLinear {
+  const void* a;
+  const void* w;
+  void* out;
+  const void* bias;
+  const void* table;
+  const void* ids;
+  const int* tile_expert;
+  const int* a_rows;
+  int* status;
+  long long lda, ldw, ldo, ld_table;
+  int M, N, K, in_f32, out_f32, act, table_off, table_cols, vocab, ids64, experts, num_a_rows;
+  float limit, scale, cap;
+};
+inline rlb::LinearEpi rlb_linear_epi(const RlbLinear& l) {
+  return rlb::LinearEpi{l.bias, l.act, l.limit, l.scale, l.cap, l.table, l.ld_table, l.table_off, l.table_cols, l.vocab, l.ids, l.ids64};
+}
 
 // ---------------------------------------------------------------- host helpers
 typedef CUresult (*RlbEncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,

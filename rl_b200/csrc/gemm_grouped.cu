@@ -42,6 +42,8 @@ struct GroupedArgs {
   long long c_expert_stride;  // reduction mode: elements between consecutive experts' outputs
   int out_fp32;
   int accumulate;
+  int glu;                  // rows mode, bf16: columns 2i, 2i + 1 are gate and up of a clamped gated unit, C has N / 2 columns
+  float limit;
 };
 
 // One unit of work: which tile, which k range, where B / C start.
@@ -243,6 +245,15 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
               *reinterpret_cast<float4*>(dst + q * 4) = o;
             }
           }
+        } else if (g.glu) {
+          __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(g.C) + static_cast<long long>(row) * g.ldc + col / 2;
+#pragma unroll
+          for (int q = 0; q < 4; ++q) {
+            if (col + q * 8 < g.N)
+              *reinterpret_cast<uint2*>(dst + q * 4) =
+                  make_uint2(pack_bf16x2(clamped_glu(v[q * 8], v[q * 8 + 1], g.limit), clamped_glu(v[q * 8 + 2], v[q * 8 + 3], g.limit)),
+                             pack_bf16x2(clamped_glu(v[q * 8 + 4], v[q * 8 + 5], g.limit), clamped_glu(v[q * 8 + 6], v[q * 8 + 7], g.limit)));
+          }
         } else {
           __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(g.C) + w.c_off + static_cast<long long>(row) * g.ldc + col;
 #pragma unroll
@@ -334,6 +345,31 @@ RLB_API int rlb_gemm_grouped_rows(const void* A, long long lda, const void* B, i
   const int tiles = (Mpad / BM) * ((N + BN - 1) / BN);
   return b_mn ? launch_grouped<false, true>(ta, tb, g, status, tiles, static_cast<cudaStream_t>(stream))
               : launch_grouped<false, false>(ta, tb, g, status, tiles, static_cast<cudaStream_t>(stream));
+}
+
+// rlb_gemm_grouped_rows with the clamped gated unit of LIN_GLU or no epilogue; rows of padding may hold anything.
+RLB_API int rlb_linear_grouped(const RlbLinear* l, void* stream) {
+  if (l->M <= 0 || l->N <= 0 || l->K <= 0) return 0;
+  if ((l->M % 128) || (l->lda % 8) || (l->ldo % 8) || (l->N % 8) || (l->K % 8) || l->ldw != l->K || !l->tile_expert || l->a_rows) return -2;
+  if (l->in_f32 || l->out_f32 || l->bias || (l->act != LIN_NONE && l->act != LIN_GLU)) return -2;
+  if ((reinterpret_cast<uintptr_t>(l->a) | reinterpret_cast<uintptr_t>(l->w) | reinterpret_cast<uintptr_t>(l->out)) & 15) return -3;
+  CUtensorMap ta, tb;
+  int rc = rlb_make_tmap_2d(&ta, l->a, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, l->K, l->M, l->lda * 2, BK, BM, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (rc) return -100 - rc;
+  rc = rlb_make_tmap_2d(&tb, l->w, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, l->K, static_cast<uint64_t>(l->experts) * l->N, static_cast<uint64_t>(l->K) * 2, BK,
+                        BN, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (rc) return -100 - rc;
+  GroupedArgs g{};
+  g.M = l->M;
+  g.N = l->N;
+  g.K = l->K;
+  g.num_experts = l->experts;
+  g.tile_expert = l->tile_expert;
+  g.C = l->out;
+  g.ldc = l->ldo;
+  g.glu = l->act == LIN_GLU;
+  g.limit = l->limit;
+  return launch_grouped<false, false>(ta, tb, g, l->status, (l->M / BM) * ((l->N + BN - 1) / BN), static_cast<cudaStream_t>(stream));
 }
 
 // C[e][M, N] (+)= A[rows_e, M]^T * B[rows_e, N] for every expert e with rows_e = [expert_row0[e], +expert_rows[e]).

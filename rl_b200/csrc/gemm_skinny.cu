@@ -20,8 +20,8 @@
 //     rstd = rsqrt(sum of the partials / d + eps) in its epilogue: the row scale commutes with the product.
 //   * SwiGLU: for the [gate | up] weight, a tile is 64 gate rows stacked on the 64 matching up rows (two TMA boxes into
 //     one 128-row operand, no re-layout of the weight), and the epilogue writes silu(gate) * up.
-//   * The products of parallel mixer layers (LayerEpilogue in common.cuh): squared ReLU on a column range, or the fp32
-//     residual update followed by the next layer's dynamic-tanh norm.
+//   * The products of layer-list models (LayerEpilogue in common.cuh): squared ReLU on a column range, or the fp32
+//     residual update followed by the next layer's dynamic-tanh norm; bias, clamped gated unit, gated token input, soft cap.
 //
 // Counterpart in the reference: the cuBLAS / vLLM GEMMs behind every decode-step nn.Linear
 // (nemo_rl/models/generation/vllm/vllm_worker.py:570-597).
@@ -300,6 +300,8 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
         if (p.use_layer) acc = layer_epilogue4(p.layer, acc, m, n, layer_alpha);
         if (p.out_fp32) {
           *reinterpret_cast<float4*>(reinterpret_cast<float*>(p.Y) + static_cast<long long>(m) * p.ldy + n) = acc;
+        } else if (p.use_layer && p.layer.lin.act == LIN_GLU) {
+          *reinterpret_cast<uint32_t*>(reinterpret_cast<__nv_bfloat16*>(p.Y) + static_cast<long long>(m) * p.ldy + n / 2) = pack_bf16x2(acc.x, acc.y);
         } else {
           uint2 o;
           o.x = pack_bf16x2(acc.x, acc.y);
@@ -485,9 +487,38 @@ RLB_API int rlb_gemm_skinny_layer(const void* X, const void* W, void* out, int M
   p.status = status;
   p.use_layer = 1;
   p.layer = LayerEpilogue{x, ldx, e, static_cast<const __nv_bfloat16*>(step), static_cast<const __nv_bfloat16*>(alpha),
-                          static_cast<const __nv_bfloat16*>(nw), static_cast<const __nv_bfloat16*>(nb), act_from};
+                          static_cast<const __nv_bfloat16*>(nw), static_cast<const __nv_bfloat16*>(nb), act_from, LinearEpi{}};
   return launch_skinny_nt(NT, tw, tx, p, rlb_gemm_skinny_split(N, K), static_cast<cudaStream_t>(stream));
 }
+
+// rlb_linear_tiled for M <= 256 rows on the weight-streaming kernel; out bf16 or fp32 (fp32: no gated unit).
+RLB_API int rlb_linear_skinny(const RlbLinear* l, void* stream) {
+  if (l->M <= 0 || l->N <= 0 || l->K <= 0) return 0;
+  if (l->M > 256) return -7;
+  if ((l->lda % 8) || (l->ldw % 8) || (l->ldo % (l->out_f32 ? 4 : 8)) || (l->N % 8) || (l->K % 8) || l->in_f32 || l->tile_expert) return -2;
+  if (l->out_f32 && l->act == LIN_GLU) return -2;
+  if ((reinterpret_cast<uintptr_t>(l->a) | reinterpret_cast<uintptr_t>(l->w) | reinterpret_cast<uintptr_t>(l->out) | reinterpret_cast<uintptr_t>(l->bias)) & 15) return -3;
+  const int NT = l->M <= 32 ? 32 : (l->M <= 64 ? 64 : (l->M <= 128 ? 128 : 256));
+  CUtensorMap tw, tx;
+  int rc = rlb_make_tmap_2d(&tw, l->w, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, l->K, l->N, l->ldw * 2, SK_BK, SK_BM, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (rc) return -100 - rc;
+  rc = rlb_make_tmap_2d(&tx, l->a, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, l->K, l->M, l->lda * 2, SK_BK, NT, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (rc) return -100 - rc;
+  SkinnyParams p{};
+  p.Y = l->out;
+  p.ldy = l->ldo;
+  p.M = l->M;
+  p.N = l->N;
+  p.K = l->K;
+  p.out_fp32 = l->out_f32;
+  p.w_static = g_sk_static_w;
+  p.status = l->status;
+  p.use_layer = 1;
+  p.layer.act_from = 1 << 30;
+  p.layer.lin = rlb_linear_epi(*l);
+  return launch_skinny_nt(NT, tw, tx, p, rlb_gemm_skinny_split(l->N, l->K), static_cast<cudaStream_t>(stream));
+}
+
 RLB_API int rlb_gemm_skinny(const void* X, const void* W, void* Y, int M, int N, int K, long long ldx, long long ldw,
                             long long ldy, int out_fp32, const float* bias, const void* residual, long long ldr,
                             int split, int* status, void* stream) {

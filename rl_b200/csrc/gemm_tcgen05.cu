@@ -303,13 +303,14 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
         }
       } else if (EPI == EPI_LAYER) {
         const float alpha = ep.layer.x ? __bfloat162float(*ep.layer.alpha) : 0.f;
+        const bool glu = ep.layer.lin.act == LIN_GLU;
         for (int c = 0; c < BN / 32; ++c) {
           uint32_t r[32];
           tmem_ld_32x32b_x32(taddr + c * 32, r);
           tmem_ld_wait();
           const int col = col0 + c * 32;
           if (!row_ok || col >= N) continue;
-          __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(ep.C) + static_cast<long long>(row) * ep.ldc + col;
+          __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(ep.C) + static_cast<long long>(row) * ep.ldc + (glu ? col / 2 : col);
 #pragma unroll
           for (int q = 0; q < 4; ++q) {
             if (col + q * 8 < N) {
@@ -317,6 +318,10 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
                                                                      __uint_as_float(r[q * 8 + 2]), __uint_as_float(r[q * 8 + 3])), row, col + q * 8, alpha);
               const float4 b = layer_epilogue4(ep.layer, make_float4(__uint_as_float(r[q * 8 + 4]), __uint_as_float(r[q * 8 + 5]),
                                                                      __uint_as_float(r[q * 8 + 6]), __uint_as_float(r[q * 8 + 7])), row, col + q * 8 + 4, alpha);
+              if (glu) {
+                *reinterpret_cast<uint2*>(dst + q * 4) = make_uint2(pack_bf16x2(a.x, a.y), pack_bf16x2(b.x, b.y));
+                continue;
+              }
               *reinterpret_cast<uint4*>(dst + q * 8) = make_uint4(pack_bf16x2(a.x, a.y), pack_bf16x2(a.z, a.w), pack_bf16x2(b.x, b.y), pack_bf16x2(b.z, b.w));
             }
           }
@@ -578,8 +583,24 @@ RLB_API int rlb_gemm_layer(const void* A, const void* W, void* out, int M, int N
   ep.C = out;
   ep.ldc = ldo;
   ep.layer = LayerEpilogue{x, ldx, e, static_cast<const __nv_bfloat16*>(step), static_cast<const __nv_bfloat16*>(alpha),
-                           static_cast<const __nv_bfloat16*>(nw), static_cast<const __nv_bfloat16*>(nb), act_from};
+                           static_cast<const __nv_bfloat16*>(nw), static_cast<const __nv_bfloat16*>(nb), act_from, LinearEpi{}};
   return launch_gemm<false, false, EPI_LAYER>(ta, tb, M, N, K, ep, status, 0, static_cast<cudaStream_t>(stream));
+}
+
+// out (bf16) = epilogue(a w^T); N, K and the row strides multiples of 8.
+RLB_API int rlb_linear_tiled(const RlbLinear* l, void* stream) {
+  if (l->M <= 0 || l->N <= 0 || l->K <= 0) return 0;
+  if ((l->lda % 8) || (l->ldw % 8) || (l->ldo % 8) || (l->N % 8) || (l->K % 8) || l->in_f32 || l->out_f32 || l->tile_expert) return -2;
+  if ((reinterpret_cast<uintptr_t>(l->a) | reinterpret_cast<uintptr_t>(l->w) | reinterpret_cast<uintptr_t>(l->out) | reinterpret_cast<uintptr_t>(l->bias)) & 15) return -3;
+  CUtensorMap ta, tb;
+  int rc = make_operand_maps(l->a, l->w, l->M, l->N, l->K, l->lda, l->ldw, false, false, &ta, &tb);
+  if (rc) return -100 - rc;
+  EpiParams ep{};
+  ep.C = l->out;
+  ep.ldc = l->ldo;
+  ep.layer.act_from = 1 << 30;
+  ep.layer.lin = rlb_linear_epi(*l);
+  return launch_gemm<false, false, EPI_LAYER>(ta, tb, l->M, l->N, l->K, ep, l->status, 0, static_cast<cudaStream_t>(stream));
 }
 
 // Number of n-tiles the vocab-projection epilogues split N into (size of the partial buffers).

@@ -10,6 +10,8 @@
 //   warp 1      tcgen05.mma issuer: S = Q K^T over dim + rot_dim in 16-wide steps, O += P V
 //   warps 2..5  softmax, one thread per query row, stale-maximum rescaling; the epilogue normalises, multiplies by sigmoid(gate) and
 //               writes over the gate columns of the projected rows
+// The same kernel serves grouped-query attention (rlb_flash_gqa): no rotated source of its own (the rotation is in the queries and keys), several
+// query heads per key / value head, keys and values read from column ranges of one matrix, no gate, output rows of their own.
 // Query rows stand at the end of their context: row r of a portion of n tokens in a context of c sees keys up to c - n + r.
 #include "common.cuh"
 
@@ -47,9 +49,13 @@ struct FlashLatentParams {
   int vcols;                       // columns of the PV product: vdim rounded up to 16
   int tmem_cols;
   float scale_log2;
-  __nv_bfloat16* p;
+  __nv_bfloat16* p;                // output rows, first column of head 0 (gated: the gates stand there)
   long long ldp;
   int* status;
+  int per_kv;                      // query heads per key / value head
+  int k_col, v_col;                // first key / value column of kv head 0
+  int ctx_row0;                    // row of the key / value matrix that cu_ctx counts from
+  int gated;
 };
 
 __global__ void __launch_bounds__(LA_THREADS, 2)
@@ -102,7 +108,7 @@ flash_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + 64;
-  const int q_row0 = p.row0 + info[0], n_q = info[1], q0 = info[2] * LA_BQ, c_row0 = info[3], n_ctx = info[4];
+  const int q_row0 = p.row0 + info[0], n_q = info[1], q0 = info[2] * LA_BQ, c_row0 = p.ctx_row0 + info[3], n_ctx = info[4];
   const int q_rows = min(LA_BQ, n_q - q0);
   const int shift = n_ctx - n_q;                                     // query row i of the portion sees keys <= shift + i
   const int n_kv = (shift + q0 + q_rows + LA_BKV - 1) / LA_BKV;
@@ -121,13 +127,13 @@ flash_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
         const int row = c_row0 + j * LA_BKV;
         if (!mbar_wait(smem_u32(k_empty), ph ^ 1, abort_flag, p.status, RLB_ERR_WAIT_EMPTY)) break;
         mbar_arrive_expect_tx(smem_u32(k_full), atoms_q * LA_KV_ATOM);
-        for (int a = 0; a < p.atoms_n; ++a) tma_load_2d(smem_u32(k_s + a * LA_KV_ATOM), &tmap_kv, smem_u32(k_full), head * p.dim + a * 64, row);
+        for (int a = 0; a < p.atoms_n; ++a) tma_load_2d(smem_u32(k_s + a * LA_KV_ATOM), &tmap_kv, smem_u32(k_full), p.k_col + head / p.per_kv * p.dim + a * 64, row);
         for (int a = 0; a < p.atoms_r; ++a)
           tma_load_2d(smem_u32(k_s + (p.atoms_n + a) * LA_KV_ATOM), &tmap_lat, smem_u32(k_full), p.rank + a * 64, row);
         if (!mbar_wait(smem_u32(v_empty), ph ^ 1, abort_flag, p.status, RLB_ERR_WAIT_EMPTY)) break;
         mbar_arrive_expect_tx(smem_u32(v_full), p.atoms_v * LA_KV_ATOM);
         for (int a = 0; a < p.atoms_v; ++a)
-          tma_load_2d(smem_u32(v_s + a * LA_KV_ATOM), &tmap_kv, smem_u32(v_full), p.heads * p.dim + head * p.vdim + a * 64, row);
+          tma_load_2d(smem_u32(v_s + a * LA_KV_ATOM), &tmap_kv, smem_u32(v_full), p.v_col + head / p.per_kv * p.vdim + a * 64, row);
       }
     }
   } else if (warp == 1) {
@@ -242,7 +248,7 @@ flash_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
     if (ok && mbar_wait(smem_u32(v_empty), (n_kv - 1) & 1, abort_flag, p.status, RLB_ERR_WAIT_TMEM_EMPTY)) {
       tc_fence_after();
       const float inv_l = l > 0.f ? 1.f / l : 0.f;
-      __nv_bfloat16* dst = p.p + static_cast<long long>(q_row0 + q0 + r) * p.ldp + p.mix_off + head * p.vdim;
+      __nv_bfloat16* dst = p.p + static_cast<long long>(q_row0 + q0 + r) * p.ldp + p.mix_off + head * p.vdim;      // (gqa: mix_off is 0)
       for (int c = 0; c < p.vdim; c += 32) {
         uint32_t o[32];
         tmem_ld_32x32b_x32(tmem_o + lane_addr + c, o);
@@ -251,8 +257,16 @@ flash_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
 #pragma unroll
           for (int q = 0; q < 4; ++q) {
             if (c + q * 8 < p.vdim) {
-              uint4 g = *reinterpret_cast<uint4*>(dst + c + q * 8);
+              uint4 g = make_uint4(0, 0, 0, 0);
               uint32_t* gw = reinterpret_cast<uint32_t*>(&g);
+              if (!p.gated) {
+#pragma unroll
+                for (int w = 0; w < 4; ++w)
+                  gw[w] = pack_bf16x2(__uint_as_float(o[q * 8 + 2 * w]) * inv_l, __uint_as_float(o[q * 8 + 2 * w + 1]) * inv_l);
+                *reinterpret_cast<uint4*>(dst + c + q * 8) = g;
+                continue;
+              }
+              g = *reinterpret_cast<uint4*>(dst + c + q * 8);
 #pragma unroll
               for (int w = 0; w < 4; ++w) {
                 const float2 gf = unpack_bf16x2(gw[w]);
@@ -287,6 +301,18 @@ __global__ void latent_gather_kernel(const uint4* __restrict__ cache, const long
     }
     out[i] = cache[s * vecs + (i - t * vecs)];
   }
+}
+
+int launch_flash(const CUtensorMap& tq, const CUtensorMap& tkv, const CUtensorMap& tl, const FlashLatentParams& f, int max_tiles, cudaStream_t stream) {
+  const int smem = (f.atoms_n + f.atoms_r) * (LA_Q_ATOM + LA_KV_ATOM) + f.atoms_v * LA_KV_ATOM + LA_P_BYTES + 256 + 1024;
+  static int configured = 0;
+  if (smem > configured) {
+    cudaError_t e = cudaFuncSetAttribute(flash_latent_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    configured = smem;
+  }
+  flash_latent_kernel<<<dim3(max_tiles, f.heads), LA_THREADS, smem, stream>>>(tq, tkv, tl, f);
+  return static_cast<int>(cudaGetLastError());
 }
 }  // namespace
 
@@ -337,6 +363,11 @@ RLB_API int rlb_flash_latent(void* p, long long rows, long long ldp, int in_widt
   f.p = static_cast<__nv_bfloat16*>(p);
   f.ldp = ldp;
   f.status = status;
+  f.per_kv = 1;
+  f.k_col = 0;
+  f.v_col = heads * dim;
+  f.ctx_row0 = 0;
+  f.gated = 1;
   const long long kvw = static_cast<long long>(heads) * (dim + vdim);
   CUtensorMap tq, tkv, tl;
   int rc = rlb_make_tmap_2d(&tq, p, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, in_width, rows, ldp * 2, 64, LA_BQ, CU_TENSOR_MAP_SWIZZLE_128B);
@@ -346,13 +377,44 @@ RLB_API int rlb_flash_latent(void* p, long long rows, long long ldp, int in_widt
   rc = rlb_make_tmap_2d(&tl, lat, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, width, ctx_rows, static_cast<uint64_t>(width) * 2, 64, LA_BKV,
                         CU_TENSOR_MAP_SWIZZLE_128B);
   if (rc) return -100 - rc;
-  const int smem = (f.atoms_n + f.atoms_r) * (LA_Q_ATOM + LA_KV_ATOM) + f.atoms_v * LA_KV_ATOM + LA_P_BYTES + 256 + 1024;
-  static int configured = 0;
-  if (smem > configured) {
-    cudaError_t e = cudaFuncSetAttribute(flash_latent_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    if (e != cudaSuccess) return static_cast<int>(e);
-    configured = smem;
-  }
-  flash_latent_kernel<<<dim3(max_tiles, heads), LA_THREADS, smem, static_cast<cudaStream_t>(stream)>>>(tq, tkv, tl, f);
-  return static_cast<int>(cudaGetLastError());
+  return launch_flash(tq, tkv, tl, f, max_tiles, static_cast<cudaStream_t>(stream));
+}
+
+// Grouped-query attention of prompt portions. p: projected rows with normed and rotated queries at q_off; the portions are its rows
+// [row0, row0 + cu_q[portions]). Keys of kv head g: columns [k_col + g * dim, + dim) of kv [kv_rows, kv_width], values [v_col + g * vdim, + vdim);
+// row ctx_row0 + cu_ctx[i] is the first of portion i's context (kv may be p itself). y [rows, heads * vdim]: outputs. dim a multiple of 16, vdim of 8.
+RLB_API int rlb_flash_gqa(void* p, long long rows, long long ldp, int in_width, int row0, const void* kv, long long kv_rows, long long ldkv, int kv_width,
+                          int ctx_row0, int k_col, int v_col, const int* cu_q, const int* cu_ctx, int portions, int heads, int kv_heads, int dim, int vdim,
+                          int q_off, float scale, int max_tiles, void* y, long long ldy, int* status, void* stream) {
+  if (portions <= 0 || rows <= 0 || max_tiles <= 0) return 0;
+  if (!rlb_flash_latent_supported(dim, 0, vdim, 8) || kv_heads < 1 || heads % kv_heads) return -2;
+  if (ldp % 8 || ldkv % 8 || ldy % 8 || q_off % 8 || k_col % 8 || v_col % 8 || heads > 65535) return -2;
+  if ((reinterpret_cast<uintptr_t>(p) | reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(y)) & 15) return -3;
+  FlashLatentParams f{};
+  f.cu_q = cu_q;
+  f.cu_ctx = cu_ctx;
+  f.portions = portions;
+  f.row0 = row0;
+  f.heads = heads;
+  f.dim = dim;
+  f.vdim = vdim;
+  f.q_off = q_off;
+  f.atoms_n = (dim + 63) / 64;
+  f.atoms_v = (vdim + 63) / 64;
+  f.vcols = (vdim + 15) / 16 * 16;
+  f.tmem_cols = 64 + (vdim + 31) / 32 * 32 <= 128 ? 128 : (64 + (vdim + 31) / 32 * 32 <= 256 ? 256 : 512);
+  f.scale_log2 = scale * LA_LOG2E;
+  f.p = static_cast<__nv_bfloat16*>(y);
+  f.ldp = ldy;
+  f.status = status;
+  f.per_kv = heads / kv_heads;
+  f.k_col = k_col;
+  f.v_col = v_col;
+  f.ctx_row0 = ctx_row0;
+  CUtensorMap tq, tkv;
+  int rc = rlb_make_tmap_2d(&tq, p, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, in_width, rows, ldp * 2, 64, LA_BQ, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (rc) return -100 - rc;
+  rc = rlb_make_tmap_2d(&tkv, kv, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, kv_width, kv_rows, ldkv * 2, 64, LA_BKV, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (rc) return -100 - rc;
+  return launch_flash(tq, tkv, tkv, f, max_tiles, static_cast<cudaStream_t>(stream));
 }

@@ -33,7 +33,7 @@ __device__ __forceinline__ void st<__nv_bfloat16>(__nv_bfloat16* p, float v) {
 }
 
 // ---------------------------------------------------------------- start of the residual stream
-// x = table[id] * scale (kept in e), + step; h = w * tanh(alpha x) + b
+// x = table[id] * scale (kept in e), + step; h = w * tanh(alpha x) + b, or x itself where there is no norm (alpha null)
 template <typename T>
 __global__ void embed_rows_kernel(const void* ids, int ids64, const T* __restrict__ table, float* __restrict__ x, float* __restrict__ e,
                                   T* __restrict__ h, const T* __restrict__ step, const T* __restrict__ alpha, const T* __restrict__ nw,
@@ -44,13 +44,13 @@ __global__ void embed_rows_kernel(const void* ids, int ids64, const T* __restric
     if (threadIdx.x == 0 && status) atomicCAS(status, 0, RLB_ERR_BOUNDS);
     id = 0;
   }
-  const float a = ld(alpha);
+  const float a = alpha ? ld(alpha) : 0.f;
   for (int c = threadIdx.x; c < d; c += blockDim.x) {
     float v = ld(table + id * d + c) * scale;
     if (e) e[row * d + c] = v;
     if (step) v += ld(step + c);
     x[row * d + c] = v;
-    st(h + row * d + c, tanhf(a * v) * ld(nw + c) + ld(nb + c));
+    st(h + row * d + c, alpha ? tanhf(a * v) * ld(nw + c) + ld(nb + c) : v);
   }
 }
 
@@ -69,6 +69,10 @@ struct RowsGemm {
   const void* alpha;
   const void* nw;
   const void* nb;
+  LinearEpi lin;
+  const int* tile_expert;   // expert of each 128-row tile (null: one weight); its weight starts expert * N * ldw further on
+  const int* a_rows;        // row of `a` that each row reads (-1 or out of range: zeros); null: its own
+  int num_a_rows;
 };
 
 constexpr int RG_T = 64, RG_K = 16;
@@ -80,11 +84,21 @@ __global__ void __launch_bounds__(256) gemm_rows_kernel(RowsGemm g) {
   const TI* W = static_cast<const TI*>(g.w);
   const int m0 = blockIdx.y * RG_T, n0 = blockIdx.x * RG_T;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  if (g.tile_expert) {
+    const int e = g.tile_expert[m0 / 128];
+    if (e < 0) return;
+    W += static_cast<long long>(e) * g.N * g.ldw;
+  }
   float acc[4][4] = {};
   for (int k0 = 0; k0 < g.K; k0 += RG_K) {
     for (int i = threadIdx.x; i < RG_T * RG_K; i += 256) {
       const int r = i / RG_K, k = i % RG_K;
-      as[k][r] = (m0 + r < g.M && k0 + k < g.K) ? ld(A + static_cast<long long>(m0 + r) * g.lda + k0 + k) : 0.f;
+      int row = m0 + r < g.M ? m0 + r : -1;
+      if (g.a_rows && row >= 0) {
+        row = g.a_rows[row];
+        if (row >= g.num_a_rows) row = -1;
+      }
+      as[k][r] = (row >= 0 && k0 + k < g.K) ? ld(A + static_cast<long long>(row) * g.lda + k0 + k) : 0.f;
       ws[k][r] = (n0 + r < g.N && k0 + k < g.K) ? ld(W + static_cast<long long>(n0 + r) * g.ldw + k0 + k) : 0.f;
     }
     __syncthreads();
@@ -113,6 +127,21 @@ __global__ void __launch_bounds__(256) gemm_rows_kernel(RowsGemm g) {
       const int n = n0 + tx * 4 + j;
       if (n >= g.N) continue;
       float v = acc[i][j];
+      if (g.lin.bias) v += ld(static_cast<const TI*>(g.lin.bias) + n);
+      if (g.lin.act == LIN_GLU) {          // N is even: the pair of an even column is there
+        if (j & 1) continue;
+        float u = acc[i][j + 1];
+        if (g.lin.bias) u += ld(static_cast<const TI*>(g.lin.bias) + n + 1);
+        st(static_cast<TO*>(g.out) + static_cast<long long>(m) * g.ldo + n / 2, clamped_glu(v, u, g.lin.limit));
+        continue;
+      }
+      if (g.lin.act == LIN_GELU_MUL) {
+        const TI* t = static_cast<const TI*>(g.lin.table) + lin_token(g.lin, m) * g.lin.ld_table + g.lin.table_off;
+        v = n < g.lin.table_cols ? 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v))) * ld(t + n) : 0.f;
+      } else if (g.lin.act == LIN_CAP) {
+        v *= g.lin.scale;
+        if (g.lin.cap > 0.f) v = g.lin.cap * tanhf(v / g.lin.cap);
+      }
       TO* o = static_cast<TO*>(g.out) + static_cast<long long>(m) * g.ldo + n;
       if (g.x) {
         float* xp = g.x + static_cast<long long>(m) * g.ldx + n;
@@ -385,6 +414,16 @@ retention_rows_kernel(T* __restrict__ p, RetentionShape s, int row0, const int* 
   }
 }
 
+int launch_rows(const RowsGemm& g, int in_f32, int out_f32, cudaStream_t s) {
+  const dim3 grid((g.N + RG_T - 1) / RG_T, (g.M + RG_T - 1) / RG_T);
+  if (grid.y > 65535) return -2;
+  if (in_f32 && out_f32) gemm_rows_kernel<float, float><<<grid, 256, 0, s>>>(g);
+  else if (in_f32) gemm_rows_kernel<float, __nv_bfloat16><<<grid, 256, 0, s>>>(g);
+  else if (out_f32) gemm_rows_kernel<__nv_bfloat16, float><<<grid, 256, 0, s>>>(g);
+  else gemm_rows_kernel<__nv_bfloat16, __nv_bfloat16><<<grid, 256, 0, s>>>(g);
+  return static_cast<int>(cudaGetLastError());
+}
+
 int smem_attr(const void* kernel, size_t bytes) {
   if (bytes <= 48 * 1024) return 0;
   if (bytes > 220 * 1024) return -2;
@@ -414,15 +453,17 @@ RLB_API int rlb_gemm_rows(const void* a, const void* w, void* out, int M, int N,
                           const void* nw, const void* nb, void* stream) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   if (x && (!alpha || !nw || !nb)) return -2;
-  RowsGemm g{a, w, out, M, N, K, lda, ldw, ldo, act_from, x, ldx, e, step, alpha, nw, nb};
-  const dim3 grid((N + RG_T - 1) / RG_T, (M + RG_T - 1) / RG_T);
-  if (grid.y > 65535) return -2;
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (in_f32 && out_f32) gemm_rows_kernel<float, float><<<grid, 256, 0, s>>>(g);
-  else if (in_f32) gemm_rows_kernel<float, __nv_bfloat16><<<grid, 256, 0, s>>>(g);
-  else if (out_f32) gemm_rows_kernel<__nv_bfloat16, float><<<grid, 256, 0, s>>>(g);
-  else gemm_rows_kernel<__nv_bfloat16, __nv_bfloat16><<<grid, 256, 0, s>>>(g);
-  return static_cast<int>(cudaGetLastError());
+  RowsGemm g{a, w, out, M, N, K, lda, ldw, ldo, act_from, x, ldx, e, step, alpha, nw, nb, LinearEpi{}, nullptr, nullptr, 0};
+  return launch_rows(g, in_f32, out_f32, static_cast<cudaStream_t>(stream));
+}
+
+// The product of RlbLinear for any sizes, bf16 or fp32, one weight or one per expert.
+RLB_API int rlb_linear_rows(const RlbLinear* l, void* stream) {
+  if (l->M <= 0 || l->N <= 0 || l->K <= 0) return 0;
+  if ((l->act == LIN_GLU && l->N % 2) || (l->tile_expert && l->M % 128)) return -2;
+  RowsGemm g{l->a, l->w, l->out, l->M, l->N, l->K, l->lda, l->ldw, l->ldo, 1 << 30, nullptr, 0, nullptr, nullptr, nullptr, nullptr, nullptr,
+             rlb_linear_epi(*l), l->tile_expert, l->a_rows, l->num_a_rows};
+  return launch_rows(g, l->in_f32, l->out_f32, static_cast<cudaStream_t>(stream));
 }
 
 RLB_API int rlb_latent_prep(void* p, int f32, long long rows, long long ldp, int q_off, int lat_off, int heads, int dim, int rot_dim, int rank,

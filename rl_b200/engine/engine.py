@@ -21,11 +21,14 @@ from typing import Optional, Sequence
 
 import torch
 
+from rl_b200.models.config import RECURRENT_MIXERS
 from rl_b200.models.transformer import CausalLM, PackedBatch
 from rl_b200.ops import engine_ops as E
 from rl_b200.ops import functional as F
+from rl_b200.ops import layer_ops as Y
 from rl_b200.ops import lib as _L
 from rl_b200.ops import mixer_ops as X
+from rl_b200.ops import sequence_ops as S
 from rl_b200.parallel.tensor import gather_cols, row_linear
 
 _P, _I, _LL = C.c_void_p, C.c_int, C.c_longlong
@@ -431,7 +434,7 @@ class GenerationEngine:
         # ``_hybrid_block``. Prefixes are not shared between sequences (pages carry no state) and decode runs eagerly.
         self.hybrid = bool(self.cfg.is_hybrid)
         self._attn_layers = [i for i, l in enumerate(model.layers) if l.self_attn is not None]
-        # layer-list models (Gadarax): one cache or state pool per layer RUN (a looped layer has one per pass), see ``_mixer_forward``
+        # layer-list models (Gadarax, Redarax): one cache or state pool per layer RUN (a looped layer has one per pass), see ``_mixer_forward``
         self.mixer = bool(self.cfg.is_mixer)
         self.runs = self.cfg.layer_runs if self.mixer else []
         self.stateful = bool(self.cfg.is_recurrent)   # sequences own a row of the state pools: prefixes are not shared by pages
@@ -449,7 +452,8 @@ class GenerationEngine:
         self.mamba_conv: Optional[list] = None
         self.mamba_ssm: Optional[list] = None
         self.latent_cache: Optional[list] = None      # per run: [pages, page size, latent width] (latent attention)
-        self.ret_state: Optional[list] = None         # per run: [state rows, heads, dim, vdim] fp32 (retention)
+        self.rec_state: Optional[list] = None         # per run: [state rows, heads, dim, vdim] fp32 (retention, Mamba-2, delta rule)
+        self.conv_ring: Optional[list] = None         # per run: [state rows, taps, channels], last inputs of a short convolution
         self._step_ids: dict = {}                     # requests driven through ``step``: caller's id -> sequence id
         self._step_next = 0
         self._state_row: dict[int, int] = {}
@@ -475,7 +479,7 @@ class GenerationEngine:
                 free, _ = torch.cuda.mem_get_info(self.device)
                 per_block = 2 * max(1, len(self._attn_layers)) * self.hkv * block_size * c.head_dim * 2
                 if self.mixer:
-                    per_block = max(1, sum(self._latent_width(i) for i, _ in self.runs)) * block_size * model.embed_tokens.element_size()
+                    per_block = max(1, sum(self._cache_width(i) for i, _ in self.runs)) * block_size * model.embed_tokens.element_size()
                 num_blocks = max(16, int(free * gpu_memory_utilization) // per_block)
             else:
                 num_blocks = 256
@@ -553,22 +557,27 @@ class GenerationEngine:
             self.mamba_ssm = [torch.zeros((R, c.mamba_num_heads, c.mamba_head_dim, c.ssm_state_size), dtype=torch.float32, device=self.device)
                               if l.kind == "mamba" else None for l in self.model.layers]
 
-    def _latent_width(self, layer: int) -> int:
+    def _cache_width(self, layer: int) -> int:
+        """Elements per token that a layer keeps in pages."""
         m = self.model.layers[layer].mixer
+        if m.kind == "attention":
+            return m.kv_heads * (m.dim + m.vdim)
         return m.latent_width if m.kind == "latent_attention" else 0
 
     def _wake_mixer(self) -> None:
-        """Pools of a layer-list model, one per layer run: latent pages for latent attention, fp32 state rows (row 0 is scratch for the
-        padding rows of a decode batch) for retention."""
-        dt, dev = self.model.dtype, self.device
+        """Pools of a layer-list model, one per layer run: key / value pages for attention, latent pages for latent attention, fp32 state rows
+        (row 0 is scratch for the padding rows of a decode batch) for the recurrent mixers, with the last inputs of their convolution."""
+        dt, dev, n, bs = self.model.dtype, self.device, self.num_blocks, self.block_size
         mx = [self.model.layers[i].mixer for i, _ in self.runs]
-        self.k_cache = self.v_cache = []     # (no key / value pages)
-        self.latent_cache = [torch.zeros((self.num_blocks, self.block_size, m.latent_width), dtype=dt, device=dev)
-                             if m.kind == "latent_attention" else None for m in mx]
-        self.ret_state = [torch.zeros((self.max_running + 1, m.heads, m.dim, m.vdim), dtype=torch.float32, device=dev)
-                          if m.kind == "retention" else None for m in mx]
-        # portions of prompts attend tile-wise when every latent-attention layer has a shape the tensor-core kernel takes
-        self._portion_tiles = self.native and all(X.portion_tiles(m, dt) for m in mx if m.kind == "latent_attention")
+        zeros = lambda *shape, dtype=dt: torch.zeros(shape, dtype=dtype, device=dev)   # noqa: E731
+        self.k_cache = [zeros(n, m.kv_heads, bs, m.dim) if m.kind == "attention" else None for m in mx]
+        self.v_cache = [zeros(n, m.kv_heads, bs, m.vdim) if m.kind == "attention" else None for m in mx]
+        self.latent_cache = [zeros(n, bs, m.latent_width) if m.kind == "latent_attention" else None for m in mx]
+        self.rec_state = [zeros(self.max_running + 1, m.heads, m.dim, m.vdim, dtype=torch.float32) if m.kind in RECURRENT_MIXERS else None for m in mx]
+        self.conv_ring = [zeros(self.max_running + 1, m.taps, m.channels) if hasattr(m, "taps") else None for m in mx]
+        # portions of prompts attend tile-wise when every attention layer has a shape its tensor-core kernel takes
+        tiles = {"latent_attention": X.portion_tiles, "attention": S.portion_tiles}
+        self._portion_tiles = self.native and all(tiles[m.kind](m, dt) for m in mx if m.kind in tiles)
 
     def sleep(self, free_kv_cache: bool = True) -> None:
         """Ends a generation phase: drops all requests; optionally returns the KV cache memory (captured graphs are
@@ -582,14 +591,14 @@ class GenerationEngine:
             self._static = None
             self.k_cache = self.v_cache = None
             self.mamba_conv = self.mamba_ssm = None
-            self.latent_cache = self.ret_state = None
+            self.latent_cache = self.rec_state = self.conv_ring = None
             if self.device.type == "cuda":
                 torch.cuda.empty_cache()
 
     def kv_cache_bytes(self) -> int:
         c = self.cfg
         if self.mixer:
-            return sum(self._latent_width(i) for i, _ in self.runs) * self.num_blocks * self.block_size * self.model.embed_tokens.element_size()
+            return sum(self._cache_width(i) for i, _ in self.runs) * self.num_blocks * self.block_size * self.model.embed_tokens.element_size()
         return 2 * len(self._attn_layers) * self.num_blocks * self.hkv * self.block_size * c.head_dim * self.model.dtype.itemsize if hasattr(self.model.dtype, "itemsize") else 0
 
     # ------------------------------------------------------------------ routed-expert recording (rollout routing replay)
@@ -861,6 +870,8 @@ class GenerationEngine:
         Per layer run: fused input product, mixer, fused output product; the last one's epilogue also updates the fp32 residual
         stream, makes the loop's additions and applies the next layer's norm."""
         m, c, runs = self.model, self.cfg, self.runs
+        if c.norm_place == "post":
+            return self._post_norm_forward(b, rows)
         norms = [m.layers[i].norm for i, _ in runs] + [m.norm]
 
         def begins(r):    # (embeddings are added again, step vector) when run r is the first of a pass of the loop
@@ -876,12 +887,32 @@ class GenerationEngine:
             if mx.kind == "latent_attention":
                 X.latent_attention_(p, mx, b, self.latent_cache[r])
             else:
-                X.retention_(p, mx, b, self.ret_state[r])
+                X.retention_(p, mx, b, self.rec_state[r])
             again, step = begins(r + 1)
             h = X.out_proj_(x, p[:, mx.mix_off : mx.mix_off + layer.out_width], layer.out_proj, e if again else None, step, norms[r + 1])
         if rows is not None:
             h = h.index_select(0, rows)
         return X.logits(h, m.output_weight, self.logits_dtype)
+
+    def _post_norm_forward(self, b: "X.TokenBatch", rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """``_mixer_forward`` of post-norm layers. Each sublayer is a product, the mixer or gated unit, a product, and the step that norms its
+        output and joins it to the fp32 stream; the last one of all applies the final norm."""
+        m, c = self.model, self.cfg
+        mult, eps, last = c.residual_mult, c.rms_norm_eps, len(self.runs) - 1
+        x, h = Y.embed(b.ids, m.embed_tokens, c.embed_scale)
+        for r, (i, _) in enumerate(self.runs):
+            layer = m.layers[i]
+            mx, end = layer.mixer, m.norm if r == last else None      # the final norm rides on the last join
+            p = Y.linear(h, mx.in_proj, mx.in_bias)
+            a = S.attention(p, mx, b, self.k_cache[r], self.v_cache[r]) if mx.kind == "attention" else S.recurrent(p, mx, b, self.conv_ring[r], self.rec_state[r])
+            h = Y.add_normed_(x, Y.linear(a, mx.out_proj, mx.out_bias), layer.norm1, mult, eps, end if layer.ff is None and not layer.side_dim else None)
+            if layer.ff is not None:
+                h = Y.feed_forward_(x, h, layer.ff, layer.norm2, mult, eps, end if not layer.side_dim else None)
+            if layer.side_dim:
+                h = Y.token_side_(x, h, b.ids, layer, m.side_embed, mult, eps, end)
+        if rows is not None:
+            h = h.index_select(0, rows)
+        return Y.capped_logits(h, m.output_weight, c.logit_scale, c.final_logit_softcap, self.logits_dtype)
 
     def _token_batch(self, items) -> tuple:
         """Rows of one step from ``items`` = [(sequence id, tokens, first position)]. Single tokens come first, then portions in order of
@@ -914,9 +945,12 @@ class GenerationEngine:
             cu[1, 1:] = torch.tensor(ctx, dtype=torch.int64).cumsum(0)
             cu = cu.to(dev)
             b.cu_q, b.cu_ctx, b.q_tiles = cu[0], cu[1], sum(-(-lens[j] // 128) for j in tiled)
+            b.whole = all(items[order[j]][2] == 0 for j in tiled)
             b.ctx_slots = torch.cat([self.sched.slots(sids[j], 0, n) for j, n in zip(tiled, ctx)]).to(dev)
         if self.stateful:
-            b.state_rows = torch.tensor([self._state_row[s] for s in sids], dtype=torch.int64, device=dev)
+            srow = torch.tensor([self._state_row[s] for s in sids], dtype=torch.int64)
+            b.state_rows, b.row_state = srow.to(dev), srow[of_row].to(dev)
+            b.row_off = torch.cat([torch.arange(n, dtype=torch.int32) for n in lens]).to(dev)
         if n_single < len(lens):
             cu = torch.zeros(len(lens) - n_single + 1, dtype=torch.int32)
             cu[1:] = torch.tensor(lens[n_single:], dtype=torch.int64).cumsum(0)
@@ -1549,6 +1583,11 @@ class GenerationEngine:
                         if cache is not None:
                             raw = cache.view(torch.bfloat16)
                             E.block_copy(raw, raw, src, dst)
+                    for kc, vc in zip(self.k_cache, self.v_cache) if self.mixer else ():
+                        if kc is not None:
+                            for cache in (kc, vc):
+                                raw = cache.view(torch.bfloat16)
+                                E.block_copy(raw, raw, src, dst)
                     for li in self._attn_layers:
                         E.block_copy(self.k_cache[li], self.v_cache[li], src, dst)
                 new = list(prefill) + list(shared)

@@ -1,0 +1,212 @@
+"""Row operators of post-norm layers (``rl_b200/models/post_norm.py``) in the generation engine: products with what follows them, the
+normed join with the residual stream, the gated feed-forwards and the token input.
+
+Each operator has the native sm_100a body (CUDA tensors, bf16 or fp32) and a plain PyTorch statement (CPU tensors). ``x`` is the fp32
+residual stream, updated in place; ``h`` what the next sublayer reads (x in the model's type). fp32 models run every product in true fp32.
+"""
+
+from __future__ import annotations
+
+import ctypes as C
+from typing import Optional
+
+import torch
+import torch.nn.functional as TF
+
+from . import functional as F
+from . import lib as _L
+from .lib import F as CF
+from .lib import I, L as LL, P, call, ptr, register, stream_ptr, use_native
+from .mixer_ops import _aligned, _f32
+
+register("rlb_linear_rows", [P, P])
+register("rlb_linear_tiled", [P, P])
+register("rlb_linear_skinny", [P, P])
+register("rlb_linear_grouped", [P, P])
+register("rlb_add_normed", [P, P, LL, I, P, P, I, I, P, I, P, P, P, LL, I, CF, CF, P])
+register("rlb_group_norm_rows", [P, LL, I, P, LL, I, I, CF, P])
+register("rlb_cap_rows", [P, LL, CF, CF, P])
+register("rlb_moe_choose", [P, LL, I, I, P, I, I, I, P, P, P, P, P])
+register("rlb_moe_place", [P, P, LL, I, P, I, I, P, P, P, P, LL, P, I, P, P])
+
+NONE, GLU, GELU_MUL, CAP = range(4)      # what follows a product (RlbLinearAct)
+
+
+class _Linear(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("a", "w", "out", "bias", "table", "ids", "tile_expert", "a_rows", "status")] + \
+               [(n, C.c_longlong) for n in ("lda", "ldw", "ldo", "ld_table")] + \
+               [(n, C.c_int) for n in ("M", "N", "K", "in_f32", "out_f32", "act", "table_off", "table_cols", "vocab", "ids64", "experts", "num_a_rows")] + \
+               [(n, C.c_float) for n in ("limit", "scale", "cap")]
+
+
+def _desc(a, w, out, act=NONE, limit=0.0, bias=None) -> _Linear:
+    d = _Linear()
+    d.a, d.w, d.out, d.bias, d.status = ptr(a), ptr(w), ptr(out), ptr(bias), ptr(_L.status_word(a.device))
+    d.M, (d.N, d.K) = a.shape[0], w.shape[-2:]
+    d.lda, d.ldw, d.ldo = a.stride(0), w.stride(-2), out.stride(0)
+    d.in_f32, d.out_f32, d.act, d.limit = _f32(a), _f32(out), act, limit
+    return d
+
+
+def _run(d: _Linear, fast: bool) -> None:
+    name = "rlb_linear_rows"
+    if fast and d.N % 8 == 0 and d.K % 8 == 0:
+        if d.M <= 256 and d.K >= 256:
+            name = "rlb_linear_skinny"
+        elif not d.out_f32:
+            name = "rlb_linear_tiled"
+    call(name, C.byref(d), stream_ptr())
+
+
+def clamped_glu_ref(p: torch.Tensor, limit: float) -> torch.Tensor:
+    g, u = p[:, 0::2].float().clamp(max=limit), p[:, 1::2].float().clamp(-limit, limit)
+    return (g * torch.sigmoid(1.702 * g) * (u + 1)).to(p.dtype)
+
+
+def linear(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, glu: Optional[float] = None) -> torch.Tensor:
+    """a w^T (+ bias); ``glu``: the limit of a clamped gated unit over neighbouring columns, half as wide."""
+    if not use_native(a):
+        p = a @ w.t() if bias is None else a @ w.t() + bias
+        return p if glu is None else clamped_glu_ref(p, glu)
+    out = torch.empty((a.shape[0], w.shape[0] // (1 if glu is None else 2)), dtype=a.dtype, device=a.device)
+    _run(_desc(a, w, out, NONE if glu is None else GLU, glu or 0.0, bias), _aligned(a, w, out))
+    return out
+
+
+# --------------------------------------------------------------------------------------- residual stream
+def embed(ids: torch.Tensor, table: torch.Tensor, scale: float):
+    """(x, h): the tokens' rows in fp32 and in the model's type."""
+    if not use_native(table):
+        x = table[ids.long()].float() * scale
+        return x, x.to(table.dtype)
+    T, d = ids.shape[0], table.shape[1]
+    x = torch.empty((T, d), dtype=torch.float32, device=table.device)
+    h = torch.empty((T, d), dtype=table.dtype, device=table.device)
+    call("rlb_embed_rows", ptr(ids), int(ids.dtype == torch.int64), ptr(table), _f32(table), ptr(x), None, ptr(h), None, None, None, None, T, d,
+         table.shape[0], float(scale), ptr(_L.status_word(table.device)), stream_ptr())
+    return x, h
+
+
+def _rms(x: torch.Tensor, eps: float) -> torch.Tensor:
+    return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+
+
+def add_normed_(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, mult: float, eps: float, next_norm: Optional[torch.Tensor] = None,
+                experts: Optional[tuple] = None) -> torch.Tensor:
+    """x += mult * rms(y) * w in place; returns x in the model's type, or rms(x) * next_norm. ``experts`` = (row of every copy, weight of
+    every copy, the experts' counts to reset): y holds expert rows, a token's value is the weighted sum of its copies' rows."""
+    if not use_native(x):
+        x += mult * (_rms(y.float(), eps) * w.float())
+        return (x if next_norm is None else _rms(x, eps) * next_norm.float()).to(w.dtype)
+    T, d = x.shape
+    h = torch.empty((T, d), dtype=w.dtype, device=x.device)
+    rows, wt, counts = experts if experts is not None else (None, None, None)
+    call("rlb_add_normed", ptr(x), ptr(y), y.stride(0), _f32(y), ptr(rows), ptr(wt), wt.shape[1] if wt is not None else 0, y.shape[0], ptr(counts),
+         counts.numel() if counts is not None else 0, ptr(w), ptr(next_norm), ptr(h), T, d, float(mult), float(eps), stream_ptr())
+    return h
+
+
+def group_norm_(y: torch.Tensor, w: torch.Tensor, groups: int, eps: float) -> None:
+    """The leading w.numel() columns of ``y`` in ``groups`` equal parts, each over its root mean square, times w; in place."""
+    n = w.numel()
+    if not use_native(y):
+        y[:, :n] = (_rms(y[:, :n].float().view(y.shape[0], groups, -1), eps).reshape(-1, n) * w.float()).to(y.dtype)
+        return
+    call("rlb_group_norm_rows", ptr(y), y.stride(0), _f32(y), ptr(w), y.shape[0], groups, n // groups, float(eps), stream_ptr())
+
+
+# --------------------------------------------------------------------------------------- feed-forwards
+def feed_forward_(x: torch.Tensor, h: torch.Tensor, ff, norm: torch.Tensor, mult: float, eps: float, next_norm=None) -> torch.Tensor:
+    """x += mult * rms(ff(h)) * norm. ``ff``: the layer's ``ClampedGLU`` or ``ClampedExperts``."""
+    if hasattr(ff, "router"):
+        y, experts = clamped_experts(h, ff)
+        return add_normed_(x, y, norm, mult, eps, next_norm, experts)
+    return add_normed_(x, linear(linear(h, ff.gate_up, glu=ff.limit), ff.down), norm, mult, eps, next_norm)
+
+
+def clamped_experts(h: torch.Tensor, m):
+    """(expert rows, (row of every copy, weights, counts)) on the native path, (summed outputs, None) otherwise."""
+    T, d = h.shape
+    if not use_native(h):
+        w, idx = m.choose(h.float() @ m.router.float().t())
+        y = torch.zeros((T, d), dtype=torch.float32)
+        for e in range(m.experts):
+            tok, slot = (idx == e).nonzero(as_tuple=True)
+            if tok.numel():
+                y.index_add_(0, tok, (clamped_glu_ref(h[tok] @ m.gate_up[e].t(), m.limit) @ m.down[e].t()).float() * w[tok, slot, None])
+        return y, None
+    dev, E, k = h.device, m.experts, m.top
+    st = ptr(_L.status_word(dev))
+    z = router_logits(h, m.router)
+    wt = torch.empty((T, k), dtype=torch.float32, device=dev)
+    idx, rank, copy_row = torch.empty((3, T, k), dtype=torch.int32, device=dev)
+    counts = _expert_counts(m, dev)
+    call("rlb_moe_choose", ptr(z), z.stride(0), T, E, ptr(m.correction), m.groups, m.keep, k, ptr(wt), ptr(idx), ptr(rank), ptr(counts), stream_ptr())
+    mpad = -(-(T * k + E * 127) // 128) * 128
+    tiles = torch.empty(mpad // 128, dtype=torch.int32, device=dev)
+    fast = _aligned(h, m.gate_up[0], m.down[0]) and m.gate_up.shape[1] % 8 == 0 and d % 8 == 0
+    xp = torch.empty((mpad, d), dtype=h.dtype, device=dev) if fast else h
+    src = None if fast else torch.full((mpad,), -1, dtype=torch.int32, device=dev)
+    call("rlb_moe_place", ptr(idx), ptr(rank), T * k, k, ptr(counts), E, mpad, ptr(copy_row), ptr(tiles), ptr(src), ptr(h),
+         h.stride(0) * h.element_size() if fast else 0, ptr(xp) if fast else None, d * h.element_size() if fast else 0, st, stream_ptr())
+    a = torch.empty((mpad, m.down.shape[2]), dtype=h.dtype, device=dev)
+    y = torch.empty((mpad, d), dtype=h.dtype, device=dev)
+    for first, inp, w, out in ((True, xp, m.gate_up, a), (False, a, m.down, y)):
+        q = _desc(inp, w, out, GLU if first else NONE, m.limit)
+        q.M, q.experts, q.tile_expert = mpad, E, ptr(tiles)
+        if first and not fast:
+            q.a_rows, q.num_a_rows = ptr(src), T
+        call("rlb_linear_grouped" if fast else "rlb_linear_rows", C.byref(q), stream_ptr())
+    return y, (copy_row, wt, counts)
+
+
+def router_logits(h: torch.Tensor, router: torch.Tensor) -> torch.Tensor:
+    if _aligned(h, router) and router.shape[0] % 8 == 0 and router.shape[1] % 8 == 0:
+        return F.gemm(h, router, out_dtype=torch.float32)
+    z = torch.empty((h.shape[0], router.shape[0]), dtype=torch.float32, device=h.device)
+    _run(_desc(h, router, z), False)
+    return z
+
+
+_COUNTS: dict = {}
+
+
+def _expert_counts(m, dev) -> torch.Tensor:
+    """Zeros that the router counts in and the join resets: one buffer per device serves all layers of a stream's step."""
+    c = _COUNTS.get((dev, m.experts))
+    if c is None:
+        c = _COUNTS[(dev, m.experts)] = torch.zeros(m.experts, dtype=torch.int32, device=dev)
+    return c
+
+
+# --------------------------------------------------------------------------------------- token input, logits
+def token_side_(x: torch.Tensor, h: torch.Tensor, ids: torch.Tensor, layer, table: torch.Tensor, mult: float, eps: float, next_norm=None) -> torch.Tensor:
+    """x += mult * rms(proj(gelu(gate h) * e)) * norm with e the tokens' rows of the layer's columns of ``table``."""
+    n, off = layer.side_dim, layer.layer_idx * layer.side_dim
+    if not use_native(h):
+        e = table[ids.long()][:, off : off + n].float()
+        g = TF.pad(TF.gelu((h @ layer.side_gate.t()).float(), approximate="tanh")[:, :n] * e, (0, layer.side_gate.shape[0] - n)).to(h.dtype)
+    else:
+        g = torch.empty((h.shape[0], layer.side_gate.shape[0]), dtype=h.dtype, device=h.device)
+        d = _desc(h, layer.side_gate, g, GELU_MUL)
+        d.table, d.ld_table, d.table_off, d.table_cols, d.vocab = ptr(table), table.stride(0), off, n, table.shape[0]
+        d.ids, d.ids64 = ptr(ids), int(ids.dtype == torch.int64)
+        _run(d, _aligned(h, layer.side_gate, g))
+    return add_normed_(x, linear(g, layer.side_proj), layer.side_norm, mult, eps, next_norm)
+
+
+def capped_logits(h: torch.Tensor, w: torch.Tensor, scale: float, cap: float, out_dtype: torch.dtype = torch.float32) -> torch.Tensor:
+    """(h w^T) * scale, soft-capped where cap > 0."""
+    if not use_native(h):
+        z = (h.float() @ w.float().t()) * scale
+        return (cap * torch.tanh(z / cap) if cap else z).to(out_dtype)
+    z = torch.empty((h.shape[0], w.shape[0]), dtype=torch.float32, device=h.device)
+    ok = _aligned(h, w) and w.shape[0] % 8 == 0 and w.shape[1] % 8 == 0
+    if ok and (h.shape[0] > 256 or h.shape[1] < 256):
+        F.gemm(h, w, out=z)
+        call("rlb_cap_rows", ptr(z), z.numel(), float(scale), float(cap), stream_ptr())
+    elif z.numel():
+        d = _desc(h, w, z, CAP)
+        d.scale, d.cap = float(scale), float(cap)
+        _run(d, ok)
+    return z.to(out_dtype)

@@ -80,6 +80,9 @@ class TokenBatch:
     cu_ctx: Optional[torch.Tensor] = None       # int32
     ctx_slots: Optional[torch.Tensor] = None    # int64
     q_tiles: int = 0                 # 128-row query tiles of those portions
+    row_off: Optional[torch.Tensor] = None      # int32 [T]: rows of the same piece before each row (None: all rows are singles)
+    row_state: Optional[torch.Tensor] = None    # int64 [T]: state row of each row's sequence (None: ``state_rows``)
+    whole: bool = False              # the tile-wise portions start at position 0
     max_ctx: int = 0                 # upper bound of seq_lens (a host number, fixed while a graph is captured)
 
     @property

@@ -1,0 +1,142 @@
+"""Sequence mixers of post-norm layers in the generation engine: grouped-query attention over paged keys and values, and the recurrent
+mixers with a short convolution (Mamba-2, gated delta rule), over a batch of token rows that mixes single decoded tokens and portions of
+prompts (``mixer_ops.TokenBatch``).
+
+Each operator takes the projected rows ``p`` of the layer's mixer module and returns the rows [T, mix_width] that its output product reads.
+CUDA tensors run the native kernels: tensor-core forms for bf16 shapes they take, kernels for any size otherwise and for fp32 models;
+CPU tensors run the plain PyTorch statement.
+"""
+
+from __future__ import annotations
+
+import torch
+
+from . import engine_ops as E
+from . import lib as _L
+from .layer_ops import group_norm_
+from .lib import F as CF
+from .lib import I, L as LL, P, call, ptr, register, stream_ptr, use_native
+from .mixer_ops import TokenBatch, _f32, _page_rows
+
+register("rlb_gqa_prep", [P, I, LL, LL, I, I, I, I, I, I, I, I, I, P, P, P, P, P, I, CF, CF, P, P, P, P])
+register("rlb_gqa_rows", [P, I, I, LL, I, I, I, I, I, I, I, P, P, P, I, P, CF, P, LL, P, P])
+register("rlb_gqa_gather", [P, P, P, P, LL, I, I, I, I, LL, P, P])
+register("rlb_flash_gqa", [P, LL, LL, I, I, P, LL, LL, I, I, I, I, P, P, I, I, I, I, I, I, CF, I, P, LL, P, P])
+register("rlb_conv_rows", [P, I, LL, P, LL, LL, I, I, P, P, P, P, P, P, LL, P, P])
+register("rlb_conv_state", [P, I, LL, I, I, P, I, I, P, P, P, LL, P])
+register("rlb_mamba2_rows", [P, I, LL, P, LL, P, LL, I, I, I, I, I, I, I, I, P, P, P, P, LL, P, P, P, P, P])
+register("rlb_delta_rows", [P, I, LL, P, LL, P, LL, I, I, I, I, I, I, I, I, I, P, P, P, P, LL, P, P, P, CF, CF, P, P])
+
+
+def _rows_out(p: torch.Tensor, m) -> torch.Tensor:
+    n = m.heads * m.vdim
+    return (torch.zeros if m.mix_width > n else torch.empty)((p.shape[0], m.mix_width), dtype=p.dtype, device=p.device)
+
+
+# --------------------------------------------------------------------------------------- attention
+def attention(p: torch.Tensor, m, b: TokenBatch, k_cache: torch.Tensor, v_cache: torch.Tensor) -> torch.Tensor:
+    """``m``: the layer's ``GroupedAttentionMixer``; caches [pages, kv_heads, page size, dim / vdim]. The rows' own keys and values are
+    written first; ``p`` is left with normed and rotated queries and keys."""
+    bs, H, G = k_cache.shape[2], m.heads, m.kv_heads
+    y = _rows_out(p, m)
+    if not use_native(p):
+        q, k, v = m.qkv(p, b.positions)
+        ok = b.slots >= 0
+        page, off = (b.slots[ok] // bs).long(), (b.slots[ok] % bs).long()
+        k_cache[page, :, off], v_cache[page, :, off] = k[ok].to(k_cache.dtype), v[ok].to(v_cache.dtype)
+        q = q.to(p.dtype).float()
+        for i in range(p.shape[0]):
+            n = int(b.seq_lens[i])
+            if n == 0:
+                y[i] = 0
+                continue
+            rows = _page_rows(b.block_table[i], n, bs)
+            ks, vs = (c[rows // bs, :, rows % bs].float().transpose(0, 1) for c in (k_cache, v_cache))      # [kv_heads, n, dim]
+            w = torch.softmax(q[i].view(G, H // G, m.dim) @ ks.transpose(1, 2) * m.scale, dim=-1)
+            y[i, : H * m.vdim] = (w @ vs).reshape(-1).to(p.dtype)
+        return y
+    T, st = p.shape[0], ptr(_L.status_word(p.device))
+    call("rlb_gqa_prep", ptr(p), _f32(p), T, p.stride(0), m.q_off, m.k_off, m.v_off, H, G, m.dim, m.vdim, bs, k_cache.shape[0], ptr(b.positions),
+         ptr(b.slots), ptr(m.q_norm), ptr(m.k_norm), ptr(m.freq), m.freq.numel(), float(m.gain), float(m.eps), ptr(k_cache), ptr(v_cache), st, stream_ptr())
+    if b.n_paged:
+        if decode_tiles(p, m, bs):
+            splits = E.choose_splits(b.n_paged, G, max(b.max_ctx // 2, 1), bs)
+            E.paged_decode(p[: b.n_paged, m.q_off : m.q_off + H * m.dim], k_cache, v_cache, b.block_table, b.seq_lens, H, G, m.dim, scale=m.scale,
+                           num_splits=splits, out=y[: b.n_paged])
+        else:
+            call("rlb_gqa_rows", ptr(p), _f32(p), b.n_paged, p.stride(0), m.q_off, H, G, m.dim, m.vdim, bs, k_cache.shape[0], ptr(k_cache),
+                 ptr(v_cache), ptr(b.block_table), b.block_table.stride(0), ptr(b.seq_lens), float(m.scale), ptr(y), y.stride(0), st, stream_ptr())
+    if b.n_paged < T:
+        if b.whole:       # nothing cached before these portions: their keys and values stand in the projected rows
+            kv, rows, row0, k0, v0 = p, T, b.n_paged, m.k_off, m.v_off
+        else:
+            rows, row0, k0, v0 = b.ctx_slots.numel(), 0, 0, G * m.dim
+            kv = torch.empty((rows, G * (m.dim + m.vdim)), dtype=p.dtype, device=p.device)
+            call("rlb_gqa_gather", ptr(k_cache), ptr(v_cache), ptr(b.ctx_slots), ptr(kv), rows, G, m.dim, m.vdim, bs, k_cache.shape[0] * bs, st, stream_ptr())
+        call("rlb_flash_gqa", ptr(p), T, p.stride(0), p.shape[1], b.n_paged, ptr(kv), rows, kv.stride(0), kv.shape[1], row0, k0, v0, ptr(b.cu_q),
+             ptr(b.cu_ctx), b.cu_q.numel() - 1, H, G, m.dim, m.vdim, m.q_off, float(m.scale), b.q_tiles, ptr(y), y.stride(0), st, stream_ptr())
+    return y
+
+
+def decode_tiles(p: torch.Tensor, m, block_size: int) -> bool:
+    """Whether the tensor-core decode kernel takes this layer's shape."""
+    return p.dtype == torch.bfloat16 and m.dim == 128 and m.vdim == 128 and m.heads // m.kv_heads <= 8 and block_size in (16, 32, 64)
+
+
+def portion_tiles(m, dtype: torch.dtype) -> bool:
+    """Whether the tensor-core prefill kernel takes this layer's shape."""
+    return dtype == torch.bfloat16 and m.dim % 16 == 0 and m.vdim % 8 == 0 and bool(_L.lib().rlb_flash_latent_supported(m.dim, 0, m.vdim, 8))
+
+
+# --------------------------------------------------------------------------------------- recurrent mixers
+def _pieces(b: TokenBatch) -> list:
+    cuts = list(range(b.n_single)) + ([b.n_single + c for c in b.cu.tolist()] if b.cu is not None else [b.n_single])
+    return list(zip(cuts[:-1], cuts[1:]))
+
+
+def recurrent(p: torch.Tensor, m, b: TokenBatch, ring: torch.Tensor, state: torch.Tensor, plain: bool = False) -> torch.Tensor:
+    """Mamba-2 or delta-rule mixing of all rows: every sequence's row of ``ring`` [rows, taps, channels] (the convolution's last inputs, by
+    position modulo taps) and of ``state`` [rows, heads, dim, vdim] (fp32) is advanced by its tokens; a piece that starts at position 0
+    starts from zeros. ``plain``: the token-by-token kernels for every shape (they serve fp32 models and odd sizes)."""
+    y = _rows_out(p, m)
+    if not use_native(p):
+        return _recurrent_ref(p, m, b, ring, state, y)
+    st, T = ptr(_L.status_word(p.device)), p.shape[0]
+    x = p[:, m.conv_off : m.conv_off + m.channels]
+    u = torch.empty((T, -(-m.channels // 8) * 8), dtype=p.dtype, device=p.device)
+    call("rlb_conv_rows", ptr(x), _f32(p), p.stride(0), ptr(u), u.stride(0), T, m.channels, m.taps, ptr(m.conv), ptr(m.conv_bias), ptr(ring),
+         ptr(b.positions), ptr(b.row_off), ptr(b.row_state if b.row_state is not None else b.state_rows), ring.shape[0], st, stream_ptr())
+    for row0, pieces, cu, rows in ((0, b.n_single, None, b.state_rows),
+                                   (b.n_single, b.cu.numel() - 1 if b.cu is not None else 0, b.cu, b.state_rows[b.n_single :])):
+        if not pieces:
+            continue
+        if m.taps > 1:
+            call("rlb_conv_state", ptr(x), _f32(p), p.stride(0), row0, pieces, ptr(cu), m.channels, m.taps, ptr(ring), ptr(b.positions), ptr(rows),
+                 ring.shape[0], stream_ptr())
+        if m.kind == "mamba2":
+            call("rlb_mamba2_rows", ptr(u), _f32(p), u.stride(0), ptr(p), p.stride(0), ptr(y), y.stride(0), m.z_off, m.dt_off, m.heads, m.groups, m.dim,
+                 m.vdim, row0, pieces, ptr(cu), ptr(b.positions), ptr(rows), ptr(state), state.shape[0], ptr(m.A_log), ptr(m.dt_bias), ptr(m.D), st,
+                 stream_ptr())
+        else:
+            call("rlb_delta_rows", ptr(u), _f32(p), u.stride(0), ptr(p), p.stride(0), ptr(y), y.stride(0), m.g_off, m.b_off, m.a_off, m.heads,
+                 m.kv_heads, m.dim, m.vdim, row0, pieces, ptr(cu), ptr(b.positions), ptr(rows), ptr(state), state.shape[0], ptr(m.A_log),
+                 ptr(m.dt_bias), ptr(m.norm), float(m.unit_eps), float(m.eps), st, stream_ptr())
+    if m.kind == "mamba2":
+        group_norm_(y, m.norm, m.norm_groups, m.eps)
+    return y
+
+
+def _recurrent_ref(p, m, b, ring, state, y):
+    n = m.taps - 1
+    for j, (s, e) in enumerate(_pieces(b)):
+        r, pos = int(b.state_rows[j]), int(b.positions[s])
+        before = torch.stack([ring[r, t % m.taps] if t >= 0 else torch.zeros_like(ring[r, 0]) for t in range(pos - n, pos)]) if n else p.new_zeros(0, m.channels)
+        x = p[s:e, m.conv_off : m.conv_off + m.channels]
+        u = m.convolve(x, before)
+        S = state[r] if pos else torch.zeros_like(state[r])
+        o, S = m.scan(u, p[s:e], S)
+        y[s:e, : m.heads * m.vdim] = m.finish(o, p[s:e]).reshape(e - s, -1)
+        state[r] = S
+        for t in range(max(s, e - n), e):
+            ring[r, (pos + t - s) % m.taps] = x[t - s]
+    return y
