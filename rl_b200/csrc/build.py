@@ -31,7 +31,7 @@ NVCC_FLAGS = [
     "--use_fast_math",
 ]
 # sources whose tanh / sine / cosine / exponential / division must be the accurate ones
-PRECISE = {"mixers.cu", "retention.cu", "layers.cu", "attention.cu", "recurrent.cu", "ssd.cu", "delta.cu"}
+PRECISE = {"mixers.cu", "retention.cu", "layers.cu", "attention.cu", "recurrent.cu", "recurrent_tiles.cu"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread"]
 
 

@@ -1,5 +1,5 @@
 // Recurrent mixers with a short convolution (Mamba2LayerMixer, DeltaMixer) one token after another, for every size and for bf16 and fp32
-// models. The chunked and single-step forms for bf16 are in ssd.cu and delta.cu.
+// models. The chunked and single-step forms for bf16 are in recurrent_tiles.cu.
 //
 // State of a sequence: the last inputs of the convolution, a ring [taps, channels] indexed by position % taps in the model's type, and
 // S [heads, dim, vdim] in fp32. A piece that starts at position 0 starts from zeros, whatever its rows held before.

@@ -14,7 +14,7 @@
 // Decode: one CTA per (row, head) streams the fp32 state once (read, decay, rank-one update, write, dot with q).
 //
 // This file is compiled without fast math.
-#include "common.cuh"
+#include "recurrent.cuh"
 
 #include <math.h>
 
@@ -37,10 +37,7 @@ struct RetShape {
   int* status;
 };
 
-constexpr int RT_C = 128;                 // tokens per chunk
 constexpr int RT_THREADS = 512;
-constexpr int RT_ATOM = RT_C * 128;       // 128 rows x 64 columns of bf16
-constexpr int RT_SATOM = 64 * 128;        // 64 state rows x 64 value columns
 
 __global__ void rotation_table_kernel(const int* __restrict__ positions, const float* __restrict__ freq, int half, float gain, float* __restrict__ cs,
                                       long long n) {
@@ -54,21 +51,6 @@ __global__ void rotation_table_kernel(const int* __restrict__ positions, const f
   }
 }
 
-__device__ __forceinline__ uint32_t rt_sw(int row, int piece) { return row * 128 + ((piece ^ (row & 7)) << 4); }
-
-// Splits 8 fp32 values into bf16 high and low parts and stores them as 16-byte pieces.
-__device__ __forceinline__ void store_split(uint8_t* hi, uint8_t* lo, uint32_t off, const float (&v)[8]) {
-  uint32_t h[4], l[4];
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    h[i] = pack_bf16x2(v[2 * i], v[2 * i + 1]);
-    const float2 hf = unpack_bf16x2(h[i]);
-    l[i] = pack_bf16x2(v[2 * i] - hf.x, v[2 * i + 1] - hf.y);
-  }
-  *reinterpret_cast<uint4*>(hi + off) = make_uint4(h[0], h[1], h[2], h[3]);
-  *reinterpret_cast<uint4*>(lo + off) = make_uint4(l[0], l[1], l[2], l[3]);
-}
-
 // Eight consecutive dimensions d0.. of one head's row: the raw piece and, where the halves layout rotates whole pieces, its partner.
 struct RawPiece {
   uint4 own, other;
@@ -79,15 +61,6 @@ __device__ __forceinline__ RawPiece load_piece(const __nv_bfloat16* row, int d0,
   if (d0 < 2 * half && half % 8 == 0) r.other = *reinterpret_cast<const uint4*>(row + (d0 < half ? d0 + half : d0 - half));
   else r.other = make_uint4(0, 0, 0, 0);
   return r;
-}
-__device__ __forceinline__ void unpack8(const uint4& r, float (&v)[8]) {
-  const uint32_t w[4] = {r.x, r.y, r.z, r.w};
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const float2 f = unpack_bf16x2(w[i]);
-    v[2 * i] = f.x;
-    v[2 * i + 1] = f.y;
-  }
 }
 // The rotation of that piece in fp32 (d0 a multiple of 8).
 __device__ __forceinline__ void rotate_piece(const RawPiece& raw, const __nv_bfloat16* row, int d0, int half, const float* cs, float (&v)[8]) {

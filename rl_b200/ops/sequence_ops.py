@@ -9,6 +9,8 @@ CPU tensors run the plain PyTorch statement.
 
 from __future__ import annotations
 
+import ctypes as C
+
 import torch
 
 from . import engine_ops as E
@@ -26,6 +28,19 @@ register("rlb_conv_rows", [P, I, LL, P, LL, LL, I, I, P, P, P, P, P, P, LL, P, P
 register("rlb_conv_state", [P, I, LL, I, I, P, I, I, P, P, P, LL, P])
 register("rlb_mamba2_rows", [P, I, LL, P, LL, P, LL, I, I, I, I, I, I, I, I, P, P, P, P, LL, P, P, P, P, P])
 register("rlb_delta_rows", [P, I, LL, P, LL, P, LL, I, I, I, I, I, I, I, I, I, P, P, P, P, LL, P, P, P, CF, CF, P, P])
+register("rlb_rec_supported", [I, I, I])
+register("rlb_conv_runs", [P, LL, P, LL, LL, I, I, P, P, P, P, P, P, LL, P, P])
+register("rlb_rec_step", [P, P])
+register("rlb_rec_portions", [P, P])
+
+
+class _RecArgs(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("p", "u", "conv_w", "conv_bias", "A_log", "dt_bias", "D", "norm", "y", "ring", "positions", "piece_chunk",
+                                          "chunk_row", "chunk_rows", "state_rows", "state", "cum", "wt", "unit", "start", "u0", "w_hi", "w_lo", "kt_hi",
+                                          "kt_lo", "uu_hi", "uu_lo", "status")] + \
+               [(n, C.c_longlong) for n in ("ldp", "ldu", "ldy", "num_states", "rows")] + \
+               [(n, C.c_int) for n in ("delta", "heads", "groups", "dim", "vdim", "taps", "channels", "conv_off", "gate_off", "a_off", "b_off", "row0",
+                                       "pieces", "chunks")] + [("unit_eps", C.c_float), ("eps", C.c_float)]
 
 
 def _rows_out(p: torch.Tensor, m) -> torch.Tensor:
@@ -101,6 +116,11 @@ def recurrent(p: torch.Tensor, m, b: TokenBatch, ring: torch.Tensor, state: torc
     y = _rows_out(p, m)
     if not use_native(p):
         return _recurrent_ref(p, m, b, ring, state, y)
+    if not plain and rec_tiles(p, m):
+        _recurrent_tiles(p, m, b, ring, state, y)
+        if m.kind == "mamba2":
+            group_norm_(y, m.norm, m.norm_groups, m.eps)
+        return y
     st, T = ptr(_L.status_word(p.device)), p.shape[0]
     x = p[:, m.conv_off : m.conv_off + m.channels]
     u = torch.empty((T, -(-m.channels // 8) * 8), dtype=p.dtype, device=p.device)
@@ -124,6 +144,56 @@ def recurrent(p: torch.Tensor, m, b: TokenBatch, ring: torch.Tensor, state: torc
     if m.kind == "mamba2":
         group_norm_(y, m.norm, m.norm_groups, m.eps)
     return y
+
+
+def rec_tiles(p: torch.Tensor, m) -> bool:
+    """Whether the tensor-core and single-step kernels take this layer's shape."""
+    return p.dtype == torch.bfloat16 and m.conv_off % 8 == 0 and p.stride(0) % 8 == 0 and \
+        bool(_L.lib().rlb_rec_supported(int(m.kind == "delta"), m.dim, m.vdim))
+
+
+def _recurrent_tiles(p, m, b, ring, state, y) -> None:
+    dev, T, delta = p.device, p.shape[0], m.kind == "delta"
+    H, G = m.heads, m.kv_heads if delta else m.groups
+    st = ptr(_L.status_word(dev))
+    a = _RecArgs()
+    a.p, a.y, a.ldp, a.ldy, a.rows, a.status = ptr(p), ptr(y), p.stride(0), y.stride(0), T, st
+    a.conv_w, a.conv_bias, a.A_log, a.dt_bias, a.norm = ptr(m.conv), ptr(m.conv_bias), ptr(m.A_log), ptr(m.dt_bias), ptr(m.norm) if delta else None
+    a.D = None if delta else ptr(m.D)
+    a.ring, a.state, a.num_states, a.positions = ptr(ring), ptr(state), state.shape[0], ptr(b.positions)
+    a.delta, a.heads, a.groups, a.dim, a.vdim, a.taps, a.channels, a.conv_off = int(delta), H, G, m.dim, m.vdim, m.taps, m.channels, m.conv_off
+    a.gate_off, a.a_off, a.b_off = (m.g_off, m.a_off, m.b_off) if delta else (m.z_off, m.dt_off, -1)
+    a.unit_eps, a.eps = float(m.unit_eps) if delta else 0.0, float(m.eps)
+    if b.n_single:
+        a.pieces, a.state_rows = b.n_single, ptr(b.state_rows)
+        call("rlb_rec_step", C.byref(a), stream_ptr())
+    if b.cu is None:
+        return
+    n0, n, pieces = b.n_single, b.chunk_row.numel(), b.cu.numel() - 1
+    R, x = T - n0, p[n0:, m.conv_off : m.conv_off + m.channels]
+    u = torch.empty((T, -(-m.channels // 8) * 8), dtype=p.dtype, device=dev)
+    uv, rows = u[n0:], b.state_rows[n0:]
+    if 2 <= m.taps <= 4 and m.channels % 8 == 0:
+        call("rlb_conv_runs", ptr(x), p.stride(0), ptr(uv), u.stride(0), R, m.channels, m.taps, ptr(m.conv), ptr(m.conv_bias), ptr(ring),
+             ptr(b.positions[n0:]), ptr(b.row_off[n0:]), ptr(b.row_state[n0:]), ring.shape[0], st, stream_ptr())
+    else:
+        call("rlb_conv_rows", ptr(x), 0, p.stride(0), ptr(uv), u.stride(0), R, m.channels, m.taps, ptr(m.conv), ptr(m.conv_bias), ptr(ring),
+             ptr(b.positions[n0:]), ptr(b.row_off[n0:]), ptr(b.row_state[n0:]), ring.shape[0], st, stream_ptr())
+    if m.taps > 1:
+        call("rlb_conv_state", ptr(p[:, m.conv_off :]), 0, p.stride(0), n0, pieces, ptr(b.cu), m.channels, m.taps, ptr(ring), ptr(b.positions), ptr(rows),
+             ring.shape[0], stream_ptr())
+    f32 = lambda *s: torch.empty(s, dtype=torch.float32, device=dev)   # noqa: E731
+    cw, start = f32(2, H, R), f32(n, H, m.dim, m.vdim)
+    a.cum, a.wt, a.start = ptr(cw[0]), ptr(cw[1]), ptr(start)
+    if delta:
+        unit, u0 = f32(2, G, R), f32(n * H, 128, m.vdim)
+        tiles, writes = torch.empty((4, n * H * 128, 128), dtype=p.dtype, device=dev), torch.empty((2, R, H * m.vdim), dtype=p.dtype, device=dev)
+        a.unit, a.u0 = ptr(unit), ptr(u0)
+        a.w_hi, a.w_lo, a.kt_hi, a.kt_lo = (ptr(t) for t in tiles)
+        a.uu_hi, a.uu_lo = ptr(writes[0]), ptr(writes[1])
+    a.u, a.ldu, a.row0, a.pieces, a.chunks, a.state_rows = ptr(u), u.stride(0), n0, pieces, n, ptr(rows)
+    a.piece_chunk, a.chunk_row, a.chunk_rows = ptr(b.piece_chunk), ptr(b.chunk_row), ptr(b.chunk_rows)
+    call("rlb_rec_portions", C.byref(a), stream_ptr())
 
 
 def _recurrent_ref(p, m, b, ring, state, y):
