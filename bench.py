@@ -4,6 +4,7 @@
     python bench.py --config qwen3-32b-tp4dp2 --gpus 8 ...   (other model / layout configurations, see CONFIGS)
     python bench.py --config refit-sweep --gpus 8            (weight re-shard times, trainer layout -> serving layouts)
     python bench.py --config gadarax-serving                 (prefill / decode of a layer-list model beside Llama at equal size)
+    python bench.py --config redarax-serving                 (the same for a post-norm layer-list model, beside Qwen3-MoE)
     python bench.py --impl reference ...                     (the unmodified reference, when it can be installed)
 
 Default (headline) configuration ``llama8b-dp``: one GRPO step (generation + refit + log-probabilities + training) on
@@ -49,6 +50,7 @@ CONFIGS = {
                               train_mb_tokens=8192, logprob_mb_tokens=16384, act_ckpt="on"),
     "refit-sweep": dict(),
     "gadarax-serving": dict(),
+    "redarax-serving": dict(),
 }
 
 
@@ -171,10 +173,12 @@ def main() -> int:
 
         return sweep_main(steps=args.steps, warmup=args.warmup)
 
-    if args.config == "gadarax-serving":
+    if args.config in ("gadarax-serving", "redarax-serving"):
         from rl_b200.csrc.build import build_all
-        from rl_b200.engine.bench_mixers import main as serving_main
+        from rl_b200.engine import bench_mixers
         from rl_b200.ops import lib as L
+
+        serving_main = bench_mixers.main if args.config == "gadarax-serving" else bench_mixers.redarax_main
 
         if not L.available():
             build_all()

@@ -1,7 +1,7 @@
-"""Serving throughput of layer-list models (Gadarax) beside the Llama architecture at equal size, and the kernels' distance from
-their rooflines beside the like kernels of the Llama path.
+"""Serving throughput of layer-list models beside the framework's closest model at equal size (Gadarax: the Llama architecture, Redarax:
+Qwen3-MoE), and the kernels' distance from their rooflines beside the like kernels of the closest path.
 
-    python bench.py --config gadarax-serving [--steps K --warmup W]
+    python bench.py --config gadarax-serving | redarax-serving [--steps K --warmup W]
 
 Random weights, random prompts. Whole-model figures come from ``GenerationEngine``: prefill of packed prompts (device time of the
 forward pass) and decoding through the captured step (device time of the graph replays). Kernel figures are CUDA-event times of a
@@ -28,6 +28,7 @@ SIZES = {   # (preset, Llama twin: same width and run count, MHA with 128-wide h
     "gadarax-1b": dict(hidden_size=2048, num_attention_heads=16),
     "gadarax-4b": dict(hidden_size=4096, num_attention_heads=32),
 }
+REDARAX = ("redarax-2b", "redarax-7b")
 PREFILL = ((1, 4096), (8, 1024))      # (prompts, tokens each)
 DECODE = ((16, 4096), (64, 2048))     # (sequences, context)
 
@@ -49,6 +50,19 @@ def llama_twin(name: str) -> ModelConfig:
     ff = round((mean - 4 * d * d) / (3 * d) / 128) * 128
     return ModelConfig(model_type="llama", vocab_size=c.vocab_size, intermediate_size=ff, num_hidden_layers=len(runs), head_dim=128,
                        num_key_value_heads=base["num_attention_heads"], rms_norm_eps=1e-5, rope_theta=500000.0, tie_word_embeddings=True, **base)
+
+
+def moe_twin(name: str) -> ModelConfig:
+    """Qwen3-MoE model of the same width, layers, attention heads, experts and choice, the experts' width set for the same number of weights."""
+    c = preset(name)
+    att = next(e["mixer"] for e in c.mixers if e["type"] == "attention")
+    r = next(e["mlp"]["router"] for e in c.mixers if e["mlp"] and e["mlp"]["kind"] == "moe")
+    t = ModelConfig(model_type="qwen3_moe", vocab_size=c.vocab_size, hidden_size=c.hidden_size, intermediate_size=c.intermediate_size,
+                    num_hidden_layers=c.num_hidden_layers, num_attention_heads=att["heads"], num_key_value_heads=att["kv_heads"], head_dim=att["dim"],
+                    rms_norm_eps=1e-6, rope_theta=1e6, qk_norm=True, num_experts=r["experts"], num_experts_per_tok=r["top"], moe_intermediate_size=0)
+    per = c.num_hidden_layers * r["experts"] * 3 * c.hidden_size
+    t.moe_intermediate_size = round((c.num_parameters() - t.num_parameters()) / per / 64) * 64
+    return t
 
 
 def timed(fn, steps: int, warmup: int) -> float:
@@ -174,27 +188,6 @@ def kernel_table(name: str) -> list:
         roof = max(flops / pk["flops"], nbytes / pk["hbm"]) * 1e3
         out.append(dict(kernel=label, ms=round(ms, 4), roofline_ms=round(roof, 4), fraction=round(roof / ms, 3)))
 
-    def copies(make, nbytes):
-        return [make() for _ in range(max(2, min(24, math.ceil(200e6 / max(1, nbytes)))))]
-
-    def rows_batch(n, ctx):
-        pages = ctx // 64
-        bt = torch.arange(n * pages, dtype=torch.int32, device=dev).view(n, pages)
-        pos = torch.full((n,), ctx - 1, dtype=torch.int32, device=dev)
-        return X.TokenBatch(ids=None, positions=pos, slots=bt[:, -1].long() * 64 + 63, n_single=n, n_paged=n, block_table=bt,
-                            seq_lens=pos + 1, state_rows=torch.arange(n, device=dev), max_ctx=ctx)
-
-    def portion_batch(n, length):
-        T, pages = n * length, length // 64
-        cu = torch.arange(n + 1, dtype=torch.int32, device=dev) * length
-        slots = torch.arange(T, device=dev)
-        pos = torch.arange(length, dtype=torch.int32, device=dev).repeat(n)
-        pc, cr, cn = (t.to(dev) for t in X.chunk_lists([length] * n))
-        bt = torch.zeros((0, pages), dtype=torch.int32, device=dev)
-        return X.TokenBatch(ids=None, positions=pos, slots=slots, n_single=0, n_paged=0, block_table=bt, seq_lens=pos[:0],
-                            state_rows=torch.arange(n, device=dev), cu=cu, piece_chunk=pc, chunk_row=cr, chunk_rows=cn, cu_q=cu, cu_ctx=cu,
-                            ctx_slots=slots, q_tiles=n * -(-length // 128))
-
     with torch.no_grad():
         # products (decode and prefill rows)
         for T in (64, 4096):
@@ -279,30 +272,185 @@ def kernel_table(name: str) -> list:
     return out
 
 
+def copies(make, nbytes):
+    """Buffer sets that together are larger than L2."""
+    return [make() for _ in range(max(2, min(24, math.ceil(200e6 / max(1, nbytes)))))]
+
+
+def rows_batch(n, ctx, dev="cuda"):
+    pages = ctx // 64
+    bt = torch.arange(n * pages, dtype=torch.int32, device=dev).view(n, pages)
+    pos = torch.full((n,), ctx - 1, dtype=torch.int32, device=dev)
+    return X.TokenBatch(ids=None, positions=pos, slots=bt[:, -1].long() * 64 + 63, n_single=n, n_paged=n, block_table=bt, seq_lens=pos + 1,
+                        state_rows=torch.arange(n, device=dev), max_ctx=ctx)
+
+
+def portion_batch(n, length, dev="cuda"):
+    T, pages = n * length, length // 64
+    cu = torch.arange(n + 1, dtype=torch.int32, device=dev) * length
+    pos = torch.arange(length, dtype=torch.int32, device=dev).repeat(n)
+    pc, cr, cn = (t.to(dev) for t in X.chunk_lists([length] * n))
+    return X.TokenBatch(ids=None, positions=pos, slots=torch.arange(T, device=dev), n_single=0, n_paged=0, seq_lens=pos[:0],
+                        block_table=torch.zeros((0, pages), dtype=torch.int32, device=dev), state_rows=torch.arange(n, device=dev), cu=cu, piece_chunk=pc,
+                        chunk_row=cr, chunk_rows=cn, cu_q=cu, cu_ctx=cu, ctx_slots=torch.arange(T, device=dev), q_tiles=n * -(-length // 128), whole=True,
+                        row_off=pos, row_state=torch.arange(n, device=dev).repeat_interleave(length))
+
+
+def redarax_table(name: str) -> list:
+    """``kernel_table`` of a post-norm layer-list preset."""
+    from rl_b200.models.mixers import RetentionMixer
+    from rl_b200.models.moe import MoEMLP
+    from rl_b200.ops import layer_ops as Y
+    from rl_b200.ops import sequence_ops as S
+
+    pk, c, dev, bf = peaks(), preset(name), "cuda", torch.bfloat16
+    model = build_model(c, device=dev, dtype=bf, seed=0)
+    pick = lambda kind: next(l for l in model.layers if l.mixer.kind == kind)   # noqa: E731
+    d, out = c.hidden_size, []
+
+    def add(label, ms, flops=0.0, nbytes=0.0):
+        roof = max(flops / pk["flops"], nbytes / pk["hbm"]) * 1e3
+        out.append(dict(kernel=label, ms=round(ms, 4), roofline_ms=round(roof, 4), fraction=round(roof / ms, 3)))
+
+    rows = lambda T, n: torch.randn(T, n, device=dev).to(bf)   # noqa: E731
+    with torch.no_grad():
+        # products with what follows them
+        dl, at = pick("delta"), pick("attention")
+        glu = next(l.ff for l in model.layers if l.ff is not None and not hasattr(l.ff, "router"))
+        for T in (64, 4096):
+            for label, w, bias, lim in (("delta in_proj", dl.mixer.in_proj, None, None), ("attention in_proj + bias", at.mixer.in_proj, at.mixer.in_bias, None),
+                                        ("out_proj", dl.mixer.out_proj, None, None), ("gate_up + clamped unit", glu.gate_up, None, glu.limit)):
+                N, K = w.shape
+                nb = 2 * (N * K + T * (K + (N if lim is None else N // 2)))
+                sets = copies(lambda: (rows(T, K), w.detach().clone()), nb)
+                add(f"{label} [{N} x {K}], {T} rows", timed_graph([lambda s=s: Y.linear(s[0], s[1], bias, lim) for s in sets]), 2.0 * T * N * K, nb)
+                add("like: plain GEMM", timed_graph([lambda s=s: F.gemm(s[0], s[1]) for s in sets]), 2.0 * T * N * K, 2 * (N * K + T * (N + K)))
+                del sets
+            # the join beside the residual add + RMS norm of the closest model
+            sets = copies(lambda: (torch.randn(T, d, device=dev), rows(T, d), rows(T, d)), 12 * T * d)
+            add(f"join: x += m norm(y), {T} rows", timed_graph([lambda s=s: Y.add_normed_(s[0], s[1], dl.norm1, 0.5, 1e-6) for s in sets]), 0.0, 12 * T * d)
+            add("like: RMS norm", timed_graph([lambda s=s: F.rmsnorm(s[1], dl.norm1, 1e-6) for s in sets]), 0.0, 4 * T * d)
+            # token input
+            sd = c.token_side["dim"]
+            ids = torch.randint(0, c.vocab_size, (T,), device=dev, dtype=torch.int32)
+            nb = 2 * (2 * sd * d + T * (d + 3 * sd)) + 12 * T * d
+            sets = copies(lambda: (torch.randn(T, d, device=dev), rows(T, d)), nb)
+            add(f"token input (all kernels), {T} rows", timed_graph([lambda s=s: Y.token_side_(s[0], s[1], ids, dl, model.side_embed, 0.5, 1e-6) for s in sets]),
+                4.0 * T * d * sd, nb)
+            add("like: its two products as plain GEMMs", timed_graph([lambda s=s: F.gemm(F.gemm(s[1], dl.side_gate), dl.side_proj) for s in sets]), 4.0 * T * d * sd,
+                2 * (2 * sd * d + T * (2 * d + 2 * sd)))
+            # experts
+            ff = next(l.ff for l in model.layers if hasattr(l.ff, "router"))
+            mc = ModelConfig(model_type="qwen3_moe", hidden_size=d, num_experts=ff.experts, num_experts_per_tok=ff.top, moe_intermediate_size=ff.ff)
+            twin = MoEMLP(mc, bf, dev)
+            for prm in twin.parameters():
+                prm.normal_(std=0.02)
+            used = min(ff.experts, T * ff.top)
+            nb = 2 * (3 * used * d * ff.ff + T * ff.top * (2 * d + 2 * ff.ff)) + 12 * T * d
+            fl = 6.0 * T * ff.top * d * ff.ff
+            sets = copies(lambda: (torch.randn(T, d, device=dev), rows(T, d)), 16 * T * d)
+            ms = timed_graph([lambda s=s: Y.feed_forward_(s[0], s[1], ff, dl.norm1, 0.5, 1e-6) for s in sets[:4]])
+            add(f"experts with router and join (all kernels), {T} rows", ms, fl, nb)
+            ms = timed(lambda: twin(sets[0][1], sets[1][1]), 5, 3) if T > 256 else timed_graph([lambda s=s: twin(s[1], s[1]) for s in sets[:4]])
+            add(f"like: Qwen3-MoE block, {T} rows", ms, fl, nb - 8 * T * d)
+            del sets, twin
+        # attention
+        m = at.mixer
+        H, G = m.heads, m.kv_heads
+        for n, ctx in DECODE:
+            b = rows_batch(n, ctx)
+            nb = n * ctx * G * (m.dim + m.vdim) * 2
+            sets = copies(lambda: (rows(n, m.in_width), *(torch.randn(n * ctx // 64, G, 64, w, device=dev).to(bf) for w in (m.dim, m.vdim))), nb)
+            add(f"attention decode (all kernels), {n} x {ctx}", timed_graph([lambda s=s: S.attention(s[0], m, b, s[1], s[2]) for s in sets]), 4.0 * n * ctx * H * m.dim, nb)
+            sp = E.choose_splits(n, G, ctx // 2, 64)
+            add("like: paged decode attention", timed_graph([lambda s=s: E.paged_decode(s[0][:, : H * m.dim], s[1], s[2], b.block_table, b.seq_lens, H, G, m.dim,
+                                                                                      num_splits=sp) for s in sets]), 4.0 * n * ctx * H * m.dim, nb)
+            del sets
+        for n, length in PREFILL:
+            b, T, pairs = portion_batch(n, length), n * length, n * length * length / 2
+            kc, vc = (torch.zeros((T // 64, G, 64, w), dtype=bf, device=dev) for w in (m.dim, m.vdim))
+            nb = 2 * T * (m.in_width + m.mix_width + G * (m.dim + m.vdim))
+            sets = copies(lambda: rows(T, m.in_width), nb)
+            add(f"attention prefill (all kernels), {n} x {length}", timed_graph([lambda s=s: S.attention(s, m, b, kc, vc) for s in sets]), 2.0 * pairs * H * (m.dim + m.vdim), nb)
+            add("like: flash attention", timed_graph([lambda s=s: F.attention_varlen(s, b.cu_q, length, H, G, m.dim) for s in sets]), 4.0 * pairs * H * m.dim, nb)
+            del sets
+        # recurrent mixers beside retention at the same heads and state
+        class RC:
+            rms_norm_eps = 1e-6
+
+        for kind in ("mamba2", "delta"):
+            m = pick(kind).mixer
+            ret = RetentionMixer(dict(heads=m.heads, dim=m.dim, vdim=m.vdim, rot={"dims": m.dim, "base": 1e4}, decay=[0.99] * m.heads), RC, bf, dev)
+            G = m.groups if kind == "mamba2" else m.kv_heads
+            for n, _ in DECODE:
+                b = rows_batch(n, 64)
+                nb = n * m.heads * m.dim * m.vdim * 8
+                sets = copies(lambda: (rows(n, m.in_width), torch.randn(n, m.taps, m.channels, device=dev).to(bf), torch.randn(n, m.heads, m.dim, m.vdim, device=dev),
+                                       rows(n, ret.in_width)), nb)
+                add(f"{kind} decode (all kernels), {n} rows", timed_graph([lambda s=s: S.recurrent(s[0], m, b, s[1], s[2]) for s in sets]), 0.0, nb)
+                add("like: retention decode", timed_graph([lambda s=s: X.retention_(s[3], ret, b, s[2]) for s in sets]), 0.0, nb)
+                del sets
+            for n, length in PREFILL:
+                b, T, C = portion_batch(n, length), n * length, X.CHUNK
+                ring, st = torch.zeros((n, m.taps, m.channels), dtype=bf, device=dev), torch.zeros((n, m.heads, m.dim, m.vdim), device=dev)
+                sets = copies(lambda: (rows(T, m.in_width), rows(T, ret.in_width)), 2 * T * (m.in_width + ret.in_width))
+                states = (T // C) * m.heads * m.dim * m.vdim * 16
+                nb = 2 * T * (3 * m.channels + 2 * m.heads * m.vdim) + states       # in, convolved, read; gate, out; chunk states
+                fl = 2.0 * T * m.heads * (C / 2 * (m.dim + m.vdim) + 2 * m.dim * m.vdim)
+                if kind == "delta":      # K K^T, T K, T V, W S more; W, keys, values and writes of the chunks
+                    fl += 2.0 * T * m.heads * (C / 2 * (2 * m.dim + m.vdim) + m.dim * m.vdim)
+                    nb += 2 * T * m.heads * (4 * m.dim * 2 + 2 * m.vdim * 2 + 2 * m.vdim * 2)
+                add(f"{kind} prefill (all kernels), {n} x {length}", timed_graph([lambda s=s: S.recurrent(s[0], m, b, ring, st) for s in sets]), fl, nb)
+                nb = 2 * T * m.heads * (3 * m.dim + 3 * m.vdim) + states
+                add("like: retention prefill", timed_graph([lambda s=s: X.retention_(s[1], ret, b, st) for s in sets]),
+                    2.0 * T * m.heads * (C / 2 * (m.dim + m.vdim) + 2 * m.dim * m.vdim), nb)
+                del sets
+    return out
+
+
+def redarax_main(steps: int = 5, warmup: int = 3, sizes=None, clocks=None) -> int:
+    torch.backends.cuda.matmul.allow_tf32 = False
+    L.lib()
+    res = dict(metric="post-norm layer-list model serving (device time)", unit="tokens/s", dtype="bf16", data="synthetic (random weights and tokens)", models={}, kernels={})
+    for name in sizes or REDARAX:
+        for kind in ("redarax", "qwen3_moe"):
+            res["models"][f"{name}:{kind}"] = serving_row(preset(name) if kind == "redarax" else moe_twin(name), steps, warmup)
+        res["kernels"][name] = redarax_table(name)
+        torch.cuda.empty_cache()
+    return finish(res, clocks)
+
+
+def serving_row(cfg: ModelConfig, steps: int, warmup: int) -> dict:
+    row = dict(weights_gb=round(2e-9 * cfg.num_parameters(), 2), runs=len(cfg.layer_runs))
+    need = max(max(n * c for n, c in DECODE), max(n * c for n, c in PREFILL))
+    eng = engine_for(cfg, need, max(n for n, _ in DECODE), max(c for _, c in DECODE) + 64)
+    for n, length in PREFILL:
+        ms = prefill_ms(eng, n, length, steps, warmup)
+        row[f"prefill {n}x{length}"] = dict(ms=round(ms, 3), tokens_per_s=round(n * length / ms * 1e3))
+    for n, ctx in DECODE:
+        ms = decode_ms(eng, n, ctx, steps, warmup)
+        row[f"decode {n}x{ctx}"] = dict(ms=round(ms, 3), tokens_per_s=round(n / ms * 1e3))
+    eng.sleep(True)
+    del eng
+    torch.cuda.empty_cache()
+    return row
+
+
+def finish(res: dict, clocks) -> int:
+    res["status"] = L.check_status()
+    if clocks is not None:
+        res["clocks"] = clocks()
+    print(json.dumps(res), flush=True)
+    return 0
+
+
 def main(steps: int = 5, warmup: int = 3, sizes=None, clocks=None) -> int:
     torch.backends.cuda.matmul.allow_tf32 = False
     L.lib()
     res = dict(metric="layer-list model serving (device time)", unit="tokens/s", dtype="bf16", data="synthetic (random weights and tokens)", models={}, kernels={})
     for name in sizes or SIZES:
         for kind in ("gadarax", "llama"):
-            cfg = preset(name) if kind == "gadarax" else llama_twin(name)
-            row = dict(weights_gb=round(2e-9 * cfg.num_parameters(), 2), runs=len(cfg.layer_runs))
-            need = max(max(n * c for n, c in DECODE), max(n * c for n, c in PREFILL))
-            eng = engine_for(cfg, need, max(n for n, _ in DECODE), max(c for _, c in DECODE) + 64)
-            for n, length in PREFILL:
-                ms = prefill_ms(eng, n, length, steps, warmup)
-                row[f"prefill {n}x{length}"] = dict(ms=round(ms, 3), tokens_per_s=round(n * length / ms * 1e3))
-            for n, ctx in DECODE:
-                ms = decode_ms(eng, n, ctx, steps, warmup)
-                row[f"decode {n}x{ctx}"] = dict(ms=round(ms, 3), tokens_per_s=round(n / ms * 1e3))
-            res["models"][f"{name}:{kind}"] = row
-            eng.sleep(True)
-            del eng
-            torch.cuda.empty_cache()
+            res["models"][f"{name}:{kind}"] = serving_row(preset(name) if kind == "gadarax" else llama_twin(name), steps, warmup)
         res["kernels"][name] = kernel_table(name)
         torch.cuda.empty_cache()
-    res["status"] = L.check_status()
-    if clocks is not None:
-        res["clocks"] = clocks()
-    print(json.dumps(res), flush=True)
-    return 0
+    return finish(res, clocks)
