@@ -30,78 +30,121 @@ struct GqaShape {
   int block_size, num_blocks;
 };
 
-// One warp per head of a row: RMS norm and rotation of a query or key head in place, keys and values into the cache. A lane keeps pairs
-// (2i, 2i + 1), which is also what the rotation turns.
+// One CTA per row, a warp per head in turn: RMS norm and rotation of the query and key heads in place, keys and values into the cache. The
+// row's cosines and sines are computed once for all heads. A lane keeps pairs (2i, 2i + 1), which is also what the rotation turns. Few rows
+// are spread over several CTAs each (blockIdx.y).
 constexpr int GP_WARPS = 8, GP_KEEP = 4;      // pairs a lane keeps in registers
+template <typename T>
+struct Pair;
+template <>
+struct Pair<float> {
+  static __device__ __forceinline__ float2 load(const float* p, bool aligned) { return aligned ? *reinterpret_cast<const float2*>(p) : make_float2(p[0], p[1]); }
+  static __device__ __forceinline__ void store(float* p, float a, float b, bool aligned) {
+    if (aligned) {
+      *reinterpret_cast<float2*>(p) = make_float2(a, b);
+    } else {
+      p[0] = a;
+      p[1] = b;
+    }
+  }
+};
+template <>
+struct Pair<__nv_bfloat16> {
+  static __device__ __forceinline__ float2 load(const __nv_bfloat16* p, bool aligned) {
+    return aligned ? unpack_bf16x2(*reinterpret_cast<const uint32_t*>(p)) : make_float2(__bfloat162float(p[0]), __bfloat162float(p[1]));
+  }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, float a, float b, bool aligned) {
+    if (aligned) {
+      *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(a, b);
+    } else {
+      p[0] = __float2bfloat16(a);
+      p[1] = __float2bfloat16(b);
+    }
+  }
+};
+
 template <typename T>
 __global__ void __launch_bounds__(GP_WARPS * 32)
 gqa_prep_kernel(T* __restrict__ p, GqaShape s, const int* __restrict__ positions, const long long* __restrict__ slots, const T* __restrict__ q_norm,
                 const T* __restrict__ k_norm, const float* __restrict__ freq, int half, float gain, float eps, T* __restrict__ k_cache,
                 T* __restrict__ v_cache, int* status) {
-  pdl_sync();
+  extern __shared__ float2 turn[];      // [half] (cosine, sine)
   const int lane = threadIdx.x & 31;
   const long long row = blockIdx.x;
-  const int unit = blockIdx.y * GP_WARPS + (threadIdx.x >> 5);
-  if (unit >= s.heads + 2 * s.kv_heads) return;
-  T* pr = p + row * s.ldp;
-  const bool is_q = unit < s.heads, is_k = !is_q && unit < s.heads + s.kv_heads;
-  const int head = is_q ? unit : (is_k ? unit - s.heads : unit - s.heads - s.kv_heads);
+  pdl_sync();
+  const float pos = static_cast<float>(positions[row]);
   const long long slot = slots[row];
+  for (int i = threadIdx.x; i < half; i += GP_WARPS * 32) {
+    float sn, cs;
+    sincosf(pos * freq[i], &sn, &cs);
+    turn[i] = make_float2(cs * gain, sn * gain);
+  }
+  T* pr = p + row * s.ldp;
   const bool bad = slot >= static_cast<long long>(s.num_blocks) * s.block_size;
-  if (bad && lane == 0 && status) atomicCAS(status, 0, RLB_ERR_BOUNDS);
+  if (bad && threadIdx.x == 0 && status) atomicCAS(status, 0, RLB_ERR_BOUNDS);
   const bool cached = slot >= 0 && !bad;
   const long long page = cached ? slot / s.block_size : 0, off = cached ? slot % s.block_size : 0;
-  if (!is_q && !is_k) {
-    if (!cached) return;
-    const T* v = pr + s.v_off + head * s.vdim;
-    T* c = v_cache + ((page * s.kv_heads + head) * s.block_size + off) * s.vdim;
-    for (int i = lane; i < s.vdim; i += 32) c[i] = v[i];
-    return;
-  }
-  T* x = pr + (is_q ? s.q_off : s.k_off) + head * s.dim;
-  const T* w = is_q ? q_norm : k_norm;
-  T* c = is_k && cached ? k_cache + ((page * s.kv_heads + head) * s.block_size + off) * s.dim : nullptr;
+  const bool even = s.dim % 2 == 0 && s.ldp % 2 == 0, veven = s.vdim % 2 == 0 && s.ldp % 2 == 0;      // pairs are aligned
   const int pairs = (s.dim + 1) / 2;
-  float u[GP_KEEP], v[GP_KEEP];
-  float ss = 0.f;
-#pragma unroll
-  for (int j = 0; j < GP_KEEP; ++j) {
-    const int i = lane + j * 32;
-    u[j] = 2 * i < s.dim ? ldf(x + 2 * i) : 0.f;
-    v[j] = 2 * i + 1 < s.dim ? ldf(x + 2 * i + 1) : 0.f;
-    ss += u[j] * u[j] + v[j] * v[j];
-  }
-  for (int i = lane + GP_KEEP * 32; i < pairs; i += 32) {
-    const float a = ldf(x + 2 * i), b = 2 * i + 1 < s.dim ? ldf(x + 2 * i + 1) : 0.f;
-    ss += a * a + b * b;
-  }
-  ss = warp_sum(ss);
-  const float rstd = 1.f / sqrtf(ss / static_cast<float>(s.dim) + eps);
-  const float pos = static_cast<float>(positions[row]);
-  auto finish = [&](int i, float a, float b) {
-    if (2 * i >= s.dim) return;
-    const bool two = 2 * i + 1 < s.dim;
-    a *= rstd * ldf(w + 2 * i);
-    if (two) b *= rstd * ldf(w + 2 * i + 1);
-    if (i < half) {
-      float sn, cs;
-      sincosf(pos * freq[i], &sn, &cs);
-      sn *= gain;
-      cs *= gain;
-      const float a0 = a;
-      a = a0 * cs - b * sn;
-      b = b * cs + a0 * sn;
+  __syncthreads();
+  for (int unit = blockIdx.y * GP_WARPS + (threadIdx.x >> 5); unit < s.heads + 2 * s.kv_heads; unit += gridDim.y * GP_WARPS) {
+    const bool is_q = unit < s.heads, is_k = !is_q && unit < s.heads + s.kv_heads;
+    const int head = is_q ? unit : (is_k ? unit - s.heads : unit - s.heads - s.kv_heads);
+    if (!is_q && !is_k) {
+      if (!cached) continue;
+      const T* v = pr + s.v_off + head * s.vdim;
+      T* c = v_cache + ((page * s.kv_heads + head) * s.block_size + off) * s.vdim;
+      if (veven) {
+        for (int i = lane * 2; i < s.vdim; i += 64) {
+          const float2 t = Pair<T>::load(v + i, true);
+          Pair<T>::store(c + i, t.x, t.y, true);
+        }
+      } else {
+        for (int i = lane; i < s.vdim; i += 32) c[i] = v[i];
+      }
+      continue;
     }
-    stf(x + 2 * i, a);
-    if (two) stf(x + 2 * i + 1, b);
-    if (c) {
-      stf(c + 2 * i, a);
-      if (two) stf(c + 2 * i + 1, b);
-    }
-  };
+    T* x = pr + (is_q ? s.q_off : s.k_off) + head * s.dim;
+    const T* w = is_q ? q_norm : k_norm;
+    T* c = is_k && cached ? k_cache + ((page * s.kv_heads + head) * s.block_size + off) * s.dim : nullptr;
+    auto load = [&](int i) {      // pair i, zeros past the end
+      if (2 * i + 1 < s.dim) return Pair<T>::load(x + 2 * i, even);
+      return make_float2(2 * i < s.dim ? ldf(x + 2 * i) : 0.f, 0.f);
+    };
+    float2 u[GP_KEEP];
+    float ss = 0.f;
 #pragma unroll
-  for (int j = 0; j < GP_KEEP; ++j) finish(lane + j * 32, u[j], v[j]);
-  for (int i = lane + GP_KEEP * 32; i < pairs; i += 32) finish(i, ldf(x + 2 * i), 2 * i + 1 < s.dim ? ldf(x + 2 * i + 1) : 0.f);
+    for (int j = 0; j < GP_KEEP; ++j) {
+      u[j] = load(lane + j * 32);
+      ss += u[j].x * u[j].x + u[j].y * u[j].y;
+    }
+    for (int i = lane + GP_KEEP * 32; i < pairs; i += 32) {
+      const float2 t = load(i);
+      ss += t.x * t.x + t.y * t.y;
+    }
+    ss = warp_sum(ss);
+    const float rstd = 1.f / sqrtf(ss / static_cast<float>(s.dim) + eps);
+    auto finish = [&](int i, float2 t) {
+      if (2 * i >= s.dim) return;
+      const bool two = 2 * i + 1 < s.dim;
+      t.x *= rstd * ldf(w + 2 * i);
+      if (two) t.y *= rstd * ldf(w + 2 * i + 1);
+      if (i < half) {
+        const float2 r = turn[i];
+        t = make_float2(t.x * r.x - t.y * r.y, t.y * r.x + t.x * r.y);
+      }
+      if (two) {
+        Pair<T>::store(x + 2 * i, t.x, t.y, even);
+        if (c) Pair<T>::store(c + 2 * i, t.x, t.y, even);
+      } else {
+        stf(x + 2 * i, t.x);
+        if (c) stf(c + 2 * i, t.x);
+      }
+    };
+#pragma unroll
+    for (int j = 0; j < GP_KEEP; ++j) finish(lane + j * 32, u[j]);
+    for (int i = lane + GP_KEEP * 32; i < pairs; i += 32) finish(i, load(i));
+  }
 }
 
 // One CTA per (row, query head): tiles of 128 keys, online softmax, everything in fp32.
@@ -190,14 +233,16 @@ RLB_API int rlb_gqa_prep(void* p, int f32, long long rows, long long ldp, int q_
   if (rows <= 0) return 0;
   if (2 * half > dim || kv_heads < 1 || heads % kv_heads) return -2;
   GqaShape s{ldp, q_off, k_off, v_off, heads, kv_heads, dim, vdim, block_size, num_blocks};
-  const dim3 grid(static_cast<unsigned>(rows), (heads + 2 * kv_heads + GP_WARPS - 1) / GP_WARPS), block(GP_WARPS * 32);
-  if (grid.y > 65535) return -2;
+  const int per_row = (heads + 2 * kv_heads + GP_WARPS - 1) / GP_WARPS;
+  const dim3 grid(static_cast<unsigned>(rows), rows >= 148 * 8 ? 1 : (per_row < 64 ? per_row : 64)), block(GP_WARPS * 32);
+  const size_t sm = sizeof(float2) * half;
+  if (sm > 48 * 1024) return -2;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (f32)
-    return static_cast<int>(rlb_launch_pdl(gqa_prep_kernel<float>, grid, block, 0, st, static_cast<float*>(p), s, positions, slots,
+    return static_cast<int>(rlb_launch_pdl(gqa_prep_kernel<float>, grid, block, sm, st, static_cast<float*>(p), s, positions, slots,
                                            static_cast<const float*>(q_norm), static_cast<const float*>(k_norm), freq, half, gain, eps,
                                            static_cast<float*>(k_cache), static_cast<float*>(v_cache), status));
-  return static_cast<int>(rlb_launch_pdl(gqa_prep_kernel<__nv_bfloat16>, grid, block, 0, st, static_cast<__nv_bfloat16*>(p), s, positions, slots,
+  return static_cast<int>(rlb_launch_pdl(gqa_prep_kernel<__nv_bfloat16>, grid, block, sm, st, static_cast<__nv_bfloat16*>(p), s, positions, slots,
                                          static_cast<const __nv_bfloat16*>(q_norm), static_cast<const __nv_bfloat16*>(k_norm), freq, half, gain, eps,
                                          static_cast<__nv_bfloat16*>(k_cache), static_cast<__nv_bfloat16*>(v_cache), status));
 }

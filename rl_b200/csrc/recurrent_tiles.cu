@@ -985,18 +985,53 @@ struct RecStep {
   int* status;
 };
 
-__device__ __forceinline__ float step_conv(const RecStep& s, long long row, long long sr, int pos, int c, bool owner) {
-  const __nv_bfloat16 in = s.p[row * s.ldp + s.conv_off + c];
-  __nv_bfloat16* ring = s.ring + sr * s.taps * s.channels + c;
-  float v = s.bias ? __bfloat162float(s.bias[c]) : 0.f;
-  const __nv_bfloat16* w = s.w + static_cast<long long>(c) * s.taps;
-  for (int j = 0; j < s.taps - 1; ++j) {
-    const int back = s.taps - 1 - j;
-    if (back <= pos) v = fmaf(__bfloat162float(w[j]), __bfloat162float(ring[static_cast<long long>((pos - back) % s.taps) * s.channels]), v);
+// A channel's inputs in registers (up to four taps), so that a thread has the loads of several channels in flight.
+constexpr int SC_TAPS = 4;
+struct StepChannel {
+  __nv_bfloat16 in, past[SC_TAPS - 1];
+  float w[SC_TAPS], b;
+  __device__ __forceinline__ void fetch(const RecStep& s, long long row, long long sr, int pos, int c) {
+    in = s.p[row * s.ldp + s.conv_off + c];
+    b = s.bias ? __bfloat162float(s.bias[c]) : 0.f;
+    const __nv_bfloat16* ring = s.ring + sr * s.taps * s.channels + c;
+    const __nv_bfloat16* wc = s.w + static_cast<long long>(c + 1) * s.taps - 1;      // the current token's tap
+    w[0] = __bfloat162float(*wc);
+#pragma unroll
+    for (int back = 1; back < SC_TAPS; ++back) {
+      const bool live = back < s.taps && back <= pos;
+      past[back - 1] = live ? ring[static_cast<long long>((pos - back) % s.taps) * s.channels] : __float2bfloat16(0.f);
+      w[back] = live ? __bfloat162float(wc[-back]) : 0.f;
+    }
   }
-  v = fmaf(__bfloat162float(w[s.taps - 1]), __bfloat162float(in), v);
-  if (owner) ring[static_cast<long long>(pos % s.taps) * s.channels] = in;
-  return __bfloat162float(__float2bfloat16(rc_silu(v)));      // (as the portions' convolution leaves it)
+  // The convolved and activated value, rounded as the portions' convolution leaves it.
+  __device__ __forceinline__ float finish(const RecStep& s, long long sr, int pos, int c, bool owner) const {
+    float v = b;
+    __nv_bfloat16* ring = s.ring + sr * s.taps * s.channels + c;
+    for (int back = s.taps - 1; back >= SC_TAPS; --back)
+      if (back <= pos)
+        v = fmaf(__bfloat162float(s.w[static_cast<long long>(c + 1) * s.taps - 1 - back]),
+                 __bfloat162float(ring[static_cast<long long>((pos - back) % s.taps) * s.channels]), v);
+#pragma unroll
+    for (int back = SC_TAPS - 1; back > 0; --back) v = fmaf(w[back], __bfloat162float(past[back - 1]), v);
+    v = fmaf(w[0], __bfloat162float(in), v);
+    if (owner) ring[static_cast<long long>(pos % s.taps) * s.channels] = in;
+    return __bfloat162float(__float2bfloat16(rc_silu(v)));
+  }
+};
+// out[i] = channel(i) for i < n; `channel` and `owner` name the convolved channel and whether this CTA keeps its ring. Two channels per
+// thread in flight.
+template <typename Channel, typename Owner, typename Store>
+__device__ __forceinline__ void step_convolve(const RecStep& s, long long row, long long sr, int pos, int n, Channel channel, Owner owner, Store store) {
+  const int step = blockDim.x;
+  for (int i = threadIdx.x; i < n; i += 2 * step) {
+    StepChannel a, b;
+    const bool two = i + step < n;
+    const int ca = channel(i), cb = two ? channel(i + step) : ca;
+    a.fetch(s, row, sr, pos, ca);
+    if (two) b.fetch(s, row, sr, pos, cb);
+    store(i, a.finish(s, sr, pos, ca, owner(i)));
+    if (two) store(i + step, b.finish(s, sr, pos, cb, owner(i + step)));
+  }
 }
 
 __global__ void __launch_bounds__(256) mamba2_step_kernel(RecStep s) {
@@ -1012,13 +1047,14 @@ __global__ void __launch_bounds__(256) mamba2_step_kernel(RecStep s) {
   }
   const int pos = s.positions[row], inner = s.heads * s.vdim;
   const bool first = head % (s.heads / s.groups) == 0;
-  const float dt = rc_softplus(__bfloat162float(s.p[row * s.ldp + s.a_off + head]) + __bfloat162float(s.dt_bias[head]));
-  const float dec = expf(-expf(__bfloat162float(s.A_log[head])) * dt);
-  for (int i = tid; i < s.vdim + 2 * s.dim; i += 256) {
-    const bool is_x = i < s.vdim, is_b = i < s.vdim + s.dim;
-    const int c = is_x ? head * s.vdim + i : (is_b ? inner + group * s.dim + i - s.vdim : inner + (s.groups + group) * s.dim + i - s.vdim - s.dim);
-    sm[i] = step_conv(s, row, sr, pos, c, is_x || first) * (!is_x && is_b ? dt : 1.f);
-  }
+  const float dt_in = __bfloat162float(s.p[row * s.ldp + s.a_off + head]), dt_b = __bfloat162float(s.dt_bias[head]), A_log = __bfloat162float(s.A_log[head]);
+  step_convolve(s, row, sr, pos, s.vdim + 2 * s.dim,
+                [&](int i) {
+                  return i < s.vdim ? head * s.vdim + i
+                                    : (i < s.vdim + s.dim ? inner + group * s.dim + i - s.vdim : inner + (s.groups + group) * s.dim + i - s.vdim - s.dim);
+                },
+                [&](int i) { return i < s.vdim || first; }, [&](int i, float v) { sm[i] = v; });
+  const float dt = rc_softplus(dt_in + dt_b), dec = expf(-expf(A_log) * dt);
   __syncthreads();
   const int c4 = s.vdim / 4, slices = 256 / c4, slice = tid / c4, col = tid % c4;
   if (slice < slices) {
@@ -1037,7 +1073,7 @@ __global__ void __launch_bounds__(256) mamba2_step_kernel(RecStep s) {
       for (int q = 0; q < U; ++q) {
         const int i = i0 + q * slices;
         if (i < s.dim) {
-          const float b = B[i], c = C[i];
+          const float b = dt * B[i], c = C[i];
           a[q] = make_float4(fmaf(dec, a[q].x, b * v.x), fmaf(dec, a[q].y, b * v.y), fmaf(dec, a[q].z, b * v.z), fmaf(dec, a[q].w, b * v.w));
           S[static_cast<long long>(i) * c4] = a[q];
           acc.x = fmaf(a[q].x, c, acc.x);
@@ -1066,13 +1102,14 @@ __global__ void __launch_bounds__(256) mamba2_step_kernel(RecStep s) {
   }
 }
 
-// KEEP: the state stays in registers between the read-out and the write (at most 16 float4 per thread).
+// KEEP: the state stays in registers between the read-out and the write (at most 8 float4 per thread).
+constexpr int DD_THREADS = 512;
 template <bool KEEP>
-__global__ void __launch_bounds__(256) delta_step_kernel(RecStep s) {
+__global__ void __launch_bounds__(DD_THREADS, 2) delta_step_kernel(RecStep s) {
   extern __shared__ float sm[];
   __shared__ float red[32];
   float *q = sm, *k = q + s.dim, *v = k + s.dim;            // v: the value, then what is written
-  float4* part = reinterpret_cast<float4*>(v + s.vdim);     // [2][256]
+  float4* part = reinterpret_cast<float4*>(v + s.vdim);     // [2][DD_THREADS]
   const int row = blockIdx.x, head = blockIdx.y, tid = threadIdx.x, per = s.heads / s.groups, group = head / per, n = s.groups * s.dim;
   pdl_sync();
   const long long sr = s.state_rows[row];
@@ -1081,10 +1118,10 @@ __global__ void __launch_bounds__(256) delta_step_kernel(RecStep s) {
     return;
   }
   const int pos = s.positions[row];
-  const int c4 = s.vdim / 4, slices = 256 / c4, slice = tid / c4, col = tid % c4;
+  const int c4 = s.vdim / 4, slices = DD_THREADS / c4, slice = tid / c4, col = tid % c4;
   const bool live = slice < slices;
   float4* S = reinterpret_cast<float4*>(s.state + (sr * s.heads + head) * static_cast<long long>(s.dim) * s.vdim) + col;
-  constexpr int U = 16;
+  constexpr int U = 8;
   float4 a[U];
   if (KEEP) {
 #pragma unroll
@@ -1093,24 +1130,25 @@ __global__ void __launch_bounds__(256) delta_step_kernel(RecStep s) {
       a[u] = live && i < s.dim && pos != 0 ? S[static_cast<long long>(i) * c4] : make_float4(0.f, 0.f, 0.f, 0.f);
     }
   }
-  float qq = 0.f, kk = 0.f, qk = 0.f;
-  for (int i = tid; i < s.dim; i += 256) {
-    const float qv = step_conv(s, row, sr, pos, group * s.dim + i, head % per == 0), kv = step_conv(s, row, sr, pos, n + group * s.dim + i, head % per == 0);
-    q[i] = qv;
-    k[i] = kv;
+  const float beta_in = __bfloat162float(s.p[row * s.ldp + s.b_off + head]), dt_in = __bfloat162float(s.p[row * s.ldp + s.a_off + head]);
+  const float dt_b = __bfloat162float(s.dt_bias[head]), A_log = __bfloat162float(s.A_log[head]);
+  const bool first = head % per == 0;
+  step_convolve(s, row, sr, pos, 2 * s.dim + s.vdim,
+                [&](int i) { return i < s.dim ? group * s.dim + i : (i < 2 * s.dim ? n + group * s.dim + i - s.dim : 2 * n + head * s.vdim + i - 2 * s.dim); },
+                [&](int i) { return i >= 2 * s.dim || first; }, [&](int i, float x) { sm[i] = x; });
+  __syncthreads();
+  float qq = 0.f, kk = 0.f, qk = 0.f;      // every warp for itself
+  for (int i = tid & 31; i < s.dim; i += 32) {
+    const float qv = q[i], kv = k[i];
     qq += qv * qv;
     kk += kv * kv;
     qk += qv * kv;
   }
-  for (int i = tid; i < s.vdim; i += 256) v[i] = step_conv(s, row, sr, pos, 2 * n + head * s.vdim + i, true);
-  qq = block_sum(qq, red);
-  kk = block_sum(kk, red);
-  qk = block_sum(qk, red);
+  qq = warp_sum(qq);
+  kk = warp_sum(kk);
+  qk = warp_sum(qk);
   const float qf = 1.f / (sqrtf(qq + s.unit_eps) * sqrtf(static_cast<float>(s.dim))), kf = 1.f / sqrtf(kk + s.unit_eps);
-  const float beta = 1.f / (1.f + expf(-__bfloat162float(s.p[row * s.ldp + s.b_off + head])));
-  const float dec = expf(-expf(__bfloat162float(s.A_log[head])) *
-                         rc_softplus(__bfloat162float(s.p[row * s.ldp + s.a_off + head]) + __bfloat162float(s.dt_bias[head])));
-  __syncthreads();
+  const float beta = 1.f / (1.f + expf(-beta_in)), dec = expf(-expf(A_log) * rc_softplus(dt_in + dt_b));
   float4 sk = make_float4(0.f, 0.f, 0.f, 0.f), sq = sk;
   auto read = [&](const float4& t, int i) {
     const float kv = k[i], qv = q[i];
@@ -1127,14 +1165,14 @@ __global__ void __launch_bounds__(256) delta_step_kernel(RecStep s) {
       for (int i = slice; i < s.dim; i += slices) read(S[static_cast<long long>(i) * c4], i);
     }
     part[tid] = sk;
-    part[256 + tid] = sq;
+    part[DD_THREADS + tid] = sq;
   }
   __syncthreads();
   float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
   if (tid < c4) {
     float4 t = o;
     for (int j = 0; j < slices; ++j) {
-      const float4 x = part[j * c4 + tid], y = part[256 + j * c4 + tid];
+      const float4 x = part[j * c4 + tid], y = part[DD_THREADS + j * c4 + tid];
       t.x += x.x; t.y += x.y; t.z += x.z; t.w += x.w;
       o.x += y.x; o.y += y.y; o.z += y.z; o.w += y.w;
     }
@@ -1228,11 +1266,11 @@ RLB_API int rlb_rec_step(const RecArgs* a, void* stream) {
             a->eps, static_cast<__nv_bfloat16*>(a->y), a->ldy, a->status};
   const dim3 grid(a->pieces, a->heads), block(256);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const size_t sm = sizeof(float) * (a->vdim + 2 * a->dim) + sizeof(float4) * 256 * (a->delta ? 2 : 1);
+  const size_t sm = sizeof(float) * (a->vdim + 2 * a->dim) + sizeof(float4) * (a->delta ? 2 * DD_THREADS : 256);
   if (!a->delta) return static_cast<int>(rlb_launch_pdl(mamba2_step_kernel, grid, block, sm, st, s));
-  const int slices = 256 / (a->vdim / 4);
-  if (a->dim <= 16 * slices) return static_cast<int>(rlb_launch_pdl(delta_step_kernel<true>, grid, block, sm, st, s));
-  return static_cast<int>(rlb_launch_pdl(delta_step_kernel<false>, grid, block, sm, st, s));
+  const int slices = DD_THREADS / (a->vdim / 4);
+  if (a->dim <= 8 * slices) return static_cast<int>(rlb_launch_pdl(delta_step_kernel<true>, grid, dim3(DD_THREADS), sm, st, s));
+  return static_cast<int>(rlb_launch_pdl(delta_step_kernel<false>, grid, dim3(DD_THREADS), sm, st, s));
 }
 
 // Portions: rows [row0, rows) of u, p, y in chunks of at most 128 rows (chunk_row counts from row0); piece i owns chunks [piece_chunk[i],
