@@ -147,6 +147,94 @@ gqa_prep_kernel(T* __restrict__ p, GqaShape s, const int* __restrict__ positions
   }
 }
 
+// The same for bf16 rows with even dim <= 64 * KEEP and even vdim: one warp per row (and share of its heads). A lane turns the same pairs of every
+// head, so cosines, sines and norm weights stay in its registers; four heads are in flight.
+template <int KEEP>
+__global__ void __launch_bounds__(GP_WARPS * 32)
+gqa_prep_rows_kernel(__nv_bfloat16* __restrict__ p, GqaShape s, long long rows, const int* __restrict__ positions, const long long* __restrict__ slots,
+                     const __nv_bfloat16* __restrict__ q_norm, const __nv_bfloat16* __restrict__ k_norm, const float* __restrict__ freq, int half,
+                     float gain, float eps, __nv_bfloat16* __restrict__ k_cache, __nv_bfloat16* __restrict__ v_cache, int* status) {
+  constexpr int AHEAD = 4;
+  const int lane = threadIdx.x & 31;
+  const long long row = static_cast<long long>(blockIdx.x) * GP_WARPS + (threadIdx.x >> 5);
+  float2 wq[KEEP], wk[KEEP], turn[KEEP];
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int i = lane + j * 32;
+    const bool live = 2 * i < s.dim;
+    wq[j] = live ? Pair<__nv_bfloat16>::load(q_norm + 2 * i, true) : make_float2(0.f, 0.f);
+    wk[j] = live ? Pair<__nv_bfloat16>::load(k_norm + 2 * i, true) : make_float2(0.f, 0.f);
+  }
+  pdl_sync();
+  if (row >= rows) return;
+  const float pos = static_cast<float>(positions[row]);
+  const long long slot = slots[row];
+  const bool bad = slot >= static_cast<long long>(s.num_blocks) * s.block_size;
+  if (bad && lane == 0 && status) atomicCAS(status, 0, RLB_ERR_BOUNDS);
+  const bool cached = slot >= 0 && !bad;
+  const unsigned at = cached ? static_cast<unsigned>(slot) : 0u, page = at / s.block_size, off = at - page * s.block_size;
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int i = lane + j * 32;
+    turn[j] = make_float2(1.f, 0.f);
+    if (i < half) {
+      float sn, cs;
+      sincosf(pos * freq[i], &sn, &cs);
+      turn[j] = make_float2(cs * gain, sn * gain);
+    }
+  }
+  __nv_bfloat16* pr = p + row * s.ldp;
+  const int units = s.heads + s.kv_heads;
+  for (int u0 = blockIdx.y * AHEAD; u0 < units; u0 += gridDim.y * AHEAD) {
+    float2 v[AHEAD][KEEP];
+    float ss[AHEAD];
+#pragma unroll
+    for (int a = 0; a < AHEAD; ++a) {
+      const int unit = u0 + a;
+      const __nv_bfloat16* x = pr + (unit < s.heads ? s.q_off + unit * s.dim : s.k_off + (unit - s.heads) * s.dim);
+#pragma unroll
+      for (int j = 0; j < KEEP; ++j) {
+        const int i = lane + j * 32;
+        v[a][j] = unit < units && 2 * i < s.dim ? Pair<__nv_bfloat16>::load(x + 2 * i, true) : make_float2(0.f, 0.f);
+      }
+    }
+#pragma unroll
+    for (int a = 0; a < AHEAD; ++a) {
+      ss[a] = 0.f;
+#pragma unroll
+      for (int j = 0; j < KEEP; ++j) ss[a] += v[a][j].x * v[a][j].x + v[a][j].y * v[a][j].y;
+    }
+#pragma unroll
+    for (int a = 0; a < AHEAD; ++a) ss[a] = warp_sum(ss[a]);
+#pragma unroll
+    for (int a = 0; a < AHEAD; ++a) {
+      const int unit = u0 + a;
+      if (unit >= units) break;
+      const bool is_q = unit < s.heads;
+      const int head = is_q ? unit : unit - s.heads;
+      const float rstd = 1.f / sqrtf(ss[a] / static_cast<float>(s.dim) + eps);
+      __nv_bfloat16* x = pr + (is_q ? s.q_off : s.k_off) + head * s.dim;
+      __nv_bfloat16* c = k_cache + ((static_cast<long long>(page) * s.kv_heads + head) * s.block_size + off) * s.dim;
+#pragma unroll
+      for (int j = 0; j < KEEP; ++j) {
+        const int i = lane + j * 32;
+        if (2 * i >= s.dim) continue;
+        const float2 w = is_q ? wq[j] : wk[j];
+        const float a0 = v[a][j].x * rstd * w.x, b0 = v[a][j].y * rstd * w.y;
+        const uint32_t o = pack_bf16x2(a0 * turn[j].x - b0 * turn[j].y, b0 * turn[j].x + a0 * turn[j].y);
+        *reinterpret_cast<uint32_t*>(x + 2 * i) = o;
+        if (!is_q && cached) *reinterpret_cast<uint32_t*>(c + 2 * i) = o;
+      }
+    }
+  }
+  if (!cached) return;
+  for (int g = blockIdx.y; g < s.kv_heads; g += gridDim.y) {
+    const __nv_bfloat16* x = pr + s.v_off + g * s.vdim;
+    __nv_bfloat16* c = v_cache + ((static_cast<long long>(page) * s.kv_heads + g) * s.block_size + off) * s.vdim;
+    for (int i = lane * 2; i < s.vdim; i += 64) *reinterpret_cast<uint32_t*>(c + i) = *reinterpret_cast<const uint32_t*>(x + i);
+  }
+}
+
 // One CTA per (row, query head): tiles of 128 keys, online softmax, everything in fp32.
 constexpr int GR_TILE = 128;
 template <typename T>
@@ -238,6 +326,15 @@ RLB_API int rlb_gqa_prep(void* p, int f32, long long rows, long long ldp, int q_
   const size_t sm = sizeof(float2) * half;
   if (sm > 48 * 1024) return -2;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (!f32 && dim % 2 == 0 && vdim % 2 == 0 && ldp % 2 == 0 && dim <= 256 && (q_off | k_off | v_off) % 2 == 0 &&
+      static_cast<long long>(num_blocks) * block_size < 0x7fffffffll) {
+    const int share = (heads + kv_heads + 3) / 4;
+    const dim3 g(static_cast<unsigned>((rows + GP_WARPS - 1) / GP_WARPS), rows >= 148 * 16 ? 1 : (share < 64 ? share : 64));
+    auto k = dim <= 128 ? gqa_prep_rows_kernel<2> : gqa_prep_rows_kernel<4>;
+    return static_cast<int>(rlb_launch_pdl(k, g, block, 0, st, static_cast<__nv_bfloat16*>(p), s, rows, positions, slots,
+                                           static_cast<const __nv_bfloat16*>(q_norm), static_cast<const __nv_bfloat16*>(k_norm), freq, half, gain, eps,
+                                           static_cast<__nv_bfloat16*>(k_cache), static_cast<__nv_bfloat16*>(v_cache), status));
+  }
   if (f32)
     return static_cast<int>(rlb_launch_pdl(gqa_prep_kernel<float>, grid, block, sm, st, static_cast<float*>(p), s, positions, slots,
                                            static_cast<const float*>(q_norm), static_cast<const float*>(k_norm), freq, half, gain, eps,

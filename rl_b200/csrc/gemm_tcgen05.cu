@@ -21,6 +21,7 @@
 //                kernel folds the partials into logprob / entropy / logsumexp per row.
 //   EPI_LAYER    products of a parallel mixer layer (LayerEpilogue in common.cuh): squared ReLU on a column range, or
 //                residual update + dynamic-tanh norm
+//   EPI_LINEAR   products of post-norm layers (LinearEpi in common.cuh): bias, then clamped gated unit or gated token input
 //   EPI_DLOGITS  recomputes the logits tile and writes coef[row]*(onehot - softmax)*inv_temp in
 //                bf16, the gradient that the dH / dW GEMMs consume.
 // Replaces the cuBLAS calls behind nn.Linear and the chunked hidden->logprob path of the reference
@@ -50,7 +51,7 @@ constexpr int NUM_THREADS = 192;
 constexpr int TMEM_COLS = 512;
 constexpr int GROUP_M = 16;  // rasterisation: 16 m-tiles share each sweep over n
 
-enum { EPI_STORE = 0, EPI_LOGPROB = 1, EPI_DLOGITS = 2, EPI_LAYER = 3 };
+enum { EPI_STORE = 0, EPI_LOGPROB = 1, EPI_DLOGITS = 2, EPI_LAYER = 3, EPI_LINEAR = 4 };
 
 struct EpiParams {
   void* C;              // output (EPI_STORE, EPI_DLOGITS)
@@ -303,14 +304,13 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
         }
       } else if (EPI == EPI_LAYER) {
         const float alpha = ep.layer.x ? __bfloat162float(*ep.layer.alpha) : 0.f;
-        const bool glu = ep.layer.lin.act == LIN_GLU;
         for (int c = 0; c < BN / 32; ++c) {
           uint32_t r[32];
           tmem_ld_32x32b_x32(taddr + c * 32, r);
           tmem_ld_wait();
           const int col = col0 + c * 32;
           if (!row_ok || col >= N) continue;
-          __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(ep.C) + static_cast<long long>(row) * ep.ldc + (glu ? col / 2 : col);
+          __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(ep.C) + static_cast<long long>(row) * ep.ldc + col;
 #pragma unroll
           for (int q = 0; q < 4; ++q) {
             if (col + q * 8 < N) {
@@ -318,13 +318,72 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
                                                                      __uint_as_float(r[q * 8 + 2]), __uint_as_float(r[q * 8 + 3])), row, col + q * 8, alpha);
               const float4 b = layer_epilogue4(ep.layer, make_float4(__uint_as_float(r[q * 8 + 4]), __uint_as_float(r[q * 8 + 5]),
                                                                      __uint_as_float(r[q * 8 + 6]), __uint_as_float(r[q * 8 + 7])), row, col + q * 8 + 4, alpha);
-              if (glu) {
-                *reinterpret_cast<uint2*>(dst + q * 4) = make_uint2(pack_bf16x2(a.x, a.y), pack_bf16x2(b.x, b.y));
-                continue;
-              }
               *reinterpret_cast<uint4*>(dst + q * 8) = make_uint4(pack_bf16x2(a.x, a.y), pack_bf16x2(a.z, a.w), pack_bf16x2(b.x, b.y), pack_bf16x2(b.z, b.w));
             }
           }
+        }
+      } else if (EPI == EPI_LINEAR) {
+        const LinearEpi& le = ep.layer.lin;
+        const __nv_bfloat16* table = nullptr;
+        if (le.act == LIN_GELU_MUL && row_ok) table = static_cast<const __nv_bfloat16*>(le.table) + lin_token(le, row) * le.ld_table + le.table_off;
+        const bool wide = le.act == LIN_GELU_MUL && ((le.ld_table | le.table_off) & 3) == 0;      // table pieces of four columns are aligned
+        for (int c = 0; c < BN / 32; ++c) {
+          uint32_t r[32];
+          tmem_ld_32x32b_x32(taddr + c * 32, r);
+          tmem_ld_wait();
+          const int col = col0 + c * 32;
+          if (!row_ok || col >= N) continue;
+          float v[32];
+#pragma unroll
+          for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
+          if (le.bias) {
+#pragma unroll
+            for (int q = 0; q < 4; ++q)
+              if (col + q * 8 < N) {
+                const uint4 b = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(le.bias) + col + q * 8);
+                const float2 b0 = unpack_bf16x2(b.x), b1 = unpack_bf16x2(b.y), b2 = unpack_bf16x2(b.z), b3 = unpack_bf16x2(b.w);
+                v[q * 8 + 0] += b0.x; v[q * 8 + 1] += b0.y; v[q * 8 + 2] += b1.x; v[q * 8 + 3] += b1.y;
+                v[q * 8 + 4] += b2.x; v[q * 8 + 5] += b2.y; v[q * 8 + 6] += b3.x; v[q * 8 + 7] += b3.y;
+              }
+          }
+          if (le.act == LIN_GLU) {
+            __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(ep.C) + static_cast<long long>(row) * ep.ldc + col / 2;
+            uint32_t o[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i)
+              o[i] = pack_bf16x2(clamped_glu(v[4 * i], v[4 * i + 1], le.limit), clamped_glu(v[4 * i + 2], v[4 * i + 3], le.limit));
+#pragma unroll
+            for (int q = 0; q < 4; ++q)
+              if (col + q * 8 < N) *reinterpret_cast<uint2*>(dst + q * 4) = make_uint2(o[2 * q], o[2 * q + 1]);
+            continue;
+          }
+          if (le.act == LIN_GELU_MUL) {
+#pragma unroll
+            for (int q = 0; q < 8; ++q) {
+              float t[4] = {0.f, 0.f, 0.f, 0.f};
+              const int x = col + q * 4;
+              if (wide && x + 4 <= le.table_cols) {
+                const uint2 raw = *reinterpret_cast<const uint2*>(table + x);
+                const float2 a = unpack_bf16x2(raw.x), b = unpack_bf16x2(raw.y);
+                t[0] = a.x; t[1] = a.y; t[2] = b.x; t[3] = b.y;
+              } else {
+#pragma unroll
+                for (int k = 0; k < 4; ++k)
+                  if (x + k < le.table_cols) t[k] = __bfloat162float(table[x + k]);
+              }
+#pragma unroll
+              for (int k = 0; k < 4; ++k) {      // 0.5 z (1 + tanh y) = z / (1 + exp(-2 y))
+                const float z = v[q * 4 + k];
+                v[q * 4 + k] = x + k < le.table_cols ? z / (1.f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z))) * t[k] : 0.f;
+              }
+            }
+          }
+          __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(ep.C) + static_cast<long long>(row) * ep.ldc + col;
+#pragma unroll
+          for (int q = 0; q < 4; ++q)
+            if (col + q * 8 < N)
+              *reinterpret_cast<uint4*>(dst + q * 8) = make_uint4(pack_bf16x2(v[q * 8], v[q * 8 + 1]), pack_bf16x2(v[q * 8 + 2], v[q * 8 + 3]),
+                                                                  pack_bf16x2(v[q * 8 + 4], v[q * 8 + 5]), pack_bf16x2(v[q * 8 + 6], v[q * 8 + 7]));
         }
       } else if (EPI == EPI_LOGPROB) {
         // Online softmax statistics of this row over the tile's columns.
@@ -590,17 +649,17 @@ RLB_API int rlb_gemm_layer(const void* A, const void* W, void* out, int M, int N
 // out (bf16) = epilogue(a w^T); N, K and the row strides multiples of 8.
 RLB_API int rlb_linear_tiled(const RlbLinear* l, void* stream) {
   if (l->M <= 0 || l->N <= 0 || l->K <= 0) return 0;
-  if ((l->lda % 8) || (l->ldw % 8) || (l->ldo % 8) || (l->N % 8) || (l->K % 8) || l->in_f32 || l->out_f32 || l->tile_expert) return -2;
+  if ((l->lda % 8) || (l->ldw % 8) || (l->ldo % 8) || (l->N % 8) || (l->K % 8) || l->in_f32 || l->out_f32 || l->tile_expert || l->act == LIN_CAP) return -2;
   if ((reinterpret_cast<uintptr_t>(l->a) | reinterpret_cast<uintptr_t>(l->w) | reinterpret_cast<uintptr_t>(l->out) | reinterpret_cast<uintptr_t>(l->bias)) & 15) return -3;
+  if (l->act == LIN_GELU_MUL && (reinterpret_cast<uintptr_t>(l->table) & 7)) return -3;
   CUtensorMap ta, tb;
   int rc = make_operand_maps(l->a, l->w, l->M, l->N, l->K, l->lda, l->ldw, false, false, &ta, &tb);
   if (rc) return -100 - rc;
   EpiParams ep{};
   ep.C = l->out;
   ep.ldc = l->ldo;
-  ep.layer.act_from = 1 << 30;
   ep.layer.lin = rlb_linear_epi(*l);
-  return launch_gemm<false, false, EPI_LAYER>(ta, tb, l->M, l->N, l->K, ep, l->status, 0, static_cast<cudaStream_t>(stream));
+  return launch_gemm<false, false, EPI_LINEAR>(ta, tb, l->M, l->N, l->K, ep, l->status, 0, static_cast<cudaStream_t>(stream));
 }
 
 // Number of n-tiles the vocab-projection epilogues split N into (size of the partial buffers).

@@ -52,9 +52,8 @@ struct AddNormed {
   float mult, eps;
 };
 
-constexpr int AN_KEEP = 8;   // groups of four columns that a thread keeps in registers
-
-template <typename T, int THREADS>
+// AN_KEEP: groups of four columns that a thread keeps in registers
+template <typename T, int THREADS, int AN_KEEP>
 __global__ void __launch_bounds__(THREADS) add_normed_kernel(AddNormed a) {
   __shared__ float red[32];
   pdl_sync();
@@ -77,20 +76,30 @@ __global__ void __launch_bounds__(THREADS) add_normed_kernel(AddNormed a) {
       if (!a.copy_row) v[i] = ld4(Y + row * a.ldy + c);
     }
     if (a.copy_row) {
-      for (int j = 0; j < a.k; ++j) {
-        const int r = a.copy_row[row * a.k + j];
-        const float wt = a.weight[row * a.k + j];
-        if (r < 0 || r >= a.y_rows) continue;
+      constexpr int AHEAD = AN_KEEP <= 2 ? 4 : 2;      // copies in flight
+      for (int j0 = 0; j0 < a.k; j0 += AHEAD) {
+        float4 e[AHEAD][AN_KEEP];
+        float wt[AHEAD];
 #pragma unroll
-        for (int i = 0; i < AN_KEEP; ++i) {
-          const int c = (threadIdx.x + i * THREADS) * 4;
-          if (c >= a.d) continue;
-          const float4 e = ld4(Y + r * a.ldy + c);
-          v[i].x = fmaf(wt, e.x, v[i].x);
-          v[i].y = fmaf(wt, e.y, v[i].y);
-          v[i].z = fmaf(wt, e.z, v[i].z);
-          v[i].w = fmaf(wt, e.w, v[i].w);
+        for (int j = 0; j < AHEAD; ++j) {
+          const int r = j0 + j < a.k ? a.copy_row[row * a.k + j0 + j] : -1;
+          const bool live = r >= 0 && r < a.y_rows;
+          wt[j] = live ? a.weight[row * a.k + j0 + j] : 0.f;
+#pragma unroll
+          for (int i = 0; i < AN_KEEP; ++i) {
+            const int c = (threadIdx.x + i * THREADS) * 4;
+            e[j][i] = live && c < a.d ? ld4(Y + r * a.ldy + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+          }
         }
+#pragma unroll
+        for (int j = 0; j < AHEAD; ++j)
+#pragma unroll
+          for (int i = 0; i < AN_KEEP; ++i) {
+            v[i].x = fmaf(wt[j], e[j][i].x, v[i].x);
+            v[i].y = fmaf(wt[j], e[j][i].y, v[i].y);
+            v[i].z = fmaf(wt[j], e[j][i].z, v[i].z);
+            v[i].w = fmaf(wt[j], e[j][i].w, v[i].w);
+          }
       }
     }
 #pragma unroll
@@ -190,6 +199,47 @@ __global__ void __launch_bounds__(256) group_norm_rows_kernel(T* __restrict__ y,
   ss = block_sum(ss, red);
   const float f = 1.f / sqrtf(ss / static_cast<float>(n) + eps);
   for (int c = threadIdx.x; c < n; c += 256) st1(p + c, ldv(p + c) * f * ldv(wg + c));
+}
+
+// The same for bf16 parts of at most 2048 columns: one warp per part.
+__global__ void __launch_bounds__(256)
+group_norm_warp_kernel(__nv_bfloat16* __restrict__ y, long long ldy, const __nv_bfloat16* __restrict__ w, long long parts, int groups, int n, float eps) {
+  pdl_sync();
+  const int lane = threadIdx.x & 31;
+  const long long i = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+  if (i >= parts) return;
+  const long long row = i / groups;
+  const int g = static_cast<int>(i - row * groups);
+  __nv_bfloat16* p = y + row * ldy + static_cast<long long>(g) * n;
+  const __nv_bfloat16* wg = w + static_cast<long long>(g) * n;
+  uint4 raw[8];
+  float ss = 0.f;
+#pragma unroll
+  for (int q = 0; q < 8; ++q) {
+    const int c = (lane + q * 32) * 8;
+    raw[q] = c < n ? *reinterpret_cast<const uint4*>(p + c) : make_uint4(0, 0, 0, 0);
+  }
+#pragma unroll
+  for (int q = 0; q < 8; ++q) {
+    const float2 a = unpack_bf16x2(raw[q].x), b = unpack_bf16x2(raw[q].y), c = unpack_bf16x2(raw[q].z), d = unpack_bf16x2(raw[q].w);
+    ss += a.x * a.x + a.y * a.y + b.x * b.x + b.y * b.y + c.x * c.x + c.y * c.y + d.x * d.x + d.y * d.y;
+  }
+  ss = warp_sum(ss);
+  const float f = 1.f / sqrtf(ss / static_cast<float>(n) + eps);
+#pragma unroll
+  for (int q = 0; q < 8; ++q) {
+    const int c = (lane + q * 32) * 8;
+    if (c >= n) continue;
+    const uint4 wr = *reinterpret_cast<const uint4*>(wg + c);
+    const uint32_t in[4] = {raw[q].x, raw[q].y, raw[q].z, raw[q].w}, wv[4] = {wr.x, wr.y, wr.z, wr.w};
+    uint32_t o[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const float2 a = unpack_bf16x2(in[k]), b = unpack_bf16x2(wv[k]);
+      o[k] = pack_bf16x2(a.x * f * b.x, a.y * f * b.y);
+    }
+    *reinterpret_cast<uint4*>(p + c) = make_uint4(o[0], o[1], o[2], o[3]);
+  }
 }
 
 __global__ void __launch_bounds__(256) cap_rows_kernel(float* __restrict__ z, long long n, float scale, float cap) {
@@ -354,9 +404,13 @@ RLB_API int rlb_add_normed(float* x, const void* y, long long ldy, int f32, cons
   AddNormed a{x, y, ldy, copy_row, weight, k, y_rows, counts, experts, w, next_w, h, d, mult, eps};
   const dim3 grid(static_cast<unsigned>(rows));
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (f32) return static_cast<int>(rlb_launch_pdl(add_normed_kernel<float, 256>, grid, dim3(256), 0, s, a));
-  if (d > 1024 && rows < 148 * 4) return static_cast<int>(rlb_launch_pdl(add_normed_kernel<__nv_bfloat16, 512>, grid, dim3(512), 0, s, a));
-  return static_cast<int>(rlb_launch_pdl(add_normed_kernel<__nv_bfloat16, 256>, grid, dim3(256), 0, s, a));
+  if (f32) return static_cast<int>(rlb_launch_pdl(add_normed_kernel<float, 256, 8>, grid, dim3(256), 0, s, a));
+  const bool few = rows < 148 * 4;      // few rows: more threads per row
+  auto kernel = few && d > 1024 ? (d <= 2048 ? add_normed_kernel<__nv_bfloat16, 512, 1> : (d <= 4096 ? add_normed_kernel<__nv_bfloat16, 512, 2>
+                                                                                                : add_normed_kernel<__nv_bfloat16, 512, 4>))
+                           : (d <= 1024 ? add_normed_kernel<__nv_bfloat16, 256, 1> : (d <= 2048 ? add_normed_kernel<__nv_bfloat16, 256, 2>
+                              : (d <= 4096 ? add_normed_kernel<__nv_bfloat16, 256, 4> : add_normed_kernel<__nv_bfloat16, 256, 8>)));
+  return static_cast<int>(rlb_launch_pdl(kernel, grid, dim3(few && d > 1024 ? 512 : 256), 0, s, a));
 }
 
 // y [rows, ldy]: each of `groups` neighbouring parts of n columns divided by its root mean square, times w [groups * n]; in place.
@@ -368,6 +422,11 @@ RLB_API int rlb_group_norm_rows(void* y, long long ldy, int f32, const void* w, 
   if (f32)
     return static_cast<int>(rlb_launch_pdl(group_norm_rows_kernel<float>, grid, dim3(256), 0, s, static_cast<float*>(y), ldy, static_cast<const float*>(w),
                                            groups, n, eps));
+  if (n % 8 == 0 && n <= 2048 && ldy % 8 == 0 && !((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(w)) & 15)) {
+    const long long parts = rows * groups;
+    return static_cast<int>(rlb_launch_pdl(group_norm_warp_kernel, dim3(static_cast<unsigned>((parts + 7) / 8)), dim3(256), 0, s,
+                                           static_cast<__nv_bfloat16*>(y), ldy, static_cast<const __nv_bfloat16*>(w), parts, groups, n, eps));
+  }
   return static_cast<int>(rlb_launch_pdl(group_norm_rows_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, static_cast<__nv_bfloat16*>(y), ldy,
                                          static_cast<const __nv_bfloat16*>(w), groups, n, eps));
 }

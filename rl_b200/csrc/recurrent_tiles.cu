@@ -73,41 +73,54 @@ conv_runs_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, __nv_bfloat
     for (int j = 0; j < TAPS; ++j) wv[k][j] = __bfloat162float(w[static_cast<long long>(c + k) * TAPS + j]);
   }
   const long long r0 = static_cast<long long>(blockIdx.x) * CV_RUN, r1 = min(rows, r0 + CV_RUN);
-  for (long long r = r0; r < r1; ++r) {
-    const int off = row_off[r];
-    if (r == r0 || off == 0) {      // the inputs before this row: of the same piece, of the ring, or none
-      const int pos = positions[r];
-      long long sr = row_state[r];
-      if (sr < 0 || sr >= num_states) {
-        if (c == 0 && status) atomicCAS(status, 0, RLB_ERR_BOUNDS);
-        sr = 0;
-      }
+  constexpr int AHEAD = 4;
+  for (long long rb = r0; rb < r1; rb += AHEAD) {
+    uint4 raw[AHEAD];
+    int offs[AHEAD];
 #pragma unroll
-      for (int j = 0; j < TAPS - 1; ++j) {
-        const int back = TAPS - 1 - j;
-        uint4 raw = make_uint4(0, 0, 0, 0);
-        if (back <= off) raw = *reinterpret_cast<const uint4*>(x + (r - back) * ldx + c);
-        else if (back <= pos) raw = *reinterpret_cast<const uint4*>(ring + (sr * TAPS + (pos - back) % TAPS) * channels + c);
-        unpack8(raw, win[j]);
-      }
+    for (int a = 0; a < AHEAD; ++a) {
+      raw[a] = rb + a < r1 ? *reinterpret_cast<const uint4*>(x + (rb + a) * ldx + c) : make_uint4(0, 0, 0, 0);
+      offs[a] = rb + a < r1 ? row_off[rb + a] : 1;
     }
-    unpack8(*reinterpret_cast<const uint4*>(x + r * ldx + c), win[TAPS - 1]);
-    uint32_t o[4];
 #pragma unroll
-    for (int k = 0; k < 8; k += 2) {
-      float a0 = b[k], a1 = b[k + 1];
+    for (int a = 0; a < AHEAD; ++a) {
+      const long long r = rb + a;
+      if (r >= r1) break;
+      const int off = offs[a];
+      if (r == r0 || off == 0) {      // the inputs before this row: of the same piece, of the ring, or none
+        const int pos = positions[r];
+        long long sr = row_state[r];
+        if (sr < 0 || sr >= num_states) {
+          if (c == 0 && status) atomicCAS(status, 0, RLB_ERR_BOUNDS);
+          sr = 0;
+        }
 #pragma unroll
-      for (int j = 0; j < TAPS; ++j) {
-        a0 = fmaf(wv[k][j], win[j][k], a0);
-        a1 = fmaf(wv[k + 1][j], win[j][k + 1], a1);
+        for (int j = 0; j < TAPS - 1; ++j) {
+          const int back = TAPS - 1 - j;
+          uint4 before = make_uint4(0, 0, 0, 0);
+          if (back <= off) before = *reinterpret_cast<const uint4*>(x + (r - back) * ldx + c);
+          else if (back <= pos) before = *reinterpret_cast<const uint4*>(ring + (sr * TAPS + (pos - back) % TAPS) * channels + c);
+          unpack8(before, win[j]);
+        }
       }
-      o[k / 2] = pack_bf16x2(rc_silu(a0), rc_silu(a1));
+      unpack8(raw[a], win[TAPS - 1]);
+      uint32_t o[4];
+#pragma unroll
+      for (int k = 0; k < 8; k += 2) {
+        float a0 = b[k], a1 = b[k + 1];
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) {
+          a0 = fmaf(wv[k][j], win[j][k], a0);
+          a1 = fmaf(wv[k + 1][j], win[j][k + 1], a1);
+        }
+        o[k / 2] = pack_bf16x2(a0 / (1.f + __expf(-a0)), a1 / (1.f + __expf(-a1)));
+      }
+      *reinterpret_cast<uint4*>(u + r * ldu + c) = make_uint4(o[0], o[1], o[2], o[3]);
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+        for (int k = 0; k < 8; ++k) win[j][k] = win[j + 1][k];
     }
-    *reinterpret_cast<uint4*>(u + r * ldu + c) = make_uint4(o[0], o[1], o[2], o[3]);
-#pragma unroll
-    for (int j = 0; j < TAPS - 1; ++j)
-#pragma unroll
-      for (int k = 0; k < 8; ++k) win[j][k] = win[j + 1][k];
   }
 }
 
@@ -659,10 +672,18 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmap_whi, const __grid_con
       S[q * 4] = v.x; S[q * 4 + 1] = v.y; S[q * 4 + 2] = v.z; S[q * 4 + 3] = v.w;
     }
     bool ok = true;
+    float4 u[DS_VB / 4];
+    auto fetch = [&](int c) {      // the row's part of V' of chunk c
+      const float* up = p.u0 + ((static_cast<long long>(c) * p.heads + head) * RT_C + row) * p.vdim + v0;
+#pragma unroll
+      for (int q = 0; q < DS_VB / 4; ++q) u[q] = v0 + q * 4 < p.vdim ? *reinterpret_cast<const float4*>(up + q * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+    };
+    fetch(c0);
     for (int c = c0; c < c1; ++c) {
       const uint32_t ph = (c - c0) & 1;
       const long long tile = static_cast<long long>(c) * p.heads + head;
       const int first = p.chunk_row[c], rows = p.chunk_rows[c];
+      const float f = exp2f(p.cum[head * p.rows + first + rows - 1]);
       // the state as operand (the products that read the tiles before have completed), the chunk's start state for the outputs
 #pragma unroll
       for (int q = 0; q < DS_VB / 8; ++q) {
@@ -671,24 +692,11 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmap_whi, const __grid_con
       }
       fence_proxy_async();
       mbar_arrive(smem_u32(s_ready));
-      float4 u[DS_VB / 4];
-      const float* up = p.u0 + (tile * RT_C + row) * p.vdim + v0;
-#pragma unroll
-      for (int q = 0; q < DS_VB / 4; ++q) u[q] = v0 + q * 4 < p.vdim ? *reinterpret_cast<const float4*>(up + q * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
-      const float f = exp2f(p.cum[head * p.rows + first + rows - 1]);
-      if (mine) {
-        float* so = p.start + (tile * p.dim + row) * p.vdim + v0;
-#pragma unroll
-        for (int q = 0; q < DS_VB / 4; ++q)
-          if (v0 + q * 4 < p.vdim) *reinterpret_cast<float4*>(so + q * 4) = make_float4(S[q * 4], S[q * 4 + 1], S[q * 4 + 2], S[q * 4 + 3]);
-      }
       if (!mbar_wait(smem_u32(acc1), ph, abort_flag, p.status, RLB_ERR_WAIT_TMEM_FULL)) {
         ok = false;
         break;
       }
       tc_fence_after();
-      __nv_bfloat16 *gh = p.uu_hi + (first + row) * static_cast<long long>(p.heads * p.vdim) + head * p.vdim + v0,
-                    *gl = p.uu_lo + (first + row) * static_cast<long long>(p.heads * p.vdim) + head * p.vdim + v0;
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         uint32_t r[32];
@@ -705,15 +713,30 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmap_whi, const __grid_con
           const uint32_t o = rt_sw(row, half * 4 + q);
           *reinterpret_cast<uint4*>(u_hi + o) = hi;
           *reinterpret_cast<uint4*>(u_lo + o) = lo;
-          if (row < rows && v0 + half * 32 + q * 8 < p.vdim) {
-            *reinterpret_cast<uint4*>(gh + half * 32 + q * 8) = hi;
-            *reinterpret_cast<uint4*>(gl + half * 32 + q * 8) = lo;
-          }
         }
       }
       fence_proxy_async();
       tc_fence_before();
       mbar_arrive(smem_u32(u_ready));
+      // under the second product: the next chunk's V', the chunk's start state and its writes (the warp's own rows, line by line)
+      if (c + 1 < c1) fetch(c + 1);
+      if (mine) {
+        float* so = p.start + (tile * p.dim + row) * p.vdim + v0;
+#pragma unroll
+        for (int q = 0; q < DS_VB / 4; ++q)
+          if (v0 + q * 4 < p.vdim) *reinterpret_cast<float4*>(so + q * 4) = make_float4(S[q * 4], S[q * 4 + 1], S[q * 4 + 2], S[q * 4 + 3]);
+      }
+      __syncwarp();
+#pragma unroll
+      for (int q = 0; q < 8; ++q) {
+        const int r = quarter * 32 + q * 4 + (lane >> 3), piece = lane & 7;
+        if (r < rows && v0 + piece * 8 < p.vdim) {
+          const long long g = (first + r) * static_cast<long long>(p.heads * p.vdim) + head * p.vdim + v0 + piece * 8;
+          *reinterpret_cast<uint4*>(p.uu_hi + g) = *reinterpret_cast<const uint4*>(u_hi + rt_sw(r, piece));
+          *reinterpret_cast<uint4*>(p.uu_lo + g) = *reinterpret_cast<const uint4*>(u_lo + rt_sw(r, piece));
+        }
+      }
+      __syncwarp();
       if (!mbar_wait(smem_u32(acc2), ph, abort_flag, p.status, RLB_ERR_WAIT_TMEM_FULL)) {
         ok = false;
         break;
@@ -1102,41 +1125,48 @@ __global__ void __launch_bounds__(256) mamba2_step_kernel(RecStep s) {
   }
 }
 
-// KEEP: the state stays in registers between the read-out and the write (at most 8 float4 per thread).
-constexpr int DD_THREADS = 512;
-template <bool KEEP>
-__global__ void __launch_bounds__(DD_THREADS, 2) delta_step_kernel(RecStep s) {
-  extern __shared__ float sm[];
+// The head's state is contiguous (at most 64 KB): one bulk copy brings it to shared memory while the convolution runs, the read-out and the
+// write work there, one bulk copy takes it back. The state's last writer stands far enough back on the stream for the copy to start before
+// the dependency wait: a kernel may start once its predecessor has seen all work before it complete.
+constexpr int DD_THREADS = 256;
+__global__ void __launch_bounds__(DD_THREADS, 3) delta_step_kernel(RecStep s) {
+  extern __shared__ __align__(16) float sm[];
   __shared__ float red[32];
-  float *q = sm, *k = q + s.dim, *v = k + s.dim;            // v: the value, then what is written
+  __shared__ __align__(8) uint64_t bar;
+  __shared__ int abort_flag;
+  float4* S = reinterpret_cast<float4*>(sm);                // [dim][vdim / 4]
+  float *q = sm + s.dim * s.vdim, *k = q + s.dim, *v = k + s.dim;      // v: the value, then what is written
   float4* part = reinterpret_cast<float4*>(v + s.vdim);     // [2][DD_THREADS]
   const int row = blockIdx.x, head = blockIdx.y, tid = threadIdx.x, per = s.heads / s.groups, group = head / per, n = s.groups * s.dim;
-  pdl_sync();
   const long long sr = s.state_rows[row];
-  if (sr < 0 || sr >= s.num_states) {
+  const bool good = sr >= 0 && sr < s.num_states;
+  float* state = s.state + ((good ? sr : 0) * s.heads + head) * static_cast<long long>(s.dim) * s.vdim;
+  const uint32_t bytes = s.dim * s.vdim * 4;
+  if (tid == 0) {
+    mbar_init(smem_u32(&bar), 1);
+    abort_flag = 0;
+    mbar_fence_init();
+    fence_proxy_async();
+    if (good) {
+      mbar_arrive_expect_tx(smem_u32(&bar), bytes);
+      asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(sm)), "l"(state), "r"(bytes),
+                   "r"(smem_u32(&bar))
+                   : "memory");
+    }
+  }
+  pdl_sync();
+  if (!good) {      // uniform
     if (tid == 0 && s.status) atomicCAS(s.status, 0, RLB_ERR_BOUNDS);
     return;
   }
   const int pos = s.positions[row];
-  const int c4 = s.vdim / 4, slices = DD_THREADS / c4, slice = tid / c4, col = tid % c4;
-  const bool live = slice < slices;
-  float4* S = reinterpret_cast<float4*>(s.state + (sr * s.heads + head) * static_cast<long long>(s.dim) * s.vdim) + col;
-  constexpr int U = 8;
-  float4 a[U];
-  if (KEEP) {
-#pragma unroll
-    for (int u = 0; u < U; ++u) {
-      const int i = slice + u * slices;
-      a[u] = live && i < s.dim && pos != 0 ? S[static_cast<long long>(i) * c4] : make_float4(0.f, 0.f, 0.f, 0.f);
-    }
-  }
   const float beta_in = __bfloat162float(s.p[row * s.ldp + s.b_off + head]), dt_in = __bfloat162float(s.p[row * s.ldp + s.a_off + head]);
   const float dt_b = __bfloat162float(s.dt_bias[head]), A_log = __bfloat162float(s.A_log[head]);
   const bool first = head % per == 0;
   step_convolve(s, row, sr, pos, 2 * s.dim + s.vdim,
                 [&](int i) { return i < s.dim ? group * s.dim + i : (i < 2 * s.dim ? n + group * s.dim + i - s.dim : 2 * n + head * s.vdim + i - 2 * s.dim); },
-                [&](int i) { return i >= 2 * s.dim || first; }, [&](int i, float x) { sm[i] = x; });
-  __syncthreads();
+                [&](int i) { return i >= 2 * s.dim || first; }, [&](int i, float x) { q[i] = x; });
+  __syncthreads();      // (also: the barrier has been initialised)
   float qq = 0.f, kk = 0.f, qk = 0.f;      // every warp for itself
   for (int i = tid & 31; i < s.dim; i += 32) {
     const float qv = q[i], kv = k[i];
@@ -1149,24 +1179,21 @@ __global__ void __launch_bounds__(DD_THREADS, 2) delta_step_kernel(RecStep s) {
   qk = warp_sum(qk);
   const float qf = 1.f / (sqrtf(qq + s.unit_eps) * sqrtf(static_cast<float>(s.dim))), kf = 1.f / sqrtf(kk + s.unit_eps);
   const float beta = 1.f / (1.f + expf(-beta_in)), dec = expf(-expf(A_log) * rc_softplus(dt_in + dt_b));
+  const int c4 = s.vdim / 4, slices = DD_THREADS / c4, slice = tid / c4, col = tid % c4;
+  const bool live = slice < slices;
+  const bool ok = mbar_wait(smem_u32(&bar), 0, &abort_flag, s.status, RLB_ERR_WAIT_FULL);
   float4 sk = make_float4(0.f, 0.f, 0.f, 0.f), sq = sk;
-  auto read = [&](const float4& t, int i) {
-    const float kv = k[i], qv = q[i];
-    sk.x = fmaf(t.x, kv, sk.x); sk.y = fmaf(t.y, kv, sk.y); sk.z = fmaf(t.z, kv, sk.z); sk.w = fmaf(t.w, kv, sk.w);
-    sq.x = fmaf(t.x, qv, sq.x); sq.y = fmaf(t.y, qv, sq.y); sq.z = fmaf(t.z, qv, sq.z); sq.w = fmaf(t.w, qv, sq.w);
-  };
-  if (live) {
-    if (KEEP) {
-#pragma unroll
-      for (int u = 0; u < U; ++u)
-        if (slice + u * slices < s.dim) read(a[u], slice + u * slices);
-    } else if (pos != 0) {
+  if (live && pos != 0) {
 #pragma unroll 4
-      for (int i = slice; i < s.dim; i += slices) read(S[static_cast<long long>(i) * c4], i);
+    for (int i = slice; i < s.dim; i += slices) {
+      const float4 t = S[i * c4 + col];
+      const float kv = k[i], qv = q[i];
+      sk.x = fmaf(t.x, kv, sk.x); sk.y = fmaf(t.y, kv, sk.y); sk.z = fmaf(t.z, kv, sk.z); sk.w = fmaf(t.w, kv, sk.w);
+      sq.x = fmaf(t.x, qv, sq.x); sq.y = fmaf(t.y, qv, sq.y); sq.z = fmaf(t.z, qv, sq.z); sq.w = fmaf(t.w, qv, sq.w);
     }
-    part[tid] = sk;
-    part[DD_THREADS + tid] = sq;
   }
+  part[tid] = sk;
+  part[DD_THREADS + tid] = sq;
   __syncthreads();
   float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
   if (tid < c4) {
@@ -1186,18 +1213,18 @@ __global__ void __launch_bounds__(DD_THREADS, 2) delta_step_kernel(RecStep s) {
   __syncthreads();
   if (live) {
     const float4 w = reinterpret_cast<const float4*>(v)[col];
-    auto write = [&](const float4& t, int i) {
-      const float kv = k[i];
-      S[static_cast<long long>(i) * c4] = make_float4(fmaf(dec, t.x, kv * w.x), fmaf(dec, t.y, kv * w.y), fmaf(dec, t.z, kv * w.z), fmaf(dec, t.w, kv * w.w));
-    };
-    if (KEEP) {
-#pragma unroll
-      for (int u = 0; u < U; ++u)
-        if (slice + u * slices < s.dim) write(a[u], slice + u * slices);
-    } else {
 #pragma unroll 4
-      for (int i = slice; i < s.dim; i += slices) write(pos != 0 ? S[static_cast<long long>(i) * c4] : make_float4(0.f, 0.f, 0.f, 0.f), i);
+    for (int i = slice; i < s.dim; i += slices) {
+      const float4 t = pos != 0 ? S[i * c4 + col] : make_float4(0.f, 0.f, 0.f, 0.f);
+      const float kv = k[i];
+      S[i * c4 + col] = make_float4(fmaf(dec, t.x, kv * w.x), fmaf(dec, t.y, kv * w.y), fmaf(dec, t.z, kv * w.z), fmaf(dec, t.w, kv * w.w));
     }
+  }
+  fence_proxy_async();
+  __syncthreads();
+  if (tid == 0 && ok) {
+    asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(state), "r"(smem_u32(sm)), "r"(bytes) : "memory");
+    tma_store_commit();
   }
   const float ss = block_sum(o.x * o.x + o.y * o.y + o.z * o.z + o.w * o.w, red);
   if (tid < c4) {
@@ -1209,6 +1236,7 @@ __global__ void __launch_bounds__(DD_THREADS, 2) delta_step_kernel(RecStep s) {
         make_uint2(pack_bf16x2(o.x * rstd * w0.x * rc_silu(g0.x), o.y * rstd * w0.y * rc_silu(g0.y)),
                    pack_bf16x2(o.z * rstd * w1.x * rc_silu(g1.x), o.w * rstd * w1.y * rc_silu(g1.y)));
   }
+  if (tid == 0) tma_store_wait<0>();
 }
 
 int set_smem(const void* kernel, int bytes, int* configured) {
@@ -1266,11 +1294,14 @@ RLB_API int rlb_rec_step(const RecArgs* a, void* stream) {
             a->eps, static_cast<__nv_bfloat16*>(a->y), a->ldy, a->status};
   const dim3 grid(a->pieces, a->heads), block(256);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const size_t sm = sizeof(float) * (a->vdim + 2 * a->dim) + sizeof(float4) * (a->delta ? 2 * DD_THREADS : 256);
-  if (!a->delta) return static_cast<int>(rlb_launch_pdl(mamba2_step_kernel, grid, block, sm, st, s));
-  const int slices = DD_THREADS / (a->vdim / 4);
-  if (a->dim <= 8 * slices) return static_cast<int>(rlb_launch_pdl(delta_step_kernel<true>, grid, dim3(DD_THREADS), sm, st, s));
-  return static_cast<int>(rlb_launch_pdl(delta_step_kernel<false>, grid, dim3(DD_THREADS), sm, st, s));
+  const int vec = a->vdim + 2 * a->dim;
+  if (!a->delta) return static_cast<int>(rlb_launch_pdl(mamba2_step_kernel, grid, block, sizeof(float) * vec + sizeof(float4) * 256, st, s));
+  if (reinterpret_cast<uintptr_t>(a->state) & 15) return -3;
+  const int sm = static_cast<int>(sizeof(float)) * (a->dim * a->vdim + vec) + static_cast<int>(sizeof(float4)) * 2 * DD_THREADS;
+  static int conf = 0;
+  const int rc = set_smem(reinterpret_cast<const void*>(delta_step_kernel), sm, &conf);
+  if (rc) return rc;
+  return static_cast<int>(rlb_launch_pdl(delta_step_kernel, grid, dim3(DD_THREADS), sm, st, s));
 }
 
 // Portions: rows [row0, rows) of u, p, y in chunks of at most 128 rows (chunk_row counts from row0); piece i owns chunks [piece_chunk[i],
