@@ -283,9 +283,13 @@ gqa_rows_kernel(const T* __restrict__ p, GqaShape s, const T* __restrict__ k_cac
     if (tid < n) sc[tid] = pj;
     __syncthreads();
     for (int i = tid; i < s.vdim; i += 128) {
-      float v = o[i] * c;
-      for (int j = 0; j < n; ++j) v = fmaf(sc[j], ldf(v_cache + rows[j] * s.vdim + i), v);
-      o[i] = v;
+      float v[4] = {0.f, 0.f, 0.f, 0.f};
+      int j = 0;
+      for (; j + 4 <= n; j += 4)
+#pragma unroll
+        for (int q = 0; q < 4; ++q) v[q] = fmaf(sc[j + q], ldf(v_cache + rows[j + q] * s.vdim + i), v[q]);
+      for (; j < n; ++j) v[0] = fmaf(sc[j], ldf(v_cache + rows[j] * s.vdim + i), v[0]);
+      o[i] = fmaf(o[i], c, (v[0] + v[1]) + (v[2] + v[3]));
     }
   }
   const float inv = l > 0.f ? 1.f / l : 0.f;

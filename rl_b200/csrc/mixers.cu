@@ -102,6 +102,7 @@ __global__ void __launch_bounds__(256) gemm_rows_kernel(RowsGemm g) {
       ws[k][r] = (n0 + r < g.N && k0 + k < g.K) ? ld(W + static_cast<long long>(n0 + r) * g.ldw + k0 + k) : 0.f;
     }
     __syncthreads();
+    float part[4][4] = {};      // summed apart: chains of RG_K terms round less than one of K
 #pragma unroll
     for (int k = 0; k < RG_K; ++k) {
       float av[4], wv[4];
@@ -113,8 +114,12 @@ __global__ void __launch_bounds__(256) gemm_rows_kernel(RowsGemm g) {
 #pragma unroll
       for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], wv[j], acc[i][j]);
+        for (int j = 0; j < 4; ++j) part[i][j] = fmaf(av[i], wv[j], part[i][j]);
     }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[i][j] += part[i][j];
     __syncthreads();
   }
   const float alpha = g.x ? ld(static_cast<const TI*>(g.alpha)) : 0.f;

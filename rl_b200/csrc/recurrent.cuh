@@ -12,6 +12,9 @@ __device__ __forceinline__ void rc_st(__nv_bfloat16* p, float v) { *p = __float2
 __device__ __forceinline__ float rc_softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 __device__ __forceinline__ float rc_silu(float x) { return x / (1.f + expf(-x)); }
 
+// For activations that are rounded to bf16 right away (the approximate exponential and quotient err by a few units of 2^-22).
+__device__ __forceinline__ float rc_silu_bf16(float x) { return __fdividef(x, 1.f + __expf(-x)); }
+
 // Shared-memory operand tiles of the chunked forms: rows of 64 bf16 (128 bytes, 128-byte swizzle), one atom per 64 columns. The same tile is
 // a K-major operand (rows along M or N) or an MN-major one (rows along K).
 constexpr int RT_C = 128;                 // tokens per chunk

@@ -12,7 +12,7 @@
 //   rec_unit      per (row, group): factors that make delta-rule queries and keys unit vectors
 //   ssd_state, ssd_scan      per (chunk, head) the sum over j, then per piece the chunks' start states
 //   delta_wy      per (chunk, head): A, its inverse (16 x 16 blocks by substitution, then block by block), W, V', decayed keys
-//   delta_scan    per (piece, head, 64 value columns), chunk after chunk: U and the state; both products of a chunk on the tensor cores, the
+//   delta_scan    per (piece, head, 32 or 64 value columns), chunk after chunk: U and the state; both products of a chunk on the tensor cores, the
 //                 next chunk's tiles in flight under them
 //   rec_out       per (chunk, head): scores, decays, both output terms, the mixer's gate (and head norm), store
 //
@@ -58,7 +58,7 @@ struct RecTiles {
 // ---------------------------------------------------------------- convolution of runs of rows, 8 channels per thread
 constexpr int CV_RUN = 16;
 template <int TAPS>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, 5)
 conv_runs_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, __nv_bfloat16* __restrict__ u, long long ldu, long long rows, int channels,
                  const __nv_bfloat16* __restrict__ w, const __nv_bfloat16* __restrict__ bias, const __nv_bfloat16* __restrict__ ring,
                  const int* __restrict__ positions, const int* __restrict__ row_off, const long long* __restrict__ row_state, long long num_states,
@@ -66,11 +66,20 @@ conv_runs_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, __nv_bfloat
   const int c = (blockIdx.y * 128 + threadIdx.x) * 8;
   if (c >= channels) return;
   float wv[8][TAPS], b[8], win[TAPS][8];
+  {
+    float wf[8 * TAPS];      // the channels' taps are contiguous
 #pragma unroll
-  for (int k = 0; k < 8; ++k) {
-    b[k] = bias ? __bfloat162float(bias[c + k]) : 0.f;
+    for (int q = 0; q < TAPS; ++q) {
+      float t[8];
+      unpack8(*reinterpret_cast<const uint4*>(w + static_cast<long long>(c) * TAPS + q * 8), t);
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j) wv[k][j] = __bfloat162float(w[static_cast<long long>(c + k) * TAPS + j]);
+      for (int k = 0; k < 8; ++k) wf[q * 8 + k] = t[k];
+    }
+#pragma unroll
+    for (int k = 0; k < 8; ++k)
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) wv[k][j] = wf[k * TAPS + j];
+    unpack8(bias ? *reinterpret_cast<const uint4*>(bias + c) : make_uint4(0, 0, 0, 0), b);
   }
   const long long r0 = static_cast<long long>(blockIdx.x) * CV_RUN, r1 = min(rows, r0 + CV_RUN);
   constexpr int AHEAD = 4;
@@ -113,7 +122,7 @@ conv_runs_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, __nv_bfloat
           a0 = fmaf(wv[k][j], win[j][k], a0);
           a1 = fmaf(wv[k + 1][j], win[j][k + 1], a1);
         }
-        o[k / 2] = pack_bf16x2(a0 / (1.f + __expf(-a0)), a1 / (1.f + __expf(-a1)));
+        o[k / 2] = pack_bf16x2(rc_silu_bf16(a0), rc_silu_bf16(a1));
       }
       *reinterpret_cast<uint4*>(u + r * ldu + c) = make_uint4(o[0], o[1], o[2], o[3]);
 #pragma unroll
@@ -570,7 +579,10 @@ delta_wy_kernel(const __grid_constant__ CUtensorMap tmap_v, RecTiles p, int atom
 }
 
 // ---------------------------------------------------------------- delta rule: chunk after chunk
-constexpr int DS_THREADS = 192, DS_VB = 64;
+// VB value columns per CTA. High and low parts of the state (and of the writes) stand side by side as one operand of 2 VB columns, so that
+// hi * [hi | lo] is one product; the epilogue adds the two halves.
+constexpr int DS_THREADS = 192;
+template <int VB>
 __global__ void __launch_bounds__(DS_THREADS, 1)
 delta_scan_kernel(const __grid_constant__ CUtensorMap tmap_whi, const __grid_constant__ CUtensorMap tmap_wlo, const __grid_constant__ CUtensorMap tmap_khi,
                   const __grid_constant__ CUtensorMap tmap_klo, RecTiles p, const int* __restrict__ piece_chunk, const int* __restrict__ positions,
@@ -578,14 +590,17 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmap_whi, const __grid_con
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t *w_s = smem, *k_s = smem + 4 * RT_ATOM;                 // each [hi: 2 atoms | lo: 2 atoms]
-  uint8_t *s_hi = smem + 8 * RT_ATOM, *s_lo = s_hi + RT_ATOM, *u_hi = s_lo + RT_ATOM, *u_lo = u_hi + RT_ATOM;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(u_lo + RT_ATOM);
+  constexpr int ATOMS = VB / 32, PIECES = VB / 8;                 // atoms and 16-byte pieces per part of the state and write operands
+  uint8_t *s_s = smem + 8 * RT_ATOM, *u_s = s_s + ATOMS * RT_ATOM;
+  auto hi_at = [](int row, int q) { return rt_sw(row, q); };
+  auto lo_at = [](int row, int q) { return VB == 64 ? RT_ATOM + rt_sw(row, q) : rt_sw(row, q + 4); };
+  uint64_t* bars = reinterpret_cast<uint64_t*>(u_s + ATOMS * RT_ATOM);
   uint64_t *w_full = bars, *w_empty = bars + 1, *k_full = bars + 2, *k_empty = bars + 3, *acc1 = bars + 4, *acc2 = bars + 5, *s_ready = bars + 6,
            *u_ready = bars + 7;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 8);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int v0 = blockIdx.x * DS_VB, head = blockIdx.y, piece = blockIdx.z;
+  const int v0 = blockIdx.x * VB, head = blockIdx.y, piece = blockIdx.z;
   const long long sr = state_rows[piece];
   if (sr < 0 || sr >= num_states) {      // uniform
     if (threadIdx.x == 0 && p.status) atomicCAS(p.status, 0, RLB_ERR_BOUNDS);
@@ -600,7 +615,7 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmap_whi, const __grid_con
     fence_proxy_async();
   }
   if (warp == 1) {
-    tmem_alloc(smem_u32(tmem_slot), 128);
+    tmem_alloc(smem_u32(tmem_slot), 4 * VB);
     tmem_relinquish();
   }
   tc_fence_before();
@@ -630,29 +645,30 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmap_whi, const __grid_con
     }
   } else if (warp == 1) {
     if (lane == 0) {
-      constexpr uint32_t idesc_w = make_idesc_bf16(RT_C, DS_VB, false, true), idesc_k = make_idesc_bf16(RT_C, DS_VB, true, true);
+      constexpr uint32_t idesc_w2 = make_idesc_bf16(RT_C, 2 * VB, false, true), idesc_w1 = make_idesc_bf16(RT_C, VB, false, true);
+      constexpr uint32_t idesc_k2 = make_idesc_bf16(RT_C, 2 * VB, true, true), idesc_k1 = make_idesc_bf16(RT_C, VB, true, true);
       const int steps = (p.dim + 15) / 16;
       for (int c = c0; c < c1; ++c) {
         const uint32_t ph = (c - c0) & 1;
         if (!mbar_wait(smem_u32(w_full), ph, abort_flag, p.status, RLB_ERR_WAIT_FULL)) break;
         if (!mbar_wait(smem_u32(s_ready), ph, abort_flag, p.status, RLB_ERR_WAIT_FLAG)) break;
         tc_fence_after();
-        for (int part = 0; part < 3; ++part) {      // W S
-          const uint32_t w = smem_u32(w_s + (part == 2 ? 2 * RT_ATOM : 0)), s = smem_u32(part == 1 ? s_lo : s_hi);
+        for (int part = 0; part < 2; ++part) {      // W S: hi [hi | lo], then lo hi
+          const uint32_t w = smem_u32(w_s + part * 2 * RT_ATOM);
           for (int kk = 0; kk < steps; ++kk)
-            umma_f16(tmem, make_smem_desc_sw128(w + (kk >> 2) * RT_ATOM + (kk & 3) * 32, 16, 1024), make_smem_desc_sw128(s + kk * 2048, RT_ATOM, 1024),
-                     idesc_w, (part | kk) != 0 ? 1u : 0u);
+            umma_f16(tmem, make_smem_desc_sw128(w + (kk >> 2) * RT_ATOM + (kk & 3) * 32, 16, 1024), make_smem_desc_sw128(smem_u32(s_s) + kk * 2048, RT_ATOM, 1024),
+                     part ? idesc_w1 : idesc_w2, (part | kk) != 0 ? 1u : 0u);
         }
         umma_commit(smem_u32(w_empty));
         umma_commit(smem_u32(acc1));
         if (!mbar_wait(smem_u32(k_full), ph, abort_flag, p.status, RLB_ERR_WAIT_FULL)) break;
         if (!mbar_wait(smem_u32(u_ready), ph, abort_flag, p.status, RLB_ERR_WAIT_FLAG)) break;
         tc_fence_after();
-        for (int part = 0; part < 3; ++part) {      // K^T U
-          const uint32_t k = smem_u32(k_s + (part == 2 ? 2 * RT_ATOM : 0)), u = smem_u32(part == 1 ? u_lo : u_hi);
+        for (int part = 0; part < 2; ++part) {      // K^T U
+          const uint32_t k = smem_u32(k_s + part * 2 * RT_ATOM);
           for (int kk = 0; kk < RT_C / 16; ++kk)
-            umma_f16(tmem + DS_VB, make_smem_desc_sw128(k + kk * 2048, RT_ATOM, 1024), make_smem_desc_sw128(u + kk * 2048, RT_ATOM, 1024), idesc_k,
-                     (part | kk) != 0 ? 1u : 0u);
+            umma_f16(tmem + 2 * VB, make_smem_desc_sw128(k + kk * 2048, RT_ATOM, 1024), make_smem_desc_sw128(smem_u32(u_s) + kk * 2048, RT_ATOM, 1024),
+                     part ? idesc_k1 : idesc_k2, (part | kk) != 0 ? 1u : 0u);
         }
         umma_commit(smem_u32(k_empty));
         umma_commit(smem_u32(acc2));
@@ -663,20 +679,20 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmap_whi, const __grid_con
     const uint32_t lane_addr = static_cast<uint32_t>(quarter * 32) << 16;
     const bool mine = row < p.dim;
     float* st = state + ((sr * p.heads + head) * p.dim + row) * static_cast<long long>(p.vdim) + v0;
-    float S[DS_VB];
+    float S[VB];
     const bool fresh = positions[p.row0 + p.chunk_row[c0]] == 0;
 #pragma unroll
-    for (int q = 0; q < DS_VB / 4; ++q) {
+    for (int q = 0; q < VB / 4; ++q) {
       float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
       if (mine && !fresh && v0 + q * 4 < p.vdim) v = *reinterpret_cast<const float4*>(st + q * 4);
       S[q * 4] = v.x; S[q * 4 + 1] = v.y; S[q * 4 + 2] = v.z; S[q * 4 + 3] = v.w;
     }
     bool ok = true;
-    float4 u[DS_VB / 4];
+    float4 u[VB / 4];
     auto fetch = [&](int c) {      // the row's part of V' of chunk c
       const float* up = p.u0 + ((static_cast<long long>(c) * p.heads + head) * RT_C + row) * p.vdim + v0;
 #pragma unroll
-      for (int q = 0; q < DS_VB / 4; ++q) u[q] = v0 + q * 4 < p.vdim ? *reinterpret_cast<const float4*>(up + q * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int q = 0; q < VB / 4; ++q) u[q] = v0 + q * 4 < p.vdim ? *reinterpret_cast<const float4*>(up + q * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
     };
     fetch(c0);
     for (int c = c0; c < c1; ++c) {
@@ -686,9 +702,12 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmap_whi, const __grid_con
       const float f = exp2f(p.cum[head * p.rows + first + rows - 1]);
       // the state as operand (the products that read the tiles before have completed), the chunk's start state for the outputs
 #pragma unroll
-      for (int q = 0; q < DS_VB / 8; ++q) {
+      for (int q = 0; q < VB / 8; ++q) {
         const float v[8] = {S[q * 8], S[q * 8 + 1], S[q * 8 + 2], S[q * 8 + 3], S[q * 8 + 4], S[q * 8 + 5], S[q * 8 + 6], S[q * 8 + 7]};
-        store_split(s_hi, s_lo, rt_sw(row, q), v);
+        uint4 hi, lo;
+        split8(v, hi, lo);
+        *reinterpret_cast<uint4*>(s_s + hi_at(row, q)) = hi;
+        *reinterpret_cast<uint4*>(s_s + lo_at(row, q)) = lo;
       }
       fence_proxy_async();
       mbar_arrive(smem_u32(s_ready));
@@ -698,10 +717,13 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmap_whi, const __grid_con
       }
       tc_fence_after();
 #pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        uint32_t r[32];
+      for (int half = 0; half < ATOMS; ++half) {
+        uint32_t r[32], r2[32];
         tmem_ld_32x32b_x32(tmem + lane_addr + half * 32, r);
+        tmem_ld_32x32b_x32(tmem + VB + lane_addr + half * 32, r2);
         tmem_ld_wait();
+#pragma unroll
+        for (int k = 0; k < 32; ++k) r[k] = __float_as_uint(__uint_as_float(r[k]) + __uint_as_float(r2[k]));
 #pragma unroll
         for (int q = 0; q < 4; ++q) {
           const float4 a = u[half * 8 + q * 2], b = u[half * 8 + q * 2 + 1];
@@ -710,9 +732,8 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmap_whi, const __grid_con
                               b.z - __uint_as_float(r[q * 8 + 6]), b.w - __uint_as_float(r[q * 8 + 7])};
           uint4 hi, lo;
           split8(v, hi, lo);
-          const uint32_t o = rt_sw(row, half * 4 + q);
-          *reinterpret_cast<uint4*>(u_hi + o) = hi;
-          *reinterpret_cast<uint4*>(u_lo + o) = lo;
+          *reinterpret_cast<uint4*>(u_s + hi_at(row, half * 4 + q)) = hi;
+          *reinterpret_cast<uint4*>(u_s + lo_at(row, half * 4 + q)) = lo;
         }
       }
       fence_proxy_async();
@@ -723,17 +744,17 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmap_whi, const __grid_con
       if (mine) {
         float* so = p.start + (tile * p.dim + row) * p.vdim + v0;
 #pragma unroll
-        for (int q = 0; q < DS_VB / 4; ++q)
+        for (int q = 0; q < VB / 4; ++q)
           if (v0 + q * 4 < p.vdim) *reinterpret_cast<float4*>(so + q * 4) = make_float4(S[q * 4], S[q * 4 + 1], S[q * 4 + 2], S[q * 4 + 3]);
       }
       __syncwarp();
 #pragma unroll
-      for (int q = 0; q < 8; ++q) {
-        const int r = quarter * 32 + q * 4 + (lane >> 3), piece = lane & 7;
+      for (int q = 0; q < PIECES; ++q) {
+        const int r = quarter * 32 + q * (32 / PIECES) + lane / PIECES, piece = lane % PIECES;
         if (r < rows && v0 + piece * 8 < p.vdim) {
           const long long g = (first + r) * static_cast<long long>(p.heads * p.vdim) + head * p.vdim + v0 + piece * 8;
-          *reinterpret_cast<uint4*>(p.uu_hi + g) = *reinterpret_cast<const uint4*>(u_hi + rt_sw(r, piece));
-          *reinterpret_cast<uint4*>(p.uu_lo + g) = *reinterpret_cast<const uint4*>(u_lo + rt_sw(r, piece));
+          *reinterpret_cast<uint4*>(p.uu_hi + g) = *reinterpret_cast<const uint4*>(u_s + hi_at(r, piece));
+          *reinterpret_cast<uint4*>(p.uu_lo + g) = *reinterpret_cast<const uint4*>(u_s + lo_at(r, piece));
         }
       }
       __syncwarp();
@@ -743,18 +764,19 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmap_whi, const __grid_con
       }
       tc_fence_after();
 #pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        uint32_t r[32];
-        tmem_ld_32x32b_x32(tmem + DS_VB + lane_addr + half * 32, r);
+      for (int half = 0; half < ATOMS; ++half) {
+        uint32_t r[32], r2[32];
+        tmem_ld_32x32b_x32(tmem + 2 * VB + lane_addr + half * 32, r);
+        tmem_ld_32x32b_x32(tmem + 3 * VB + lane_addr + half * 32, r2);
         tmem_ld_wait();
 #pragma unroll
-        for (int k = 0; k < 32; ++k) S[half * 32 + k] = fmaf(S[half * 32 + k], f, __uint_as_float(r[k]));
+        for (int k = 0; k < 32; ++k) S[half * 32 + k] = fmaf(S[half * 32 + k], f, __uint_as_float(r[k]) + __uint_as_float(r2[k]));
       }
       tc_fence_before();
     }
     if (ok && mine) {
 #pragma unroll
-      for (int q = 0; q < DS_VB / 4; ++q)
+      for (int q = 0; q < VB / 4; ++q)
         if (v0 + q * 4 < p.vdim) *reinterpret_cast<float4*>(st + q * 4) = make_float4(S[q * 4], S[q * 4 + 1], S[q * 4 + 2], S[q * 4 + 3]);
     }
   }
@@ -762,7 +784,7 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmap_whi, const __grid_con
   __syncthreads();
   if (warp == 1) {
     tc_fence_after();
-    tmem_dealloc(tmem, 128);
+    tmem_dealloc(tmem, 4 * VB);
   }
 }
 
@@ -965,7 +987,7 @@ rec_out_kernel(const __grid_constant__ CUtensorMap tmap_v, const __grid_constant
 #pragma unroll
           for (int k = 0; k < 8; ++k) {
             const float acc = __uint_as_float(r[q * 8 + k]);
-            g[k] = (DELTA ? acc * rstd * w[k] : fmaf(Dh, w[k], acc)) * rc_silu(g[k]);
+            g[k] = (DELTA ? acc * rstd * w[k] : fmaf(Dh, w[k], acc)) * rc_silu_bf16(g[k]);
           }
 #pragma unroll
           for (int k = 0; k < 4; ++k) o[k] = pack_bf16x2(g[2 * k], g[2 * k + 1]);
@@ -1272,7 +1294,9 @@ RLB_API int rlb_conv_runs(const void* x, long long ldx, void* u, long long ldu, 
                           void* stream) {
   if (rows <= 0) return 0;
   if (taps < 2 || taps > 4 || channels % 8 || ldx % 8 || ldu % 8 || !row_off || !row_state) return -2;
-  if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(u) | reinterpret_cast<uintptr_t>(ring)) & 15) return -3;
+  if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(u) | reinterpret_cast<uintptr_t>(ring) | reinterpret_cast<uintptr_t>(w) |
+       reinterpret_cast<uintptr_t>(bias)) & 15)
+    return -3;
   const dim3 grid(static_cast<unsigned>((rows + CV_RUN - 1) / CV_RUN), (channels / 8 + 127) / 128);
   auto k = taps == 2 ? conv_runs_kernel<2> : (taps == 3 ? conv_runs_kernel<3> : conv_runs_kernel<4>);
   k<<<grid, 128, 0, static_cast<cudaStream_t>(stream)>>>(static_cast<const __nv_bfloat16*>(x), ldx, static_cast<__nv_bfloat16*>(u), ldu, rows, channels,
@@ -1360,7 +1384,7 @@ RLB_API int rlb_rec_portions(const RecArgs* a, void* stream) {
   if (rc) return -100 - rc;
   const int smem_out = 4 * RT_ATOM + 2 * av * RT_SATOM + (a->delta ? 2 : 1) * av * RT_ATOM + (4 * RT_C + RC_THREADS) * 4 + 64 + 1024;
   const int cols_out = vpad <= 128 ? 256 : 512;
-  static int conf_state = 0, conf_out[2] = {0, 0}, conf_wy = 0, conf_scan = 0;
+  static int conf_state = 0, conf_out[2] = {0, 0}, conf_wy = 0, conf_scan[2] = {0, 0};
   if (!a->delta) {
     const int smem_state = (4 + av) * RT_ATOM + RT_C * 4 + 64 + 1024;
     if ((rc = set_smem(reinterpret_cast<const void*>(ssd_state_kernel), smem_state, &conf_state))) return rc;
@@ -1383,12 +1407,14 @@ RLB_API int rlb_rec_portions(const RecArgs* a, void* stream) {
     if (rc) return -100 - rc;
   }
   const int smem_wy = 4 * RT_ATOM + 68 * 1024 + av * RT_ATOM + (WY_TMP + 5 * RT_C) * 4 + 64 + 1024;
-  const int smem_scan = 12 * RT_ATOM + 128 + 1024;
+  const bool narrow = static_cast<long long>(a->pieces) * a->heads * ((a->vdim + 63) / 64) <= 74;      // few chains: more, narrower CTAs
+  const int vb = narrow ? 32 : 64, smem_scan = (8 + vb / 16) * RT_ATOM + 128 + 1024;
+  auto scan = narrow ? delta_scan_kernel<32> : delta_scan_kernel<64>;
   if ((rc = set_smem(reinterpret_cast<const void*>(delta_wy_kernel), smem_wy, &conf_wy))) return rc;
-  if ((rc = set_smem(reinterpret_cast<const void*>(delta_scan_kernel), smem_scan, &conf_scan))) return rc;
+  if ((rc = set_smem(reinterpret_cast<const void*>(scan), smem_scan, &conf_scan[narrow]))) return rc;
   if ((rc = set_smem(reinterpret_cast<const void*>(rec_out_kernel<true>), smem_out, &conf_out[1]))) return rc;
   delta_wy_kernel<<<grid, RC_THREADS, smem_wy, st>>>(tv, t, av);
-  delta_scan_kernel<<<dim3((a->vdim + DS_VB - 1) / DS_VB, a->heads, a->pieces), DS_THREADS, smem_scan, st>>>(tm[0], tm[1], tm[2], tm[3], t, a->piece_chunk,
+  scan<<<dim3((a->vdim + vb - 1) / vb, a->heads, a->pieces), DS_THREADS, smem_scan, st>>>(tm[0], tm[1], tm[2], tm[3], t, a->piece_chunk,
       a->positions, a->state_rows, a->state, a->num_states);
   rec_out_kernel<true><<<grid, RC_THREADS, smem_out, st>>>(tm[4], tm[5], t, av, cols_out);
   return static_cast<int>(cudaGetLastError());
