@@ -28,11 +28,20 @@ struct GqaShape {
   int q_off, k_off, v_off;
   int heads, kv_heads, dim, vdim;
   int block_size, num_blocks;
+  int halves;            // rotated pairs are (i, i + half) instead of (2i, 2i + 1)
+};
+
+// Values of a layer that mixes them with an earlier layer's: v <- (1 - share) v + share v_first.
+template <typename T>
+struct ValueMix {
+  const T* first;        // column of kv head 0 of the earlier layer's projected rows (null: no mixing)
+  long long ld;
+  const T* share;        // one number
 };
 
 // One CTA per row, a warp per head in turn: RMS norm and rotation of the query and key heads in place, keys and values into the cache. The
-// row's cosines and sines are computed once for all heads. A lane keeps pairs (2i, 2i + 1), which is also what the rotation turns. Few rows
-// are spread over several CTAs each (blockIdx.y).
+// row's cosines and sines are computed once for all heads. A lane keeps pairs (2i, 2i + 1), which is also what the interleaved rotation
+// turns. Few rows are spread over several CTAs each (blockIdx.y).
 constexpr int GP_WARPS = 8, GP_KEEP = 4;      // pairs a lane keeps in registers
 template <typename T>
 struct Pair;
@@ -65,8 +74,8 @@ struct Pair<__nv_bfloat16> {
 
 template <typename T>
 __global__ void __launch_bounds__(GP_WARPS * 32)
-gqa_prep_kernel(T* __restrict__ p, GqaShape s, const int* __restrict__ positions, const long long* __restrict__ slots, const T* __restrict__ q_norm,
-                const T* __restrict__ k_norm, const float* __restrict__ freq, int half, float gain, float eps, T* __restrict__ k_cache,
+gqa_prep_kernel(T* __restrict__ p, GqaShape s, ValueMix<T> mix, const int* __restrict__ positions, const long long* __restrict__ slots,
+                const T* __restrict__ q_norm, const T* __restrict__ k_norm, const float* __restrict__ freq, int half, float gain, float eps, T* __restrict__ k_cache,
                 T* __restrict__ v_cache, int* status) {
   extern __shared__ float2 turn[];      // [half] (cosine, sine)
   const int lane = threadIdx.x & 31;
@@ -91,8 +100,14 @@ gqa_prep_kernel(T* __restrict__ p, GqaShape s, const int* __restrict__ positions
     const bool is_q = unit < s.heads, is_k = !is_q && unit < s.heads + s.kv_heads;
     const int head = is_q ? unit : (is_k ? unit - s.heads : unit - s.heads - s.kv_heads);
     if (!is_q && !is_k) {
+      T* v = pr + s.v_off + head * s.vdim;
+      if (mix.first) {
+        const T* f = mix.first + row * mix.ld + head * s.vdim;
+        const float share = ldf(mix.share);
+        for (int i = lane; i < s.vdim; i += 32) stf(v + i, (1.f - share) * ldf(v + i) + share * ldf(f + i));
+        __syncwarp();
+      }
       if (!cached) continue;
-      const T* v = pr + s.v_off + head * s.vdim;
       T* c = v_cache + ((page * s.kv_heads + head) * s.block_size + off) * s.vdim;
       if (veven) {
         for (int i = lane * 2; i < s.vdim; i += 64) {
@@ -124,6 +139,20 @@ gqa_prep_kernel(T* __restrict__ p, GqaShape s, const int* __restrict__ positions
     }
     ss = warp_sum(ss);
     const float rstd = 1.f / sqrtf(ss / static_cast<float>(s.dim) + eps);
+    if (s.halves) {      // a lane turns entries i and i + half; the sum's shuffles stand between the loads above and these stores
+      auto put = [&](int i, float t) {
+        stf(x + i, t);
+        if (c) stf(c + i, t);
+      };
+      for (int i = lane; i < half; i += 32) {
+        const float a = ldf(x + i) * rstd * ldf(w + i), b = ldf(x + i + half) * rstd * ldf(w + i + half);
+        const float2 r = turn[i];
+        put(i, a * r.x - b * r.y);
+        put(i + half, b * r.x + a * r.y);
+      }
+      for (int i = 2 * half + lane; i < s.dim; i += 32) put(i, ldf(x + i) * rstd * ldf(w + i));
+      continue;
+    }
     auto finish = [&](int i, float2 t) {
       if (2 * i >= s.dim) return;
       const bool two = 2 * i + 1 < s.dim;
@@ -147,20 +176,27 @@ gqa_prep_kernel(T* __restrict__ p, GqaShape s, const int* __restrict__ positions
   }
 }
 
-// The same for bf16 rows with even dim <= 64 * KEEP and even vdim: one warp per row (and share of its heads). A lane turns the same pairs of every
-// head, so cosines, sines and norm weights stay in its registers; four heads are in flight.
-template <int KEEP>
+// The same for bf16 rows with even dim <= 64 * KEEP and even vdim: one warp per row (and share of its heads). A lane keeps the same 32-bit words
+// (two entries) of every head, so cosines, sines and norm weights stay in its registers; four heads are in flight. Interleaved pairs: word
+// lane + 32 j is one pair. HALVES (half even): words 2 s and 2 s + 1 of a lane are r and r + half / 2 with r = lane + 32 s, two pairs, or two
+// neighbours behind the rotated part.
+template <int KEEP, bool HALVES>
 __global__ void __launch_bounds__(GP_WARPS * 32)
-gqa_prep_rows_kernel(__nv_bfloat16* __restrict__ p, GqaShape s, long long rows, const int* __restrict__ positions, const long long* __restrict__ slots,
+gqa_prep_rows_kernel(__nv_bfloat16* __restrict__ p, GqaShape s, ValueMix<__nv_bfloat16> mix, long long rows, const int* __restrict__ positions, const long long* __restrict__ slots,
                      const __nv_bfloat16* __restrict__ q_norm, const __nv_bfloat16* __restrict__ k_norm, const float* __restrict__ freq, int half,
                      float gain, float eps, __nv_bfloat16* __restrict__ k_cache, __nv_bfloat16* __restrict__ v_cache, int* status) {
   constexpr int AHEAD = 4;
   const int lane = threadIdx.x & 31;
   const long long row = static_cast<long long>(blockIdx.x) * GP_WARPS + (threadIdx.x >> 5);
   float2 wq[KEEP], wk[KEEP], turn[KEEP];
+  auto word = [&](int j) {      // may lie behind the head
+    if (!HALVES) return lane + j * 32;
+    const int r = lane + (j >> 1) * 32, hw = half / 2;
+    return r < hw ? r + (j & 1) * hw : half + 2 * (r - hw) + (j & 1);
+  };
 #pragma unroll
   for (int j = 0; j < KEEP; ++j) {
-    const int i = lane + j * 32;
+    const int i = word(j);
     const bool live = 2 * i < s.dim;
     wq[j] = live ? Pair<__nv_bfloat16>::load(q_norm + 2 * i, true) : make_float2(0.f, 0.f);
     wk[j] = live ? Pair<__nv_bfloat16>::load(k_norm + 2 * i, true) : make_float2(0.f, 0.f);
@@ -175,7 +211,7 @@ gqa_prep_rows_kernel(__nv_bfloat16* __restrict__ p, GqaShape s, long long rows, 
   const unsigned at = cached ? static_cast<unsigned>(slot) : 0u, page = at / s.block_size, off = at - page * s.block_size;
 #pragma unroll
   for (int j = 0; j < KEEP; ++j) {
-    const int i = lane + j * 32;
+    const int i = HALVES ? 2 * (lane + (j >> 1) * 32) + (j & 1) : lane + j * 32;      // pair
     turn[j] = make_float2(1.f, 0.f);
     if (i < half) {
       float sn, cs;
@@ -194,7 +230,7 @@ gqa_prep_rows_kernel(__nv_bfloat16* __restrict__ p, GqaShape s, long long rows, 
       const __nv_bfloat16* x = pr + (unit < s.heads ? s.q_off + unit * s.dim : s.k_off + (unit - s.heads) * s.dim);
 #pragma unroll
       for (int j = 0; j < KEEP; ++j) {
-        const int i = lane + j * 32;
+        const int i = word(j);
         v[a][j] = unit < units && 2 * i < s.dim ? Pair<__nv_bfloat16>::load(x + 2 * i, true) : make_float2(0.f, 0.f);
       }
     }
@@ -215,6 +251,24 @@ gqa_prep_rows_kernel(__nv_bfloat16* __restrict__ p, GqaShape s, long long rows, 
       const float rstd = 1.f / sqrtf(ss[a] / static_cast<float>(s.dim) + eps);
       __nv_bfloat16* x = pr + (is_q ? s.q_off : s.k_off) + head * s.dim;
       __nv_bfloat16* c = k_cache + ((static_cast<long long>(page) * s.kv_heads + head) * s.block_size + off) * s.dim;
+      if (HALVES) {
+#pragma unroll
+        for (int j = 0; j < KEEP; j += 2) {
+          const int i0 = word(j), i1 = word(j + 1);
+          const float2 w0 = is_q ? wq[j] : wk[j], w1 = is_q ? wq[j + 1] : wk[j + 1], t0 = turn[j], t1 = turn[j + 1];
+          const float2 e = make_float2(v[a][j].x * rstd * w0.x, v[a][j].y * rstd * w0.y), f = make_float2(v[a][j + 1].x * rstd * w1.x, v[a][j + 1].y * rstd * w1.y);
+          const uint32_t o0 = pack_bf16x2(e.x * t0.x - f.x * t0.y, e.y * t1.x - f.y * t1.y), o1 = pack_bf16x2(f.x * t0.x + e.x * t0.y, f.y * t1.x + e.y * t1.y);
+          if (2 * i0 < s.dim) {
+            *reinterpret_cast<uint32_t*>(x + 2 * i0) = o0;
+            if (!is_q && cached) *reinterpret_cast<uint32_t*>(c + 2 * i0) = o0;
+          }
+          if (2 * i1 < s.dim) {
+            *reinterpret_cast<uint32_t*>(x + 2 * i1) = o1;
+            if (!is_q && cached) *reinterpret_cast<uint32_t*>(c + 2 * i1) = o1;
+          }
+        }
+        continue;
+      }
 #pragma unroll
       for (int j = 0; j < KEEP; ++j) {
         const int i = lane + j * 32;
@@ -227,20 +281,31 @@ gqa_prep_rows_kernel(__nv_bfloat16* __restrict__ p, GqaShape s, long long rows, 
       }
     }
   }
-  if (!cached) return;
+  if (!cached && !mix.first) return;
+  const float share = mix.first ? __bfloat162float(*mix.share) : 0.f;
   for (int g = blockIdx.y; g < s.kv_heads; g += gridDim.y) {
-    const __nv_bfloat16* x = pr + s.v_off + g * s.vdim;
+    __nv_bfloat16* x = pr + s.v_off + g * s.vdim;
+    const __nv_bfloat16* f = mix.first + row * mix.ld + g * s.vdim;
     __nv_bfloat16* c = v_cache + ((static_cast<long long>(page) * s.kv_heads + g) * s.block_size + off) * s.vdim;
-    for (int i = lane * 2; i < s.vdim; i += 64) *reinterpret_cast<uint32_t*>(c + i) = *reinterpret_cast<const uint32_t*>(x + i);
+    for (int i = lane * 2; i < s.vdim; i += 64) {
+      uint32_t t = *reinterpret_cast<const uint32_t*>(x + i);
+      if (mix.first) {
+        const float2 own = unpack_bf16x2(t), old = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(f + i));
+        t = pack_bf16x2((1.f - share) * own.x + share * old.x, (1.f - share) * own.y + share * old.y);
+        *reinterpret_cast<uint32_t*>(x + i) = t;
+      }
+      if (cached) *reinterpret_cast<uint32_t*>(c + i) = t;
+    }
   }
 }
 
-// One CTA per (row, query head): tiles of 128 keys, online softmax, everything in fp32.
+// One CTA per (row, query head): tiles of 128 keys, online softmax, everything in fp32. chunk > 0: only the keys of the row's own run of
+// `chunk` positions are visible.
 constexpr int GR_TILE = 128;
 template <typename T>
 __global__ void __launch_bounds__(128)
 gqa_rows_kernel(const T* __restrict__ p, GqaShape s, const T* __restrict__ k_cache, const T* __restrict__ v_cache, const int* __restrict__ block_table,
-                int bt_stride, const int* __restrict__ seq_lens, float scale, T* __restrict__ y, long long ldy, int* status) {
+                int bt_stride, const int* __restrict__ seq_lens, int chunk, float scale, T* __restrict__ y, long long ldy, int* status) {
   extern __shared__ float sm[];
   __shared__ float red[32];
   float* q = sm;                        // [dim]
@@ -253,7 +318,7 @@ gqa_rows_kernel(const T* __restrict__ p, GqaShape s, const T* __restrict__ k_cac
   for (int i = tid; i < s.vdim; i += 128) o[i] = 0.f;
   const int len = min(seq_lens[row], bt_stride * s.block_size);
   float m = -INFINITY, l = 0.f;
-  for (int t0 = 0; t0 < len; t0 += GR_TILE) {
+  for (int t0 = chunk > 0 && len > 0 ? (len - 1) / chunk * chunk : 0; t0 < len; t0 += GR_TILE) {
     const int n = min(GR_TILE, len - t0);
     __syncthreads();
     if (tid < n) {
@@ -317,53 +382,59 @@ __global__ void gqa_gather_kernel(const uint4* __restrict__ k_cache, const uint4
 }
 }  // namespace
 
-// In place on the projected rows p: RMS norm (weight [dim]) and rotation of the first 2 * half dimensions (interleaved pairs) of every query
-// and key head; keys and values of rows with a slot go to the cache.
+// In place on the projected rows p: RMS norm (weight [dim]) and rotation of the first 2 * half dimensions (pairs (2i, 2i + 1), or (i, i + half)
+// when `halves`) of every query and key head; v_first (row stride ld_first, null: none): values become (1 - share) v + share v_first; keys and
+// values of rows with a slot go to the cache.
 RLB_API int rlb_gqa_prep(void* p, int f32, long long rows, long long ldp, int q_off, int k_off, int v_off, int heads, int kv_heads, int dim, int vdim,
                          int block_size, int num_blocks, const int* positions, const long long* slots, const void* q_norm, const void* k_norm,
-                         const float* freq, int half, float gain, float eps, void* k_cache, void* v_cache, int* status, void* stream) {
+                         const float* freq, int half, int halves, float gain, float eps, const void* v_first, long long ld_first, const void* share,
+                         void* k_cache, void* v_cache, int* status, void* stream) {
   if (rows <= 0) return 0;
-  if (2 * half > dim || kv_heads < 1 || heads % kv_heads) return -2;
-  GqaShape s{ldp, q_off, k_off, v_off, heads, kv_heads, dim, vdim, block_size, num_blocks};
+  if (2 * half > dim || kv_heads < 1 || heads % kv_heads || (v_first && !share)) return -2;
+  GqaShape s{ldp, q_off, k_off, v_off, heads, kv_heads, dim, vdim, block_size, num_blocks, halves};
+  const ValueMix<float> mix32{static_cast<const float*>(v_first), ld_first, static_cast<const float*>(share)};
+  const ValueMix<__nv_bfloat16> mix16{static_cast<const __nv_bfloat16*>(v_first), ld_first, static_cast<const __nv_bfloat16*>(share)};
   const int per_row = (heads + 2 * kv_heads + GP_WARPS - 1) / GP_WARPS;
   const dim3 grid(static_cast<unsigned>(rows), rows >= 148 * 8 ? 1 : (per_row < 64 ? per_row : 64)), block(GP_WARPS * 32);
   const size_t sm = sizeof(float2) * half;
   if (sm > 48 * 1024) return -2;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (!f32 && dim % 2 == 0 && vdim % 2 == 0 && ldp % 2 == 0 && dim <= 256 && (q_off | k_off | v_off) % 2 == 0 &&
+  if (!f32 && dim % 2 == 0 && vdim % 2 == 0 && ldp % 2 == 0 && dim <= 256 && (q_off | k_off | v_off) % 2 == 0 && (!halves || half % 2 == 0) &&
+      ld_first % 2 == 0 && reinterpret_cast<uintptr_t>(v_first) % 4 == 0 &&
       static_cast<long long>(num_blocks) * block_size < 0x7fffffffll) {
     const int share = (heads + kv_heads + 3) / 4;
     const dim3 g(static_cast<unsigned>((rows + GP_WARPS - 1) / GP_WARPS), rows >= 148 * 16 ? 1 : (share < 64 ? share : 64));
-    auto k = dim <= 128 ? gqa_prep_rows_kernel<2> : gqa_prep_rows_kernel<4>;
-    return static_cast<int>(rlb_launch_pdl(k, g, block, 0, st, static_cast<__nv_bfloat16*>(p), s, rows, positions, slots,
+    auto k = halves ? (dim <= 128 ? gqa_prep_rows_kernel<2, true> : gqa_prep_rows_kernel<4, true>)
+                    : (dim <= 128 ? gqa_prep_rows_kernel<2, false> : gqa_prep_rows_kernel<4, false>);
+    return static_cast<int>(rlb_launch_pdl(k, g, block, 0, st, static_cast<__nv_bfloat16*>(p), s, mix16, rows, positions, slots,
                                            static_cast<const __nv_bfloat16*>(q_norm), static_cast<const __nv_bfloat16*>(k_norm), freq, half, gain, eps,
                                            static_cast<__nv_bfloat16*>(k_cache), static_cast<__nv_bfloat16*>(v_cache), status));
   }
   if (f32)
-    return static_cast<int>(rlb_launch_pdl(gqa_prep_kernel<float>, grid, block, sm, st, static_cast<float*>(p), s, positions, slots,
+    return static_cast<int>(rlb_launch_pdl(gqa_prep_kernel<float>, grid, block, sm, st, static_cast<float*>(p), s, mix32, positions, slots,
                                            static_cast<const float*>(q_norm), static_cast<const float*>(k_norm), freq, half, gain, eps,
                                            static_cast<float*>(k_cache), static_cast<float*>(v_cache), status));
-  return static_cast<int>(rlb_launch_pdl(gqa_prep_kernel<__nv_bfloat16>, grid, block, sm, st, static_cast<__nv_bfloat16*>(p), s, positions, slots,
+  return static_cast<int>(rlb_launch_pdl(gqa_prep_kernel<__nv_bfloat16>, grid, block, sm, st, static_cast<__nv_bfloat16*>(p), s, mix16, positions, slots,
                                          static_cast<const __nv_bfloat16*>(q_norm), static_cast<const __nv_bfloat16*>(k_norm), freq, half, gain, eps,
                                          static_cast<__nv_bfloat16*>(k_cache), static_cast<__nv_bfloat16*>(v_cache), status));
 }
 
 RLB_API int rlb_gqa_rows(const void* p, int f32, int rows, long long ldp, int q_off, int heads, int kv_heads, int dim, int vdim, int block_size,
                          int num_blocks, const void* k_cache, const void* v_cache, const int* block_table, int bt_stride, const int* seq_lens,
-                         float scale, void* y, long long ldy, int* status, void* stream) {
+                         int chunk, float scale, void* y, long long ldy, int* status, void* stream) {
   if (rows <= 0) return 0;
   if (kv_heads < 1 || heads % kv_heads || heads > 65535 || dim + vdim > 12000) return -2;
-  GqaShape s{ldp, q_off, 0, 0, heads, kv_heads, dim, vdim, block_size, num_blocks};
+  GqaShape s{ldp, q_off, 0, 0, heads, kv_heads, dim, vdim, block_size, num_blocks, 0};
   const size_t sm = sizeof(float) * ((dim + vdim + GR_TILE + 1) & ~1) + sizeof(long long) * GR_TILE;
   if (sm > 48 * 1024) return -2;
   const dim3 grid(rows, heads);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (f32)
     gqa_rows_kernel<float><<<grid, 128, sm, st>>>(static_cast<const float*>(p), s, static_cast<const float*>(k_cache), static_cast<const float*>(v_cache),
-                                                  block_table, bt_stride, seq_lens, scale, static_cast<float*>(y), ldy, status);
+                                                  block_table, bt_stride, seq_lens, chunk, scale, static_cast<float*>(y), ldy, status);
   else
     gqa_rows_kernel<__nv_bfloat16><<<grid, 128, sm, st>>>(static_cast<const __nv_bfloat16*>(p), s, static_cast<const __nv_bfloat16*>(k_cache),
-                                                          static_cast<const __nv_bfloat16*>(v_cache), block_table, bt_stride, seq_lens, scale,
+                                                          static_cast<const __nv_bfloat16*>(v_cache), block_table, bt_stride, seq_lens, chunk, scale,
                                                           static_cast<__nv_bfloat16*>(y), ldy, status);
   return static_cast<int>(cudaGetLastError());
 }

@@ -343,9 +343,9 @@ __device__ __forceinline__ float tanh_acc(float x) {
   return copysignf(1.f - 2.f / (1.f + expf(2.f * a)), x);
 }
 
-// What follows a product in a layer-list model. LIN_GLU: columns 2i and 2i + 1 are gate and up of a clamped gated unit, the output has
-// N / 2 columns. LIN_GELU_MUL: gelu_tanh times a table row chosen by the row's token. LIN_CAP: scale, then soft cap (cap > 0).
-enum RlbLinearAct : int { LIN_NONE = 0, LIN_GLU = 1, LIN_GELU_MUL = 2, LIN_CAP = 3 };
+// What follows a product in a layer-list model. LIN_GLU, LIN_SILU: columns 2i and 2i + 1 are gate and up of a gated unit (clamped, or silu
+// without limits), the output has N / 2 columns. LIN_GELU_MUL: gelu_tanh times a table row chosen by the row's token. LIN_CAP: scale, then soft cap (cap > 0).
+enum RlbLinearAct : int { LIN_NONE = 0, LIN_GLU = 1, LIN_GELU_MUL = 2, LIN_CAP = 3, LIN_SILU = 4 };
 struct LinearEpi {
   const void* bias;      // [N] in the weights' type, or null: added to the product
   int act;
@@ -356,12 +356,15 @@ struct LinearEpi {
   int table_off, table_cols, vocab;
   const void* ids;       // [rows] int32 or int64
   int ids64;
+  const float* row_scale;   // [rows] or null: the product's rows are multiplied by it first
 };
 __device__ __forceinline__ float clamped_glu(float g, float u, float limit) {
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
   return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
 }
+__device__ __forceinline__ float gated_unit(int act, float g, float u, float limit) { return act == LIN_SILU ? g / (1.f + expf(-g)) * u : clamped_glu(g, u, limit); }
+__host__ __device__ inline bool lin_gated(int act) { return act == LIN_GLU || act == LIN_SILU; }
 __device__ __forceinline__ float gelu_tanh_acc(float z) { return 0.5f * z * (1.f + tanh_acc(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
 __device__ __forceinline__ float soft_cap(float z, float scale, float cap) {
   z *= scale;
@@ -386,7 +389,7 @@ struct LayerEpilogue {
   int act_from;
   LinearEpi lin;
 };
-// Four consecutive columns of one row (col a multiple of 4). LIN_GLU: the two outputs are in .x and .y.
+// Four consecutive columns of one row (col a multiple of 4). Gated units: the two outputs are in .x and .y.
 __device__ __forceinline__ float4 layer_epilogue4(const LayerEpilogue& le, float4 v, long long row, int col, float alpha) {
   if (le.lin.bias) {
     const uint2 bv = *reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(le.lin.bias) + col);
@@ -413,9 +416,9 @@ __device__ __forceinline__ float4 layer_epilogue4(const LayerEpilogue& le, float
     v.y = tanh_acc(alpha * v.y) * w0.y + b0.y;
     v.z = tanh_acc(alpha * v.z) * w1.x + b1.x;
     v.w = tanh_acc(alpha * v.w) * w1.y + b1.y;
-  } else if (le.lin.act == LIN_GLU) {
-    v.x = clamped_glu(v.x, v.y, le.lin.limit);
-    v.y = clamped_glu(v.z, v.w, le.lin.limit);
+  } else if (lin_gated(le.lin.act)) {
+    v.x = gated_unit(le.lin.act, v.x, v.y, le.lin.limit);
+    v.y = gated_unit(le.lin.act, v.z, v.w, le.lin.limit);
   } else if (le.lin.act == LIN_GELU_MUL) {
     const __nv_bfloat16* t = static_cast<const __nv_bfloat16*>(le.lin.table) + lin_token(le.lin, row) * le.lin.ld_table + le.lin.table_off;
     float* f = reinterpret_cast<float*>(&v);
@@ -457,7 +460,8 @@ __device__ __forceinline__ float block_max(float v, float* red) {
 
 // A product and what follows it: out = epilogue(a w^T), for rlb_linear_rows (any size, bf16 or fp32), rlb_linear_tiled and
 // rlb_linear_skinny (bf16 shapes that TMA can address) and rlb_linear_grouped. Grouped: 128-row tile t of `a` belongs to expert
-// tile_expert[t] (-1: unused) whose weight is w + expert * N * ldw; rlb_linear_rows may read row r of `a` from a_rows[r] (-1: zeros).
+// tile_expert[t] (-1: unused) whose weight is w + expert * N * ldw; rlb_linear_rows may read row r of `a` from a_rows[r] (-1: zeros). row_scale
+// [M] (rlb_linear_grouped and rlb_linear_rows): row r of the product is multiplied by row_scale[r] before anything else.
 struct RlbLinear {
   const void* a;
   const void* w;
@@ -468,12 +472,13 @@ struct RlbLinear {
   const int* tile_expert;
   const int* a_rows;
   int* status;
+  const float* row_scale;
   long long lda, ldw, ldo, ld_table;
   int M, N, K, in_f32, out_f32, act, table_off, table_cols, vocab, ids64, experts, num_a_rows;
   float limit, scale, cap;
 };
 inline rlb::LinearEpi rlb_linear_epi(const RlbLinear& l) {
-  return rlb::LinearEpi{l.bias, l.act, l.limit, l.scale, l.cap, l.table, l.ld_table, l.table_off, l.table_cols, l.vocab, l.ids, l.ids64};
+  return rlb::LinearEpi{l.bias, l.act, l.limit, l.scale, l.cap, l.table, l.ld_table, l.table_off, l.table_cols, l.vocab, l.ids, l.ids64, l.row_scale};
 }
 
 // ---------------------------------------------------------------- host helpers

@@ -42,8 +42,9 @@ struct GroupedArgs {
   long long c_expert_stride;  // reduction mode: elements between consecutive experts' outputs
   int out_fp32;
   int accumulate;
-  int glu;                  // rows mode, bf16: columns 2i, 2i + 1 are gate and up of a clamped gated unit, C has N / 2 columns
+  int act;                  // rows mode, bf16: LIN_GLU or LIN_SILU: columns 2i, 2i + 1 are gate and up of a gated unit, C has N / 2 columns
   float limit;
+  const float* row_scale;   // rows mode: [M] or null, multiplies the product's rows
 };
 
 // One unit of work: which tile, which k range, where B / C start.
@@ -223,6 +224,7 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
       const bool row_ok = row < g.M;
       const uint32_t taddr = tmem_base + (static_cast<uint32_t>(quarter * 32) << 16) + acc * BN;
       const int col0 = w.n_blk * BN;
+      const float scale = g.row_scale && row_ok ? g.row_scale[row] : 1.f;
       for (int c = 0; c < BN / 32; ++c) {
         uint32_t r[32];
         tmem_ld_32x32b_x32(taddr + c * 32, r);
@@ -231,7 +233,7 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
         if (!row_ok || col >= g.N) continue;
         float v[32];
 #pragma unroll
-        for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
+        for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]) * scale;
         if (g.out_fp32) {
           float* dst = reinterpret_cast<float*>(g.C) + w.c_off + static_cast<long long>(row) * g.ldc + col;
 #pragma unroll
@@ -245,14 +247,14 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
               *reinterpret_cast<float4*>(dst + q * 4) = o;
             }
           }
-        } else if (g.glu) {
+        } else if (g.act != LIN_NONE) {
           __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(g.C) + static_cast<long long>(row) * g.ldc + col / 2;
 #pragma unroll
           for (int q = 0; q < 4; ++q) {
             if (col + q * 8 < g.N)
               *reinterpret_cast<uint2*>(dst + q * 4) =
-                  make_uint2(pack_bf16x2(clamped_glu(v[q * 8], v[q * 8 + 1], g.limit), clamped_glu(v[q * 8 + 2], v[q * 8 + 3], g.limit)),
-                             pack_bf16x2(clamped_glu(v[q * 8 + 4], v[q * 8 + 5], g.limit), clamped_glu(v[q * 8 + 6], v[q * 8 + 7], g.limit)));
+                  make_uint2(pack_bf16x2(gated_unit(g.act, v[q * 8], v[q * 8 + 1], g.limit), gated_unit(g.act, v[q * 8 + 2], v[q * 8 + 3], g.limit)),
+                             pack_bf16x2(gated_unit(g.act, v[q * 8 + 4], v[q * 8 + 5], g.limit), gated_unit(g.act, v[q * 8 + 6], v[q * 8 + 7], g.limit)));
           }
         } else {
           __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(g.C) + w.c_off + static_cast<long long>(row) * g.ldc + col;
@@ -347,11 +349,11 @@ RLB_API int rlb_gemm_grouped_rows(const void* A, long long lda, const void* B, i
               : launch_grouped<false, false>(ta, tb, g, status, tiles, static_cast<cudaStream_t>(stream));
 }
 
-// rlb_gemm_grouped_rows with the clamped gated unit of LIN_GLU or no epilogue; rows of padding may hold anything.
+// rlb_gemm_grouped_rows with a gated unit or no epilogue, and a factor per row; rows of padding may hold anything.
 RLB_API int rlb_linear_grouped(const RlbLinear* l, void* stream) {
   if (l->M <= 0 || l->N <= 0 || l->K <= 0) return 0;
   if ((l->M % 128) || (l->lda % 8) || (l->ldo % 8) || (l->N % 8) || (l->K % 8) || l->ldw != l->K || !l->tile_expert || l->a_rows) return -2;
-  if (l->in_f32 || l->out_f32 || l->bias || (l->act != LIN_NONE && l->act != LIN_GLU)) return -2;
+  if (l->in_f32 || l->out_f32 || l->bias || (l->act != LIN_NONE && !lin_gated(l->act))) return -2;
   if ((reinterpret_cast<uintptr_t>(l->a) | reinterpret_cast<uintptr_t>(l->w) | reinterpret_cast<uintptr_t>(l->out)) & 15) return -3;
   CUtensorMap ta, tb;
   int rc = rlb_make_tmap_2d(&ta, l->a, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, l->K, l->M, l->lda * 2, BK, BM, CU_TENSOR_MAP_SWIZZLE_128B);
@@ -367,8 +369,9 @@ RLB_API int rlb_linear_grouped(const RlbLinear* l, void* stream) {
   g.tile_expert = l->tile_expert;
   g.C = l->out;
   g.ldc = l->ldo;
-  g.glu = l->act == LIN_GLU;
+  g.act = l->act;
   g.limit = l->limit;
+  g.row_scale = l->row_scale;
   return launch_grouped<false, false>(ta, tb, g, l->status, (l->M / BM) * ((l->N + BN - 1) / BN), static_cast<cudaStream_t>(stream));
 }
 

@@ -300,7 +300,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
         if (p.use_layer) acc = layer_epilogue4(p.layer, acc, m, n, layer_alpha);
         if (p.out_fp32) {
           *reinterpret_cast<float4*>(reinterpret_cast<float*>(p.Y) + static_cast<long long>(m) * p.ldy + n) = acc;
-        } else if (p.use_layer && p.layer.lin.act == LIN_GLU) {
+        } else if (p.use_layer && lin_gated(p.layer.lin.act)) {
           *reinterpret_cast<uint32_t*>(reinterpret_cast<__nv_bfloat16*>(p.Y) + static_cast<long long>(m) * p.ldy + n / 2) = pack_bf16x2(acc.x, acc.y);
         } else {
           uint2 o;
@@ -495,8 +495,8 @@ RLB_API int rlb_gemm_skinny_layer(const void* X, const void* W, void* out, int M
 RLB_API int rlb_linear_skinny(const RlbLinear* l, void* stream) {
   if (l->M <= 0 || l->N <= 0 || l->K <= 0) return 0;
   if (l->M > 256) return -7;
-  if ((l->lda % 8) || (l->ldw % 8) || (l->ldo % (l->out_f32 ? 4 : 8)) || (l->N % 8) || (l->K % 8) || l->in_f32 || l->tile_expert) return -2;
-  if (l->out_f32 && l->act == LIN_GLU) return -2;
+  if ((l->lda % 8) || (l->ldw % 8) || (l->ldo % (l->out_f32 ? 4 : 8)) || (l->N % 8) || (l->K % 8) || l->in_f32 || l->tile_expert || l->row_scale) return -2;
+  if (l->out_f32 && lin_gated(l->act)) return -2;
   if ((reinterpret_cast<uintptr_t>(l->a) | reinterpret_cast<uintptr_t>(l->w) | reinterpret_cast<uintptr_t>(l->out) | reinterpret_cast<uintptr_t>(l->bias)) & 15) return -3;
   const int NT = l->M <= 32 ? 32 : (l->M <= 64 ? 64 : (l->M <= 128 ? 128 : 256));
   CUtensorMap tw, tx;

@@ -346,12 +346,12 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
                 v[q * 8 + 4] += b2.x; v[q * 8 + 5] += b2.y; v[q * 8 + 6] += b3.x; v[q * 8 + 7] += b3.y;
               }
           }
-          if (le.act == LIN_GLU) {
+          if (lin_gated(le.act)) {
             __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(ep.C) + static_cast<long long>(row) * ep.ldc + col / 2;
             uint32_t o[8];
 #pragma unroll
             for (int i = 0; i < 8; ++i)
-              o[i] = pack_bf16x2(clamped_glu(v[4 * i], v[4 * i + 1], le.limit), clamped_glu(v[4 * i + 2], v[4 * i + 3], le.limit));
+              o[i] = pack_bf16x2(gated_unit(le.act, v[4 * i], v[4 * i + 1], le.limit), gated_unit(le.act, v[4 * i + 2], v[4 * i + 3], le.limit));
 #pragma unroll
             for (int q = 0; q < 4; ++q)
               if (col + q * 8 < N) *reinterpret_cast<uint2*>(dst + q * 4) = make_uint2(o[2 * q], o[2 * q + 1]);
@@ -649,7 +649,7 @@ RLB_API int rlb_gemm_layer(const void* A, const void* W, void* out, int M, int N
 // out (bf16) = epilogue(a w^T); N, K and the row strides multiples of 8.
 RLB_API int rlb_linear_tiled(const RlbLinear* l, void* stream) {
   if (l->M <= 0 || l->N <= 0 || l->K <= 0) return 0;
-  if ((l->lda % 8) || (l->ldw % 8) || (l->ldo % 8) || (l->N % 8) || (l->K % 8) || l->in_f32 || l->out_f32 || l->tile_expert || l->act == LIN_CAP) return -2;
+  if ((l->lda % 8) || (l->ldw % 8) || (l->ldo % 8) || (l->N % 8) || (l->K % 8) || l->in_f32 || l->out_f32 || l->tile_expert || l->row_scale || l->act == LIN_CAP) return -2;
   if ((reinterpret_cast<uintptr_t>(l->a) | reinterpret_cast<uintptr_t>(l->w) | reinterpret_cast<uintptr_t>(l->out) | reinterpret_cast<uintptr_t>(l->bias)) & 15) return -3;
   if (l->act == LIN_GELU_MUL && (reinterpret_cast<uintptr_t>(l->table) & 7)) return -3;
   CUtensorMap ta, tb;

@@ -8,11 +8,12 @@
 //               64 keys. K and V have one buffer and one pair of barriers each: the next K tile streams in as soon as the QK product
 //               has read the current one, i.e. under the softmax and the PV product, the next V tile under the next QK and softmax
 //   warp 1      tcgen05.mma issuer: S = Q K^T over dim + rot_dim in 16-wide steps, O += P V
-//   warps 2..5  softmax, one thread per query row, stale-maximum rescaling; the epilogue normalises, multiplies by sigmoid(gate) and
-//               writes over the gate columns of the projected rows
+//   warps 2..5  softmax, one thread per query row, stale-maximum rescaling; the epilogue normalises and, where the output columns hold
+//               gates, multiplies by sigmoid(gate)
 // The same kernel serves grouped-query attention (rlb_flash_gqa): no rotated source of its own (the rotation is in the queries and keys), several
 // query heads per key / value head, keys and values read from column ranges of one matrix, no gate, output rows of their own.
-// Query rows stand at the end of their context: row r of a portion of n tokens in a context of c sees keys up to c - n + r.
+// Query rows stand at the end of their context: row r of a portion of n tokens in a context of c sees keys up to c - n + r. With chunks of C
+// positions (the context then begins at a chunk's border) row i sees keys from i - i % C on, and a tile starts where its first row's chunk does.
 #include "common.cuh"
 
 #include <math.h>
@@ -49,13 +50,14 @@ struct FlashLatentParams {
   int vcols;                       // columns of the PV product: vdim rounded up to 16
   int tmem_cols;
   float scale_log2;
-  __nv_bfloat16* p;                // output rows, first column of head 0 (gated: the gates stand there)
+  __nv_bfloat16* p;                // output rows (gated: the gates stand there)
   long long ldp;
   int* status;
   int per_kv;                      // query heads per key / value head
   int k_col, v_col;                // first key / value column of kv head 0
   int ctx_row0;                    // row of the key / value matrix that cu_ctx counts from
   int gated;
+  int chunk;                       // > 0: keys of the row's own chunk only
 };
 
 __global__ void __launch_bounds__(LA_THREADS, 2)
@@ -111,7 +113,8 @@ flash_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
   const int q_row0 = p.row0 + info[0], n_q = info[1], q0 = info[2] * LA_BQ, c_row0 = p.ctx_row0 + info[3], n_ctx = info[4];
   const int q_rows = min(LA_BQ, n_q - q0);
   const int shift = n_ctx - n_q;                                     // query row i of the portion sees keys <= shift + i
-  const int n_kv = (shift + q0 + q_rows + LA_BKV - 1) / LA_BKV;
+  const int first_tile = p.chunk > 0 ? (shift + q0) / p.chunk * p.chunk / LA_BKV : 0;
+  const int n_kv = (shift + q0 + q_rows + LA_BKV - 1) / LA_BKV - first_tile;      // tiles of 64 keys
 
   if (warp == 0) {
     if (lane == 0) {
@@ -124,7 +127,7 @@ flash_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
         tma_load_2d(smem_u32(q_s + a * LA_Q_ATOM), &tmap_q, smem_u32(q_full), a < p.atoms_n ? qx + a * 64 : qx + p.dim + (a - p.atoms_n) * 64, q_row0 + q0);
       for (int j = 0; j < n_kv; ++j) {
         const uint32_t ph = j & 1;
-        const int row = c_row0 + j * LA_BKV;
+        const int row = c_row0 + (first_tile + j) * LA_BKV;
         if (!mbar_wait(smem_u32(k_empty), ph ^ 1, abort_flag, p.status, RLB_ERR_WAIT_EMPTY)) break;
         mbar_arrive_expect_tx(smem_u32(k_full), atoms_q * LA_KV_ATOM);
         for (int a = 0; a < p.atoms_n; ++a) tma_load_2d(smem_u32(k_s + a * LA_KV_ATOM), &tmap_kv, smem_u32(k_full), p.k_col + head / p.per_kv * p.dim + a * 64, row);
@@ -171,6 +174,7 @@ flash_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
     const int quarter = warp & 3, r = quarter * 32 + lane;
     const uint32_t lane_addr = static_cast<uint32_t>(quarter * 32) << 16;
     const int qi = shift + q0 + r;      // last key this row sees
+    const int lo = p.chunk > 0 ? qi - qi % p.chunk : 0, lo_last = p.chunk > 0 ? (shift + q0 + LA_BQ - 1) / p.chunk * p.chunk : 0;      // first key
     float m_ref = -INFINITY, l = 0.f;
     bool ok = true;
     for (int j = 0; j < n_kv; ++j) {
@@ -183,15 +187,15 @@ flash_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
       tmem_ld_32x32b_x32(tmem_s + lane_addr, s0);
       tmem_ld_32x32b_x32(tmem_s + lane_addr + 32, s1);
       tmem_ld_wait();
-      const int k0 = j * LA_BKV;
-      const bool diag = k0 + LA_BKV - 1 > shift + q0;
+      const int k0 = (first_tile + j) * LA_BKV;
+      const bool edge = k0 + LA_BKV - 1 > shift + q0 || k0 < lo_last;
       float mx = -INFINITY;
 #pragma unroll
       for (int i = 0; i < 32; ++i) {
         float a = __uint_as_float(s0[i]) * p.scale_log2, b = __uint_as_float(s1[i]) * p.scale_log2;
-        if (diag) {
-          if (k0 + i > qi) a = -INFINITY;
-          if (k0 + 32 + i > qi) b = -INFINITY;
+        if (edge) {
+          if (k0 + i > qi || k0 + i < lo) a = -INFINITY;
+          if (k0 + 32 + i > qi || k0 + 32 + i < lo) b = -INFINITY;
         }
         s0[i] = __float_as_uint(a);
         s1[i] = __float_as_uint(b);
@@ -248,7 +252,7 @@ flash_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
     if (ok && mbar_wait(smem_u32(v_empty), (n_kv - 1) & 1, abort_flag, p.status, RLB_ERR_WAIT_TMEM_EMPTY)) {
       tc_fence_after();
       const float inv_l = l > 0.f ? 1.f / l : 0.f;
-      __nv_bfloat16* dst = p.p + static_cast<long long>(q_row0 + q0 + r) * p.ldp + p.mix_off + head * p.vdim;      // (gqa: mix_off is 0)
+      __nv_bfloat16* dst = p.p + static_cast<long long>(q_row0 + q0 + r) * p.ldp + p.mix_off + head * p.vdim;
       for (int c = 0; c < p.vdim; c += 32) {
         uint32_t o[32];
         tmem_ld_32x32b_x32(tmem_o + lane_addr + c, o);
@@ -333,16 +337,17 @@ RLB_API int rlb_flash_latent_supported(int dim, int rot_dim, int vdim, int rank)
   return dim > 0 && dim % 16 == 0 && rot_dim % 8 == 0 && vdim % 8 == 0 && rank % 8 == 0 && an + ar <= 4 && av <= 4 && vdim > 0;
 }
 
-// p: projected rows (bf16, row stride ldp); the portions are rows [row0, row0 + cu_q[portions]). kv [ctx_rows, heads * (dim + vdim)]:
-// decompressed keys and values of the gathered context, lat [ctx_rows, width]: its latent rows. max_tiles >= number of 128-row tiles.
-RLB_API int rlb_flash_latent(void* p, long long rows, long long ldp, int in_width, int row0, const void* kv, const void* lat, long long ctx_rows,
+// q [rows, q_width] (bf16, row stride ldq): prepared queries from column q_off; the portions are rows [row0, row0 + cu_q[portions]). kv [ctx_rows,
+// heads * (dim + vdim)]: decompressed keys and values of the gathered context, lat [ctx_rows, width]: its latent rows. out (row stride ldo, may be
+// the rows of q): head outputs from column mix_off, gated by what stands there when `gated`. max_tiles >= number of 128-row tiles.
+RLB_API int rlb_flash_latent(const void* q, long long rows, long long ldq, int q_width, int row0, const void* kv, const void* lat, long long ctx_rows,
                              int width, const int* cu_q, const int* cu_ctx, int portions, int heads, int dim, int rot_dim, int vdim, int rank,
-                             int q_off, int mix_off, float scale, int max_tiles, int* status, void* stream) {
+                             int q_off, void* out, long long ldo, int mix_off, int gated, float scale, int max_tiles, int* status, void* stream) {
   if (portions <= 0 || rows <= 0 || max_tiles <= 0) return 0;
   if (!rlb_flash_latent_supported(dim, rot_dim, vdim, rank)) return -2;
-  if (ldp % 8 || width % 8 || q_off % 8 || mix_off % 8 || (dim + rot_dim) % 8 || heads > 65535) return -2;
-  if ((reinterpret_cast<uintptr_t>(p) | reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(lat)) & 15) return -3;
-  FlashLatentParams f;
+  if (ldq % 8 || ldo % 8 || width % 8 || q_off % 8 || mix_off % 8 || (dim + rot_dim) % 8 || heads > 65535) return -2;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(lat)) & 15) return -3;
+  FlashLatentParams f{};
   f.cu_q = cu_q;
   f.cu_ctx = cu_ctx;
   f.portions = portions;
@@ -360,17 +365,17 @@ RLB_API int rlb_flash_latent(void* p, long long rows, long long ldp, int in_widt
   f.vcols = (vdim + 15) / 16 * 16;
   f.tmem_cols = 64 + (vdim + 31) / 32 * 32 <= 128 ? 128 : (64 + (vdim + 31) / 32 * 32 <= 256 ? 256 : 512);
   f.scale_log2 = scale * LA_LOG2E;
-  f.p = static_cast<__nv_bfloat16*>(p);
-  f.ldp = ldp;
+  f.p = static_cast<__nv_bfloat16*>(out);
+  f.ldp = ldo;
   f.status = status;
   f.per_kv = 1;
   f.k_col = 0;
   f.v_col = heads * dim;
   f.ctx_row0 = 0;
-  f.gated = 1;
+  f.gated = gated;
   const long long kvw = static_cast<long long>(heads) * (dim + vdim);
   CUtensorMap tq, tkv, tl;
-  int rc = rlb_make_tmap_2d(&tq, p, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, in_width, rows, ldp * 2, 64, LA_BQ, CU_TENSOR_MAP_SWIZZLE_128B);
+  int rc = rlb_make_tmap_2d(&tq, q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, q_width, rows, ldq * 2, 64, LA_BQ, CU_TENSOR_MAP_SWIZZLE_128B);
   if (rc) return -100 - rc;
   rc = rlb_make_tmap_2d(&tkv, kv, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, kvw, ctx_rows, kvw * 2, 64, LA_BKV, CU_TENSOR_MAP_SWIZZLE_128B);
   if (rc) return -100 - rc;
@@ -382,10 +387,11 @@ RLB_API int rlb_flash_latent(void* p, long long rows, long long ldp, int in_widt
 
 // Grouped-query attention of prompt portions. p: projected rows with normed and rotated queries at q_off; the portions are its rows
 // [row0, row0 + cu_q[portions]). Keys of kv head g: columns [k_col + g * dim, + dim) of kv [kv_rows, kv_width], values [v_col + g * vdim, + vdim);
-// row ctx_row0 + cu_ctx[i] is the first of portion i's context (kv may be p itself). y [rows, heads * vdim]: outputs. dim a multiple of 16, vdim of 8.
+// row ctx_row0 + cu_ctx[i] is the first of portion i's context (kv may be p itself), with chunk > 0 the first of a chunk. y [rows, heads * vdim]:
+// outputs. dim a multiple of 16, vdim of 8.
 RLB_API int rlb_flash_gqa(void* p, long long rows, long long ldp, int in_width, int row0, const void* kv, long long kv_rows, long long ldkv, int kv_width,
                           int ctx_row0, int k_col, int v_col, const int* cu_q, const int* cu_ctx, int portions, int heads, int kv_heads, int dim, int vdim,
-                          int q_off, float scale, int max_tiles, void* y, long long ldy, int* status, void* stream) {
+                          int q_off, int chunk, float scale, int max_tiles, void* y, long long ldy, int* status, void* stream) {
   if (portions <= 0 || rows <= 0 || max_tiles <= 0) return 0;
   if (!rlb_flash_latent_supported(dim, 0, vdim, 8) || kv_heads < 1 || heads % kv_heads) return -2;
   if (ldp % 8 || ldkv % 8 || ldy % 8 || q_off % 8 || k_col % 8 || v_col % 8 || heads > 65535) return -2;
@@ -411,6 +417,7 @@ RLB_API int rlb_flash_gqa(void* p, long long rows, long long ldp, int in_width, 
   f.k_col = k_col;
   f.v_col = v_col;
   f.ctx_row0 = ctx_row0;
+  f.chunk = chunk;
   CUtensorMap tq, tkv;
   int rc = rlb_make_tmap_2d(&tq, p, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, in_width, rows, ldp * 2, 64, LA_BQ, CU_TENSOR_MAP_SWIZZLE_128B);
   if (rc) return -100 - rc;

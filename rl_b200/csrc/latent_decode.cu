@@ -5,7 +5,7 @@
 //   attention    one CTA per (row, group of HN heads, split of the context): a tile of 64 latent rows is both K and V and is fetched once,
 //                by TMA, into a ring of 64-column chunks
 //   combine      joins the splits
-//   heads GEMM   y[t, h, :] = o[t, h, :] W_uv[h]^T * sigmoid(gate) (tcgen05), written over the gate columns of the projected rows
+//   heads GEMM   y[t, h, :] = o[t, h, :] W_uv[h]^T (tcgen05), times sigmoid(gate) where the output columns hold gates
 //
 // The attention products have 16 or 32 rows (heads) only. A tcgen05.mma with 128 latent rows on the M side and 16 heads on the N side
 // occupies its pipe for about 120 cycles (measured: the issuing thread is held that long per instruction, although the tensor pipe is
@@ -509,15 +509,16 @@ RLB_API int rlb_latent_decode_supported(int dim, int rot_dim, int vdim, int rank
 }
 
 // q_lat [rows, heads, width] (bf16): columns [rank, width) hold the rotated query part (zero padded) already; columns [0, rank) are
-// computed here. o_lat [rows, heads * rank] is scratch. part_o / part_ml: scratch for num_splits > 1. Only rows [0, rows) of p.
-RLB_API int rlb_latent_decode(void* p, int rows, long long ldp, int in_width, int q_off, int mix_off, int heads, int dim, int rot_dim, int vdim,
+// computed here from the queries q [rows, q_width]. o_lat [rows, heads * rank] is scratch. part_o / part_ml: scratch for num_splits > 1. out (may
+// be the rows of q): head outputs from column mix_off, gated by what stands there when `gated`.
+RLB_API int rlb_latent_decode(const void* q, int rows, long long ldq, int q_width, int q_off, void* out, long long ldo, int mix_off, int gated, int heads, int dim, int rot_dim, int vdim,
                               int rank, int width, int block_size, int num_blocks, const void* cache, const int* block_table, int bt_stride,
                               const int* seq_lens, const void* kv_up, float scale, void* q_lat, void* o_lat, int num_splits, float* part_o,
                               float* part_ml, int* status, void* stream) {
   if (rows <= 0) return 0;
   if (!rlb_latent_decode_supported(dim, rot_dim, vdim, rank, width, block_size) || heads > 65535 || num_splits < 1 || num_splits > 32) return -2;
-  if (ldp % 8 || q_off % 8 || mix_off % 8 || (dim + rot_dim) % 8 || (num_splits > 1 && (!part_o || !part_ml))) return -2;
-  if ((reinterpret_cast<uintptr_t>(p) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(kv_up) | reinterpret_cast<uintptr_t>(q_lat) |
+  if (ldq % 8 || ldo % 8 || q_off % 8 || mix_off % 8 || (dim + rot_dim) % 8 || (num_splits > 1 && (!part_o || !part_ml))) return -2;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(kv_up) | reinterpret_cast<uintptr_t>(q_lat) |
        reinterpret_cast<uintptr_t>(o_lat)) & 15)
     return -3;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
@@ -531,7 +532,7 @@ RLB_API int rlb_latent_decode(void* p, int rows, long long ldp, int in_width, in
   const auto BF = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   const auto SW = CU_TENSOR_MAP_SWIZZLE_128B;
   CUtensorMap ta, tb, tl;
-  int rc = rlb_make_tmap_2d(&ta, p, BF, 2, in_width, rows, ldp * 2, HG_K, HG_T, SW);
+  int rc = rlb_make_tmap_2d(&ta, q, BF, 2, q_width, rows, ldq * 2, HG_K, HG_T, SW);
   if (!rc) rc = rlb_make_tmap_2d(&tb, kv_up, BF, 2, rank, static_cast<uint64_t>(heads) * (dim + vdim), static_cast<uint64_t>(rank) * 2, 64, HG_K, SW);
   if (rc) return -100 - rc;
   HeadsGemm g{rows, rank, dim, q_off, dim + rot_dim, 0, dim, static_cast<__nv_bfloat16*>(q_lat), static_cast<long long>(heads) * width, 0, width, 0, status};
@@ -568,7 +569,7 @@ RLB_API int rlb_latent_decode(void* p, int rows, long long ldp, int in_width, in
   rc = rlb_make_tmap_2d(&ta, o_lat, BF, 2, static_cast<uint64_t>(heads) * rank, rows, static_cast<uint64_t>(heads) * rank * 2, HG_K, HG_T, SW);
   if (!rc) rc = rlb_make_tmap_2d(&tb, kv_up, BF, 2, rank, static_cast<uint64_t>(heads) * (dim + vdim), static_cast<uint64_t>(rank) * 2, HG_K, 32, SW);
   if (rc) return -100 - rc;
-  HeadsGemm u{rows, vdim, rank, 0, rank, heads * dim, vdim, static_cast<__nv_bfloat16*>(p), ldp, mix_off, vdim, 1, status};
+  HeadsGemm u{rows, vdim, rank, 0, rank, heads * dim, vdim, static_cast<__nv_bfloat16*>(out), ldo, mix_off, vdim, gated, status};
   e = rlb_launch_pdl(gemm_heads_kernel<false, 32, 8>, dim3((vdim + 31) / 32, (rows + HG_T - 1) / HG_T, heads), dim3(HG_THREADS), HgCfg<32, 8>::SMEM, s, ta, tb, u);
   return static_cast<int>(e);
 }

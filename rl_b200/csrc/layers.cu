@@ -1,9 +1,9 @@
-// Row kernels of post-norm layers (models/post_norm.py), for every size and for bf16 and fp32 models: the step that norms a sublayer's
+// Row kernels of post-norm and pre-norm layers (models/post_norm.py, models/pre_norm.py), for every size and for bf16 and fp32 models: the step that norms a sublayer's
 // output and joins it to the residual stream, the sigmoid router with group-limited choice, the placement of the tokens' copies in
 // per-expert row ranges, and the soft cap of the logits.
 //
-//   add_normed   x += m * rms(y) * w on the fp32 stream, and what the next sublayer reads: x itself in the model's type, or its RMS norm
-//                behind the last layer. y is a product's output or the weighted sum of a token's expert rows (combined here, never stored).
+//   add_normed   x += m * rms(y) * w (post-norm layers) or x += y (pre-norm layers) on the fp32 stream, and what the next sublayer reads: x
+//                itself in the model's type, or its RMS norm. y is a product's output or the weighted sum of a token's expert rows (combined here, never stored).
 //   moe_choose   one warp per token: scores, group choice, top-k; every copy takes a number among its expert's copies.
 //   moe_place    row ranges of the experts (multiples of 128 rows) from their counts, the row of every copy, and its token's row moved there.
 //
@@ -41,15 +41,17 @@ struct AddNormed {
   const void* y;           // [rows, ldy], or the experts' rows when copy_row is set
   long long ldy;
   const int* copy_row;     // [rows, k] row of each of a token's copies in y (out of [0, y_rows): skipped)
-  const float* weight;     // [rows, k]
+  const float* weight;     // [rows, k] (null: 1)
   int k, y_rows;
   int* counts;             // the experts' counts [experts], set to zero for the next layer
   int experts;
-  const void* w;           // norm weight of the sublayer
-  const void* next_w;      // weight of the norm behind the last layer (null: h is x)
+  const void* w;           // norm weight of the sublayer (null: its output joins as it is)
+  const void* next_w;      // weight of the next norm (null: h is x)
   void* h;                 // [rows, d]
   int d;
   float mult, eps;
+  const void* also;        // [rows, ld_also] or null: added to the sublayer's output
+  long long ld_also;
 };
 
 // AN_KEEP: groups of four columns that a thread keeps in registers
@@ -63,7 +65,7 @@ __global__ void __launch_bounds__(THREADS) add_normed_kernel(AddNormed a) {
   const T* Y = static_cast<const T*>(a.y);
   float* x = a.x + row * a.d;
   T* h = static_cast<T*>(a.h) + row * a.d;
-  const T *w = static_cast<const T*>(a.w), *nw = static_cast<const T*>(a.next_w);
+  const T *w = static_cast<const T*>(a.w), *nw = static_cast<const T*>(a.next_w), *also = static_cast<const T*>(a.also);
   if (a.d % 4 == 0 && a.d <= AN_KEEP * 4 * THREADS) {
     float4 v[AN_KEEP], xv[AN_KEEP];
     float ss = 0.f;
@@ -74,6 +76,10 @@ __global__ void __launch_bounds__(THREADS) add_normed_kernel(AddNormed a) {
       if (c >= a.d) continue;
       xv[i] = ld4(x + c);
       if (!a.copy_row) v[i] = ld4(Y + row * a.ldy + c);
+      if (also) {
+        const float4 t = ld4(also + row * a.ld_also + c);
+        v[i].x += t.x; v[i].y += t.y; v[i].z += t.z; v[i].w += t.w;
+      }
     }
     if (a.copy_row) {
       constexpr int AHEAD = AN_KEEP <= 2 ? 4 : 2;      // copies in flight
@@ -84,7 +90,7 @@ __global__ void __launch_bounds__(THREADS) add_normed_kernel(AddNormed a) {
         for (int j = 0; j < AHEAD; ++j) {
           const int r = j0 + j < a.k ? a.copy_row[row * a.k + j0 + j] : -1;
           const bool live = r >= 0 && r < a.y_rows;
-          wt[j] = live ? a.weight[row * a.k + j0 + j] : 0.f;
+          wt[j] = live ? (a.weight ? a.weight[row * a.k + j0 + j] : 1.f) : 0.f;
 #pragma unroll
           for (int i = 0; i < AN_KEEP; ++i) {
             const int c = (threadIdx.x + i * THREADS) * 4;
@@ -102,16 +108,19 @@ __global__ void __launch_bounds__(THREADS) add_normed_kernel(AddNormed a) {
           }
       }
     }
+    float f = a.mult;
+    if (w) {
 #pragma unroll
-    for (int i = 0; i < AN_KEEP; ++i) ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
-    ss = block_sum(ss, red);
-    const float f = a.mult / sqrtf(ss / static_cast<float>(a.d) + a.eps);
+      for (int i = 0; i < AN_KEEP; ++i) ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+      ss = block_sum(ss, red);
+      f = a.mult / sqrtf(ss / static_cast<float>(a.d) + a.eps);
+    }
     float s2 = 0.f;
 #pragma unroll
     for (int i = 0; i < AN_KEEP; ++i) {
       const int c = (threadIdx.x + i * THREADS) * 4;
       if (c >= a.d) continue;
-      const float4 wv = ld4(w + c);
+      const float4 wv = w ? ld4(w + c) : make_float4(1.f, 1.f, 1.f, 1.f);
       xv[i].x = fmaf(v[i].x * f, wv.x, xv[i].x);
       xv[i].y = fmaf(v[i].y * f, wv.y, xv[i].y);
       xv[i].z = fmaf(v[i].z * f, wv.z, xv[i].z);
@@ -134,23 +143,26 @@ __global__ void __launch_bounds__(THREADS) add_normed_kernel(AddNormed a) {
     return;
   }
   auto value = [&](int c) {
-    if (!a.copy_row) return ldv(Y + row * a.ldy + c);
-    float v = 0.f;
+    float v = also ? ldv(also + row * a.ld_also + c) : 0.f;
+    if (!a.copy_row) return v + ldv(Y + row * a.ldy + c);
     for (int j = 0; j < a.k; ++j) {
       const int r = a.copy_row[row * a.k + j];
-      if (r >= 0 && r < a.y_rows) v = fmaf(a.weight[row * a.k + j], ldv(Y + r * a.ldy + c), v);
+      if (r >= 0 && r < a.y_rows) v = fmaf(a.weight ? a.weight[row * a.k + j] : 1.f, ldv(Y + r * a.ldy + c), v);
     }
     return v;
   };
   float ss = 0.f, s2 = 0.f;
-  for (int c = threadIdx.x; c < a.d; c += THREADS) {
-    const float v = value(c);
-    ss += v * v;
+  float f = a.mult;
+  if (w) {
+    for (int c = threadIdx.x; c < a.d; c += THREADS) {
+      const float v = value(c);
+      ss += v * v;
+    }
+    ss = block_sum(ss, red);
+    f = a.mult / sqrtf(ss / static_cast<float>(a.d) + a.eps);
   }
-  ss = block_sum(ss, red);
-  const float f = a.mult / sqrtf(ss / static_cast<float>(a.d) + a.eps);
   for (int c = threadIdx.x; c < a.d; c += THREADS) {
-    const float v = fmaf(value(c) * f, ldv(w + c), x[c]);
+    const float v = fmaf(value(c) * f, w ? ldv(w + c) : 1.f, x[c]);
     x[c] = v;
     if (!nw) st1(h + c, v);
     s2 += v * v;
@@ -279,7 +291,7 @@ moe_choose_kernel(const float* __restrict__ logits, long long ld, int T, int E, 
   for (int e = lane; e < E; e += 32) {
     const float v = 1.f / (1.f + expf(-logits[static_cast<long long>(t) * ld + e]));
     s[e] = v;
-    c[e] = v + correction[e];
+    c[e] = correction ? v + correction[e] : v;
   }
   __syncwarp();
   if (groups > 1) {
@@ -348,7 +360,8 @@ constexpr int MP_MAX_E = 1024;
 __global__ void __launch_bounds__(256)
 moe_place_kernel(const int* __restrict__ idx, const int* __restrict__ rank, long long copies, int k, const int* __restrict__ counts, int E, int mpad,
                  int* __restrict__ copy_row, int* __restrict__ tile_expert, int* __restrict__ a_rows,
-                 const uint4* __restrict__ x, long long x_vecs, uint4* __restrict__ x_out, int vecs, int* status) {
+                 const uint4* __restrict__ x, long long x_vecs, uint4* __restrict__ x_out, int vecs, const float* __restrict__ weight,
+                 float* __restrict__ row_weight, int* status) {
   __shared__ int row0[MP_MAX_E + 1];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   pdl_sync();
@@ -385,6 +398,7 @@ moe_place_kernel(const int* __restrict__ idx, const int* __restrict__ rank, long
     if (lane == 0) {
       copy_row[c] = row;
       if (a_rows && row >= 0) a_rows[row] = static_cast<int>(c / k);
+      if (row_weight && row >= 0) row_weight[row] = weight[c];
     }
     if (x_out && row >= 0) {
       const uint4* src = x + (c / k) * x_vecs;
@@ -395,13 +409,13 @@ moe_place_kernel(const int* __restrict__ idx, const int* __restrict__ rank, long
 }
 }  // namespace
 
-// x [rows, d] fp32 += mult * rms(y) * w; h [rows, d] = x, or rms(x) * next_w. With copy_row [rows, k]: y of a row is the sum of its k
-// weighted rows of y [y_rows, ldy], and counts [experts] are set to zero.
+// x [rows, d] fp32 += mult * rms(y) * w (w null: mult * y); h [rows, d] = x, or rms(x) * next_w. With copy_row [rows, k]: y of a row is the
+// sum of its k weighted (weight null: plain) rows of y [y_rows, ldy], and counts [experts] are set to zero. also [rows, ld_also]: added to y.
 RLB_API int rlb_add_normed(float* x, const void* y, long long ldy, int f32, const int* copy_row, const float* weight, int k, int y_rows, int* counts, int experts,
-                           const void* w, const void* next_w, void* h, long long rows, int d, float mult, float eps, void* stream) {
+                           const void* also, long long ld_also, const void* w, const void* next_w, void* h, long long rows, int d, float mult, float eps, void* stream) {
   if (rows <= 0) return 0;
-  if (d % 4 == 0 && ldy % 4) return -2;
-  AddNormed a{x, y, ldy, copy_row, weight, k, y_rows, counts, experts, w, next_w, h, d, mult, eps};
+  if (d % 4 == 0 && (ldy % 4 || (also && ld_also % 4))) return -2;
+  AddNormed a{x, y, ldy, copy_row, weight, k, y_rows, counts, experts, w, next_w, h, d, mult, eps, also, ld_also};
   const dim3 grid(static_cast<unsigned>(rows));
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (f32) return static_cast<int>(rlb_launch_pdl(add_normed_kernel<float, 256, 8>, grid, dim3(256), 0, s, a));
@@ -438,7 +452,7 @@ RLB_API int rlb_cap_rows(float* z, long long n, float scale, float cap, void* st
   return static_cast<int>(cudaGetLastError());
 }
 
-// Scores sigmoid(logits [T, E]), choice by score + correction among the `keep` best of `groups` groups. counts [E] (zero before the call)
+// Scores sigmoid(logits [T, E]), choice by score + correction (null: none) among the `keep` best of `groups` groups. counts [E] (zero before the call)
 // receives the experts' copies, out_rank each copy's number among them.
 RLB_API int rlb_moe_choose(const float* logits, long long ld, int T, int E, const float* correction, int groups, int keep, int k, float* out_w,
                            int* out_idx, int* out_rank, int* counts, void* stream) {
@@ -450,14 +464,15 @@ RLB_API int rlb_moe_choose(const float* logits, long long ld, int T, int E, cons
 }
 
 // mpad: a multiple of 128, at least copies + E * 127. a_rows (with x_out null) must hold -1 everywhere before the call. row_bytes and the
-// row stride of x: multiples of 16 (only with x_out).
+// row stride of x: multiples of 16 (only with x_out). row_weight [mpad] (or null): each copy's weight [copies] at its row.
 RLB_API int rlb_moe_place(const int* idx, const int* rank, long long copies, int k, const int* counts, int E, int mpad, int* copy_row,
-                          int* tile_expert, int* a_rows, const void* x, long long x_stride_bytes, void* x_out, int row_bytes, int* status, void* stream) {
+                          int* tile_expert, int* a_rows, const void* x, long long x_stride_bytes, void* x_out, int row_bytes, const float* weight,
+                          float* row_weight, int* status, void* stream) {
   if (copies <= 0) return 0;
   if (E < 1 || E > MP_MAX_E || mpad % 128 || mpad < copies + static_cast<long long>(E) * 127) return -2;
   if (x_out && ((row_bytes % 16) || (x_stride_bytes % 16) || ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(x_out)) & 15))) return -3;
   const long long want = (copies + 7) / 8;
   return static_cast<int>(rlb_launch_pdl(moe_place_kernel, dim3(static_cast<unsigned>(want < 148 * 4 ? want : 148 * 4)), dim3(256), 0,
                                          static_cast<cudaStream_t>(stream), idx, rank, copies, k, counts, E, mpad, copy_row, tile_expert, a_rows,
-                                         static_cast<const uint4*>(x), x_stride_bytes / 16, static_cast<uint4*>(x_out), row_bytes / 16, status));
+                                         static_cast<const uint4*>(x), x_stride_bytes / 16, static_cast<uint4*>(x_out), row_bytes / 16, weight, row_weight, status));
 }

@@ -33,11 +33,12 @@ __device__ __forceinline__ void st<__nv_bfloat16>(__nv_bfloat16* p, float v) {
 }
 
 // ---------------------------------------------------------------- start of the residual stream
-// x = table[id] * scale (kept in e), + step; h = w * tanh(alpha x) + b, or x itself where there is no norm (alpha null)
+// x = table[id] * scale (kept in e), + step; h = w * tanh(alpha x) + b, or x / rms(x) * w (alpha null), or x itself (no norm)
 template <typename T>
 __global__ void embed_rows_kernel(const void* ids, int ids64, const T* __restrict__ table, float* __restrict__ x, float* __restrict__ e,
                                   T* __restrict__ h, const T* __restrict__ step, const T* __restrict__ alpha, const T* __restrict__ nw,
-                                  const T* __restrict__ nb, int d, int vocab, float scale, int* status) {
+                                  const T* __restrict__ nb, int d, int vocab, float scale, float eps, int* status) {
+  __shared__ float red[32];
   const long long row = blockIdx.x;
   long long id = ids64 ? static_cast<const long long*>(ids)[row] : static_cast<const int*>(ids)[row];
   if (id < 0 || id >= vocab) {
@@ -45,13 +46,19 @@ __global__ void embed_rows_kernel(const void* ids, int ids64, const T* __restric
     id = 0;
   }
   const float a = alpha ? ld(alpha) : 0.f;
+  float ss = 0.f;
   for (int c = threadIdx.x; c < d; c += blockDim.x) {
     float v = ld(table + id * d + c) * scale;
     if (e) e[row * d + c] = v;
     if (step) v += ld(step + c);
     x[row * d + c] = v;
-    st(h + row * d + c, alpha ? tanhf(a * v) * ld(nw + c) + ld(nb + c) : v);
+    ss += v * v;
+    if (alpha || !nw) st(h + row * d + c, alpha ? tanhf(a * v) * ld(nw + c) + ld(nb + c) : v);
   }
+  if (alpha || !nw) return;
+  ss = block_sum(ss, red);
+  const float rstd = 1.f / sqrtf(ss / static_cast<float>(d) + eps);
+  for (int c = threadIdx.x; c < d; c += blockDim.x) st(h + row * d + c, x[row * d + c] * rstd * ld(nw + c));     // (each thread reads what it wrote)
 }
 
 // ---------------------------------------------------------------- product with the layer epilogues
@@ -127,17 +134,22 @@ __global__ void __launch_bounds__(256) gemm_rows_kernel(RowsGemm g) {
   for (int i = 0; i < 4; ++i) {
     const int m = m0 + ty * 4 + i;
     if (m >= g.M) continue;
+    if (g.lin.row_scale) {
+      const float f = g.lin.row_scale[m];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[i][j] *= f;
+    }
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
       if (n >= g.N) continue;
       float v = acc[i][j];
       if (g.lin.bias) v += ld(static_cast<const TI*>(g.lin.bias) + n);
-      if (g.lin.act == LIN_GLU) {          // N is even: the pair of an even column is there
+      if (lin_gated(g.lin.act)) {          // N is even: the pair of an even column is there
         if (j & 1) continue;
         float u = acc[i][j + 1];
         if (g.lin.bias) u += ld(static_cast<const TI*>(g.lin.bias) + n + 1);
-        st(static_cast<TO*>(g.out) + static_cast<long long>(m) * g.ldo + n / 2, clamped_glu(v, u, g.lin.limit));
+        st(static_cast<TO*>(g.out) + static_cast<long long>(m) * g.ldo + n / 2, gated_unit(g.lin.act, v, u, g.lin.limit));
         continue;
       }
       if (g.lin.act == LIN_GELU_MUL) {
@@ -166,11 +178,13 @@ __global__ void __launch_bounds__(256) gemm_rows_kernel(RowsGemm g) {
 
 // ---------------------------------------------------------------- latent attention
 struct LatentShape {
-  long long ldp;                       // row stride of the projected rows
-  int q_off, lat_off, mix_off;         // columns of queries, latent and gate
+  long long ldp, ldq, ldo;             // row strides of the rows with the latent, of the queries, of the output
+  int q_off, lat_off, mix_off;         // columns of queries, latent and output
   int heads, dim, rot_dim, vdim, rank; // per head: dim unrotated + rot_dim rotated query / key dimensions
   int width;                           // row width of the latent cache
   int block_size, num_blocks;
+  int halves;                          // rotated pairs are (i, i + half) instead of (2i, 2i + 1)
+  int gated;                           // the output columns hold gates: out = y * sigmoid(gate)
 };
 
 // Two CTAs per row. blockIdx.y 0: latent / rms * w and the rotated shared key into the cache row of the token. blockIdx.y 1: the
@@ -180,21 +194,46 @@ struct LatentShape {
 constexpr int LP_KEEP = 8;     // latent columns a thread keeps in registers
 template <typename T>
 __global__ void __launch_bounds__(128)
-latent_prep_kernel(T* __restrict__ p, LatentShape s, const int* __restrict__ positions, const long long* __restrict__ slots,
+latent_prep_kernel(const T* __restrict__ p, T* __restrict__ queries, LatentShape s, const int* __restrict__ positions, const long long* __restrict__ slots,
                    const T* __restrict__ norm_w, const float* __restrict__ freq, int half, float gain, float eps,
                    T* __restrict__ cache, T* __restrict__ q_lat, int q_rows, int* status) {
   __shared__ float red[32];
   const int tid = threadIdx.x;
   pdl_sync();
   const long long row = blockIdx.x;
-  T* pr = p + row * s.ldp;
   const float pos = static_cast<float>(positions[row]);
   if (blockIdx.y == 1) {
     const int tail = s.width - s.rank, pairs = (tail + 1) / 2, qd = s.dim + s.rot_dim;
     const bool decode = q_lat && row < q_rows;
+    T* qr = queries + row * s.ldq + s.q_off + s.dim;
+    if (s.halves) {      // a thread turns pairs (f, f + half), or passes on a column behind the rotated ones
+      const int units = tail - half;
+      for (int i = tid; i < s.heads * units; i += 128) {
+        const int h = i / units, f = i % units;
+        T* q = qr + h * qd;
+        T* o = q_lat + (row * s.heads + h) * s.width + s.rank;
+        if (f >= half) {
+          if (decode) st(o + f + half, f + half < s.rot_dim ? ld(q + f + half) : 0.f);
+          continue;
+        }
+        const float u = ld(q + f), v = ld(q + f + half);
+        float sn, c;
+        sincosf(pos * freq[f], &sn, &c);
+        c *= gain;
+        sn *= gain;
+        const float a = u * c - v * sn, b = v * c + u * sn;
+        st(q + f, a);
+        st(q + f + half, b);
+        if (decode) {
+          st(o + f, a);
+          st(o + f + half, b);
+        }
+      }
+      return;
+    }
     for (int i = tid; i < s.heads * pairs; i += 128) {
       const int h = i / pairs, f = i % pairs, j = 2 * f;
-      T* q = pr + s.q_off + h * qd + s.dim + j;
+      T* q = qr + h * qd + j;
       float u = j < s.rot_dim ? ld(q) : 0.f, v = j + 1 < s.rot_dim ? ld(q + 1) : 0.f;
       if (f < half) {
         float sn, c;
@@ -216,7 +255,7 @@ latent_prep_kernel(T* __restrict__ p, LatentShape s, const int* __restrict__ pos
     return;
   }
   const long long slot = slots[row];
-  const T* lat = pr + s.lat_off;
+  const T* lat = p + row * s.ldp + s.lat_off;
   float keep[LP_KEEP];
   float ss = 0.f;
 #pragma unroll
@@ -237,10 +276,11 @@ latent_prep_kernel(T* __restrict__ p, LatentShape s, const int* __restrict__ pos
     for (int j = tid; j < s.width - s.rank; j += 128) {      // rotated key part, then padding
       float v = j < s.rot_dim ? ld(lat + s.rank + j) : 0.f;
       if (j < 2 * half) {
+        const bool second = s.halves ? j >= half : (j & 1);
         float sn, c;
-        sincosf(pos * freq[j >> 1], &sn, &c);
-        const float o = ld(lat + s.rank + (j ^ 1));
-        v = ((j & 1) ? v * c + o * sn : v * c - o * sn) * gain;
+        sincosf(pos * freq[s.halves ? j - (second ? half : 0) : j >> 1], &sn, &c);
+        const float o = ld(lat + s.rank + (s.halves ? (second ? j - half : j + half) : (j ^ 1)));
+        v = (second ? v * c + o * sn : v * c - o * sn) * gain;
       }
       st(cr + s.rank + j, v);
     }
@@ -257,11 +297,11 @@ latent_prep_kernel(T* __restrict__ p, LatentShape s, const int* __restrict__ pos
 }
 
 // One CTA per (row, head): the query is carried into the latent space (q^T W_uk), the keys are the cached rows, the weighted
-// latent is carried to the values (W_uv) and gated. Everything in fp32.
+// latent is carried to the values (W_uv), and gated where the output columns hold gates. Everything in fp32.
 constexpr int LR_TILE = 128;
 template <typename T>
 __global__ void __launch_bounds__(128)
-latent_rows_kernel(T* __restrict__ p, LatentShape s, const T* __restrict__ cache, const int* __restrict__ block_table, int bt_stride,
+latent_rows_kernel(const T* queries, T* out, LatentShape s, const T* __restrict__ cache, const int* __restrict__ block_table, int bt_stride,
                    const int* __restrict__ seq_lens, const T* __restrict__ kv_up, float scale, int* status) {
   extern __shared__ float sm[];
   __shared__ float red[32];
@@ -270,8 +310,7 @@ latent_rows_kernel(T* __restrict__ p, LatentShape s, const T* __restrict__ cache
   float* sc = o + s.rank;               // [LR_TILE]
   long long* rows = reinterpret_cast<long long*>(sm + ((s.width + s.rank + LR_TILE + 1) & ~1));   // [LR_TILE]
   const int row = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  T* pr = p + row * s.ldp;
-  const T* q = pr + s.q_off + h * (s.dim + s.rot_dim);
+  const T* q = queries + row * s.ldq + s.q_off + h * (s.dim + s.rot_dim);
   for (int r = tid; r < s.width; r += 128) {
     float v = 0.f;
     if (r < s.rank) {
@@ -327,8 +366,8 @@ latent_rows_kernel(T* __restrict__ p, LatentShape s, const T* __restrict__ cache
     for (int r = lane; r < s.rank; r += 32) y = fmaf(o[r], ld(w + r), y);
     y = warp_sum(y) * inv;
     if (lane == 0) {
-      T* g = pr + s.mix_off + h * s.vdim + v;
-      st(g, y / (1.f + expf(-ld(g))));
+      T* g = out + row * s.ldo + s.mix_off + h * s.vdim + v;
+      st(g, s.gated ? y / (1.f + expf(-ld(g))) : y);
     }
   }
 }
@@ -437,17 +476,17 @@ int smem_attr(const void* kernel, size_t bytes) {
 }  // namespace
 
 RLB_API int rlb_embed_rows(const void* ids, int ids64, const void* table, int f32, float* x, float* e, void* h, const void* step,
-                           const void* alpha, const void* nw, const void* nb, long long rows, int d, int vocab, float scale, int* status,
+                           const void* alpha, const void* nw, const void* nb, long long rows, int d, int vocab, float scale, float eps, int* status,
                            void* stream) {
   if (rows <= 0) return 0;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (f32)
     embed_rows_kernel<float><<<static_cast<unsigned>(rows), 256, 0, s>>>(ids, ids64, static_cast<const float*>(table), x, e, static_cast<float*>(h),
-        static_cast<const float*>(step), static_cast<const float*>(alpha), static_cast<const float*>(nw), static_cast<const float*>(nb), d, vocab, scale, status);
+        static_cast<const float*>(step), static_cast<const float*>(alpha), static_cast<const float*>(nw), static_cast<const float*>(nb), d, vocab, scale, eps, status);
   else
     embed_rows_kernel<__nv_bfloat16><<<static_cast<unsigned>(rows), 256, 0, s>>>(ids, ids64, static_cast<const __nv_bfloat16*>(table), x, e,
         static_cast<__nv_bfloat16*>(h), static_cast<const __nv_bfloat16*>(step), static_cast<const __nv_bfloat16*>(alpha),
-        static_cast<const __nv_bfloat16*>(nw), static_cast<const __nv_bfloat16*>(nb), d, vocab, scale, status);
+        static_cast<const __nv_bfloat16*>(nw), static_cast<const __nv_bfloat16*>(nb), d, vocab, scale, eps, status);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -465,47 +504,51 @@ RLB_API int rlb_gemm_rows(const void* a, const void* w, void* out, int M, int N,
 // The product of RlbLinear for any sizes, bf16 or fp32, one weight or one per expert.
 RLB_API int rlb_linear_rows(const RlbLinear* l, void* stream) {
   if (l->M <= 0 || l->N <= 0 || l->K <= 0) return 0;
-  if ((l->act == LIN_GLU && l->N % 2) || (l->tile_expert && l->M % 128)) return -2;
+  if ((lin_gated(l->act) && l->N % 2) || (l->tile_expert && l->M % 128)) return -2;
   RowsGemm g{l->a, l->w, l->out, l->M, l->N, l->K, l->lda, l->ldw, l->ldo, 1 << 30, nullptr, 0, nullptr, nullptr, nullptr, nullptr, nullptr,
              rlb_linear_epi(*l), l->tile_expert, l->a_rows, l->num_a_rows};
   return launch_rows(g, l->in_f32, l->out_f32, static_cast<cudaStream_t>(stream));
 }
 
-RLB_API int rlb_latent_prep(void* p, int f32, long long rows, long long ldp, int q_off, int lat_off, int heads, int dim, int rot_dim, int rank,
-                            int width, int block_size, int num_blocks, const int* positions, const long long* slots, const void* norm_w,
-                            const float* freq, int half, float gain, float eps, void* cache, void* q_lat, int q_rows, int* status, void* stream) {
+// p: rows with the latent (lat_off) and the shared key part behind it; q: rows with the queries (may be p). halves: rotated pairs are
+// (i, i + half) instead of (2i, 2i + 1).
+RLB_API int rlb_latent_prep(const void* p, int f32, long long rows, long long ldp, int lat_off, void* q, long long ldq, int q_off, int heads, int dim,
+                            int rot_dim, int rank, int width, int block_size, int num_blocks, const int* positions, const long long* slots,
+                            const void* norm_w, const float* freq, int half, int halves, float gain, float eps, void* cache, void* q_lat, int q_rows,
+                            int* status, void* stream) {
   if (rows <= 0) return 0;
   if (2 * half > rot_dim || rank + rot_dim > width) return -2;
-  LatentShape s{ldp, q_off, lat_off, 0, heads, dim, rot_dim, 0, rank, width, block_size, num_blocks};
+  LatentShape s{ldp, ldq, 0, q_off, lat_off, 0, heads, dim, rot_dim, 0, rank, width, block_size, num_blocks, halves, 0};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const dim3 grid(static_cast<unsigned>(rows), 2), block(128);
   if (f32)
-    rlb_launch_pdl(latent_prep_kernel<float>, grid, block, 0, st, static_cast<float*>(p), s, positions, slots, static_cast<const float*>(norm_w),
-                                                                            freq, half, gain, eps, static_cast<float*>(cache), static_cast<float*>(q_lat), q_rows, status);
+    rlb_launch_pdl(latent_prep_kernel<float>, grid, block, 0, st, static_cast<const float*>(p), static_cast<float*>(q), s, positions, slots,
+                   static_cast<const float*>(norm_w), freq, half, gain, eps, static_cast<float*>(cache), static_cast<float*>(q_lat), q_rows, status);
   else
-    rlb_launch_pdl(latent_prep_kernel<__nv_bfloat16>, grid, block, 0, st, static_cast<__nv_bfloat16*>(p), s, positions, slots,
+    rlb_launch_pdl(latent_prep_kernel<__nv_bfloat16>, grid, block, 0, st, static_cast<const __nv_bfloat16*>(p), static_cast<__nv_bfloat16*>(q), s, positions, slots,
         static_cast<const __nv_bfloat16*>(norm_w), freq, half, gain, eps, static_cast<__nv_bfloat16*>(cache),
         static_cast<__nv_bfloat16*>(q_lat), q_rows, status);
   return static_cast<int>(cudaGetLastError());
 }
 
-RLB_API int rlb_latent_rows(void* p, int f32, int rows, long long ldp, int q_off, int mix_off, int heads, int dim, int rot_dim, int vdim, int rank,
+// q: prepared queries; out (row stride ldo, may be the same rows): head outputs from column mix_off, gated by what stands there when `gated`.
+RLB_API int rlb_latent_rows(const void* q, int f32, int rows, long long ldq, int q_off, void* out, long long ldo, int mix_off, int gated, int heads, int dim, int rot_dim, int vdim, int rank,
                             int width, int block_size, int num_blocks, const void* cache, const int* block_table, int bt_stride,
                             const int* seq_lens, const void* kv_up, float scale, int* status, void* stream) {
   if (rows <= 0) return 0;
   if (rank + rot_dim > width || heads > 65535) return -2;
-  LatentShape s{ldp, q_off, 0, mix_off, heads, dim, rot_dim, vdim, rank, width, block_size, num_blocks};
+  LatentShape s{0, ldq, ldo, q_off, 0, mix_off, heads, dim, rot_dim, vdim, rank, width, block_size, num_blocks, 0, gated};
   const size_t sm = sizeof(float) * ((width + rank + LR_TILE + 1) & ~1) + sizeof(long long) * LR_TILE;
   const dim3 grid(rows, heads);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   int rc;
   if (f32) {
     if ((rc = smem_attr(reinterpret_cast<const void*>(latent_rows_kernel<float>), sm))) return rc;
-    latent_rows_kernel<float><<<grid, 128, sm, st>>>(static_cast<float*>(p), s, static_cast<const float*>(cache), block_table, bt_stride, seq_lens,
+    latent_rows_kernel<float><<<grid, 128, sm, st>>>(static_cast<const float*>(q), static_cast<float*>(out), s, static_cast<const float*>(cache), block_table, bt_stride, seq_lens,
                                                      static_cast<const float*>(kv_up), scale, status);
   } else {
     if ((rc = smem_attr(reinterpret_cast<const void*>(latent_rows_kernel<__nv_bfloat16>), sm))) return rc;
-    latent_rows_kernel<__nv_bfloat16><<<grid, 128, sm, st>>>(static_cast<__nv_bfloat16*>(p), s, static_cast<const __nv_bfloat16*>(cache), block_table,
+    latent_rows_kernel<__nv_bfloat16><<<grid, 128, sm, st>>>(static_cast<const __nv_bfloat16*>(q), static_cast<__nv_bfloat16*>(out), s, static_cast<const __nv_bfloat16*>(cache), block_table,
                                                              bt_stride, seq_lens, static_cast<const __nv_bfloat16*>(kv_up), scale, status);
   }
   return static_cast<int>(cudaGetLastError());

@@ -10,7 +10,7 @@
 // CUDA cores never touch K or V. Warp roles: warp 0 streams K and V tiles with TMA (one buffer each; the next K tile is
 // requested as soon as the QK MMAs of the current one have completed, the next V tile after the PV MMAs), warp 1 issues
 // the MMAs, warps 2-5 own one token row of S^T / one dim row of O^T each and keep the running max / sum / output in
-// registers. Every wait is bounded (status word, no hang).
+// registers. Every wait is bounded (status word, no hang). With chunks of C positions only the keys of the query's own chunk are read.
 //
 // The CUDA-core kernel in paged_decode_tma.cu (same contract) is kept as the fallback for block sizes / head dims this
 // kernel does not cover. Reference counterpart: the FlashInfer / vLLM paged-attention decode kernels behind
@@ -46,6 +46,7 @@ struct DmParams {
   __nv_bfloat16* out;
   long long out_stride;
   int* status;
+  int chunk;               // > 0: only the query's own run of `chunk` positions is visible
 };
 
 __device__ __forceinline__ void named_bar_sync(int id, int count) {
@@ -108,8 +109,9 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
   const int G = p.G, Hq = p.Hkv * G;
   const int len = p.seq_lens[seq];
   const int bs = p.block_size;
-  const int per_split = ((len + p.num_splits - 1) / p.num_splits + DM_TOK - 1) / DM_TOK * DM_TOK;
-  const int t_begin = split * per_split;
+  const int t_first = p.chunk > 0 && len > 0 ? (len - 1) / p.chunk * p.chunk : 0, t_base = t_first / DM_TOK * DM_TOK;      // first key, its tile
+  const int per_split = ((len - t_base + p.num_splits - 1) / p.num_splits + DM_TOK - 1) / DM_TOK * DM_TOK;
+  const int t_begin = t_base + split * per_split;
   const int t_end = min(len, t_begin + per_split);
   const int n_tiles = t_end > t_begin ? (t_end - t_begin + DM_TOK - 1) / DM_TOK : 0;
 
@@ -244,7 +246,8 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(s_empty));
-      const bool valid = t_begin + i * DM_TOK + r < t_end;
+      const int tok = t_begin + i * DM_TOK + r;
+      const bool valid = tok >= t_first && tok < t_end;
       float s[8], pr[8], c[8];
 #pragma unroll
       for (int g = 0; g < 8; ++g) {
@@ -332,10 +335,10 @@ __global__ void dm_combine_kernel(const float* __restrict__ part_o, const float*
 }
 }  // namespace
 
-// Same contract as rlb_paged_decode_tma. Supported: head_dim 128, Hq / Hkv <= 8, block_size 16, 32, 64 or a multiple of 128.
+// Same contract as rlb_paged_decode_tma; chunk > 0: only the query's own chunk of positions is visible. Supported: head_dim 128, Hq / Hkv <= 8, block_size 16, 32, 64 or a multiple of 128.
 RLB_API int rlb_paged_decode_mma(const void* q, long long q_stride, const void* k_cache, const void* v_cache, int num_blocks,
                                  const int* block_table, int max_blocks_per_seq, const int* seq_lens, int B, int Hq, int Hkv, int D,
-                                 int block_size, float scale, int num_splits, float* part_o, float* part_ml, void* out,
+                                 int block_size, int chunk, float scale, int num_splits, float* part_o, float* part_ml, void* out,
                                  long long out_stride, int* status, void* stream) {
   if (B <= 0) return 0;
   if (D != DM_D || Hq % Hkv || Hq / Hkv > 8) return -2;
@@ -367,6 +370,7 @@ RLB_API int rlb_paged_decode_mma(const void* q, long long q_stride, const void* 
   p.out = static_cast<__nv_bfloat16*>(out);
   p.out_stride = out_stride;
   p.status = status;
+  p.chunk = chunk;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(paged_decode_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, DM_SMEM);

@@ -434,7 +434,7 @@ class GenerationEngine:
         # ``_hybrid_block``. Prefixes are not shared between sequences (pages carry no state) and decode runs eagerly.
         self.hybrid = bool(self.cfg.is_hybrid)
         self._attn_layers = [i for i, l in enumerate(model.layers) if l.self_attn is not None]
-        # layer-list models (Gadarax, Redarax): one cache or state pool per layer RUN (a looped layer has one per pass), see ``_mixer_forward``
+        # layer-list models (Gadarax, Redarax, Kikivik): one cache or state pool per layer RUN (a looped layer has one per pass), see ``_mixer_forward``
         self.mixer = bool(self.cfg.is_mixer)
         self.runs = self.cfg.layer_runs if self.mixer else []
         self.stateful = bool(self.cfg.is_recurrent)   # sequences own a row of the state pools: prefixes are not shared by pages
@@ -577,6 +577,7 @@ class GenerationEngine:
         self.conv_ring = [zeros(self.max_running + 1, m.taps, m.channels) if hasattr(m, "taps") else None for m in mx]
         # portions of prompts attend tile-wise when every attention layer has a shape its tensor-core kernel takes
         tiles = {"latent_attention": X.portion_tiles, "attention": S.portion_tiles}
+        self._chunks = sorted({m.chunk for m in mx if getattr(m, "chunk", 0)})
         self._portion_tiles = self.native and all(tiles[m.kind](m, dt) for m in mx if m.kind in tiles)
 
     def sleep(self, free_kv_cache: bool = True) -> None:
@@ -870,8 +871,8 @@ class GenerationEngine:
         Per layer run: fused input product, mixer, fused output product; the last one's epilogue also updates the fp32 residual
         stream, makes the loop's additions and applies the next layer's norm."""
         m, c, runs = self.model, self.cfg, self.runs
-        if c.norm_place == "post":
-            return self._post_norm_forward(b, rows)
+        if c.layer_form != "parallel":
+            return (self._post_norm_forward if c.layer_form == "post" else self._pre_norm_forward)(b, rows)
         norms = [m.layers[i].norm for i, _ in runs] + [m.norm]
 
         def begins(r):    # (embeddings are added again, step vector) when run r is the first of a pass of the loop
@@ -914,6 +915,29 @@ class GenerationEngine:
             h = h.index_select(0, rows)
         return Y.capped_logits(h, m.output_weight, c.logit_scale, c.final_logit_softcap, self.logits_dtype)
 
+    def _pre_norm_forward(self, b: "X.TokenBatch", rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """``_mixer_forward`` of pre-norm layers. Each sublayer is a product, the mixer or gated unit, a product, and the step that joins its
+        output to the fp32 stream and applies the next sublayer's norm (the final norm behind the last)."""
+        m, c = self.model, self.cfg
+        eps, last, values = c.rms_norm_eps, len(self.runs) - 1, None
+        x, h = Y.embed(b.ids, m.embed_tokens, c.embed_scale, m.layers[self.runs[0][0]].norm1, eps)
+        for r, (i, _) in enumerate(self.runs):
+            layer = m.layers[i]
+            mx, end = layer.mixer, m.norm if r == last else m.layers[self.runs[r + 1][0]].norm1
+            p = Y.linear(h, mx.in_proj, getattr(mx, "in_bias", None))
+            if mx.kind == "latent_attention":
+                a = X.latent_attention(p, mx, b, self.latent_cache[r])
+            else:
+                a = S.attention(p, mx, b, self.k_cache[r], self.v_cache[r], values if mx.v_mix else None)
+                if mx.v_mix and values is None:
+                    values = mx.values(p)
+            h = Y.add_normed_(x, Y.linear(a, mx.out_proj, getattr(mx, "out_bias", None)), None, 1.0, eps, end if layer.ff is None else layer.norm2)
+            if layer.ff is not None:
+                h = Y.feed_forward_(x, h, layer.ff, None, 1.0, eps, end)
+        if rows is not None:
+            h = h.index_select(0, rows)
+        return X.logits(h, m.output_weight, self.logits_dtype)
+
     def _token_batch(self, items) -> tuple:
         """Rows of one step from ``items`` = [(sequence id, tokens, first position)]. Single tokens come first, then portions in order of
         length; returns (batch, first row of every item in the order of ``items``)."""
@@ -947,6 +971,12 @@ class GenerationEngine:
             b.cu_q, b.cu_ctx, b.q_tiles = cu[0], cu[1], sum(-(-lens[j] // 128) for j in tiled)
             b.whole = all(items[order[j]][2] == 0 for j in tiled)
             b.ctx_slots = torch.cat([self.sched.slots(sids[j], 0, n) for j, n in zip(tiled, ctx)]).to(dev)
+            for size in self._chunks:      # what layers that see chunks of positions need: from the border before each portion on
+                lo = [items[order[j]][2] // size * size for j in tiled]
+                cu = torch.zeros(len(tiled) + 1, dtype=torch.int32)
+                cu[1:] = torch.tensor([n - s for n, s in zip(ctx, lo)], dtype=torch.int64).cumsum(0)
+                slots = torch.cat([self.sched.slots(sids[j], s, n - s) for j, n, s in zip(tiled, ctx, lo)])
+                b.chunk_ctx[size] = (cu.to(dev), slots.to(dev), all(items[order[j]][2] == s for j, s in zip(tiled, lo)))
         if self.stateful:
             srow = torch.tensor([self._state_row[s] for s in sids], dtype=torch.int64)
             b.state_rows, b.row_state = srow.to(dev), srow[of_row].to(dev)

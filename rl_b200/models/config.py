@@ -5,10 +5,12 @@ One dataclass covers Llama (2/3/3.1/3.2), Mistral, Qwen2/2.5, Qwen3, Qwen3-MoE a
 before and after each block, scaled embeddings, sliding-window layers with their own RoPE base, a fixed attention scale). ``from_hf_dict`` reads a
 HuggingFace ``config.json`` dictionary; ``PRESETS`` names the architectures used by the benchmark configs.
 
-Models described layer by layer (Gadarax, Redarax) keep their layer list in ``mixers``: each entry names the sequence mixer, its sizes
+Models described layer by layer (Gadarax, Redarax, Kikivik) keep their layer list in ``mixers``: each entry names the sequence mixer, its sizes
 and its MLP. ``LAYER_LISTS`` says which mixers and MLPs each architecture has and how its configuration maps to ``ModelConfig``:
 Gadarax runs mixer and MLP side by side behind one norm (``layer_loop`` repeats a range of layers with the same weights), Redarax runs
-them one after the other and norms what they return (``norm_place`` "post"), with an input per layer and token (``token_side``).
+them one after the other and norms what they return (``norm_place`` "post"), with an input per layer and token (``token_side``), Kikivik
+runs them one after the other on norms of the residual stream. What an architecture fixes for all its mixers of a kind (biases, gates, the
+layout of rotated pairs) is in ``traits`` and joins each layer's sizes (``mixer_spec``, ``mlp_spec``).
 """
 
 from __future__ import annotations
@@ -95,7 +97,7 @@ class ModelConfig:
     moe_latent_size: Optional[int] = None      # routed experts work in a narrower space between two shared projections
     moe_shared_expert_intermediate_size: int = 0
 
-    # models described layer by layer (Gadarax, Redarax): the layers differ in their mixers, sizes and MLPs
+    # models described layer by layer (Gadarax, Redarax, Kikivik): the layers differ in their mixers, sizes and MLPs
     mixers: Optional[list] = None      # per layer: {"type": name of the mixer, "mixer": {sizes}, "mlp": {"kind", sizes} or None}
     layer_loop: Optional[dict] = None  # {"start", "stop", "times"}: layers start .. stop - 1 run `times` times in a row with the same weights
     norm_kind: str = "rms"             # "rms" | "dyt" (dynamic tanh: w * tanh(alpha x) + b, no statistics)
@@ -103,6 +105,7 @@ class ModelConfig:
     residual_mult: float = 1.0         # what sublayer outputs are multiplied by when they join the residual stream
     token_side: Optional[dict] = None  # {"dim"}: every layer adds an input looked up by token in a table of its own (gated by the stream)
     logit_scale: float = 1.0           # logits are multiplied by this (before the soft cap)
+    traits: dict = field(default_factory=dict)   # kind of mixer or MLP: what the architecture fixes for it, in the words of its class
 
     @property
     def is_hybrid(self) -> bool:
@@ -111,6 +114,18 @@ class ModelConfig:
     @property
     def is_mixer(self) -> bool:
         return self.mixers is not None
+
+    @property
+    def layer_form(self) -> str:
+        """How the layers of a layer-list model are put together: "parallel" | "post" | "pre" (see the three block classes)."""
+        return "post" if self.norm_place == "post" else "parallel" if self.norm_kind == "dyt" else "pre"
+
+    def mixer_spec(self, i: int) -> dict:
+        return {**self.traits.get(self.mixers[i]["type"], {}), **self.mixers[i]["mixer"]}
+
+    def mlp_spec(self, i: int) -> dict:
+        mlp = self.mixers[i]["mlp"]
+        return {**self.traits.get(mlp.get("kind", "dense"), {}), **mlp}
 
     @property
     def is_recurrent(self) -> bool:
@@ -194,6 +209,22 @@ class ModelConfig:
                     n += d + (r["experts"] * (3 * d * mlp["expert"]["ff"] + d + 1) if r else 3 * d * mlp["ff"])
                 n += 2 * d * sd + (d if sd else 0)
             return n
+        if self.model_type == "kikivik":
+            n = 2 * self.vocab_size * d + d
+            for e in self.mixers:
+                m, mlp = e["mixer"], e.get("mlp")
+                H, kd, vd = m["heads"], m["dim"], m["vdim"]
+                if e["type"] == "attention":
+                    n += d * (H * kd + m["kv_heads"] * (kd + vd)) + 2 * kd + (1 if m.get("v_mix") else 0)
+                else:
+                    R, Q, rd = m["kv_rank"], m["q_rank"], m["rot_dim"]
+                    n += d * (Q + R + rd) + Q + R + H * (kd + rd) * Q + H * (kd + vd) * R
+                n += d + H * vd * d
+                if mlp and mlp["kind"] == "moe":
+                    n += d + mlp["router"]["experts"] * (3 * d * mlp["expert"]["ff"] + d) + (3 * d * mlp["shared"]["ff"] if mlp.get("shared") else 0)
+                elif mlp:
+                    n += d + 3 * d * mlp["ff"]
+            return n
         if self.mixers is not None:
             n = self.vocab_size * d + 2 * d + 1 + (self.layer_loop["times"] * d if self.layer_loop else 0)
             for e in self.mixers:
@@ -225,6 +256,9 @@ class ModelConfig:
         return L * (attn + ffn + norms) + emb + d
 
     def to_hf_dict(self) -> dict:
+        if self.model_type == "kikivik":
+            return {"architecture": "Kikivik", "vocab": self.vocab_size, "width": self.hidden_size, "embedding": {"scale": self.embed_scale},
+                    "norm": {"eps": self.rms_norm_eps}, "layers": self.mixers, "torch_dtype": self.torch_dtype}
         if self.model_type == "redarax":
             out = {"architecture": "Redarax", "vocab": self.vocab_size, "width": self.hidden_size, "norm": {"eps": self.rms_norm_eps},
                    "residual_mult": self.residual_mult, "logit_scale": self.logit_scale, "layers": self.mixers, "torch_dtype": self.torch_dtype}
@@ -240,7 +274,7 @@ class ModelConfig:
                 "gemma3_text": "Gemma3ForCausalLM", "deepseek_v3": "DeepseekV3ForCausalLM",
                 "nemotron_h": "NemotronHForCausalLM"}.get(self.model_type, "LlamaForCausalLM")
         d = asdict(self)
-        for k in ("mixers", "layer_loop", "norm_kind", "norm_place", "residual_mult", "token_side", "logit_scale"):
+        for k in ("mixers", "layer_loop", "norm_kind", "norm_place", "residual_mult", "token_side", "logit_scale", "traits"):
             d.pop(k)
         nh = {k: d.pop(k) for k in ("layers_block_type", "use_rope", "mlp_gated", "mlp_bias", "mamba_num_heads", "mamba_head_dim", "ssm_state_size",
                                     "mamba_n_groups", "mamba_d_conv", "mamba_chunk_size", "mamba_conv_bias", "mamba_proj_bias", "mamba_dt_limit",
@@ -397,6 +431,7 @@ class ModelConfig:
             need = MIXER_SIZES[e["type"]] if e["type"] in mixers else None
             if need is None:
                 raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
+            need = need + (("q_rank",) if hf["architecture"] == "Kikivik" and e["type"] == "latent_attention" else ())
             missing = [k for k in need if k not in e["mixer"]]
             if missing:
                 raise ValueError(f"layer {i}: the {e['type']} mixer lacks {missing}")
@@ -408,6 +443,9 @@ class ModelConfig:
                 g = r.get("groups") or {"count": 1, "keep": 1}
                 if r["experts"] % g["count"] or not 1 <= g["keep"] <= g["count"] or not 1 <= r["top"] <= g["keep"] * (r["experts"] // g["count"]):
                     raise ValueError(f"layer {i}: router {r} does not fit its groups")
+        mixing = {(e["mixer"]["kv_heads"], e["mixer"]["vdim"]) for e in layers if e["type"] == "attention" and e["mixer"].get("v_mix")}
+        if len(mixing) > 1:
+            raise ValueError(f"layers that mix their values have unequal (key / value heads, value sizes): {sorted(mixing)}")
         lp = hf.get("loop")
         if lp and not (0 <= lp["start"] < lp["stop"] <= len(layers) and lp["times"] >= 1):
             raise ValueError(f"layer loop {lp} does not fit {len(layers)} layers")
@@ -456,6 +494,8 @@ def _check_mixer(i: int, kind: str, m: dict) -> None:
         raise ValueError(f"layer {i}: {m['heads'] * m['vdim']} channels do not divide into {m['norm_groups']} norm groups")
     if m.get("conv", 1) < 1:
         raise ValueError(f"layer {i}: a convolution needs at least one tap")
+    if m.get("mask") and m["mask"]["size"] < 1:
+        raise ValueError(f"layer {i}: chunks of {m['mask']['size']} positions")
 
 
 def _ff_width(mlp: dict) -> int:
@@ -471,9 +511,18 @@ def _redarax(hf: dict) -> dict:
                 final_logit_softcap=float(hf.get("logit_softcap") or 0.0), token_side=dict(hf["token_side"]) if hf.get("token_side") else None)
 
 
+KIKIVIK_TRAITS = {"latent_attention": {"gate": False, "interleaved": False}, "attention": {"bias": False, "interleaved": False},
+                  "moe": {"weigh_input": True, "corrected": False}}
+
+
+def _kikivik(hf: dict) -> dict:
+    return dict(model_type="kikivik", embed_scale=float(hf["embedding"]["scale"]), traits=KIKIVIK_TRAITS)
+
+
 # architecture -> (its mixers, its kinds of MLP, configuration -> further ModelConfig fields)
 LAYER_LISTS = {"Gadarax": (("latent_attention", "retention"), ("dense",), _gadarax),
-               "Redarax": (("attention", "mamba2", "delta"), ("dense", "moe"), _redarax)}
+               "Redarax": (("attention", "mamba2", "delta"), ("dense", "moe"), _redarax),
+               "Kikivik": (("latent_attention", "attention"), ("dense", "moe"), _kikivik)}
 
 
 def rope_inv_freq(cfg: ModelConfig, device=None) -> torch.Tensor:
@@ -513,15 +562,18 @@ def rope_inv_freq(cfg: ModelConfig, device=None) -> torch.Tensor:
 
 def rotary_table(rot: dict) -> tuple[torch.Tensor, float]:
     """Angle per position of each rotated pair [dims / 2] (fp32) and the factor on cosine and sine, for a rotation described by
-    ``{"dims", "base"}`` and optionally ``"scaling"`` = YaRN's ``{"factor", "original", "fast", "slow"}``: pairs that turn more than
-    ``fast`` times within the original context keep their frequency, pairs that turn less than ``slow`` times are slowed down by
-    ``factor``, with a linear ramp between the two (upper end clamped at the last dimension)."""
+    ``{"dims", "base"}`` and optionally ``"scaling"``: ``{"factor"}`` alone slows every pair down by ``factor``, YaRN's ``{"factor",
+    "original", "fast", "slow"}`` keeps the frequency of pairs that turn more than ``fast`` times within the original context and slows
+    down by ``factor`` those that turn less than ``slow`` times, with a linear ramp between the two (upper end clamped at the last
+    dimension)."""
     n, base = int(rot["dims"]), float(rot["base"])
     f = base ** (-2.0 * torch.arange(n // 2, dtype=torch.float64) / n) if n else torch.zeros(0, dtype=torch.float64)
     s = rot.get("scaling")
     if not s:
         return f.float(), 1.0
     factor = float(s["factor"])
+    if "original" not in s:
+        return (f / factor).float(), 1.0
 
     def dim_of(turns):
         return n * math.log(float(s["original"]) / (2 * math.pi * float(turns))) / (2 * math.log(base))

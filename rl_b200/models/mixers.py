@@ -1,5 +1,5 @@
-"""Sequence mixers of models that are described layer by layer, and the parallel layer (mixer and MLP side by side); the layer whose
-sublayers run one after the other is in ``post_norm.py``.
+"""Sequence mixers of models that are described layer by layer, and the parallel layer (mixer and MLP side by side); the layers whose
+sublayers run one after the other are in ``post_norm.py`` and ``pre_norm.py``.
 
 A parallel layer computes ``h = norm(x)`` once and adds ``mixer(h) + mlp(h)`` to the residual stream, so all its input projections
 read the same rows and both its output projections write the same rows. The layer therefore holds two fused weights:
@@ -12,11 +12,13 @@ Segments start at multiples of 8 columns (16-byte rows for TMA); padding rows an
 
 Mixers:
   * ``LatentAttentionMixer``: causal attention whose keys and values are decompressed from one normalised latent per token; only
-    the latent and a rotated key part shared by the heads are cached. Own softmax scale, output gate, interleaved rotation.
+    the latent and a rotated key part shared by the heads are cached. Own softmax scale; queries plain or through a normed latent of their
+    own, output gate or none, rotated pairs interleaved or in halves.
   * ``RetentionMixer``: linear attention with one fixed decay per head, a unit-RMS norm per head and a SiLU gate. The state
     [heads, dim, vdim] is fp32.
-  * ``GroupedAttentionMixer``: causal attention with fewer key / value heads than query heads, biases, RMS norms per head on queries and
-    keys, interleaved partial rotation, own scale, keys and values of unequal size.
+  * ``GroupedAttentionMixer``: causal attention with fewer key / value heads than query heads, RMS norms per head on queries and keys,
+    partial rotation (pairs interleaved or in halves), own scale, keys and values of unequal size; optionally biases, keys of the query's
+    own chunk of positions only, values mixed with those of the first such layer.
   * ``Mamba2LayerMixer``: state-space duality with a short convolution in front and a gated norm in equal parts behind.
   * ``DeltaMixer``: gated delta rule: a linear-attention state that forgets by a decay per token and corrects what it stores under a key.
 
@@ -71,6 +73,9 @@ def rotate_pairs(x: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor, g
 
 
 class LatentAttentionMixer(nn.Module):
+    """Spec, beside the sizes: "q_rank" (queries go through a normed latent of this width), "gate" (output gate, default yes), "interleaved"
+    (rotated pairs are (2i, 2i + 1), default yes; else (i, i + dims / 2))."""
+
     kind = "latent_attention"
 
     def __init__(self, spec: dict, cfg: ModelConfig, dtype, device):
@@ -80,19 +85,38 @@ class LatentAttentionMixer(nn.Module):
         self.qdim = self.dim + self.rot_dim
         self.latent_width = pad8(self.rank + self.rot_dim)       # row width of the cache: [latent | rotated key | padding]
         H = self.heads
-        self.q_off, self.lat_off = 0, pad8(H * self.qdim)
-        self.mix_off = self.lat_off + pad8(self.rank + self.rot_dim)
+        self.q_rank, self.gate, self.interleaved = spec.get("q_rank", 0), bool(spec.get("gate", True)), bool(spec.get("interleaved", True))
+        self.q_off, self.lat_off = 0, pad8(self.q_rank or H * self.qdim)
         self.mix_width = pad8(H * self.vdim)
-        self.in_width = self.mix_off + self.mix_width
+        end = self.lat_off + pad8(self.rank + self.rot_dim)
+        # with a gate the head outputs are written over its columns of the projected rows, else to rows of their own
+        self.mix_off, self.in_width = (end, end + self.mix_width) if self.gate else (0, end)
+        if self.q_rank:
+            self.q_norm = nn.Parameter(torch.ones(self.q_rank, dtype=dtype, device=device))
+            self.q_up = nn.Parameter(torch.zeros(pad8(H * self.qdim), pad8(self.q_rank), dtype=dtype, device=device))
         self.kv_norm = nn.Parameter(torch.ones(self.rank, dtype=dtype, device=device))
         self.kv_up = nn.Parameter(torch.empty(H * (self.dim + self.vdim), self.rank, dtype=dtype, device=device))   # [keys | values]
         freq, self.gain = rotary_table(spec["rot"])
         self.register_buffer("freq", freq.to(device), persistent=False)
 
+    def add_projections(self, d: int, dtype, device) -> None:
+        """Projections of the mixer's own, in layers that do not fuse them with the MLP's."""
+        self.in_proj = nn.Parameter(torch.zeros(self.in_width, d, dtype=dtype, device=device))
+        self.out_proj = nn.Parameter(torch.zeros(d, self.mix_width, dtype=dtype, device=device))
+
+    def tensors(self) -> list:
+        """(checkpoint leaf, view of a parameter); with projections of the mixer's own."""
+        out = [(leaf, self.in_proj[r : r + n]) for leaf, r, n in self.in_rows()]
+        out += [(leaf, getattr(self, p) if n is None else getattr(self, p)[r : r + n]) for leaf, p, r, n in self.own_tensors()]
+        if self.q_rank:
+            out += [("dq.norm", self.q_norm), ("uq", self.q_up[: self.heads * self.qdim, : self.q_rank])]
+        return out + [("o", self.out_proj[:, : self.heads * self.vdim])]
+
     def in_rows(self) -> list:
         """(checkpoint leaf, first row, rows) of this mixer's slices of ``in_proj``."""
         H = self.heads
-        return [("q", self.q_off, H * self.qdim), ("dkv", self.lat_off, self.rank + self.rot_dim), ("g", self.mix_off, H * self.vdim)]
+        out = [("dq", self.q_off, self.q_rank) if self.q_rank else ("q", self.q_off, H * self.qdim), ("dkv", self.lat_off, self.rank + self.rot_dim)]
+        return out + ([("g", self.mix_off, H * self.vdim)] if self.gate else [])
 
     def own_tensors(self) -> list:
         """(checkpoint leaf, parameter name, first row, rows or None)."""
@@ -104,21 +128,28 @@ class LatentAttentionMixer(nn.Module):
         lat = p[:, self.lat_off : self.lat_off + self.rank].float()
         lat = lat * torch.rsqrt(lat.pow(2).mean(-1, keepdim=True) + self.eps) * self.kv_norm.float()
         kr = p[:, self.lat_off + self.rank : self.lat_off + self.rank + self.rot_dim]
-        return lat, rotate_pairs(kr[:, None], positions, self.freq, self.gain, True)[:, 0]
+        return lat, rotate_pairs(kr[:, None], positions, self.freq, self.gain, self.interleaved)[:, 0]
+
+    def project_queries(self, p: torch.Tensor) -> torch.Tensor:
+        """Rows with the queries from column ``q_off`` on: the projected rows, or the product of the normed query latent."""
+        if not self.q_rank:
+            return p
+        c = rms_unit(p[:, : self.q_rank].float(), self.eps) * self.q_norm.float()
+        return _linear(TF.pad(c, (0, self.q_up.shape[1] - self.q_rank)).to(p.dtype), self.q_up)
 
     def queries(self, p: torch.Tensor, positions: torch.Tensor):
         q = p[:, self.q_off : self.q_off + self.heads * self.qdim].reshape(-1, self.heads, self.qdim)
-        return torch.cat([q[..., : self.dim].float(), rotate_pairs(q[..., self.dim :], positions, self.freq, self.gain, True)], dim=-1)
+        return torch.cat([q[..., : self.dim].float(), rotate_pairs(q[..., self.dim :], positions, self.freq, self.gain, self.interleaved)], dim=-1)
 
     def sequence(self, p: torch.Tensor, positions: torch.Tensor, cu_seqlens: torch.Tensor) -> torch.Tensor:
-        """Gated head outputs [T, heads * vdim] of packed whole sequences."""
+        """Head outputs [T, heads * vdim] of packed whole sequences, gated where the mixer has a gate."""
         T, H = p.shape[0], self.heads
         lat, kr = self.key_parts(p, positions)
         lat = lat.to(p.dtype)
         k = TF.linear(lat, self.kv_up[: H * self.dim]).reshape(T, H, self.dim)
         v = TF.linear(lat, self.kv_up[H * self.dim :]).reshape(T, H, self.vdim).float()
         k = torch.cat([k.float(), kr[:, None].expand(T, H, self.rot_dim)], dim=-1)
-        q = self.queries(p, positions)
+        q = self.queries(self.project_queries(p), positions)
         out = []
         cu = cu_seqlens.tolist()
         for s, e in zip(cu[:-1], cu[1:]):
@@ -126,6 +157,8 @@ class LatentAttentionMixer(nn.Module):
             z = z.masked_fill(torch.ones(e - s, e - s, dtype=torch.bool, device=z.device).triu(1), float("-inf"))
             out.append(torch.einsum("hij,jhd->ihd", torch.softmax(z, -1), v[s:e]))
         y = torch.cat(out).reshape(T, H * self.vdim)
+        if not self.gate:
+            return y.to(p.dtype)
         return (y * torch.sigmoid(p[:, self.mix_off : self.mix_off + H * self.vdim].float())).to(p.dtype)
 
 
@@ -200,6 +233,10 @@ def rms_unit(x: torch.Tensor, eps: float) -> torch.Tensor:
 
 
 class GroupedAttentionMixer(nn.Module):
+    """Spec, beside the sizes: "bias" (default yes), "interleaved" (rotated pairs are (2i, 2i + 1), default yes; else (i, i + dims / 2)),
+    "mask" = {"size"} (position i sees j <= i of the same run of ``size`` positions, counted from the sequence's first), "v_mix" (values
+    become (1 - share) v + share v_first with v_first the first such layer's)."""
+
     kind = "attention"
 
     def __init__(self, spec: dict, cfg: ModelConfig, dtype, device):
@@ -212,9 +249,15 @@ class GroupedAttentionMixer(nn.Module):
         self.mix_width = pad8(self.heads * self.vdim)
         d = cfg.hidden_size
         self.in_proj = nn.Parameter(torch.zeros(self.in_width, d, dtype=dtype, device=device))
-        self.in_bias = nn.Parameter(torch.zeros(self.in_width, dtype=dtype, device=device))
         self.out_proj = nn.Parameter(torch.zeros(d, self.mix_width, dtype=dtype, device=device))
-        self.out_bias = nn.Parameter(torch.zeros(d, dtype=dtype, device=device))
+        self.in_bias = self.out_bias = None
+        if spec.get("bias", True):
+            self.in_bias = nn.Parameter(torch.zeros(self.in_width, dtype=dtype, device=device))
+            self.out_bias = nn.Parameter(torch.zeros(d, dtype=dtype, device=device))
+        self.interleaved, self.chunk = bool(spec.get("interleaved", True)), int((spec.get("mask") or {"size": 0})["size"])
+        self.v_mix = bool(spec.get("v_mix"))
+        if self.v_mix:
+            self.v_share = nn.Parameter(torch.full((), 0.5, dtype=dtype, device=device))
         self.q_norm = nn.Parameter(torch.ones(self.dim, dtype=dtype, device=device))
         self.k_norm = nn.Parameter(torch.ones(self.dim, dtype=dtype, device=device))
         freq, self.gain = rotary_table(spec["rot"])
@@ -224,29 +267,40 @@ class GroupedAttentionMixer(nn.Module):
         """(checkpoint leaf, view of a parameter)."""
         out = []
         for leaf, r, n in (("q", self.q_off, self.heads * self.dim), ("k", self.k_off, self.kv_heads * self.dim), ("v", self.v_off, self.kv_heads * self.vdim)):
-            out += [(leaf, self.in_proj[r : r + n]), (leaf + ".b", self.in_bias[r : r + n])]
-        return out + [("q.norm", self.q_norm), ("k.norm", self.k_norm), ("o", self.out_proj[:, : self.heads * self.vdim]), ("o.b", self.out_bias)]
+            out += [(leaf, self.in_proj[r : r + n])] + ([(leaf + ".b", self.in_bias[r : r + n])] if self.in_bias is not None else [])
+        out += [("q.norm", self.q_norm), ("k.norm", self.k_norm), ("o", self.out_proj[:, : self.heads * self.vdim])]
+        return out + ([("o.b", self.out_bias)] if self.out_bias is not None else []) + ([("vmix", self.v_share)] if self.v_mix else [])
 
-    def qkv(self, p: torch.Tensor, positions: torch.Tensor):
-        """fp32 normed and rotated queries [T, heads, dim] and keys [T, kv_heads, dim], values [T, kv_heads, vdim]."""
+    def values(self, p: torch.Tensor) -> torch.Tensor:
+        """The layer's own values, columns of the projected rows."""
+        return p[:, self.v_off : self.v_off + self.kv_heads * self.vdim]
+
+    def qkv(self, p: torch.Tensor, positions: torch.Tensor, first=None):
+        """fp32 normed and rotated queries [T, heads, dim] and keys [T, kv_heads, dim], values [T, kv_heads, vdim] (mixed with ``first``)."""
         q = p[:, self.q_off : self.q_off + self.heads * self.dim].reshape(-1, self.heads, self.dim).float()
         k = p[:, self.k_off : self.k_off + self.kv_heads * self.dim].reshape(-1, self.kv_heads, self.dim).float()
-        v = p[:, self.v_off : self.v_off + self.kv_heads * self.vdim].reshape(-1, self.kv_heads, self.vdim).float()
-        q = rotate_pairs(rms_unit(q, self.eps) * self.q_norm.float(), positions, self.freq, self.gain, True)
-        k = rotate_pairs(rms_unit(k, self.eps) * self.k_norm.float(), positions, self.freq, self.gain, True)
+        v = self.values(p).float()
+        if first is not None:
+            v = (1 - self.v_share.float()) * v + self.v_share.float() * first.float()
+        v = v.reshape(-1, self.kv_heads, self.vdim)
+        q = rotate_pairs(rms_unit(q, self.eps) * self.q_norm.float(), positions, self.freq, self.gain, self.interleaved)
+        k = rotate_pairs(rms_unit(k, self.eps) * self.k_norm.float(), positions, self.freq, self.gain, self.interleaved)
         return q, k, v
 
-    def sequence(self, p: torch.Tensor, positions: torch.Tensor, cu_seqlens: torch.Tensor) -> torch.Tensor:
+    def sequence(self, p: torch.Tensor, positions: torch.Tensor, cu_seqlens: torch.Tensor, first=None) -> torch.Tensor:
         """Head outputs [T, heads * vdim] of packed whole sequences."""
-        q, k, v = self.qkv(p, positions)
+        q, k, v = self.qkv(p, positions, first)
         n = self.heads // self.kv_heads
         k, v = k.repeat_interleave(n, dim=1), v.repeat_interleave(n, dim=1)
         out = []
         cu = cu_seqlens.tolist()
         for s, e in zip(cu[:-1], cu[1:]):
             z = torch.einsum("ihd,jhd->hij", q[s:e], k[s:e]) * self.scale
-            z = z.masked_fill(torch.ones(e - s, e - s, dtype=torch.bool, device=z.device).triu(1), float("-inf"))
-            out.append(torch.einsum("hij,jhd->ihd", torch.softmax(z, -1), v[s:e]))
+            hidden = torch.ones(e - s, e - s, dtype=torch.bool, device=z.device).triu(1)
+            if self.chunk:
+                c = torch.arange(e - s, device=z.device) // self.chunk
+                hidden = hidden | (c[:, None] != c[None, :])
+            out.append(torch.einsum("hij,jhd->ihd", torch.softmax(z.masked_fill(hidden, float("-inf")), -1), v[s:e]))
         return torch.cat(out).reshape(-1, self.heads * self.vdim).to(p.dtype)
 
 
@@ -407,7 +461,7 @@ class ParallelBlock(nn.Module):
         entry = cfg.mixers[layer_idx]
         d = cfg.hidden_size
         self.norm = DynamicTanh(d, dtype, device)
-        self.mixer = MIXERS[entry["type"]](entry["mixer"], cfg, dtype, device)
+        self.mixer = MIXERS[entry["type"]](cfg.mixer_spec(layer_idx), cfg, dtype, device)
         self.ff = entry["mlp"]["ff"] if entry.get("mlp") else 0
         self.up_off = self.mixer.in_width                  # first MLP column of the projected rows; squared ReLU from here on
         self.in_width = self.up_off + pad8(self.ff)

@@ -523,8 +523,9 @@ class CausalLM(nn.Module):
         if cfg.is_mixer:
             from .mixers import DynamicTanh, ParallelBlock
             from .post_norm import PostNormBlock
+            from .pre_norm import PreNormBlock
 
-            block = PostNormBlock if cfg.norm_place == "post" else ParallelBlock
+            block = {"parallel": ParallelBlock, "post": PostNormBlock, "pre": PreNormBlock}[cfg.layer_form]
             if tpw > 1 or pp_size > 1 or self.cp is not None or (ep is not None and ep.world > 1) or self.lora_cfg or cfg.value_head:
                 raise NotImplementedError("layer-list models run data parallel only, without LoRA or value heads")
         if cfg.is_hybrid and self.tp.sequence_parallel:
@@ -729,12 +730,14 @@ class CausalLM(nn.Module):
     def _run_layer_runs(self, h: torch.Tensor, batch: PackedBatch) -> torch.Tensor:
         """Layers in the order of ``cfg.layer_runs``. A pass of the loop begins with the embeddings added again (not in the first)
         and with its step vector added."""
-        e, loop = h, self.cfg.layer_loop
+        e, loop, carries, values = h, self.cfg.layer_loop, self.cfg.layer_form == "pre", None
         for i, t in self.cfg.layer_runs:
             if t is not None and i == loop["start"]:
                 h = (h + e if t else h) + self.loop_step[t].float()
-            args = (h, batch.positions, self.side_rows(batch.input_ids, i), batch.cu_seqlens, batch.max_seqlen)
+            args = (h, batch.positions, values if carries else self.side_rows(batch.input_ids, i), batch.cu_seqlens, batch.max_seqlen)
             h = ckpt.checkpoint(self.layers[i], *args, use_reentrant=False) if (self.activation_checkpointing and torch.is_grad_enabled()) else self.layers[i](*args)
+            if carries:        # pre-norm layers hand on the values that later ones mix in
+                h, values = h
         return h
 
     def side_rows(self, ids: torch.Tensor, layer: int) -> Optional[torch.Tensor]:

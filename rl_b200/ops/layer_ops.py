@@ -1,5 +1,5 @@
-"""Row operators of post-norm layers (``rl_b200/models/post_norm.py``) in the generation engine: products with what follows them, the
-normed join with the residual stream, the gated feed-forwards and the token input.
+"""Row operators of post-norm and pre-norm layers (``rl_b200/models/post_norm.py``, ``pre_norm.py``) in the generation engine: products with
+what follows them, the join with the residual stream, the gated feed-forwards and the token input.
 
 Each operator has the native sm_100a body (CUDA tensors, bf16 or fp32) and a plain PyTorch statement (CPU tensors). ``x`` is the fp32
 residual stream, updated in place; ``h`` what the next sublayer reads (x in the model's type). fp32 models run every product in true fp32.
@@ -23,17 +23,17 @@ register("rlb_linear_rows", [P, P])
 register("rlb_linear_tiled", [P, P])
 register("rlb_linear_skinny", [P, P])
 register("rlb_linear_grouped", [P, P])
-register("rlb_add_normed", [P, P, LL, I, P, P, I, I, P, I, P, P, P, LL, I, CF, CF, P])
+register("rlb_add_normed", [P, P, LL, I, P, P, I, I, P, I, P, LL, P, P, P, LL, I, CF, CF, P])
 register("rlb_group_norm_rows", [P, LL, I, P, LL, I, I, CF, P])
 register("rlb_cap_rows", [P, LL, CF, CF, P])
 register("rlb_moe_choose", [P, LL, I, I, P, I, I, I, P, P, P, P, P])
-register("rlb_moe_place", [P, P, LL, I, P, I, I, P, P, P, P, LL, P, I, P, P])
+register("rlb_moe_place", [P, P, LL, I, P, I, I, P, P, P, P, LL, P, I, P, P, P, P])
 
-NONE, GLU, GELU_MUL, CAP = range(4)      # what follows a product (RlbLinearAct)
+NONE, GLU, GELU_MUL, CAP, SILU = range(5)      # what follows a product (RlbLinearAct)
 
 
 class _Linear(C.Structure):
-    _fields_ = [(n, C.c_void_p) for n in ("a", "w", "out", "bias", "table", "ids", "tile_expert", "a_rows", "status")] + \
+    _fields_ = [(n, C.c_void_p) for n in ("a", "w", "out", "bias", "table", "ids", "tile_expert", "a_rows", "status", "row_scale")] + \
                [(n, C.c_longlong) for n in ("lda", "ldw", "ldo", "ld_table")] + \
                [(n, C.c_int) for n in ("M", "N", "K", "in_f32", "out_f32", "act", "table_off", "table_cols", "vocab", "ids64", "experts", "num_a_rows")] + \
                [(n, C.c_float) for n in ("limit", "scale", "cap")]
@@ -63,6 +63,24 @@ def clamped_glu_ref(p: torch.Tensor, limit: float) -> torch.Tensor:
     return (g * torch.sigmoid(1.702 * g) * (u + 1)).to(p.dtype)
 
 
+def silu_glu_ref(p: torch.Tensor) -> torch.Tensor:
+    return (TF.silu(p[:, 0::2].float()) * p[:, 1::2].float()).to(p.dtype)
+
+
+def gated_ref(p: torch.Tensor, limit: Optional[float]) -> torch.Tensor:
+    """Gated unit over neighbouring columns: clamped to ``limit``, or silu without limits (None)."""
+    return silu_glu_ref(p) if limit is None else clamped_glu_ref(p, limit)
+
+
+def gated_linear(a: torch.Tensor, w: torch.Tensor, limit: Optional[float]) -> torch.Tensor:
+    """``gated_ref`` of a w^T, in the product's epilogue."""
+    if not use_native(a):
+        return gated_ref(a @ w.t(), limit)
+    out = torch.empty((a.shape[0], w.shape[0] // 2), dtype=a.dtype, device=a.device)
+    _run(_desc(a, w, out, SILU if limit is None else GLU, limit or 0.0), _aligned(a, w, out))
+    return out
+
+
 def linear(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, glu: Optional[float] = None) -> torch.Tensor:
     """a w^T (+ bias); ``glu``: the limit of a clamped gated unit over neighbouring columns, half as wide."""
     if not use_native(a):
@@ -74,16 +92,16 @@ def linear(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
 
 
 # --------------------------------------------------------------------------------------- residual stream
-def embed(ids: torch.Tensor, table: torch.Tensor, scale: float):
-    """(x, h): the tokens' rows in fp32 and in the model's type."""
+def embed(ids: torch.Tensor, table: torch.Tensor, scale: float, norm: Optional[torch.Tensor] = None, eps: float = 0.0):
+    """(x, h): the tokens' rows in fp32, and in the model's type as they are or rms(x) * norm."""
     if not use_native(table):
         x = table[ids.long()].float() * scale
-        return x, x.to(table.dtype)
+        return x, (x if norm is None else _rms(x, eps) * norm.float()).to(table.dtype)
     T, d = ids.shape[0], table.shape[1]
     x = torch.empty((T, d), dtype=torch.float32, device=table.device)
     h = torch.empty((T, d), dtype=table.dtype, device=table.device)
-    call("rlb_embed_rows", ptr(ids), int(ids.dtype == torch.int64), ptr(table), _f32(table), ptr(x), None, ptr(h), None, None, None, None, T, d,
-         table.shape[0], float(scale), ptr(_L.status_word(table.device)), stream_ptr())
+    call("rlb_embed_rows", ptr(ids), int(ids.dtype == torch.int64), ptr(table), _f32(table), ptr(x), None, ptr(h), None, None, ptr(norm), None, T, d,
+         table.shape[0], float(scale), float(eps), ptr(_L.status_word(table.device)), stream_ptr())
     return x, h
 
 
@@ -91,18 +109,20 @@ def _rms(x: torch.Tensor, eps: float) -> torch.Tensor:
     return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
 
 
-def add_normed_(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, mult: float, eps: float, next_norm: Optional[torch.Tensor] = None,
-                experts: Optional[tuple] = None) -> torch.Tensor:
-    """x += mult * rms(y) * w in place; returns x in the model's type, or rms(x) * next_norm. ``experts`` = (row of every copy, weight of
-    every copy, the experts' counts to reset): y holds expert rows, a token's value is the weighted sum of its copies' rows."""
+def add_normed_(x: torch.Tensor, y: torch.Tensor, w: Optional[torch.Tensor], mult: float, eps: float, next_norm: Optional[torch.Tensor] = None,
+                experts: Optional[tuple] = None, also: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x += mult * rms(y) * w in place (w None: mult * y); returns x in the model's type, or rms(x) * next_norm. ``experts`` = (row of every
+    copy, weight of every copy or None, the experts' counts to reset): y holds expert rows, a token's value is the (weighted) sum of its
+    copies' rows. ``also``: rows added to y first."""
     if not use_native(x):
-        x += mult * (_rms(y.float(), eps) * w.float())
-        return (x if next_norm is None else _rms(x, eps) * next_norm.float()).to(w.dtype)
+        y = y.float() if also is None else y.float() + also.float()
+        x += mult * (y if w is None else _rms(y, eps) * w.float())
+        return (x if next_norm is None else _rms(x, eps) * next_norm.float()).to((next_norm if w is None else w).dtype)
     T, d = x.shape
-    h = torch.empty((T, d), dtype=w.dtype, device=x.device)
+    h = torch.empty((T, d), dtype=y.dtype, device=x.device)
     rows, wt, counts = experts if experts is not None else (None, None, None)
-    call("rlb_add_normed", ptr(x), ptr(y), y.stride(0), _f32(y), ptr(rows), ptr(wt), wt.shape[1] if wt is not None else 0, y.shape[0], ptr(counts),
-         counts.numel() if counts is not None else 0, ptr(w), ptr(next_norm), ptr(h), T, d, float(mult), float(eps), stream_ptr())
+    call("rlb_add_normed", ptr(x), ptr(y), y.stride(0), _f32(y), ptr(rows), ptr(wt), rows.shape[1] if rows is not None else 0, y.shape[0], ptr(counts),
+         counts.numel() if counts is not None else 0, ptr(also), also.stride(0) if also is not None else 0, ptr(w), ptr(next_norm), ptr(h), T, d, float(mult), float(eps), stream_ptr())
     return h
 
 
@@ -116,16 +136,22 @@ def group_norm_(y: torch.Tensor, w: torch.Tensor, groups: int, eps: float) -> No
 
 
 # --------------------------------------------------------------------------------------- feed-forwards
-def feed_forward_(x: torch.Tensor, h: torch.Tensor, ff, norm: torch.Tensor, mult: float, eps: float, next_norm=None) -> torch.Tensor:
-    """x += mult * rms(ff(h)) * norm. ``ff``: the layer's ``ClampedGLU`` or ``ClampedExperts``."""
+def feed_forward_(x: torch.Tensor, h: torch.Tensor, ff, norm: Optional[torch.Tensor], mult: float, eps: float, next_norm=None) -> torch.Tensor:
+    """x += mult * rms(ff(h)) * norm (norm None: mult * ff(h)). ``ff``: the layer's ``GatedUnit`` or ``GatedExperts``."""
     if hasattr(ff, "router"):
-        y, experts = clamped_experts(h, ff)
-        return add_normed_(x, y, norm, mult, eps, next_norm, experts)
-    return add_normed_(x, linear(linear(h, ff.gate_up, glu=ff.limit), ff.down), norm, mult, eps, next_norm)
+        shared = unit(h, ff.shared) if ff.shared is not None else None
+        y, experts = gated_experts(h, ff)
+        return add_normed_(x, y, norm, mult, eps, next_norm, experts, shared)
+    return add_normed_(x, unit(h, ff), norm, mult, eps, next_norm)
 
 
-def clamped_experts(h: torch.Tensor, m):
-    """(expert rows, (row of every copy, weights, counts)) on the native path, (summed outputs, None) otherwise."""
+def unit(h: torch.Tensor, m) -> torch.Tensor:
+    return linear(gated_linear(h, m.gate_up, m.limit), m.down)
+
+
+def gated_experts(h: torch.Tensor, m):
+    """Routed part of ``m`` (``GatedExperts``): (expert rows, (row of every copy, weights or None, counts)) on the native path, (summed
+    outputs, None) otherwise. Weights on the experts' inputs are factors of the first product's rows."""
     T, d = h.shape
     if not use_native(h):
         w, idx = m.choose(h.float() @ m.router.float().t())
@@ -133,7 +159,9 @@ def clamped_experts(h: torch.Tensor, m):
         for e in range(m.experts):
             tok, slot = (idx == e).nonzero(as_tuple=True)
             if tok.numel():
-                y.index_add_(0, tok, (clamped_glu_ref(h[tok] @ m.gate_up[e].t(), m.limit) @ m.down[e].t()).float() * w[tok, slot, None])
+                p, wt = h[tok] @ m.gate_up[e].t(), w[tok, slot, None]
+                a = gated_ref((p.float() * wt).to(p.dtype) if m.weigh_input else p, m.limit)
+                y.index_add_(0, tok, (a @ m.down[e].t()).float() * (1.0 if m.weigh_input else wt))
         return y, None
     dev, E, k = h.device, m.experts, m.top
     st = ptr(_L.status_word(dev))
@@ -147,17 +175,21 @@ def clamped_experts(h: torch.Tensor, m):
     fast = _aligned(h, m.gate_up[0], m.down[0]) and m.gate_up.shape[1] % 8 == 0 and d % 8 == 0
     xp = torch.empty((mpad, d), dtype=h.dtype, device=dev) if fast else h
     src = None if fast else torch.full((mpad,), -1, dtype=torch.int32, device=dev)
+    factor = torch.empty(mpad, dtype=torch.float32, device=dev) if m.weigh_input else None
     call("rlb_moe_place", ptr(idx), ptr(rank), T * k, k, ptr(counts), E, mpad, ptr(copy_row), ptr(tiles), ptr(src), ptr(h),
-         h.stride(0) * h.element_size() if fast else 0, ptr(xp) if fast else None, d * h.element_size() if fast else 0, st, stream_ptr())
+         h.stride(0) * h.element_size() if fast else 0, ptr(xp) if fast else None, d * h.element_size() if fast else 0, ptr(wt) if m.weigh_input else None,
+         ptr(factor), st, stream_ptr())
     a = torch.empty((mpad, m.down.shape[2]), dtype=h.dtype, device=dev)
     y = torch.empty((mpad, d), dtype=h.dtype, device=dev)
     for first, inp, w, out in ((True, xp, m.gate_up, a), (False, a, m.down, y)):
-        q = _desc(inp, w, out, GLU if first else NONE, m.limit)
+        q = _desc(inp, w, out, NONE if not first else SILU if m.limit is None else GLU, m.limit or 0.0)
         q.M, q.experts, q.tile_expert = mpad, E, ptr(tiles)
+        if first:
+            q.row_scale = ptr(factor)
         if first and not fast:
             q.a_rows, q.num_a_rows = ptr(src), T
         call("rlb_linear_grouped" if fast else "rlb_linear_rows", C.byref(q), stream_ptr())
-    return y, (copy_row, wt, counts)
+    return y, (copy_row, None if m.weigh_input else wt, counts)
 
 
 def router_logits(h: torch.Tensor, router: torch.Tensor) -> torch.Tensor:

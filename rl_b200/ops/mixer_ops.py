@@ -1,4 +1,4 @@
-"""Operators of parallel mixer layers (``rl_b200/models/mixers.py``) in the generation engine, over a batch of token rows that mixes
+"""Operators of parallel mixer layers (``rl_b200/models/mixers.py``), and latent attention of every kind of layer, in the generation engine, over a batch of token rows that mixes
 single decoded tokens and portions of prompts.
 
 Each operator has the native sm_100a body (CUDA tensors, bf16 or fp32) and a plain PyTorch statement (CPU tensors). A layer is
@@ -12,7 +12,7 @@ so nothing but the two products and the mixer touches memory. fp32 models run ev
 
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from typing import Optional
 
 import torch
@@ -22,17 +22,17 @@ from . import lib as _L
 from .lib import F as CF
 from .lib import I, L as LL, P, call, ptr, register, stream_ptr, use_native
 
-register("rlb_embed_rows", [P, I, P, I, P, P, P, P, P, P, P, LL, I, I, CF, P, P])
+register("rlb_embed_rows", [P, I, P, I, P, P, P, P, P, P, P, LL, I, I, CF, CF, P, P])
 register("rlb_gemm_rows", [P, P, P, I, I, I, LL, LL, LL, I, I, I, P, LL, P, P, P, P, P, P])
 register("rlb_gemm_layer", [P, P, P, I, I, I, LL, LL, LL, I, P, LL, P, P, P, P, P, P, P])
 register("rlb_gemm_skinny_layer", [P, P, P, I, I, I, LL, LL, LL, I, P, LL, P, P, P, P, P, P, P])
-register("rlb_latent_prep", [P, I, LL, LL, I, I, I, I, I, I, I, I, I, P, P, P, P, I, CF, CF, P, P, I, P, P])
+register("rlb_latent_prep", [P, I, LL, LL, I, P, LL, I, I, I, I, I, I, I, I, P, P, P, P, I, I, CF, CF, P, P, I, P, P])
 register("rlb_latent_gather", [P, P, P, LL, I, LL, P, P])
 register("rlb_flash_latent_supported", [I, I, I, I])
-register("rlb_flash_latent", [P, LL, LL, I, I, P, P, LL, I, P, P, I, I, I, I, I, I, I, I, CF, I, P, P])
+register("rlb_flash_latent", [P, LL, LL, I, I, P, P, LL, I, P, P, I, I, I, I, I, I, I, P, LL, I, I, CF, I, P, P])
 register("rlb_latent_decode_supported", [I, I, I, I, I, I])
-register("rlb_latent_decode", [P, I, LL, I, I, I, I, I, I, I, I, I, I, I, P, P, I, P, P, CF, P, P, I, P, P, P, P])
-register("rlb_latent_rows", [P, I, I, LL, I, I, I, I, I, I, I, I, I, I, P, P, I, P, P, CF, P, P])
+register("rlb_latent_decode", [P, I, LL, I, I, P, LL, I, I, I, I, I, I, I, I, I, I, P, P, I, P, P, CF, P, P, I, P, P, P, P])
+register("rlb_latent_rows", [P, I, I, LL, I, P, LL, I, I, I, I, I, I, I, I, I, I, P, P, I, P, P, CF, P, P])
 register("rlb_retention_rows", [P, I, I, I, LL, I, I, I, I, I, I, I, P, P, P, P, LL, P, P, I, CF, CF, CF, P, P])
 register("rlb_retention_supported", [I, I])
 register("rlb_retention_step", [P, I, LL, I, I, I, I, I, I, I, P, P, P, LL, P, P, I, CF, CF, CF, P, P])
@@ -83,6 +83,7 @@ class TokenBatch:
     row_off: Optional[torch.Tensor] = None      # int32 [T]: rows of the same piece before each row (None: all rows are singles)
     row_state: Optional[torch.Tensor] = None    # int64 [T]: state row of each row's sequence (None: ``state_rows``)
     whole: bool = False              # the tile-wise portions start at position 0
+    chunk_ctx: dict = field(default_factory=dict)   # chunk size: (cu_ctx, ctx_slots, whole) of layers that see chunks, from the border before each portion
     max_ctx: int = 0                 # upper bound of seq_lens (a host number, fixed while a graph is captured)
 
     @property
@@ -112,7 +113,7 @@ def embed_rows(ids, table, scale: float, step: Optional[torch.Tensor], norm, kee
     e = torch.empty_like(x) if keep else None
     h = torch.empty((T, d), dtype=table.dtype, device=dev)
     call("rlb_embed_rows", ptr(ids), int(ids.dtype == torch.int64), ptr(table), _f32(table), ptr(x), ptr(e), ptr(h), ptr(step),
-         ptr(norm.alpha), ptr(norm.weight), ptr(norm.bias), T, d, table.shape[0], float(scale), ptr(_L.status_word(dev)), stream_ptr())
+         ptr(norm.alpha), ptr(norm.weight), ptr(norm.bias), T, d, table.shape[0], float(scale), 0.0, ptr(_L.status_word(dev)), stream_ptr())
     return x, e, h
 
 
@@ -173,10 +174,27 @@ def _page_rows(table_row: torch.Tensor, n: int, block_size: int) -> torch.Tensor
     return table_row.long()[t // block_size] * block_size + t % block_size
 
 
-def latent_attention_(p: torch.Tensor, m, b: TokenBatch, cache: torch.Tensor) -> None:
+def latent_attention(p: torch.Tensor, m, b: TokenBatch, cache: torch.Tensor) -> torch.Tensor:
+    """Rows [T, mix_width] of latent attention without an output gate, its queries taken from their own latent where the mixer has one
+    (normed in place in ``p``)."""
+    from .layer_ops import group_norm_, linear
+
+    q = p
+    if m.q_rank:
+        group_norm_(p, m.q_norm, 1, m.eps)
+        q = linear(p[:, : m.q_up.shape[1]], m.q_up)
+    n = m.heads * m.vdim
+    y = (torch.zeros if m.mix_width > n else torch.empty)((p.shape[0], m.mix_width), dtype=p.dtype, device=p.device)
+    latent_attention_(p, m, b, cache, q, y)
+    return y
+
+
+def latent_attention_(p: torch.Tensor, m, b: TokenBatch, cache: torch.Tensor, q=None, out=None) -> None:
     """Latent attention of all rows of ``p`` over the paged latent cache [pages, page size, width]; the rows' own latents are
-    written first. ``m``: the layer's ``LatentAttentionMixer``."""
+    written first. ``m``: the layer's ``LatentAttentionMixer``. Queries are columns of ``q`` (None: of ``p``; rotated in place), head outputs
+    columns of ``out`` (None: of ``p``, over the gates)."""
     bs = cache.shape[1]
+    q, out = p if q is None else q, p if out is None else out
     if not use_native(p):
         lat, kr = m.key_parts(p, b.positions)
         ok = b.slots >= 0
@@ -184,12 +202,12 @@ def latent_attention_(p: torch.Tensor, m, b: TokenBatch, cache: torch.Tensor) ->
         rows[:, : m.rank], rows[:, m.rank : m.rank + m.rot_dim] = lat.to(p.dtype), kr.to(p.dtype)
         flat = cache.view(-1, m.latent_width)
         flat[b.slots[ok].long()] = rows[ok]
-        q, H = m.queries(p, b.positions).to(p.dtype).float(), m.heads
+        q, H = m.queries(q, b.positions).to(p.dtype).float(), m.heads
         uk = m.kv_up[: H * m.dim].float().view(H, m.dim, m.rank)
         uv = m.kv_up[H * m.dim :].float().view(H, m.vdim, m.rank)
         for i in range(p.shape[0]):
             n = int(b.seq_lens[i])
-            g = p[i, m.mix_off : m.mix_off + H * m.vdim]
+            g = out[i, m.mix_off : m.mix_off + H * m.vdim]
             if n == 0:
                 g.zero_()
                 continue
@@ -197,33 +215,34 @@ def latent_attention_(p: torch.Tensor, m, b: TokenBatch, cache: torch.Tensor) ->
             qa = torch.cat([torch.einsum("hd,hdr->hr", q[i, :, : m.dim], uk), q[i, :, m.dim :]], dim=1)
             w = torch.softmax(qa @ c[:, : m.rank + m.rot_dim].t() * m.scale, dim=-1)
             y = torch.einsum("hr,hvr->hv", w @ c[:, : m.rank], uv).reshape(-1)
-            g.copy_((y * torch.sigmoid(g.float())).to(p.dtype))
+            g.copy_((y * torch.sigmoid(g.float()) if m.gate else y).to(p.dtype))
         return
     dev, T, H, W = p.device, p.shape[0], m.heads, m.latent_width
     st = ptr(_L.status_word(dev))
     decode = b.n_paged > 0 and decode_tiles(p, m, bs)
     q_lat = torch.empty((b.n_paged, H, W), dtype=p.dtype, device=dev) if decode else None
-    call("rlb_latent_prep", ptr(p), _f32(p), T, p.stride(0), m.q_off, m.lat_off, H, m.dim, m.rot_dim, m.rank, W, bs, cache.shape[0], ptr(b.positions),
-         ptr(b.slots), ptr(m.kv_norm), ptr(m.freq), m.freq.numel(), float(m.gain), float(m.eps), ptr(cache), ptr(q_lat),
-         b.n_paged if decode else 0, st, stream_ptr())
+    call("rlb_latent_prep", ptr(p), _f32(p), T, p.stride(0), m.lat_off, ptr(q), q.stride(0), m.q_off, H, m.dim, m.rot_dim, m.rank, W, bs,
+         cache.shape[0], ptr(b.positions), ptr(b.slots), ptr(m.kv_norm), ptr(m.freq), m.freq.numel(), int(not m.interleaved), float(m.gain), float(m.eps),
+         ptr(cache), ptr(q_lat), b.n_paged if decode else 0, st, stream_ptr())
     if decode:
         splits = split_count(b.n_paged * -(-H // (32 if H > 16 else 16)), b.max_ctx)
         o_lat = torch.empty((b.n_paged, H * m.rank), dtype=p.dtype, device=dev)
         po = torch.empty(b.n_paged * H * splits * m.rank, dtype=torch.float32, device=dev) if splits > 1 else None
         pml = torch.empty(b.n_paged * H * splits * 2, dtype=torch.float32, device=dev) if splits > 1 else None
-        call("rlb_latent_decode", ptr(p), b.n_paged, p.stride(0), p.shape[1], m.q_off, m.mix_off, H, m.dim, m.rot_dim, m.vdim, m.rank, W, bs,
+        call("rlb_latent_decode", ptr(q), b.n_paged, q.stride(0), q.shape[1], m.q_off, ptr(out), out.stride(0), m.mix_off, int(m.gate), H, m.dim, m.rot_dim, m.vdim, m.rank, W, bs,
              cache.shape[0], ptr(cache), ptr(b.block_table), b.block_table.stride(0), ptr(b.seq_lens), ptr(m.kv_up), float(m.scale), ptr(q_lat),
              ptr(o_lat), splits, ptr(po), ptr(pml), st, stream_ptr())
     elif b.n_paged:
-        call("rlb_latent_rows", ptr(p), _f32(p), b.n_paged, p.stride(0), m.q_off, m.mix_off, H, m.dim, m.rot_dim, m.vdim, m.rank, W, bs,
+        call("rlb_latent_rows", ptr(q), _f32(p), b.n_paged, q.stride(0), m.q_off, ptr(out), out.stride(0), m.mix_off, int(m.gate), H, m.dim, m.rot_dim, m.vdim, m.rank, W, bs,
              cache.shape[0], ptr(cache), ptr(b.block_table), b.block_table.stride(0), ptr(b.seq_lens), ptr(m.kv_up), float(m.scale), st, stream_ptr())
     if b.n_paged < T:
         n = b.ctx_slots.numel()
         lat = torch.empty((n, W), dtype=p.dtype, device=dev)
         call("rlb_latent_gather", ptr(cache), ptr(b.ctx_slots), ptr(lat), n, W, cache.shape[0] * bs, st, stream_ptr())
         kv = F.gemm(lat[:, : m.rank], m.kv_up)
-        call("rlb_flash_latent", ptr(p), T, p.stride(0), p.shape[1], b.n_paged, ptr(kv), ptr(lat), n, W, ptr(b.cu_q), ptr(b.cu_ctx),
-             b.cu_q.numel() - 1, H, m.dim, m.rot_dim, m.vdim, m.rank, m.q_off, m.mix_off, float(m.scale), b.q_tiles, st, stream_ptr())
+        call("rlb_flash_latent", ptr(q), T, q.stride(0), q.shape[1], b.n_paged, ptr(kv), ptr(lat), n, W, ptr(b.cu_q), ptr(b.cu_ctx),
+             b.cu_q.numel() - 1, H, m.dim, m.rot_dim, m.vdim, m.rank, m.q_off, ptr(out), out.stride(0), m.mix_off, int(m.gate), float(m.scale),
+             b.q_tiles, st, stream_ptr())
 
 
 def decode_tiles(p: torch.Tensor, m, block_size: int) -> bool:

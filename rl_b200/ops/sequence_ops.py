@@ -1,4 +1,4 @@
-"""Sequence mixers of post-norm layers in the generation engine: grouped-query attention over paged keys and values, and the recurrent
+"""Sequence mixers of post-norm and pre-norm layers in the generation engine: grouped-query attention over paged keys and values, and the recurrent
 mixers with a short convolution (Mamba-2, gated delta rule), over a batch of token rows that mixes single decoded tokens and portions of
 prompts (``mixer_ops.TokenBatch``).
 
@@ -10,6 +10,7 @@ CPU tensors run the plain PyTorch statement.
 from __future__ import annotations
 
 import ctypes as C
+from typing import Optional
 
 import torch
 
@@ -20,10 +21,10 @@ from .lib import F as CF
 from .lib import I, L as LL, P, call, ptr, register, stream_ptr, use_native
 from .mixer_ops import TokenBatch, _f32, _page_rows
 
-register("rlb_gqa_prep", [P, I, LL, LL, I, I, I, I, I, I, I, I, I, P, P, P, P, P, I, CF, CF, P, P, P, P])
-register("rlb_gqa_rows", [P, I, I, LL, I, I, I, I, I, I, I, P, P, P, I, P, CF, P, LL, P, P])
+register("rlb_gqa_prep", [P, I, LL, LL, I, I, I, I, I, I, I, I, I, P, P, P, P, P, I, I, CF, CF, P, LL, P, P, P, P, P])
+register("rlb_gqa_rows", [P, I, I, LL, I, I, I, I, I, I, I, P, P, P, I, P, I, CF, P, LL, P, P])
 register("rlb_gqa_gather", [P, P, P, P, LL, I, I, I, I, LL, P, P])
-register("rlb_flash_gqa", [P, LL, LL, I, I, P, LL, LL, I, I, I, I, P, P, I, I, I, I, I, I, CF, I, P, LL, P, P])
+register("rlb_flash_gqa", [P, LL, LL, I, I, P, LL, LL, I, I, I, I, P, P, I, I, I, I, I, I, I, CF, I, P, LL, P, P])
 register("rlb_conv_rows", [P, I, LL, P, LL, LL, I, I, P, P, P, P, P, P, LL, P, P])
 register("rlb_conv_state", [P, I, LL, I, I, P, I, I, P, P, P, LL, P])
 register("rlb_mamba2_rows", [P, I, LL, P, LL, P, LL, I, I, I, I, I, I, I, I, P, P, P, P, LL, P, P, P, P, P])
@@ -49,13 +50,14 @@ def _rows_out(p: torch.Tensor, m) -> torch.Tensor:
 
 
 # --------------------------------------------------------------------------------------- attention
-def attention(p: torch.Tensor, m, b: TokenBatch, k_cache: torch.Tensor, v_cache: torch.Tensor) -> torch.Tensor:
+def attention(p: torch.Tensor, m, b: TokenBatch, k_cache: torch.Tensor, v_cache: torch.Tensor, first: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``m``: the layer's ``GroupedAttentionMixer``; caches [pages, kv_heads, page size, dim / vdim]. The rows' own keys and values are
-    written first; ``p`` is left with normed and rotated queries and keys."""
+    written first; ``p`` is left with normed and rotated queries and keys. ``first`` [T, kv_heads * vdim]: an earlier layer's values of the
+    rows, of which the layer's own take over a share before they are written."""
     bs, H, G = k_cache.shape[2], m.heads, m.kv_heads
     y = _rows_out(p, m)
     if not use_native(p):
-        q, k, v = m.qkv(p, b.positions)
+        q, k, v = m.qkv(p, b.positions, first)
         ok = b.slots >= 0
         page, off = (b.slots[ok] // bs).long(), (b.slots[ok] % bs).long()
         k_cache[page, :, off], v_cache[page, :, off] = k[ok].to(k_cache.dtype), v[ok].to(v_cache.dtype)
@@ -65,31 +67,33 @@ def attention(p: torch.Tensor, m, b: TokenBatch, k_cache: torch.Tensor, v_cache:
             if n == 0:
                 y[i] = 0
                 continue
-            rows = _page_rows(b.block_table[i], n, bs)
+            rows = _page_rows(b.block_table[i], n, bs)[(n - 1) // m.chunk * m.chunk if m.chunk else 0 :]
             ks, vs = (c[rows // bs, :, rows % bs].float().transpose(0, 1) for c in (k_cache, v_cache))      # [kv_heads, n, dim]
             w = torch.softmax(q[i].view(G, H // G, m.dim) @ ks.transpose(1, 2) * m.scale, dim=-1)
             y[i, : H * m.vdim] = (w @ vs).reshape(-1).to(p.dtype)
         return y
     T, st = p.shape[0], ptr(_L.status_word(p.device))
     call("rlb_gqa_prep", ptr(p), _f32(p), T, p.stride(0), m.q_off, m.k_off, m.v_off, H, G, m.dim, m.vdim, bs, k_cache.shape[0], ptr(b.positions),
-         ptr(b.slots), ptr(m.q_norm), ptr(m.k_norm), ptr(m.freq), m.freq.numel(), float(m.gain), float(m.eps), ptr(k_cache), ptr(v_cache), st, stream_ptr())
+         ptr(b.slots), ptr(m.q_norm), ptr(m.k_norm), ptr(m.freq), m.freq.numel(), int(not m.interleaved), float(m.gain), float(m.eps), ptr(first),
+         first.stride(0) if first is not None else 0, ptr(m.v_share) if first is not None else None, ptr(k_cache), ptr(v_cache), st, stream_ptr())
     if b.n_paged:
         if decode_tiles(p, m, bs):
-            splits = E.choose_splits(b.n_paged, G, max(b.max_ctx // 2, 1), bs)
+            splits = E.choose_splits(b.n_paged, G, max((min(b.max_ctx, m.chunk) if m.chunk else b.max_ctx) // 2, 1), bs)
             E.paged_decode(p[: b.n_paged, m.q_off : m.q_off + H * m.dim], k_cache, v_cache, b.block_table, b.seq_lens, H, G, m.dim, scale=m.scale,
-                           num_splits=splits, out=y[: b.n_paged])
+                           num_splits=splits, out=y[: b.n_paged], chunk=m.chunk)
         else:
             call("rlb_gqa_rows", ptr(p), _f32(p), b.n_paged, p.stride(0), m.q_off, H, G, m.dim, m.vdim, bs, k_cache.shape[0], ptr(k_cache),
-                 ptr(v_cache), ptr(b.block_table), b.block_table.stride(0), ptr(b.seq_lens), float(m.scale), ptr(y), y.stride(0), st, stream_ptr())
+                 ptr(v_cache), ptr(b.block_table), b.block_table.stride(0), ptr(b.seq_lens), m.chunk, float(m.scale), ptr(y), y.stride(0), st, stream_ptr())
     if b.n_paged < T:
-        if b.whole:       # nothing cached before these portions: their keys and values stand in the projected rows
+        cu_ctx, slots, whole = b.chunk_ctx.get(m.chunk, (b.cu_ctx, b.ctx_slots, b.whole))
+        if whole:         # no cached key is visible to these portions: theirs, and their values, stand in the projected rows
             kv, rows, row0, k0, v0 = p, T, b.n_paged, m.k_off, m.v_off
         else:
-            rows, row0, k0, v0 = b.ctx_slots.numel(), 0, 0, G * m.dim
+            rows, row0, k0, v0 = slots.numel(), 0, 0, G * m.dim
             kv = torch.empty((rows, G * (m.dim + m.vdim)), dtype=p.dtype, device=p.device)
-            call("rlb_gqa_gather", ptr(k_cache), ptr(v_cache), ptr(b.ctx_slots), ptr(kv), rows, G, m.dim, m.vdim, bs, k_cache.shape[0] * bs, st, stream_ptr())
+            call("rlb_gqa_gather", ptr(k_cache), ptr(v_cache), ptr(slots), ptr(kv), rows, G, m.dim, m.vdim, bs, k_cache.shape[0] * bs, st, stream_ptr())
         call("rlb_flash_gqa", ptr(p), T, p.stride(0), p.shape[1], b.n_paged, ptr(kv), rows, kv.stride(0), kv.shape[1], row0, k0, v0, ptr(b.cu_q),
-             ptr(b.cu_ctx), b.cu_q.numel() - 1, H, G, m.dim, m.vdim, m.q_off, float(m.scale), b.q_tiles, ptr(y), y.stride(0), st, stream_ptr())
+             ptr(cu_ctx), b.cu_q.numel() - 1, H, G, m.dim, m.vdim, m.q_off, m.chunk, float(m.scale), b.q_tiles, ptr(y), y.stride(0), st, stream_ptr())
     return y
 
 

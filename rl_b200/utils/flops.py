@@ -268,12 +268,32 @@ def redarax_flops(hf, seq: int) -> float:
     return total + head_flops(seq, d, _g(hf, "vocab_size"))
 
 
+def kikivik_flops(hf, seq: int) -> float:
+    """Pre-norm layer-list models: latent attention with a query latent or (chunked) grouped attention, dense or expert gated units."""
+    d, total = _g(hf, "hidden_size"), 0.0
+    for e in _g(hf, "mixers"):
+        m, mlp = e["mixer"], e.get("mlp")
+        H, kd, vd = m["heads"], m["dim"], m["vdim"]
+        if e["type"] == "latent_attention":
+            total += mla_attention_flops(seq, d, H, m["q_rank"], m["kv_rank"], kd, m["rot_dim"], vd)
+        else:      # pairs (query, key) of the causal triangles of the chunks
+            size = min(m["mask"]["size"], seq) if m.get("mask") else seq
+            pairs = (seq // size * size * size + (seq % size) ** 2) / 2
+            total += 2 * seq * d * (H * kd + m["kv_heads"] * (kd + vd) + H * vd) + 2 * pairs * H * (kd + vd)
+        if mlp and mlp.get("kind") == "moe":
+            total += 2 * seq * d * mlp["router"]["experts"] + mlp["router"]["top"] * mlp_flops(seq, d, mlp["expert"]["ff"], gated=True)
+            total += mlp_flops(seq, d, mlp["shared"]["ff"], gated=True) if mlp.get("shared") else 0.0
+        elif mlp:
+            total += mlp_flops(seq, d, mlp["ff"], gated=True)
+    return total + head_flops(seq, d, _g(hf, "vocab_size"))
+
+
 FAMILY_FLOPS = {
     "llama": llama_flops, "mistral": mistral_flops, "qwen2": qwen2_flops, "qwen3": qwen3_flops, "gemma3": gemma3_flops,
     "gemma3_text": gemma3_flops,
     "gpt2": gpt_flops, "gpt3": gpt_flops, "nemotron": nemotron_flops, "mixtral": mixtral_flops, "qwen3_moe": qwen3_moe_flops,
     "qwen2_moe": moe_decoder_flops, "deepseek_v3": deepseek_v3_flops, "deepseek_v2": deepseek_v3_flops, "nemotron_h": nemotron_h_flops,
-    "bert": bert_flops, "gadarax": gadarax_flops, "redarax": redarax_flops,
+    "bert": bert_flops, "gadarax": gadarax_flops, "redarax": redarax_flops, "kikivik": kikivik_flops,
 }
 
 

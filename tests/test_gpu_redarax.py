@@ -12,7 +12,7 @@ from test_redarax import Cfg, standout_case
 from rl_b200.engine.engine import SamplingParams
 from rl_b200.models.config import preset
 from rl_b200.models.mixers import DeltaMixer, GroupedAttentionMixer, Mamba2LayerMixer
-from rl_b200.models.post_norm import ClampedExperts, ClampedGLU
+from rl_b200.models.gated import GatedExperts, GatedUnit
 from rl_b200.models.transformer import build_model
 from rl_b200.ops import layer_ops as Y
 from rl_b200.ops import lib as L
@@ -247,13 +247,13 @@ def test_expert_kernels(spec, width, T):
     h = torch.randn(T, width, dtype=F64).to(BF)
     nw = torch.rand(width) + 0.5
     for dt, tol in ((F32, 1e-4), (BF, 0.02)):
-        m = R.module_weights(ClampedExperts(spec, C2, dt, DEV), w)
+        m = R.module_weights(GatedExperts(spec, C2, dt, DEV), w)
         x = torch.zeros(T, width, device=DEV)
         with torch.no_grad():
             z = Y.router_logits(h.to(DEV, dt), m.router)
             assert torch.allclose(z.double().cpu(), h.double() @ w["router"].T, atol=1e-4)
             Y.feed_forward_(x, h.to(DEV, dt), m, nw.to(DEV, dt), 0.7, 1e-3)
-        ref = ClampedExperts(spec, C2, F32, "cpu")
+        ref = GatedExperts(spec, C2, F32, "cpu")
         R.module_weights(ref, w)
         with torch.no_grad():
             y = ref(h.float()).double()
@@ -305,7 +305,7 @@ def test_joins(d, dt):
 
 
 def test_dense_unit_of_odd_width():
-    m = R.module_weights(ClampedGLU(R.dense(ff=13), Cfg, BF, DEV), {k: v for k, v in O.below(R.weights(R.config([(R.delta(), R.dense(ff=13))]), 1), "l0.mlp.").items()})
+    m = R.module_weights(GatedUnit(R.dense(ff=13), Cfg, BF, DEV), {k: v for k, v in O.below(R.weights(R.config([(R.delta(), R.dense(ff=13))]), 1), "l0.mlp.").items()})
     h = torch.randn(70, 56, device=DEV).to(BF)
     with torch.no_grad():
         assert rel(Y.linear(Y.linear(h, m.gate_up, glu=m.limit), m.down), m(h)) < 1e-2

@@ -14,7 +14,7 @@ from rl_b200.engine.engine import SamplingParams
 from rl_b200.models.config import ModelConfig, preset
 from rl_b200.models.hf_io import load_pretrained, save_pretrained
 from rl_b200.models.mixers import DeltaMixer, GroupedAttentionMixer, Mamba2LayerMixer
-from rl_b200.models.post_norm import ClampedExperts, ClampedGLU, clamped_glu
+from rl_b200.models.gated import GatedExperts, GatedUnit, clamped_glu
 from rl_b200.models.transformer import PackedBatch, build_model
 from rl_b200.ops import layer_ops as Y
 from rl_b200.ops import mixer_ops as X
@@ -107,7 +107,7 @@ def test_clamped_unit_and_its_limits():
     assert torch.allclose(got.double(), want, atol=1e-6) and torch.allclose(clamped_glu(p.float(), 1.5).double(), want, atol=1e-6)
     for spec in (R.dense(), R.dense(ff=9, limit=0.3)):
         w = {k: v.to(F64) for k, v in O.below(R.weights(R.config([(R.delta(), spec)]), 1), "l0.mlp.").items()}
-        m = R.module_weights(ClampedGLU(spec, Cfg, torch.float32, "cpu"), w)
+        m = R.module_weights(GatedUnit(spec, Cfg, torch.float32, "cpu"), w)
         h = torch.randn(30, 56, dtype=F64)
         assert torch.allclose(m(h.float()).double(), O.clamped_glu(w, h, spec["limit"]), atol=2e-5)
         assert torch.allclose(Y.linear(Y.linear(h.float(), m.gate_up, glu=m.limit), m.down).double(), O.clamped_glu(w, h, spec["limit"]), atol=2e-5)
@@ -117,17 +117,17 @@ def test_clamped_unit_and_its_limits():
                                   R.moe(experts=6, top=2, groups=(6, 3)), R.moe(experts=8, top=2, groups=(2, 1))])
 def test_experts_alone(spec):
     w = {k: v.to(F64) for k, v in O.below(R.weights(R.config([(R.delta(), spec)]), 5), "l0.mlp.").items()}
-    m = R.module_weights(ClampedExperts(spec, Cfg, torch.float32, "cpu"), w)
+    m = R.module_weights(GatedExperts(spec, Cfg, torch.float32, "cpu"), w)
     h = torch.randn(60, 56, dtype=F64)
     want = O.experts(w, h, spec)
     assert torch.allclose(m(h.float()).double(), want, atol=3e-5)
-    assert torch.allclose(Y.clamped_experts(h.float(), m)[0].double(), want, atol=3e-5)
+    assert torch.allclose(Y.gated_experts(h.float(), m)[0].double(), want, atol=3e-5)
 
 
 def test_router_masks_groups_with_minus_infinity():
     """All choice scores negative: experts of dropped groups must not win over eligible ones (a mask of 0 would let them)."""
     spec = R.moe(experts=6, top=2, groups=(3, 1))
-    m = ClampedExperts(spec, Cfg, torch.float32, "cpu")
+    m = GatedExperts(spec, Cfg, torch.float32, "cpu")
     m.correction.copy_(torch.tensor([-3.0, -3.0, -2.0, -2.0, -4.0, -1.9]))
     wt, idx = m.choose(torch.zeros(1, 6))
     assert sorted(idx[0].tolist()) == [2, 3] and torch.allclose(wt, torch.full((1, 2), 0.5))
