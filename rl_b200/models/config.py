@@ -608,7 +608,30 @@ def _redarax_preset(width: int, kinds: str, attention: dict, mamba2: dict, delta
                 norm_place="post", residual_mult=0.5, logit_scale=0.5, final_logit_softcap=30.0, token_side={"dim": side} if side else None)
 
 
+def _kikivik_preset(width: int, kinds: str, latent: dict, attention: dict, ff: int, moe: dict, vocab: int) -> dict:
+    """Preset of a pre-norm layer-list model: ``kinds`` has two letters per layer, the mixer (L latent attention, A chunked attention) and the
+    feed-forward (d dense, e experts, - none)."""
+    mix = {"L": ("latent_attention", dict(latent, scale=(latent["dim"] + latent["rot_dim"]) ** -0.5, rot={"dims": latent["rot_dim"], "base": 5e5})),
+           "A": ("attention", dict(attention, scale=attention["dim"] ** -0.5, v_mix=True))}
+    mlp = {"d": {"kind": "dense", "ff": ff, "limit": 7.0}, "e": dict(moe, kind="moe"), "-": None}
+    layers = [{"type": mix[k][0], "mixer": mix[k][1], "mlp": mlp[f]} for k, f in zip(kinds[::2], kinds[1::2])]
+    m0 = layers[0]["mixer"]
+    return dict(model_type="kikivik", vocab_size=vocab, hidden_size=width, num_hidden_layers=len(layers), intermediate_size=max(ff, moe["expert"]["ff"]),
+                num_attention_heads=m0["heads"], num_key_value_heads=m0["heads"], head_dim=m0["dim"], rms_norm_eps=1e-6, mixers=layers,
+                embed_scale=2.0, traits=KIKIVIK_TRAITS)
+
+
 PRESETS: dict[str, dict] = {
+    # Kikivik at the size of small production models: latent and chunked attention layers, dense and expert feed-forwards
+    "kikivik-2b": _kikivik_preset(2048, "AdLeLdAeLeLdAeLe", dict(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=768),
+                                  dict(heads=16, kv_heads=4, dim=128, vdim=128, mask={"size": 1024}, rot={"dims": 128, "base": 1e6, "scaling": {"factor": 4.0}}),
+                                  6144, dict(expert={"ff": 768}, router={"experts": 64, "top": 8}, shared={"ff": 768}), 65536),
+    "kikivik-7b": _kikivik_preset(4096, "AdLeLdAeLeLdAeLe", dict(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=1536),
+                                  dict(heads=32, kv_heads=8, dim=128, vdim=128, mask={"size": 1024}, rot={"dims": 128, "base": 1e6, "scaling": {"factor": 4.0}}),
+                                  12288, dict(expert={"ff": 1536}, router={"experts": 64, "top": 8}, shared={"ff": 1536}), 65536),
+    "tiny-kikivik": _kikivik_preset(96, "AeLdAdL-", dict(heads=3, dim=16, rot_dim=8, vdim=24, kv_rank=40, q_rank=48),
+                                    dict(heads=4, kv_heads=2, dim=24, vdim=16, mask={"size": 20}, rot={"dims": 16, "base": 1e4, "scaling": {"factor": 2.0}}),
+                                    160, dict(expert={"ff": 48}, router={"experts": 8, "top": 2}, shared={"ff": 40}), 264),
     # Redarax at the size of small production models: delta-rule, Mamba-2 and grouped-query attention layers, dense and expert feed-forwards
     "redarax-2b": _redarax_preset(2048, "DdDeMeAeDdDeMeAe", dict(heads=16, kv_heads=4, dim=128, vdim=128, rot={"dims": 64, "base": 1e6}),
                                   dict(heads=32, vdim=128, state=128, groups=4, norm_groups=4, conv=4), dict(heads=16, kv_heads=8, dim=128, vdim=128, conv=4),
