@@ -5,6 +5,7 @@
     python bench.py --config refit-sweep --gpus 8            (weight re-shard times, trainer layout -> serving layouts)
     python bench.py --config gadarax-serving                 (prefill / decode of a layer-list model beside Llama at equal size)
     python bench.py --config redarax-serving                 (the same for a post-norm layer-list model, beside Qwen3-MoE)
+    python bench.py --config kikivik-serving                 (the same for a pre-norm layer-list model, beside Qwen3-MoE)
     python bench.py --impl reference ...                     (the unmodified reference, when it can be installed)
 
 Default (headline) configuration ``llama8b-dp``: one GRPO step (generation + refit + log-probabilities + training) on
@@ -51,6 +52,7 @@ CONFIGS = {
     "refit-sweep": dict(),
     "gadarax-serving": dict(),
     "redarax-serving": dict(),
+    "kikivik-serving": dict(),
 }
 
 
@@ -173,12 +175,12 @@ def main() -> int:
 
         return sweep_main(steps=args.steps, warmup=args.warmup)
 
-    if args.config in ("gadarax-serving", "redarax-serving"):
+    if args.config in ("gadarax-serving", "redarax-serving", "kikivik-serving"):
         from rl_b200.csrc.build import build_all
         from rl_b200.engine import bench_mixers
         from rl_b200.ops import lib as L
 
-        serving_main = bench_mixers.main if args.config == "gadarax-serving" else bench_mixers.redarax_main
+        serving_main = {"gadarax-serving": bench_mixers.main, "redarax-serving": bench_mixers.redarax_main, "kikivik-serving": bench_mixers.kikivik_main}[args.config]
 
         if not L.available():
             build_all()

@@ -436,7 +436,8 @@ RLB_API int rlb_group_norm_rows(void* y, long long ldy, int f32, const void* w, 
   if (f32)
     return static_cast<int>(rlb_launch_pdl(group_norm_rows_kernel<float>, grid, dim3(256), 0, s, static_cast<float*>(y), ldy, static_cast<const float*>(w),
                                            groups, n, eps));
-  if (n % 8 == 0 && n <= 2048 && ldy % 8 == 0 && !((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(w)) & 15)) {
+  const bool few = rows * groups < 148 * 2 && n >= 256;      // few parts: a CTA each
+  if (!few && n % 8 == 0 && n <= 2048 && ldy % 8 == 0 && !((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(w)) & 15)) {
     const long long parts = rows * groups;
     return static_cast<int>(rlb_launch_pdl(group_norm_warp_kernel, dim3(static_cast<unsigned>((parts + 7) / 8)), dim3(256), 0, s,
                                            static_cast<__nv_bfloat16*>(y), ldy, static_cast<const __nv_bfloat16*>(w), parts, groups, n, eps));

@@ -61,6 +61,59 @@ __global__ void embed_rows_kernel(const void* ids, int ids64, const T* __restric
   for (int c = threadIdx.x; c < d; c += blockDim.x) st(h + row * d + c, x[row * d + c] * rstd * ld(nw + c));     // (each thread reads what it wrote)
 }
 
+// The same without a loop's copies and steps, d a multiple of 4 and at most 4 * EM_KEEP * EM_THREADS: h = x, or x / rms(x) * w. A thread keeps its
+// columns in registers, all loads are issued before the first is used.
+constexpr int EM_THREADS = 512, EM_KEEP = 4;
+__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 ld4(const __nv_bfloat16* p) {
+  const uint2 r = *reinterpret_cast<const uint2*>(p);
+  const float2 a = unpack_bf16x2(r.x), b = unpack_bf16x2(r.y);
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void st4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void st4(__nv_bfloat16* p, float4 v) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+}
+template <typename T>
+__global__ void __launch_bounds__(EM_THREADS)
+embed_wide_kernel(const void* ids, int ids64, const T* __restrict__ table, float* __restrict__ x, T* __restrict__ h, const T* __restrict__ nw, int d,
+                  int vocab, float scale, float eps, int* status) {
+  __shared__ float red[32];
+  const long long row = blockIdx.x;
+  const int n = blockDim.x;
+  float4 w[EM_KEEP], v[EM_KEEP];
+#pragma unroll
+  for (int i = 0; i < EM_KEEP; ++i) {
+    const int c = (threadIdx.x + i * n) * 4;
+    w[i] = nw && c < d ? ld4(nw + c) : make_float4(1.f, 1.f, 1.f, 1.f);
+  }
+  long long id = ids64 ? static_cast<const long long*>(ids)[row] : static_cast<const int*>(ids)[row];
+  if (id < 0 || id >= vocab) {
+    if (threadIdx.x == 0 && status) atomicCAS(status, 0, RLB_ERR_BOUNDS);
+    id = 0;
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < EM_KEEP; ++i) {
+    const int c = (threadIdx.x + i * n) * 4;
+    v[i] = c < d ? ld4(table + id * d + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+#pragma unroll
+  for (int i = 0; i < EM_KEEP; ++i) {
+    const int c = (threadIdx.x + i * n) * 4;
+    v[i] = make_float4(v[i].x * scale, v[i].y * scale, v[i].z * scale, v[i].w * scale);
+    ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    if (c < d) st4(x + row * d + c, v[i]);
+  }
+  float f = 1.f;
+  if (nw) f = 1.f / sqrtf(block_sum(ss, red) / static_cast<float>(d) + eps);
+#pragma unroll
+  for (int i = 0; i < EM_KEEP; ++i) {
+    const int c = (threadIdx.x + i * n) * 4;
+    if (c < d) st4(h + row * d + c, make_float4(v[i].x * f * w[i].x, v[i].y * f * w[i].y, v[i].z * f * w[i].z, v[i].w * f * w[i].w));
+  }
+}
+
 // ---------------------------------------------------------------- product with the layer epilogues
 struct RowsGemm {
   const void* a;
@@ -480,6 +533,17 @@ RLB_API int rlb_embed_rows(const void* ids, int ids64, const void* table, int f3
                            void* stream) {
   if (rows <= 0) return 0;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (!e && !step && !alpha && d % 4 == 0 && d <= 4 * EM_KEEP * EM_THREADS) {
+    const int threads = d > 4096 ? EM_THREADS : (d > 1024 ? 256 : 128);
+    if (f32)
+      embed_wide_kernel<float><<<static_cast<unsigned>(rows), threads, 0, s>>>(ids, ids64, static_cast<const float*>(table), x, static_cast<float*>(h),
+                                                                               static_cast<const float*>(nw), d, vocab, scale, eps, status);
+    else
+      embed_wide_kernel<__nv_bfloat16><<<static_cast<unsigned>(rows), threads, 0, s>>>(ids, ids64, static_cast<const __nv_bfloat16*>(table), x,
+                                                                                       static_cast<__nv_bfloat16*>(h), static_cast<const __nv_bfloat16*>(nw), d,
+                                                                                       vocab, scale, eps, status);
+    return static_cast<int>(cudaGetLastError());
+  }
   if (f32)
     embed_rows_kernel<float><<<static_cast<unsigned>(rows), 256, 0, s>>>(ids, ids64, static_cast<const float*>(table), x, e, static_cast<float*>(h),
         static_cast<const float*>(step), static_cast<const float*>(alpha), static_cast<const float*>(nw), static_cast<const float*>(nb), d, vocab, scale, eps, status);

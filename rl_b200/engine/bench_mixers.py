@@ -1,7 +1,7 @@
-"""Serving throughput of layer-list models beside the framework's closest model at equal size (Gadarax: the Llama architecture, Redarax:
-Qwen3-MoE), and the kernels' distance from their rooflines beside the like kernels of the closest path.
+"""Serving throughput of layer-list models beside the framework's closest model at equal size (Gadarax: the Llama architecture, Redarax and
+Kikivik: Qwen3-MoE), and the kernels' distance from their rooflines beside the like kernels of the closest path.
 
-    python bench.py --config gadarax-serving | redarax-serving [--steps K --warmup W]
+    python bench.py --config gadarax-serving | redarax-serving | kikivik-serving [--steps K --warmup W]
 
 Random weights, random prompts. Whole-model figures come from ``GenerationEngine``: prefill of packed prompts (device time of the
 forward pass) and decoding through the captured step (device time of the graph replays). Kernel figures are CUDA-event times of a
@@ -29,6 +29,7 @@ SIZES = {   # (preset, Llama twin: same width and run count, MHA with 128-wide h
     "gadarax-4b": dict(hidden_size=4096, num_attention_heads=32),
 }
 REDARAX = ("redarax-2b", "redarax-7b")
+KIKIVIK = ("kikivik-2b", "kikivik-7b")
 PREFILL = ((1, 4096), (8, 1024))      # (prompts, tokens each)
 DECODE = ((16, 4096), (64, 2048))     # (sequences, context)
 
@@ -406,6 +407,132 @@ def redarax_table(name: str) -> list:
                     2.0 * T * m.heads * (C / 2 * (m.dim + m.vdim) + 2 * m.dim * m.vdim), nb)
                 del sets
     return out
+
+
+def kikivik_table(name: str) -> list:
+    """``kernel_table`` of a pre-norm layer-list preset. The like kernels are those of the layer-list models that it is closest to: latent
+    attention with an output gate and plain queries, causal grouped attention with biases, clamped experts without a shared unit, normed joins;
+    and flash and paged decode attention of the plain models."""
+    from rl_b200.models.gated import GatedExperts
+    from rl_b200.models.mixers import GroupedAttentionMixer, LatentAttentionMixer
+    from rl_b200.ops import layer_ops as Y
+    from rl_b200.ops import sequence_ops as S
+
+    pk, c, dev, bf = peaks(), preset(name), "cuda", torch.bfloat16
+    model = build_model(c, device=dev, dtype=bf, seed=0)
+    la, at = (next(l for l in model.layers if l.mixer.kind == kind) for kind in ("latent_attention", "attention"))
+    glu = next(l.ff for l in model.layers if l.ff is not None and not hasattr(l.ff, "router"))
+    moe = next(l.ff for l in model.layers if hasattr(l.ff, "router"))
+    d, out = c.hidden_size, []
+
+    def add(label, ms, flops=0.0, nbytes=0.0):
+        roof = max(flops / pk["flops"], nbytes / pk["hbm"]) * 1e3
+        out.append(dict(kernel=label, ms=round(ms, 4), roofline_ms=round(roof, 4), fraction=round(roof / ms, 3)))
+
+    rows = lambda T, n: torch.randn(T, n, device=dev).to(bf)   # noqa: E731
+    with torch.no_grad():
+        m, g = la.mixer, at.mixer
+        for T in (64, 4096):
+            # products with what follows them
+            for label, w, unit in (("latent in_proj", m.in_proj, None), ("query up-projection", m.q_up, None), ("latent out_proj", m.out_proj, None),
+                                   ("attention in_proj", g.in_proj, None), ("gate_up + clamped unit", glu.gate_up, glu), ("gate_up + silu unit", moe.shared.gate_up, moe.shared)):
+                N, K = w.shape
+                nb = 2 * (N * K + T * (K + (N if unit is None else N // 2)))
+                sets = copies(lambda: (rows(T, K), w.detach().clone()), nb)
+                fn = Y.linear if unit is None else lambda a, b, unit=unit: Y.gated_linear(a, b, unit.limit)
+                add(f"{label} [{N} x {K}], {T} rows", timed_graph([lambda s=s: fn(s[0], s[1]) for s in sets]), 2.0 * T * N * K, nb)
+                add("like: plain GEMM", timed_graph([lambda s=s: F.gemm(s[0], s[1]) for s in sets]), 2.0 * T * N * K, 2 * (N * K + T * (N + K)))
+                del sets
+            # joins, norms, the start
+            sets = copies(lambda: (torch.randn(T, d, device=dev), rows(T, d), rows(T, d)), 12 * T * d)
+            add(f"join: x += y, next norm, {T} rows", timed_graph([lambda s=s: Y.add_normed_(s[0], s[1], None, 1.0, 1e-6, la.norm1) for s in sets]), 0.0, 12 * T * d)
+            add("like: normed join", timed_graph([lambda s=s: Y.add_normed_(s[0], s[1], la.norm1, 0.5, 1e-6) for s in sets]), 0.0, 12 * T * d)
+            ids = torch.randint(0, c.vocab_size, (T,), device=dev, dtype=torch.int32)
+            add(f"embedding + first norm, {T} rows", timed_graph([lambda: Y.embed(ids, model.embed_tokens, 2.0, la.norm1, 1e-6) for _ in range(8)]), 0.0, 8 * T * d)
+            add("like: embedding", timed_graph([lambda: Y.embed(ids, model.embed_tokens, 2.0) for _ in range(8)]), 0.0, 8 * T * d)
+            sets = copies(lambda: rows(T, m.in_width), 4 * T * m.q_rank)
+            add(f"query latent norm, {T} rows", timed_graph([lambda s=s: Y.group_norm_(s, m.q_norm, 1, 1e-6) for s in sets]), 0.0, 4 * T * m.q_rank)
+            add("like: RMS norm", timed_graph([lambda s=s: F.rmsnorm(s[:, : m.q_rank], m.q_norm, 1e-6) for s in sets]), 0.0, 4 * T * m.q_rank)
+            del sets
+            # experts
+            sh = moe.shared
+            like = GatedExperts(dict(router={"experts": moe.experts, "top": moe.top, "groups": {"count": 8, "keep": 4}}, expert={"ff": moe.ff, "limit": 7.0}), c, bf, dev)
+            for prm in like.parameters():
+                prm.normal_(std=0.02)
+            used = min(moe.experts, T * moe.top)
+            nb = 2 * (3 * used * d * moe.ff + T * moe.top * (2 * d + 2 * moe.ff)) + 12 * T * d
+            fl = 6.0 * T * moe.top * d * moe.ff
+            nbs, fls = 2 * (3 * d * sh.ff + T * (d + 2 * sh.ff)), 6.0 * T * d * sh.ff
+            sets = copies(lambda: (torch.randn(T, d, device=dev), rows(T, d)), 16 * T * d)
+            ms = timed_graph([lambda s=s: Y.feed_forward_(s[0], s[1], moe, None, 1.0, 1e-6, la.norm1) for s in sets[:4]])
+            add(f"experts with router, shared unit and join (all kernels), {T} rows", ms, fl + fls, nb + nbs)
+            ms = timed_graph([lambda s=s: Y.feed_forward_(s[0], s[1], like, la.norm1, 0.5, 1e-6) for s in sets[:4]])
+            add("like: clamped experts with router and join", ms, fl, nb)
+            del sets, like
+        # chunked attention beside causal attention over as many keys as a query sees here
+        C = g.chunk
+        H, G = g.heads, g.kv_heads
+        twin = GroupedAttentionMixer(dict(heads=H, kv_heads=G, dim=g.dim, vdim=g.vdim, scale=g.scale, rot={"dims": g.dim, "base": 1e6}), c, bf, dev)
+        for n, ctx in DECODE:
+            for label, mx, seen in (("chunked attention", g, ctx - (ctx - 1) // C * C), ("like: causal attention", twin, C)):
+                b = rows_batch(n, ctx if mx is g else seen)
+                nb, pages = n * seen * G * (g.dim + g.vdim) * 2, n * ctx // 64
+                sets = copies(lambda: (rows(n, mx.in_width), *(torch.randn(pages, G, 64, w, device=dev).to(bf) for w in (g.dim, g.vdim)), rows(n, G * g.vdim)), nb)
+                add(f"{label} decode (all kernels), {n} rows, {seen} keys seen", timed_graph([lambda s=s: S.attention(s[0], mx, b, s[1], s[2], s[3] if mx.v_mix else None) for s in sets]),
+                    4.0 * n * seen * H * g.dim, nb)
+                if mx is twin:
+                    sp = E.choose_splits(n, G, seen // 2, 64)
+                    add("like: paged decode attention", timed_graph([lambda s=s: E.paged_decode(s[0][:, : H * g.dim], s[1], s[2], b.block_table, b.seq_lens, H, G, g.dim, num_splits=sp)
+                                                                     for s in sets]), 4.0 * n * seen * H * g.dim, nb)
+                del sets
+        for n, length in PREFILL:
+            for label, mx, per in (("chunked attention", g, min(C, length)), ("like: causal attention", twin, length)):
+                b, T = portion_batch(n, length), n * length
+                kc, vc = (torch.zeros((T // 64, G, 64, w), dtype=bf, device=dev) for w in (g.dim, g.vdim))
+                nb = 2 * T * (mx.in_width + mx.mix_width + G * (g.dim + g.vdim))
+                sets = copies(lambda: (rows(T, mx.in_width), rows(T, G * g.vdim)), nb)
+                add(f"{label} prefill (all kernels), {n} x {length}", timed_graph([lambda s=s: S.attention(s[0], mx, b, kc, vc, s[1] if mx.v_mix else None) for s in sets]),
+                    2.0 * T * per / 2 * H * (g.dim + g.vdim), nb)
+                if mx is twin:      # over sequences of a chunk's length
+                    cu = torch.arange(0, T + 1, min(C, length), dtype=torch.int32, device=dev)
+                    add(f"like: flash attention, {T // min(C, length)} x {min(C, length)}", timed_graph([lambda s=s: F.attention_varlen(s[0], cu, min(C, length), H, G, g.dim) for s in sets]),
+                        2.0 * T * min(C, length) / 2 * H * (g.dim + g.vdim), nb)
+                del sets
+        # latent attention: queries through their latent, no gate, beside gated latent attention whose queries stand in the projected rows
+        gated = LatentAttentionMixer(dict(heads=m.heads, dim=m.dim, rot_dim=m.rot_dim, vdim=m.vdim, kv_rank=m.rank, scale=m.scale, rot={"dims": m.rot_dim, "base": 5e5}), c, bf, dev)
+        gated.kv_up.normal_(std=0.02)
+        qb = m.q_up.numel() * 2
+        for n, ctx in DECODE:
+            b = rows_batch(n, ctx)
+            nb, fl = n * ctx * m.latent_width * 2 + m.kv_up.numel() * 2, 2.0 * n * ctx * m.heads * (2 * m.rank + m.rot_dim)
+            sets = copies(lambda: (rows(n, m.in_width), torch.randn(n * ctx // 64, 64, m.latent_width, device=dev).to(bf), rows(n, gated.in_width)), nb)
+            add(f"latent attention decode with query up-projection (all kernels), {n} x {ctx}", timed_graph([lambda s=s: X.latent_attention(s[0], m, b, s[1]) for s in sets]), fl, nb + qb)
+            add("like: gated latent attention decode", timed_graph([lambda s=s: X.latent_attention_(s[2], gated, b, s[1]) for s in sets]), fl, nb)
+            del sets
+        for n, length in PREFILL:
+            b, T = portion_batch(n, length), n * length
+            pairs = n * length * length / 2
+            cache = torch.zeros((T // 64, 64, m.latent_width), dtype=bf, device=dev)
+            fl = 2.0 * pairs * m.heads * (m.dim + m.rot_dim + m.vdim) + 2.0 * T * m.kv_up.numel()
+            nb = 2 * T * (m.in_width + m.q_up.shape[0] + m.mix_width + 2 * m.heads * (m.dim + m.vdim))
+            sets = copies(lambda: (rows(T, m.in_width), rows(T, gated.in_width)), nb)
+            add(f"latent attention prefill with query up-projection (all kernels), {n} x {length}", timed_graph([lambda s=s: X.latent_attention(s[0], m, b, cache) for s in sets]),
+                fl + 2.0 * T * m.q_up.numel(), nb)
+            add("like: gated latent attention prefill", timed_graph([lambda s=s: X.latent_attention_(s[1], gated, b, cache) for s in sets]), fl, nb)
+            del sets
+    return out
+
+
+def kikivik_main(steps: int = 5, warmup: int = 3, sizes=None, clocks=None) -> int:
+    torch.backends.cuda.matmul.allow_tf32 = False
+    L.lib()
+    res = dict(metric="pre-norm layer-list model serving (device time)", unit="tokens/s", dtype="bf16", data="synthetic (random weights and tokens)", models={}, kernels={})
+    for name in sizes or KIKIVIK:
+        for kind in ("kikivik", "qwen3_moe"):
+            res["models"][f"{name}:{kind}"] = serving_row(preset(name) if kind == "kikivik" else moe_twin(name), steps, warmup)
+        res["kernels"][name] = kikivik_table(name)
+        torch.cuda.empty_cache()
+    return finish(res, clocks)
 
 
 def redarax_main(steps: int = 5, warmup: int = 3, sizes=None, clocks=None) -> int:
