@@ -5,11 +5,13 @@ One dataclass covers Llama (2/3/3.1/3.2), Mistral, Qwen2/2.5, Qwen3, Qwen3-MoE a
 before and after each block, scaled embeddings, sliding-window layers with their own RoPE base, a fixed attention scale). ``from_hf_dict`` reads a
 HuggingFace ``config.json`` dictionary; ``PRESETS`` names the architectures used by the benchmark configs.
 
-Models described layer by layer (Gadarax, Redarax, Kikivik) keep their layer list in ``mixers``: each entry names the sequence mixer, its sizes
+Models described layer by layer (Gadarax, Redarax, Kikivik, Zonidra) keep their layer list in ``mixers``: each entry names the sequence mixer, its sizes
 and its MLP. ``LAYER_LISTS`` says which mixers and MLPs each architecture has and how its configuration maps to ``ModelConfig``:
 Gadarax runs mixer and MLP side by side behind one norm (``layer_loop`` repeats a range of layers with the same weights), Redarax runs
 them one after the other and norms what they return (``norm_place`` "post"), with an input per layer and token (``token_side``), Kikivik
-runs them one after the other on norms of the residual stream. What an architecture fixes for all its mixers of a kind (biases, gates, the
+runs them one after the other on norms of the residual stream, Zonidra does that and norms and scales what they return as well
+(``norm_place`` "both", ``layer_scale``), its mixers read a blend with the token before (``token_shift``) and its embedding has a second
+table over pairs of tokens (``bigram``). What an architecture fixes for all its mixers of a kind (biases, gates, the
 layout of rotated pairs) is in ``traits`` and joins each layer's sizes (``mixer_spec``, ``mlp_spec``).
 """
 
@@ -97,13 +99,16 @@ class ModelConfig:
     moe_latent_size: Optional[int] = None      # routed experts work in a narrower space between two shared projections
     moe_shared_expert_intermediate_size: int = 0
 
-    # models described layer by layer (Gadarax, Redarax, Kikivik): the layers differ in their mixers, sizes and MLPs
+    # models described layer by layer (Gadarax, Redarax, Kikivik, Zonidra): the layers differ in their mixers, sizes and MLPs
     mixers: Optional[list] = None      # per layer: {"type": name of the mixer, "mixer": {sizes}, "mlp": {"kind", sizes} or None}
     layer_loop: Optional[dict] = None  # {"start", "stop", "times"}: layers start .. stop - 1 run `times` times in a row with the same weights
     norm_kind: str = "rms"             # "rms" | "dyt" (dynamic tanh: w * tanh(alpha x) + b, no statistics)
-    norm_place: str = "pre"            # "pre": sublayers read norm(x); "post": they read x, and norm(output) joins the residual stream
+    norm_place: str = "pre"            # "pre": sublayers read norm(x); "post": they read x, and norm(output) joins the residual stream; "both"
     residual_mult: float = 1.0         # what sublayer outputs are multiplied by when they join the residual stream
     token_side: Optional[dict] = None  # {"dim"}: every layer adds an input looked up by token in a table of its own (gated by the stream)
+    layer_scale: bool = False          # sublayer outputs are multiplied element by element when they join the residual stream
+    token_shift: bool = False          # mixers read h + (h of the token before - h) * s, element by element
+    bigram: Optional[dict] = None      # {"buckets", "mul_prev", "mul_cur"}: embeddings get a row looked up by (token before, token)
     logit_scale: float = 1.0           # logits are multiplied by this (before the soft cap)
     traits: dict = field(default_factory=dict)   # kind of mixer or MLP: what the architecture fixes for it, in the words of its class
 
@@ -129,8 +134,8 @@ class ModelConfig:
 
     @property
     def is_recurrent(self) -> bool:
-        """Some layer carries a per-sequence state beside (or instead of) cache pages: prefixes cannot be shared by pages."""
-        return self.is_hybrid or (self.mixers is not None and any(m["type"] in RECURRENT_MIXERS for m in self.mixers))
+        """The model carries a per-sequence state beside (or instead of) cache pages: prefixes cannot be shared by pages."""
+        return self.is_hybrid or self.token_shift or bool(self.bigram) or (self.mixers is not None and any(m["type"] in RECURRENT_MIXERS for m in self.mixers))
 
     @property
     def caps_logits(self) -> bool:
@@ -225,6 +230,19 @@ class ModelConfig:
                 elif mlp:
                     n += d + 3 * d * mlp["ff"]
             return n
+        if self.model_type == "zonidra":
+            n = 2 * self.vocab_size * d + d + ((self.bigram["buckets"] + 1) * d if self.bigram else 0)
+            for e in self.mixers:
+                m, mlp = e["mixer"], e.get("mlp")
+                H, kd, vd = m["heads"], m["dim"], m["vdim"]
+                n += d * (H * kd + 2 * H * vd + (m["kv_heads"] * (kd + vd) if m.get("kv_from") is None else 0)) + H + 4 * d
+                if mlp and mlp["kind"] == "moe":
+                    r, sh = mlp["router"], mlp.get("shared")
+                    n += r["experts"] * 3 * d * mlp["expert"]["ff"] + (r["experts"] + r.get("identity", 0)) * (d + 1) + (3 * d * sh["ff"] + d if sh else 0)
+                elif mlp:
+                    n += 2 * d * mlp["ff"] + 4
+                n += 3 * d if mlp else 0
+            return n
         if self.mixers is not None:
             n = self.vocab_size * d + 2 * d + 1 + (self.layer_loop["times"] * d if self.layer_loop else 0)
             for e in self.mixers:
@@ -259,6 +277,10 @@ class ModelConfig:
         if self.model_type == "kikivik":
             return {"architecture": "Kikivik", "vocab": self.vocab_size, "width": self.hidden_size, "embedding": {"scale": self.embed_scale},
                     "norm": {"eps": self.rms_norm_eps}, "layers": self.mixers, "torch_dtype": self.torch_dtype}
+        if self.model_type == "zonidra":
+            emb = {"scale": self.embed_scale, **({"bigram": self.bigram} if self.bigram else {})}
+            return {"architecture": "Zonidra", "vocab": self.vocab_size, "width": self.hidden_size, "embedding": emb,
+                    "norm": {"eps": self.rms_norm_eps}, "layers": self.mixers, "torch_dtype": self.torch_dtype}
         if self.model_type == "redarax":
             out = {"architecture": "Redarax", "vocab": self.vocab_size, "width": self.hidden_size, "norm": {"eps": self.rms_norm_eps},
                    "residual_mult": self.residual_mult, "logit_scale": self.logit_scale, "layers": self.mixers, "torch_dtype": self.torch_dtype}
@@ -274,7 +296,7 @@ class ModelConfig:
                 "gemma3_text": "Gemma3ForCausalLM", "deepseek_v3": "DeepseekV3ForCausalLM",
                 "nemotron_h": "NemotronHForCausalLM"}.get(self.model_type, "LlamaForCausalLM")
         d = asdict(self)
-        for k in ("mixers", "layer_loop", "norm_kind", "norm_place", "residual_mult", "token_side", "logit_scale", "traits"):
+        for k in ("mixers", "layer_loop", "norm_kind", "norm_place", "residual_mult", "token_side", "layer_scale", "token_shift", "bigram", "logit_scale", "traits"):
             d.pop(k)
         nh = {k: d.pop(k) for k in ("layers_block_type", "use_rope", "mlp_gated", "mlp_bias", "mamba_num_heads", "mamba_head_dim", "ssm_state_size",
                                     "mamba_n_groups", "mamba_d_conv", "mamba_chunk_size", "mamba_conv_bias", "mamba_proj_bias", "mamba_dt_limit",
@@ -441,8 +463,10 @@ class ModelConfig:
             if e.get("mlp") and e["mlp"].get("kind") == "moe":
                 r = e["mlp"]["router"]
                 g = r.get("groups") or {"count": 1, "keep": 1}
-                if r["experts"] % g["count"] or not 1 <= g["keep"] <= g["count"] or not 1 <= r["top"] <= g["keep"] * (r["experts"] // g["count"]):
+                n = r["experts"] + r.get("identity", 0)
+                if n % g["count"] or not 1 <= g["keep"] <= g["count"] or not 1 <= r["top"] <= g["keep"] * (n // g["count"]):
                     raise ValueError(f"layer {i}: router {r} does not fit its groups")
+            _check_source(i, layers)
         mixing = {(e["mixer"]["kv_heads"], e["mixer"]["vdim"]) for e in layers if e["type"] == "attention" and e["mixer"].get("v_mix")}
         if len(mixing) > 1:
             raise ValueError(f"layers that mix their values have unequal (key / value heads, value sizes): {sorted(mixing)}")
@@ -494,8 +518,21 @@ def _check_mixer(i: int, kind: str, m: dict) -> None:
         raise ValueError(f"layer {i}: {m['heads'] * m['vdim']} channels do not divide into {m['norm_groups']} norm groups")
     if m.get("conv", 1) < 1:
         raise ValueError(f"layer {i}: a convolution needs at least one tap")
-    if m.get("mask") and m["mask"]["size"] < 1:
-        raise ValueError(f"layer {i}: chunks of {m['mask']['size']} positions")
+    if m.get("mask") and (m["mask"]["size"] < 1 or m["mask"].get("keep_first", 0) < 0):
+        raise ValueError(f"layer {i}: mask {m['mask']}")
+
+
+def _check_source(i: int, layers: list) -> None:
+    """A layer that reads another layer's keys and values comes behind it and has its key / value heads and sizes."""
+    m = layers[i]["mixer"]
+    j = m.get("kv_from")
+    if j is None:
+        return
+    if not 0 <= j < i or layers[j]["type"] != "attention" or layers[j]["mixer"].get("kv_from") is not None:
+        raise ValueError(f"layer {i}: layer {j} has no keys and values to share")
+    unequal = [k for k in ("kv_heads", "dim", "vdim") if m.get(k) != layers[j]["mixer"].get(k)]
+    if unequal:
+        raise ValueError(f"layer {i}: {unequal} differ from those of layer {j}, whose keys and values it reads")
 
 
 def _ff_width(mlp: dict) -> int:
@@ -519,10 +556,21 @@ def _kikivik(hf: dict) -> dict:
     return dict(model_type="kikivik", embed_scale=float(hf["embedding"]["scale"]), traits=KIKIVIK_TRAITS)
 
 
+ZONIDRA_TRAITS = {"attention": {"bias": False, "qk_norm": False, "interleaved": False, "gate": True, "weights": "sigmoid", "mask_kind": "window"},
+                  "dense": {"act": "poly"}, "moe": {"score": "softmax", "shared_gate": True}}
+
+
+def _zonidra(hf: dict) -> dict:
+    big = hf["embedding"].get("bigram")
+    return dict(model_type="zonidra", embed_scale=float(hf["embedding"]["scale"]), norm_place="both", layer_scale=True, token_shift=True,
+                bigram={k: int(big[k]) for k in ("buckets", "mul_prev", "mul_cur")} if big else None, traits=ZONIDRA_TRAITS)
+
+
 # architecture -> (its mixers, its kinds of MLP, configuration -> further ModelConfig fields)
 LAYER_LISTS = {"Gadarax": (("latent_attention", "retention"), ("dense",), _gadarax),
                "Redarax": (("attention", "mamba2", "delta"), ("dense", "moe"), _redarax),
-               "Kikivik": (("latent_attention", "attention"), ("dense", "moe"), _kikivik)}
+               "Kikivik": (("latent_attention", "attention"), ("dense", "moe"), _kikivik),
+               "Zonidra": (("attention",), ("dense", "moe"), _zonidra)}
 
 
 def rope_inv_freq(cfg: ModelConfig, device=None) -> torch.Tensor:
@@ -562,7 +610,9 @@ def rope_inv_freq(cfg: ModelConfig, device=None) -> torch.Tensor:
 
 def rotary_table(rot: dict) -> tuple[torch.Tensor, float]:
     """Angle per position of each rotated pair [dims / 2] (fp32) and the factor on cosine and sine, for a rotation described by
-    ``{"dims", "base"}`` and optionally ``"scaling"``: ``{"factor"}`` alone slows every pair down by ``factor``, YaRN's ``{"factor",
+    ``{"dims", "base"}`` and optionally ``"scaling"``: ``{"factor"}`` alone slows every pair down by ``factor``, Llama 3.1's ``{"factor",
+    "original", "low", "high"}`` keeps pairs that turn more than ``high`` times within the original context, slows down by ``factor`` those that
+    turn less than ``low`` times and mixes the two linearly in the turns between them, YaRN's ``{"factor",
     "original", "fast", "slow"}`` keeps the frequency of pairs that turn more than ``fast`` times within the original context and slows
     down by ``factor`` those that turn less than ``slow`` times, with a linear ramp between the two (upper end clamped at the last
     dimension)."""
@@ -574,6 +624,11 @@ def rotary_table(rot: dict) -> tuple[torch.Tensor, float]:
     factor = float(s["factor"])
     if "original" not in s:
         return (f / factor).float(), 1.0
+
+    if "low" in s:
+        turns, lo, hi = float(s["original"]) * f / (2 * math.pi), float(s["low"]), float(s["high"])
+        t = ((turns - lo) / (hi - lo)).clamp(0, 1) if hi > lo else (turns >= lo).double()
+        return ((1 - t) * f / factor + t * f).float(), 1.0
 
     def dim_of(turns):
         return n * math.log(float(s["original"]) / (2 * math.pi * float(turns))) / (2 * math.log(base))
@@ -621,7 +676,33 @@ def _kikivik_preset(width: int, kinds: str, latent: dict, attention: dict, ff: i
                 embed_scale=2.0, traits=KIKIVIK_TRAITS)
 
 
+def _zonidra_preset(width: int, kinds: str, attention: dict, ff: int, moe: dict, bigram: dict, vocab: int) -> dict:
+    """Preset of a layer-list model with norms on both sides of its sublayers: ``kinds`` has two letters per layer, the attention (A with keys and
+    values of its own, S with those of the layer before it that has some) and the feed-forward (d dense, e experts, - none)."""
+    rot = {"dims": attention["dim"], "base": 5e5, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}
+    att = dict(attention, scale=attention["dim"] ** -0.5, rot=attention.get("rot", rot))
+    mlp = {"d": {"kind": "dense", "ff": ff}, "e": dict(moe, kind="moe"), "-": None}
+    layers, source = [], 0
+    for i, (k, f) in enumerate(zip(kinds[::2], kinds[1::2])):
+        source = i if k == "A" else source
+        layers.append({"type": "attention", "mixer": dict(att, kv_from=source) if k == "S" else att, "mlp": mlp[f]})
+    return dict(model_type="zonidra", vocab_size=vocab, hidden_size=width, num_hidden_layers=len(layers), intermediate_size=max(ff, moe["expert"]["ff"]),
+                num_attention_heads=att["heads"], num_key_value_heads=att["heads"], head_dim=att["dim"], rms_norm_eps=1e-6, mixers=layers,
+                embed_scale=float(width) ** 0.5, norm_place="both", layer_scale=True, token_shift=True, bigram=bigram, traits=ZONIDRA_TRAITS)
+
+
 PRESETS: dict[str, dict] = {
+    # Zonidra at the size of small production models: windowed sigmoid attention, every second layer on another's keys and values
+    "zonidra-2b": _zonidra_preset(2048, "AdSeAeSeAdSeAeSe", dict(heads=16, kv_heads=4, dim=128, vdim=128, mask={"size": 1024, "keep_first": 64}), 8192,
+                                  dict(expert={"ff": 768}, router={"experts": 64, "identity": 8, "top": 8, "scale": 2.5}, shared={"ff": 768}),
+                                  {"buckets": 65521, "mul_prev": 40503, "mul_cur": 1}, 65536),
+    "zonidra-7b": _zonidra_preset(4096, "AdSeAeSeAdSeAeSe", dict(heads=32, kv_heads=8, dim=128, vdim=128, mask={"size": 1024, "keep_first": 64}), 16384,
+                                  dict(expert={"ff": 1536}, router={"experts": 64, "identity": 8, "top": 8, "scale": 2.5}, shared={"ff": 1536}),
+                                  {"buckets": 65521, "mul_prev": 40503, "mul_cur": 1}, 65536),
+    "tiny-zonidra": _zonidra_preset(96, "AeSdAdS-", dict(heads=4, kv_heads=2, dim=24, vdim=16, mask={"size": 20, "keep_first": 3},
+                                                         rot={"dims": 16, "base": 1e4, "scaling": {"factor": 2.0, "low": 1.0, "high": 3.0, "original": 64}}),
+                                    160, dict(expert={"ff": 48}, router={"experts": 6, "identity": 2, "top": 3, "scale": 1.5}, shared={"ff": 40}),
+                                    {"buckets": 97, "mul_prev": 31, "mul_cur": 5}, 264),
     # Kikivik at the size of small production models: latent and chunked attention layers, dense and expert feed-forwards
     "kikivik-2b": _kikivik_preset(2048, "AdLeLdAeLeLdAeLe", dict(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=768),
                                   dict(heads=16, kv_heads=4, dim=128, vdim=128, mask={"size": 1024}, rot={"dims": 128, "base": 1e6, "scaling": {"factor": 4.0}}),

@@ -1,12 +1,12 @@
-"""Gated feed-forwards of models that are described layer by layer.
+"""Feed-forwards of models that are described layer by layer.
 
-A unit is ``down(act(gate h, up h))`` with one of two activations of neighbouring columns (g, u):
+A gated unit is ``down(act(gate h, up h))`` with one of two activations of neighbouring columns (g, u):
 
     clamped to a limit     g sigmoid(1.702 g) (u + 1),  g = min(gate, limit), u = clamp(up, +-limit)
     silu (no limit)        g sigmoid(g) u
 
 ``GatedUnit`` is one unit, ``GatedExperts`` many small ones of which every token uses a few, with an optional unit for every token beside
-them. Gate and up rows are interleaved in one weight (row 2i gate, row 2i + 1 up), so that a pair stands in neighbouring columns of the
+them. ``PolyUnit`` is ``down(act(up h))`` with a polynomial of normed powers as its activation. Gate and up rows are interleaved in one weight (row 2i gate, row 2i + 1 up), so that a pair stands in neighbouring columns of the
 product and the unit is evaluated in its epilogue. Widths are padded to multiples of 8 with zero rows and columns.
 
 The modules' ``forward`` methods are the differentiable PyTorch statement (training, CPU); the generation engine runs the same weights
@@ -22,7 +22,7 @@ import torch.nn as nn
 import torch.nn.functional as TF
 
 from .config import ModelConfig
-from .mixers import _linear, pad8
+from .mixers import _linear, pad8, rms_unit
 from .moe import limit_groups
 
 
@@ -60,10 +60,40 @@ class GatedUnit(nn.Module):
         return _linear(gated(_linear(h, self.gate_up), self.limit), self.down)
 
 
+def poly_norm(z: torch.Tensor, coef: torch.Tensor, eps: float) -> torch.Tensor:
+    """c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3 with N(y) = y over the root mean square of its row, in fp32. For every row that is one cubic
+    polynomial of the entries."""
+    z, c = z.float(), coef.float()
+    y = c[3]
+    for i in range(3):
+        y = y + c[i] * rms_unit(z ** (i + 1), eps)
+    return y
+
+
+class PolyUnit(nn.Module):
+    def __init__(self, spec: dict, cfg: ModelConfig, dtype, device):
+        super().__init__()
+        self.ff, self.eps = spec["ff"], cfg.rms_norm_eps
+        d, n = cfg.hidden_size, pad8(self.ff)
+        self.up = nn.Parameter(torch.zeros(n, d, dtype=dtype, device=device))
+        self.down = nn.Parameter(torch.zeros(d, n, dtype=dtype, device=device))
+        self.coef = nn.Parameter(torch.tensor([1 / 3, 1 / 3, 1 / 3, 0.0], dtype=dtype, device=device))
+
+    def tensors(self) -> list:
+        return [("up", self.up[: self.ff]), ("down", self.down[:, : self.ff]), ("act", self.coef)]
+
+    def forward(self, h: torch.Tensor) -> torch.Tensor:
+        p = _linear(h, self.up)
+        a = poly_norm(p[:, : self.ff], self.coef, self.eps).to(p.dtype)
+        return _linear(TF.pad(a, (0, p.shape[1] - self.ff)), self.down)
+
+
 class GatedExperts(nn.Module):
-    """Sigmoid router in fp32: experts are chosen by score (+ correction) among the best groups and weighted by the scores themselves, on
-    their outputs or (``weigh_input``) on their inputs, i.e. on the rows of their first product. Spec: "router", "expert", optionally
-    "shared" (a unit for every token), "weigh_input", "corrected" (whether there is a correction; default yes)."""
+    """Router in fp32: experts are chosen by score (+ correction) among the best groups and weighted by the scores themselves (times a
+    constant), on their outputs or (``weigh_input``) on their inputs, i.e. on the rows of their first product. Spec: "router" ("experts", "top",
+    optionally "groups", "scale", "identity": that many more outputs, behind the experts', which stand for the input itself), "expert",
+    optionally "shared" (a unit for every token), "shared_gate" (its output is multiplied by a sigmoid, one number per token), "score" ("sigmoid",
+    the default, or "softmax" over all outputs), "weigh_input", "corrected" (whether there is a correction; default yes)."""
 
     def __init__(self, spec: dict, cfg: ModelConfig, dtype, device):
         super().__init__()
@@ -72,31 +102,44 @@ class GatedExperts(nn.Module):
         self.experts, self.top, self.groups, self.keep = r["experts"], r["top"], g["count"], g["keep"]
         self.ff, self.limit, self.weigh_input = spec["expert"]["ff"], _limit(spec["expert"]), bool(spec.get("weigh_input"))
         d, n = cfg.hidden_size, pad8(self.ff)
-        self.router = nn.Parameter(torch.zeros(self.experts, d, dtype=dtype, device=device))
+        self.identity, self.scale, self.softmax = r.get("identity", 0), float(r.get("scale", 1.0)), spec.get("score", "sigmoid") == "softmax"
+        self.outputs = self.experts + self.identity
+        self.shared_gate = bool(spec.get("shared") and spec.get("shared_gate"))
+        assert not (self.weigh_input and self.identity), "weights on the experts' inputs and identity outputs"
+        # the shared unit's gate is one more row behind the outputs
+        rows = self.outputs + int(self.shared_gate)
+        self.router = nn.Parameter(torch.zeros(rows if rows == self.experts else pad8(rows), d, dtype=dtype, device=device))
         self.gate_up = nn.Parameter(torch.zeros(self.experts, 2 * n, d, dtype=dtype, device=device))
         self.down = nn.Parameter(torch.zeros(self.experts, d, n, dtype=dtype, device=device))
         # shifts the choice; not trained by gradient
-        self.register_buffer("correction", torch.zeros(self.experts, dtype=torch.float32, device=device) if spec.get("corrected", True) else None)
+        self.register_buffer("correction", torch.zeros(self.outputs, dtype=torch.float32, device=device) if spec.get("corrected", True) else None)
         self.shared = GatedUnit(spec["shared"], cfg, dtype, device) if spec.get("shared") else None
 
     def tensors(self) -> list:
-        n, out = self.ff, [("router", self.router)]
+        n, out = self.ff, [("router", self.router[: self.outputs])]
         if self.correction is not None:
             out.append(("correction", self.correction))
         for e in range(self.experts):
             out += [(f"e{e}.gate", self.gate_up[e, 0 : 2 * n : 2]), (f"e{e}.up", self.gate_up[e, 1 : 2 * n : 2]), (f"e{e}.down", self.down[e, :, :n])]
+        if self.shared_gate:
+            out.append(("shared.sg", self.router[self.outputs : self.outputs + 1]))
         return out + ([(f"shared.{leaf}", t) for leaf, t in self.shared.tensors()] if self.shared is not None else [])
 
     def choose(self, z: torch.Tensor):
-        """Router logits [T, experts] fp32 -> (weights, expert ids) [T, top]."""
-        s = torch.sigmoid(z)
+        """Router logits [T, outputs] fp32 -> (weights, indices) [T, top]."""
+        s = torch.softmax(z, -1) if self.softmax else torch.sigmoid(z)
         c = s if self.correction is None else s + self.correction
         idx = limit_groups(c, self.groups, self.keep, float("-inf")).topk(self.top, dim=-1)[1]
-        return s.gather(1, idx), idx
+        return s.gather(1, idx) * self.scale, idx
 
     def forward(self, h: torch.Tensor) -> torch.Tensor:
-        w, idx = self.choose(h.float() @ self.router.float().t())
+        z = h.float() @ self.router.float().t()
+        w, idx = self.choose(z[:, : self.outputs])
         y = torch.zeros(h.shape, dtype=torch.float32, device=h.device) if self.shared is None else self.shared(h).float()
+        if self.shared_gate:
+            y = y * torch.sigmoid(z[:, self.outputs, None])
+        if self.identity:
+            y = y + h.float() * (w * (idx >= self.experts)).sum(-1, keepdim=True)
         for e in range(self.experts):
             tok, slot = (idx == e).nonzero(as_tuple=True)
             if tok.numel():
@@ -108,4 +151,5 @@ class GatedExperts(nn.Module):
 
 
 def feed_forward(spec: dict, cfg: ModelConfig, dtype, device) -> nn.Module:
-    return (GatedExperts if spec["kind"] == "moe" else GatedUnit)(spec, cfg, dtype, device)
+    kind = GatedExperts if spec["kind"] == "moe" else PolyUnit if spec.get("act") == "poly" else GatedUnit
+    return kind(spec, cfg, dtype, device)

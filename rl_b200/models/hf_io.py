@@ -175,10 +175,12 @@ def _model_map(model: CausalLM):
 def iter_hf_shards(model: CausalLM) -> Iterator[tuple[str, torch.Tensor, Optional[tuple[int, int, int]]]]:
     """Yields (hf_name, local tensor view, hf_slice) for every logical HF tensor (or shard of one) this rank holds."""
     cfg = model.cfg
-    if cfg.is_mixer:    # layer-list models (Gadarax, Redarax, Kikivik) keep their checkpoint's own tensor names
+    if cfg.is_mixer:    # layer-list models (Gadarax, Redarax, Kikivik, Zonidra) keep their checkpoint's own tensor names
         yield "embed", model.embed_tokens, None
         if model.side_embed is not None:
             yield "side.embed", model.side_embed, None
+        if model.bigram is not None:
+            yield "bigram", model.bigram, None
         if model.loop_step is not None:
             yield "loop.step", model.loop_step, None
         for i, layer in enumerate(model.layers):

@@ -17,8 +17,9 @@ Mixers:
   * ``RetentionMixer``: linear attention with one fixed decay per head, a unit-RMS norm per head and a SiLU gate. The state
     [heads, dim, vdim] is fp32.
   * ``GroupedAttentionMixer``: causal attention with fewer key / value heads than query heads, RMS norms per head on queries and keys,
-    partial rotation (pairs interleaved or in halves), own scale, keys and values of unequal size; optionally biases, keys of the query's
-    own chunk of positions only, values mixed with those of the first such layer.
+    partial rotation (pairs interleaved or in halves), own scale, keys and values of unequal size; optionally biases, an output gate, keys of
+    the query's own chunk of positions or of a sliding window with kept first tokens only, values mixed with those of the first such layer,
+    another layer's keys and values in place of own ones, sigmoid weights in place of the soft-max.
   * ``Mamba2LayerMixer``: state-space duality with a short convolution in front and a gated norm in equal parts behind.
   * ``DeltaMixer``: gated delta rule: a linear-attention state that forgets by a decay per token and corrects what it stores under a key.
 
@@ -27,6 +28,8 @@ engine runs the same weights through ``rl_b200/ops/mixer_ops.py`` (latent attent
 """
 
 from __future__ import annotations
+
+import math
 
 import torch
 import torch.nn as nn
@@ -233,9 +236,16 @@ def rms_unit(x: torch.Tensor, eps: float) -> torch.Tensor:
 
 
 class GroupedAttentionMixer(nn.Module):
-    """Spec, beside the sizes: "bias" (default yes), "interleaved" (rotated pairs are (2i, 2i + 1), default yes; else (i, i + dims / 2)),
-    "mask" = {"size"} (position i sees j <= i of the same run of ``size`` positions, counted from the sequence's first), "v_mix" (values
-    become (1 - share) v + share v_first with v_first the first such layer's)."""
+    """Spec, beside the sizes:
+      "bias"         biases on the projections (default yes)
+      "qk_norm"      RMS norms per head on queries and keys (default yes)
+      "interleaved"  rotated pairs are (2i, 2i + 1) (default yes); else (i, i + dims / 2)
+      "mask"         with "mask_kind" "chunk" (default) {"size"}: position i sees j <= i of the same run of ``size`` positions, counted from the
+                     sequence's first; with "window" {"size", "keep_first"}: it sees j <= i with i - j < size or j < keep_first
+      "weights"      "softmax" (default), or "sigmoid": every visible key weighs sigmoid(score + a number per head), unnormalised
+      "gate"         the head outputs are multiplied by sigmoid of a projection of the mixer's input (default no)
+      "v_mix"        values become (1 - share) v + share v_first with v_first the first such layer's
+      "kv_from"      index of the layer whose keys and values are read; the layer projects none of its own"""
 
     kind = "attention"
 
@@ -243,10 +253,16 @@ class GroupedAttentionMixer(nn.Module):
         super().__init__()
         self.heads, self.kv_heads, self.dim, self.vdim = spec["heads"], spec["kv_heads"], spec["dim"], spec["vdim"]
         self.scale, self.eps = float(spec["scale"]), cfg.rms_norm_eps
-        self.q_off, self.k_off = 0, pad8(self.heads * self.dim)
-        self.v_off = self.k_off + pad8(self.kv_heads * self.dim)
-        self.in_width = self.v_off + pad8(self.kv_heads * self.vdim)
+        self.kv_from = spec.get("kv_from")
+        self.gate, self.sigmoid = bool(spec.get("gate")), spec.get("weights", "softmax") == "sigmoid"
+        self.q_off, end = 0, pad8(self.heads * self.dim)
+        self.k_off = self.v_off = end
+        if self.kv_from is None:
+            self.v_off = self.k_off + pad8(self.kv_heads * self.dim)
+            end = self.v_off + pad8(self.kv_heads * self.vdim)
         self.mix_width = pad8(self.heads * self.vdim)
+        # with a gate the head outputs are written over its columns of the projected rows, else to rows of their own
+        self.mix_off, self.in_width = (end, end + self.mix_width) if self.gate else (0, end)
         d = cfg.hidden_size
         self.in_proj = nn.Parameter(torch.zeros(self.in_width, d, dtype=dtype, device=device))
         self.out_proj = nn.Parameter(torch.zeros(d, self.mix_width, dtype=dtype, device=device))
@@ -254,54 +270,98 @@ class GroupedAttentionMixer(nn.Module):
         if spec.get("bias", True):
             self.in_bias = nn.Parameter(torch.zeros(self.in_width, dtype=dtype, device=device))
             self.out_bias = nn.Parameter(torch.zeros(d, dtype=dtype, device=device))
-        self.interleaved, self.chunk = bool(spec.get("interleaved", True)), int((spec.get("mask") or {"size": 0})["size"])
+        self.interleaved, mask = bool(spec.get("interleaved", True)), spec.get("mask")
+        windowed = spec.get("mask_kind", "chunk") == "window"
+        self.chunk = int(mask["size"]) if mask and not windowed else 0
+        self.window, self.keep = (int(mask["size"]), int(mask.get("keep_first", 0))) if mask and windowed else (0, 0)
         self.v_mix = bool(spec.get("v_mix"))
         if self.v_mix:
             self.v_share = nn.Parameter(torch.full((), 0.5, dtype=dtype, device=device))
-        self.q_norm = nn.Parameter(torch.ones(self.dim, dtype=dtype, device=device))
-        self.k_norm = nn.Parameter(torch.ones(self.dim, dtype=dtype, device=device))
+        self.qk_norm = bool(spec.get("qk_norm", True))
+        self.q_norm = self.k_norm = self.offset = None
+        if self.qk_norm:
+            self.q_norm = nn.Parameter(torch.ones(self.dim, dtype=dtype, device=device))
+            self.k_norm = nn.Parameter(torch.ones(self.dim, dtype=dtype, device=device))
+        if self.sigmoid:       # added to the scores; starts where as many keys as the mask shows weigh about one together
+            self.offset = nn.Parameter(torch.full((self.heads,), -math.log(self.window or self.chunk or 1024), dtype=dtype, device=device))
         freq, self.gain = rotary_table(spec["rot"])
         self.register_buffer("freq", freq.to(device), persistent=False)
 
     def tensors(self) -> list:
         """(checkpoint leaf, view of a parameter)."""
+        own = self.kv_from is None
+        rows = [("q", self.q_off, self.heads * self.dim)]
+        if own:
+            rows += [("k", self.k_off, self.kv_heads * self.dim), ("v", self.v_off, self.kv_heads * self.vdim)]
+        if self.gate:
+            rows.append(("g", self.mix_off, self.heads * self.vdim))
         out = []
-        for leaf, r, n in (("q", self.q_off, self.heads * self.dim), ("k", self.k_off, self.kv_heads * self.dim), ("v", self.v_off, self.kv_heads * self.vdim)):
+        for leaf, r, n in rows:
             out += [(leaf, self.in_proj[r : r + n])] + ([(leaf + ".b", self.in_bias[r : r + n])] if self.in_bias is not None else [])
-        out += [("q.norm", self.q_norm), ("k.norm", self.k_norm), ("o", self.out_proj[:, : self.heads * self.vdim])]
+        if self.qk_norm:
+            out += [("q.norm", self.q_norm)] + ([("k.norm", self.k_norm)] if own else [])
+        if self.sigmoid:
+            out.append(("pb", self.offset))
+        out.append(("o", self.out_proj[:, : self.heads * self.vdim]))
         return out + ([("o.b", self.out_bias)] if self.out_bias is not None else []) + ([("vmix", self.v_share)] if self.v_mix else [])
 
     def values(self, p: torch.Tensor) -> torch.Tensor:
         """The layer's own values, columns of the projected rows."""
         return p[:, self.v_off : self.v_off + self.kv_heads * self.vdim]
 
-    def qkv(self, p: torch.Tensor, positions: torch.Tensor, first=None):
-        """fp32 normed and rotated queries [T, heads, dim] and keys [T, kv_heads, dim], values [T, kv_heads, vdim] (mixed with ``first``)."""
-        q = p[:, self.q_off : self.q_off + self.heads * self.dim].reshape(-1, self.heads, self.dim).float()
-        k = p[:, self.k_off : self.k_off + self.kv_heads * self.dim].reshape(-1, self.kv_heads, self.dim).float()
+    def _prepared(self, x: torch.Tensor, norm, positions: torch.Tensor) -> torch.Tensor:
+        x = x.float()
+        if self.qk_norm:
+            x = rms_unit(x, self.eps) * norm.float()
+        return rotate_pairs(x, positions, self.freq, self.gain, self.interleaved)
+
+    def queries(self, p: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
+        """fp32 normed and rotated queries [T, heads, dim]."""
+        return self._prepared(p[:, self.q_off : self.q_off + self.heads * self.dim].reshape(-1, self.heads, self.dim), self.q_norm, positions)
+
+    def keys_values(self, p: torch.Tensor, positions: torch.Tensor, first=None):
+        """fp32 normed and rotated keys [T, kv_heads, dim], values [T, kv_heads, vdim] (mixed with ``first``)."""
         v = self.values(p).float()
         if first is not None:
             v = (1 - self.v_share.float()) * v + self.v_share.float() * first.float()
-        v = v.reshape(-1, self.kv_heads, self.vdim)
-        q = rotate_pairs(rms_unit(q, self.eps) * self.q_norm.float(), positions, self.freq, self.gain, self.interleaved)
-        k = rotate_pairs(rms_unit(k, self.eps) * self.k_norm.float(), positions, self.freq, self.gain, self.interleaved)
-        return q, k, v
+        k = self._prepared(p[:, self.k_off : self.k_off + self.kv_heads * self.dim].reshape(-1, self.kv_heads, self.dim), self.k_norm, positions)
+        return k, v.reshape(-1, self.kv_heads, self.vdim)
 
-    def sequence(self, p: torch.Tensor, positions: torch.Tensor, cu_seqlens: torch.Tensor, first=None) -> torch.Tensor:
-        """Head outputs [T, heads * vdim] of packed whole sequences."""
-        q, k, v = self.qkv(p, positions, first)
+    def qkv(self, p: torch.Tensor, positions: torch.Tensor, first=None):
+        return (self.queries(p, positions), *self.keys_values(p, positions, first))
+
+    def hidden(self, i: torch.Tensor, j: torch.Tensor) -> torch.Tensor:
+        """Whether position i does not see position j (tensors that broadcast)."""
+        h = j > i
+        if self.chunk:
+            h = h | (i // self.chunk != j // self.chunk)
+        if self.window:
+            h = h | ((i - j >= self.window) & (j >= self.keep))
+        return h
+
+    def weigh(self, z: torch.Tensor, hidden: torch.Tensor) -> torch.Tensor:
+        """Weights of the keys from scaled scores [..., heads, queries, keys]."""
+        if self.sigmoid:
+            return torch.sigmoid(z + self.offset.float()[:, None, None]).masked_fill(hidden, 0.0)
+        return torch.softmax(z.masked_fill(hidden, float("-inf")), -1)
+
+    def gated(self, y: torch.Tensor, p: torch.Tensor) -> torch.Tensor:
+        """Head outputs [T, heads * vdim] behind the output gate where there is one."""
+        return y * torch.sigmoid(p[:, self.mix_off : self.mix_off + self.heads * self.vdim].float()) if self.gate else y
+
+    def sequence(self, p: torch.Tensor, positions: torch.Tensor, cu_seqlens: torch.Tensor, first=None, kv=None) -> torch.Tensor:
+        """Head outputs [T, heads * vdim] of packed whole sequences. ``kv``: prepared keys and values (None: the layer's own)."""
+        q = self.queries(p, positions)
+        k, v = self.keys_values(p, positions, first) if kv is None else kv
         n = self.heads // self.kv_heads
         k, v = k.repeat_interleave(n, dim=1), v.repeat_interleave(n, dim=1)
         out = []
         cu = cu_seqlens.tolist()
         for s, e in zip(cu[:-1], cu[1:]):
             z = torch.einsum("ihd,jhd->hij", q[s:e], k[s:e]) * self.scale
-            hidden = torch.ones(e - s, e - s, dtype=torch.bool, device=z.device).triu(1)
-            if self.chunk:
-                c = torch.arange(e - s, device=z.device) // self.chunk
-                hidden = hidden | (c[:, None] != c[None, :])
-            out.append(torch.einsum("hij,jhd->ihd", torch.softmax(z.masked_fill(hidden, float("-inf")), -1), v[s:e]))
-        return torch.cat(out).reshape(-1, self.heads * self.vdim).to(p.dtype)
+            t = torch.arange(e - s, device=z.device)
+            out.append(torch.einsum("hij,jhd->ihd", self.weigh(z, self.hidden(t[:, None], t[None, :])), v[s:e]))
+        return self.gated(torch.cat(out).reshape(-1, self.heads * self.vdim), p).to(p.dtype)
 
 
 class RecurrentMixer(nn.Module):

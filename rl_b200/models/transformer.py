@@ -544,6 +544,8 @@ class CausalLM(nn.Module):
         # token inputs of the layers: one table, the layers' columns side by side
         side = cfg.token_side["dim"] * L if cfg.token_side else 0
         self.side_embed = nn.Parameter(torch.empty(cfg.vocab_size, side, dtype=dtype, device=device)) if side else None
+        # pairs of tokens: one row per bucket of the pairs' hash, and one for first tokens
+        self.bigram = nn.Parameter(torch.empty(cfg.bigram["buckets"] + 1, d, dtype=dtype, device=device)) if cfg.bigram else None
         # looped layers: one learned vector per pass joins the residual stream when the pass begins
         self.loop_step = nn.Parameter(torch.zeros(cfg.layer_loop["times"], d, dtype=dtype, device=device)) if cfg.layer_loop else None
         self.register_buffer("inv_freq", rope_inv_freq(cfg, device) if not cfg.is_mixer else torch.zeros(0, device=device), persistent=False)
@@ -596,7 +598,7 @@ class CausalLM(nn.Module):
         from .hf_io import iter_hf_shards, hf_full_shape
 
         for name, p in self.named_parameters():
-            if name.endswith("norm") or name.rsplit(".", 1)[-1] in ("norm1", "norm2") or name.endswith("layernorm") or name.endswith("norm.weight"):
+            if name.endswith("norm") or name.rsplit(".", 1)[-1] in ("norm1", "norm2", "norm1b", "norm2b") or name.endswith("layernorm") or name.endswith("norm.weight"):
                 p.fill_(1.0)
             elif name.endswith("bias"):
                 p.zero_()
@@ -711,8 +713,14 @@ class CausalLM(nn.Module):
         h = self._embed(batch)
         s = self.cfg.embed_scale
         if self.cfg.is_mixer:      # fp32 residual stream
-            return h.float() * s
+            return h.float() * s if self.bigram is None else h.float() * s + nn.functional.embedding(self.pair_rows(batch), self.bigram).float()
         return h if s == 1.0 else h * torch.tensor(s, dtype=h.dtype, device=h.device)   # the scale is rounded to the model dtype first
+
+    def pair_rows(self, batch: PackedBatch) -> torch.Tensor:
+        """Row of the pair table for every token of packed whole sequences."""
+        g, ids = self.cfg.bigram, batch.input_ids.long()
+        rows = (torch.roll(ids, 1) * g["mul_prev"] + ids * g["mul_cur"]) % g["buckets"]
+        return rows.masked_fill(batch.positions == 0, g["buckets"])
 
     def _embed(self, batch: PackedBatch) -> torch.Tensor:
         if self.sharder is not None:
@@ -730,14 +738,14 @@ class CausalLM(nn.Module):
     def _run_layer_runs(self, h: torch.Tensor, batch: PackedBatch) -> torch.Tensor:
         """Layers in the order of ``cfg.layer_runs``. A pass of the loop begins with the embeddings added again (not in the first)
         and with its step vector added."""
-        e, loop, carries, values = h, self.cfg.layer_loop, self.cfg.layer_form == "pre", None
+        e, loop, carries, handed = h, self.cfg.layer_loop, self.cfg.layer_form == "pre", {}
         for i, t in self.cfg.layer_runs:
             if t is not None and i == loop["start"]:
                 h = (h + e if t else h) + self.loop_step[t].float()
-            args = (h, batch.positions, values if carries else self.side_rows(batch.input_ids, i), batch.cu_seqlens, batch.max_seqlen)
+            args = (h, batch.positions, handed if carries else self.side_rows(batch.input_ids, i), batch.cu_seqlens, batch.max_seqlen)
             h = ckpt.checkpoint(self.layers[i], *args, use_reentrant=False) if (self.activation_checkpointing and torch.is_grad_enabled()) else self.layers[i](*args)
-            if carries:        # pre-norm layers hand on the values that later ones mix in
-                h, values = h
+            if carries:        # pre-norm layers hand on values that later ones mix in, keys and values that later ones read
+                h, handed = h
         return h
 
     def side_rows(self, ids: torch.Tensor, layer: int) -> Optional[torch.Tensor]:

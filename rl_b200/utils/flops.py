@@ -288,12 +288,36 @@ def kikivik_flops(hf, seq: int) -> float:
     return total + head_flops(seq, d, _g(hf, "vocab_size"))
 
 
+def zonidra_flops(hf, seq: int) -> float:
+    """Layer-list models with windowed grouped attention behind an output gate (some layers without keys and values of their own), two-matrix or
+    expert feed-forwards. Identity outputs of the router count as chosen at random."""
+    d, total = _g(hf, "hidden_size"), 0.0
+    for e in _g(hf, "mixers"):
+        m, mlp = e["mixer"], e.get("mlp")
+        H, kd, vd = m["heads"], m["dim"], m["vdim"]
+        size = min(m["mask"]["size"], seq) if m.get("mask") else seq
+        pairs = size * (size + 1) / 2 + (seq - size) * size
+        if m.get("mask"):      # kept first tokens that the window has left behind
+            keep = min(m["mask"].get("keep_first", 0), seq - size)
+            pairs += keep * (seq - size) - keep * (keep - 1) / 2
+        total += 2 * seq * d * (H * kd + 2 * H * vd + (m["kv_heads"] * (kd + vd) if m.get("kv_from") is None else 0)) + 2 * pairs * H * (kd + vd)
+        if mlp and mlp.get("kind") == "moe":
+            r = mlp["router"]
+            n = r["experts"] + r.get("identity", 0)
+            total += 2 * seq * d * n + r["top"] * r["experts"] / n * mlp_flops(seq, d, mlp["expert"]["ff"], gated=True)
+            total += mlp_flops(seq, d, mlp["shared"]["ff"], gated=True) if mlp.get("shared") else 0.0
+        elif mlp:
+            total += mlp_flops(seq, d, mlp["ff"], gated=False)
+    return total + head_flops(seq, d, _g(hf, "vocab_size"))
+
+
 FAMILY_FLOPS = {
     "llama": llama_flops, "mistral": mistral_flops, "qwen2": qwen2_flops, "qwen3": qwen3_flops, "gemma3": gemma3_flops,
     "gemma3_text": gemma3_flops,
     "gpt2": gpt_flops, "gpt3": gpt_flops, "nemotron": nemotron_flops, "mixtral": mixtral_flops, "qwen3_moe": qwen3_moe_flops,
     "qwen2_moe": moe_decoder_flops, "deepseek_v3": deepseek_v3_flops, "deepseek_v2": deepseek_v3_flops, "nemotron_h": nemotron_h_flops,
     "bert": bert_flops, "gadarax": gadarax_flops, "redarax": redarax_flops, "kikivik": kikivik_flops,
+    "zonidra": zonidra_flops,
 }
 
 
