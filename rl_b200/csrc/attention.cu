@@ -29,6 +29,7 @@ struct GqaShape {
   int heads, kv_heads, dim, vdim;
   int block_size, num_blocks;
   int halves;            // rotated pairs are (i, i + half) instead of (2i, 2i + 1)
+  int own_kv;            // the rows hold keys and values of the layer's own
 };
 
 // Values of a layer that mixes them with an earlier layer's: v <- (1 - share) v + share v_first.
@@ -96,7 +97,7 @@ gqa_prep_kernel(T* __restrict__ p, GqaShape s, ValueMix<T> mix, const int* __res
   const bool even = s.dim % 2 == 0 && s.ldp % 2 == 0, veven = s.vdim % 2 == 0 && s.ldp % 2 == 0;      // pairs are aligned
   const int pairs = (s.dim + 1) / 2;
   __syncthreads();
-  for (int unit = blockIdx.y * GP_WARPS + (threadIdx.x >> 5); unit < s.heads + 2 * s.kv_heads; unit += gridDim.y * GP_WARPS) {
+  for (int unit = blockIdx.y * GP_WARPS + (threadIdx.x >> 5); unit < s.heads + (s.own_kv ? 2 * s.kv_heads : 0); unit += gridDim.y * GP_WARPS) {
     const bool is_q = unit < s.heads, is_k = !is_q && unit < s.heads + s.kv_heads;
     const int head = is_q ? unit : (is_k ? unit - s.heads : unit - s.heads - s.kv_heads);
     if (!is_q && !is_k) {
@@ -120,7 +121,8 @@ gqa_prep_kernel(T* __restrict__ p, GqaShape s, ValueMix<T> mix, const int* __res
       continue;
     }
     T* x = pr + (is_q ? s.q_off : s.k_off) + head * s.dim;
-    const T* w = is_q ? q_norm : k_norm;
+    const T* w = is_q ? q_norm : k_norm;      // null: no norm
+    auto weight = [&](int i) { return w ? ldf(w + i) : 1.f; };
     T* c = is_k && cached ? k_cache + ((page * s.kv_heads + head) * s.block_size + off) * s.dim : nullptr;
     auto load = [&](int i) {      // pair i, zeros past the end
       if (2 * i + 1 < s.dim) return Pair<T>::load(x + 2 * i, even);
@@ -138,26 +140,26 @@ gqa_prep_kernel(T* __restrict__ p, GqaShape s, ValueMix<T> mix, const int* __res
       ss += t.x * t.x + t.y * t.y;
     }
     ss = warp_sum(ss);
-    const float rstd = 1.f / sqrtf(ss / static_cast<float>(s.dim) + eps);
+    const float rstd = w ? 1.f / sqrtf(ss / static_cast<float>(s.dim) + eps) : 1.f;
     if (s.halves) {      // a lane turns entries i and i + half; the sum's shuffles stand between the loads above and these stores
       auto put = [&](int i, float t) {
         stf(x + i, t);
         if (c) stf(c + i, t);
       };
       for (int i = lane; i < half; i += 32) {
-        const float a = ldf(x + i) * rstd * ldf(w + i), b = ldf(x + i + half) * rstd * ldf(w + i + half);
+        const float a = ldf(x + i) * rstd * weight(i), b = ldf(x + i + half) * rstd * weight(i + half);
         const float2 r = turn[i];
         put(i, a * r.x - b * r.y);
         put(i + half, b * r.x + a * r.y);
       }
-      for (int i = 2 * half + lane; i < s.dim; i += 32) put(i, ldf(x + i) * rstd * ldf(w + i));
+      for (int i = 2 * half + lane; i < s.dim; i += 32) put(i, ldf(x + i) * rstd * weight(i));
       continue;
     }
     auto finish = [&](int i, float2 t) {
       if (2 * i >= s.dim) return;
       const bool two = 2 * i + 1 < s.dim;
-      t.x *= rstd * ldf(w + 2 * i);
-      if (two) t.y *= rstd * ldf(w + 2 * i + 1);
+      t.x *= rstd * weight(2 * i);
+      if (two) t.y *= rstd * weight(2 * i + 1);
       if (i < half) {
         const float2 r = turn[i];
         t = make_float2(t.x * r.x - t.y * r.y, t.y * r.x + t.x * r.y);
@@ -198,8 +200,8 @@ gqa_prep_rows_kernel(__nv_bfloat16* __restrict__ p, GqaShape s, ValueMix<__nv_bf
   for (int j = 0; j < KEEP; ++j) {
     const int i = word(j);
     const bool live = 2 * i < s.dim;
-    wq[j] = live ? Pair<__nv_bfloat16>::load(q_norm + 2 * i, true) : make_float2(0.f, 0.f);
-    wk[j] = live ? Pair<__nv_bfloat16>::load(k_norm + 2 * i, true) : make_float2(0.f, 0.f);
+    wq[j] = live && q_norm ? Pair<__nv_bfloat16>::load(q_norm + 2 * i, true) : make_float2(1.f, 1.f);
+    wk[j] = live && k_norm ? Pair<__nv_bfloat16>::load(k_norm + 2 * i, true) : make_float2(1.f, 1.f);
   }
   pdl_sync();
   if (row >= rows) return;
@@ -220,7 +222,7 @@ gqa_prep_rows_kernel(__nv_bfloat16* __restrict__ p, GqaShape s, ValueMix<__nv_bf
     }
   }
   __nv_bfloat16* pr = p + row * s.ldp;
-  const int units = s.heads + s.kv_heads;
+  const int units = s.heads + (s.own_kv ? s.kv_heads : 0);
   for (int u0 = blockIdx.y * AHEAD; u0 < units; u0 += gridDim.y * AHEAD) {
     float2 v[AHEAD][KEEP];
     float ss[AHEAD];
@@ -248,7 +250,7 @@ gqa_prep_rows_kernel(__nv_bfloat16* __restrict__ p, GqaShape s, ValueMix<__nv_bf
       if (unit >= units) break;
       const bool is_q = unit < s.heads;
       const int head = is_q ? unit : unit - s.heads;
-      const float rstd = 1.f / sqrtf(ss[a] / static_cast<float>(s.dim) + eps);
+      const float rstd = (is_q ? q_norm : k_norm) ? 1.f / sqrtf(ss[a] / static_cast<float>(s.dim) + eps) : 1.f;
       __nv_bfloat16* x = pr + (is_q ? s.q_off : s.k_off) + head * s.dim;
       __nv_bfloat16* c = k_cache + ((static_cast<long long>(page) * s.kv_heads + head) * s.block_size + off) * s.dim;
       if (HALVES) {
@@ -281,7 +283,7 @@ gqa_prep_rows_kernel(__nv_bfloat16* __restrict__ p, GqaShape s, ValueMix<__nv_bf
       }
     }
   }
-  if (!cached && !mix.first) return;
+  if (!s.own_kv || (!cached && !mix.first)) return;
   const float share = mix.first ? __bfloat162float(*mix.share) : 0.f;
   for (int g = blockIdx.y; g < s.kv_heads; g += gridDim.y) {
     __nv_bfloat16* x = pr + s.v_off + g * s.vdim;
@@ -299,13 +301,17 @@ gqa_prep_rows_kernel(__nv_bfloat16* __restrict__ p, GqaShape s, ValueMix<__nv_bf
   }
 }
 
-// One CTA per (row, query head): tiles of 128 keys, online softmax, everything in fp32. chunk > 0: only the keys of the row's own run of
-// `chunk` positions are visible.
+// One CTA per (row, query head): tiles of 128 keys, everything in fp32; online softmax, or with `offset` the weights sigmoid(score + offset[head]).
+// What a row at position i sees: chunk > 0: the keys of its own run of `chunk` positions; window > 0: keys j with i - j < window or j < keep.
+// gated: the output's place holds gates, out = y * sigmoid(gate).
+struct RowsMask {
+  int chunk, window, keep, gated;
+};
 constexpr int GR_TILE = 128;
 template <typename T>
 __global__ void __launch_bounds__(128)
-gqa_rows_kernel(const T* __restrict__ p, GqaShape s, const T* __restrict__ k_cache, const T* __restrict__ v_cache, const int* __restrict__ block_table,
-                int bt_stride, const int* __restrict__ seq_lens, int chunk, float scale, T* __restrict__ y, long long ldy, int* status) {
+gqa_rows_kernel(const T* p, GqaShape s, const T* __restrict__ k_cache, const T* __restrict__ v_cache, const int* __restrict__ block_table,
+                int bt_stride, const int* __restrict__ seq_lens, RowsMask mask, const T* __restrict__ offset, float scale, T* y, long long ldy, int* status) {
   extern __shared__ float sm[];
   __shared__ float red[32];
   float* q = sm;                        // [dim]
@@ -317,9 +323,15 @@ gqa_rows_kernel(const T* __restrict__ p, GqaShape s, const T* __restrict__ k_cac
   for (int i = tid; i < s.dim; i += 128) q[i] = ldf(qp + i) * scale;
   for (int i = tid; i < s.vdim; i += 128) o[i] = 0.f;
   const int len = min(seq_lens[row], bt_stride * s.block_size);
+  const float off = offset ? ldf(offset + h) : 0.f;
   float m = -INFINITY, l = 0.f;
-  for (int t0 = chunk > 0 && len > 0 ? (len - 1) / chunk * chunk : 0; t0 < len; t0 += GR_TILE) {
-    const int n = min(GR_TILE, len - t0);
+  int first = 0;                        // first visible key behind the kept ones
+  if (len > 0 && mask.chunk > 0) first = (len - 1) / mask.chunk * mask.chunk;
+  if (mask.window > 0) first = max(0, len - mask.window);
+  const int kept = mask.window > 0 ? min(mask.keep, first) : 0;
+  int t0 = kept > 0 ? 0 : first;
+  while (t0 < len) {
+    const int n = min(GR_TILE, (t0 < kept ? kept : len) - t0);
     __syncthreads();
     if (tid < n) {
       const int t = t0 + tid;
@@ -339,13 +351,18 @@ gqa_rows_kernel(const T* __restrict__ p, GqaShape s, const T* __restrict__ k_cac
       if (lane == 0) sc[j] = v;
     }
     __syncthreads();
-    const float mine = tid < n ? sc[tid] : -INFINITY;
-    const float mn = fmaxf(m, block_max(mine, red));
-    const float pj = tid < n ? expf(mine - mn) : 0.f;
-    const float c = m == -INFINITY ? 0.f : expf(m - mn);
-    l = l * c + block_sum(pj, red);
-    m = mn;
-    if (tid < n) sc[tid] = pj;
+    float c = 1.f;
+    if (offset) {
+      if (tid < n) sc[tid] = 1.f / (1.f + expf(-(sc[tid] + off)));
+    } else {
+      const float mine = tid < n ? sc[tid] : -INFINITY;
+      const float mn = fmaxf(m, block_max(mine, red));
+      const float pj = tid < n ? expf(mine - mn) : 0.f;
+      c = m == -INFINITY ? 0.f : expf(m - mn);
+      l = l * c + block_sum(pj, red);
+      m = mn;
+      if (tid < n) sc[tid] = pj;
+    }
     __syncthreads();
     for (int i = tid; i < s.vdim; i += 128) {
       float v[4] = {0.f, 0.f, 0.f, 0.f};
@@ -356,9 +373,13 @@ gqa_rows_kernel(const T* __restrict__ p, GqaShape s, const T* __restrict__ k_cac
       for (; j < n; ++j) v[0] = fmaf(sc[j], ldf(v_cache + rows[j] * s.vdim + i), v[0]);
       o[i] = fmaf(o[i], c, (v[0] + v[1]) + (v[2] + v[3]));
     }
+    t0 = t0 < kept && t0 + n >= kept ? first : t0 + n;
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
-  for (int i = tid; i < s.vdim; i += 128) stf(y + row * ldy + h * s.vdim + i, o[i] * inv);     // (each thread reads what it wrote)
+  const float inv = offset ? 1.f : (l > 0.f ? 1.f / l : 0.f);
+  for (int i = tid; i < s.vdim; i += 128) {     // (each thread reads what it wrote)
+    T* d = y + row * ldy + h * s.vdim + i;
+    stf(d, mask.gated ? o[i] * inv / (1.f + expf(-ldf(d))) : o[i] * inv);
+  }
 }
 
 // out[i] = [keys of all kv heads | values of all kv heads] of cache slot slots[i]; dim and vdim in 16-byte pieces.
@@ -382,19 +403,19 @@ __global__ void gqa_gather_kernel(const uint4* __restrict__ k_cache, const uint4
 }
 }  // namespace
 
-// In place on the projected rows p: RMS norm (weight [dim]) and rotation of the first 2 * half dimensions (pairs (2i, 2i + 1), or (i, i + half)
+// In place on the projected rows p: RMS norm (weight [dim]; null: none) and rotation of the first 2 * half dimensions (pairs (2i, 2i + 1), or (i, i + half)
 // when `halves`) of every query and key head; v_first (row stride ld_first, null: none): values become (1 - share) v + share v_first; keys and
-// values of rows with a slot go to the cache.
+// values of rows with a slot go to the cache. own_kv 0: the rows hold queries only.
 RLB_API int rlb_gqa_prep(void* p, int f32, long long rows, long long ldp, int q_off, int k_off, int v_off, int heads, int kv_heads, int dim, int vdim,
                          int block_size, int num_blocks, const int* positions, const long long* slots, const void* q_norm, const void* k_norm,
-                         const float* freq, int half, int halves, float gain, float eps, const void* v_first, long long ld_first, const void* share,
+                         const float* freq, int half, int halves, float gain, float eps, const void* v_first, long long ld_first, const void* share, int own_kv,
                          void* k_cache, void* v_cache, int* status, void* stream) {
   if (rows <= 0) return 0;
   if (2 * half > dim || kv_heads < 1 || heads % kv_heads || (v_first && !share)) return -2;
-  GqaShape s{ldp, q_off, k_off, v_off, heads, kv_heads, dim, vdim, block_size, num_blocks, halves};
+  GqaShape s{ldp, q_off, k_off, v_off, heads, kv_heads, dim, vdim, block_size, num_blocks, halves, own_kv};
   const ValueMix<float> mix32{static_cast<const float*>(v_first), ld_first, static_cast<const float*>(share)};
   const ValueMix<__nv_bfloat16> mix16{static_cast<const __nv_bfloat16*>(v_first), ld_first, static_cast<const __nv_bfloat16*>(share)};
-  const int per_row = (heads + 2 * kv_heads + GP_WARPS - 1) / GP_WARPS;
+  const int per_row = (heads + (own_kv ? 2 * kv_heads : 0) + GP_WARPS - 1) / GP_WARPS;
   const dim3 grid(static_cast<unsigned>(rows), rows >= 148 * 8 ? 1 : (per_row < 64 ? per_row : 64)), block(GP_WARPS * 32);
   const size_t sm = sizeof(float2) * half;
   if (sm > 48 * 1024) return -2;
@@ -402,7 +423,7 @@ RLB_API int rlb_gqa_prep(void* p, int f32, long long rows, long long ldp, int q_
   if (!f32 && dim % 2 == 0 && vdim % 2 == 0 && ldp % 2 == 0 && dim <= 256 && (q_off | k_off | v_off) % 2 == 0 && (!halves || half % 2 == 0) &&
       ld_first % 2 == 0 && reinterpret_cast<uintptr_t>(v_first) % 4 == 0 &&
       static_cast<long long>(num_blocks) * block_size < 0x7fffffffll) {
-    const int share = (heads + kv_heads + 3) / 4;
+    const int share = (heads + (own_kv ? kv_heads : 0) + 3) / 4;
     const dim3 g(static_cast<unsigned>((rows + GP_WARPS - 1) / GP_WARPS), rows >= 148 * 16 ? 1 : (share < 64 ? share : 64));
     auto k = halves ? (dim <= 128 ? gqa_prep_rows_kernel<2, true> : gqa_prep_rows_kernel<4, true>)
                     : (dim <= 128 ? gqa_prep_rows_kernel<2, false> : gqa_prep_rows_kernel<4, false>);
@@ -421,21 +442,23 @@ RLB_API int rlb_gqa_prep(void* p, int f32, long long rows, long long ldp, int q_
 
 RLB_API int rlb_gqa_rows(const void* p, int f32, int rows, long long ldp, int q_off, int heads, int kv_heads, int dim, int vdim, int block_size,
                          int num_blocks, const void* k_cache, const void* v_cache, const int* block_table, int bt_stride, const int* seq_lens,
-                         int chunk, float scale, void* y, long long ldy, int* status, void* stream) {
+                         int chunk, int window, int keep, const void* offset, int gated, float scale, void* y, long long ldy, int* status, void* stream) {
   if (rows <= 0) return 0;
-  if (kv_heads < 1 || heads % kv_heads || heads > 65535 || dim + vdim > 12000) return -2;
-  GqaShape s{ldp, q_off, 0, 0, heads, kv_heads, dim, vdim, block_size, num_blocks, 0};
+  if (kv_heads < 1 || heads % kv_heads || heads > 65535 || dim + vdim > 12000 || (chunk > 0 && window > 0)) return -2;
+  GqaShape s{ldp, q_off, 0, 0, heads, kv_heads, dim, vdim, block_size, num_blocks, 0, 0};
+  const RowsMask mask{chunk, window, keep, gated};
   const size_t sm = sizeof(float) * ((dim + vdim + GR_TILE + 1) & ~1) + sizeof(long long) * GR_TILE;
   if (sm > 48 * 1024) return -2;
   const dim3 grid(rows, heads);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (f32)
     gqa_rows_kernel<float><<<grid, 128, sm, st>>>(static_cast<const float*>(p), s, static_cast<const float*>(k_cache), static_cast<const float*>(v_cache),
-                                                  block_table, bt_stride, seq_lens, chunk, scale, static_cast<float*>(y), ldy, status);
+                                                  block_table, bt_stride, seq_lens, mask, static_cast<const float*>(offset), scale, static_cast<float*>(y),
+                                                  ldy, status);
   else
     gqa_rows_kernel<__nv_bfloat16><<<grid, 128, sm, st>>>(static_cast<const __nv_bfloat16*>(p), s, static_cast<const __nv_bfloat16*>(k_cache),
-                                                          static_cast<const __nv_bfloat16*>(v_cache), block_table, bt_stride, seq_lens, chunk, scale,
-                                                          static_cast<__nv_bfloat16*>(y), ldy, status);
+                                                          static_cast<const __nv_bfloat16*>(v_cache), block_table, bt_stride, seq_lens, mask,
+                                                          static_cast<const __nv_bfloat16*>(offset), scale, static_cast<__nv_bfloat16*>(y), ldy, status);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -9,11 +9,14 @@
 //               has read the current one, i.e. under the softmax and the PV product, the next V tile under the next QK and softmax
 //   warp 1      tcgen05.mma issuer: S = Q K^T over dim + rot_dim in 16-wide steps, O += P V
 //   warps 2..5  softmax, one thread per query row, stale-maximum rescaling; the epilogue normalises and, where the output columns hold
-//               gates, multiplies by sigmoid(gate)
+//               gates, multiplies by sigmoid(gate). With sigmoid weights (SIG) there is no maximum and no sum: every visible key weighs
+//               sigmoid(score + a number per head), O only accumulates
 // The same kernel serves grouped-query attention (rlb_flash_gqa): no rotated source of its own (the rotation is in the queries and keys), several
-// query heads per key / value head, keys and values read from column ranges of one matrix, no gate, output rows of their own.
+// query heads per key / value head, keys and values read from column ranges of one matrix, a gate or none.
 // Query rows stand at the end of their context: row r of a portion of n tokens in a context of c sees keys up to c - n + r. With chunks of C
 // positions (the context then begins at a chunk's border) row i sees keys from i - i % C on, and a tile starts where its first row's chunk does.
+// With a window of W and the first K tokens kept it sees keys j with i - j < W or j < K: a tile visits the kept tokens' tiles and those from its
+// first row's window on. The context may leave out whole tiles between the two (`skip` positions per portion).
 #include "common.cuh"
 
 #include <math.h>
@@ -58,8 +61,24 @@ struct FlashLatentParams {
   int ctx_row0;                    // row of the key / value matrix that cu_ctx counts from
   int gated;
   int chunk;                       // > 0: keys of the row's own chunk only
+  int window, keep;                // window > 0: keys nearer than that, or among the first `keep` tokens
+  const int* skip;                 // [portions] positions left out of the context behind the kept tokens' tiles (null: none)
+  const __nv_bfloat16* offset;     // [heads] added to the scaled scores (sigmoid weights)
 };
 
+// 1 / (1 + 2^x_i) for four x (above 30 they count as 30): one reciprocal serves all of them.
+__device__ __forceinline__ void la_sigmoid4(float (&x)[4]) {
+  float d[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) d[i] = 1.f + exp2f(fminf(x[i], 30.f));
+  const float ab = d[0] * d[1], cd = d[2] * d[3], r = __fdividef(1.f, ab * cd), rab = r * cd, rcd = r * ab;
+  x[0] = rab * d[1];
+  x[1] = rab * d[0];
+  x[2] = rcd * d[3];
+  x[3] = rcd * d[2];
+}
+
+template <bool SIG>
 __global__ void __launch_bounds__(LA_THREADS, 2)
 flash_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_kv,
                     const __grid_constant__ CUtensorMap tmap_lat, FlashLatentParams p) {
@@ -74,7 +93,7 @@ flash_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
   uint64_t *q_full = bars, *k_full = bars + 1, *v_full = bars + 2, *k_empty = bars + 3, *v_empty = bars + 4, *s_full = bars + 5, *p_full = bars + 6;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 7);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
-  int* info = reinterpret_cast<int*>(tmem_slot + 2);   // first query row, portion rows, tile, first context row, context rows, valid
+  int* info = reinterpret_cast<int*>(tmem_slot + 2);   // first query row, portion rows, tile, first context row, context rows, valid, skip
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int head = blockIdx.y;
@@ -93,6 +112,7 @@ flash_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
       info[2] = tile;
       info[3] = p.cu_ctx[s];
       info[4] = p.cu_ctx[s + 1] - p.cu_ctx[s];
+      info[6] = p.skip ? p.skip[s] : 0;
     }
     for (int i = 0; i < 6; ++i) mbar_init(smem_u32(bars + i), 1);
     mbar_init(smem_u32(p_full), 128);
@@ -112,9 +132,18 @@ flash_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
   const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + 64;
   const int q_row0 = p.row0 + info[0], n_q = info[1], q0 = info[2] * LA_BQ, c_row0 = p.ctx_row0 + info[3], n_ctx = info[4];
   const int q_rows = min(LA_BQ, n_q - q0);
-  const int shift = n_ctx - n_q;                                     // query row i of the portion sees keys <= shift + i
-  const int first_tile = p.chunk > 0 ? (shift + q0) / p.chunk * p.chunk / LA_BKV : 0;
-  const int n_kv = (shift + q0 + q_rows + LA_BKV - 1) / LA_BKV - first_tile;      // tiles of 64 keys
+  const int skip = info[6];
+  const int shift = n_ctx - n_q + skip;                              // query row i of the portion sees keys <= shift + i
+  // tiles of 64 context rows: the kept tokens' (`sinks` of them, when tiles that no row sees follow), then all from first_tile on
+  const int lo0 = p.chunk > 0 ? (shift + q0) / p.chunk * p.chunk : (p.window > 0 ? max(0, shift + q0 - p.window + 1) : 0);
+  const int kept_tiles = p.window > 0 ? (p.keep + LA_BKV - 1) / LA_BKV : 0;
+  int first_tile = max(0, lo0 - skip) / LA_BKV, sinks = kept_tiles;
+  if (first_tile <= kept_tiles) {
+    sinks = 0;
+    if (kept_tiles > 0) first_tile = 0;
+  }
+  const int n_kv = sinks + (shift - skip + q0 + q_rows + LA_BKV - 1) / LA_BKV - first_tile;
+  auto tile_of = [&](int j) { return j < sinks ? j : first_tile + j - sinks; };
 
   if (warp == 0) {
     if (lane == 0) {
@@ -127,7 +156,7 @@ flash_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
         tma_load_2d(smem_u32(q_s + a * LA_Q_ATOM), &tmap_q, smem_u32(q_full), a < p.atoms_n ? qx + a * 64 : qx + p.dim + (a - p.atoms_n) * 64, q_row0 + q0);
       for (int j = 0; j < n_kv; ++j) {
         const uint32_t ph = j & 1;
-        const int row = c_row0 + (first_tile + j) * LA_BKV;
+        const int row = c_row0 + tile_of(j) * LA_BKV;
         if (!mbar_wait(smem_u32(k_empty), ph ^ 1, abort_flag, p.status, RLB_ERR_WAIT_EMPTY)) break;
         mbar_arrive_expect_tx(smem_u32(k_full), atoms_q * LA_KV_ATOM);
         for (int a = 0; a < p.atoms_n; ++a) tma_load_2d(smem_u32(k_s + a * LA_KV_ATOM), &tmap_kv, smem_u32(k_full), p.k_col + head / p.per_kv * p.dim + a * 64, row);
@@ -174,7 +203,10 @@ flash_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
     const int quarter = warp & 3, r = quarter * 32 + lane;
     const uint32_t lane_addr = static_cast<uint32_t>(quarter * 32) << 16;
     const int qi = shift + q0 + r;      // last key this row sees
-    const int lo = p.chunk > 0 ? qi - qi % p.chunk : 0, lo_last = p.chunk > 0 ? (shift + q0 + LA_BQ - 1) / p.chunk * p.chunk : 0;      // first key
+    // first key behind the kept ones: of this row, of the last row
+    const int lo = p.chunk > 0 ? qi - qi % p.chunk : (p.window > 0 ? max(0, qi - p.window + 1) : 0), last = shift + q0 + LA_BQ - 1;
+    const int lo_last = p.chunk > 0 ? last / p.chunk * p.chunk : (p.window > 0 ? max(0, last - p.window + 1) : 0);
+    const float off = SIG ? __bfloat162float(p.offset[head]) * LA_LOG2E : 0.f;
     float m_ref = -INFINITY, l = 0.f;
     bool ok = true;
     for (int j = 0; j < n_kv; ++j) {
@@ -187,60 +219,90 @@ flash_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
       tmem_ld_32x32b_x32(tmem_s + lane_addr, s0);
       tmem_ld_32x32b_x32(tmem_s + lane_addr + 32, s1);
       tmem_ld_wait();
-      const int k0 = (first_tile + j) * LA_BKV;
-      const bool edge = k0 + LA_BKV - 1 > shift + q0 || k0 < lo_last;
-      float mx = -INFINITY;
-#pragma unroll
-      for (int i = 0; i < 32; ++i) {
-        float a = __uint_as_float(s0[i]) * p.scale_log2, b = __uint_as_float(s1[i]) * p.scale_log2;
-        if (edge) {
-          if (k0 + i > qi || k0 + i < lo) a = -INFINITY;
-          if (k0 + 32 + i > qi || k0 + 32 + i < lo) b = -INFINITY;
-        }
-        s0[i] = __float_as_uint(a);
-        s1[i] = __float_as_uint(b);
-        mx = fmaxf(mx, fmaxf(a, b));
-      }
-      float factor = 1.f;
-      bool need = false;
-      if (mx > m_ref + LA_RESCALE || m_ref == -INFINITY) {
-        const float m_new = fmaxf(mx, m_ref);
-        if (m_new != -INFINITY) {
-          factor = m_ref == -INFINITY ? 0.f : exp2f(m_ref - m_new);
-          need = m_ref != -INFINITY;
-          m_ref = m_new;
-        }
-      }
-      l *= factor;
-      float rowsum = 0.f;
+      const int tile = tile_of(j), k0 = tile * LA_BKV + (tile >= kept_tiles ? skip : 0);
+      const bool edge = k0 + LA_BKV - 1 > shift + q0 || (k0 < lo_last && k0 + LA_BKV > p.keep);
       uint32_t pk[32];
-      const float mr = m_ref == -INFINITY ? 0.f : m_ref;
+      if constexpr (SIG) {
 #pragma unroll
-      for (int i = 0; i < 16; ++i) {
-        const float e0 = exp2f(__uint_as_float(s0[2 * i]) - mr), e1 = exp2f(__uint_as_float(s0[2 * i + 1]) - mr);
-        const float f0 = exp2f(__uint_as_float(s1[2 * i]) - mr), f1 = exp2f(__uint_as_float(s1[2 * i + 1]) - mr);
-        rowsum += (e0 + e1) + (f0 + f1);
-        pk[i] = pack_bf16x2(e0, e1);
-        pk[16 + i] = pack_bf16x2(f0, f1);
-      }
-      l += rowsum;
-      if (j > 0) {
-        if (!mbar_wait(smem_u32(v_empty), (j - 1) & 1, abort_flag, p.status, RLB_ERR_WAIT_TMEM_EMPTY)) {
+        for (int i = 0; i < 32; i += 4) {
+          float a[4], b[4];
+#pragma unroll
+          for (int q = 0; q < 4; ++q) {
+            a[q] = -fmaf(__uint_as_float(s0[i + q]), p.scale_log2, off);
+            b[q] = -fmaf(__uint_as_float(s1[i + q]), p.scale_log2, off);
+          }
+          la_sigmoid4(a);
+          la_sigmoid4(b);
+          if (edge) {
+#pragma unroll
+            for (int q = 0; q < 4; ++q) {
+              const int ka = k0 + i + q, kb = ka + 32;
+              if (ka > qi || (ka < lo && ka >= p.keep)) a[q] = 0.f;
+              if (kb > qi || (kb < lo && kb >= p.keep)) b[q] = 0.f;
+            }
+          }
+          pk[i / 2] = pack_bf16x2(a[0], a[1]);
+          pk[i / 2 + 1] = pack_bf16x2(a[2], a[3]);
+          pk[16 + i / 2] = pack_bf16x2(b[0], b[1]);
+          pk[16 + i / 2 + 1] = pack_bf16x2(b[2], b[3]);
+        }
+        if (j > 0 && !mbar_wait(smem_u32(v_empty), (j - 1) & 1, abort_flag, p.status, RLB_ERR_WAIT_TMEM_EMPTY)) {
           ok = false;
           break;
         }
-        tc_fence_after();
-      }
-      if (__any_sync(0xffffffffu, need)) {
-        for (int c = 0; c < p.vcols; c += 32) {   // (the last 32 columns may reach past vcols: allocated, never read as output)
-          uint32_t o[32];
-          tmem_ld_32x32b_x32(tmem_o + lane_addr + c, o);
-          tmem_ld_wait();
+      } else {
+        float mx = -INFINITY;
 #pragma unroll
-          for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * factor);
-          la_tmem_st_x32(tmem_o + lane_addr + c, o);
+        for (int i = 0; i < 32; ++i) {
+          float a = __uint_as_float(s0[i]) * p.scale_log2, b = __uint_as_float(s1[i]) * p.scale_log2;
+          if (edge) {
+            if (k0 + i > qi || (k0 + i < lo && k0 + i >= p.keep)) a = -INFINITY;
+            if (k0 + 32 + i > qi || (k0 + 32 + i < lo && k0 + 32 + i >= p.keep)) b = -INFINITY;
+          }
+          s0[i] = __float_as_uint(a);
+          s1[i] = __float_as_uint(b);
+          mx = fmaxf(mx, fmaxf(a, b));
         }
-        tmem_st_wait();
+        float factor = 1.f;
+        bool need = false;
+        if (mx > m_ref + LA_RESCALE || m_ref == -INFINITY) {
+          const float m_new = fmaxf(mx, m_ref);
+          if (m_new != -INFINITY) {
+            factor = m_ref == -INFINITY ? 0.f : exp2f(m_ref - m_new);
+            need = m_ref != -INFINITY;
+            m_ref = m_new;
+          }
+        }
+        l *= factor;
+        float rowsum = 0.f;
+        const float mr = m_ref == -INFINITY ? 0.f : m_ref;
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const float e0 = exp2f(__uint_as_float(s0[2 * i]) - mr), e1 = exp2f(__uint_as_float(s0[2 * i + 1]) - mr);
+          const float f0 = exp2f(__uint_as_float(s1[2 * i]) - mr), f1 = exp2f(__uint_as_float(s1[2 * i + 1]) - mr);
+          rowsum += (e0 + e1) + (f0 + f1);
+          pk[i] = pack_bf16x2(e0, e1);
+          pk[16 + i] = pack_bf16x2(f0, f1);
+        }
+        l += rowsum;
+        if (j > 0) {
+          if (!mbar_wait(smem_u32(v_empty), (j - 1) & 1, abort_flag, p.status, RLB_ERR_WAIT_TMEM_EMPTY)) {
+            ok = false;
+            break;
+          }
+          tc_fence_after();
+        }
+        if (__any_sync(0xffffffffu, need)) {
+          for (int c = 0; c < p.vcols; c += 32) {   // (the last 32 columns may reach past vcols: allocated, never read as output)
+            uint32_t o[32];
+            tmem_ld_32x32b_x32(tmem_o + lane_addr + c, o);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * factor);
+            la_tmem_st_x32(tmem_o + lane_addr + c, o);
+          }
+          tmem_st_wait();
+        }
       }
 #pragma unroll
       for (int c = 0; c < 8; ++c)
@@ -251,7 +313,7 @@ flash_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_con
     }
     if (ok && mbar_wait(smem_u32(v_empty), (n_kv - 1) & 1, abort_flag, p.status, RLB_ERR_WAIT_TMEM_EMPTY)) {
       tc_fence_after();
-      const float inv_l = l > 0.f ? 1.f / l : 0.f;
+      const float inv_l = SIG ? 1.f : (l > 0.f ? 1.f / l : 0.f);
       __nv_bfloat16* dst = p.p + static_cast<long long>(q_row0 + q0 + r) * p.ldp + p.mix_off + head * p.vdim;
       for (int c = 0; c < p.vdim; c += 32) {
         uint32_t o[32];
@@ -309,13 +371,15 @@ __global__ void latent_gather_kernel(const uint4* __restrict__ cache, const long
 
 int launch_flash(const CUtensorMap& tq, const CUtensorMap& tkv, const CUtensorMap& tl, const FlashLatentParams& f, int max_tiles, cudaStream_t stream) {
   const int smem = (f.atoms_n + f.atoms_r) * (LA_Q_ATOM + LA_KV_ATOM) + f.atoms_v * LA_KV_ATOM + LA_P_BYTES + 256 + 1024;
-  static int configured = 0;
-  if (smem > configured) {
-    cudaError_t e = cudaFuncSetAttribute(flash_latent_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  static int configured[2] = {0, 0};
+  const bool sig = f.offset != nullptr;
+  auto kernel = sig ? flash_latent_kernel<true> : flash_latent_kernel<false>;
+  if (smem > configured[sig]) {
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return static_cast<int>(e);
-    configured = smem;
+    configured[sig] = smem;
   }
-  flash_latent_kernel<<<dim3(max_tiles, f.heads), LA_THREADS, smem, stream>>>(tq, tkv, tl, f);
+  kernel<<<dim3(max_tiles, f.heads), LA_THREADS, smem, stream>>>(tq, tkv, tl, f);
   return static_cast<int>(cudaGetLastError());
 }
 }  // namespace
@@ -387,13 +451,16 @@ RLB_API int rlb_flash_latent(const void* q, long long rows, long long ldq, int q
 
 // Grouped-query attention of prompt portions. p: projected rows with normed and rotated queries at q_off; the portions are its rows
 // [row0, row0 + cu_q[portions]). Keys of kv head g: columns [k_col + g * dim, + dim) of kv [kv_rows, kv_width], values [v_col + g * vdim, + vdim);
-// row ctx_row0 + cu_ctx[i] is the first of portion i's context (kv may be p itself), with chunk > 0 the first of a chunk. y [rows, heads * vdim]:
-// outputs. dim a multiple of 16, vdim of 8.
+// row ctx_row0 + cu_ctx[i] is the first of portion i's context (kv may be p itself), with chunk > 0 the first of a chunk. window > 0: keys
+// j with i - j < window or j < keep; skip [portions] (null: zeros; multiples of 64): positions that portion i's context leaves out behind its first
+// ceil(keep / 64) * 64 rows. offset [heads] (bf16; null: soft-max): the weights are sigmoid(score + offset), unnormalised. y (row stride ldy, may be
+// the rows of p): head outputs, with `gated` multiplied by sigmoid of what stands there. dim a multiple of 16, vdim of 8.
 RLB_API int rlb_flash_gqa(void* p, long long rows, long long ldp, int in_width, int row0, const void* kv, long long kv_rows, long long ldkv, int kv_width,
                           int ctx_row0, int k_col, int v_col, const int* cu_q, const int* cu_ctx, int portions, int heads, int kv_heads, int dim, int vdim,
-                          int q_off, int chunk, float scale, int max_tiles, void* y, long long ldy, int* status, void* stream) {
+                          int q_off, int chunk, int window, int keep, const int* skip, const void* offset, int gated, float scale, int max_tiles, void* y, long long ldy,
+                          int* status, void* stream) {
   if (portions <= 0 || rows <= 0 || max_tiles <= 0) return 0;
-  if (!rlb_flash_latent_supported(dim, 0, vdim, 8) || kv_heads < 1 || heads % kv_heads) return -2;
+  if (!rlb_flash_latent_supported(dim, 0, vdim, 8) || kv_heads < 1 || heads % kv_heads || (chunk > 0 && window > 0) || (skip && window <= 0)) return -2;
   if (ldp % 8 || ldkv % 8 || ldy % 8 || q_off % 8 || k_col % 8 || v_col % 8 || heads > 65535) return -2;
   if ((reinterpret_cast<uintptr_t>(p) | reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(y)) & 15) return -3;
   FlashLatentParams f{};
@@ -418,6 +485,11 @@ RLB_API int rlb_flash_gqa(void* p, long long rows, long long ldp, int in_width, 
   f.v_col = v_col;
   f.ctx_row0 = ctx_row0;
   f.chunk = chunk;
+  f.window = window;
+  f.keep = window > 0 ? keep : 0;
+  f.skip = skip;
+  f.offset = static_cast<const __nv_bfloat16*>(offset);
+  f.gated = gated;
   CUtensorMap tq, tkv;
   int rc = rlb_make_tmap_2d(&tq, p, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, in_width, rows, ldp * 2, 64, LA_BQ, CU_TENSOR_MAP_SWIZZLE_128B);
   if (rc) return -100 - rc;

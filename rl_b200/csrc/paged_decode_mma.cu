@@ -10,7 +10,9 @@
 // CUDA cores never touch K or V. Warp roles: warp 0 streams K and V tiles with TMA (one buffer each; the next K tile is
 // requested as soon as the QK MMAs of the current one have completed, the next V tile after the PV MMAs), warp 1 issues
 // the MMAs, warps 2-5 own one token row of S^T / one dim row of O^T each and keep the running max / sum / output in
-// registers. Every wait is bounded (status word, no hang). With chunks of C positions only the keys of the query's own chunk are read.
+// registers. Every wait is bounded (status word, no hang). With chunks of C positions only the keys of the query's own chunk are read,
+// with a window of W and K kept first tokens the keys nearer than W and the first K. With sigmoid weights (SIG) there is no running maximum and no
+// sum: a key weighs sigmoid(score + a number per head), splits only add up. Where the output's place holds gates, out = y * sigmoid(gate).
 //
 // The CUDA-core kernel in paged_decode_tma.cu (same contract) is kept as the fallback for block sizes / head dims this
 // kernel does not cover. Reference counterpart: the FlashInfer / vLLM paged-attention decode kernels behind
@@ -47,7 +49,14 @@ struct DmParams {
   long long out_stride;
   int* status;
   int chunk;               // > 0: only the query's own run of `chunk` positions is visible
+  int window, keep;        // window > 0: only keys nearer than that, or among the first `keep` tokens
+  const __nv_bfloat16* offset;   // [Hq] added to the scaled scores (sigmoid weights)
+  int gated;
 };
+
+__device__ __forceinline__ float dm_gated(float v, const __nv_bfloat16* gate, int gated) {
+  return gated ? v / (1.f + __expf(-__bfloat162float(*gate))) : v;
+}
 
 __device__ __forceinline__ void named_bar_sync(int id, int count) {
   asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(count) : "memory");
@@ -60,6 +69,7 @@ __device__ __forceinline__ uint32_t sw128_off(int row, int col, int chunk_bytes)
   return chunk * chunk_bytes + (row >> 3) * 1024 + (row & 7) * 128 + ((((c * 2) >> 4) ^ (row & 7)) << 4) + ((c * 2) & 15);
 }
 
+template <bool SIG>
 __global__ void __launch_bounds__(DM_THREADS, 2)
 paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v, DmParams p) {
   extern __shared__ uint8_t smem_raw[];
@@ -109,13 +119,20 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
   const int G = p.G, Hq = p.Hkv * G;
   const int len = p.seq_lens[seq];
   const int bs = p.block_size;
-  const int t_first = p.chunk > 0 && len > 0 ? (len - 1) / p.chunk * p.chunk : 0, t_base = t_first / DM_TOK * DM_TOK;      // first key, its tile
-  const int per_split = ((len - t_base + p.num_splits - 1) / p.num_splits + DM_TOK - 1) / DM_TOK * DM_TOK;
-  const int t_begin = t_base + split * per_split;
-  const int t_end = min(len, t_begin + per_split);
-  const int n_tiles = t_end > t_begin ? (t_end - t_begin + DM_TOK - 1) / DM_TOK : 0;
+  // first key behind the kept ones; tiles of 128 keys: the kept tokens' (`sinks` of them, when unseen ones follow), then all from first_tile on
+  const int t_first = len <= 0 ? 0 : (p.chunk > 0 ? (len - 1) / p.chunk * p.chunk : (p.window > 0 ? max(0, len - p.window) : 0));
+  const int keep = p.window > 0 ? p.keep : 0, kept_tiles = (keep + DM_TOK - 1) / DM_TOK;
+  int first_tile = t_first / DM_TOK, sinks = kept_tiles;
+  if (first_tile <= kept_tiles) {
+    sinks = 0;
+    if (keep > 0) first_tile = 0;
+  }
+  const int all_tiles = len > 0 ? sinks + (len + DM_TOK - 1) / DM_TOK - first_tile : 0;
+  const int per_split = (all_tiles + p.num_splits - 1) / p.num_splits;
+  const int i_begin = split * per_split, n_tiles = max(0, min(all_tiles, i_begin + per_split) - i_begin);
+  auto tile_start = [&](int i) { return (i_begin + i < sinks ? i_begin + i : first_tile + i_begin + i - sinks) * DM_TOK; };
 
-  // Q (pre-scaled) and a zeroed P^T, both in the swizzled K-major operand layout: 256 pieces of 16 bytes each
+  // Q (pre-scaled for the soft-max) and a zeroed P^T, both in the swizzled K-major operand layout: 256 pieces of 16 bytes each
   for (int i = threadIdx.x; i < 2 * DM_QP_BYTES / 16; i += DM_THREADS) {
     uint4 val = make_uint4(0, 0, 0, 0);
     const int which = i / (DM_QP_BYTES / 16);          // 0: Q, 1: P
@@ -129,7 +146,7 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
         const float2 f = unpack_bf16x2(w[k]);
-        o[k] = pack_bf16x2(f.x * p.scale, f.y * p.scale);
+        o[k] = SIG ? w[k] : pack_bf16x2(f.x * p.scale, f.y * p.scale);
       }
       val = make_uint4(o[0], o[1], o[2], o[3]);
     }
@@ -152,7 +169,7 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
       bool ok = true;
       for (int i = 0; i < n_tiles && ok; ++i) {
         const uint32_t ph = i & 1;
-        const int t0 = t_begin + i * DM_TOK;
+        const int t0 = tile_start(i);
         for (int kv = 0; kv < 2 && ok; ++kv) {
           uint64_t* empty = kv == 0 ? k_empty : v_empty;
           uint64_t* full = kv == 0 ? k_full : v_full;
@@ -230,6 +247,9 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
       l_run[g] = 0.f;
       o_run[g] = 0.f;
     }
+    float off[8];
+#pragma unroll
+    for (int g = 0; g < 8; ++g) off[g] = SIG && g < G ? __bfloat162float(p.offset[kvh * G + g]) : 0.f;
     float* red_max = red;                 // [4][16]
     float* red_sum = red + 4 * DM_N;      // [4][16]
     bool ok = true;
@@ -246,8 +266,32 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(s_empty));
-      const int tok = t_begin + i * DM_TOK + r;
-      const bool valid = tok >= t_first && tok < t_end;
+      const int tok = tile_start(i) + r;
+      const bool valid = tok < len && (tok >= t_first || tok < keep);
+      if constexpr (SIG) {
+#pragma unroll
+        for (int g = 0; g < 8; ++g) {
+          const float z = fmaf(__uint_as_float(sr[g]), p.scale, off[g]);
+          if (g < G) *reinterpret_cast<__nv_bfloat16*>(p_sm + sw128_off(g, r, DM_N * 128)) = __float2bfloat16(valid ? 1.f / (1.f + __expf(-z)) : 0.f);
+        }
+        fence_proxy_async();         // P^T is read by the tensor core (async proxy)
+        named_bar_sync(1, 128);
+        if (threadIdx.x == 64) mbar_arrive(smem_u32(p_ready));
+        if (!mbar_wait(smem_u32(o_full), ph, abort_flag, p.status, RLB_ERR_WAIT_TMEM_FULL)) {
+          ok = false;
+          break;
+        }
+        tc_fence_after();
+        uint32_t orr[16];
+        tmem_ld_32x32b_x16(tmem_o + lane_addr, orr);
+        tmem_ld_wait();
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(smem_u32(o_empty));
+#pragma unroll
+        for (int g = 0; g < 8; ++g) o_run[g] += __uint_as_float(orr[g]);
+        continue;
+      }
       float s[8], pr[8], c[8];
 #pragma unroll
       for (int g = 0; g < 8; ++g) {
@@ -298,11 +342,12 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
       if (g >= G) break;
       const int hq = kvh * G + g;
       if (p.num_splits == 1) {
-        p.out[seq * p.out_stride + static_cast<long long>(hq) * DM_D + r] = __float2bfloat16(l_run[g] > 0.f ? o_run[g] / l_run[g] : 0.f);
+        __nv_bfloat16* dst = p.out + seq * p.out_stride + static_cast<long long>(hq) * DM_D + r;
+        *dst = __float2bfloat16(dm_gated(SIG ? o_run[g] : (l_run[g] > 0.f ? o_run[g] / l_run[g] : 0.f), dst, p.gated));
       } else {
         const long long pi = (static_cast<long long>(seq) * Hq + hq) * p.num_splits + split;
         p.part_o[pi * DM_D + r] = o_run[g];
-        if (r == 0) {
+        if (!SIG && r == 0) {
           p.part_ml[pi * 2] = m_run[g];
           p.part_ml[pi * 2 + 1] = l_run[g];
         }
@@ -317,11 +362,18 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid
   }
 }
 
-__global__ void dm_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int num_splits, int Hq,
+__global__ void dm_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int num_splits, int Hq, int sig, int gated,
                                   __nv_bfloat16* __restrict__ out, long long out_stride) {
   pdl_sync();
   const int seq = blockIdx.x, hq = blockIdx.y, d = threadIdx.x;
   const long long base = (static_cast<long long>(seq) * Hq + hq) * num_splits;
+  __nv_bfloat16* dst = out + seq * out_stride + static_cast<long long>(hq) * DM_D + d;
+  if (sig) {
+    float acc = 0.f;
+    for (int s = 0; s < num_splits; ++s) acc += part_o[(base + s) * DM_D + d];
+    *dst = __float2bfloat16(dm_gated(acc, dst, gated));
+    return;
+  }
   float mm = -INFINITY;
   for (int s = 0; s < num_splits; ++s) mm = fmaxf(mm, part_ml[(base + s) * 2]);
   float ll = 0.f, acc = 0.f;
@@ -331,20 +383,22 @@ __global__ void dm_combine_kernel(const float* __restrict__ part_o, const float*
     ll += part_ml[(base + s) * 2 + 1] * c;
     acc += part_o[(base + s) * DM_D + d] * c;
   }
-  out[seq * out_stride + static_cast<long long>(hq) * DM_D + d] = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
+  *dst = __float2bfloat16(dm_gated(ll > 0.f ? acc / ll : 0.f, dst, gated));
 }
 }  // namespace
 
-// Same contract as rlb_paged_decode_tma; chunk > 0: only the query's own chunk of positions is visible. Supported: head_dim 128, Hq / Hkv <= 8, block_size 16, 32, 64 or a multiple of 128.
+// Same contract as rlb_paged_decode_tma; chunk > 0: only the query's own chunk of positions is visible; window > 0: only keys nearer than
+// that or among the first `keep`; offset [Hq] (null: soft-max): weights sigmoid(score + offset); gated: out holds gates. Supported: head_dim 128, Hq / Hkv <= 8, block_size 16, 32, 64 or a multiple of 128.
 RLB_API int rlb_paged_decode_mma(const void* q, long long q_stride, const void* k_cache, const void* v_cache, int num_blocks,
                                  const int* block_table, int max_blocks_per_seq, const int* seq_lens, int B, int Hq, int Hkv, int D,
-                                 int block_size, int chunk, float scale, int num_splits, float* part_o, float* part_ml, void* out,
+                                 int block_size, int chunk, int window, int keep, const void* offset, int gated, float scale, int num_splits, float* part_o, float* part_ml, void* out,
                                  long long out_stride, int* status, void* stream) {
   if (B <= 0) return 0;
   if (D != DM_D || Hq % Hkv || Hq / Hkv > 8) return -2;
   if (!(block_size == 16 || block_size == 32 || block_size == 64 || block_size % 128 == 0)) return -2;
   if (num_splits < 1) num_splits = 1;
   if (num_splits > 1 && (!part_o || !part_ml)) return -3;
+  if (chunk > 0 && window > 0) return -2;
   const int box_rows = block_size < DM_TOK ? block_size : DM_TOK;
   const unsigned long long rows = static_cast<unsigned long long>(num_blocks) * Hkv * block_size;
   CUtensorMap tk, tv;
@@ -371,18 +425,24 @@ RLB_API int rlb_paged_decode_mma(const void* q, long long q_stride, const void* 
   p.out_stride = out_stride;
   p.status = status;
   p.chunk = chunk;
-  static bool configured = false;
-  if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(paged_decode_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, DM_SMEM);
+  p.window = window;
+  p.keep = keep;
+  p.offset = static_cast<const __nv_bfloat16*>(offset);
+  p.gated = gated;
+  static bool configured[2] = {false, false};
+  const bool sig = offset != nullptr;
+  auto kernel = sig ? paged_decode_mma_kernel<true> : paged_decode_mma_kernel<false>;
+  if (!configured[sig]) {
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, DM_SMEM);
     if (e != cudaSuccess) return static_cast<int>(e);
-    configured = true;
+    configured[sig] = true;
   }
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   dim3 grid(B, Hkv, num_splits);
-  rlb_launch_pdl(paged_decode_mma_kernel, grid, dim3(DM_THREADS), DM_SMEM, s, tk, tv, p);
+  rlb_launch_pdl(kernel, grid, dim3(DM_THREADS), DM_SMEM, s, tk, tv, p);
   if (num_splits > 1) {
     dim3 g2(B, Hq);
-    rlb_launch_pdl(dm_combine_kernel, g2, dim3(DM_D), 0, s, part_o, part_ml, num_splits, Hq, static_cast<__nv_bfloat16*>(out), out_stride);
+    rlb_launch_pdl(dm_combine_kernel, g2, dim3(DM_D), 0, s, part_o, part_ml, num_splits, Hq, static_cast<int>(sig), gated, static_cast<__nv_bfloat16*>(out), out_stride);
   }
   return static_cast<int>(cudaGetLastError());
 }
