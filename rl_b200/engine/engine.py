@@ -434,7 +434,7 @@ class GenerationEngine:
         # ``_hybrid_block``. Prefixes are not shared between sequences (pages carry no state) and decode runs eagerly.
         self.hybrid = bool(self.cfg.is_hybrid)
         self._attn_layers = [i for i, l in enumerate(model.layers) if l.self_attn is not None]
-        # layer-list models (Gadarax, Redarax, Kikivik): one cache or state pool per layer RUN (a looped layer has one per pass), see ``_mixer_forward``
+        # layer-list models (Gadarax, Redarax, Kikivik, Zonidra): one cache or state pool per layer RUN (a looped layer has one per pass), see ``_mixer_forward``
         self.mixer = bool(self.cfg.is_mixer)
         self.runs = self.cfg.layer_runs if self.mixer else []
         self.stateful = bool(self.cfg.is_recurrent)   # sequences own a row of the state pools: prefixes are not shared by pages
@@ -454,6 +454,7 @@ class GenerationEngine:
         self.latent_cache: Optional[list] = None      # per run: [pages, page size, latent width] (latent attention)
         self.rec_state: Optional[list] = None         # per run: [state rows, heads, dim, vdim] fp32 (retention, Mamba-2, delta rule)
         self.conv_ring: Optional[list] = None         # per run: [state rows, taps, channels], last inputs of a short convolution
+        self.carry: Optional[Y.Carry] = None          # per sequence: last token, its normed stream where the next token blends it in
         self._step_ids: dict = {}                     # requests driven through ``step``: caller's id -> sequence id
         self._step_next = 0
         self._state_row: dict[int, int] = {}
@@ -561,22 +562,31 @@ class GenerationEngine:
         """Elements per token that a layer keeps in pages."""
         m = self.model.layers[layer].mixer
         if m.kind == "attention":
-            return m.kv_heads * (m.dim + m.vdim)
+            return m.kv_heads * (m.dim + m.vdim) if m.kv_from is None else 0
         return m.latent_width if m.kind == "latent_attention" else 0
 
     def _wake_mixer(self) -> None:
-        """Pools of a layer-list model, one per layer run: key / value pages for attention, latent pages for latent attention, fp32 state rows
-        (row 0 is scratch for the padding rows of a decode batch) for the recurrent mixers, with the last inputs of their convolution."""
+        """Pools of a layer-list model, one per layer run: key / value pages for attention (a layer that reads
+        another one's has that one's), latent pages for latent attention, fp32 state rows (row 0 is scratch for the padding rows of a decode batch) for the recurrent mixers, with the last inputs of their convolution."""
         dt, dev, n, bs = self.model.dtype, self.device, self.num_blocks, self.block_size
         mx = [self.model.layers[i].mixer for i, _ in self.runs]
         zeros = lambda *shape, dtype=dt: torch.zeros(shape, dtype=dtype, device=dev)   # noqa: E731
-        self.k_cache = [zeros(n, m.kv_heads, bs, m.dim) if m.kind == "attention" else None for m in mx]
-        self.v_cache = [zeros(n, m.kv_heads, bs, m.vdim) if m.kind == "attention" else None for m in mx]
+        own = [m.kind == "attention" and m.kv_from is None for m in mx]
+        self.k_cache = [zeros(n, m.kv_heads, bs, m.dim) if o else None for m, o in zip(mx, own)]
+        self.v_cache = [zeros(n, m.kv_heads, bs, m.vdim) if o else None for m, o in zip(mx, own)]
+        for r, m in enumerate(mx):
+            if m.kind == "attention" and m.kv_from is not None:
+                src = next(q for q, (i, _) in enumerate(self.runs) if i == m.kv_from)
+                self.k_cache[r], self.v_cache[r] = self.k_cache[src], self.v_cache[src]
         self.latent_cache = [zeros(n, bs, m.latent_width) if m.kind == "latent_attention" else None for m in mx]
         self.rec_state = [zeros(self.max_running + 1, m.heads, m.dim, m.vdim, dtype=torch.float32) if m.kind in RECURRENT_MIXERS else None for m in mx]
         self.conv_ring = [zeros(self.max_running + 1, m.taps, m.channels) if hasattr(m, "taps") else None for m in mx]
+        c = self.cfg
+        if c.token_shift or c.bigram:
+            self.carry = Y.Carry(self.max_running + 1, len(self.runs) if c.token_shift else 0, c.hidden_size, bool(c.bigram), dev)
         # portions of prompts attend tile-wise when every attention layer has a shape its tensor-core kernel takes
         tiles = {"latent_attention": X.portion_tiles, "attention": S.portion_tiles}
+        self._windows = sorted({(m.window, m.keep) for m in mx if getattr(m, "window", 0)})
         self._chunks = sorted({m.chunk for m in mx if getattr(m, "chunk", 0)})
         self._portion_tiles = self.native and all(tiles[m.kind](m, dt) for m in mx if m.kind in tiles)
 
@@ -592,7 +602,7 @@ class GenerationEngine:
             self._static = None
             self.k_cache = self.v_cache = None
             self.mamba_conv = self.mamba_ssm = None
-            self.latent_cache = self.rec_state = self.conv_ring = None
+            self.latent_cache = self.rec_state = self.conv_ring = self.carry = None
             if self.device.type == "cuda":
                 torch.cuda.empty_cache()
 
@@ -916,11 +926,20 @@ class GenerationEngine:
         return Y.capped_logits(h, m.output_weight, c.logit_scale, c.final_logit_softcap, self.logits_dtype)
 
     def _pre_norm_forward(self, b: "X.TokenBatch", rows: Optional[torch.Tensor] = None) -> torch.Tensor:
-        """``_mixer_forward`` of pre-norm layers. Each sublayer is a product, the mixer or gated unit, a product, and the step that joins its
-        output to the fp32 stream and applies the next sublayer's norm (the final norm behind the last)."""
+        """``_mixer_forward`` of pre-norm layers. Each sublayer is a product, the mixer or feed-forward, a product, and the step that joins its
+        output to the fp32 stream (normed and scaled where the model does that) and applies the next sublayer's norm (the final norm behind the
+        last) and blend with the token before."""
         m, c = self.model, self.cfg
-        eps, last, values = c.rms_norm_eps, len(self.runs) - 1, None
-        x, h = Y.embed(b.ids, m.embed_tokens, c.embed_scale, m.layers[self.runs[0][0]].norm1, eps)
+        eps, last, values, lent = c.rms_norm_eps, len(self.runs) - 1, None, {}
+
+        def blend(r):
+            return Y.Shift(m.layers[self.runs[r][0]].shift, r, self.carry, b) if c.token_shift and r <= last else None
+
+        norm = m.layers[self.runs[0][0]].norm1
+        if self.carry is not None:
+            x, h = Y.start(b, m.embed_tokens, c.embed_scale, norm, eps, m.bigram, c.bigram, blend(0) or Y.Shift(None, 0, self.carry, b))
+        else:
+            x, h = Y.embed(b.ids, m.embed_tokens, c.embed_scale, norm, eps)
         for r, (i, _) in enumerate(self.runs):
             layer = m.layers[i]
             mx, end = layer.mixer, m.norm if r == last else m.layers[self.runs[r + 1][0]].norm1
@@ -928,12 +947,19 @@ class GenerationEngine:
             if mx.kind == "latent_attention":
                 a = X.latent_attention(p, mx, b, self.latent_cache[r])
             else:
-                a = S.attention(p, mx, b, self.k_cache[r], self.v_cache[r], values if mx.v_mix else None)
+                if layer.lends:
+                    lent[i] = S.KeyValues(p, mx)
+                a = S.attention(p, mx, b, self.k_cache[r], self.v_cache[r], values if mx.v_mix else None, lent.get(i if mx.kv_from is None else mx.kv_from))
                 if mx.v_mix and values is None:
                     values = mx.values(p)
-            h = Y.add_normed_(x, Y.linear(a, mx.out_proj, getattr(mx, "out_bias", None)), None, 1.0, eps, end if layer.ff is None else layer.norm2)
-            if layer.ff is not None:
-                h = Y.feed_forward_(x, h, layer.ff, None, 1.0, eps, end)
+            y = Y.linear(a, mx.out_proj, getattr(mx, "out_bias", None))
+            if layer.ff is None:
+                x, h = Y.join(x, y, layer.norm1b, 1.0, eps, end, ls=layer.ls1, shift=blend(r + 1))
+            else:
+                x, h = Y.join(x, y, layer.norm1b, 1.0, eps, layer.norm2, ls=layer.ls1)
+                x, h = Y.feed_forward(x, h, layer.ff, layer.norm2b, 1.0, eps, end, layer.ls2, blend(r + 1))
+        if self.carry is not None:
+            self.carry.commit(b)
         if rows is not None:
             h = h.index_select(0, rows)
         return X.logits(h, m.output_weight, self.logits_dtype)
@@ -977,6 +1003,16 @@ class GenerationEngine:
                 cu[1:] = torch.tensor([n - s for n, s in zip(ctx, lo)], dtype=torch.int64).cumsum(0)
                 slots = torch.cat([self.sched.slots(sids[j], s, n - s) for j, n, s in zip(tiled, ctx, lo)])
                 b.chunk_ctx[size] = (cu.to(dev), slots.to(dev), all(items[order[j]][2] == s for j, s in zip(tiled, lo)))
+            for size, keep in self._windows:    # and windows: whole tiles of kept first tokens, then from the window of each portion's first token on
+                k0, parts, skip = -(-keep // X.KEY_TILE) * X.KEY_TILE, [], []
+                for j, n in zip(tiled, ctx):
+                    lo = max(0, items[order[j]][2] - size + 1) // X.KEY_TILE * X.KEY_TILE
+                    skip.append(max(0, lo - k0))
+                    parts.append([(0, n)] if lo <= k0 else [(0, k0), (lo, n)])
+                cu = torch.zeros(len(tiled) + 1, dtype=torch.int32)
+                cu[1:] = torch.tensor([sum(e - s for s, e in q) for q in parts], dtype=torch.int64).cumsum(0)
+                slots_w = torch.cat([self.sched.slots(sids[j], s, e - s) for j, q in zip(tiled, parts) for s, e in q if e > s])
+                b.window_ctx[size, keep] = (cu.to(dev), slots_w.to(dev), torch.tensor(skip, dtype=torch.int32).to(dev))
         if self.stateful:
             srow = torch.tensor([self._state_row[s] for s in sids], dtype=torch.int64)
             b.state_rows, b.row_state = srow.to(dev), srow[of_row].to(dev)

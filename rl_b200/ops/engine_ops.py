@@ -100,16 +100,20 @@ def _paged_decode_gather(q, k_cache, v_cache, block_table, seq_lens, Hq, Hkv, D,
 def paged_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor,
                  seq_lens: torch.Tensor, Hq: int, Hkv: int, D: int, *, scale: Optional[float] = None,
                  num_splits: int = 1, scratch: Optional[tuple[torch.Tensor, torch.Tensor]] = None,
-                 out: Optional[torch.Tensor] = None, window: int = 0, chunk: int = 0) -> torch.Tensor:
+                 out: Optional[torch.Tensor] = None, window: int = 0, chunk: int = 0, keep: int = 0,
+                 offset: Optional[torch.Tensor] = None, gated: bool = False) -> torch.Tensor:
     """Attention of one query token per sequence against its paged KV. ``q`` [B, Hq*D] (rows may be strided). ``window`` > 0:
-    only the last ``window`` cached tokens are visible (sliding-window layers; served by the gather path). ``chunk`` > 0: only the cached
-    tokens of the query's own run of ``chunk`` positions are."""
+    only the last ``window`` cached tokens are visible (sliding-window layers; served by the gather path, or with ``offset`` by the tensor-core
+    kernel) and, with ``keep``, the sequence's first ``keep``. ``chunk`` > 0: only the cached tokens of the query's own run of ``chunk`` positions
+    are. ``offset`` [Hq]: the weights are sigmoid(score + offset), unnormalised. ``gated``: ``out`` holds gates, and becomes output * sigmoid(gate)."""
     B = q.shape[0]
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
     block_size = k_cache.shape[2]
     if out is None:
         out = torch.empty((B, Hq * D), dtype=q.dtype, device=q.device)
+    special = offset is not None or gated or keep > 0       # (forms that the tensor-core kernel alone has)
     if not use_native(q):
+        assert not special
         g = Hq // Hkv
         for b in range(B):
             n = int(seq_lens[b])
@@ -125,7 +129,9 @@ def paged_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, 
             p = torch.softmax(qb @ k.transpose(1, 2), dim=-1)
             out[b] = (p @ v).reshape(Hq * D).to(out.dtype)
         return out
-    if D != 128 or window:
+    if special:
+        assert D == 128 and Hq // Hkv <= 8 and (block_size in (16, 32, 64) or block_size % 128 == 0), "shape of the tensor-core decode kernel"
+    elif D != 128 or window:
         return _paged_decode_gather(q, k_cache, v_cache, block_table, seq_lens, Hq, Hkv, D, scale, out, window=window, chunk=chunk)
     po = pml = None
     if num_splits > 1:
@@ -135,11 +141,11 @@ def paged_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, 
                        torch.empty(nml, dtype=torch.float32, device=q.device))
         po, pml = scratch
     kernel = os.environ.get("RLB_DECODE_KERNEL", "mma")
-    if kernel == "mma" and D == 128 and Hq // Hkv <= 8 and (block_size in (16, 32, 64) or block_size % 128 == 0):
+    if (kernel == "mma" or special) and D == 128 and Hq // Hkv <= 8 and (block_size in (16, 32, 64) or block_size % 128 == 0):
         # tensor-core flash-decoding kernel (tcgen05: QK^T and PV as MMAs over 128-token tiles)
         call("rlb_paged_decode_mma", ptr(q), q.stride(0), ptr(k_cache), ptr(v_cache), k_cache.shape[0], ptr(block_table),
-             block_table.stride(0), ptr(seq_lens), B, Hq, Hkv, D, block_size, chunk, scale, num_splits, ptr(po), ptr(pml), ptr(out),
-             out.stride(0), ptr(_L.status_word(q.device)), stream_ptr())
+             block_table.stride(0), ptr(seq_lens), B, Hq, Hkv, D, block_size, chunk, window, keep, ptr(offset), int(gated), scale, num_splits, ptr(po), ptr(pml),
+             ptr(out), out.stride(0), ptr(_L.status_word(q.device)), stream_ptr())
         return out
     if chunk:
         return _paged_decode_gather(q, k_cache, v_cache, block_table, seq_lens, Hq, Hkv, D, scale, out, chunk=chunk)

@@ -1,5 +1,5 @@
 """Row operators of post-norm and pre-norm layers (``rl_b200/models/post_norm.py``, ``pre_norm.py``) in the generation engine: products with
-what follows them, the join with the residual stream, the gated feed-forwards and the token input.
+what follows them, the join with the residual stream, the blend with the token before, the feed-forwards and the token input.
 
 Each operator has the native sm_100a body (CUDA tensors, bf16 or fp32) and a plain PyTorch statement (CPU tensors). ``x`` is the fp32
 residual stream, updated in place; ``h`` what the next sublayer reads (x in the model's type). fp32 models run every product in true fp32.
@@ -8,6 +8,7 @@ residual stream, updated in place; ``h`` what the next sublayer reads (x in the 
 from __future__ import annotations
 
 import ctypes as C
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
@@ -17,16 +18,19 @@ from . import functional as F
 from . import lib as _L
 from .lib import F as CF
 from .lib import I, L as LL, P, call, ptr, register, stream_ptr, use_native
-from .mixer_ops import _aligned, _f32
+from .mixer_ops import TokenBatch, _aligned, _f32
 
 register("rlb_linear_rows", [P, P])
 register("rlb_linear_tiled", [P, P])
 register("rlb_linear_skinny", [P, P])
 register("rlb_linear_grouped", [P, P])
-register("rlb_add_normed", [P, P, LL, I, P, P, I, I, P, I, P, LL, P, P, P, LL, I, CF, CF, P])
+register("rlb_add_normed", [P, P])
+register("rlb_shift_rows", [P, P, P])
+register("rlb_commit_states", [P, P, LL, P, P, P, I, LL, P, P])
+register("rlb_poly_norm_rows", [P, LL, I, P, LL, I, CF, P])
 register("rlb_group_norm_rows", [P, LL, I, P, LL, I, I, CF, P])
 register("rlb_cap_rows", [P, LL, CF, CF, P])
-register("rlb_moe_choose", [P, LL, I, I, P, I, I, I, P, P, P, P, P])
+register("rlb_moe_choose", [P, LL, I, I, P, I, I, I, I, CF, I, P, P, P, P, P, P, P])
 register("rlb_moe_place", [P, P, LL, I, P, I, I, P, P, P, P, LL, P, I, P, P, P, P])
 
 NONE, GLU, GELU_MUL, CAP, SILU = range(5)      # what follows a product (RlbLinearAct)
@@ -109,21 +113,146 @@ def _rms(x: torch.Tensor, eps: float) -> torch.Tensor:
     return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
 
 
-def add_normed_(x: torch.Tensor, y: torch.Tensor, w: Optional[torch.Tensor], mult: float, eps: float, next_norm: Optional[torch.Tensor] = None,
-                experts: Optional[tuple] = None, also: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """x += mult * rms(y) * w in place (w None: mult * y); returns x in the model's type, or rms(x) * next_norm. ``experts`` = (row of every
-    copy, weight of every copy or None, the experts' counts to reset): y holds expert rows, a token's value is the (weighted) sum of its
-    copies' rows. ``also``: rows added to y first."""
+class _Join(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("x", "y", "copy_row", "weight", "counts", "w", "ls", "next_w", "also", "own", "also_f", "own_f", "h", "x_out")] + \
+               [(n, C.c_longlong) for n in ("ldy", "ld_also", "ld_own", "rows")] + [(n, C.c_int) for n in ("f32", "k", "y_rows", "experts", "d")] + \
+               [(n, C.c_float) for n in ("mult", "eps")]
+
+
+class _Shift(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("s", "positions", "row_off", "row_state", "state", "next", "ids", "table", "pairs", "token", "token_next", "status")] + \
+               [(n, C.c_longlong) for n in ("num_states", "ld_state", "mul_prev", "mul_cur")] + [(n, C.c_int) for n in ("n_single", "vocab", "buckets")] + \
+               [("scale", C.c_float)]
+
+
+class Carry:
+    """What sequences carry from step to step beside their cache pages, a row per sequence: the normed stream of their last token at every place
+    where the next token blends it in (``state`` [rows, places, d], fp32), and the token itself. Portions leave theirs in second buffers until the
+    step is through (``commit``): another CTA may still have to read the old one."""
+
+    def __init__(self, rows: int, places: int, d: int, tokens: bool, device):
+        self.state = torch.zeros((rows, places, d), dtype=torch.float32, device=device) if places else None
+        self.next = torch.zeros_like(self.state) if places else None
+        self.token = torch.zeros(rows, dtype=torch.int32, device=device) if tokens else None
+        self.token_next = torch.zeros_like(self.token) if tokens else None
+        self.rows = rows
+
+    def commit(self, b: TokenBatch) -> None:
+        """Takes over what the portions of ``b`` left."""
+        rows = b.state_rows[b.n_single :]
+        if not rows.numel() or not rows.is_cuda:
+            return
+        call("rlb_commit_states", ptr(self.state), ptr(self.next), self.state[0].numel() if self.state is not None else 0, ptr(self.token), ptr(self.token_next),
+             ptr(rows), rows.numel(), self.rows, ptr(_L.status_word(rows.device)), stream_ptr())
+
+
+@dataclass
+class Shift:
+    """Blend of a normed stream with that of the token before: h + (h' - h) * s, at one of the ``places`` of ``carry`` (s None: no blend)."""
+
+    s: Optional[torch.Tensor]
+    place: int
+    carry: Carry
+    b: TokenBatch
+
+
+def _pieces(b: TokenBatch) -> list:
+    cuts = list(range(b.n_single)) + ([b.n_single + c for c in b.cu.tolist()] if b.cu is not None else [b.n_single])
+    return list(zip(cuts[:-1], cuts[1:]))
+
+
+def _shift_ref(h: torch.Tensor, t: Shift) -> torch.Tensor:
+    """``h`` fp32."""
+    if t.s is None:
+        return h
+    before, state = torch.cat([h[:1], h[:-1]]), t.carry.state[:, t.place]
+    for j, (s, e) in enumerate(_pieces(t.b)):
+        r = int(t.b.state_rows[j])
+        before[s] = state[r] if int(t.b.positions[s]) else 0.0
+        state[r] = h[e - 1]
+    return h + (before - h) * t.s.float()
+
+
+def _shift_desc(t: Shift) -> _Shift:
+    b, c, q = t.b, t.carry, _Shift()
+    q.s, q.positions, q.row_off, q.n_single = ptr(t.s), ptr(b.positions), ptr(b.row_off), b.n_single
+    q.row_state = ptr(b.row_state if b.row_state is not None else b.state_rows)
+    q.num_states, q.status = c.rows, ptr(_L.status_word(b.positions.device))
+    if t.s is not None:
+        q.state, q.next, q.ld_state = ptr(c.state[:, t.place]), ptr(c.next[:, t.place]), c.state.stride(0)
+    return q
+
+
+def start(b: TokenBatch, table: torch.Tensor, scale: float, norm: torch.Tensor, eps: float, pairs: Optional[torch.Tensor], bigram: Optional[dict], t: Shift):
+    """(x, h): the tokens' rows of ``table`` times ``scale`` plus, with ``pairs``, the rows of (token before, token) in the pair table, and rms(x) *
+    norm blended by ``t``. Sequences' last tokens are kept in ``t.carry``."""
+    c, T = t.carry, b.rows
+    if not use_native(table):
+        x = table[b.ids.long()].float() * scale
+        if pairs is not None:
+            rows = torch.empty(T, dtype=torch.int64)
+            for j, (s, e) in enumerate(_pieces(b)):
+                r, ids = int(b.state_rows[j]), b.ids[s:e].long()
+                before = torch.cat([c.token[r : r + 1].long(), ids[:-1]])
+                rows[s:e] = (before * bigram["mul_prev"] + ids * bigram["mul_cur"]) % bigram["buckets"]
+                if int(b.positions[s]) == 0:
+                    rows[s] = bigram["buckets"]
+                c.token[r] = int(ids[-1])
+            x = x + pairs[rows].float()
+        return x, _shift_ref(_rms(x, eps) * norm.float(), t).to(table.dtype)
+    d = table.shape[1]
+    x = torch.empty((T, d), dtype=torch.float32, device=table.device)
+    h = torch.empty((T, d), dtype=table.dtype, device=table.device)
+    j, q = _Join(), _shift_desc(t)
+    j.x_out, j.h, j.next_w, j.rows, j.d, j.f32, j.eps = ptr(x), ptr(h), ptr(norm), T, d, _f32(table), eps
+    ids = b.ids if b.ids.dtype == torch.int32 else b.ids.int()
+    q.ids, q.table, q.vocab, q.scale = ptr(ids), ptr(table), table.shape[0], float(scale)
+    if pairs is not None:
+        q.pairs, q.buckets, q.mul_prev, q.mul_cur = ptr(pairs), bigram["buckets"], bigram["mul_prev"], bigram["mul_cur"]
+        q.token, q.token_next = ptr(c.token), ptr(c.token_next)
+    call("rlb_shift_rows", C.byref(j), C.byref(q), stream_ptr())
+    return x, h
+
+
+def join(x: torch.Tensor, y: torch.Tensor, w: Optional[torch.Tensor], mult: float, eps: float, next_norm: Optional[torch.Tensor] = None,
+         experts: Optional[tuple] = None, also: Optional[torch.Tensor] = None, also_f: Optional[torch.Tensor] = None, own: Optional[torch.Tensor] = None,
+         own_f: Optional[torch.Tensor] = None, ls: Optional[torch.Tensor] = None, shift: Optional[Shift] = None):
+    """(x, h) with x + mult * rms(y) * w * ls (w None: mult * y; ls None: ones) and h: x in the model's type, or rms(x) * next_norm, blended by
+    ``shift``. x is updated in place, with ``shift`` it moves to a new buffer. ``experts`` = (row of every copy, weight of every copy or None, the
+    experts' counts to reset): y holds expert rows, a token's value is the (weighted) sum of its copies' rows. ``also`` / ``own``: rows added to y
+    first, times ``also_f`` (None: 1) / ``own_f`` [T]."""
     if not use_native(x):
-        y = y.float() if also is None else y.float() + also.float()
-        x += mult * (y if w is None else _rms(y, eps) * w.float())
-        return (x if next_norm is None else _rms(x, eps) * next_norm.float()).to((next_norm if w is None else w).dtype)
+        y = y.float()
+        if also is not None:
+            y = y + also.float() * (1.0 if also_f is None else also_f[:, None])
+        if own is not None:
+            y = y + own.float() * own_f[:, None]
+        z = mult * (y if w is None else _rms(y, eps) * w.float())
+        x += z if ls is None else z * ls.float()
+        h = x if next_norm is None else _rms(x, eps) * next_norm.float()
+        return x, (h if shift is None else _shift_ref(h, shift)).to((next_norm if w is None else w).dtype)
     T, d = x.shape
     h = torch.empty((T, d), dtype=y.dtype, device=x.device)
+    out = x if shift is None else torch.empty_like(x)
     rows, wt, counts = experts if experts is not None else (None, None, None)
-    call("rlb_add_normed", ptr(x), ptr(y), y.stride(0), _f32(y), ptr(rows), ptr(wt), rows.shape[1] if rows is not None else 0, y.shape[0], ptr(counts),
-         counts.numel() if counts is not None else 0, ptr(also), also.stride(0) if also is not None else 0, ptr(w), ptr(next_norm), ptr(h), T, d, float(mult), float(eps), stream_ptr())
-    return h
+    j = _Join()
+    j.x, j.y, j.copy_row, j.weight, j.counts, j.w, j.ls, j.next_w = ptr(x), ptr(y), ptr(rows), ptr(wt), ptr(counts), ptr(w), ptr(ls), ptr(next_norm)
+    j.also, j.also_f, j.own, j.own_f, j.h, j.x_out = ptr(also), ptr(also_f), ptr(own), ptr(own_f), ptr(h), ptr(out)
+    j.ldy, j.ld_also, j.ld_own, j.rows, j.d = y.stride(0), also.stride(0) if also is not None else 0, own.stride(0) if own is not None else 0, T, d
+    j.f32, j.k, j.y_rows, j.experts = _f32(y), rows.shape[1] if rows is not None else 0, y.shape[0], counts.numel() if counts is not None else 0
+    j.mult, j.eps = mult, eps
+    if shift is None:
+        call("rlb_add_normed", C.byref(j), stream_ptr())
+    else:
+        q = _shift_desc(shift)
+        call("rlb_shift_rows", C.byref(j), C.byref(q), stream_ptr())
+    return out, h
+
+
+def add_normed_(x: torch.Tensor, y: torch.Tensor, w: Optional[torch.Tensor], mult: float, eps: float, next_norm: Optional[torch.Tensor] = None,
+                experts: Optional[tuple] = None, also: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``join`` in place; returns h."""
+    return join(x, y, w, mult, eps, next_norm, experts, also)[1]
 
 
 def group_norm_(y: torch.Tensor, w: torch.Tensor, groups: int, eps: float) -> None:
@@ -137,39 +266,65 @@ def group_norm_(y: torch.Tensor, w: torch.Tensor, groups: int, eps: float) -> No
 
 # --------------------------------------------------------------------------------------- feed-forwards
 def feed_forward_(x: torch.Tensor, h: torch.Tensor, ff, norm: Optional[torch.Tensor], mult: float, eps: float, next_norm=None) -> torch.Tensor:
-    """x += mult * rms(ff(h)) * norm (norm None: mult * ff(h)). ``ff``: the layer's ``GatedUnit`` or ``GatedExperts``."""
+    """x += mult * rms(ff(h)) * norm (norm None: mult * ff(h)). ``ff``: the layer's feed-forward module."""
+    return feed_forward(x, h, ff, norm, mult, eps, next_norm)[1]
+
+
+def feed_forward(x: torch.Tensor, h: torch.Tensor, ff, norm: Optional[torch.Tensor], mult: float, eps: float, next_norm=None, ls=None, shift: Optional[Shift] = None):
+    """``join`` of the feed-forward's output with the stream."""
     if hasattr(ff, "router"):
         shared = unit(h, ff.shared) if ff.shared is not None else None
-        y, experts = gated_experts(h, ff)
-        return add_normed_(x, y, norm, mult, eps, next_norm, experts, shared)
-    return add_normed_(x, unit(h, ff), norm, mult, eps, next_norm)
+        y, experts, own_f, gate = gated_experts(h, ff)
+        return join(x, y, norm, mult, eps, next_norm, experts, shared, gate, h if own_f is not None else None, own_f, ls, shift)
+    return join(x, poly_unit(h, ff) if hasattr(ff, "coef") else unit(h, ff), norm, mult, eps, next_norm, ls=ls, shift=shift)
 
 
 def unit(h: torch.Tensor, m) -> torch.Tensor:
     return linear(gated_linear(h, m.gate_up, m.limit), m.down)
 
 
+def poly_unit(h: torch.Tensor, m) -> torch.Tensor:
+    """``m``: a ``PolyUnit``. (The padding columns of the first product are zeros, and so are the weights that read them.)"""
+    return linear(poly_norm_(linear(h, m.up), m.coef, m.ff, m.eps), m.down)
+
+
+def poly_norm_(z: torch.Tensor, coef: torch.Tensor, n: int, eps: float) -> torch.Tensor:
+    """The leading n columns of ``z`` become c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3, N dividing a row by its root mean square; in place."""
+    if not use_native(z):
+        v, c = z[:, :n].float(), coef.float()
+        z[:, :n] = (c[0] * _rms(v, eps) + c[1] * _rms(v ** 2, eps) + c[2] * _rms(v ** 3, eps) + c[3]).to(z.dtype)
+        return z
+    call("rlb_poly_norm_rows", ptr(z), z.stride(0), _f32(z), ptr(coef), z.shape[0], n, float(eps), stream_ptr())
+    return z
+
+
 def gated_experts(h: torch.Tensor, m):
-    """Routed part of ``m`` (``GatedExperts``): (expert rows, (row of every copy, weights or None, counts)) on the native path, (summed
-    outputs, None) otherwise. Weights on the experts' inputs are factors of the first product's rows."""
+    """Routed part of ``m`` (``GatedExperts``): (y, experts, weight of the token's own row [T] or None, factor of the shared unit [T] or None).
+    Native path: y are expert rows, experts = (row of every copy, weights or None, counts); otherwise y are summed outputs and experts None.
+    Weights on the experts' inputs are factors of the first product's rows."""
     T, d = h.shape
+    E, k, n = m.experts, m.top, m.outputs
     if not use_native(h):
-        w, idx = m.choose(h.float() @ m.router.float().t())
+        z = h.float() @ m.router.float().t()
+        w, idx = m.choose(z[:, :n])
         y = torch.zeros((T, d), dtype=torch.float32)
-        for e in range(m.experts):
+        for e in range(E):
             tok, slot = (idx == e).nonzero(as_tuple=True)
             if tok.numel():
                 p, wt = h[tok] @ m.gate_up[e].t(), w[tok, slot, None]
                 a = gated_ref((p.float() * wt).to(p.dtype) if m.weigh_input else p, m.limit)
                 y.index_add_(0, tok, (a @ m.down[e].t()).float() * (1.0 if m.weigh_input else wt))
-        return y, None
-    dev, E, k = h.device, m.experts, m.top
+        return y, None, (w * (idx >= E)).sum(-1) if m.identity else None, torch.sigmoid(z[:, n]) if m.shared_gate else None
+    dev = h.device
     st = ptr(_L.status_word(dev))
     z = router_logits(h, m.router)
     wt = torch.empty((T, k), dtype=torch.float32, device=dev)
     idx, rank, copy_row = torch.empty((3, T, k), dtype=torch.int32, device=dev)
+    own_f = torch.empty(T, dtype=torch.float32, device=dev) if m.identity else None
+    gate = torch.empty(T, dtype=torch.float32, device=dev) if m.shared_gate else None
     counts = _expert_counts(m, dev)
-    call("rlb_moe_choose", ptr(z), z.stride(0), T, E, ptr(m.correction), m.groups, m.keep, k, ptr(wt), ptr(idx), ptr(rank), ptr(counts), stream_ptr())
+    call("rlb_moe_choose", ptr(z), z.stride(0), T, n, ptr(m.correction), m.groups, m.keep, k, int(m.softmax), m.scale, E, ptr(wt), ptr(idx), ptr(rank), ptr(counts),
+         ptr(own_f), ptr(gate), stream_ptr())
     mpad = -(-(T * k + E * 127) // 128) * 128
     tiles = torch.empty(mpad // 128, dtype=torch.int32, device=dev)
     fast = _aligned(h, m.gate_up[0], m.down[0]) and m.gate_up.shape[1] % 8 == 0 and d % 8 == 0
@@ -189,7 +344,7 @@ def gated_experts(h: torch.Tensor, m):
         if first and not fast:
             q.a_rows, q.num_a_rows = ptr(src), T
         call("rlb_linear_grouped" if fast else "rlb_linear_rows", C.byref(q), stream_ptr())
-    return y, (copy_row, None if m.weigh_input else wt, counts)
+    return y, (copy_row, None if m.weigh_input else wt, counts), own_f, gate
 
 
 def router_logits(h: torch.Tensor, router: torch.Tensor) -> torch.Tensor:

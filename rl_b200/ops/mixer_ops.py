@@ -40,6 +40,7 @@ register("rlb_retention_portions", [P, LL, LL, I, I, I, I, I, I, I, I, I, I, I, 
 
 NO_ACT = 1 << 30
 CHUNK = 128          # rows per chunk of the chunked recurrences
+KEY_TILE = 64        # keys per tile of the attention of prompt portions
 PAGED_PORTION = 16   # portions of at most this many tokens attend row by row over the pages (decode kernels)
 
 
@@ -84,6 +85,7 @@ class TokenBatch:
     row_state: Optional[torch.Tensor] = None    # int64 [T]: state row of each row's sequence (None: ``state_rows``)
     whole: bool = False              # the tile-wise portions start at position 0
     chunk_ctx: dict = field(default_factory=dict)   # chunk size: (cu_ctx, ctx_slots, whole) of layers that see chunks, from the border before each portion
+    window_ctx: dict = field(default_factory=dict)  # (window, kept): (cu_ctx, ctx_slots, skip) of layers that see windows, without what no row of a portion sees
     max_ctx: int = 0                 # upper bound of seq_lens (a host number, fixed while a graph is captured)
 
     @property

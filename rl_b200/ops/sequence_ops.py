@@ -10,21 +10,22 @@ CPU tensors run the plain PyTorch statement.
 from __future__ import annotations
 
 import ctypes as C
-from typing import Optional
+from dataclasses import dataclass, field
+from typing import Any, Optional
 
 import torch
 
 from . import engine_ops as E
 from . import lib as _L
-from .layer_ops import group_norm_
+from .layer_ops import _pieces, group_norm_
 from .lib import F as CF
 from .lib import I, L as LL, P, call, ptr, register, stream_ptr, use_native
 from .mixer_ops import TokenBatch, _f32, _page_rows
 
-register("rlb_gqa_prep", [P, I, LL, LL, I, I, I, I, I, I, I, I, I, P, P, P, P, P, I, I, CF, CF, P, LL, P, P, P, P, P])
-register("rlb_gqa_rows", [P, I, I, LL, I, I, I, I, I, I, I, P, P, P, I, P, I, CF, P, LL, P, P])
+register("rlb_gqa_prep", [P, I, LL, LL, I, I, I, I, I, I, I, I, I, P, P, P, P, P, I, I, CF, CF, P, LL, P, I, P, P, P, P])
+register("rlb_gqa_rows", [P, I, I, LL, I, I, I, I, I, I, I, P, P, P, I, P, I, I, I, P, I, CF, P, LL, P, P])
 register("rlb_gqa_gather", [P, P, P, P, LL, I, I, I, I, LL, P, P])
-register("rlb_flash_gqa", [P, LL, LL, I, I, P, LL, LL, I, I, I, I, P, P, I, I, I, I, I, I, I, CF, I, P, LL, P, P])
+register("rlb_flash_gqa", [P, LL, LL, I, I, P, LL, LL, I, I, I, I, P, P, I, I, I, I, I, I, I, I, I, P, P, I, CF, I, P, LL, P, P])
 register("rlb_conv_rows", [P, I, LL, P, LL, LL, I, I, P, P, P, P, P, P, LL, P, P])
 register("rlb_conv_state", [P, I, LL, I, I, P, I, I, P, P, P, LL, P])
 register("rlb_mamba2_rows", [P, I, LL, P, LL, P, LL, I, I, I, I, I, I, I, I, P, P, P, P, LL, P, P, P, P, P])
@@ -50,50 +51,82 @@ def _rows_out(p: torch.Tensor, m) -> torch.Tensor:
 
 
 # --------------------------------------------------------------------------------------- attention
-def attention(p: torch.Tensor, m, b: TokenBatch, k_cache: torch.Tensor, v_cache: torch.Tensor, first: Optional[torch.Tensor] = None) -> torch.Tensor:
+@dataclass
+class KeyValues:
+    """Keys and values of one layer in one step, for the layers that read them: its projected rows (whole portions attend to those) and, by mask,
+    what was gathered from its cache."""
+
+    p: torch.Tensor
+    m: Any
+    gathered: dict = field(default_factory=dict)
+
+
+def attention(p: torch.Tensor, m, b: TokenBatch, k_cache: torch.Tensor, v_cache: torch.Tensor, first: Optional[torch.Tensor] = None,
+              kv: Optional[KeyValues] = None) -> torch.Tensor:
     """``m``: the layer's ``GroupedAttentionMixer``; caches [pages, kv_heads, page size, dim / vdim]. The rows' own keys and values are
     written first; ``p`` is left with normed and rotated queries and keys. ``first`` [T, kv_heads * vdim]: an earlier layer's values of the
-    rows, of which the layer's own take over a share before they are written."""
+    rows, of which the layer's own take over a share before they are written. A layer without keys and values of its own reads those of ``kv``, and
+    the caches are that layer's. With an output gate the outputs stand over the gates in ``p``."""
     bs, H, G = k_cache.shape[2], m.heads, m.kv_heads
-    y = _rows_out(p, m)
+    own = m.kv_from is None
     if not use_native(p):
-        q, k, v = m.qkv(p, b.positions, first)
-        ok = b.slots >= 0
-        page, off = (b.slots[ok] // bs).long(), (b.slots[ok] % bs).long()
-        k_cache[page, :, off], v_cache[page, :, off] = k[ok].to(k_cache.dtype), v[ok].to(v_cache.dtype)
+        y = _rows_out(p, m)
+        q = m.queries(p, b.positions)
+        if own:
+            k, v = m.keys_values(p, b.positions, first)
+            ok = b.slots >= 0
+            page, off = (b.slots[ok] // bs).long(), (b.slots[ok] % bs).long()
+            k_cache[page, :, off], v_cache[page, :, off] = k[ok].to(k_cache.dtype), v[ok].to(v_cache.dtype)
         q = q.to(p.dtype).float()
         for i in range(p.shape[0]):
             n = int(b.seq_lens[i])
             if n == 0:
                 y[i] = 0
                 continue
-            rows = _page_rows(b.block_table[i], n, bs)[(n - 1) // m.chunk * m.chunk if m.chunk else 0 :]
+            t = torch.arange(n)
+            t = t[~m.hidden(torch.tensor(n - 1), t)]
+            rows = _page_rows(b.block_table[i], n, bs)[t]
             ks, vs = (c[rows // bs, :, rows % bs].float().transpose(0, 1) for c in (k_cache, v_cache))      # [kv_heads, n, dim]
-            w = torch.softmax(q[i].view(G, H // G, m.dim) @ ks.transpose(1, 2) * m.scale, dim=-1)
-            y[i, : H * m.vdim] = (w @ vs).reshape(-1).to(p.dtype)
+            z = (q[i].view(G, H // G, m.dim) @ ks.transpose(1, 2) * m.scale).view(H, 1, -1)
+            w = m.weigh(z, torch.zeros((), dtype=torch.bool)).view(G, H // G, -1)
+            y[i, : H * m.vdim] = m.gated((w @ vs).reshape(1, -1), p[i : i + 1])[0].to(p.dtype)
         return y
     T, st = p.shape[0], ptr(_L.status_word(p.device))
+    y = p[:, m.mix_off : m.mix_off + m.mix_width] if m.gate else _rows_out(p, m)
     call("rlb_gqa_prep", ptr(p), _f32(p), T, p.stride(0), m.q_off, m.k_off, m.v_off, H, G, m.dim, m.vdim, bs, k_cache.shape[0], ptr(b.positions),
          ptr(b.slots), ptr(m.q_norm), ptr(m.k_norm), ptr(m.freq), m.freq.numel(), int(not m.interleaved), float(m.gain), float(m.eps), ptr(first),
-         first.stride(0) if first is not None else 0, ptr(m.v_share) if first is not None else None, ptr(k_cache), ptr(v_cache), st, stream_ptr())
+         first.stride(0) if first is not None else 0, ptr(m.v_share) if first is not None else None, int(own), ptr(k_cache), ptr(v_cache), st, stream_ptr())
     if b.n_paged:
         if decode_tiles(p, m, bs):
-            splits = E.choose_splits(b.n_paged, G, max((min(b.max_ctx, m.chunk) if m.chunk else b.max_ctx) // 2, 1), bs)
+            seen = min(b.max_ctx, m.chunk) // 2 if m.chunk else min(b.max_ctx // 2, m.window + m.keep) if m.window else b.max_ctx // 2
             E.paged_decode(p[: b.n_paged, m.q_off : m.q_off + H * m.dim], k_cache, v_cache, b.block_table, b.seq_lens, H, G, m.dim, scale=m.scale,
-                           num_splits=splits, out=y[: b.n_paged], chunk=m.chunk)
+                           num_splits=E.choose_splits(b.n_paged, G, max(seen, 1), bs), out=y[: b.n_paged], chunk=m.chunk, window=m.window, keep=m.keep,
+                           offset=m.offset, gated=m.gate)
         else:
             call("rlb_gqa_rows", ptr(p), _f32(p), b.n_paged, p.stride(0), m.q_off, H, G, m.dim, m.vdim, bs, k_cache.shape[0], ptr(k_cache),
-                 ptr(v_cache), ptr(b.block_table), b.block_table.stride(0), ptr(b.seq_lens), m.chunk, float(m.scale), ptr(y), y.stride(0), st, stream_ptr())
+                 ptr(v_cache), ptr(b.block_table), b.block_table.stride(0), ptr(b.seq_lens), m.chunk, m.window, m.keep, ptr(m.offset), int(m.gate),
+                 float(m.scale), ptr(y), y.stride(0), st, stream_ptr())
     if b.n_paged < T:
-        cu_ctx, slots, whole = b.chunk_ctx.get(m.chunk, (b.cu_ctx, b.ctx_slots, b.whole))
+        cu_ctx, slots, whole, skip = b.cu_ctx, b.ctx_slots, b.whole, None
+        if m.chunk in b.chunk_ctx:
+            cu_ctx, slots, whole = b.chunk_ctx[m.chunk]
+        elif not whole and (m.window, m.keep) in b.window_ctx:
+            cu_ctx, slots, skip = b.window_ctx[m.window, m.keep]
         if whole:         # no cached key is visible to these portions: theirs, and their values, stand in the projected rows
-            kv, rows, row0, k0, v0 = p, T, b.n_paged, m.k_off, m.v_off
+            rows, row0 = T, b.n_paged
+            src, k0, v0 = (p, m.k_off, m.v_off) if own else (kv.p, kv.m.k_off, kv.m.v_off)
         else:
             rows, row0, k0, v0 = slots.numel(), 0, 0, G * m.dim
-            kv = torch.empty((rows, G * (m.dim + m.vdim)), dtype=p.dtype, device=p.device)
-            call("rlb_gqa_gather", ptr(k_cache), ptr(v_cache), ptr(slots), ptr(kv), rows, G, m.dim, m.vdim, bs, k_cache.shape[0] * bs, st, stream_ptr())
-        call("rlb_flash_gqa", ptr(p), T, p.stride(0), p.shape[1], b.n_paged, ptr(kv), rows, kv.stride(0), kv.shape[1], row0, k0, v0, ptr(b.cu_q),
-             ptr(cu_ctx), b.cu_q.numel() - 1, H, G, m.dim, m.vdim, m.q_off, m.chunk, float(m.scale), b.q_tiles, ptr(y), y.stride(0), st, stream_ptr())
+            seen = (m.chunk, m.window, m.keep)
+            src = kv.gathered.get(seen) if kv is not None else None
+            if src is None:
+                src = torch.empty((rows, G * (m.dim + m.vdim)), dtype=p.dtype, device=p.device)
+                call("rlb_gqa_gather", ptr(k_cache), ptr(v_cache), ptr(slots), ptr(src), rows, G, m.dim, m.vdim, bs, k_cache.shape[0] * bs, st, stream_ptr())
+                if kv is not None:
+                    kv.gathered[seen] = src
+        call("rlb_flash_gqa", ptr(p), T, p.stride(0), p.shape[1], b.n_paged, ptr(src), rows, src.stride(0), src.shape[1], row0, k0, v0, ptr(b.cu_q),
+             ptr(cu_ctx), b.cu_q.numel() - 1, H, G, m.dim, m.vdim, m.q_off, m.chunk, m.window, m.keep, ptr(skip), ptr(m.offset), int(m.gate), float(m.scale),
+             b.q_tiles, ptr(y), y.stride(0), st, stream_ptr())
     return y
 
 
@@ -108,11 +141,6 @@ def portion_tiles(m, dtype: torch.dtype) -> bool:
 
 
 # --------------------------------------------------------------------------------------- recurrent mixers
-def _pieces(b: TokenBatch) -> list:
-    cuts = list(range(b.n_single)) + ([b.n_single + c for c in b.cu.tolist()] if b.cu is not None else [b.n_single])
-    return list(zip(cuts[:-1], cuts[1:]))
-
-
 def recurrent(p: torch.Tensor, m, b: TokenBatch, ring: torch.Tensor, state: torch.Tensor, plain: bool = False) -> torch.Tensor:
     """Mamba-2 or delta-rule mixing of all rows: every sequence's row of ``ring`` [rows, taps, channels] (the convolution's last inputs, by
     position modulo taps) and of ``state`` [rows, heads, dim, vdim] (fp32) is advanced by its tokens; a piece that starts at position 0
