@@ -56,7 +56,7 @@ _SIGS: dict[str, list[Any]] = {
     "rlb_rope_kv_cache_write": [P, P, P, P, P, P, L, I, I, I, I, L, L, P, P],
     "rlb_paged_decode": [P, L, P, P, P, I, P, I, I, I, I, I, F, I, P, P, P, L, P],
     "rlb_paged_decode_tma": [P, L, P, P, I, P, I, P, I, I, I, I, I, F, I, P, P, P, L, P, P],
-    "rlb_paged_decode_mma": [P, L, P, P, I, P, I, P, I, I, I, I, I, I, F, I, P, P, P, L, P, P],
+    "rlb_paged_decode_mma": [P, L, P, P, I, P, I, P, I, I, I, I, I, I, I, I, P, I, F, I, P, P, P, L, P, P],
     "rlb_sample": [P, I, L, I, I, P, P, P, F, I, F, I, U64, U64, P, P, P, P, P],
     "rlb_decode_advance": [P, P, P, P, P, P, P, P, I, P, P, P, P, I, P, P, I, I, P, I, I, P],
     "rlb_block_copy": [P, P, P, P, I, L, P],
