@@ -6,6 +6,7 @@
     python bench.py --config gadarax-serving                 (prefill / decode of a layer-list model beside Llama at equal size)
     python bench.py --config redarax-serving                 (the same for a post-norm layer-list model, beside Qwen3-MoE)
     python bench.py --config kikivik-serving                 (the same for a pre-norm layer-list model, beside Qwen3-MoE)
+    python bench.py --config zonidra-serving                 (the same for a layer-list model with norms on both sides, beside Kikivik)
     python bench.py --impl reference ...                     (the unmodified reference, when it can be installed)
 
 Default (headline) configuration ``llama8b-dp``: one GRPO step (generation + refit + log-probabilities + training) on
@@ -53,6 +54,7 @@ CONFIGS = {
     "gadarax-serving": dict(),
     "redarax-serving": dict(),
     "kikivik-serving": dict(),
+    "zonidra-serving": dict(),
 }
 
 
@@ -175,12 +177,13 @@ def main() -> int:
 
         return sweep_main(steps=args.steps, warmup=args.warmup)
 
-    if args.config in ("gadarax-serving", "redarax-serving", "kikivik-serving"):
+    if args.config in ("gadarax-serving", "redarax-serving", "kikivik-serving", "zonidra-serving"):
         from rl_b200.csrc.build import build_all
         from rl_b200.engine import bench_mixers
         from rl_b200.ops import lib as L
 
-        serving_main = {"gadarax-serving": bench_mixers.main, "redarax-serving": bench_mixers.redarax_main, "kikivik-serving": bench_mixers.kikivik_main}[args.config]
+        serving_main = {"gadarax-serving": bench_mixers.main, "redarax-serving": bench_mixers.redarax_main, "kikivik-serving": bench_mixers.kikivik_main,
+                        "zonidra-serving": bench_mixers.zonidra_main}[args.config]
 
         if not L.available():
             build_all()

@@ -1,7 +1,7 @@
 """Serving throughput of layer-list models beside the framework's closest model at equal size (Gadarax: the Llama architecture, Redarax and
-Kikivik: Qwen3-MoE), and the kernels' distance from their rooflines beside the like kernels of the closest path.
+Kikivik: Qwen3-MoE, Zonidra: Kikivik), and the kernels' distance from their rooflines beside the like kernels of the closest path.
 
-    python bench.py --config gadarax-serving | redarax-serving | kikivik-serving [--steps K --warmup W]
+    python bench.py --config gadarax-serving | redarax-serving | kikivik-serving | zonidra-serving [--steps K --warmup W]
 
 Random weights, random prompts. Whole-model figures come from ``GenerationEngine``: prefill of packed prompts (device time of the
 forward pass) and decoding through the captured step (device time of the graph replays). Kernel figures are CUDA-event times of a
@@ -30,6 +30,7 @@ SIZES = {   # (preset, Llama twin: same width and run count, MHA with 128-wide h
 }
 REDARAX = ("redarax-2b", "redarax-7b")
 KIKIVIK = ("kikivik-2b", "kikivik-7b")
+ZONIDRA = ("zonidra-2b", "zonidra-7b")
 PREFILL = ((1, 4096), (8, 1024))      # (prompts, tokens each)
 DECODE = ((16, 4096), (64, 2048))     # (sequences, context)
 
@@ -64,6 +65,28 @@ def moe_twin(name: str) -> ModelConfig:
     per = c.num_hidden_layers * r["experts"] * 3 * c.hidden_size
     t.moe_intermediate_size = round((c.num_parameters() - t.num_parameters()) / per / 64) * 64
     return t
+
+
+def kikivik_twin(name: str) -> ModelConfig:
+    """Kikivik model of the same width, layers, attention heads, experts and choice: chunks as long as the window, gated units of the same number of
+    weights, the experts' width set for the same number of weights altogether."""
+    c = preset(name)
+    layers = []
+    for e in c.mixers:
+        m, mlp = {k: v for k, v in e["mixer"].items() if k != "kv_from"}, e["mlp"]
+        m.update(mask={"size": m["mask"]["size"]}, rot={"dims": m["dim"], "base": 1e6, "scaling": {"factor": 4.0}}, v_mix=True)
+        if mlp["kind"] == "dense":
+            mlp = {"kind": "dense", "ff": round(mlp["ff"] * 2 / 3 / 64) * 64, "limit": 7.0}
+        else:
+            mlp = {"kind": "moe", "expert": dict(mlp["expert"]), "router": {"experts": mlp["router"]["experts"], "top": mlp["router"]["top"]}, "shared": dict(mlp["shared"])}
+        layers.append({"type": "attention", "mixer": m, "mlp": mlp})
+    hf = {"architecture": "Kikivik", "vocab": c.vocab_size, "width": c.hidden_size, "embedding": {"scale": 2.0}, "norm": {"eps": 1e-6}, "layers": layers}
+    moe = [e["mlp"] for e in layers if e["mlp"]["kind"] == "moe"]
+    per = sum(m["router"]["experts"] * 3 * c.hidden_size for m in moe)
+    more = c.num_parameters() - c.bigram["buckets"] * c.hidden_size - ModelConfig.from_hf_dict(hf).num_parameters()      # (of the pair table a few rows are read)
+    for m in moe:
+        m["expert"]["ff"] += round(more / per / 8) * 8
+    return ModelConfig.from_hf_dict(hf)
 
 
 def timed(fn, steps: int, warmup: int) -> float:
@@ -521,6 +544,117 @@ def kikivik_table(name: str) -> list:
             add("like: gated latent attention prefill", timed_graph([lambda s=s: X.latent_attention_(s[1], gated, b, cache) for s in sets]), fl, nb)
             del sets
     return out
+
+
+def zonidra_table(name: str) -> list:
+    """``kernel_table`` of a layer-list preset with norms on both sides. The like kernels are those of Kikivik at the same sizes: its joins, embedding,
+    silu experts with a shared unit, chunked soft-max attention; for the polynomial activation the RMS norm over as many columns."""
+    from rl_b200.models.gated import GatedExperts
+    from rl_b200.models.mixers import GroupedAttentionMixer
+    from rl_b200.ops import layer_ops as Y
+    from rl_b200.ops import sequence_ops as S
+
+    pk, c, dev, bf = peaks(), preset(name), "cuda", torch.bfloat16
+    model = build_model(c, device=dev, dtype=bf, seed=0)
+    own, lent = model.layers[0], model.layers[1]
+    poly = next(l.ff for l in model.layers if hasattr(l.ff, "coef"))
+    moe = next(l.ff for l in model.layers if hasattr(l.ff, "router"))
+    d, out = c.hidden_size, []
+
+    def add(label, ms, flops=0.0, nbytes=0.0):
+        roof = max(flops / pk["flops"], nbytes / pk["hbm"]) * 1e3
+        out.append(dict(kernel=label, ms=round(ms, 4), roofline_ms=round(roof, 4), fraction=round(roof / ms, 3)))
+
+    rows = lambda T, n: torch.randn(T, n, device=dev).to(bf)   # noqa: E731
+    with torch.no_grad():
+        g = own.mixer
+        for T in (64, 4096):
+            for label, w in (("in_proj", g.in_proj), ("in_proj without keys and values", lent.mixer.in_proj), ("out_proj", g.out_proj), ("up", poly.up), ("down", poly.down),
+                             ("router and shared gate", moe.router)):
+                N, K = w.shape
+                nb = 2 * (N * K + T * (K + N)) + (2 * T * N if w is moe.router else 0)
+                sets = copies(lambda: (rows(T, K), w.detach().clone()), nb)
+                fn = Y.router_logits if w is moe.router else Y.linear
+                add(f"{label} [{N} x {K}], {T} rows", timed_graph([lambda s=s: fn(s[0], s[1]) for s in sets]), 2.0 * T * N * K, nb)
+                add("like: plain GEMM", timed_graph([lambda s=s: F.gemm(s[0], s[1]) for s in sets]), 2.0 * T * N * K, 2 * (N * K + T * (N + K)))
+                del sets
+            sets = copies(lambda: rows(T, poly.ff), 4 * T * poly.ff)
+            one = torch.ones(poly.ff, dtype=bf, device=dev)
+            add(f"polynomial activation, {T} rows", timed_graph([lambda s=s: Y.poly_norm_(s, poly.coef, poly.ff, 1e-6) for s in sets]), 0.0, 4 * T * poly.ff)
+            add("like: RMS norm", timed_graph([lambda s=s: F.rmsnorm(s, one, 1e-6) for s in sets]), 0.0, 4 * T * poly.ff)
+            del sets
+            # joins: T single rows, and one portion of T rows
+            sets = copies(lambda: (torch.randn(T, d, device=dev), rows(T, d)), 12 * T * d)
+            add(f"join: x += ls norm(y), next norm, {T} rows", timed_graph([lambda s=s: Y.join(s[0], s[1], own.norm1b, 1.0, 1e-6, own.norm2, ls=own.ls1) for s in sets]), 0.0, 12 * T * d)
+            add("like: join and next norm", timed_graph([lambda s=s: Y.join(s[0], s[1], None, 1.0, 1e-6, own.norm2) for s in sets]), 0.0, 12 * T * d)
+            b = rows_batch(T, 64) if T == 64 else portion_batch(1, T)
+            b.state_rows = b.state_rows + 1
+            b.row_state = b.row_state + 1 if b.row_state is not None else None
+            carry = Y.Carry(T + 1 if T == 64 else 2, 2, d, True, dev)
+            state = 8 * T * d if T == 64 else 0
+            sh = Y.Shift(own.shift, 0, carry, b)
+            add(f"join with token shift, {T} rows", timed_graph([lambda s=s: Y.join(s[0], s[1], own.norm1b, 1.0, 1e-6, own.norm1, ls=own.ls1, shift=sh) for s in sets]), 0.0, 12 * T * d + state)
+            add("like: join and next norm", timed_graph([lambda s=s: Y.join(s[0], s[1], None, 1.0, 1e-6, own.norm1) for s in sets]), 0.0, 12 * T * d)
+            del sets
+            b.ids = torch.randint(0, c.vocab_size, (T,), device=dev, dtype=torch.int32)
+            add(f"embedding with pairs, first norm, token shift, {T} rows", timed_graph([lambda: Y.start(b, model.embed_tokens, 2.0, own.norm1, 1e-6, model.bigram, c.bigram, sh) for _ in range(8)]), 0.0,
+                10 * T * d + state)
+            add("like: embedding + first norm", timed_graph([lambda: Y.embed(b.ids, model.embed_tokens, 2.0, own.norm1, 1e-6) for _ in range(8)]), 0.0, 8 * T * d)
+            # experts
+            unit = moe.shared
+            like = GatedExperts(dict(router={"experts": moe.experts, "top": moe.top}, expert={"ff": moe.ff}, shared={"ff": unit.ff}, weigh_input=True, corrected=False), c, bf, dev)
+            for prm in like.parameters():
+                prm.normal_(std=0.02)
+            nbs, fls = 2 * (3 * d * unit.ff + T * (d + 2 * unit.ff)), 6.0 * T * d * unit.ff
+
+            def cost(copies_):
+                used = min(moe.experts, copies_)
+                return 6.0 * copies_ * d * moe.ff + fls, 2 * (3 * used * d * moe.ff + copies_ * (2 * d + 2 * moe.ff)) + 12 * T * d + nbs
+
+            sets = copies(lambda: (torch.randn(T, d, device=dev), rows(T, d)), 16 * T * d)
+            real = round(T * moe.top * moe.experts / moe.outputs)
+            ms = timed_graph([lambda s=s: Y.feed_forward(s[0], s[1], moe, own.norm1b, 1.0, 1e-6, own.norm1, own.ls1) for s in sets[:4]])
+            add(f"experts with identity outputs, router, gated shared unit and join (all kernels), {T} rows", ms, *cost(real))
+            ms = timed_graph([lambda s=s: Y.feed_forward(s[0], s[1], like, None, 1.0, 1e-6, own.norm1) for s in sets[:4]])
+            add("like: experts with router, shared unit and join", ms, *cost(T * moe.top))
+            del sets, like
+        # attention beside chunked soft-max attention over as many keys as a query sees here
+        W, H, G = g.window, g.heads, g.kv_heads
+        twin = GroupedAttentionMixer(dict(heads=H, kv_heads=G, dim=g.dim, vdim=g.vdim, scale=g.scale, rot={"dims": g.dim, "base": 1e6}, bias=False, interleaved=False), c, bf, dev)
+        m2 = lent.mixer
+        for n, ctx in DECODE:
+            seen = min(ctx, W) + g.keep
+            for label, mx, keys in (("windowed sigmoid attention", g, seen), ("the same on another layer's keys", m2, seen), ("like: soft-max attention", twin, -(-seen // 64) * 64)):
+                b, pages = rows_batch(n, ctx if mx is not twin else keys), n * ctx // 64
+                nb = n * keys * G * (g.dim + g.vdim) * 2
+                sets = copies(lambda: (rows(n, mx.in_width), *(torch.randn(pages, G, 64, w, device=dev).to(bf) for w in (g.dim, g.vdim))), nb)
+                add(f"{label} decode (all kernels), {n} rows, {keys} keys seen", timed_graph([lambda s=s: S.attention(s[0], mx, b, s[1], s[2]) for s in sets]), 4.0 * n * keys * H * g.dim, nb)
+                del sets
+        for n, length in PREFILL:
+            for label, mx in (("windowed sigmoid attention", g), ("like: soft-max attention", twin)):
+                b, T = portion_batch(n, length), n * length
+                size = min(W, length) if mx is g else length
+                pairs = n * (size * (size + 1) / 2 + (length - size) * size)
+                if mx is g:
+                    pairs += n * g.keep * max(0, length - size)
+                kc, vc = (torch.zeros((T // 64, G, 64, w), dtype=bf, device=dev) for w in (g.dim, g.vdim))
+                nb = 2 * T * (mx.in_width + mx.mix_width + G * (g.dim + g.vdim))
+                sets = copies(lambda: rows(T, mx.in_width), nb)
+                add(f"{label} prefill (all kernels), {n} x {length}", timed_graph([lambda s=s: S.attention(s, mx, b, kc, vc) for s in sets]), 2.0 * pairs * H * (g.dim + g.vdim), nb)
+                del sets
+    return out
+
+
+def zonidra_main(steps: int = 5, warmup: int = 3, sizes=None, clocks=None) -> int:
+    torch.backends.cuda.matmul.allow_tf32 = False
+    L.lib()
+    res = dict(metric="layer-list model with norms on both sides, serving (device time)", unit="tokens/s", dtype="bf16", data="synthetic (random weights and tokens)", models={}, kernels={})
+    for name in sizes or ZONIDRA:
+        for kind in ("zonidra", "kikivik"):
+            res["models"][f"{name}:{kind}"] = serving_row(preset(name) if kind == "zonidra" else kikivik_twin(name), steps, warmup)
+        res["kernels"][name] = zonidra_table(name)
+        torch.cuda.empty_cache()
+    return finish(res, clocks)
 
 
 def kikivik_main(steps: int = 5, warmup: int = 3, sizes=None, clocks=None) -> int:

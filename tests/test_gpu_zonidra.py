@@ -272,6 +272,7 @@ def test_shift_of_many_rows(lens, d, dt):
     w, ls, nw, s = (torch.rand(d, device=DEV).to(dt) for _ in range(4))
     rows, wt, f1, f2 = torch.randint(-1, T, (T, k), device=DEV, dtype=torch.int32), torch.rand(T, k, device=DEV), torch.rand(T, device=DEV), torch.rand(T, device=DEV)
     counts = torch.ones(6, dtype=torch.int32, device=DEV)
+    carry.next.copy_(carry.state)      # (a step fills all places)
     before = carry.state.clone()
     gx, gh = Y.join(x, y, w, 1.0, 1e-3, nw, (rows, wt, counts), also, f1, h, f2, ls, Y.Shift(s, 1, carry, b))
     carry.commit(b)
