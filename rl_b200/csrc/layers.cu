@@ -5,9 +5,10 @@
 //   add_normed   x += m * rms(y) * w * ls (norms behind the sublayer) or x += y (pre-norm layers) on the fp32 stream, and what the next sublayer reads: x
 //                itself in the model's type, or its RMS norm. y is a product's output or the weighted sum of a token's expert rows (combined here, never
 //                stored), with rows of a shared unit and of the sublayer's own input added, each times a factor per row.
-//   shift_rows   the same (or the start of the stream from the embedding tables), and behind the norm the blend with the token before: h + (h' - h) s.
-//                A CTA walks a run of rows and computes the row in front of its run again, so that the rows need no order among the CTAs; the
-//                stream is written to a second buffer for that. Sequences continue from a state row [d] per place, see ShiftArgs.
+//   shift_rows   the same (or the start of the stream from the embedding tables), and behind the norm the blend with the token before: h + (h' - h) s,
+//                for few rows. A CTA computes the row in front of its own again, so that the rows need no order among the CTAs; the stream is
+//                written to a second buffer for that. Sequences continue from a state row [d] per place, see ShiftArgs.
+//   blend_rows   the norm and the blend alone, for many rows: the first pass has left the stream and its rows' reciprocal root mean squares.
 //   moe_choose   one warp per token: scores, group choice, top-k; every copy takes a number among its expert's copies.
 //   moe_place    row ranges of the experts (multiples of 128 rows) from their counts, the row of every copy, and its token's row moved there.
 //
@@ -54,6 +55,7 @@ struct AddNormed {
   const void* next_w;      // weight of the next norm (null: h is x)
   void* h;                 // [rows, d]
   float* x_out;            // [rows, d]; x itself, except in shift_rows
+  float* rstd;             // [rows] reciprocal root mean square of the new stream, in place of h (null: h)
   int d;
   float mult, eps;
   const void* also;        // [rows, ld_also] or null: added to the sublayer's output
@@ -64,8 +66,8 @@ struct AddNormed {
   const float* own_f;
 };
 
-// Columns (threadIdx.x + i * THREADS) * 4 of the sublayer's output of one row; KEEP groups of four columns per thread.
-template <typename T, int THREADS, int KEEP>
+// Columns (threadIdx.x + i * THREADS) * 4 of the sublayer's output of one row; KEEP groups of four columns per thread. EXPERTS: copy_row is set.
+template <typename T, int THREADS, int KEEP, bool EXPERTS>
 __device__ __forceinline__ void sublayer_row(const AddNormed& a, long long row, float4 (&v)[KEEP]) {
   const T *Y = static_cast<const T*>(a.y), *also = static_cast<const T*>(a.also), *own = static_cast<const T*>(a.own);
   const float fa = also && a.also_f ? a.also_f[row] : 1.f, fo = own ? a.own_f[row] : 0.f;
@@ -74,7 +76,7 @@ __device__ __forceinline__ void sublayer_row(const AddNormed& a, long long row, 
     const int c = (threadIdx.x + i * THREADS) * 4;
     v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (c >= a.d) continue;
-    if (!a.copy_row) v[i] = ld4(Y + row * a.ldy + c);
+    if (!EXPERTS) v[i] = ld4(Y + row * a.ldy + c);
     if (also) {
       const float4 t = ld4(also + row * a.ld_also + c);
       v[i].x = fmaf(fa, t.x, v[i].x); v[i].y = fmaf(fa, t.y, v[i].y); v[i].z = fmaf(fa, t.z, v[i].z); v[i].w = fmaf(fa, t.w, v[i].w);
@@ -84,7 +86,7 @@ __device__ __forceinline__ void sublayer_row(const AddNormed& a, long long row, 
       v[i].x = fmaf(fo, t.x, v[i].x); v[i].y = fmaf(fo, t.y, v[i].y); v[i].z = fmaf(fo, t.z, v[i].z); v[i].w = fmaf(fo, t.w, v[i].w);
     }
   }
-  if (!a.copy_row) return;
+  if (!EXPERTS) return;
   constexpr int AHEAD = KEEP <= 2 ? 4 : 2;      // copies in flight
   for (int j0 = 0; j0 < a.k; j0 += AHEAD) {
     float4 e[AHEAD][KEEP];
@@ -170,8 +172,8 @@ __device__ __forceinline__ float join_factor(const AddNormed& a, long long row, 
 }
 
 // AN_KEEP: groups of four columns that a thread keeps in registers
-template <typename T, int THREADS, int AN_KEEP>
-__global__ void __launch_bounds__(THREADS) add_normed_kernel(AddNormed a) {
+template <typename T, int THREADS, int AN_KEEP, bool EXPERTS>
+__global__ void __launch_bounds__(THREADS, THREADS * AN_KEEP <= 512 ? 1024 / THREADS : (THREADS * AN_KEEP <= 1024 ? 768 / THREADS : 1)) add_normed_kernel(AddNormed a) {
   __shared__ float red[32];
   pdl_sync();
   const long long row = blockIdx.x;
@@ -187,7 +189,7 @@ __global__ void __launch_bounds__(THREADS) add_normed_kernel(AddNormed a) {
       const int c = (threadIdx.x + i * THREADS) * 4;
       if (c < a.d) xv[i] = ld4(a.x + row * a.d + c);
     }
-    sublayer_row<T, THREADS, AN_KEEP>(a, row, v);
+    sublayer_row<T, THREADS, AN_KEEP, EXPERTS>(a, row, v);
     join_row<T, THREADS, AN_KEEP>(a, v, xv, red);
     float s2 = 0.f;
 #pragma unroll
@@ -195,10 +197,13 @@ __global__ void __launch_bounds__(THREADS) add_normed_kernel(AddNormed a) {
       const int c = (threadIdx.x + i * THREADS) * 4;
       if (c >= a.d) continue;
       st4(x + c, xv[i]);
-      if (!nw) st4(h + c, xv[i]);
+      if (!nw && !a.rstd) st4(h + c, xv[i]);
       s2 += xv[i].x * xv[i].x + xv[i].y * xv[i].y + xv[i].z * xv[i].z + xv[i].w * xv[i].w;
     }
-    if (nw) {
+    if (a.rstd) {
+      s2 = block_sum(s2, red);
+      if (threadIdx.x == 0) a.rstd[row] = 1.f / sqrtf(s2 / static_cast<float>(a.d) + a.eps);
+    } else if (nw) {
       s2 = block_sum(s2, red);
       const float g = 1.f / sqrtf(s2 / static_cast<float>(a.d) + a.eps);
 #pragma unroll
@@ -251,10 +256,15 @@ struct ShiftArgs {
   float* state;            // [states, ld_state], this place's columns
   float* next;
   long long rows;
-  int n_single, run;       // rows per CTA
+  int n_single;
   int* status;
 };
 
+__device__ __forceinline__ bool last_of_piece(const ShiftArgs& s, long long row) { return !s.row_off || row + 1 == s.rows || s.row_off[row + 1] == 0; }
+// Where the last row of a piece leaves its normed stream (null: another row).
+__device__ __forceinline__ float* leaves(const ShiftArgs& s, long long row, long long st) {
+  return s.s && last_of_piece(s, row) ? (row < s.n_single ? s.state : s.next) + st * s.ld_state : nullptr;
+}
 __device__ __forceinline__ long long state_row(const ShiftArgs& s, long long row) {
   const long long r = s.row_state[row];
   if (r >= 0 && r < s.num_states) return r;
@@ -282,30 +292,30 @@ __device__ __forceinline__ void start_rows(const StartArgs& e, const ShiftArgs& 
 }
 
 template <typename T, int THREADS, int KEEP, bool START>
-__global__ void __launch_bounds__(THREADS) shift_rows_kernel(AddNormed a, ShiftArgs s, StartArgs e) {
+__global__ void __launch_bounds__(THREADS, 1) shift_rows_kernel(AddNormed a, ShiftArgs s, StartArgs e) {
   __shared__ float red[32];
   pdl_sync();
-  if (!START && blockIdx.x == 0 && a.counts)
+  const long long row = blockIdx.x;
+  if (!START && row == 0 && a.counts)
     for (int i = threadIdx.x; i < a.experts; i += THREADS) a.counts[i] = 0;
-  const long long row0 = static_cast<long long>(blockIdx.x) * s.run, row1 = min(row0 + s.run, s.rows);
   const T *nw = static_cast<const T*>(a.next_w), *sw = static_cast<const T*>(s.s), *table = static_cast<const T*>(e.table), *pairs = static_cast<const T*>(e.pairs);
-  auto last_of_piece = [&](long long row) { return !s.row_off || row + 1 == s.rows || s.row_off[row + 1] == 0; };
-  auto leaves = [&](long long row, long long st) {      // where the last row of a piece leaves its normed stream
-    return sw && last_of_piece(row) ? (row < s.n_single ? s.state : s.next) + st * s.ld_state : nullptr;
-  };
-  auto leave_token = [&](long long row, long long st) {
-    if (START && e.token && last_of_piece(row)) {
-      __syncthreads();                                   // (everyone has read the old one)
-      if (threadIdx.x == 0) (row < s.n_single ? e.token : e.token_next)[st] = e.ids[row];
-    }
-  };
+  const long long st = state_row(s, row);
+  const bool first = !s.row_off || s.row_off[row] == 0, fresh = first && s.positions[row] == 0;
+  const bool again = sw && !first && !a.rstd;            // the row in front is computed again
+  float* keep = a.rstd ? nullptr : leaves(s, row, st);
+  const float* from = s.state + st * s.ld_state;
   if (a.d % 4 == 0 && a.d <= KEEP * 4 * THREADS) {
     float4 prev[KEEP];
-    for (long long row = row0 - (sw && s.row_off && s.row_off[row0] > 0 ? 1 : 0); row < row1; ++row) {
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+      const int c = (threadIdx.x + i * THREADS) * 4;
+      prev[i] = sw && first && !fresh && !a.rstd && c < a.d ? ld4(from + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    for (long long r = row - (again ? 1 : 0); r <= row; ++r) {
       float4 v[KEEP], xv[KEEP];
       if (START) {
         long long tok, pair;
-        start_rows(e, s, row, a.d, tok, pair);
+        start_rows(e, s, r, a.d, tok, pair);
 #pragma unroll
         for (int i = 0; i < KEEP; ++i) {
           const int c = (threadIdx.x + i * THREADS) * 4;
@@ -318,12 +328,13 @@ __global__ void __launch_bounds__(THREADS) shift_rows_kernel(AddNormed a, ShiftA
 #pragma unroll
         for (int i = 0; i < KEEP; ++i) {
           const int c = (threadIdx.x + i * THREADS) * 4;
-          if (c < a.d) xv[i] = ld4(a.x + row * a.d + c);
+          if (c < a.d) xv[i] = ld4(a.x + r * a.d + c);
         }
-        sublayer_row<T, THREADS, KEEP>(a, row, v);
+        if (a.copy_row) sublayer_row<T, THREADS, KEEP, true>(a, r, v);
+        else sublayer_row<T, THREADS, KEEP, false>(a, r, v);
         join_row<T, THREADS, KEEP>(a, v, xv, red);
       }
-      const bool mine = row >= row0;
+      const bool mine = r == row;
       float s2 = 0.f;
 #pragma unroll
       for (int i = 0; i < KEEP; ++i) {
@@ -334,37 +345,31 @@ __global__ void __launch_bounds__(THREADS) shift_rows_kernel(AddNormed a, ShiftA
       }
       s2 = block_sum(s2, red);
       const float g = 1.f / sqrtf(s2 / static_cast<float>(a.d) + a.eps);
-      const long long st = mine ? state_row(s, row) : 0;
-      const bool first = mine && (!s.row_off || s.row_off[row] == 0), fresh = first && s.positions[row] == 0;
-      float* keep = mine ? leaves(row, st) : nullptr;
-      const float* from = s.state + st * s.ld_state;
+      if (a.rstd) {
+        if (threadIdx.x == 0) a.rstd[row] = g;
+        break;
+      }
 #pragma unroll
       for (int i = 0; i < KEEP; ++i) {
         const int c = (threadIdx.x + i * THREADS) * 4;
         if (c >= a.d) continue;
-        const float4 wv = ld4(nw + c);
+        const float4 wv = ld4(nw + c), b = prev[i];
         const float4 h = make_float4(xv[i].x * g * wv.x, xv[i].y * g * wv.y, xv[i].z * g * wv.z, xv[i].w * g * wv.w);
-        if (mine) {
-          const float4 b = !sw || fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : (first ? ld4(from + c) : prev[i]);
-          const float4 f = sw ? ld4(sw + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-          st4(static_cast<T*>(a.h) + row * a.d + c, make_float4(fmaf(b.x - h.x, f.x, h.x), fmaf(b.y - h.y, f.y, h.y), fmaf(b.z - h.z, f.z, h.z), fmaf(b.w - h.w, f.w, h.w)));
-          if (keep) st4(keep + c, h);
-        }
         prev[i] = h;
+        if (!mine) continue;
+        const float4 f = sw ? ld4(sw + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        st4(static_cast<T*>(a.h) + row * a.d + c, make_float4(fmaf(b.x - h.x, f.x, h.x), fmaf(b.y - h.y, f.y, h.y), fmaf(b.z - h.z, f.z, h.z), fmaf(b.w - h.w, f.w, h.w)));
+        if (keep) st4(keep + c, h);
       }
-      if (mine) leave_token(row, st);
     }
-    return;
-  }
-  for (long long row = row0; row < row1; ++row) {        // any size: the row in front is computed again for every row
-    const bool first = !s.row_off || s.row_off[row] == 0, fresh = first && s.positions[row] == 0;
+  } else {                                               // any size
     float f[2] = {0.f, 0.f}, g[2] = {0.f, 0.f};
     long long tok[2] = {0, 0}, pair[2] = {-1, -1};
     auto value = [&](int q, int c) {                     // stream of row `row - q`
       if (START) return fmaf(ldv(table + tok[q] + c), e.scale, pair[q] >= 0 ? ldv(pairs + pair[q] + c) : 0.f);
       return join_value<T>(a, row - q, c, f[q]);
     };
-    for (int q = 0; q < (first || !sw ? 1 : 2); ++q) {
+    for (int q = 0; q < (again ? 2 : 1); ++q) {
       if (START) start_rows(e, s, row - q, a.d, tok[q], pair[q]);
       else f[q] = join_factor<T, THREADS>(a, row - q, red);
       float s2 = 0.f;
@@ -374,9 +379,6 @@ __global__ void __launch_bounds__(THREADS) shift_rows_kernel(AddNormed a, ShiftA
       }
       g[q] = 1.f / sqrtf(block_sum(s2, red) / static_cast<float>(a.d) + a.eps);
     }
-    const long long st = state_row(s, row);
-    float* keep = leaves(row, st);
-    const float* from = s.state + st * s.ld_state;
     for (int c = threadIdx.x; c < a.d; c += THREADS) {
       const float v = value(0, c), n = ldv(nw + c), h = v * g[0] * n;
       const float b = !sw || fresh ? 0.f : (first ? from[c] : value(1, c) * g[1] * n);
@@ -384,7 +386,46 @@ __global__ void __launch_bounds__(THREADS) shift_rows_kernel(AddNormed a, ShiftA
       st1(static_cast<T*>(a.h) + row * a.d + c, fmaf(b - h, sw ? ldv(sw + c) : 0.f, h));
       if (keep) keep[c] = h;
     }
-    leave_token(row, st);
+  }
+  if (START && e.token && last_of_piece(s, row)) {
+    __syncthreads();                                     // (everyone has read the old one)
+    if (threadIdx.x == 0) (row < s.n_single ? e.token : e.token_next)[st] = e.ids[row];
+  }
+}
+
+// h = n + (n' - n) * s with n = x * rstd * nw of the row and n' that of the token before. A thread walks BR_RUN rows of its four columns.
+constexpr int BR_THREADS = 128, BR_RUN = 8;
+template <typename T>
+__global__ void __launch_bounds__(BR_THREADS) blend_rows_kernel(const float* __restrict__ x, const float* __restrict__ rstd, const T* __restrict__ nw, T* __restrict__ h,
+                                                                int d, ShiftArgs s) {
+  const int c = (blockIdx.y * BR_THREADS + threadIdx.x) * 4;
+  const long long row0 = static_cast<long long>(blockIdx.x) * BR_RUN;
+  pdl_sync();
+  if (c >= d) return;
+  const float4 wv = ld4(nw + c), f = ld4(static_cast<const T*>(s.s) + c);
+  float4 xv[BR_RUN + 1];
+#pragma unroll
+  for (int i = 0; i <= BR_RUN; ++i) {
+    const long long r = row0 - 1 + i;
+    xv[i] = r >= 0 && r < s.rows ? ld4(x + r * d + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  auto normed = [&](float4 v, long long r) {
+    const float g = rstd[r];
+    return make_float4(v.x * g * wv.x, v.y * g * wv.y, v.z * g * wv.z, v.w * g * wv.w);
+  };
+  float4 prev = row0 > 0 ? normed(xv[0], row0 - 1) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < BR_RUN; ++i) {
+    const long long row = row0 + i;
+    if (row >= s.rows) break;
+    const float4 n = normed(xv[i + 1], row);
+    const bool first = !s.row_off || s.row_off[row] == 0;
+    long long st = 0;
+    if (first || last_of_piece(s, row)) st = state_row(s, row);
+    if (first) prev = s.positions[row] > 0 ? ld4(s.state + st * s.ld_state + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    st4(h + row * d + c, make_float4(fmaf(prev.x - n.x, f.x, n.x), fmaf(prev.y - n.y, f.y, n.y), fmaf(prev.z - n.z, f.z, n.z), fmaf(prev.w - n.w, f.w, n.w)));
+    if (float* keep = leaves(s, row, st)) st4(keep + c, n);
+    prev = n;
   }
 }
 
@@ -751,7 +792,7 @@ struct RlbJoin {
   const void *w, *ls, *next_w, *also, *own;
   const float *also_f, *own_f;
   void* h;
-  float* x_out;
+  float *x_out, *rstd;
   long long ldy, ld_also, ld_own, rows;
   int f32, k, y_rows, experts, d;
   float mult, eps;
@@ -775,7 +816,8 @@ namespace {
 int join_args(const RlbJoin& j, AddNormed& a) {
   if (j.d % 4 == 0 && ((j.y && j.ldy % 4) || (j.also && j.ld_also % 4) || (j.own && j.ld_own % 4))) return -2;
   if (j.own && !j.own_f) return -2;
-  a = AddNormed{j.x, j.y, j.ldy, j.copy_row, j.weight, j.k, j.y_rows, j.counts, j.experts, j.w, j.ls, j.next_w, j.h, j.x_out, j.d, j.mult, j.eps,
+  if (j.rstd && (j.d % 4 || j.d > 4096)) return -2;
+  a = AddNormed{j.x, j.y, j.ldy, j.copy_row, j.weight, j.k, j.y_rows, j.counts, j.experts, j.w, j.ls, j.next_w, j.h, j.x_out, j.rstd, j.d, j.mult, j.eps,
                 j.also, j.ld_also, j.also_f, j.own, j.ld_own, j.own_f};
   return 0;
 }
@@ -783,6 +825,7 @@ int join_args(const RlbJoin& j, AddNormed& a) {
 
 // x [rows, d] fp32 += mult * rms(y) * w * ls (w null: mult * y * ls); h [rows, d] = x, or rms(x) * next_w. With copy_row [rows, k]: y of a row is the
 // sum of its k weighted (weight null: plain) rows of y [y_rows, ldy], and counts [experts] are set to zero. also, own: added to y times their factors.
+// rstd [rows] (d a multiple of 4, at most 4096): written in place of h, for rlb_blend_rows.
 RLB_API int rlb_add_normed(const RlbJoin* j, void* stream) {
   if (j->rows <= 0) return 0;
   AddNormed a;
@@ -791,17 +834,18 @@ RLB_API int rlb_add_normed(const RlbJoin* j, void* stream) {
   const int d = j->d;
   const dim3 grid(static_cast<unsigned>(rows));
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (j->f32) return static_cast<int>(rlb_launch_pdl(add_normed_kernel<float, 256, 8>, grid, dim3(256), 0, s, a));
-  const bool few = rows < 148 * 4;      // few rows: more threads per row
-  auto kernel = few && d > 1024 ? (d <= 2048 ? add_normed_kernel<__nv_bfloat16, 512, 1> : (d <= 4096 ? add_normed_kernel<__nv_bfloat16, 512, 2>
-                                                                                                : add_normed_kernel<__nv_bfloat16, 512, 4>))
-                           : (d <= 1024 ? add_normed_kernel<__nv_bfloat16, 256, 1> : (d <= 2048 ? add_normed_kernel<__nv_bfloat16, 256, 2>
-                              : (d <= 4096 ? add_normed_kernel<__nv_bfloat16, 256, 4> : add_normed_kernel<__nv_bfloat16, 256, 8>)));
-  return static_cast<int>(rlb_launch_pdl(kernel, grid, dim3(few && d > 1024 ? 512 : 256), 0, s, a));
+  auto go = [&](auto kernel, int threads) { return static_cast<int>(rlb_launch_pdl(kernel, grid, dim3(threads), 0, s, a)); };
+#define RLB_ADD(T, THREADS, KEEP) (a.copy_row ? go(add_normed_kernel<T, THREADS, KEEP, true>, THREADS) : go(add_normed_kernel<T, THREADS, KEEP, false>, THREADS))
+  if (j->f32) return RLB_ADD(float, 256, 8);
+  if (rows < 148 * 4 && d > 1024)       // few rows: more threads per row
+    return d <= 2048 ? RLB_ADD(__nv_bfloat16, 512, 1) : (d <= 4096 ? RLB_ADD(__nv_bfloat16, 512, 2) : RLB_ADD(__nv_bfloat16, 512, 4));
+  return d <= 1024 ? RLB_ADD(__nv_bfloat16, 256, 1) : (d <= 2048 ? RLB_ADD(__nv_bfloat16, 256, 2) : (d <= 4096 ? RLB_ADD(__nv_bfloat16, 256, 4)
+                                                                                                                : RLB_ADD(__nv_bfloat16, 256, 8)));
+#undef RLB_ADD
 }
 
 // rlb_add_normed into x_out, or with ids the embedding, and h = n + (n' - n) * s with n = rms(x) * next_w and n' that of the sequence's token
-// before (s null, with ids only: h = n).
+// before (s null, with ids only: h = n). With rstd only the stream and the reciprocal root mean squares are written.
 RLB_API int rlb_shift_rows(const RlbJoin* j, const RlbShift* t, void* stream) {
   if (j->rows <= 0) return 0;
   AddNormed a;
@@ -812,11 +856,9 @@ RLB_API int rlb_shift_rows(const RlbJoin* j, const RlbShift* t, void* stream) {
   if (j->d % 4 == 0 && t->ld_state % 4) return -2;
   const long long rows = j->rows;
   const int d = j->d;
-  // a run of rows costs one row more; few rows are a matter of latency
-  const int run = rows < 148 * 4 ? 1 : (rows < 148 * 16 ? 2 : 4);
-  ShiftArgs s{t->s, t->positions, t->row_off, t->row_state, t->num_states, t->ld_state, t->state, t->next, rows, t->n_single, run, t->status};
+  ShiftArgs s{t->s, t->positions, t->row_off, t->row_state, t->num_states, t->ld_state, t->state, t->next, rows, t->n_single, t->status};
   StartArgs e{t->ids, t->table, t->vocab, t->scale, t->pairs, t->buckets, t->mul_prev, t->mul_cur, t->token, t->token_next};
-  const dim3 grid(static_cast<unsigned>((rows + run - 1) / run));
+  const dim3 grid(static_cast<unsigned>(rows));
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   auto go = [&](auto kernel, int threads) { return static_cast<int>(rlb_launch_pdl(kernel, grid, dim3(threads), 0, st, a, s, e)); };
 #define RLB_SHIFT(T, THREADS, KEEP) (start ? go(shift_rows_kernel<T, THREADS, KEEP, true>, THREADS) : go(shift_rows_kernel<T, THREADS, KEEP, false>, THREADS))
@@ -825,6 +867,18 @@ RLB_API int rlb_shift_rows(const RlbJoin* j, const RlbShift* t, void* stream) {
   return d <= 1024 ? RLB_SHIFT(__nv_bfloat16, 256, 1) : (d <= 2048 ? RLB_SHIFT(__nv_bfloat16, 256, 2) : (d <= 4096 ? RLB_SHIFT(__nv_bfloat16, 256, 4)
                                                                                                                 : RLB_SHIFT(__nv_bfloat16, 512, 4)));
 #undef RLB_SHIFT
+}
+
+// h [rows, d] = n + (n' - n) * t->s with n = x * rstd * nw; d a multiple of 4.
+RLB_API int rlb_blend_rows(const float* x, const float* rstd, const void* nw, void* h, int f32, long long rows, int d, const RlbShift* t, void* stream) {
+  if (rows <= 0) return 0;
+  if (d % 4 || t->ld_state % 4 || !t->s || !t->state || !t->next) return -2;
+  ShiftArgs s{t->s, t->positions, t->row_off, t->row_state, t->num_states, t->ld_state, t->state, t->next, rows, t->n_single, t->status};
+  const dim3 grid(static_cast<unsigned>((rows + BR_RUN - 1) / BR_RUN), (d / 4 + BR_THREADS - 1) / BR_THREADS);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (f32) return static_cast<int>(rlb_launch_pdl(blend_rows_kernel<float>, grid, dim3(BR_THREADS), 0, st, x, rstd, static_cast<const float*>(nw), static_cast<float*>(h), d, s));
+  return static_cast<int>(rlb_launch_pdl(blend_rows_kernel<__nv_bfloat16>, grid, dim3(BR_THREADS), 0, st, x, rstd, static_cast<const __nv_bfloat16*>(nw),
+                                         static_cast<__nv_bfloat16*>(h), d, s));
 }
 
 // state [num_states, width] and token [num_states] (null: none) of the state rows `rows` [n] take over what the step left in the second buffers.

@@ -26,6 +26,7 @@ register("rlb_linear_skinny", [P, P])
 register("rlb_linear_grouped", [P, P])
 register("rlb_add_normed", [P, P])
 register("rlb_shift_rows", [P, P, P])
+register("rlb_blend_rows", [P, P, P, P, I, LL, I, P, P])
 register("rlb_commit_states", [P, P, LL, P, P, P, I, LL, P, P])
 register("rlb_poly_norm_rows", [P, LL, I, P, LL, I, CF, P])
 register("rlb_group_norm_rows", [P, LL, I, P, LL, I, I, CF, P])
@@ -114,7 +115,7 @@ def _rms(x: torch.Tensor, eps: float) -> torch.Tensor:
 
 
 class _Join(C.Structure):
-    _fields_ = [(n, C.c_void_p) for n in ("x", "y", "copy_row", "weight", "counts", "w", "ls", "next_w", "also", "own", "also_f", "own_f", "h", "x_out")] + \
+    _fields_ = [(n, C.c_void_p) for n in ("x", "y", "copy_row", "weight", "counts", "w", "ls", "next_w", "also", "own", "also_f", "own_f", "h", "x_out", "rstd")] + \
                [(n, C.c_longlong) for n in ("ldy", "ld_also", "ld_own", "rows")] + [(n, C.c_int) for n in ("f32", "k", "y_rows", "experts", "d")] + \
                [(n, C.c_float) for n in ("mult", "eps")]
 
@@ -154,6 +155,13 @@ class Shift:
     place: int
     carry: Carry
     b: TokenBatch
+
+
+FUSED_SHIFT_ROWS = 148 * 4      # fewer rows are blended by the kernel that joins or embeds them, more in a pass of their own
+
+
+def _blend_after(T: int, d: int, t: Optional[Shift]) -> bool:
+    return t is not None and t.s is not None and T >= FUSED_SHIFT_ROWS and d % 4 == 0 and d <= 4096
 
 
 def _pieces(b: TokenBatch) -> list:
@@ -210,7 +218,11 @@ def start(b: TokenBatch, table: torch.Tensor, scale: float, norm: torch.Tensor, 
     if pairs is not None:
         q.pairs, q.buckets, q.mul_prev, q.mul_cur = ptr(pairs), bigram["buckets"], bigram["mul_prev"], bigram["mul_cur"]
         q.token, q.token_next = ptr(c.token), ptr(c.token_next)
+    after = torch.empty(T, dtype=torch.float32, device=x.device) if _blend_after(T, d, t) else None
+    j.rstd = ptr(after)
     call("rlb_shift_rows", C.byref(j), C.byref(q), stream_ptr())
+    if after is not None:
+        call("rlb_blend_rows", ptr(x), ptr(after), ptr(norm), ptr(h), _f32(h), T, d, C.byref(q), stream_ptr())
     return x, h
 
 
@@ -218,7 +230,7 @@ def join(x: torch.Tensor, y: torch.Tensor, w: Optional[torch.Tensor], mult: floa
          experts: Optional[tuple] = None, also: Optional[torch.Tensor] = None, also_f: Optional[torch.Tensor] = None, own: Optional[torch.Tensor] = None,
          own_f: Optional[torch.Tensor] = None, ls: Optional[torch.Tensor] = None, shift: Optional[Shift] = None):
     """(x, h) with x + mult * rms(y) * w * ls (w None: mult * y; ls None: ones) and h: x in the model's type, or rms(x) * next_norm, blended by
-    ``shift``. x is updated in place, with ``shift`` it moves to a new buffer. ``experts`` = (row of every copy, weight of every copy or None, the
+    ``shift``. x is updated in place, or with ``shift`` moves to a new buffer. ``experts`` = (row of every copy, weight of every copy or None, the
     experts' counts to reset): y holds expert rows, a token's value is the (weighted) sum of its copies' rows. ``also`` / ``own``: rows added to y
     first, times ``also_f`` (None: 1) / ``own_f`` [T]."""
     if not use_native(x):
@@ -233,16 +245,21 @@ def join(x: torch.Tensor, y: torch.Tensor, w: Optional[torch.Tensor], mult: floa
         return x, (h if shift is None else _shift_ref(h, shift)).to((next_norm if w is None else w).dtype)
     T, d = x.shape
     h = torch.empty((T, d), dtype=y.dtype, device=x.device)
-    out = x if shift is None else torch.empty_like(x)
+    after = torch.empty(T, dtype=torch.float32, device=x.device) if _blend_after(T, d, shift) else None
+    out = x if shift is None or after is not None else torch.empty_like(x)
     rows, wt, counts = experts if experts is not None else (None, None, None)
     j = _Join()
     j.x, j.y, j.copy_row, j.weight, j.counts, j.w, j.ls, j.next_w = ptr(x), ptr(y), ptr(rows), ptr(wt), ptr(counts), ptr(w), ptr(ls), ptr(next_norm)
     j.also, j.also_f, j.own, j.own_f, j.h, j.x_out = ptr(also), ptr(also_f), ptr(own), ptr(own_f), ptr(h), ptr(out)
     j.ldy, j.ld_also, j.ld_own, j.rows, j.d = y.stride(0), also.stride(0) if also is not None else 0, own.stride(0) if own is not None else 0, T, d
     j.f32, j.k, j.y_rows, j.experts = _f32(y), rows.shape[1] if rows is not None else 0, y.shape[0], counts.numel() if counts is not None else 0
-    j.mult, j.eps = mult, eps
+    j.mult, j.eps, j.rstd = mult, eps, ptr(after)
     if shift is None:
         call("rlb_add_normed", C.byref(j), stream_ptr())
+    elif after is not None:
+        call("rlb_add_normed", C.byref(j), stream_ptr())
+        q = _shift_desc(shift)
+        call("rlb_blend_rows", ptr(out), ptr(after), ptr(next_norm), ptr(h), _f32(h), T, d, C.byref(q), stream_ptr())
     else:
         q = _shift_desc(shift)
         call("rlb_shift_rows", C.byref(j), C.byref(q), stream_ptr())

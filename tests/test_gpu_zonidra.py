@@ -274,7 +274,7 @@ def test_shift_of_many_rows(lens, d, dt):
     counts = torch.ones(6, dtype=torch.int32, device=DEV)
     carry.next.copy_(carry.state)      # (a step fills all places)
     before = carry.state.clone()
-    gx, gh = Y.join(x, y, w, 1.0, 1e-3, nw, (rows, wt, counts), also, f1, h, f2, ls, Y.Shift(s, 1, carry, b))
+    gx, gh = Y.join(x.clone(), y, w, 1.0, 1e-3, nw, (rows, wt, counts), also, f1, h, f2, ls, Y.Shift(s, 1, carry, b))
     carry.commit(b)
     v = (torch.where(rows[..., None] >= 0, y[rows.clamp(min=0).long()].double(), 0.0) * wt[..., None].double()).sum(1) + also.double() * f1[:, None] + h.double() * f2[:, None]
     want = x.double() + O.rms(v, 1e-3) * w.double() * ls.double()
