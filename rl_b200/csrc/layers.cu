@@ -70,21 +70,23 @@ struct AddNormed {
 template <typename T, int THREADS, int KEEP, bool EXPERTS>
 __device__ __forceinline__ void sublayer_row(const AddNormed& a, long long row, float4 (&v)[KEEP]) {
   const T *Y = static_cast<const T*>(a.y), *also = static_cast<const T*>(a.also), *own = static_cast<const T*>(a.own);
-  const float fa = also && a.also_f ? a.also_f[row] : 1.f, fo = own ? a.own_f[row] : 0.f;
 #pragma unroll
   for (int i = 0; i < KEEP; ++i) {
     const int c = (threadIdx.x + i * THREADS) * 4;
-    v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (c >= a.d) continue;
-    if (!EXPERTS) v[i] = ld4(Y + row * a.ldy + c);
-    if (also) {
-      const float4 t = ld4(also + row * a.ld_also + c);
-      v[i].x = fmaf(fa, t.x, v[i].x); v[i].y = fmaf(fa, t.y, v[i].y); v[i].z = fmaf(fa, t.z, v[i].z); v[i].w = fmaf(fa, t.w, v[i].w);
+    v[i] = !EXPERTS && c < a.d ? ld4(Y + row * a.ldy + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  auto add = [&](const T* p, float f) {
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+      const int c = (threadIdx.x + i * THREADS) * 4;
+      const float4 t = c < a.d ? ld4(p + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      v[i].x = fmaf(f, t.x, v[i].x); v[i].y = fmaf(f, t.y, v[i].y); v[i].z = fmaf(f, t.z, v[i].z); v[i].w = fmaf(f, t.w, v[i].w);
     }
-    if (fo != 0.f) {
-      const float4 t = ld4(own + row * a.ld_own + c);
-      v[i].x = fmaf(fo, t.x, v[i].x); v[i].y = fmaf(fo, t.y, v[i].y); v[i].z = fmaf(fo, t.z, v[i].z); v[i].w = fmaf(fo, t.w, v[i].w);
-    }
+  };
+  if (also) add(also + row * a.ld_also, a.also_f ? a.also_f[row] : 1.f);
+  if (own) {
+    const float f = a.own_f[row];
+    if (f != 0.f) add(own + row * a.ld_own, f);
   }
   if (!EXPERTS) return;
   constexpr int AHEAD = KEEP <= 2 ? 4 : 2;      // copies in flight
@@ -126,19 +128,27 @@ __device__ __forceinline__ void join_row(const AddNormed& a, const float4 (&v)[K
     ss = block_sum(ss, red);
     f = a.mult / sqrtf(ss / static_cast<float>(a.d) + a.eps);
   }
+  auto add = [&](auto weight) {
 #pragma unroll
-  for (int i = 0; i < KEEP; ++i) {
-    const int c = (threadIdx.x + i * THREADS) * 4;
-    if (c >= a.d) continue;
-    float4 wv = w ? ld4(w + c) : make_float4(1.f, 1.f, 1.f, 1.f);
-    if (ls) {
-      const float4 l = ld4(ls + c);
-      wv.x *= l.x; wv.y *= l.y; wv.z *= l.z; wv.w *= l.w;
+    for (int i = 0; i < KEEP; ++i) {
+      const int c = (threadIdx.x + i * THREADS) * 4;
+      if (c >= a.d) continue;
+      const float4 wv = weight(c);
+      xv[i].x = fmaf(v[i].x * f, wv.x, xv[i].x);
+      xv[i].y = fmaf(v[i].y * f, wv.y, xv[i].y);
+      xv[i].z = fmaf(v[i].z * f, wv.z, xv[i].z);
+      xv[i].w = fmaf(v[i].w * f, wv.w, xv[i].w);
     }
-    xv[i].x = fmaf(v[i].x * f, wv.x, xv[i].x);
-    xv[i].y = fmaf(v[i].y * f, wv.y, xv[i].y);
-    xv[i].z = fmaf(v[i].z * f, wv.z, xv[i].z);
-    xv[i].w = fmaf(v[i].w * f, wv.w, xv[i].w);
+  };
+  if (w && ls) {
+    add([&](int c) {
+      const float4 x = ld4(w + c), y = ld4(ls + c);
+      return make_float4(x.x * y.x, x.y * y.y, x.z * y.z, x.w * y.w);
+    });
+  } else if (w || ls) {
+    add([&](int c) { return ld4((w ? w : ls) + c); });
+  } else {
+    add([](int) { return make_float4(1.f, 1.f, 1.f, 1.f); });
   }
 }
 
@@ -171,7 +181,7 @@ __device__ __forceinline__ float join_factor(const AddNormed& a, long long row, 
   return a.mult / sqrtf(block_sum(ss, red) / static_cast<float>(a.d) + a.eps);
 }
 
-// AN_KEEP: groups of four columns that a thread keeps in registers
+// d a multiple of 4, at most 4 * AN_KEEP * THREADS: AN_KEEP groups of four columns stay in a thread's registers.
 template <typename T, int THREADS, int AN_KEEP, bool EXPERTS>
 __global__ void __launch_bounds__(THREADS, THREADS * AN_KEEP <= 512 ? 1024 / THREADS : (THREADS * AN_KEEP <= 1024 ? 768 / THREADS : 1)) add_normed_kernel(AddNormed a) {
   __shared__ float red[32];
@@ -182,43 +192,53 @@ __global__ void __launch_bounds__(THREADS, THREADS * AN_KEEP <= 512 ? 1024 / THR
   float* x = a.x_out + row * a.d;
   T* h = static_cast<T*>(a.h) + row * a.d;
   const T* nw = static_cast<const T*>(a.next_w);
-  if (a.d % 4 == 0 && a.d <= AN_KEEP * 4 * THREADS) {
-    float4 v[AN_KEEP], xv[AN_KEEP];
+  float4 v[AN_KEEP], xv[AN_KEEP];
 #pragma unroll
-    for (int i = 0; i < AN_KEEP; ++i) {
-      const int c = (threadIdx.x + i * THREADS) * 4;
-      if (c < a.d) xv[i] = ld4(a.x + row * a.d + c);
-    }
-    sublayer_row<T, THREADS, AN_KEEP, EXPERTS>(a, row, v);
-    join_row<T, THREADS, AN_KEEP>(a, v, xv, red);
-    float s2 = 0.f;
+  for (int i = 0; i < AN_KEEP; ++i) {
+    const int c = (threadIdx.x + i * THREADS) * 4;
+    xv[i] = c < a.d ? ld4(a.x + row * a.d + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  sublayer_row<T, THREADS, AN_KEEP, EXPERTS>(a, row, v);
+  join_row<T, THREADS, AN_KEEP>(a, v, xv, red);
+  float s2 = 0.f;
 #pragma unroll
-    for (int i = 0; i < AN_KEEP; ++i) {
-      const int c = (threadIdx.x + i * THREADS) * 4;
-      if (c >= a.d) continue;
-      st4(x + c, xv[i]);
-      if (!nw && !a.rstd) st4(h + c, xv[i]);
-      s2 += xv[i].x * xv[i].x + xv[i].y * xv[i].y + xv[i].z * xv[i].z + xv[i].w * xv[i].w;
-    }
-    if (a.rstd) {
-      s2 = block_sum(s2, red);
-      if (threadIdx.x == 0) a.rstd[row] = 1.f / sqrtf(s2 / static_cast<float>(a.d) + a.eps);
-    } else if (nw) {
-      s2 = block_sum(s2, red);
-      const float g = 1.f / sqrtf(s2 / static_cast<float>(a.d) + a.eps);
-#pragma unroll
-      for (int i = 0; i < AN_KEEP; ++i) {
-        const int c = (threadIdx.x + i * THREADS) * 4;
-        if (c >= a.d) continue;
-        const float4 wv = ld4(nw + c);
-        st4(h + c, make_float4(xv[i].x * g * wv.x, xv[i].y * g * wv.y, xv[i].z * g * wv.z, xv[i].w * g * wv.w));
-      }
-    }
+  for (int i = 0; i < AN_KEEP; ++i) {
+    const int c = (threadIdx.x + i * THREADS) * 4;
+    if (c >= a.d) continue;
+    st4(x + c, xv[i]);
+    if (!nw && !a.rstd) st4(h + c, xv[i]);
+    s2 += xv[i].x * xv[i].x + xv[i].y * xv[i].y + xv[i].z * xv[i].z + xv[i].w * xv[i].w;
+  }
+  if (!nw && !a.rstd) return;
+  s2 = block_sum(s2, red);
+  const float g = 1.f / sqrtf(s2 / static_cast<float>(a.d) + a.eps);
+  if (a.rstd) {
+    if (threadIdx.x == 0) a.rstd[row] = g;
     return;
   }
-  const float f = join_factor<T, THREADS>(a, row, red);
+#pragma unroll
+  for (int i = 0; i < AN_KEEP; ++i) {
+    const int c = (threadIdx.x + i * THREADS) * 4;
+    if (c >= a.d) continue;
+    const float4 wv = ld4(nw + c);
+    st4(h + c, make_float4(xv[i].x * g * wv.x, xv[i].y * g * wv.y, xv[i].z * g * wv.z, xv[i].w * g * wv.w));
+  }
+}
+
+// Any size.
+template <typename T>
+__global__ void __launch_bounds__(256) add_normed_any_kernel(AddNormed a) {
+  __shared__ float red[32];
+  pdl_sync();
+  const long long row = blockIdx.x;
+  if (row == 0 && a.counts)
+    for (int e = threadIdx.x; e < a.experts; e += 256) a.counts[e] = 0;
+  float* x = a.x_out + row * a.d;
+  T* h = static_cast<T*>(a.h) + row * a.d;
+  const T* nw = static_cast<const T*>(a.next_w);
+  const float f = join_factor<T, 256>(a, row, red);
   float s2 = 0.f;
-  for (int c = threadIdx.x; c < a.d; c += THREADS) {
+  for (int c = threadIdx.x; c < a.d; c += 256) {
     const float v = join_value<T>(a, row, c, f);
     x[c] = v;
     if (!nw) st1(h + c, v);
@@ -227,7 +247,7 @@ __global__ void __launch_bounds__(THREADS, THREADS * AN_KEEP <= 512 ? 1024 / THR
   if (!nw) return;
   s2 = block_sum(s2, red);
   const float g = 1.f / sqrtf(s2 / static_cast<float>(a.d) + a.eps);
-  for (int c = threadIdx.x; c < a.d; c += THREADS) st1(h + c, x[c] * g * ldv(nw + c));
+  for (int c = threadIdx.x; c < a.d; c += 256) st1(h + c, x[c] * g * ldv(nw + c));
 }
 
 // ---------------------------------------------------------------- blend with the token before
@@ -301,15 +321,15 @@ __global__ void __launch_bounds__(THREADS, 1) shift_rows_kernel(AddNormed a, Shi
   const T *nw = static_cast<const T*>(a.next_w), *sw = static_cast<const T*>(s.s), *table = static_cast<const T*>(e.table), *pairs = static_cast<const T*>(e.pairs);
   const long long st = state_row(s, row);
   const bool first = !s.row_off || s.row_off[row] == 0, fresh = first && s.positions[row] == 0;
-  const bool again = sw && !first && !a.rstd;            // the row in front is computed again
-  float* keep = a.rstd ? nullptr : leaves(s, row, st);
+  const bool again = sw && !first;                       // the row in front is computed again
+  float* keep = leaves(s, row, st);
   const float* from = s.state + st * s.ld_state;
   if (a.d % 4 == 0 && a.d <= KEEP * 4 * THREADS) {
     float4 prev[KEEP];
 #pragma unroll
     for (int i = 0; i < KEEP; ++i) {
       const int c = (threadIdx.x + i * THREADS) * 4;
-      prev[i] = sw && first && !fresh && !a.rstd && c < a.d ? ld4(from + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      prev[i] = sw && first && !fresh && c < a.d ? ld4(from + c) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
     for (long long r = row - (again ? 1 : 0); r <= row; ++r) {
       float4 v[KEEP], xv[KEEP];
@@ -345,10 +365,6 @@ __global__ void __launch_bounds__(THREADS, 1) shift_rows_kernel(AddNormed a, Shi
       }
       s2 = block_sum(s2, red);
       const float g = 1.f / sqrtf(s2 / static_cast<float>(a.d) + a.eps);
-      if (a.rstd) {
-        if (threadIdx.x == 0) a.rstd[row] = g;
-        break;
-      }
 #pragma unroll
       for (int i = 0; i < KEEP; ++i) {
         const int c = (threadIdx.x + i * THREADS) * 4;
@@ -391,6 +407,38 @@ __global__ void __launch_bounds__(THREADS, 1) shift_rows_kernel(AddNormed a, Shi
     __syncthreads();                                     // (everyone has read the old one)
     if (threadIdx.x == 0) (row < s.n_single ? e.token : e.token_next)[st] = e.ids[row];
   }
+}
+
+// The start of the stream alone: x and rstd.
+template <typename T, int THREADS, int KEEP>
+__global__ void __launch_bounds__(THREADS) start_rows_kernel(AddNormed a, ShiftArgs s, StartArgs e) {
+  __shared__ float red[32];
+  pdl_sync();
+  const long long row = blockIdx.x;
+  const T *table = static_cast<const T*>(e.table), *pairs = static_cast<const T*>(e.pairs);
+  long long tok, pair;
+  start_rows(e, s, row, a.d, tok, pair);
+  float4 v[KEEP], w[KEEP];
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i) {
+    const int c = (threadIdx.x + i * THREADS) * 4;
+    v[i] = w[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c >= a.d) continue;
+    v[i] = ld4(table + tok + c);
+    if (pair >= 0) w[i] = ld4(pairs + pair + c);
+  }
+  float s2 = 0.f;
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i) {
+    const int c = (threadIdx.x + i * THREADS) * 4;
+    const float4 x = make_float4(fmaf(v[i].x, e.scale, w[i].x), fmaf(v[i].y, e.scale, w[i].y), fmaf(v[i].z, e.scale, w[i].z), fmaf(v[i].w, e.scale, w[i].w));
+    if (c < a.d) st4(a.x_out + row * a.d + c, x);
+    s2 += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+  }
+  s2 = block_sum(s2, red);      // (everyone has read the old token)
+  if (threadIdx.x) return;
+  a.rstd[row] = 1.f / sqrtf(s2 / static_cast<float>(a.d) + a.eps);
+  if (e.token && last_of_piece(s, row)) (row < s.n_single ? e.token : e.token_next)[state_row(s, row)] = e.ids[row];
 }
 
 // h = n + (n' - n) * s with n = x * rstd * nw of the row and n' that of the token before. A thread walks BR_RUN rows of its four columns.
@@ -836,7 +884,8 @@ RLB_API int rlb_add_normed(const RlbJoin* j, void* stream) {
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   auto go = [&](auto kernel, int threads) { return static_cast<int>(rlb_launch_pdl(kernel, grid, dim3(threads), 0, s, a)); };
 #define RLB_ADD(T, THREADS, KEEP) (a.copy_row ? go(add_normed_kernel<T, THREADS, KEEP, true>, THREADS) : go(add_normed_kernel<T, THREADS, KEEP, false>, THREADS))
-  if (j->f32) return RLB_ADD(float, 256, 8);
+  if (d % 4 || d > 8192) return j->f32 ? go(add_normed_any_kernel<float>, 256) : go(add_normed_any_kernel<__nv_bfloat16>, 256);
+  if (j->f32) return d <= 4096 ? RLB_ADD(float, 256, 4) : RLB_ADD(float, 256, 8);
   if (rows < 148 * 4 && d > 1024)       // few rows: more threads per row
     return d <= 2048 ? RLB_ADD(__nv_bfloat16, 512, 1) : (d <= 4096 ? RLB_ADD(__nv_bfloat16, 512, 2) : RLB_ADD(__nv_bfloat16, 512, 4));
   return d <= 1024 ? RLB_ADD(__nv_bfloat16, 256, 1) : (d <= 2048 ? RLB_ADD(__nv_bfloat16, 256, 2) : (d <= 4096 ? RLB_ADD(__nv_bfloat16, 256, 4)
@@ -845,7 +894,7 @@ RLB_API int rlb_add_normed(const RlbJoin* j, void* stream) {
 }
 
 // rlb_add_normed into x_out, or with ids the embedding, and h = n + (n' - n) * s with n = rms(x) * next_w and n' that of the sequence's token
-// before (s null, with ids only: h = n). With rstd only the stream and the reciprocal root mean squares are written.
+// before (s null, with ids only: h = n). With ids and rstd only the stream and the reciprocal root mean squares are written.
 RLB_API int rlb_shift_rows(const RlbJoin* j, const RlbShift* t, void* stream) {
   if (j->rows <= 0) return 0;
   AddNormed a;
@@ -862,6 +911,12 @@ RLB_API int rlb_shift_rows(const RlbJoin* j, const RlbShift* t, void* stream) {
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   auto go = [&](auto kernel, int threads) { return static_cast<int>(rlb_launch_pdl(kernel, grid, dim3(threads), 0, st, a, s, e)); };
 #define RLB_SHIFT(T, THREADS, KEEP) (start ? go(shift_rows_kernel<T, THREADS, KEEP, true>, THREADS) : go(shift_rows_kernel<T, THREADS, KEEP, false>, THREADS))
+  if (a.rstd) {
+    if (!start) return -2;
+    if (j->f32) return go(start_rows_kernel<float, 256, 4>, 256);
+    return d <= 1024 ? go(start_rows_kernel<__nv_bfloat16, 128, 2>, 128) : (d <= 2048 ? go(start_rows_kernel<__nv_bfloat16, 256, 2>, 256)
+                                                                                        : go(start_rows_kernel<__nv_bfloat16, 256, 4>, 256));
+  }
   if (j->f32) return RLB_SHIFT(float, 256, 4);
   if (rows < 148 * 4 && d > 1024) return d <= 2048 ? RLB_SHIFT(__nv_bfloat16, 512, 1) : (d <= 4096 ? RLB_SHIFT(__nv_bfloat16, 512, 2) : RLB_SHIFT(__nv_bfloat16, 512, 4));
   return d <= 1024 ? RLB_SHIFT(__nv_bfloat16, 256, 1) : (d <= 2048 ? RLB_SHIFT(__nv_bfloat16, 256, 2) : (d <= 4096 ? RLB_SHIFT(__nv_bfloat16, 256, 4)
