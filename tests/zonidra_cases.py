@@ -48,8 +48,8 @@ CASES = {
                    (attention(heads=3, kv_heads=1, dim=7, vdim=7, rot_dims=2, size=2, keep=5), dense(ff=6))], width=37, vocab=61, bigram=(12, 5, 7)),
     # causal layers, no rotation, wide groups; no pair table
     "causal": config([(attention(heads=6, kv_heads=1, dim=16, vdim=40, rot_dims=0, size=0), dense()), (attention(heads=4, kv_heads=1, dim=32, vdim=40, rot_dims=32, size=64, keep=5), moe(top=7, identity=4))], bigram=None),
-    # one bucket only, everything the token's own row
-    "narrow": config([(attention(heads=8, kv_heads=8, dim=8, vdim=8, rot_dims=8, size=33, keep=0), moe(experts=1, identity=1, top=2)), (attention(heads=2, kv_heads=1, dim=32, size=20, keep=30), dense())],
+    # one bucket and one expert only, no feed-forward at the end
+    "narrow": config([(attention(heads=8, kv_heads=8, dim=8, vdim=8, rot_dims=8, size=33, keep=0), moe(experts=1, identity=1, top=2)), (attention(heads=2, kv_heads=1, dim=32, size=20, keep=30), None)],
                      scale=0.7, eps=1e-6, bigram=(1, 3, 4)),
 }
 
